@@ -1,6 +1,6 @@
 // Paged decode attention (flash-decoding) for sm_100a: one new query token per row against that row's cached keys.
 //
-// grid = (row, kv head, key split). A CTA handles the G = Hq / Hkv query heads that share its KV head, so every cached
+// grid = (row, kv head x share, key split). A CTA handles the G = Hq / Hkv query heads that share its KV head, so every cached
 // key and value is read from HBM exactly once per row. Each of its 4 warps walks 32-key blocks of the split:
 //   scores : lane = key      - each lane reads one key row (16-byte loads) and dots it with the G queries in smem
 //   values : lane = d-slice  - the block's probabilities are broadcast by shuffle; value rows are read coalesced
@@ -55,12 +55,13 @@ __global__ void __launch_bounds__(WARPS * 32)
 paged_decode_kernel(const __nv_bfloat16* __restrict__ q, const void* __restrict__ kpool, const void* __restrict__ vpool,
                     const float* __restrict__ kscale, const float* __restrict__ vscale,
                     const int* __restrict__ page_table, const int* __restrict__ lengths, float* __restrict__ part_m,
-                    float* __restrict__ part_l, float* __restrict__ part_acc, int Hq, int Hkv, int page_size,
+                    float* __restrict__ part_l, float* __restrict__ part_acc, int Hq, int Hkv, int share, int page_size,
                     int max_pages, int splits, float scale_log2, int window) {
   constexpr int DV = D / 32;                 // value elements per lane
   const int row = blockIdx.x, hk = blockIdx.y, split = blockIdx.z;
+  const int kvh = hk / share;                  // `share` groups of query heads read the same KV head
   constexpr int GM = GT ? GT : MAX_G;          // compile-time bound of every per-head array and loop
-  const int G = GT ? GT : Hq / Hkv;
+  const int G = GT ? GT : Hq / (Hkv * share);
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   __shared__ __align__(16) float sq[GM][D];
   __shared__ float sm_m[WARPS][GM], sm_l[WARPS][GM];
@@ -97,7 +98,7 @@ paged_decode_kernel(const __nv_bfloat16* __restrict__ q, const void* __restrict_
     if (live) {
       const int page = table[key / page_size];
       tok = static_cast<long long>(page) * page_size + (key % page_size);
-      const long long base = (tok * Hkv + hk) * D;
+      const long long base = (tok * Hkv + kvh) * D;
       float dot[GM];
 #pragma unroll
       for (int g = 0; g < GM; ++g) dot[g] = 0.f;
@@ -120,7 +121,7 @@ paged_decode_kernel(const __nv_bfloat16* __restrict__ q, const void* __restrict_
             }
         }
       }
-      const float ks = KIND == KV_BF16 ? 1.f : kscale[tok * Hkv + hk];
+      const float ks = KIND == KV_BF16 ? 1.f : kscale[tok * Hkv + kvh];
 #pragma unroll
       for (int g = 0; g < GM; ++g) if (GT != 0 || g < G) s[g] = dot[g] * ks;
     }
@@ -160,7 +161,7 @@ paged_decode_kernel(const __nv_bfloat16* __restrict__ q, const void* __restrict_
       for (int jj = 0; jj < 8; ++jj) tj[jj] = stok[warp][min(j0 + jj, nkeys - 1)];
 #pragma unroll
       for (int jj = 0; jj < 8; ++jj) {
-        const long long vb = (tj[jj] * Hkv + hk) * D + lane * DV;
+        const long long vb = (tj[jj] * Hkv + kvh) * D + lane * DV;
         if (KIND == KV_BF16) {
           const __nv_bfloat16* vp = reinterpret_cast<const __nv_bfloat16*>(vpool) + vb;
           if (DV == 4) {
@@ -184,7 +185,7 @@ paged_decode_kernel(const __nv_bfloat16* __restrict__ q, const void* __restrict_
       for (int jj = 0; jj < 8; ++jj) {
         const int j = min(j0 + jj, 31);
         const bool on = j0 + jj < nkeys;
-        const float vs = KIND == KV_BF16 ? 1.f : vscale[tj[jj] * Hkv + hk];
+        const float vs = KIND == KV_BF16 ? 1.f : vscale[tj[jj] * Hkv + kvh];
         float pk[GM];
         if (GM % 4 == 0) {
 #pragma unroll
@@ -309,17 +310,19 @@ using namespace dewb::decode;
 extern "C" int dewb_paged_decode(const void* q, const void* kpool, const void* vpool, const float* kscale,
                                  const float* vscale, const int* page_table, const int* lengths, const float* sinks,
                                  void* out, float* lse, float* part_m, float* part_l, float* part_acc, int rows, int Hq,
-                                 int Hkv, int D, int page_size, int max_pages, int splits, float scale, int window,
+                                 int Hkv, int share, int D, int page_size, int max_pages, int splits, float scale, int window,
                                  int kv_kind, void* stream_ptr) {
   if (rows <= 0) return 0;
-  if ((D != 64 && D != 128 && D != 256) || Hq % Hkv != 0 || Hq / Hkv > MAX_G || splits < 1) return -3;
+  if ((D != 64 && D != 128 && D != 256) || share < 1 || Hkv < 1 || Hq % (Hkv * share) != 0 ||
+      Hq / (Hkv * share) > MAX_G || splits < 1)
+    return -3;
   cudaStream_t stream = reinterpret_cast<cudaStream_t>(stream_ptr);
   const float scale_log2 = scale * 1.4426950408889634f;
-  dim3 grid(rows, Hkv, splits);
+  dim3 grid(rows, Hkv * share, splits);
   const __nv_bfloat16* qp = reinterpret_cast<const __nv_bfloat16*>(q);
-  const int Gq = Hq / Hkv;
+  const int Gq = Hq / (Hkv * share);
 #define DEWB_DECODE_G(DD, KK, GG) paged_decode_kernel<DD, KK, GG><<<grid, WARPS * 32, 0, stream>>>( \
-    qp, kpool, vpool, kscale, vscale, page_table, lengths, part_m, part_l, part_acc, Hq, Hkv, page_size, max_pages, splits, scale_log2, window)
+    qp, kpool, vpool, kscale, vscale, page_table, lengths, part_m, part_l, part_acc, Hq, Hkv, share, page_size, max_pages, splits, scale_log2, window)
 #define DEWB_DECODE(DD, KK) do { if (Gq == 4) DEWB_DECODE_G(DD, KK, 4); else if (Gq == 8) DEWB_DECODE_G(DD, KK, 8); \
     else if (Gq == 1) DEWB_DECODE_G(DD, KK, 1); else if (Gq == 2) DEWB_DECODE_G(DD, KK, 2); else DEWB_DECODE_G(DD, KK, 0); } while (0)
 #define DEWB_DECODE_D(KK) do { if (D == 64) DEWB_DECODE(64, KK); else if (D == 128) DEWB_DECODE(128, KK); else DEWB_DECODE(256, KK); } while (0)

@@ -1,0 +1,311 @@
+// Attention against a paged cache for any head widths, and the projection epilogue in front of it, for sm_100a.
+//
+//   qk_norm_append   from the packed projection [tokens, H dk + G dk + G dv]: RMS norm of q over all its heads at once and of k likewise
+//                    (weights may be null: no norm), the query temperature 1 + coef ln(floor((p + 1) / every) + 1), the copy into heads
+//                    of the cache's (padded) width, and the append of keys and values to the page pools
+//   paged_attend     causal attention of a call's tokens against everything the cache holds of their rows (any start positions; a decode
+//                    step is the case of one token per row); scores, softmax and sums in fp32 on the CUDA cores.  It is the fp32 form,
+//                    and takes the head widths the tensor-core kernels do not.
+//
+// A query's row of work is (token, head of its group), so a group's heads share the key and value tiles.  Positions below 0 are padding:
+// nothing is appended for them and their outputs are zero.  Compiled without fast math.
+#include <cstdint>
+#include <cuda_bf16.h>
+#include <cuda_runtime.h>
+
+namespace dewb {
+namespace paged {
+
+using bf16 = __nv_bfloat16;
+
+__device__ __forceinline__ float ld(const float* p) { return *p; }
+__device__ __forceinline__ float ld(const bf16* p) { return __bfloat162float(*p); }
+__device__ __forceinline__ void st(float* p, float v) { *p = v; }
+__device__ __forceinline__ void st(bf16* p, float v) { *p = __float2bfloat16(v); }
+
+template <int V>
+__device__ __forceinline__ void load_v(const float* p, float (&f)[V]) {
+  if constexpr (V == 4) {
+    const float4 v = *reinterpret_cast<const float4*>(p);
+    f[0] = v.x; f[1] = v.y; f[2] = v.z; f[3] = v.w;
+  } else {
+    f[0] = *p;
+  }
+}
+template <int V>
+__device__ __forceinline__ void load_v(const bf16* p, float (&f)[V]) {
+  if constexpr (V == 4) {
+    const uint2 v = *reinterpret_cast<const uint2*>(p);
+    f[0] = __uint_as_float(v.x << 16); f[1] = __uint_as_float(v.x & 0xffff0000u);
+    f[2] = __uint_as_float(v.y << 16); f[3] = __uint_as_float(v.y & 0xffff0000u);
+  } else {
+    f[0] = __bfloat162float(*p);
+  }
+}
+template <int V>
+__device__ __forceinline__ void store_v(float* p, const float (&f)[V]) {
+  if constexpr (V == 4) *reinterpret_cast<float4*>(p) = make_float4(f[0], f[1], f[2], f[3]);
+  else *p = f[0];
+}
+template <int V>
+__device__ __forceinline__ void store_v(bf16* p, const float (&f)[V]) {
+  if constexpr (V == 4) {
+    __nv_bfloat162 a = __floats2bfloat162_rn(f[0], f[1]), b = __floats2bfloat162_rn(f[2], f[3]);
+    *reinterpret_cast<uint2*>(p) = make_uint2(*reinterpret_cast<uint32_t*>(&a), *reinterpret_cast<uint32_t*>(&b));
+  } else {
+    *p = __float2bfloat16(f[0]);
+  }
+}
+
+__device__ __forceinline__ float block_sum(float v, float* red) {
+#pragma unroll
+  for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nw = blockDim.x >> 5;
+  __syncthreads();
+  if (lane == 0) red[warp] = v;
+  __syncthreads();
+  float t = lane < nw ? red[lane] : 0.f;
+#pragma unroll
+  for (int o = 16; o > 0; o >>= 1) t += __shfl_xor_sync(0xffffffffu, t, o);
+  return t;
+}
+
+struct Pool {
+  const int* table;       // [store rows, max_pages]
+  int page_size, max_pages;
+  const int* row_ids;     // store row of each call row, null: the same
+};
+
+__device__ __forceinline__ long long pool_token(const Pool& p, int row, int pos) {
+  const int r = p.row_ids == nullptr ? row : p.row_ids[row];
+  return static_cast<long long>(p.table[static_cast<long long>(r) * p.max_pages + pos / p.page_size]) * p.page_size + pos % p.page_size;
+}
+
+constexpr int PREP_THREADS = 256;
+
+// grid (tokens, 3): part 0 the queries, 1 the keys, 2 the values.  `packed` [tokens, H + 2 G, D] receives all three; D >= dk, dv.
+template <typename T, int V>
+__global__ void __launch_bounds__(PREP_THREADS)
+qk_norm_append_kernel(const T* __restrict__ qkv, const T* __restrict__ qw, const T* __restrict__ kw, float eps, float coef, int every,
+                      const int* __restrict__ positions, int S, int H, int G, int dk, int dv, int D, T* __restrict__ packed,
+                      T* __restrict__ kpool, T* __restrict__ vpool, Pool pool) {
+  __shared__ float red[32];
+  const long long t = blockIdx.x;
+  const int part = blockIdx.y;
+  const int heads = part == 0 ? H : G, width = part == 2 ? dv : dk, size = heads * width;
+  const T* src = qkv + t * (static_cast<long long>(H + G) * dk + G * dv) + (part == 0 ? 0 : part == 1 ? H * dk : (H + G) * dk);
+  const T* w = part == 0 ? qw : part == 1 ? kw : nullptr;
+  const int pos = positions[t];
+  float r = 1.f;
+  if (w != nullptr) {
+    float ss = 0.f;
+    for (int i = threadIdx.x * V; i < size; i += PREP_THREADS * V) {
+      float a[V];
+      load_v<V>(src + i, a);
+#pragma unroll
+      for (int j = 0; j < V; ++j) ss += a[j] * a[j];
+    }
+    r = 1.f / sqrtf(block_sum(ss, red) / size + eps);
+  }
+  float temp = 1.f;
+  if (part == 0 && every > 0 && pos >= 0) temp = 1.f + coef * logf(static_cast<float>((pos + 1) / every + 1));
+  T* dst = packed + t * static_cast<long long>(H + 2 * G) * D + static_cast<long long>(part == 0 ? 0 : part == 1 ? H : H + G) * D;
+  T* to_pool = nullptr;
+  if (part != 0 && pos >= 0) {
+    const long long tok = pool_token(pool, static_cast<int>(t / S), pos);
+    to_pool = (part == 1 ? kpool : vpool) + tok * G * D;
+  }
+  const int padded = heads * D;                    // the padding of each head is written as zeros
+  for (int i = threadIdx.x * V; i < padded; i += PREP_THREADS * V) {
+    const int h = i / D, c = i - h * D;
+    float a[V];
+#pragma unroll
+    for (int j = 0; j < V; ++j) a[j] = 0.f;
+    if (c < width) {
+      load_v<V>(src + h * width + c, a);
+      if (w != nullptr) {
+        float b[V];
+        load_v<V>(w + h * width + c, b);
+#pragma unroll
+        for (int j = 0; j < V; ++j) a[j] = a[j] * r * b[j];
+      }
+#pragma unroll
+      for (int j = 0; j < V; ++j) a[j] *= temp;
+    }
+    store_v<V>(dst + i, a);
+    if (to_pool != nullptr) store_v<V>(to_pool + i, a);
+  }
+}
+
+constexpr int BQ = 32, BK = 32, THREADS = 256;
+
+// grid (query tiles, G, rows).  q [R, S, *, D] with a token stride; out [R, S, H, dv] contiguous.  NJ: value columns per thread / 4.
+template <typename T, int NJ>
+__global__ void __launch_bounds__(THREADS)
+paged_attend_kernel(const T* __restrict__ q, long long q_token_stride, const T* __restrict__ kpool, const T* __restrict__ vpool,
+                    const int* __restrict__ positions, int S, int H, int G, int dk, int dv, int D, float scale, T* __restrict__ out, Pool pool) {
+  extern __shared__ __align__(16) float smem[];
+  const int kst = ((dk + 3) & ~3) + 4, vst = NJ * 32 + 4;
+  float* sq = smem;                     // [BQ][kst]
+  float* sk = sq + BQ * kst;            // [BK][kst]
+  float* sv = sk + BK * kst;            // [BK][vst]
+  float* sp = sv + BK * vst;            // [BQ][BK + 1]
+  __shared__ int s_pos[BQ];
+  __shared__ long long s_tok[BK];
+  const int row = blockIdx.z, g = blockIdx.y, Gq = H / G;
+  const int r0 = blockIdx.x * BQ, rows = S * Gq;
+  const int tid = threadIdx.x;
+  if (tid < BQ) {
+    const int r = r0 + tid;
+    s_pos[tid] = r < rows ? positions[static_cast<long long>(row) * S + r / Gq] : -1;
+  }
+  __syncthreads();
+  int last = -1;
+  for (int i = 0; i < BQ; ++i) last = max(last, s_pos[i]);
+  for (int i = tid; i < BQ * kst; i += THREADS) {
+    const int r = i / kst, c = i - r * kst;
+    float v = 0.f;
+    if (c < dk && s_pos[r] >= 0) {
+      const int gr = r0 + r;
+      v = ld(q + (static_cast<long long>(row) * S + gr / Gq) * q_token_stride + static_cast<long long>(g * Gq + gr % Gq) * D + c) * scale;
+    }
+    sq[i] = v;
+  }
+  const int qr = tid >> 3, ql = tid & 7;
+  const int my_pos = s_pos[qr];
+  float m = -INFINITY, l = 0.f, acc[NJ][4];
+#pragma unroll
+  for (int j = 0; j < NJ; ++j) { acc[j][0] = acc[j][1] = acc[j][2] = acc[j][3] = 0.f; }
+  for (int k0 = 0; k0 <= last; k0 += BK) {
+    __syncthreads();
+    if (tid < BK) s_tok[tid] = k0 + tid <= last ? pool_token(pool, row, k0 + tid) : -1;
+    __syncthreads();
+    for (int i = tid; i < BK * kst; i += THREADS) {
+      const int r = i / kst, c = i - r * kst;
+      sk[i] = (c < dk && s_tok[r] >= 0) ? ld(kpool + (s_tok[r] * G + g) * D + c) : 0.f;
+    }
+    for (int i = tid; i < BK * vst; i += THREADS) {
+      const int r = i / vst, c = i - r * vst;
+      sv[i] = (c < dv && s_tok[r] >= 0) ? ld(vpool + (s_tok[r] * G + g) * D + c) : 0.f;
+    }
+    __syncthreads();
+    float s[4] = {0.f, 0.f, 0.f, 0.f};
+    for (int c = 0; c < kst - 4; c += 4) {
+      const float4 a = *reinterpret_cast<const float4*>(sq + qr * kst + c);
+#pragma unroll
+      for (int j = 0; j < 4; ++j) {
+        const float4 b = *reinterpret_cast<const float4*>(sk + (ql + 8 * j) * kst + c);
+        s[j] += a.x * b.x + a.y * b.y + a.z * b.z + a.w * b.w;
+      }
+    }
+    float bm = -INFINITY;
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+      if (k0 + ql + 8 * j > my_pos) s[j] = -INFINITY;
+      bm = fmaxf(bm, s[j]);
+    }
+#pragma unroll
+    for (int o = 4; o > 0; o >>= 1) bm = fmaxf(bm, __shfl_xor_sync(0xffffffffu, bm, o));
+    const float mn = fmaxf(m, bm);
+    const float alpha = m == -INFINITY ? 0.f : expf(m - mn);
+    float ps = 0.f;
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+      const float p = s[j] == -INFINITY ? 0.f : expf(s[j] - mn);
+      ps += p;
+      sp[qr * (BK + 1) + ql + 8 * j] = p;
+    }
+#pragma unroll
+    for (int o = 4; o > 0; o >>= 1) ps += __shfl_xor_sync(0xffffffffu, ps, o);
+    l = l * alpha + ps;
+    m = mn;
+    __syncwarp();
+#pragma unroll
+    for (int j = 0; j < NJ; ++j) { acc[j][0] *= alpha; acc[j][1] *= alpha; acc[j][2] *= alpha; acc[j][3] *= alpha; }
+    for (int k = 0; k < BK; ++k) {
+      const float p = sp[qr * (BK + 1) + k];
+#pragma unroll
+      for (int j = 0; j < NJ; ++j) {
+        const float4 v = *reinterpret_cast<const float4*>(sv + k * vst + ql * 4 + 32 * j);
+        acc[j][0] += p * v.x; acc[j][1] += p * v.y; acc[j][2] += p * v.z; acc[j][3] += p * v.w;
+      }
+    }
+  }
+  const int gr = r0 + qr;
+  if (gr >= rows) return;
+  const float inv = l > 0.f ? 1.f / l : 0.f;
+  T* o = out + ((static_cast<long long>(row) * S + gr / Gq) * H + g * Gq + gr % Gq) * dv;
+#pragma unroll
+  for (int j = 0; j < NJ; ++j)
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      const int c = ql * 4 + 32 * j + e;
+      if (c < dv) st(o + c, acc[j][e] * inv);
+    }
+}
+
+inline bool aligned(const void* p, size_t a) { return (reinterpret_cast<uintptr_t>(p) & (a - 1)) == 0; }
+
+template <typename T, int NJ>
+int attend(const T* q, long long qs, const T* kpool, const T* vpool, const int* positions, int R, int S, int H, int G, int dk, int dv, int D,
+           float scale, T* out, const Pool& pool, cudaStream_t stream) {
+  const int kst = ((dk + 3) & ~3) + 4, vst = NJ * 32 + 4;
+  const size_t smem = static_cast<size_t>(BQ * kst + BK * kst + BK * vst + BQ * (BK + 1)) * 4;
+  if (smem > 225 * 1024) return -3;
+  cudaError_t e = cudaFuncSetAttribute(paged_attend_kernel<T, NJ>, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem));
+  if (e != cudaSuccess) return static_cast<int>(e);
+  const long long tiles = (static_cast<long long>(S) * (H / G) + BQ - 1) / BQ;
+  paged_attend_kernel<T, NJ><<<dim3(static_cast<unsigned>(tiles), G, R), THREADS, smem, stream>>>(q, qs, kpool, vpool, positions, S, H, G, dk, dv, D, scale, out, pool);
+  return static_cast<int>(cudaGetLastError());
+}
+
+template <typename T>
+int attend_any(const void* q, long long qs, const void* kpool, const void* vpool, const int* positions, int R, int S, int H, int G, int dk, int dv,
+               int D, float scale, void* out, const Pool& pool, cudaStream_t stream) {
+#define DEWB_ATTEND(NN) attend<T, NN>(static_cast<const T*>(q), qs, static_cast<const T*>(kpool), static_cast<const T*>(vpool), positions, R, S, H, G, \
+                                      dk, dv, D, scale, static_cast<T*>(out), pool, stream)
+  const int nj = (dv + 31) / 32;
+  if (nj <= 1) return DEWB_ATTEND(1);
+  if (nj <= 2) return DEWB_ATTEND(2);
+  if (nj <= 4) return DEWB_ATTEND(4);
+  if (nj <= 8) return DEWB_ATTEND(8);
+  if (nj <= 16) return DEWB_ATTEND(16);
+#undef DEWB_ATTEND
+  return -3;
+}
+
+}  // namespace paged
+}  // namespace dewb
+
+using namespace dewb::paged;
+
+// qkv [R * S, H dk + G dk + G dv] -> packed [R * S, H + 2 G, D] and the pools [*, page_size, G, D].  `every` 0: no temperature.
+extern "C" int dewb_qk_norm_append(const void* qkv, const void* qw, const void* kw, float eps, float coef, int every, const int* positions, int R,
+                                   int S, int H, int G, int dk, int dv, int D, void* packed, void* kpool, void* vpool, const int* page_table,
+                                   int page_size, int max_pages, const int* row_ids, int fp32, void* stream_ptr) {
+  if (R <= 0 || S <= 0) return 0;
+  if (H < 1 || G < 1 || H % G || dk < 1 || dv < 1 || D < dk || D < dv || page_size < 1 || max_pages < 1 || every < 0) return -3;
+  cudaStream_t stream = reinterpret_cast<cudaStream_t>(stream_ptr);
+  const Pool pool{page_table, page_size, max_pages, row_ids};
+  const bool vec = dk % 4 == 0 && dv % 4 == 0 && D % 4 == 0 && aligned(qkv, 16) && aligned(qw, 16) && aligned(kw, 16) && aligned(packed, 16) &&
+                   aligned(kpool, 16) && aligned(vpool, 16);
+  const dim3 grid(static_cast<unsigned>(R) * static_cast<unsigned>(S), 3);
+#define DEWB_PREP(TT, VV) qk_norm_append_kernel<TT, VV><<<grid, PREP_THREADS, 0, stream>>>(static_cast<const TT*>(qkv), static_cast<const TT*>(qw), \
+    static_cast<const TT*>(kw), eps, coef, every, positions, S, H, G, dk, dv, D, static_cast<TT*>(packed), static_cast<TT*>(kpool), \
+    static_cast<TT*>(vpool), pool)
+  if (fp32) { if (vec) DEWB_PREP(float, 4); else DEWB_PREP(float, 1); }
+  else { if (vec) DEWB_PREP(bf16, 4); else DEWB_PREP(bf16, 1); }
+#undef DEWB_PREP
+  return static_cast<int>(cudaGetLastError());
+}
+
+extern "C" int dewb_paged_attend(const void* q, long long q_token_stride, const void* kpool, const void* vpool, const int* positions, int R, int S,
+                                 int H, int G, int dk, int dv, int D, float scale, void* out, const int* page_table, int page_size, int max_pages,
+                                 const int* row_ids, int fp32, void* stream_ptr) {
+  if (R <= 0 || S <= 0) return 0;
+  if (H < 1 || G < 1 || H % G || dk < 1 || dv < 1 || D < dk || D < dv || page_size < 1 || max_pages < 1) return -3;
+  cudaStream_t stream = reinterpret_cast<cudaStream_t>(stream_ptr);
+  const Pool pool{page_table, page_size, max_pages, row_ids};
+  if (fp32) return attend_any<float>(q, q_token_stride, kpool, vpool, positions, R, S, H, G, dk, dv, D, scale, out, pool, stream);
+  return attend_any<bf16>(q, q_token_stride, kpool, vpool, positions, R, S, H, G, dk, dv, D, scale, out, pool, stream);
+}

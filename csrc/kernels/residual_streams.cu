@@ -1,0 +1,315 @@
+// Row kernels of decoders whose residual is a bundle of fp32 streams, for sm_100a.  All are bandwidth bound: one pass over the operands,
+// 16-byte accesses, fp32 arithmetic.
+//
+//   embed_streams   H[t, s, :] = embed[token t] (+ pos[position t]) for every stream s
+//   stream_step     one residual step between two sub-layers: the pending write of the sub-layer that just ran
+//                       H'[t] = sum_s mix[s, t] H[s] + out[t] * (scale . y)
+//                   (in place), the read of the next one, u = sum_s read[s] H'[s], and its norm (layer norm without a bias, or RMS norm)
+//   clamped_glu     g sigmoid(alpha g) (u + 1) with g = min(gate, limit), u = clamp(up, -limit, limit)
+//   sigmoid_gated_norm   RMS norm over a whole row times a weight times sigmoid(gate)
+//
+// Activations are bf16 or fp32 (template T); the streams, the connection weights and every sum are fp32.  Compiled without fast math.
+#include <cstdint>
+#include <cuda_bf16.h>
+#include <cuda_runtime.h>
+
+namespace dewb {
+namespace streams {
+
+using bf16 = __nv_bfloat16;
+constexpr int MAX_STREAMS = 16;
+constexpr int THREADS = 256;
+
+// V consecutive values (V = 4 or 1) as fp32
+template <int V>
+__device__ __forceinline__ void load_v(const float* p, float (&f)[V]) {
+  if constexpr (V == 4) {
+    const float4 v = *reinterpret_cast<const float4*>(p);
+    f[0] = v.x; f[1] = v.y; f[2] = v.z; f[3] = v.w;
+  } else {
+    f[0] = *p;
+  }
+}
+template <int V>
+__device__ __forceinline__ void load_v(const bf16* p, float (&f)[V]) {
+  if constexpr (V == 4) {
+    const uint2 v = *reinterpret_cast<const uint2*>(p);
+    f[0] = __uint_as_float(v.x << 16); f[1] = __uint_as_float(v.x & 0xffff0000u);
+    f[2] = __uint_as_float(v.y << 16); f[3] = __uint_as_float(v.y & 0xffff0000u);
+  } else {
+    f[0] = __bfloat162float(*p);
+  }
+}
+template <int V>
+__device__ __forceinline__ void store_v(float* p, const float (&f)[V]) {
+  if constexpr (V == 4) *reinterpret_cast<float4*>(p) = make_float4(f[0], f[1], f[2], f[3]);
+  else *p = f[0];
+}
+template <int V>
+__device__ __forceinline__ void store_v(bf16* p, const float (&f)[V]) {
+  if constexpr (V == 4) {
+    __nv_bfloat162 a = __floats2bfloat162_rn(f[0], f[1]), b = __floats2bfloat162_rn(f[2], f[3]);
+    *reinterpret_cast<uint2*>(p) = make_uint2(*reinterpret_cast<uint32_t*>(&a), *reinterpret_cast<uint32_t*>(&b));
+  } else {
+    *p = __float2bfloat16(f[0]);
+  }
+}
+
+__device__ __forceinline__ float block_sum(float v, float* red) {
+#pragma unroll
+  for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nw = blockDim.x >> 5;
+  __syncthreads();
+  if (lane == 0) red[warp] = v;
+  __syncthreads();
+  float t = lane < nw ? red[lane] : 0.f;
+#pragma unroll
+  for (int o = 16; o > 0; o >>= 1) t += __shfl_xor_sync(0xffffffffu, t, o);
+  return t;
+}
+
+template <typename T, int V>
+__global__ void __launch_bounds__(THREADS)
+embed_streams_kernel(const long long* __restrict__ tokens, const int* __restrict__ positions, const T* __restrict__ embed,
+                     const T* __restrict__ pos, float* __restrict__ H, int n, int d, int vocab, int max_pos) {
+  const long long t = blockIdx.x;
+  const long long tok = min(max(tokens[t], 0ll), static_cast<long long>(vocab - 1));
+  const int p = min(max(positions == nullptr ? 0 : positions[t], 0), max_pos - 1);
+  for (int i = threadIdx.x * V; i < d; i += THREADS * V) {
+    float a[V];
+    load_v<V>(embed + tok * d + i, a);
+    if (pos != nullptr) {
+      float b[V];
+      load_v<V>(pos + static_cast<long long>(p) * d + i, b);
+#pragma unroll
+      for (int j = 0; j < V; ++j) a[j] += b[j];
+    }
+    for (int s = 0; s < n; ++s) store_v<V>(H + (t * n + s) * d + i, a);
+  }
+}
+
+// NS: the number of streams when it is small and known (registers sized for it), 0: any number up to MAX_STREAMS.
+template <typename T, int V, int NS>
+__global__ void __launch_bounds__(THREADS)
+stream_step_kernel(float* __restrict__ H, const T* __restrict__ y, const T* __restrict__ scale, const float* __restrict__ mix,
+                   const float* __restrict__ out, const float* __restrict__ read, const T* __restrict__ w, T* __restrict__ normed,
+                   int n_rt, int d, float eps, int rms) {
+  constexpr int NM = NS ? NS : MAX_STREAMS;
+  const int n = NS ? NS : n_rt;
+  extern __shared__ float su[];                      // u of this token
+  __shared__ float s_mix[MAX_STREAMS * MAX_STREAMS], s_out[MAX_STREAMS], s_read[MAX_STREAMS], red[32];
+  const long long t = blockIdx.x;
+  if (y != nullptr) {
+    for (int i = threadIdx.x; i < n * n; i += THREADS) s_mix[i] = mix[i];
+    for (int i = threadIdx.x; i < n; i += THREADS) s_out[i] = out[i];
+  }
+  for (int i = threadIdx.x; i < n; i += THREADS) s_read[i] = read[i];
+  __syncthreads();
+  float* Ht = H + t * n * d;
+  float sum = 0.f;
+  for (int i = threadIdx.x * V; i < d; i += THREADS * V) {
+    float x[NM][V], u[V];
+#pragma unroll
+    for (int s = 0; s < NM; ++s)
+      if (NS || s < n) load_v<V>(Ht + static_cast<long long>(s) * d + i, x[s]);
+#pragma unroll
+    for (int j = 0; j < V; ++j) u[j] = 0.f;
+    if (y != nullptr) {
+      float b[V];
+      load_v<V>(y + t * d + i, b);
+      if (scale != nullptr) {
+        float c[V];
+        load_v<V>(scale + i, c);
+#pragma unroll
+        for (int j = 0; j < V; ++j) b[j] *= c[j];
+      }
+#pragma unroll(NS ? NS : 1)
+      for (int q = 0; q < NM; ++q) {
+        if (NS || q < n) {
+          float a[V];
+#pragma unroll
+          for (int j = 0; j < V; ++j) a[j] = s_out[q] * b[j];
+#pragma unroll
+          for (int s = 0; s < NM; ++s)
+            if (NS || s < n) {
+              const float m = s_mix[s * n + q];
+#pragma unroll
+              for (int j = 0; j < V; ++j) a[j] += m * x[s][j];
+            }
+          store_v<V>(Ht + static_cast<long long>(q) * d + i, a);
+#pragma unroll
+          for (int j = 0; j < V; ++j) u[j] += s_read[q] * a[j];
+        }
+      }
+    } else {
+#pragma unroll
+      for (int s = 0; s < NM; ++s)
+        if (NS || s < n) {
+#pragma unroll
+          for (int j = 0; j < V; ++j) u[j] += s_read[s] * x[s][j];
+        }
+    }
+#pragma unroll
+    for (int j = 0; j < V; ++j) sum += rms ? u[j] * u[j] : u[j];
+    if (normed != nullptr) store_v<V>(su + i, u);
+  }
+  if (normed == nullptr) return;                     // a last write with nothing to read after it
+  sum = block_sum(sum, red);
+  float mean = 0.f, var = sum / d;
+  if (!rms) {
+    mean = sum / d;
+    float dev = 0.f;
+    for (int i = threadIdx.x * V; i < d; i += THREADS * V) {
+#pragma unroll
+      for (int j = 0; j < V; ++j) { const float e = su[i + j] - mean; dev += e * e; }
+    }
+    var = block_sum(dev, red) / d;
+  }
+  const float r = 1.f / sqrtf(var + eps);
+  for (int i = threadIdx.x * V; i < d; i += THREADS * V) {
+    float c[V], o[V];
+    load_v<V>(w + i, c);
+#pragma unroll
+    for (int j = 0; j < V; ++j) o[j] = (su[i + j] - mean) * r * c[j];
+    store_v<V>(normed + t * d + i, o);
+  }
+}
+
+template <typename T, int V>
+__global__ void __launch_bounds__(THREADS)
+clamped_glu_kernel(const T* __restrict__ gu, T* __restrict__ out, long long rows, int F, float limit, float alpha) {
+  const long long total = rows * (F / V);
+  for (long long k = blockIdx.x * static_cast<long long>(THREADS) + threadIdx.x; k < total; k += static_cast<long long>(gridDim.x) * THREADS) {
+    const long long r = k / (F / V);
+    const int i = static_cast<int>(k - r * (F / V)) * V;
+    float g[V], u[V], o[V];
+    load_v<V>(gu + r * 2 * F + i, g);
+    load_v<V>(gu + r * 2 * F + F + i, u);
+#pragma unroll
+    for (int j = 0; j < V; ++j) {
+      const float a = fminf(g[j], limit), b = fminf(fmaxf(u[j], -limit), limit);
+      const float e = sizeof(T) == 2 ? __expf(-alpha * a) : expf(-alpha * a);
+      o[j] = a / (1.f + e) * (b + 1.f);
+    }
+    store_v<V>(out + r * F + i, o);
+  }
+}
+
+template <typename T, int V>
+__global__ void __launch_bounds__(THREADS)
+sigmoid_gated_norm_kernel(const T* __restrict__ x, const T* __restrict__ gate, const T* __restrict__ w, T* __restrict__ out, int d, float eps) {
+  extern __shared__ float sx[];
+  __shared__ float red[32];
+  const long long t = blockIdx.x;
+  float ss = 0.f;
+  for (int i = threadIdx.x * V; i < d; i += THREADS * V) {
+    float a[V];
+    load_v<V>(x + t * d + i, a);
+#pragma unroll
+    for (int j = 0; j < V; ++j) ss += a[j] * a[j];
+    store_v<V>(sx + i, a);
+  }
+  const float r = 1.f / sqrtf(block_sum(ss, red) / d + eps);
+  for (int i = threadIdx.x * V; i < d; i += THREADS * V) {
+    float g[V], c[V], o[V];
+    load_v<V>(gate + t * d + i, g);
+    load_v<V>(w + i, c);
+#pragma unroll
+    for (int j = 0; j < V; ++j) {
+      const float e = sizeof(T) == 2 ? __expf(-g[j]) : expf(-g[j]);
+      o[j] = sx[i + j] * r * c[j] / (1.f + e);
+    }
+    store_v<V>(out + t * d + i, o);
+  }
+}
+
+inline bool aligned(const void* p, size_t a) { return (reinterpret_cast<uintptr_t>(p) & (a - 1)) == 0; }
+
+template <typename K>
+int allow_smem(K kernel, size_t bytes) {
+  if (bytes <= 48 * 1024) return 0;
+  if (bytes > 220 * 1024) return -3;
+  return static_cast<int>(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(bytes)));
+}
+
+template <typename T>
+int step(float* H, const T* y, const T* scale, const float* mix, const float* out, const float* read, const T* w, T* normed, long long rows,
+         int n, int d, float eps, int rms, cudaStream_t stream) {
+  const bool vec = d % 4 == 0 && aligned(H, 16) && aligned(y, 4 * sizeof(T)) && aligned(scale, 4 * sizeof(T)) && aligned(w, 4 * sizeof(T)) &&
+                   aligned(normed, 4 * sizeof(T));
+  const size_t smem = static_cast<size_t>(d) * 4;
+#define DEWB_STEP(VV, NN) do { const int r = allow_smem(stream_step_kernel<T, VV, NN>, smem); if (r) return r; \
+    stream_step_kernel<T, VV, NN><<<static_cast<unsigned>(rows), THREADS, smem, stream>>>(H, y, scale, mix, out, read, w, normed, n, d, eps, rms); } while (0)
+  if (vec) {
+    if (n == 1) DEWB_STEP(4, 1); else if (n == 2) DEWB_STEP(4, 2); else if (n == 3) DEWB_STEP(4, 3); else if (n == 4) DEWB_STEP(4, 4); else DEWB_STEP(1, 0);
+  } else {
+    DEWB_STEP(1, 0);
+  }
+#undef DEWB_STEP
+  return static_cast<int>(cudaGetLastError());
+}
+
+}  // namespace streams
+}  // namespace dewb
+
+using namespace dewb::streams;
+
+// `fp32`: activations and weights are fp32, else bf16.  `positions` / `pos` may be null.
+extern "C" int dewb_embed_streams(const long long* tokens, const int* positions, const void* embed, const void* pos, float* H, long long rows,
+                                  int n, int d, int vocab, int max_pos, int fp32, void* stream_ptr) {
+  if (rows <= 0) return 0;
+  if (n < 1 || d < 1 || vocab < 1 || (pos != nullptr && (max_pos < 1 || positions == nullptr))) return -3;
+  cudaStream_t stream = reinterpret_cast<cudaStream_t>(stream_ptr);
+  const bool vec = d % 4 == 0 && aligned(H, 16) && aligned(embed, 16) && aligned(pos, 16);
+  const unsigned grid = static_cast<unsigned>(rows);
+#define DEWB_EMBED(TT, VV) embed_streams_kernel<TT, VV><<<grid, THREADS, 0, stream>>>(tokens, positions, static_cast<const TT*>(embed), \
+    static_cast<const TT*>(pos), H, n, d, vocab, max_pos > 0 ? max_pos : 1)
+  if (fp32) { if (vec) DEWB_EMBED(float, 4); else DEWB_EMBED(float, 1); }
+  else { if (vec) DEWB_EMBED(bf16, 4); else DEWB_EMBED(bf16, 1); }
+#undef DEWB_EMBED
+  return static_cast<int>(cudaGetLastError());
+}
+
+// H [rows, n, d] fp32, updated in place when `y` [rows, d] is given; normed [rows, d] (null: write only).  mix is indexed [from, to].
+extern "C" int dewb_stream_step(float* H, const void* y, const void* scale, const float* mix, const float* out, const float* read, const void* w,
+                                void* normed, long long rows, int n, int d, float eps, int rms, int fp32, void* stream_ptr) {
+  if (rows <= 0) return 0;
+  if (n < 1 || n > MAX_STREAMS || d < 1 || read == nullptr || (y != nullptr && (mix == nullptr || out == nullptr)) || (normed != nullptr && w == nullptr)) return -3;
+  cudaStream_t stream = reinterpret_cast<cudaStream_t>(stream_ptr);
+  if (fp32) return step<float>(H, static_cast<const float*>(y), static_cast<const float*>(scale), mix, out, read, static_cast<const float*>(w),
+                               static_cast<float*>(normed), rows, n, d, eps, rms, stream);
+  return step<bf16>(H, static_cast<const bf16*>(y), static_cast<const bf16*>(scale), mix, out, read, static_cast<const bf16*>(w),
+                    static_cast<bf16*>(normed), rows, n, d, eps, rms, stream);
+}
+
+// gu [rows, 2 F] (gate half, then linear half) -> out [rows, F]
+extern "C" int dewb_clamped_glu(const void* gu, void* out, long long rows, int F, float limit, float alpha, int fp32, void* stream_ptr) {
+  if (rows <= 0) return 0;
+  if (F < 1) return -3;
+  cudaStream_t stream = reinterpret_cast<cudaStream_t>(stream_ptr);
+  const bool vec = F % 4 == 0 && aligned(gu, 16) && aligned(out, 16);
+  const long long work = rows * (vec ? F / 4 : F), want = (work + THREADS - 1) / THREADS;
+  const unsigned grid = static_cast<unsigned>(want < 148 * 32 ? want : 148 * 32);
+#define DEWB_GLU(TT, VV) clamped_glu_kernel<TT, VV><<<grid, THREADS, 0, stream>>>(static_cast<const TT*>(gu), static_cast<TT*>(out), rows, F, limit, alpha)
+  if (fp32) { if (vec) DEWB_GLU(float, 4); else DEWB_GLU(float, 1); }
+  else { if (vec) DEWB_GLU(bf16, 4); else DEWB_GLU(bf16, 1); }
+#undef DEWB_GLU
+  return static_cast<int>(cudaGetLastError());
+}
+
+extern "C" int dewb_sigmoid_gated_norm(const void* x, const void* gate, const void* w, void* out, long long rows, int d, float eps, int fp32,
+                                       void* stream_ptr) {
+  if (rows <= 0) return 0;
+  if (d < 1) return -3;
+  cudaStream_t stream = reinterpret_cast<cudaStream_t>(stream_ptr);
+  const bool vec = d % 4 == 0 && aligned(x, 16) && aligned(gate, 16) && aligned(w, 16) && aligned(out, 16);
+  const size_t smem = static_cast<size_t>(d) * 4;
+  const unsigned grid = static_cast<unsigned>(rows);
+#define DEWB_GN(TT, VV) do { const int r = allow_smem(sigmoid_gated_norm_kernel<TT, VV>, smem); if (r) return r; \
+    sigmoid_gated_norm_kernel<TT, VV><<<grid, THREADS, smem, stream>>>(static_cast<const TT*>(x), static_cast<const TT*>(gate), \
+        static_cast<const TT*>(w), static_cast<TT*>(out), d, eps); } while (0)
+  if (fp32) { if (vec) DEWB_GN(float, 4); else DEWB_GN(float, 1); }
+  else { if (vec) DEWB_GN(bf16, 4); else DEWB_GN(bf16, 1); }
+#undef DEWB_GN
+  return static_cast<int>(cudaGetLastError());
+}

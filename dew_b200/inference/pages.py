@@ -151,6 +151,17 @@ class PageLedger:
             pages.append(p)
         return Seat(pages, reused)
 
+    def extend(self, pages: List[int], total_tokens: int) -> List[int]:
+        """Grow a row's ``pages`` in place to hold ``total_tokens``; returns the pages added."""
+        need = (total_tokens + self.page_size - 1) // self.page_size - len(pages)
+        if need > self.available():
+            raise OutOfPages(f"need {need} pages, {self.available()} available")
+        added = [self._take() for _ in range(max(0, need))]
+        for p in added:
+            self.refs[p] = 1
+        pages.extend(added)
+        return added
+
     def publish(self, prompt: Sequence[int], pages: Sequence[int]) -> None:
         """After a prompt's prefill: name its full pages so later requests can re-use them."""
         if not self.prefix_cache:

@@ -15,8 +15,8 @@ from typing import Any, Callable, Deque, Dict, List, Optional, Sequence
 
 import torch
 
-from ..nn.kv_cache import KVCache, KVStore
-from ..sampling.text import Sampling, transform_logits
+from ..nn.kv_cache import KVCache
+from ..sampling.text import Sampling, make_cache, transform_logits
 from ..utils import keys as K
 from .pages import HostTier, OutOfPages, PageLedger
 
@@ -68,11 +68,12 @@ class Server:
         pages_per_row = (capacity + spec.page_size - 1) // spec.page_size
         pool = spec.pages or slots * pages_per_row
         self.spec = KVCache(spec.quantized, spec.page_size, pool, spec.groups, spec.offloaded)
-        cfg = model.config
         p = next(model.parameters())
-        hd = cfg.head_dim or cfg.emb_features // cfg.num_heads
-        kvh = getattr(model, "local_kv_heads", None) or (cfg.num_kv_heads or cfg.num_heads)
-        self.store = KVStore(self.spec, cfg.num_layers, slots, capacity, kvh, hd, p.dtype, p.device)
+        self.store = make_cache(model, slots, capacity, self.spec)
+        if self.store.recurrent:
+            prefix_cache = False          # a recurrent state stands for a whole row: no page of another row brings it along
+        if self.store.slots is not None and host_pages > 0:
+            raise NotImplementedError("the host tier copies pages of caches whose layers all keep the same heads")
         self.host_tier = HostTier(self.store, host_pages) if host_pages > 0 and prefix_cache else None
         self.ledger = PageLedger(pool, self.spec.page_size, prefix_cache, self.host_tier)
         self.chunk = chunk or 512

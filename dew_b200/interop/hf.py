@@ -151,9 +151,10 @@ class Pretrained:
     def load(directory: os.PathLike, dtype=None, device="cpu", strict: bool = True):
         """A ``CausalTransformer`` for the families of ``interop.families``; a ``ClassicDecoder`` for the older lineage of
         ``interop.classic`` (GPT-2, GPT-NeoX, Falcon, Phi, OPT, BLOOM, StarCoder2, GPTBigCode); Mamba and Mamba-2 releases through
-        ``interop.recurrent``."""
+        ``interop.recurrent``; Ragenex through ``interop.ragenex``."""
         from .classic import CLASSIC, load_classic_state, read_classic_config
         from .families import family_of, load_state, read_config
+        from .ragenex import is_ragenex, load_ragenex_state, read_ragenex_config
         from .release import GenerationConfig, Release
         rel = Release(directory, dtype=dtype or torch.bfloat16)
         if str(rel.config.get("model_type") or "").lower() in CLASSIC:
@@ -163,6 +164,12 @@ class Pretrained:
             model.unread_keys = load_classic_state(model, rel, fam, strict=strict)
             model.generation_config = GenerationConfig.read(directory)
             model.family = fam.name
+            return model
+        if is_ragenex(rel.config):
+            model = CausalTransformer(read_ragenex_config(rel.config), dtype=dtype, device=device)
+            model.unread_keys = load_ragenex_state(model, rel, strict=strict)
+            model.generation_config = GenerationConfig.read(directory)
+            model.family = "ragenex"
             return model
         if str(rel.config.get("model_type") or "").lower() in ("mamba", "mamba2"):
             from .recurrent import load_recurrent_state, read_recurrent_config
@@ -184,6 +191,12 @@ class Pretrained:
         from .families import FAMILIES, export_state, write_config
         from .release import save_release
         dtype = str(next(model.parameters()).dtype).replace("torch.", "")
+        if family is None and getattr(model, "family", None) == "ragenex":
+            family = "ragenex"
+        if family == "ragenex":
+            from .ragenex import export_ragenex_state, write_ragenex_config
+            save_release(export_ragenex_state(model), write_ragenex_config(model.config), directory, max_shard_bytes, generation, fp8_blocks)
+            return
         if family is None:
             family = next((f.name for f in FAMILIES.values() if f.architecture == architecture), None)
         if family is None:           # an architecture string outside the table: Llama naming under that label

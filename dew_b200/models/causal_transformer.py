@@ -12,7 +12,7 @@ from __future__ import annotations
 
 import contextlib
 
-from dataclasses import dataclass, field
+from dataclasses import dataclass, field, replace
 from typing import Mapping, Any, Dict, List, Optional, Sequence, Tuple
 
 import torch
@@ -20,9 +20,11 @@ import torch.nn as nn
 import torch.utils.checkpoint as ckpt
 
 from .. import ops
+from ..ops import streams as ops_streams
 from ..nn.attention import SelfAttention
-from ..nn.layers import Embedding, Linear, RMSNorm
-from ..nn.mlp import SwiGLU
+from ..nn.kv_cache import CacheSlot
+from ..nn.layers import Embedding, LayerNorm, Linear, RMSNorm, declare
+from ..nn.mlp import ClampedGLU, SwiGLU
 from ..utils.registry import register
 
 
@@ -117,12 +119,48 @@ class TransformerConfig:
     embed_multiplier: Optional[float] = None          # Granite: embeddings times this (embed_scale is the sqrt(d) special case)
     residual_multiplier: float = 1.0                  # Granite: every sub-layer's output times this before it joins the stream
     logit_divisor: float = 1.0                        # Granite: logits divided by this
+    norm: str = "rms"                                 # layer: layer norms without a bias (built for the static-stream stack)
+    hyper_dynamic: bool = True                        # False: hyper-connections of the weights alone, over fp32 streams (any number, 1 included)
+    layer_scale: bool = False                         # every sub-layer's output times a learned vector before it is written to the streams
+    learned_positions: bool = False                   # a learned vector per position joins the embedding (max_seq_len of them)
+    query_temperature: Optional[Sequence[float]] = None    # (coef, every): queries times 1 + coef ln(floor((p + 1) / every) + 1)
+    value_dim: Optional[int] = None                   # width of a head's values where it differs from head_dim
+    mlp_limit: float = 7.0                            # mlp_activation 'clamped_glu': the clamp of both halves
+    layer_options: Optional[Sequence[Optional[Mapping]]] = None    # per layer, what differs from the fields above: num_heads, num_kv_heads, head_dim, value_dim,
+                                                      # query_scale, query_temperature, decay (lightning), mlp_features, mlp_limit
 
     def __post_init__(self):
+        if self.norm not in ("rms", "layer"):
+            raise ValueError(f"unknown norm {self.norm!r}; known: rms, layer")
+        if self.layer_options is not None and len(self.layer_options) != self.num_layers:
+            raise ValueError(f"layer_options describes {len(self.layer_options)} layers of {self.num_layers}")
+        if self.static_streams:
+            if self.altup > 1 or self.mixture is not None or self.sandwich_norm or not self.pre_norm or self.residual_multiplier != 1.0 or self.remat \
+                    or self.depth_residual_block or self.engram or self.mtp_depth:
+                raise NotImplementedError("static hyper-connections are built for pre-norm layers with dense MLPs, without rematerialisation, AltUp, block "
+                                          "attention residuals, n-gram memories and multi-token prediction")
+        elif self.norm != "rms" or self.layer_scale or self.learned_positions:
+            raise NotImplementedError("layer norms, layer scale and learned positions belong to the static-stream stack (hyper_connections >= 1, "
+                                      "hyper_dynamic=False)")
         if isinstance(self.mixture, Mapping):             # a run record (JSON) carries the mixture as a plain mapping
             self.mixture = Mixture(**self.mixture)
         if isinstance(self.loop, Mapping):
             self.loop = Loop(**self.loop)
+
+    @property
+    def static_streams(self) -> bool:
+        return self.hyper_connections >= 1 and not self.hyper_dynamic
+
+    def of_layer(self, index: int) -> "TransformerConfig":
+        """The configuration as layer ``index`` sees it."""
+        o = self.layer_options[index] if self.layer_options is not None else None
+        if not o:
+            return self
+        own = {"num_heads", "num_kv_heads", "head_dim", "value_dim", "query_scale", "query_temperature", "mlp_features", "mlp_limit"}
+        if set(o) - own - {"decay"}:
+            raise ValueError(f"unknown layer option(s) {sorted(set(o) - own - {'decay'})}; known: {sorted(own | {'decay'})}")
+        mixer = {k: o[k] for k in ("num_heads", "head_dim", "value_dim", "decay") if k in o} if self.kinds()[index] == "lightning" else {}
+        return replace(self, layer_options=None, mixer_options={**self.mixer_options, **mixer}, **{k: v for k, v in o.items() if k in own})
 
     def kinds(self) -> List[str]:
         if self.layer_types is None:
@@ -140,7 +178,7 @@ def _mixer(cfg: TransformerConfig, kind: str, dtype, device, index: int = 0) -> 
                           causal=cfg.causal, window=cfg.window if kind == "local" or cfg.layer_types is None else None, bias=cfg.attn_bias,
                           softcap=cfg.attn_softcap, sinks=cfg.attention_sinks, norm_eps=cfg.norm_eps,
                           init_std=cfg.init_std, qkv_bias=cfg.qkv_bias, scale=cfg.query_scale, qk_norm_full=cfg.qk_norm_full,
-                          out_gate=cfg.attn_out_gate, dtype=dtype, device=device)
+                          out_gate=cfg.attn_out_gate, value_dim=cfg.value_dim, temperature=cfg.query_temperature, dtype=dtype, device=device)
         a.rotary = kind != "nope"                        # SmolLM3's every fourth layer attends without positions
         if kind == "local" and cfg.local_rope_theta is not None:
             a.own_rope = (float(cfg.local_rope_theta), None)
@@ -188,6 +226,12 @@ def _mixer(cfg: TransformerConfig, kind: str, dtype, device, index: int = 0) -> 
                      "gla, delta, rwkv7")
 
 
+def _norm_of(cfg: TransformerConfig, dtype, device) -> nn.Module:
+    if cfg.norm == "layer":
+        return LayerNorm(cfg.emb_features, cfg.norm_eps, bias=False, dtype=dtype, device=device)
+    return RMSNorm(cfg.emb_features, cfg.norm_eps, dtype=dtype, device=device)
+
+
 class _NoNorm(nn.Module):
     """Stands where a pre-norm would: adds the pending branch into the stream and hands the stream on unnormalised."""
     weight = None
@@ -203,17 +247,18 @@ class DecoderLayer(nn.Module):
     def __init__(self, cfg: TransformerConfig, index: int, kind: str, dtype=None, device=None):
         super().__init__()
         self.kind, self.index = kind, index
+        cfg = cfg.of_layer(index) if index < cfg.num_layers else cfg
         if not cfg.pre_norm and not cfg.sandwich_norm:
             raise ValueError("a decoder without pre-norms normalises its sub-layers' outputs: set sandwich_norm=True with pre_norm=False")
         self.has_mlp = True if cfg.layer_mlp is None else bool(list(cfg.layer_mlp)[index % len(cfg.layer_mlp)])
         if kind == "none" and not self.has_mlp:
             raise ValueError(f"layer {index} has neither a mixer nor an MLP")
-        if (kind == "none" or not self.has_mlp) and (cfg.sandwich_norm or not cfg.pre_norm or cfg.hyper_connections > 1 or cfg.altup > 1):
+        if (kind == "none" or not self.has_mlp) and (cfg.sandwich_norm or not cfg.pre_norm or (cfg.hyper_connections > 1 and cfg.hyper_dynamic) or cfg.altup > 1):
             raise NotImplementedError("layers of one sub-layer are built for the plain pre-norm block")
-        self.input_norm = RMSNorm(cfg.emb_features, cfg.norm_eps, dtype=dtype, device=device) if cfg.pre_norm else _NoNorm()
+        self.input_norm = _norm_of(cfg, dtype, device) if cfg.pre_norm else _NoNorm()
         self.mixer = None if kind == "none" else _mixer(cfg, kind, dtype, device, index)
         one = kind == "none" or not self.has_mlp                  # one sub-layer: the input norm is its only norm
-        self.post_norm = None if one else (RMSNorm(cfg.emb_features, cfg.norm_eps, dtype=dtype, device=device) if cfg.pre_norm else _NoNorm())
+        self.post_norm = None if one else (_norm_of(cfg, dtype, device) if cfg.pre_norm else _NoNorm())
         mix = cfg.mixture
         sparse = self.has_mlp and mix is not None and (mix.layers is None or index in mix.layers)
         if not self.has_mlp:
@@ -225,6 +270,8 @@ class DecoderLayer(nn.Module):
             from ..nn.moe import SparseMLP
             self.mlp = SparseMLP(cfg.emb_features, mix, cfg.mlp_features or 4 * cfg.emb_features, init_std=cfg.init_std,
                                  dtype=dtype, device=device)
+        elif cfg.mlp_activation == "clamped_glu":
+            self.mlp = ClampedGLU(cfg.emb_features, cfg.mlp_features or 4 * cfg.emb_features, cfg.mlp_limit, init_std=cfg.init_std, dtype=dtype, device=device)
         else:
             self.mlp = SwiGLU(cfg.emb_features, cfg.mlp_features or 4 * cfg.emb_features, init_std=cfg.init_std,
                               activation=cfg.mlp_activation, dtype=dtype, device=device)
@@ -235,7 +282,16 @@ class DecoderLayer(nn.Module):
         self.cross = None       # set by the model for the layers of a loop with messages: one merge per sub-layer input
         self.residual_multiplier = float(cfg.residual_multiplier)
         self.streams = None
-        if cfg.hyper_connections > 1 or cfg.altup > 1:
+        self.layer_scale = None
+        if cfg.static_streams:
+            from ..nn.streams import HyperConnections
+            subs = int(self.mixer is not None) + int(self.mlp is not None)
+            self.streams = nn.ModuleList([HyperConnections(cfg.emb_features, cfg.hyper_connections, 2 * index + j, dynamic=False, device=device)
+                                          for j in range(subs)])
+            if cfg.layer_scale:
+                self.layer_scale = nn.ParameterList([declare(nn.Parameter(torch.ones(cfg.emb_features, dtype=dtype, device=device)), ("norm",), "scale")
+                                                     for _ in range(subs)])
+        elif cfg.hyper_connections > 1 or cfg.altup > 1:
             from ..nn.streams import AltUp, HyperConnections
             if cfg.hyper_connections > 1:
                 self.streams = nn.ModuleList([HyperConnections(cfg.emb_features, cfg.hyper_connections, 2 * index + j, dtype=dtype, device=device)
@@ -243,15 +299,32 @@ class DecoderLayer(nn.Module):
             else:
                 self.streams = nn.ModuleList([AltUp(cfg.altup, 2 * index + j, device=device) for j in range(2)])
 
+    def _mix(self, n, cos, sin, positions, segment_ids, cache, slot: Optional[int]):
+        """The mixer on its normalised input; ``slot`` is the cache entry of this run of the layer (None: the layer's own index)."""
+        slot = self.index if slot is None else slot
+        if self.kind in ROTARY_KINDS:
+            return self.mixer(n, cos, sin, positions, segment_ids, cache, slot)
+        if getattr(cache, "slots", None) is not None:
+            return self.mixer(n, segment_ids=segment_ids, cache=cache, layer=slot, positions=positions)
+        return self.mixer(n, segment_ids=segment_ids, cache=cache, layer=slot)
+
+    def forward_static(self, stack, cos, sin, positions, segment_ids, cache, slot: int) -> None:
+        """The layer over a ``StreamStack``: each sub-layer's write is fused with the next one's read and norm."""
+        scale = self.layer_scale if self.layer_scale is not None else [None] * len(self.streams)
+        q = 0
+        if self.mixer is not None:
+            n = stack.enter(self.streams[q], self.input_norm)
+            stack.leave(self.streams[q], self._mix(n, cos, sin, positions, segment_ids, cache, slot), scale[q])
+            q += 1
+        if self.mlp is not None:
+            n = stack.enter(self.streams[q], self.input_norm if q == 0 else self.post_norm)
+            stack.leave(self.streams[q], self.mlp(n), scale[q])
+
     def forward_streams(self, H, cos, sin, positions, segment_ids, cache):
         """The layer over several residual streams ``H [B,S,n,d]``: each sub-layer reads its input from the streams, and its
         output is written back by the learned connection (no fused add + norm on this path)."""
         x, ctx = self.streams[0].read(H)
-        n = self.input_norm(x)
-        if self.kind in ROTARY_KINDS:
-            a = self.mixer(n, cos, sin, positions, segment_ids, cache, self.index)
-        else:
-            a = self.mixer(n, segment_ids=segment_ids, cache=cache, layer=self.index)
+        a = self._mix(self.input_norm(x), cos, sin, positions, segment_ids, cache, None)
         H = self.streams[0].write(H, a, ctx)
         x, ctx = self.streams[1].read(H)
         return self.streams[1].write(H, self.mlp(self.post_norm(x)), ctx)
@@ -282,7 +355,7 @@ class DecoderLayer(nn.Module):
         h = h + a
         return h, self.mlp(self.post_norm(self.cross[1](h, bank)))
 
-    def forward(self, h, branch, cos, sin, positions, segment_ids, cache, bank=None):
+    def forward(self, h, branch, cos, sin, positions, segment_ids, cache, bank=None, slot: Optional[int] = None):
         """(stream, pending branch) -> (stream, pending branch); the branch is added by the next norm."""
         if bank is not None and self.cross is not None:
             return self._merged(h, branch, cos, sin, positions, segment_ids, bank)
@@ -295,10 +368,7 @@ class DecoderLayer(nn.Module):
             n, h = self._norm(self.input_norm, h, branch)
         if self.mixer is None:                                    # the MLP alone
             return h, self.mlp(n) if self.residual_multiplier == 1.0 else self.mlp(n) * self.residual_multiplier
-        if self.kind in ROTARY_KINDS:
-            a = self.mixer(n, cos, sin, positions, segment_ids, cache, self.index)
-        else:
-            a = self.mixer(n, segment_ids=segment_ids, cache=cache, layer=self.index)
+        a = self._mix(n, cos, sin, positions, segment_ids, cache, slot)
         if self.mlp is None:                                      # the mixer alone
             return h, a if self.residual_multiplier == 1.0 else a * self.residual_multiplier
         if self.mixer_out_norm is not None:
@@ -341,8 +411,9 @@ class CausalTransformer(nn.Module):
         self.vocab_size = cfg.vocab_size
         self.embed = Embedding(cfg.vocab_size, cfg.emb_features, cfg.init_std, dtype=dtype, device=device)
         kinds = cfg.kinds()
+        self.position_embed = Embedding(cfg.max_seq_len, cfg.emb_features, cfg.init_std, dtype=dtype, device=device) if cfg.learned_positions else None
         self.layers = nn.ModuleList([DecoderLayer(cfg, i, k, dtype, device) for i, k in enumerate(kinds)])
-        self.final_norm = RMSNorm(cfg.emb_features, cfg.norm_eps, dtype=dtype, device=device)
+        self.final_norm = _norm_of(cfg, dtype, device)
         self.head = None if cfg.tie_embeddings else Linear(cfg.emb_features, cfg.vocab_size, axes=("embed", "vocab"),
                                                            init_std=cfg.init_std, dtype=dtype, device=device)
         self.mtp = nn.ModuleList([MTPBlock(cfg, i, dtype, device) for i in range(cfg.mtp_depth)]) if cfg.mtp_depth > 0 else None
@@ -389,6 +460,33 @@ class CausalTransformer(nn.Module):
             outs.append(h)
         return outs
 
+    # ------------------------------------------------------------------ what runs, and what it keeps
+    def runs(self, steps: Optional[int] = None) -> List[Tuple[int, int]]:
+        """``(layer, cache slot)`` in the order the layers run: a looped block appears once per pass, each pass with slots of its own."""
+        n, loop = len(self.layers), self.config.loop
+        if loop is None:
+            return [(i, i) for i in range(n)]
+        end = n if loop.end is None else loop.end
+        order = list(range(loop.first)) + list(range(loop.first, end)) * (loop.steps if steps is None else steps) + list(range(end, n))
+        return [(i, slot) for slot, i in enumerate(order)]
+
+    def cache_slots(self) -> Optional[List[CacheSlot]]:
+        """One entry per layer run where the layers differ in what they keep (heads of their own widths, recurrent states); None where one
+        shape of keys and values serves them all."""
+        cfg, kinds = self.config, self.config.kinds()
+        if not (cfg.static_streams or cfg.layer_options is not None or cfg.query_temperature is not None or cfg.value_dim is not None):
+            return None
+        if any(k not in ("nope", "lightning", "none") for k in kinds):
+            raise NotImplementedError(f"per-layer caches are built for attention without rotation ('nope') and 'lightning' layers, not {sorted(set(kinds))}")
+        out = []
+        for i, _ in self.runs():
+            m = self.layers[i].mixer
+            if kinds[i] == "nope":
+                out.append(CacheSlot(m.num_kv_heads, m.head_dim, m.value_dim))
+            else:
+                out.append(CacheSlot(state=(0,) if m is None else (m.h, m.d, m.dv)))
+        return out
+
     # ------------------------------------------------------------------ helpers
     def head_weight(self) -> torch.Tensor:
         return self.embed.weight if self.head is None else self.head.weight
@@ -417,21 +515,24 @@ class CausalTransformer(nn.Module):
     def _looped(self, h, cos, sin, positions, segment_ids, cache, train, passes: bool, steps: Optional[int]):
         """The looped trunk: returns the final-normed exit state of the last pass, or of every pass with ``passes``."""
         cfg, loop = self.config, self.config.loop
-        if cache is not None:
-            raise NotImplementedError("a looped decoder keeps one cache per pass; decoding with a KV cache is not built for it")
         steps = loop.steps if steps is None else steps
+        if cache is not None and (loop.messages > 0 or passes or steps != loop.steps):
+            raise NotImplementedError("a looped decoder's cache holds its configured passes, each with keys and values of its own; cross-pass messages, "
+                                      "per-pass exits and another number of passes run on whole sequences without a cache")
         first, end = loop.first, len(self.layers) if loop.end is None else loop.end
         remat = cfg.remat and train and torch.is_grad_enabled()
 
-        def run(layers, h, branch):
-            for layer in layers:
-                if remat:
+        def run(layers, h, branch, slot=None):
+            for j, layer in enumerate(layers):
+                if cache is not None:
+                    h, branch = layer(h, branch, cos, sin, positions, segment_ids, cache, slot=slot + j)
+                elif remat:
                     h, branch = ckpt.checkpoint(layer, h, branch, cos, sin, positions, segment_ids, None, use_reentrant=False)
                 else:
                     h, branch = layer(h, branch, cos, sin, positions, segment_ids, None)
             return h, branch
 
-        h, branch = run(self.layers[:first], h, None)
+        h, branch = run(self.layers[:first], h, None, 0)
         exits = []
         if loop.messages > 0:
             if getattr(self, "tp", None) is not None:
@@ -463,9 +564,9 @@ class CausalTransformer(nn.Module):
                     h, branch = run(self.layers[first:end], h, branch)
                 h, branch = h.detach(), (None if branch is None else branch.detach())
             else:
-                h, branch = run(self.layers[first:end], h, branch)
+                h, branch = run(self.layers[first:end], h, branch, first + s * (end - first))
             if passes or s == steps - 1:
-                exits.append(self._finish(*run(self.layers[end:], h, branch)))
+                exits.append(self._finish(*run(self.layers[end:], h, branch, first + steps * (end - first))))
         return exits if passes else exits[-1]
 
     def exit_distribution(self, states: Sequence[torch.Tensor]) -> torch.Tensor:
@@ -482,11 +583,36 @@ class CausalTransformer(nn.Module):
         out.append(torch.ones_like(states[-1][..., 0], dtype=torch.float32) if stay is None else stay)
         return torch.stack(out)
 
+    def _static(self, tokens, positions, cache, steps: Optional[int] = None, observe=None):
+        """The stack over fp32 streams, up to the final norm; ``observe(run, total)`` sees the sum of the streams after every layer run."""
+        from ..nn.streams import StreamStack
+        cfg = self.config
+        if cfg.embed_scale or cfg.embed_multiplier is not None:
+            raise NotImplementedError("scaled embeddings are not built for the static-stream stack")
+        pos = None if self.position_embed is None else self.position_embed.weight
+        if pos is not None and cache is None and tokens.shape[1] > pos.shape[0]:
+            raise ValueError(f"{tokens.shape[1]} tokens do not fit the {pos.shape[0]} learned positions")
+        runs = self.runs(steps)
+        if cache is not None and steps is not None and steps != cfg.loop.steps:
+            raise NotImplementedError("the cache holds the configured number of passes")
+        H = ops_streams.embed_streams(tokens, positions, self.embed.weight, pos, cfg.hyper_connections)
+        stack = StreamStack(H, self.embed.weight.dtype)
+        cos, sin = (None, None) if all(k not in ROTARY_KINDS or k == "nope" for k in cfg.kinds()) else self.rope_tables(H.device)
+        for r, (i, slot) in enumerate(runs):
+            self.layers[i].forward_static(stack, cos, sin, positions, None, cache, slot)
+            if observe is not None:
+                observe(r, stack.total())
+        return stack
+
     def hidden(self, tokens, positions=None, segment_ids=None, cache=None, train: bool = False, passes: bool = False, loop_steps: Optional[int] = None,
                embeddings: Optional[torch.Tensor] = None):
         """``embeddings [B, S, d]``: input embeddings computed by the caller (a vision-language model splices image features into the
         token embeddings); they replace the table lookup of ``tokens`` and are scaled like it."""
         cfg = self.config
+        if cfg.static_streams:
+            if segment_ids is not None or embeddings is not None or passes:
+                raise NotImplementedError("static hyper-connections run on token rows without packed segments, given embeddings or per-pass exits")
+            return self._static(tokens, positions, cache, loop_steps).finish(self.final_norm)
         h = self.embed(tokens) if embeddings is None else embeddings
         if cfg.embed_scale:
             h = h * (cfg.emb_features ** 0.5)

@@ -10,6 +10,7 @@ import torch
 import torch.nn as nn
 
 from .. import ops
+from ..ops import paged as P
 from .layers import Linear, RMSNorm, declare
 
 
@@ -18,7 +19,7 @@ class SelfAttention(nn.Module):
                  qk_norm: bool = False, bias: bool = False, causal: bool = True, window: Optional[int] = None,
                  softcap: float = 0.0, sinks: bool = False, norm_eps: float = 1e-6, out_zero_init: bool = False,
                  init_std: Optional[float] = None, qkv_bias: bool = False, scale: Optional[float] = None, qk_norm_full: bool = False,
-                 out_gate: bool = False, dtype=None, device=None):
+                 out_gate: bool = False, value_dim: Optional[int] = None, temperature=None, dtype=None, device=None):
         super().__init__()
         self.features, self.num_heads = features, num_heads
         # a softmax scale other than head_dim ** -0.5 is folded into the queries (after the norm and the rotation)
@@ -26,9 +27,14 @@ class SelfAttention(nn.Module):
         self.num_kv_heads = num_kv_heads or num_heads
         self.head_dim = head_dim or features // num_heads
         self.causal, self.window, self.softcap = causal, window, softcap
-        qkv_out = (self.num_heads + 2 * self.num_kv_heads) * self.head_dim
+        self.value_dim = value_dim or self.head_dim
+        self.scale = float(scale) if scale is not None else self.head_dim ** -0.5
+        # queries grow with the position: (coef, every) multiplies them by 1 + coef ln(floor((p + 1) / every) + 1)
+        self.temperature = None if temperature is None else (float(temperature[0]), int(temperature[1]))
+        self.heads = P.Heads(self.num_heads, self.num_kv_heads, self.head_dim, self.value_dim)
+        qkv_out = self.heads.packed
         self.qkv_proj = Linear(features, qkv_out, bias=bias or qkv_bias, axes=("embed", "heads"), init_std=init_std, dtype=dtype, device=device)
-        self.o_proj = Linear(self.num_heads * self.head_dim, features, bias=bias, axes=("heads", "embed"),
+        self.o_proj = Linear(self.num_heads * self.value_dim, features, bias=bias, axes=("heads", "embed"),
                              init_std=init_std, zero_init=out_zero_init, dtype=dtype, device=device)
         # Qwen3-Next: the heads' outputs pass a sigmoid gate computed from the layer's input, before the output projection
         self.gate_proj = Linear(features, self.num_heads * self.head_dim, axes=("embed", "heads"), init_std=init_std, dtype=dtype, device=device) if out_gate else None
@@ -87,8 +93,27 @@ class SelfAttention(nn.Module):
             self._own = ops.rope_tables(cos.shape[0], self.head_dim, theta, cos.device, scaling)
         return self._own
 
+    def _general(self, x, positions, segment_ids, cache, layer):
+        """Heads of any widths, the query temperature, and caches whose layers differ; no rotation."""
+        B, S, _ = x.shape
+        if self.rotary or self.window is not None or self.softcap or self.sinks is not None or self.gate_proj is not None or segment_ids is not None \
+                or not self.causal or (self.q_norm is not None and not self.qk_norm_full):
+            raise NotImplementedError("a query temperature, values of another width and per-layer caches are built for causal attention without "
+                                      "rotation, window, soft cap, sinks, output gate or packed segments, with q / k norms over all heads or none")
+        qw, kw, eps = (None, None, 0.0) if self.q_norm is None else (self.q_norm.weight, self.k_norm.weight, self.q_norm.eps)
+        qkv = self.qkv_proj(x)
+        if cache is not None:
+            o = cache.attend_slot(layer, qkv, self.heads, positions, scale=self.scale, eps=eps, q_weight=qw, k_weight=kw, temperature=self.temperature)
+        else:
+            pos = torch.arange(S, device=x.device)[None].expand(B, S) if positions is None else positions
+            q, k, v = P.prepare_reference(qkv, self.heads, qw, kw, eps, self.temperature, pos)
+            o = ops.attention(q, k, v, causal=True, scale=self.scale)
+        return self.o_proj(o.reshape(B, S, self.num_heads * self.value_dim))
+
     def forward(self, x, cos=None, sin=None, positions=None, segment_ids=None, cache=None, layer: int = 0):
         B, S, _ = x.shape
+        if getattr(cache, "slots", None) is not None or self.temperature is not None or self.value_dim != self.head_dim:
+            return self._general(x, positions, segment_ids, cache, layer)
         cos, sin = self._tables(cos, sin)
         if (cache is None and x.is_cuda and cos is not None and self.head_transform is None and self.gate_proj is None and self.q_norm is None and self.window is None and not self.softcap
                 and self.sinks is None and segment_ids is None and not self.track_qk_max and self.q_gain is None):

@@ -3,6 +3,8 @@
 Parity: src/dew/nn/kv_cache.py (``KVCache`` spec :362-408 - ``quantized``, ``page_size``, ``pages``, ``groups``,
 ``offloaded``; ``quantize`` / ``dequantize`` :411-446 per-token-per-head absmax scales; ``hadamard`` :465-479;
 ``KVStore.write / attend / decode`` :787-1180; pool layout :1297-1320; ``gather_cache_rows`` :1686).
+A decoder whose layers differ in what they keep (heads of other widths, recurrent states, a layer that runs several times) gives the store
+one ``CacheSlot`` per layer run; ``attend_slot`` and ``state`` then take the place of ``attend``.
 Pool layout here: ``[layers, pages, page_size, kv_heads, head_dim]`` for keys and for values, a page table
 ``[rows, max_pages]`` and ``lengths [rows]``; a dense cache is the special case of one page per row.
 """
@@ -12,12 +14,13 @@ import ctypes
 import math
 import os
 from dataclasses import dataclass
-from typing import Optional, Tuple
+from typing import List, Optional, Sequence, Tuple
 
 import torch
 
 from .. import ops
 from ..ops import library as L
+from ..ops import paged as P
 
 LIMITS = {"int8": 127.0, "float8_e4m3fn": 448.0}
 KINDS = {None: 0, "int8": 1, "float8_e4m3fn": 2}
@@ -34,6 +37,40 @@ class KVCache:
     def __post_init__(self):
         if self.quantized not in KINDS:
             raise ValueError(f"quantized must be one of {list(KINDS)}, got {self.quantized!r}")
+
+
+@dataclass(frozen=True)
+class CacheSlot:
+    """What one run of a layer keeps per row: keys and values of its own head count and widths, or a recurrent state (a shape, fp32)."""
+    kv_heads: int = 0
+    head_dim: int = 0
+    value_dim: int = 0
+    state: Optional[Tuple[int, ...]] = None
+
+
+@dataclass
+class Call:
+    """The integers of one forward call, computed once for all its layers.  ``key`` holds the positions tensor itself, so its memory cannot
+    be handed to another tensor while this entry can still be found."""
+    key: torch.Tensor
+    version: int
+    capturing: bool
+    row_key: Optional[torch.Tensor]
+    positions: torch.Tensor                  # int32 [R, S], below 0 = padding
+    lengths: torch.Tensor                    # int32 [R]: tokens a row holds after this call's last position (decode: position + 1)
+    row_ids: Optional[torch.Tensor]          # int32 store row of each call row, None: the same
+    table: torch.Tensor                      # int32 [R, max_pages]: the call rows' page tables
+    fresh: Optional[bool] = None             # every row starts at its first token (None: not looked at)
+
+
+def pool_width(slot: CacheSlot, dtype) -> int:
+    """Width of a slot's pool heads: what the bf16 kernels are built for (64, 128, 256) where the head fits, else the head rounded up to 8."""
+    w = max(slot.head_dim, slot.value_dim)
+    if dtype == torch.bfloat16:
+        for d in (64, 128, 256):
+            if w <= d:
+                return d
+    return (w + 7) // 8 * 8
 
 
 def hadamard(x: torch.Tensor) -> torch.Tensor:
@@ -70,8 +107,9 @@ def default_page_table(rows: int, pages_per_row: int, device=None) -> torch.Tens
 
 class KVStore:
     def __init__(self, spec: KVCache, layers: int, rows: int, max_len: int, kv_heads: int, head_dim: int,
-                 dtype=torch.bfloat16, device="cpu"):
+                 dtype=torch.bfloat16, device="cpu", slots: Optional[Sequence[CacheSlot]] = None):
         self.spec = spec
+        self.slots = None if slots is None else list(slots)
         self.layers, self.rows, self.max_len, self.kv_heads, self.head_dim = layers, rows, max_len, kv_heads, head_dim
         self.page_size = spec.page_size or max_len
         self.max_pages = (max_len + self.page_size - 1) // self.page_size
@@ -80,11 +118,21 @@ class KVStore:
         store = {0: dtype, 1: torch.int8, 2: torch.float8_e4m3fn}[self.kind]
         # one page beyond the addressable pool: writes of padding positions land there, so that a write needs no data-dependent
         # shapes (and therefore no host synchronisation); no page table entry ever names it
-        shape = (layers, self.pages + 1, self.page_size, kv_heads, head_dim)
-        self.k = torch.zeros(shape, dtype=store, device=device)
-        self.v = torch.zeros(shape, dtype=store, device=device)
-        self.k_scale = torch.ones(shape[:-1], dtype=torch.float32, device=device) if self.kind else None
-        self.v_scale = torch.ones(shape[:-1], dtype=torch.float32, device=device) if self.kind else None
+        self.states: List[Optional[torch.Tensor]] = []
+        self._call: Optional[Call] = None
+        if self.slots is not None:
+            if self.kind:
+                raise NotImplementedError("quantised storage is built for caches whose layers all keep the same heads")
+            pool = lambda s: None if s.state is not None else torch.zeros(self.pages + 1, self.page_size, s.kv_heads, pool_width(s, dtype), dtype=dtype, device=device)
+            self.k, self.v = [pool(s) for s in self.slots], [pool(s) for s in self.slots]
+            self.states = [None if s.state is None else torch.zeros(rows, *s.state, dtype=torch.float32, device=device) for s in self.slots]
+            self.k_scale = self.v_scale = None
+        else:
+            shape = (layers, self.pages + 1, self.page_size, kv_heads, head_dim)
+            self.k = torch.zeros(shape, dtype=store, device=device)
+            self.v = torch.zeros(shape, dtype=store, device=device)
+            self.k_scale = torch.ones(shape[:-1], dtype=torch.float32, device=device) if self.kind else None
+            self.v_scale = torch.ones(shape[:-1], dtype=torch.float32, device=device) if self.kind else None
         self.page_table = default_page_table(rows, self.max_pages, device) if spec.pages is None else \
             torch.zeros(rows, self.max_pages, dtype=torch.int32, device=device)
         self.lengths = torch.zeros(rows, dtype=torch.int32, device=device)
@@ -92,6 +140,81 @@ class KVStore:
         self.row_ids: Optional[torch.Tensor] = None      # rows of the store addressed by the batch rows of a call
         self._scratch = None
         self.chunk_span: Optional[Tuple[int, int]] = None      # (first position, one past the last) of the prefill chunk in flight, when the caller knows
+
+    # ------------------------------------------------------------------ layers that differ (CacheSlot)
+    @property
+    def recurrent(self) -> bool:
+        """Whether some layer keeps a state (which no page holds: a prompt's prefix cannot be taken from another row's pages)."""
+        return any(s.state is not None for s in self.slots or ())
+
+    def call(self, positions: torch.Tensor) -> Call:
+        """The integers of the call whose layers pass ``positions [R, S]``: made by the first layer, found by the others."""
+        capturing = positions.is_cuda and torch.cuda.is_current_stream_capturing()
+        c = self._call
+        if c is not None and c.key is positions and c.version == positions._version and c.capturing == capturing and c.row_key is self.row_ids:
+            return c
+        pos = positions.to(torch.int32).contiguous()
+        ids = self.row_ids
+        if ids is None and positions.shape[0] > self.rows:
+            raise ValueError(f"{positions.shape[0]} rows do not fit a cache of {self.rows}")
+        table = self.page_table[: positions.shape[0]] if ids is None else self.page_table[ids]
+        self._call = Call(positions, positions._version, capturing, ids, pos, (pos.amax(1) + 1).to(torch.int32),
+                          None if ids is None else ids.to(torch.int32), table)
+        return self._call
+
+    def is_fresh(self, c: Call) -> bool:
+        if self.chunk_span is not None:
+            return self.chunk_span[0] == 0
+        if c.fresh is None:
+            c.fresh = bool((c.positions[:, 0] <= 0).all())
+        return c.fresh
+
+    def attend_slot(self, slot: int, qkv: torch.Tensor, heads: P.Heads, positions: torch.Tensor, *, scale: float, eps: float = 1e-6, q_weight=None,
+                    k_weight=None, temperature=None) -> torch.Tensor:
+        """A layer's attention from its packed projection ``qkv [R, S, H dk + G dk + G dv]``: norms, temperature, append, causal attention
+        against everything the rows hold.  -> ``[R, S, H, dv]``.  A prompt from its first token takes the tcgen05 flash kernel, a decode
+        step the paged decode kernels, anything else (and fp32) the general paged kernel."""
+        c = self.call(positions)
+        pages = P.Pages(self.k[slot], self.v[slot], self.page_table, self.page_size, c.row_ids)
+        packed = P.qk_norm_append(qkv, heads, q_weight, k_weight, eps, temperature, c.positions, pages)
+        R, S = positions.shape
+        H, G = heads.q, heads.kv
+        D = packed.shape[-1]
+        q = packed[:, :, :H]
+        if L.use_cuda(qkv) and qkv.dtype == torch.bfloat16:
+            if S == 1 and D in (64, 128, 256):
+                return self._decode_slot(slot, packed, heads, c, scale)[:, None, :, :heads.dv]
+            if D in (64, 128) and S % 128 == 0 and self.is_fresh(c):
+                from ..ops.flash import flash_fwd
+                out, _ = flash_fwd(q, packed[:, :, H:H + G], packed[:, :, H + G:], True, scale, need_lse=False)
+                return out[..., :heads.dv]
+        return P.paged_attend(q, heads, c.positions, pages, scale)
+
+    def _decode_slot(self, slot: int, packed: torch.Tensor, heads: P.Heads, c: Call, scale: float) -> torch.Tensor:
+        lib = L.load()
+        R, D, H, G = packed.shape[0], packed.shape[-1], heads.q, heads.kv
+        out = torch.empty(R, H, D, dtype=packed.dtype, device=packed.device)
+        if D == 128 and self.page_size % 64 == 0 and H // G <= 8 and hasattr(lib, "dewb_paged_decode_persist"):
+            self._fused_decode(lib, slot, packed, (H + 2 * G) * D, c.lengths, R, H, D, None, None, out, scale=scale, kv_heads=G, table=c.table)
+            return out
+        q = packed[:, 0, :H].contiguous()
+        share = next(s for s in range(1, H // G + 1) if (H // G) % s == 0 and H // G // s <= 8)     # CTAs that share a key / value head
+        splits = 1
+        while splits < 16 and R * G * share * splits < 592 and self.max_len // (splits * 2) >= 256:
+            splits *= 2
+        pm, pl, pa = self._partials(R * H * splits, D, q.device)
+        L.check(lib.dewb_paged_decode(L.ptr(q), L.ptr(self.k[slot]), L.ptr(self.v[slot]), L.ptr(None), L.ptr(None), L.ptr(c.table), L.ptr(c.lengths),
+                                      L.ptr(None), L.ptr(out), L.ptr(None), L.ptr(pm), L.ptr(pl), L.ptr(pa), ctypes.c_int(R), ctypes.c_int(H),
+                                      ctypes.c_int(G), ctypes.c_int(share), ctypes.c_int(D), ctypes.c_int(self.page_size), ctypes.c_int(self.max_pages),
+                                      ctypes.c_int(splits), ctypes.c_float(scale), ctypes.c_int(0), ctypes.c_int(0), L.stream_ptr()), "paged_decode")
+        L.count_launches(2)
+        return out
+
+    def _partials(self, n: int, D: int, device):
+        if self._scratch is None or self._scratch[0].numel() < n or self._scratch[2].numel() < n * D:
+            self._scratch = (torch.empty(n, dtype=torch.float32, device=device), torch.empty(n, dtype=torch.float32, device=device),
+                             torch.empty(n * D, dtype=torch.float32, device=device))
+        return self._scratch
 
     # ------------------------------------------------------------------ latent rows (multi-head latent attention)
     def latent(self, layer: int, width: int) -> torch.Tensor:
@@ -187,7 +310,8 @@ class KVStore:
 
     MIN_TILES = 4            # fewest 64-key tiles one CTA of the balanced decode kernel takes (bounds the parts a row is cut into)
 
-    def _fused_decode(self, lib, layer: int, q, q_row_stride: int, lens32, R: int, Hq: int, D: int, window, sinks32, out) -> None:
+    def _fused_decode(self, lib, layer: int, q, q_row_stride: int, lens32, R: int, Hq: int, D: int, window, sinks32, out,
+                      scale: Optional[float] = None, kv_heads: Optional[int] = None, table: Optional[torch.Tensor] = None) -> None:
         """The streamed paged-attention kernel finishing its rows itself.  Up to 1024 rows take the balanced persistent form
         (every CTA moves the same number of tiles, whatever the rows' lengths); more rows take one CTA per (row, head, chunk)."""
         longest = min(self.max_len, window) if window else self.max_len
@@ -200,24 +324,23 @@ class KVStore:
             chunk = 8
             splits = max(1, -(-max_tiles // chunk))
         n = R * Hq * splits
-        if self._scratch is None or self._scratch[0].numel() < n:
-            self._scratch = (torch.empty(n, dtype=torch.float32, device=q.device), torch.empty(n, dtype=torch.float32, device=q.device),
-                             torch.empty(n * D, dtype=torch.float32, device=q.device))
-        if getattr(self, "_arrivals", None) is None or self._arrivals.numel() < R * self.kv_heads:
-            self._arrivals = torch.zeros(R * self.kv_heads, dtype=torch.int32, device=q.device)
-        pm, pl, pa = self._scratch
+        scale = 1.0 / math.sqrt(D) if scale is None else scale
+        kv_heads = self.kv_heads if kv_heads is None else kv_heads
+        pm, pl, pa = self._partials(n, D, q.device)
+        if getattr(self, "_arrivals", None) is None or self._arrivals.numel() < R * kv_heads:
+            self._arrivals = torch.zeros(R * kv_heads, dtype=torch.int32, device=q.device)
         common = (L.ptr(q), L.ptr(self.k[layer]), L.ptr(self.v[layer]), ctypes.c_longlong(self.pages * self.page_size),
-                  L.ptr(self.page_table), L.ptr(lens32), L.ptr(pm), L.ptr(pl), L.ptr(pa), L.ptr(self._arrivals), L.ptr(sinks32),
-                  L.ptr(out), ctypes.c_int(R), ctypes.c_int(Hq), ctypes.c_int(self.kv_heads), ctypes.c_int(self.page_size),
+                  L.ptr(self.page_table if table is None else table), L.ptr(lens32), L.ptr(pm), L.ptr(pl), L.ptr(pa), L.ptr(self._arrivals), L.ptr(sinks32),
+                  L.ptr(out), ctypes.c_int(R), ctypes.c_int(Hq), ctypes.c_int(kv_heads), ctypes.c_int(self.page_size),
                   ctypes.c_int(self.max_pages), ctypes.c_int(splits))
         if persist:
             if getattr(self, "_ctas", None) is None:
                 self._ctas = 2 * torch.cuda.get_device_properties(q.device).multi_processor_count
-            L.check(lib.dewb_paged_decode_persist(*common, ctypes.c_int(min_tiles), ctypes.c_float(1.0 / math.sqrt(D)),
+            L.check(lib.dewb_paged_decode_persist(*common, ctypes.c_int(min_tiles), ctypes.c_float(scale),
                                                   ctypes.c_int(window or 0), ctypes.c_longlong(q_row_stride), ctypes.c_int(self._ctas),
                                                   L.ptr(L.status(q.device)), L.stream_ptr()), "paged_decode_persist")
         else:
-            L.check(lib.dewb_paged_decode_fused(*common, ctypes.c_int(chunk), ctypes.c_float(1.0 / math.sqrt(D)),
+            L.check(lib.dewb_paged_decode_fused(*common, ctypes.c_int(chunk), ctypes.c_float(scale),
                                                 ctypes.c_int(window or 0), ctypes.c_longlong(q_row_stride),
                                                 L.ptr(L.status(q.device)), L.stream_ptr()), "paged_decode_fused")
         L.count_launches()
@@ -273,10 +396,7 @@ class KVStore:
             # the longest possible row near 512 keys so that the walk is short and there are CTAs to overlap
             splits = max(splits, min(16, (longest + 511) // 512))
             n = R * Hq * splits
-            if self._scratch is None or self._scratch[0].numel() < n:
-                self._scratch = (torch.empty(n, dtype=torch.float32, device=q.device), torch.empty(n, dtype=torch.float32, device=q.device),
-                                 torch.empty(n * D, dtype=torch.float32, device=q.device))
-            pm, pl, pa = self._scratch
+            pm, pl, pa = self._partials(n, D, q.device)
             out = torch.empty_like(q)
             qc, lens32 = q.contiguous(), lengths.to(torch.int32).contiguous()      # kept referenced across the launches below
             sinks32 = sinks.float().contiguous() if sinks is not None else None
@@ -302,7 +422,7 @@ class KVStore:
                                           L.ptr(self.v_scale[layer] if self.kind else None), L.ptr(self.page_table),
                                           L.ptr(lens32), L.ptr(sinks32), L.ptr(out), L.ptr(None),
                                           L.ptr(pm), L.ptr(pl), L.ptr(pa), ctypes.c_int(R), ctypes.c_int(Hq),
-                                          ctypes.c_int(self.kv_heads), ctypes.c_int(D), ctypes.c_int(self.page_size),
+                                          ctypes.c_int(self.kv_heads), ctypes.c_int(1), ctypes.c_int(D), ctypes.c_int(self.page_size),
                                           ctypes.c_int(self.max_pages), ctypes.c_int(splits), ctypes.c_float(scale),
                                           ctypes.c_int(window or 0), ctypes.c_int(self.kind), L.stream_ptr()), "paged_decode")
             L.count_launches(2)

@@ -80,16 +80,17 @@ class RMSNorm(nn.Module):
 
 
 class LayerNorm(nn.Module):
-    def __init__(self, features: int, eps: float = 1e-6, affine: bool = True, dtype=None, device=None):
+    def __init__(self, features: int, eps: float = 1e-6, affine: bool = True, bias: bool = True, dtype=None, device=None):
         super().__init__()
         self.features, self.eps = features, eps
         self.weight = declare(nn.Parameter(torch.ones(features, dtype=dtype, device=device)), ("norm",), "scale") if affine else None
-        self.bias = declare(nn.Parameter(torch.zeros(features, dtype=dtype, device=device)), ("norm",), "bias") if affine else None
+        self.bias = declare(nn.Parameter(torch.zeros(features, dtype=dtype, device=device)), ("norm",), "bias") if affine and bias else None
 
     def reset_parameters(self, generator=None):
         with torch.no_grad():
             if self.weight is not None:
                 self.weight.fill_(1.0)
+            if self.bias is not None:
                 self.bias.zero_()
 
     def forward(self, x):

@@ -8,6 +8,7 @@ import torch.nn as nn
 import torch.nn.functional as F
 
 from .. import ops
+from ..ops import streams
 from .layers import Linear
 
 
@@ -31,6 +32,20 @@ class SwiGLU(nn.Module):
         gu = self.gate_up_proj(x)
         g, u = gu.chunk(2, -1)                                    # GeGLU (Gemma): the gate passes through GELU
         return self.down_proj(F.gelu(g, approximate="tanh" if self.activation == "gelu_tanh" else "none") * u)
+
+
+class ClampedGLU(nn.Module):
+    """``down(g sigmoid(alpha g) (u + 1))`` with ``g = min(gate(x), limit)`` and ``u = clamp(up(x), -limit, limit)``: GPT-OSS's activation in a
+    dense block; gate and up share one ``[2F, d]`` weight, gate rows first."""
+
+    def __init__(self, features: int, hidden: int, limit: float, alpha: float = 1.702, init_std: Optional[float] = None, dtype=None, device=None):
+        super().__init__()
+        self.features, self.hidden, self.limit, self.alpha = features, hidden, float(limit), float(alpha)
+        self.gate_up_proj = Linear(features, 2 * hidden, axes=("embed", "mlp"), init_std=init_std, dtype=dtype, device=device)
+        self.down_proj = Linear(hidden, features, axes=("mlp", "embed"), init_std=init_std, dtype=dtype, device=device)
+
+    def forward(self, x):
+        return self.down_proj(streams.clamped_glu(self.gate_up_proj(x), self.limit, self.alpha))
 
 
 class GeluMLP(nn.Module):

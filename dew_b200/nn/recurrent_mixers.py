@@ -22,7 +22,7 @@ import torch.nn as nn
 import torch.nn.functional as F
 
 from .. import ops
-from ..ops import scan
+from ..ops import decayed, scan, streams
 from .layers import Linear, declare
 
 
@@ -65,33 +65,55 @@ def lightning_attention(q, k, v, rate, state=None):
 
 
 class LightningAttention(nn.Module):
+    """``decay``: the decay of every head (one number or a list) instead of the ALiBi-slope rates; ``value_dim``: values of another width."""
+
     def __init__(self, features: int, num_heads: int = 8, head_dim: int = 64, depth: int = 0, layers: int = 1, norm_eps: float = 1e-6,
-                 dtype=None, device=None):
+                 decay=None, value_dim: Optional[int] = None, dtype=None, device=None):
         super().__init__()
-        self.h, self.d = num_heads, head_dim
-        inner = num_heads * head_dim
-        self.qkv = Linear(features, 3 * inner, axes=("embed", "heads"), dtype=dtype, device=device)
+        self.h, self.d, self.dv = num_heads, head_dim, value_dim or head_dim
+        inner = num_heads * self.dv
+        self.qkv = Linear(features, 2 * num_heads * head_dim + inner, axes=("embed", "heads"), dtype=dtype, device=device)
         self.output_gate = Linear(features, inner, axes=("embed", "heads"), dtype=dtype, device=device)
         self.norm_weight = declare(nn.Parameter(torch.ones(inner, dtype=dtype, device=device)), ("norm",), "scale")
         self.out_proj = Linear(inner, features, axes=("heads", "embed"), dtype=dtype, device=device)
         self.eps = norm_eps
-        # the first layer forgets fastest: slope * (1 - depth / (layers - 1) + 1e-5)
-        factor = 1.0 - depth / max(layers - 1, 1) + 1e-5
-        self.register_buffer("rate", alibi_slopes(num_heads).float() * factor, persistent=False)
+        if decay is None:
+            # the first layer forgets fastest: slope * (1 - depth / (layers - 1) + 1e-5)
+            rate = alibi_slopes(num_heads).float() * (1.0 - depth / max(layers - 1, 1) + 1e-5)
+            values = torch.exp(-rate)
+        else:
+            values = torch.tensor(decay, dtype=torch.float64).expand(num_heads).clone()
+            rate = -torch.log(values.clamp_min(1e-300)).float()
+        self._constants = (rate.tolist(), values.tolist())
+        self.register_buffer("rate", rate, persistent=False)
+        self._decay: Optional[torch.Tensor] = None
 
-    def forward(self, x, segment_ids=None, cache=None, layer: int = 0):
+    def decay_on(self, device) -> torch.Tensor:
+        """The per-head decay in fp32 whatever the module's parameters were cast to."""
+        if self._decay is None or self._decay.device != torch.device(device):
+            self._decay = torch.tensor(self._constants[1], dtype=torch.float64).float().to(device)
+        return self._decay
+
+    def forward(self, x, segment_ids=None, cache=None, layer: int = 0, positions=None):
         B, T, _ = x.shape
-        q, k, v = F.silu(self.qkv(x)).view(B, T, 3, self.h, self.d).unbind(2)
+        if getattr(cache, "slots", None) is not None:
+            c = cache.call(positions)
+            o = decayed.decayed_attention(self.qkv(x), self.decay_on(x.device), self.h, self.d, self.dv, cache.states[layer], c.positions, c.row_ids)
+            o = streams.sigmoid_gated_norm(o.reshape(B, T, -1), self.output_gate(x), self.norm_weight, self.eps)
+            return self.out_proj(o)
+        q, k, v = F.silu(self.qkv(x)).split([self.h * self.d, self.h * self.d, self.h * self.dv], -1)
+        q, k, v = q.view(B, T, self.h, self.d), k.view(B, T, self.h, self.d), v.view(B, T, self.h, self.dv)
         state = cache.recurrent(layer, B, self) if cache is not None and hasattr(cache, "recurrent") else None
-        o, S = lightning_attention(q, k, v, self.rate.to(x.device), state["S"] if state is not None else None)
+        rate = torch.tensor(self._constants[0], device=x.device)
+        o, S = lightning_attention(q, k, v, rate, state["S"] if state is not None else None)
         if state is not None:
             state["S"].copy_(S)
-        o = ops.rms_norm(o.reshape(B, T, -1).to(x.dtype), self.norm_weight, self.eps)
-        return self.out_proj(o * torch.sigmoid(self.output_gate(x)))
+        o = streams.sigmoid_gated_norm(o.reshape(B, T, -1).to(x.dtype), self.output_gate(x), self.norm_weight, self.eps)
+        return self.out_proj(o)
 
     def fresh_state(self, batch: int) -> dict:
         p = self.out_proj.weight
-        return {"S": torch.zeros(batch, self.h, self.d, self.d, dtype=torch.float32, device=p.device)}
+        return {"S": torch.zeros(batch, self.h, self.d, self.dv, dtype=torch.float32, device=p.device)}
 
 
 # ---------------------------------------------------------------------------------------------------------------

@@ -9,6 +9,8 @@ streams (initialised to zero, so training starts from the static form).
 ``AltUp`` (K blocks): predict every block from all blocks (``P`` [K x K], identity at start), run the layer on ONE block
 (``layer % K``), and correct every block by its gate times the layer's innovation on the active block.
 
+``StreamStack`` runs a stack of static hyper-connections (``dynamic=False``: the weights alone, no input-dependent part) over fp32 streams.
+
 A stack of either with one stream / block reduces to the ordinary pre-norm residual stack.
 Reference: ``hyper_connections`` and ``altup`` fields of src/dew/nn/backbones/causal_transformer.py:165-423.
 """
@@ -17,6 +19,9 @@ from __future__ import annotations
 import torch
 import torch.nn as nn
 import torch.nn.functional as F
+
+from ..ops import streams as S
+from .layers import LayerNorm
 
 
 class HyperConnections(nn.Module):
@@ -57,6 +62,39 @@ class HyperConnections(nn.Module):
     def write(self, H: torch.Tensor, out: torch.Tensor, ctx) -> torch.Tensor:
         mix, beta = ctx
         return torch.einsum("bsij,bsid->bsjd", mix.to(H.dtype), H) + beta.to(H.dtype).unsqueeze(-1) * out.unsqueeze(2)
+
+
+class StreamStack:
+    """The fp32 streams of one forward call under static hyper-connections.  A sub-layer's write is held back until the next read, so that
+    write, read and norm are one pass over the streams (``ops.streams.stream_step``)."""
+
+    def __init__(self, H: torch.Tensor, dtype):
+        self.H, self.dtype, self.pending = H, dtype, None
+
+    def enter(self, connection: "HyperConnections", norm: nn.Module) -> torch.Tensor:
+        """The next sub-layer's normalised input."""
+        return self._step(connection.alpha, norm)
+
+    def leave(self, connection: "HyperConnections", y: torch.Tensor, scale=None) -> None:
+        """The sub-layer's output (times its layer scale), to be written back by the connection."""
+        self.pending = S.Write(y, scale, connection.mix, connection.beta)
+
+    def finish(self, norm: nn.Module) -> torch.Tensor:
+        """The final norm of the sum of the streams."""
+        return self._step(torch.ones(self.H.shape[-2], device=self.H.device), norm)
+
+    def total(self) -> torch.Tensor:
+        """The sum of the streams after everything so far."""
+        if self.pending is not None:
+            _, self.H = S.stream_step(self.H, self.pending, self.pending.out, None, 0.0, self.dtype)
+            self.pending = None
+        return self.H.sum(-2)
+
+    def _step(self, read, norm) -> torch.Tensor:
+        kind = "layer" if isinstance(norm, LayerNorm) else "rms"
+        n, self.H = S.stream_step(self.H, self.pending, read, norm.weight, norm.eps, self.dtype, kind)
+        self.pending = None
+        return n
 
 
 class AltUp(nn.Module):

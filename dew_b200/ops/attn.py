@@ -33,6 +33,7 @@ _ATTN.kernels = [
         Requirement("built", lambda c: _flash_available(), "flash kernels are not in this build of libdewb.so"),
         Requirement("dtype", lambda c: c["dtype"] == torch.bfloat16, "bf16 only"),
         Requirement("head_dim", lambda c: c["D"] in (64, 128), "head_dim must be 64 or 128"),
+        Requirement("value_dim", lambda c: c.get("Dv", c["D"]) == c["D"], "values as wide as the keys"),
         Requirement("variants", lambda c: not c["segments"] or (c["S"] == c["T"] and c["S"] % 4 == 0),
                     "packed segments need S == T and rows of ids on 16-byte boundaries"),
         Requirement("seq", lambda c: c["S"] == c["T"] and c["S"] % 128 == 0, "needs S == T and S a multiple of 128"),
@@ -61,7 +62,7 @@ def _sdpa(q, k, v, causal, scale, window, softcap, sinks, segment_ids):
 def flash_attention(q, k, v, causal=True, scale=None, window=None, softcap=0.0, sinks=None, segment_ids=None,
                     kernel: Optional[str] = None):
     B, S, Hq, D = q.shape
-    case = dict(dtype=q.dtype, D=D, S=S, T=k.shape[1], Hq=Hq, Hkv=k.shape[2], sinks=sinks is not None,
+    case = dict(dtype=q.dtype, D=D, Dv=v.shape[-1], S=S, T=k.shape[1], Hq=Hq, Hkv=k.shape[2], sinks=sinks is not None,
                 softcap=bool(softcap), window=window, segments=segment_ids is not None, causal=causal,
                 grad=torch.is_grad_enabled() and (q.requires_grad or k.requires_grad or v.requires_grad),
                 unit_d=q.stride(3) == 1 and k.stride(3) == 1 and v.stride(3) == 1)

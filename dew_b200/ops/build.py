@@ -13,7 +13,7 @@ import subprocess
 import sys
 from concurrent.futures import ThreadPoolExecutor
 from pathlib import Path
-from typing import List
+from typing import List, Optional
 
 ROOT = Path(__file__).resolve().parents[2]
 CSRC = ROOT / "csrc"
@@ -24,6 +24,16 @@ LIB = OUT_DIR / "libdewb.so"
 ARCH_FLAGS = ["-gencode", "arch=compute_100a,code=sm_100a"]
 NVCC_FLAGS = ["-O3", "-std=c++17", "-lineinfo", "--use_fast_math", "-Xcompiler", "-fPIC", "-Xptxas", "-v",
               "--expt-relaxed-constexpr"]
+
+# Files whose 32-bit arithmetic has to hold up on its own (decoders that run in fp32): compiled without fast math.
+EXACT_MATH = ("residual_streams", "paged_attention", "decayed_recurrence")
+
+# Subsets of the library a program can build alone, as ``libdewb_<part>.so``: a process that only decodes needs neither the training nor
+# the multi-GPU kernels.
+PARTS = {
+    "decoder": ("elementwise", "decode_attention", "decode_attention_tma", "flash_fwd_sm100", "gemm_sm100", "gemm_pair_sm100", "sampling")
+    + EXACT_MATH,
+}
 
 
 def nvcc() -> str:
@@ -43,8 +53,12 @@ def _digest(path: Path) -> str:
     for folder in ("common", "include"):                       # every header a kernel file may include
         for hdr in sorted((CSRC / folder).glob("*")):
             h.update(hdr.read_bytes())
-    h.update(" ".join(ARCH_FLAGS + NVCC_FLAGS).encode())
+    h.update(" ".join(ARCH_FLAGS + _flags(path)).encode())
     return h.hexdigest()[:16]
+
+
+def _flags(src: Path) -> List[str]:
+    return [f for f in NVCC_FLAGS if f != "--use_fast_math"] if src.stem in EXACT_MATH else NVCC_FLAGS
 
 
 def _compile(src: Path, verbose: bool) -> Path:
@@ -54,7 +68,7 @@ def _compile(src: Path, verbose: bool) -> Path:
         return obj
     for stale in OBJ_DIR.glob(f"{src.stem}.*.o"):
         stale.unlink()
-    cmd = [nvcc(), *ARCH_FLAGS, *NVCC_FLAGS, "-I", str(CSRC), "-c", str(src), "-o", str(obj)]
+    cmd = [nvcc(), *ARCH_FLAGS, *_flags(src), "-I", str(CSRC), "-c", str(src), "-o", str(obj)]
     res = subprocess.run(cmd, capture_output=True, text=True)
     log = OBJ_DIR / f"{src.stem}.ptxas.log"
     log.write_text(res.stdout + res.stderr)
@@ -65,25 +79,31 @@ def _compile(src: Path, verbose: bool) -> Path:
     return obj
 
 
-def build(verbose: bool = True, force: bool = False) -> Path:
-    """Compile what changed and link; returns the library path."""
+def part_path(part: str) -> Path:
+    return OUT_DIR / f"libdewb_{part}.so"
+
+
+def build(verbose: bool = True, force: bool = False, part: Optional[str] = None) -> Path:
+    """Compile what changed and link; returns the library path.  With ``part``, only the files of ``PARTS[part]``, into a library of
+    their own."""
     if force and OBJ_DIR.exists():
         shutil.rmtree(OBJ_DIR)
-    srcs = sources()
+    srcs = [p for p in sources() if part is None or p.stem in PARTS[part]]
+    lib = LIB if part is None else part_path(part)
     with ThreadPoolExecutor(max_workers=min(8, max(1, len(srcs)))) as pool:
         objs = list(pool.map(lambda s: _compile(s, verbose), srcs))
-    stamp = OBJ_DIR / "link.stamp"
+    stamp = OBJ_DIR / ("link.stamp" if part is None else f"link_{part}.stamp")
     want = " ".join(o.name for o in objs)
-    if LIB.exists() and stamp.exists() and stamp.read_text() == want:
-        return LIB
-    cmd = [nvcc(), "-shared", *ARCH_FLAGS, "-Xcompiler", "-fPIC", "-o", str(LIB), *map(str, objs), "-cudart", "static"]
+    if lib.exists() and stamp.exists() and stamp.read_text() == want:
+        return lib
+    cmd = [nvcc(), "-shared", *ARCH_FLAGS, "-Xcompiler", "-fPIC", "-o", str(lib), *map(str, objs), "-cudart", "static"]
     res = subprocess.run(cmd, capture_output=True, text=True)
     if res.returncode != 0:
         raise RuntimeError(f"link failed:\n{res.stdout}\n{res.stderr}")
     stamp.write_text(want)
     if verbose:
-        print(f"[dew_b200.build] linked {LIB}", file=sys.stderr)
-    return LIB
+        print(f"[dew_b200.build] linked {lib}", file=sys.stderr)
+    return lib
 
 
 def ptxas_report() -> str:

@@ -54,6 +54,16 @@ def load(build_if_missing: bool = False) -> ctypes.CDLL:
     return _LIB
 
 
+def load_part(part: str) -> ctypes.CDLL:
+    """Load the whole library if it is built, else the subset ``build.PARTS[part]``, building that where it is missing or out of date:
+    for a program that runs from a source checkout and needs only those kernels."""
+    global _LIB, _LIB_PATH
+    if _LIB is None and not _LIB_PATH.exists():
+        from . import build
+        _LIB_PATH = build.build(verbose=False, part=part)
+    return load()
+
+
 def use_cuda(*tensors: torch.Tensor) -> bool:
     """True when the op must run on the CUDA library (all tensors on a GPU)."""
     t = next((x for x in tensors if isinstance(x, torch.Tensor)), None)

@@ -8,7 +8,7 @@ step, so a row's continuation does not depend on which rows share its batch.
 """
 from __future__ import annotations
 
-from dataclasses import dataclass, field
+from dataclasses import dataclass, field, replace
 from typing import Any, Callable, List, Optional, Sequence, Tuple
 
 import torch
@@ -135,23 +135,116 @@ def draw(logits: torch.Tensor, s: Sampling, row_keys: Sequence[int], step: int) 
 # ---------------------------------------------------------------------------------------------------------------
 
 
-def _prefill(model, params_call, tokens, lengths, store: KVStore):
-    """Run the prompts (right-padded) through the model, filling the cache; returns last-position logits ``[R, V]``."""
-    R, S = tokens.shape
-    pos = torch.arange(S, device=tokens.device)[None].expand(R, S).clone()
-    pos[pos >= lengths[:, None]] = -1
-    logits = params_call(tokens, positions=pos, cache=store)
-    last = (lengths - 1).clamp_min(0)
-    return logits[torch.arange(R, device=tokens.device), last]
-
-
 def make_cache(model, rows: int, max_len: int, spec: Optional[KVCache] = None, device=None, dtype=None) -> KVStore:
     cfg = model.config
     hd = cfg.head_dim or cfg.emb_features // cfg.num_heads
     p = next(model.parameters())
     kvh = getattr(model, "local_kv_heads", None) or (cfg.num_kv_heads or cfg.num_heads)     # this rank's KV heads under TP
-    return KVStore(spec or KVCache(), cfg.num_layers, rows, max_len, kvh, hd,
-                   dtype or p.dtype, device or p.device)
+    slots = model.cache_slots() if hasattr(model, "cache_slots") else None
+    if slots is not None and (spec is None or spec.page_size is None):
+        spec = replace(spec or KVCache(), page_size=64)                                     # the paged decode kernels walk tiles of 64 keys
+    layers = len(model.runs()) if hasattr(model, "runs") else cfg.num_layers                # a looped block keeps a cache per pass
+    return KVStore(spec or KVCache(), layers, rows, max_len, kvh, hd, dtype or p.dtype, device or p.device, slots=slots)
+
+
+class RowBatch:
+    """Rows of token ids going through a model with one cache: the step ``generate`` loops over and a trace is replayed with.
+
+    ``feed`` takes the next tokens of every row (none for a row that rests), ``forward`` the same as device tensors.  With ``pool_tokens`` the
+    rows share a page pool of that many tokens, take pages as they grow and give them back on ``release``; without it every row has room for
+    ``max_len`` tokens from the start."""
+
+    PAGE = 64
+
+    def __init__(self, model, rows: int, max_len: int, params=None, kv_cache: Optional[KVCache] = None, pool_tokens: Optional[int] = None):
+        self.model, self.rows, self.max_len = model, rows, max_len
+        self.ledger = None
+        if pool_tokens is not None:
+            from ..inference.pages import PageLedger
+            # a row's last page may be partly empty: one page per row on top
+            pages = -(-pool_tokens // self.PAGE) + rows
+            kv_cache = KVCache(page_size=self.PAGE, pages=pages)
+            self.ledger = PageLedger(pages, self.PAGE, prefix_cache=False)
+            self.pages: List[List[int]] = [[] for _ in range(rows)]
+        self.store: KVStore = make_cache(model, rows, max_len, kv_cache)
+        self.device = self.store.device
+        self.lengths = [0] * rows
+        self.splits_head = params is None and hasattr(model, "logits")
+        if params is None:
+            self.call = lambda t, **kw: model(t, **kw)
+        else:
+            from ..utils.trees import variables_for_call
+            named = variables_for_call(model, params)
+            self.call = lambda t, **kw: torch.func.functional_call(model, named, (t,), kw)
+
+    def forward(self, ids: torch.Tensor, positions: torch.Tensor, span: Optional[Tuple[int, int]] = None, pick: Optional[torch.Tensor] = None):
+        """``ids, positions [rows, S]`` (positions below 0 = padding at a row's end) -> logits ``[n, V]`` at ``pick = (rows, places)`` or of
+        every position.  ``span``: where the tokens lie in every row, when the caller knows (saves the cache a device read)."""
+        self.store.chunk_span = span
+        try:
+            with torch.no_grad():
+                if self.splits_head:                         # the head runs on the picked positions alone
+                    hidden = self.call(ids, positions=positions, cache=self.store, return_hidden=True)
+                    if pick is not None and pick[0].numel() == 0:
+                        return None
+                    return self.model.logits(hidden if pick is None else hidden[pick])
+                logits = self.call(ids, positions=positions, cache=self.store)
+                return logits if pick is None else logits[pick]
+        finally:
+            self.store.chunk_span = None
+
+    def prefill(self, tokens: torch.Tensor, lengths: torch.Tensor) -> torch.Tensor:
+        """The prompts ``[rows, S]`` (right-padded), from their first token; returns last-position logits ``[rows, V]``."""
+        R, S = tokens.shape
+        if self.store.slots is not None and self.device.type == "cuda" and 1 < S and S % 128:
+            tokens = torch.nn.functional.pad(tokens, (0, 128 - S % 128))          # whole tiles for the flash kernel
+        pos = torch.arange(tokens.shape[1], device=tokens.device)[None].expand(R, -1)
+        pos = torch.where(pos < lengths[:, None], pos, torch.full_like(pos, -1))
+        return self.forward(tokens, pos, (0, S) if self.store.slots is not None else None,
+                            (torch.arange(R, device=tokens.device), (lengths - 1).clamp_min(0)))
+
+    def feed(self, pieces: Sequence[Sequence[int]], want: Optional[Sequence[Sequence[int]]] = None) -> Optional[torch.Tensor]:
+        """The next tokens of every row (an empty piece: the row rests); returns the logits at ``want`` (places within each piece, row by
+        row), None where nothing is wanted."""
+        if len(pieces) != self.rows:
+            raise ValueError(f"{len(pieces)} pieces for {self.rows} rows")
+        starts = self.lengths
+        width = max(len(p) for p in pieces)
+        if width == 0:
+            return None
+        vocab = getattr(self.model, "vocab_size", None)
+        for r, p in enumerate(pieces):
+            if starts[r] + len(p) > self.max_len:
+                raise ValueError(f"row {r}: {starts[r] + len(p)} tokens exceed the row capacity {self.max_len}")
+            if vocab is not None and len(p) and (min(p) < 0 or max(p) >= vocab):
+                raise ValueError(f"row {r}: token ids outside the vocabulary of {vocab}")
+        if self.store.slots is not None and self.device.type == "cuda" and width > 1:
+            width = (width + 127) // 128 * 128
+        ids, pos = torch.zeros(self.rows, width, dtype=torch.long), torch.full((self.rows, width), -1, dtype=torch.long)
+        for r, p in enumerate(pieces):
+            ids[r, :len(p)] = torch.tensor(list(p), dtype=torch.long)
+            pos[r, :len(p)] = torch.arange(starts[r], starts[r] + len(p))
+            if self.ledger is not None and len(p):
+                have = len(self.pages[r])
+                added = self.ledger.extend(self.pages[r], starts[r] + len(p))
+                if added:
+                    self.store.page_table[r, have:have + len(added)] = torch.tensor(added, dtype=torch.int32, device=self.device)
+        live = {starts[r] for r, p in enumerate(pieces) if len(p)}
+        span = (live.pop(), max(starts[r] + len(p) for r, p in enumerate(pieces))) if len(live) == 1 else None
+        if span is None and self.store.slots is not None:
+            span = (1, max(starts[r] + len(p) for r, p in enumerate(pieces)))     # rows at different places: not a fresh prompt
+        wanted = [(r, w) for r, ws in enumerate(want or ()) for w in ws]
+        pick = tuple(torch.tensor([x[j] for x in wanted], dtype=torch.long, device=self.device) for j in range(2))
+        out = self.forward(ids.to(self.device), pos.to(self.device), span, pick)
+        self.lengths = [n + len(p) for n, p in zip(starts, pieces)]
+        return out if wanted else None
+
+    def release(self, row: int) -> None:
+        """The row's sequence is finished: its pages go back to the pool, and its next tokens are a new sequence's first."""
+        self.lengths[row] = 0
+        if self.ledger is not None:
+            self.ledger.release(self.pages[row])
+            self.pages[row] = []
 
 
 def generate(model, params, inputs, max_new_tokens: int, *, key: int = 0, sampling: Sampling = Sampling(), n: int = 1,
@@ -180,21 +273,14 @@ def generate(model, params, inputs, max_new_tokens: int, *, key: int = 0, sampli
     for r, p in enumerate(prompts):
         tokens[r, :len(p)] = torch.tensor(p, device=dev)
 
-    if params is None:
-        call = lambda t, **kw: model(t, **kw)
-    else:
-        from ..utils.trees import variables_for_call
-        named = variables_for_call(model, params)
-        call = lambda t, **kw: torch.func.functional_call(model, named, (t,), kw)
-
-    store = make_cache(model, R, total, kv_cache)
+    batch = RowBatch(model, R, total, params, kv_cache)
     row_keys = [K.fold_in(K.key(key), r) for r in range(R)]
     eos = set(sampling.eos_token_ids or ())
     lengths = plen.clone()
     done = torch.zeros(R, dtype=torch.bool, device=dev)
     terminated = torch.zeros(R, dtype=torch.bool, device=dev)
     with torch.no_grad():
-        step_logits = _prefill(model, call, tokens[:, :S], plen, store)
+        step_logits = batch.prefill(tokens[:, :S], plen)
         for step in range(max_new_tokens):
             x = logits(step_logits, tokens, lengths) if logits is not None else step_logits
             x = transform_logits(x, tokens, lengths, sampling, step)
@@ -219,7 +305,7 @@ def generate(model, params, inputs, max_new_tokens: int, *, key: int = 0, sampli
             if bool(done.all()) or step == max_new_tokens - 1:
                 break
             pos = torch.where(done, torch.full_like(lengths, -1), lengths - 1)
-            step_logits = call(nxt[:, None], positions=pos[:, None], cache=store)[:, 0]
+            step_logits = batch.forward(nxt[:, None], pos[:, None])[:, 0]
     text = None
     if tokenizer is not None:
         text = [tokenizer.decode(tokens[r, int(plen[r]):int(lengths[r])].tolist()) for r in range(R)]
