@@ -2,6 +2,7 @@
 //     S_t = decay S_{t-1} + k_t v_t^T,   o_t = S_t^T q_t,   q, k, v = silu of the packed projection (or as given)
 //
 //   decayed_step        one token per row: the fp32 state is read and written once
+//   decayed_chunks      a call's tokens in chunks of 64 on the tensor cores (bf16, head widths up to 128 in multiples of 8)
 //   decayed_sequence    a call's tokens one after another, any head widths, fp32 arithmetic (the exact form; it also serves fp32 models)
 //
 // The packed projection is [rows, S, H dk | H dk | H dv] (q, k, v; heads inside each).  `state` [store rows, H, dk, dv] fp32 stays on the
@@ -10,6 +11,8 @@
 #include <cstdint>
 #include <cuda_bf16.h>
 #include <cuda_runtime.h>
+
+#include "../common/mma_bf16.cuh"
 
 namespace dewb {
 namespace decayed {
@@ -174,6 +177,224 @@ decayed_sequence_kernel(const T* __restrict__ qkv, const float* __restrict__ dec
   }
 }
 
+// Chunked form.  Within a chunk starting from state S:
+//     o_i = a^{i+1} S^T q_i + sum_{j <= i} a^{i-j} (q_i . k_j) v_j,      S' = a^n S + sum_j a^{n-1-j} k_j v_j^T
+// grid (H, ceil(dv / 64), rows), 8 warps.  The fp32 state lives in accumulator registers for the whole call.  Every factor that is not a
+// bf16 activation - the state, the decayed scores, the decayed keys - enters its product as a pair of bf16 (value and rounding rest), so the
+// products see 16 bits of it.  The next chunk's rows are fetched into registers while this one is computed.
+constexpr int CT = 64, VT = 64;       // tokens per chunk, value columns per CTA
+
+template <int DK>
+struct ChunkSmem {
+  bf16 q[CT][DK + 8], k[CT][DK + 8], v[CT][VT + 8];
+  bf16 s_big[DK][VT + 8], s_rest[DK][VT + 8];
+  float pw[CT + 1];
+  int count;
+};
+
+template <int DK>
+__global__ void __launch_bounds__(THREADS, 2)
+decayed_chunks_kernel(const bf16* __restrict__ qkv, const float* __restrict__ decay, float* __restrict__ state, const int* __restrict__ positions,
+                      const int* __restrict__ row_ids, int S_len, int H, int dk, int dv, int act, bf16* __restrict__ out) {
+  using namespace mma16;
+  extern __shared__ __align__(16) uint8_t raw[];
+  ChunkSmem<DK>& sm = *reinterpret_cast<ChunkSmem<DK>*>(raw);
+  constexpr int MT = DK / 16;                      // 16-row tiles of the state: 8 (a warp each, all columns) or 4 (two warps each, half the columns)
+  constexpr int NT = MT;                           // 8-column tiles of the state a warp owns
+  constexpr int QV = DK / 8 * CT / THREADS, VV = VT / 8 * CT / THREADS;
+  const int h = blockIdx.x, row = blockIdx.z, c0 = blockIdx.y * VT;
+  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+  const int* pos = positions + static_cast<long long>(row) * S_len;
+  const long long width = static_cast<long long>(H) * (2 * dk + dv);
+  const bf16* base = qkv + static_cast<long long>(row) * S_len * width;
+  bf16* o = out + (static_cast<long long>(row) * S_len * H + h) * dv;
+  const float a = decay[h];
+  if (tid == 0) sm.count = 0;
+  for (int i = tid; i <= CT; i += THREADS) sm.pw[i] = powf(a, static_cast<float>(i));
+  __syncthreads();
+  {
+    int live = 0;
+    for (int i = tid; i < S_len; i += THREADS) live += pos[i] >= 0;
+#pragma unroll
+    for (int s = 16; s > 0; s >>= 1) live += __shfl_xor_sync(0xffffffffu, live, s);
+    if (lane == 0) atomicAdd(&sm.count, live);
+  }
+  __syncthreads();
+  const int len = sm.count;                        // positions below 0 come last
+  const int r = row_ids == nullptr ? row : row_ids[row];
+  float* S = state == nullptr ? nullptr : state + (static_cast<long long>(r) * H + h) * dk * dv;
+  const int g = lane >> 2, t2 = (lane & 3) * 2;
+  // this warp's part of the state: rows sm_row + {g, g + 8}, columns s_col + 8 n + t2 + {0, 1}
+  const int s_row = (MT == 8 ? warp : warp & 3) * 16, s_col = MT == 8 ? 0 : (warp >> 2) * 32;
+  float st_acc[NT][4];
+  const bool load_state = S != nullptr && len > 0 && pos[0] > 0;
+#pragma unroll
+  for (int n = 0; n < NT; ++n)
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      const int kr = s_row + g + (e >> 1) * 8, vc = c0 + s_col + n * 8 + t2 + (e & 1);
+      st_acc[n][e] = (load_state && kr < dk && vc < dv) ? S[static_cast<long long>(kr) * dv + vc] : 0.f;
+    }
+  // output tile of this warp: tokens o_row + {g, g + 8}, columns o_col + ...
+  const int o_row = (warp & 3) * 16, o_col = (warp >> 2) * 32;
+  uint4 rq[QV], rk[QV], rv[VV];
+  const uint4 zero = make_uint4(0, 0, 0, 0);
+  auto fetch = [&](int t0) {
+#pragma unroll
+    for (int i = 0; i < QV; ++i) {
+      const int x = tid + i * THREADS, t = x / (DK / 8), c = (x % (DK / 8)) * 8;
+      const bool ok = t0 + t < len && c < dk;
+      const bf16* p = base + (t0 + t) * width + h * dk + c;
+      rq[i] = ok ? *reinterpret_cast<const uint4*>(p) : zero;
+      rk[i] = ok ? *reinterpret_cast<const uint4*>(p + H * dk) : zero;
+    }
+#pragma unroll
+    for (int i = 0; i < VV; ++i) {
+      const int x = tid + i * THREADS, t = x / (VT / 8), c = (x % (VT / 8)) * 8;
+      rv[i] = t0 + t < len && c0 + c < dv ? *reinterpret_cast<const uint4*>(base + (t0 + t) * width + 2 * H * dk + h * dv + c0 + c) : zero;
+    }
+  };
+  auto put = [&](bf16* dst, uint4 x) {
+    if (act) {
+      uint32_t w[4] = {x.x, x.y, x.z, x.w};
+#pragma unroll
+      for (int j = 0; j < 4; ++j) {
+        const float f0 = lo_f(w[j]), f1 = hi_f(w[j]);
+        w[j] = pack2(__fdividef(f0, 1.f + __expf(-f0)), __fdividef(f1, 1.f + __expf(-f1)));
+      }
+      x = make_uint4(w[0], w[1], w[2], w[3]);
+    }
+    *reinterpret_cast<uint4*>(dst) = x;
+  };
+  fetch(0);
+  for (int t0 = 0; t0 < len; t0 += CT) {
+    const int n = min(CT, len - t0);
+    __syncthreads();                               // the chunk before has been read
+#pragma unroll
+    for (int i = 0; i < QV; ++i) {
+      const int x = tid + i * THREADS, t = x / (DK / 8), c = (x % (DK / 8)) * 8;
+      put(&sm.q[t][c], rq[i]);
+      put(&sm.k[t][c], rk[i]);
+    }
+#pragma unroll
+    for (int i = 0; i < VV; ++i) {
+      const int x = tid + i * THREADS, t = x / (VT / 8), c = (x % (VT / 8)) * 8;
+      put(&sm.v[t][c], rv[i]);
+    }
+#pragma unroll
+    for (int j = 0; j < NT; ++j)
+#pragma unroll
+      for (int e = 0; e < 2; ++e) {
+        uint32_t big, rest;
+        split2(st_acc[j][2 * e], st_acc[j][2 * e + 1], big, rest);
+        *reinterpret_cast<uint32_t*>(&sm.s_big[s_row + g + 8 * e][s_col + j * 8 + t2]) = big;
+        *reinterpret_cast<uint32_t*>(&sm.s_rest[s_row + g + 8 * e][s_col + j * 8 + t2]) = rest;
+      }
+    __syncthreads();
+    if (t0 + CT < len) fetch(t0 + CT);
+    // ---- from the state: Q S
+    float acc[4][4];
+#pragma unroll
+    for (int j = 0; j < 4; ++j) { acc[j][0] = acc[j][1] = acc[j][2] = acc[j][3] = 0.f; }
+#pragma unroll
+    for (int kk = 0; kk < DK; kk += 16) {
+      uint32_t qa[4];
+      ldsm4(qa, smem_addr(&sm.q[o_row + (lane & 15)][kk + (lane >> 4) * 8]));
+#pragma unroll
+      for (int j = 0; j < 2; ++j) {
+        uint32_t b[4], d[4];
+        ldsm4_t(b, smem_addr(&sm.s_big[kk + (lane & 15)][o_col + j * 16 + (lane >> 4) * 8]));
+        ldsm4_t(d, smem_addr(&sm.s_rest[kk + (lane & 15)][o_col + j * 16 + (lane >> 4) * 8]));
+        mma(acc[2 * j], qa, b[0], b[1]);
+        mma(acc[2 * j + 1], qa, b[2], b[3]);
+        mma(acc[2 * j], qa, d[0], d[1]);
+        mma(acc[2 * j + 1], qa, d[2], d[3]);
+      }
+    }
+    const float w0 = sm.pw[o_row + g + 1], w1 = sm.pw[o_row + g + 9];
+#pragma unroll
+    for (int j = 0; j < 4; ++j) { acc[j][0] *= w0; acc[j][1] *= w0; acc[j][2] *= w1; acc[j][3] *= w1; }
+    // ---- from the chunk: 16 tokens at a time, up to this warp's diagonal tile
+#pragma unroll 1
+    for (int j = 0; j <= (warp & 3); ++j) {
+      float sc[2][4] = {{0.f, 0.f, 0.f, 0.f}, {0.f, 0.f, 0.f, 0.f}};
+#pragma unroll
+      for (int kk = 0; kk < DK; kk += 16) {
+        uint32_t qa[4], b[4];
+        ldsm4(qa, smem_addr(&sm.q[o_row + (lane & 15)][kk + (lane >> 4) * 8]));
+        ldsm4(b, smem_addr(&sm.k[j * 16 + (lane & 7) + (lane >> 4) * 8][kk + ((lane >> 3) & 1) * 8]));
+        mma(sc[0], qa, b[0], b[1]);
+        mma(sc[1], qa, b[2], b[3]);
+      }
+      uint32_t pa[4], pr[4];
+#pragma unroll
+      for (int half = 0; half < 2; ++half)
+#pragma unroll
+        for (int e = 0; e < 2; ++e) {
+          const int i = o_row + g + 8 * e, c = j * 16 + half * 8 + t2;
+          const float x0 = c <= i ? sc[half][2 * e] * sm.pw[max(i - c, 0)] : 0.f;
+          const float x1 = c + 1 <= i ? sc[half][2 * e + 1] * sm.pw[max(i - c - 1, 0)] : 0.f;
+          split2(x0, x1, pa[half * 2 + e], pr[half * 2 + e]);
+        }
+#pragma unroll
+      for (int m = 0; m < 2; ++m) {
+        uint32_t b[4];
+        ldsm4_t(b, smem_addr(&sm.v[j * 16 + (lane & 15)][o_col + m * 16 + (lane >> 4) * 8]));
+        mma(acc[2 * m], pa, b[0], b[1]);
+        mma(acc[2 * m + 1], pa, b[2], b[3]);
+        mma(acc[2 * m], pr, b[0], b[1]);
+        mma(acc[2 * m + 1], pr, b[2], b[3]);
+      }
+    }
+#pragma unroll
+    for (int j = 0; j < 4; ++j)
+#pragma unroll
+      for (int e = 0; e < 2; ++e) {
+        const int t = o_row + g + 8 * e, c = c0 + o_col + j * 8 + t2;
+        if (t < n && c < dv) *reinterpret_cast<uint32_t*>(o + (t0 + t) * static_cast<long long>(H) * dv + c) = pack2(acc[j][2 * e], acc[j][2 * e + 1]);
+      }
+    // ---- the state after the chunk
+    const float wn = sm.pw[n];
+#pragma unroll
+    for (int j = 0; j < NT; ++j) { st_acc[j][0] *= wn; st_acc[j][1] *= wn; st_acc[j][2] *= wn; st_acc[j][3] *= wn; }
+#pragma unroll
+    for (int kt = 0; kt < CT; kt += 16) {
+      if (kt < n) {
+        uint32_t ka[4], big[4], rest[4];
+        // A = K^T: rows are key components, the reduction runs over tokens
+        ldsm4_t(ka, smem_addr(&sm.k[kt + (lane & 7) + (lane >> 4) * 8][s_row + ((lane >> 3) & 1) * 8]));
+#pragma unroll
+        for (int x = 0; x < 4; ++x) {
+          const int tk = kt + (x >> 1) * 8 + t2;   // tokens past the end carry zero keys
+          split2(lo_f(ka[x]) * sm.pw[max(n - 1 - tk, 0)], hi_f(ka[x]) * sm.pw[max(n - 2 - tk, 0)], big[x], rest[x]);
+        }
+#pragma unroll
+        for (int m = 0; m < NT / 2; ++m) {
+          uint32_t b[4];
+          ldsm4_t(b, smem_addr(&sm.v[kt + (lane & 15)][s_col + m * 16 + (lane >> 4) * 8]));
+          mma(st_acc[2 * m], big, b[0], b[1]);
+          mma(st_acc[2 * m + 1], big, b[2], b[3]);
+          mma(st_acc[2 * m], rest, b[0], b[1]);
+          mma(st_acc[2 * m + 1], rest, b[2], b[3]);
+        }
+      }
+    }
+  }
+  if (S != nullptr && len > 0) {
+#pragma unroll
+    for (int n = 0; n < NT; ++n)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        const int kr = s_row + g + (e >> 1) * 8, vc = c0 + s_col + n * 8 + t2 + (e & 1);
+        if (kr < dk && vc < dv) S[static_cast<long long>(kr) * dv + vc] = st_acc[n][e];
+      }
+  }
+  for (int i = tid; i < (S_len - len) * (VT / 8); i += THREADS) {
+    const int t = len + i / (VT / 8), c = c0 + (i % (VT / 8)) * 8;
+    if (c < dv) *reinterpret_cast<uint4*>(o + t * static_cast<long long>(H) * dv + c) = zero;
+  }
+}
+
 template <typename T, int V, int LANES>
 int step_go(const T* qkv, const float* decay, float* state, const int* positions, const int* row_ids, int R, int H, int dk, int dv, int act, T* out,
             cudaStream_t stream) {
@@ -218,6 +439,16 @@ int seq_any(const T* qkv, const float* decay, float* state, const int* positions
   return -3;
 }
 
+template <int DK>
+int chunks_go(const bf16* qkv, const float* decay, float* state, const int* positions, const int* row_ids, int R, int S, int H, int dk, int dv, int act,
+              bf16* out, cudaStream_t stream) {
+  const int smem = static_cast<int>(sizeof(ChunkSmem<DK>));
+  cudaError_t e = cudaFuncSetAttribute(decayed_chunks_kernel<DK>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
+  if (e != cudaSuccess) return static_cast<int>(e);
+  decayed_chunks_kernel<DK><<<dim3(H, (dv + VT - 1) / VT, R), THREADS, smem, stream>>>(qkv, decay, state, positions, row_ids, S, H, dk, dv, act, out);
+  return static_cast<int>(cudaGetLastError());
+}
+
 }  // namespace decayed
 }  // namespace dewb
 
@@ -241,4 +472,15 @@ extern "C" int dewb_decayed_sequence(const void* qkv, const float* decay, float*
   cudaStream_t stream = reinterpret_cast<cudaStream_t>(stream_ptr);
   if (fp32) return seq_any<float>(static_cast<const float*>(qkv), decay, state, positions, row_ids, R, S, H, dk, dv, act, static_cast<float*>(out), stream);
   return seq_any<bf16>(static_cast<const bf16*>(qkv), decay, state, positions, row_ids, R, S, H, dk, dv, act, static_cast<bf16*>(out), stream);
+}
+
+// The chunked tensor-core form of the same (bf16; dk, dv multiples of 8, dk at most 128; qkv and out on 16-byte boundaries).
+extern "C" int dewb_decayed_chunks(const void* qkv, const float* decay, float* state, const int* positions, const int* row_ids, int R, int S, int H,
+                                   int dk, int dv, int act, void* out, void* stream_ptr) {
+  if (R <= 0 || S <= 0) return 0;
+  if (H < 1 || dk < 8 || dv < 8 || dk % 8 || dv % 8 || dk > 128 || (reinterpret_cast<uintptr_t>(qkv) & 15) || (reinterpret_cast<uintptr_t>(out) & 15)) return -3;
+  cudaStream_t stream = reinterpret_cast<cudaStream_t>(stream_ptr);
+  const bf16* x = static_cast<const bf16*>(qkv);
+  if (dk <= 64) return chunks_go<64>(x, decay, state, positions, row_ids, R, S, H, dk, dv, act, static_cast<bf16*>(out), stream);
+  return chunks_go<128>(x, decay, state, positions, row_ids, R, S, H, dk, dv, act, static_cast<bf16*>(out), stream);
 }

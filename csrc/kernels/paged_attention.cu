@@ -6,12 +6,15 @@
 //   paged_attend     causal attention of a call's tokens against everything the cache holds of their rows (any start positions; a decode
 //                    step is the case of one token per row); scores, softmax and sums in fp32 on the CUDA cores.  It is the fp32 form,
 //                    and takes the head widths the tensor-core kernels do not.
+//   paged_attend_mma   the same on the tensor cores for bf16 pools 64, 128 or 256 wide (a prompt's later portions, mixed start positions)
 //
 // A query's row of work is (token, head of its group), so a group's heads share the key and value tiles.  Positions below 0 are padding:
 // nothing is appended for them and their outputs are zero.  Compiled without fast math.
 #include <cstdint>
 #include <cuda_bf16.h>
 #include <cuda_runtime.h>
+
+#include "../common/mma_bf16.cuh"
 
 namespace dewb {
 namespace paged {
@@ -244,6 +247,163 @@ paged_attend_kernel(const T* __restrict__ q, long long q_token_stride, const T* 
     }
 }
 
+// ---- tensor-core form: 64 rows of work a CTA (4 warps of 16), key / value tiles of 64 through a two-stage cp.async ring, online softmax in
+// the log2 domain with fp32 scores and sums, probabilities in bf16 for the value product.
+constexpr int MQ = 64, MK = 64, MTHREADS = 128;
+
+__device__ __forceinline__ void cp16(uint32_t dst, const void* src, bool live) {
+  const int n = live ? 16 : 0;                     // 0: the 16 bytes are filled with zeros
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst), "l"(src), "r"(n) : "memory");
+}
+
+template <int D>
+__global__ void __launch_bounds__(MTHREADS)
+paged_attend_mma_kernel(const bf16* __restrict__ q, long long q_token_stride, const bf16* __restrict__ kpool, const bf16* __restrict__ vpool,
+                        const int* __restrict__ positions, int S, int H, int G, int dv, float scale_log2, bf16* __restrict__ out, Pool pool) {
+  using namespace mma16;
+  constexpr int ST = D + 8;                        // smem row stride
+  extern __shared__ __align__(16) uint8_t raw[];
+  bf16* sq = reinterpret_cast<bf16*>(raw);         // [MQ][ST]
+  bf16* sk = sq + MQ * ST;                         // [2][MK][ST]
+  bf16* sv = sk + 2 * MK * ST;                     // [2][MK][ST]
+  __shared__ int s_pos[MQ];
+  const int row = blockIdx.z, g = blockIdx.y, Gq = H / G;
+  const int r0 = blockIdx.x * MQ, rows = S * Gq;
+  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+  if (tid < MQ) {
+    const int r = r0 + tid;
+    s_pos[tid] = r < rows ? positions[static_cast<long long>(row) * S + r / Gq] : -1;
+  }
+  __syncthreads();
+  int last = -1;
+  for (int i = 0; i < MQ; ++i) last = max(last, s_pos[i]);
+  const int tiles = (last + MK) / MK;              // key tiles [0, last]
+  for (int i = tid; i < MQ * (D / 8); i += MTHREADS) {
+    const int r = i / (D / 8), c = (i % (D / 8)) * 8, gr = r0 + r;
+    const bool live = s_pos[r] >= 0;
+    const bf16* src = live ? q + (static_cast<long long>(row) * S + gr / Gq) * q_token_stride + static_cast<long long>(g * Gq + gr % Gq) * D + c : q;
+    cp16(smem_addr(sq + r * ST + c), src, live);
+  }
+  auto fetch = [&](int t) {
+    bf16* dk_ = sk + (t & 1) * MK * ST;
+    bf16* dv_ = sv + (t & 1) * MK * ST;
+    for (int i = tid; i < MK * (D / 8); i += MTHREADS) {
+      const int r = i / (D / 8), c = (i % (D / 8)) * 8, key = t * MK + r;
+      const bool live = key <= last;
+      const long long off = live ? (pool_token(pool, row, key) * G + g) * D + c : 0;
+      cp16(smem_addr(dk_ + r * ST + c), kpool + off, live);
+      cp16(smem_addr(dv_ + r * ST + c), vpool + off, live);
+    }
+    asm volatile("cp.async.commit_group;" ::: "memory");
+  };
+  const int lg = lane >> 2, t2 = (lane & 3) * 2;
+  const int p0 = s_pos[warp * 16 + lg], p1 = s_pos[warp * 16 + lg + 8];
+  float m0 = -INFINITY, m1 = -INFINITY, l0 = 0.f, l1 = 0.f, o[D / 8][4];
+#pragma unroll
+  for (int j = 0; j < D / 8; ++j) { o[j][0] = o[j][1] = o[j][2] = o[j][3] = 0.f; }
+  if (tiles > 0) fetch(0);
+  for (int t = 0; t < tiles; ++t) {
+    if (t + 1 < tiles) {
+      fetch(t + 1);
+      asm volatile("cp.async.wait_group 1;" ::: "memory");
+    } else {
+      asm volatile("cp.async.wait_group 0;" ::: "memory");
+    }
+    __syncthreads();
+    const bf16* tk = sk + (t & 1) * MK * ST;
+    const bf16* tv = sv + (t & 1) * MK * ST;
+    float s[8][4];
+#pragma unroll
+    for (int j = 0; j < 8; ++j) { s[j][0] = s[j][1] = s[j][2] = s[j][3] = 0.f; }
+#pragma unroll
+    for (int kk = 0; kk < D; kk += 16) {
+      uint32_t a[4];
+      ldsm4(a, smem_addr(sq + (warp * 16 + (lane & 15)) * ST + kk + (lane >> 4) * 8));
+#pragma unroll
+      for (int j = 0; j < 4; ++j) {
+        uint32_t b[4];
+        ldsm4(b, smem_addr(tk + (j * 16 + (lane & 7) + (lane >> 4) * 8) * ST + kk + ((lane >> 3) & 1) * 8));
+        mma(s[2 * j], a, b[0], b[1]);
+        mma(s[2 * j + 1], a, b[2], b[3]);
+      }
+    }
+    float x0 = -INFINITY, x1 = -INFINITY;
+#pragma unroll
+    for (int j = 0; j < 8; ++j) {
+      const int key = t * MK + j * 8 + t2;
+      s[j][0] = key <= p0 ? s[j][0] * scale_log2 : -INFINITY;
+      s[j][1] = key + 1 <= p0 ? s[j][1] * scale_log2 : -INFINITY;
+      s[j][2] = key <= p1 ? s[j][2] * scale_log2 : -INFINITY;
+      s[j][3] = key + 1 <= p1 ? s[j][3] * scale_log2 : -INFINITY;
+      x0 = fmaxf(x0, fmaxf(s[j][0], s[j][1]));
+      x1 = fmaxf(x1, fmaxf(s[j][2], s[j][3]));
+    }
+#pragma unroll
+    for (int d = 1; d < 4; d <<= 1) {
+      x0 = fmaxf(x0, __shfl_xor_sync(0xffffffffu, x0, d));
+      x1 = fmaxf(x1, __shfl_xor_sync(0xffffffffu, x1, d));
+    }
+    const float n0 = fmaxf(m0, x0), n1 = fmaxf(m1, x1);
+    const float b0 = n0 == -INFINITY ? 0.f : n0, b1 = n1 == -INFINITY ? 0.f : n1;      // a row that has seen nothing yet
+    const float f0 = exp2f(m0 - b0), f1 = exp2f(m1 - b1);
+    m0 = n0; m1 = n1;
+    l0 *= f0; l1 *= f1;
+#pragma unroll
+    for (int j = 0; j < D / 8; ++j) { o[j][0] *= f0; o[j][1] *= f0; o[j][2] *= f1; o[j][3] *= f1; }
+#pragma unroll
+    for (int j = 0; j < 8; ++j) {
+      s[j][0] = exp2f(s[j][0] - b0); s[j][1] = exp2f(s[j][1] - b0);
+      s[j][2] = exp2f(s[j][2] - b1); s[j][3] = exp2f(s[j][3] - b1);
+      l0 += s[j][0] + s[j][1];
+      l1 += s[j][2] + s[j][3];
+    }
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+      const uint32_t a[4] = {pack2(s[2 * j][0], s[2 * j][1]), pack2(s[2 * j][2], s[2 * j][3]), pack2(s[2 * j + 1][0], s[2 * j + 1][1]),
+                             pack2(s[2 * j + 1][2], s[2 * j + 1][3])};
+#pragma unroll
+      for (int n = 0; n < D / 16; ++n) {
+        uint32_t b[4];
+        ldsm4_t(b, smem_addr(tv + (j * 16 + (lane & 15)) * ST + n * 16 + (lane >> 4) * 8));
+        mma(o[2 * n], a, b[0], b[1]);
+        mma(o[2 * n + 1], a, b[2], b[3]);
+      }
+    }
+    __syncthreads();                               // the tile's stage is refilled two tiles on
+  }
+#pragma unroll
+  for (int d = 1; d < 4; d <<= 1) {
+    l0 += __shfl_xor_sync(0xffffffffu, l0, d);
+    l1 += __shfl_xor_sync(0xffffffffu, l1, d);
+  }
+  const float i0 = l0 > 0.f ? 1.f / l0 : 0.f, i1 = l1 > 0.f ? 1.f / l1 : 0.f;
+#pragma unroll
+  for (int e = 0; e < 2; ++e) {
+    const int gr = r0 + warp * 16 + lg + 8 * e;
+    if (gr >= rows) continue;
+    const float inv = e ? i1 : i0;
+    bf16* dst = out + ((static_cast<long long>(row) * S + gr / Gq) * H + g * Gq + gr % Gq) * dv;
+#pragma unroll
+    for (int j = 0; j < D / 8; ++j) {
+      const int c = j * 8 + t2;
+      if (c < dv) dst[c] = __float2bfloat16(o[j][2 * e] * inv);
+      if (c + 1 < dv) dst[c + 1] = __float2bfloat16(o[j][2 * e + 1] * inv);
+    }
+  }
+}
+
+template <int D>
+int attend_mma(const bf16* q, long long qs, const bf16* kpool, const bf16* vpool, const int* positions, int R, int S, int H, int G, int dv, float scale,
+               bf16* out, const Pool& pool, cudaStream_t stream) {
+  const int smem = (MQ + 4 * MK) * (D + 8) * 2;
+  cudaError_t e = cudaFuncSetAttribute(paged_attend_mma_kernel<D>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
+  if (e != cudaSuccess) return static_cast<int>(e);
+  const long long tiles = (static_cast<long long>(S) * (H / G) + MQ - 1) / MQ;
+  paged_attend_mma_kernel<D><<<dim3(static_cast<unsigned>(tiles), G, R), MTHREADS, smem, stream>>>(q, qs, kpool, vpool, positions, S, H, G, dv,
+                                                                                              scale * 1.4426950408889634f, out, pool);
+  return static_cast<int>(cudaGetLastError());
+}
+
 inline bool aligned(const void* p, size_t a) { return (reinterpret_cast<uintptr_t>(p) & (a - 1)) == 0; }
 
 template <typename T, int NJ>
@@ -308,4 +468,22 @@ extern "C" int dewb_paged_attend(const void* q, long long q_token_stride, const 
   const Pool pool{page_table, page_size, max_pages, row_ids};
   if (fp32) return attend_any<float>(q, q_token_stride, kpool, vpool, positions, R, S, H, G, dk, dv, D, scale, out, pool, stream);
   return attend_any<bf16>(q, q_token_stride, kpool, vpool, positions, R, S, H, G, dk, dv, D, scale, out, pool, stream);
+}
+
+// The tensor-core form (bf16; pools D = 64, 128 or 256 wide; q on 16-byte boundaries with a token stride of a multiple of 8).
+extern "C" int dewb_paged_attend_mma(const void* q, long long q_token_stride, const void* kpool, const void* vpool, const int* positions, int R, int S,
+                                     int H, int G, int dv, int D, float scale, void* out, const int* page_table, int page_size, int max_pages,
+                                     const int* row_ids, void* stream_ptr) {
+  if (R <= 0 || S <= 0) return 0;
+  if (H < 1 || G < 1 || H % G || dv < 1 || D < dv || page_size < 1 || max_pages < 1 || q_token_stride % 8 || !aligned(q, 16) || !aligned(kpool, 16) ||
+      !aligned(vpool, 16))
+    return -3;
+  cudaStream_t stream = reinterpret_cast<cudaStream_t>(stream_ptr);
+  const Pool pool{page_table, page_size, max_pages, row_ids};
+  const bf16 *qp = static_cast<const bf16*>(q), *kp = static_cast<const bf16*>(kpool), *vp = static_cast<const bf16*>(vpool);
+  bf16* op = static_cast<bf16*>(out);
+  if (D == 64) return attend_mma<64>(qp, q_token_stride, kp, vp, positions, R, S, H, G, dv, scale, op, pool, stream);
+  if (D == 128) return attend_mma<128>(qp, q_token_stride, kp, vp, positions, R, S, H, G, dv, scale, op, pool, stream);
+  if (D == 256) return attend_mma<256>(qp, q_token_stride, kp, vp, positions, R, S, H, G, dv, scale, op, pool, stream);
+  return -3;
 }

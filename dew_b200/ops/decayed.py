@@ -40,9 +40,14 @@ def decayed_attention_reference(qkv, decay, H: int, dk: int, dv: int, state=None
     return torch.stack(outs, 1).to(qkv.dtype)
 
 
+def chunks_ok(qkv: torch.Tensor, dk: int, dv: int) -> bool:
+    return qkv.dtype == torch.bfloat16 and dk % 8 == 0 and dv % 8 == 0 and 8 <= dk <= 128 and qkv.data_ptr() % 16 == 0
+
+
 def decayed_attention(qkv: torch.Tensor, decay: torch.Tensor, H: int, dk: int, dv: int, state: Optional[torch.Tensor] = None,
-                      positions: Optional[torch.Tensor] = None, row_ids: Optional[torch.Tensor] = None, silu: bool = True) -> torch.Tensor:
-    """``qkv [R, S, H (2 dk + dv)] -> [R, S, H, dv]``.  ``positions`` int32 ``[R, S]``, ``row_ids`` int32 (call row -> store row)."""
+                      positions: Optional[torch.Tensor] = None, row_ids: Optional[torch.Tensor] = None, silu: bool = True, kernel: Optional[str] = None) -> torch.Tensor:
+    """``qkv [R, S, H (2 dk + dv)] -> [R, S, H, dv]``.  ``positions`` int32 ``[R, S]``, ``row_ids`` int32 (call row -> store row).
+    ``kernel`` forces ``chunks`` (tensor cores, bf16) or ``sequence`` (fp32 arithmetic, any widths) for a call of several tokens."""
     R, S, _ = qkv.shape
     if not L.use_cuda(qkv) or qkv.dtype not in (torch.bfloat16, torch.float32):
         return decayed_attention_reference(qkv, decay, H, dk, dv, state, positions, row_ids, silu)
@@ -57,6 +62,9 @@ def decayed_attention(qkv: torch.Tensor, decay: torch.Tensor, H: int, dk: int, d
     if S == 1 and state is not None:
         L.check(lib.dewb_decayed_step(L.ptr(qkv), L.ptr(decay), L.ptr(state), L.ptr(pos), L.ptr(rows), c_int(R), c_int(H), c_int(dk), c_int(dv),
                                       c_int(int(silu)), L.ptr(out), fp32, L.stream_ptr()), "decayed_step")
+    elif (kernel or ("chunks" if chunks_ok(qkv, dk, dv) else "sequence")) == "chunks":
+        L.check(lib.dewb_decayed_chunks(L.ptr(qkv), L.ptr(decay), L.ptr(state), L.ptr(pos), L.ptr(rows), c_int(R), c_int(S), c_int(H), c_int(dk),
+                                        c_int(dv), c_int(int(silu)), L.ptr(out), L.stream_ptr()), "decayed_chunks")
     else:
         L.check(lib.dewb_decayed_sequence(L.ptr(qkv), L.ptr(decay), L.ptr(state), L.ptr(pos), L.ptr(rows), c_int(R), c_int(S), c_int(H), c_int(dk),
                                           c_int(dv), c_int(int(silu)), L.ptr(out), fp32, L.stream_ptr()), "decayed_sequence")

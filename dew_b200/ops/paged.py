@@ -105,14 +105,21 @@ def paged_attend_reference(q, heads: Heads, positions, pages: Pages, scale: floa
     return torch.einsum("rhsn,rnhd->rshd", p, vc).to(q.dtype)
 
 
-def paged_attend(q: torch.Tensor, heads: Heads, positions: torch.Tensor, pages: Pages, scale: float) -> torch.Tensor:
-    """``q [R, S, H, D]`` (a view into the packed tensor will do: unit stride in a head, heads next to each other) -> ``[R, S, H, dv]``."""
+def paged_attend(q: torch.Tensor, heads: Heads, positions: torch.Tensor, pages: Pages, scale: float, kernel: Optional[str] = None) -> torch.Tensor:
+    """``q [R, S, H, D]`` (a view into the packed tensor will do: unit stride in a head, heads next to each other) -> ``[R, S, H, dv]``.
+    ``kernel`` forces ``mma`` (bf16 pools of 64, 128, 256) or ``general``."""
     if not L.use_cuda(q):
         return paged_attend_reference(q, heads, positions, pages, scale)
     R, S, H, D = q.shape
     if q.stride(3) != 1 or q.stride(2) != D or (R > 1 and q.stride(0) != S * q.stride(1)):
         q = q.contiguous()
     out = torch.empty(R, S, H, heads.dv, dtype=q.dtype, device=q.device)
+    if (kernel or ("mma" if q.dtype == torch.bfloat16 and D in (64, 128, 256) else "general")) == "mma":
+        L.check(L.load().dewb_paged_attend_mma(L.ptr(q), c_ll(q.stride(1)), L.ptr(pages.k), L.ptr(pages.v), L.ptr(positions), c_int(R), c_int(S), c_int(H),
+                                               c_int(heads.kv), c_int(heads.dv), c_int(D), c_float(scale), L.ptr(out), L.ptr(pages.table),
+                                               c_int(pages.page_size), c_int(pages.table.shape[1]), L.ptr(pages.row_ids), L.stream_ptr()), "paged_attend_mma")
+        L.count_launches()
+        return out
     L.check(L.load().dewb_paged_attend(L.ptr(q), c_ll(q.stride(1)), L.ptr(pages.k), L.ptr(pages.v), L.ptr(positions), c_int(R), c_int(S), c_int(H),
                                        c_int(heads.kv), c_int(heads.dk), c_int(heads.dv), c_int(D), c_float(scale), L.ptr(out), L.ptr(pages.table),
                                        c_int(pages.page_size), c_int(pages.table.shape[1]), L.ptr(pages.row_ids),
