@@ -166,10 +166,22 @@ def main() -> None:
     ap.add_argument("--others", default="auto", choices=["auto", "none"],
                     help="auto: the default (dense) run also times 3 steps of the moe and hybrid configurations in child processes "
                          "and reports them under `others`")
+    ap.add_argument("--decoder", default=None, choices=["ragenex"],
+                    help="instead of the training benchmark: prefill and decode throughput of this decoder design beside the closest existing model of equal "
+                         "size, and its kernels beside theirs (dew_b200/telemetry/decoder_bench.py)")
     ap.add_argument("--compile", action="store_true", help="torch_nccl arm only: torch.compile each decoder layer")
     args = ap.parse_args()
     if args.impl == "reference":
         return reference_arm(args)
+    if args.decoder is not None:
+        from dew_b200.ops import library as L
+        from dew_b200.telemetry import decoder_bench
+        sampler = ClockSampler(0)
+        sampler.start()
+        out = decoder_bench.run()
+        L.check_status()
+        print(json.dumps({"metric": f"prefill and decode tokens/sec ({args.decoder})", "n_gpus": 1, **out, "clocks": sampler.stop()}))
+        return
     if args.impl == "torch_nccl":
         # the library arm: stock PyTorch modules / cuBLAS / cuDNN SDPA / FSDP2 over NCCL, none of this framework's code
         sys.path.insert(0, os.path.join(os.path.dirname(os.path.abspath(__file__)), "baseline"))

@@ -11,7 +11,6 @@ from dew_b200.ops import decayed, paged, streams
 
 pytestmark = pytest.mark.gpu
 DEV = "cuda"
-TOL = {torch.float32: 2e-4, torch.bfloat16: 6e-2}
 
 
 def rnd(*shape, seed=0, dtype=torch.float32):
@@ -19,6 +18,8 @@ def rnd(*shape, seed=0, dtype=torch.float32):
 
 
 def close(got, want, rel):
+    if got.numel() == 0:
+        return got.shape == want.shape
     return float((got.float() - want.float()).abs().max()) <= rel * float(want.float().abs().max().clamp_min(1e-6))
 
 
@@ -99,7 +100,7 @@ HEADS = [paged.Heads(4, 1, 96, 96), paged.Heads(8, 2, 64, 64), paged.Heads(6, 2,
 @pytest.mark.parametrize("heads", HEADS)
 def test_attention_from_the_packed_projection(dtype, heads):
     """``attend_slot``: a prompt, a portion after it at mixed positions, and decode steps with a planted key at page borders and far back."""
-    rel = 2e-5 if dtype == torch.float32 else 2e-2
+    rel = 2e-5 if dtype == torch.float32 else 6e-2      # bf16 queries and keys under sharp scores; a missed key is past 0.2
     H, G, dk, dv = heads
     rows, first, T = 3, 128, 300
     kw = dict(scale=dk ** -0.5, eps=1e-3, q_weight=rnd(H * dk, seed=1, dtype=dtype), k_weight=rnd(G * dk, seed=2, dtype=dtype), temperature=(0.3, 16))
@@ -165,9 +166,11 @@ def test_model_on_every_schedule(tmp_path, name, dtype):
     cfg, w, m = C.load(tmp_path, name, dtype, DEV)
     tokens = C.prompt(cfg, 150)
     want, _ = O.run(cfg, w, tokens)
-    tol = TOL[dtype]
-    if name == "looped" and dtype == torch.bfloat16:
-        tol = 0.2                                                      # a head whose decay is 0 normalises single products of rounded numbers
+    tol = 2e-4
+    if dtype == torch.bfloat16:
+        # what rounding alone costs this model: the plain PyTorch forms in bf16 on the CPU (sharp attention and small normalised vectors
+        # amplify it differently from model to model)
+        tol = 0.03 + 3 * C.error(C.load(tmp_path / "cpu", name, dtype)[2](torch.tensor([tokens]))[0], want)
     assert C.error(C.replay(m, [tokens]), want) < tol
     for size in (2, 50, 64, 65):
         assert C.error(C.replay(m, C.cut(tokens, size), pool_tokens=160), want) < tol, size
