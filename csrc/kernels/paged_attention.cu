@@ -15,63 +15,17 @@
 #include <cuda_runtime.h>
 
 #include "../common/mma_bf16.cuh"
+#include "../common/rows.cuh"
 
 namespace dewb {
 namespace paged {
 
-using bf16 = __nv_bfloat16;
+using namespace rows;
 
 __device__ __forceinline__ float ld(const float* p) { return *p; }
 __device__ __forceinline__ float ld(const bf16* p) { return __bfloat162float(*p); }
 __device__ __forceinline__ void st(float* p, float v) { *p = v; }
 __device__ __forceinline__ void st(bf16* p, float v) { *p = __float2bfloat16(v); }
-
-template <int V>
-__device__ __forceinline__ void load_v(const float* p, float (&f)[V]) {
-  if constexpr (V == 4) {
-    const float4 v = *reinterpret_cast<const float4*>(p);
-    f[0] = v.x; f[1] = v.y; f[2] = v.z; f[3] = v.w;
-  } else {
-    f[0] = *p;
-  }
-}
-template <int V>
-__device__ __forceinline__ void load_v(const bf16* p, float (&f)[V]) {
-  if constexpr (V == 4) {
-    const uint2 v = *reinterpret_cast<const uint2*>(p);
-    f[0] = __uint_as_float(v.x << 16); f[1] = __uint_as_float(v.x & 0xffff0000u);
-    f[2] = __uint_as_float(v.y << 16); f[3] = __uint_as_float(v.y & 0xffff0000u);
-  } else {
-    f[0] = __bfloat162float(*p);
-  }
-}
-template <int V>
-__device__ __forceinline__ void store_v(float* p, const float (&f)[V]) {
-  if constexpr (V == 4) *reinterpret_cast<float4*>(p) = make_float4(f[0], f[1], f[2], f[3]);
-  else *p = f[0];
-}
-template <int V>
-__device__ __forceinline__ void store_v(bf16* p, const float (&f)[V]) {
-  if constexpr (V == 4) {
-    __nv_bfloat162 a = __floats2bfloat162_rn(f[0], f[1]), b = __floats2bfloat162_rn(f[2], f[3]);
-    *reinterpret_cast<uint2*>(p) = make_uint2(*reinterpret_cast<uint32_t*>(&a), *reinterpret_cast<uint32_t*>(&b));
-  } else {
-    *p = __float2bfloat16(f[0]);
-  }
-}
-
-__device__ __forceinline__ float block_sum(float v, float* red) {
-#pragma unroll
-  for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
-  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nw = blockDim.x >> 5;
-  __syncthreads();
-  if (lane == 0) red[warp] = v;
-  __syncthreads();
-  float t = lane < nw ? red[lane] : 0.f;
-#pragma unroll
-  for (int o = 16; o > 0; o >>= 1) t += __shfl_xor_sync(0xffffffffu, t, o);
-  return t;
-}
 
 struct Pool {
   const int* table;       // [store rows, max_pages]
@@ -84,7 +38,7 @@ __device__ __forceinline__ long long pool_token(const Pool& p, int row, int pos)
   return static_cast<long long>(p.table[static_cast<long long>(r) * p.max_pages + pos / p.page_size]) * p.page_size + pos % p.page_size;
 }
 
-constexpr int PREP_THREADS = 256;
+constexpr int PREP_THREADS = 128;
 
 // grid (tokens, 3): part 0 the queries, 1 the keys, 2 the values.  `packed` [tokens, H + 2 G, D] receives all three; D >= dk, dv.
 template <typename T, int V>
@@ -404,8 +358,6 @@ int attend_mma(const bf16* q, long long qs, const bf16* kpool, const bf16* vpool
   return static_cast<int>(cudaGetLastError());
 }
 
-inline bool aligned(const void* p, size_t a) { return (reinterpret_cast<uintptr_t>(p) & (a - 1)) == 0; }
-
 template <typename T, int NJ>
 int attend(const T* q, long long qs, const T* kpool, const T* vpool, const int* positions, int R, int S, int H, int G, int dk, int dv, int D,
            float scale, T* out, const Pool& pool, cudaStream_t stream) {
@@ -454,7 +406,7 @@ extern "C" int dewb_qk_norm_append(const void* qkv, const void* qw, const void* 
     static_cast<const TT*>(kw), eps, coef, every, positions, S, H, G, dk, dv, D, static_cast<TT*>(packed), static_cast<TT*>(kpool), \
     static_cast<TT*>(vpool), pool)
   if (fp32) { if (vec) DEWB_PREP(float, 4); else DEWB_PREP(float, 1); }
-  else { if (vec) DEWB_PREP(bf16, 4); else DEWB_PREP(bf16, 1); }
+  else { if (vec && dk % 8 == 0 && dv % 8 == 0 && D % 8 == 0) DEWB_PREP(bf16, 8); else if (vec) DEWB_PREP(bf16, 4); else DEWB_PREP(bf16, 1); }
 #undef DEWB_PREP
   return static_cast<int>(cudaGetLastError());
 }

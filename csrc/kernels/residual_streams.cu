@@ -13,60 +13,14 @@
 #include <cuda_bf16.h>
 #include <cuda_runtime.h>
 
+#include "../common/rows.cuh"
+
 namespace dewb {
 namespace streams {
 
-using bf16 = __nv_bfloat16;
+using namespace rows;
 constexpr int MAX_STREAMS = 16;
 constexpr int THREADS = 256;
-
-// V consecutive values (V = 4 or 1) as fp32
-template <int V>
-__device__ __forceinline__ void load_v(const float* p, float (&f)[V]) {
-  if constexpr (V == 4) {
-    const float4 v = *reinterpret_cast<const float4*>(p);
-    f[0] = v.x; f[1] = v.y; f[2] = v.z; f[3] = v.w;
-  } else {
-    f[0] = *p;
-  }
-}
-template <int V>
-__device__ __forceinline__ void load_v(const bf16* p, float (&f)[V]) {
-  if constexpr (V == 4) {
-    const uint2 v = *reinterpret_cast<const uint2*>(p);
-    f[0] = __uint_as_float(v.x << 16); f[1] = __uint_as_float(v.x & 0xffff0000u);
-    f[2] = __uint_as_float(v.y << 16); f[3] = __uint_as_float(v.y & 0xffff0000u);
-  } else {
-    f[0] = __bfloat162float(*p);
-  }
-}
-template <int V>
-__device__ __forceinline__ void store_v(float* p, const float (&f)[V]) {
-  if constexpr (V == 4) *reinterpret_cast<float4*>(p) = make_float4(f[0], f[1], f[2], f[3]);
-  else *p = f[0];
-}
-template <int V>
-__device__ __forceinline__ void store_v(bf16* p, const float (&f)[V]) {
-  if constexpr (V == 4) {
-    __nv_bfloat162 a = __floats2bfloat162_rn(f[0], f[1]), b = __floats2bfloat162_rn(f[2], f[3]);
-    *reinterpret_cast<uint2*>(p) = make_uint2(*reinterpret_cast<uint32_t*>(&a), *reinterpret_cast<uint32_t*>(&b));
-  } else {
-    *p = __float2bfloat16(f[0]);
-  }
-}
-
-__device__ __forceinline__ float block_sum(float v, float* red) {
-#pragma unroll
-  for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
-  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nw = blockDim.x >> 5;
-  __syncthreads();
-  if (lane == 0) red[warp] = v;
-  __syncthreads();
-  float t = lane < nw ? red[lane] : 0.f;
-#pragma unroll
-  for (int o = 16; o > 0; o >>= 1) t += __shfl_xor_sync(0xffffffffu, t, o);
-  return t;
-}
 
 template <typename T, int V>
 __global__ void __launch_bounds__(THREADS)
@@ -175,24 +129,29 @@ stream_step_kernel(float* __restrict__ H, const T* __restrict__ y, const T* __re
   }
 }
 
+// x sigmoid(z) times a factor: fp32 models take the exact quotient, bf16 the approximate one (a few parts in 2^22)
+template <typename T>
+__device__ __forceinline__ float times_sigmoid(float x, float z) {
+  if constexpr (sizeof(T) == 2) return __fdividef(x, 1.f + __expf(-z));
+  else return x / (1.f + expf(-z));
+}
+
+// grid (rows, ceil(F / (THREADS V)))
 template <typename T, int V>
 __global__ void __launch_bounds__(THREADS)
-clamped_glu_kernel(const T* __restrict__ gu, T* __restrict__ out, long long rows, int F, float limit, float alpha) {
-  const long long total = rows * (F / V);
-  for (long long k = blockIdx.x * static_cast<long long>(THREADS) + threadIdx.x; k < total; k += static_cast<long long>(gridDim.x) * THREADS) {
-    const long long r = k / (F / V);
-    const int i = static_cast<int>(k - r * (F / V)) * V;
-    float g[V], u[V], o[V];
-    load_v<V>(gu + r * 2 * F + i, g);
-    load_v<V>(gu + r * 2 * F + F + i, u);
+clamped_glu_kernel(const T* __restrict__ gu, T* __restrict__ out, int F, float limit, float alpha) {
+  const long long r = blockIdx.x;
+  const int i = (blockIdx.y * THREADS + threadIdx.x) * V;
+  if (i >= F) return;
+  float g[V], u[V], o[V];
+  load_v<V>(gu + r * 2 * F + i, g);
+  load_v<V>(gu + r * 2 * F + F + i, u);
 #pragma unroll
-    for (int j = 0; j < V; ++j) {
-      const float a = fminf(g[j], limit), b = fminf(fmaxf(u[j], -limit), limit);
-      const float e = sizeof(T) == 2 ? __expf(-alpha * a) : expf(-alpha * a);
-      o[j] = a / (1.f + e) * (b + 1.f);
-    }
-    store_v<V>(out + r * F + i, o);
+  for (int j = 0; j < V; ++j) {
+    const float a = fminf(g[j], limit), b = fminf(fmaxf(u[j], -limit), limit);
+    o[j] = times_sigmoid<T>(a, alpha * a) * (b + 1.f);
   }
+  store_v<V>(out + r * F + i, o);
 }
 
 template <typename T, int V>
@@ -215,15 +174,10 @@ sigmoid_gated_norm_kernel(const T* __restrict__ x, const T* __restrict__ gate, c
     load_v<V>(gate + t * d + i, g);
     load_v<V>(w + i, c);
 #pragma unroll
-    for (int j = 0; j < V; ++j) {
-      const float e = sizeof(T) == 2 ? __expf(-g[j]) : expf(-g[j]);
-      o[j] = sx[i + j] * r * c[j] / (1.f + e);
-    }
+    for (int j = 0; j < V; ++j) o[j] = times_sigmoid<T>(sx[i + j] * r * c[j], g[j]);
     store_v<V>(out + t * d + i, o);
   }
 }
-
-inline bool aligned(const void* p, size_t a) { return (reinterpret_cast<uintptr_t>(p) & (a - 1)) == 0; }
 
 template <typename K>
 int allow_smem(K kernel, size_t bytes) {
@@ -287,12 +241,13 @@ extern "C" int dewb_clamped_glu(const void* gu, void* out, long long rows, int F
   if (rows <= 0) return 0;
   if (F < 1) return -3;
   cudaStream_t stream = reinterpret_cast<cudaStream_t>(stream_ptr);
-  const bool vec = F % 4 == 0 && aligned(gu, 16) && aligned(out, 16);
-  const long long work = rows * (vec ? F / 4 : F), want = (work + THREADS - 1) / THREADS;
-  const unsigned grid = static_cast<unsigned>(want < 148 * 32 ? want : 148 * 32);
-#define DEWB_GLU(TT, VV) clamped_glu_kernel<TT, VV><<<grid, THREADS, 0, stream>>>(static_cast<const TT*>(gu), static_cast<TT*>(out), rows, F, limit, alpha)
-  if (fp32) { if (vec) DEWB_GLU(float, 4); else DEWB_GLU(float, 1); }
-  else { if (vec) DEWB_GLU(bf16, 4); else DEWB_GLU(bf16, 1); }
+  const int v = F % 8 == 0 && !fp32 && aligned(gu, 16) && aligned(out, 16) ? 8 : F % 4 == 0 && aligned(gu, 16) && aligned(out, 16) ? 4 : 1;
+  const int blocks = (F + THREADS * v - 1) / (THREADS * v);
+  if (blocks > 65535) return -3;
+  const dim3 grid(static_cast<unsigned>(rows), blocks);
+#define DEWB_GLU(TT, VV) clamped_glu_kernel<TT, VV><<<grid, THREADS, 0, stream>>>(static_cast<const TT*>(gu), static_cast<TT*>(out), F, limit, alpha)
+  if (fp32) { if (v == 4) DEWB_GLU(float, 4); else DEWB_GLU(float, 1); }
+  else { if (v == 8) DEWB_GLU(bf16, 8); else if (v == 4) DEWB_GLU(bf16, 4); else DEWB_GLU(bf16, 1); }
 #undef DEWB_GLU
   return static_cast<int>(cudaGetLastError());
 }
@@ -309,7 +264,7 @@ extern "C" int dewb_sigmoid_gated_norm(const void* x, const void* gate, const vo
     sigmoid_gated_norm_kernel<TT, VV><<<grid, THREADS, smem, stream>>>(static_cast<const TT*>(x), static_cast<const TT*>(gate), \
         static_cast<const TT*>(w), static_cast<TT*>(out), d, eps); } while (0)
   if (fp32) { if (vec) DEWB_GN(float, 4); else DEWB_GN(float, 1); }
-  else { if (vec) DEWB_GN(bf16, 4); else DEWB_GN(bf16, 1); }
+  else { if (vec && d % 8 == 0) DEWB_GN(bf16, 8); else if (vec) DEWB_GN(bf16, 4); else DEWB_GN(bf16, 1); }
 #undef DEWB_GN
   return static_cast<int>(cudaGetLastError());
 }

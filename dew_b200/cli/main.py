@@ -1,4 +1,4 @@
-"""``dewb`` command line: ``train``, ``sweep``, ``profile``, ``inspect``, ``plan``, ``serve``, ``export``, ``data export | analyse | shards``, ``launch``.
+"""``dewb`` command line: ``train``, ``sweep``, ``profile``, ``inspect``, ``plan``, ``generate``, ``serve``, ``trace``, ``export``, ``data export | analyse | shards``, ``launch``.
 
 Parity: src/dew/_cli/main.py (subcommands Train with ``--set path=value``, Profile, Inspect, Export, DataExport),
 src/dew/_cli/launch.py.  Importing this module imports no CUDA library.
@@ -205,6 +205,9 @@ def cmd_serve(args) -> int:
     task = pipeline(args.checkpoint)
     if torch.cuda.is_available() and not args.cpu:
         task.model.cuda()
+    if args.tokenizer == "bytes":
+        from ..data import ByteTokenizer
+        task.tokenizer = ByteTokenizer()
     server = Server.from_task(task, slots=args.slots, capacity=args.capacity, kv_cache=KVCache(page_size=args.page_size), host_pages=args.host_pages,
                               cuda_graph=torch.cuda.is_available() and not args.cpu)
     with CompletionService(server, name=args.name or Path(args.checkpoint).name, host=args.host, port=args.port) as service:
@@ -218,11 +221,41 @@ def cmd_serve(args) -> int:
     return 0
 
 
+def cmd_generate(args) -> int:
+    """Continue prompts with a run's or a released checkpoint's model: token ids (``--ids 5,17,3``, repeated) or text (``--prompt``)."""
+    import torch
+
+    from ..inference import pipeline
+    from ..sampling.text import Sampling
+    cuda = torch.cuda.is_available() and not args.cpu
+    task = pipeline(args.checkpoint, dtype=getattr(torch, args.dtype), device="cuda" if cuda else "cpu")
+    if args.tokenizer == "bytes":
+        from ..data import ByteTokenizer
+        task.tokenizer = ByteTokenizer()
+    prompts = [[int(t) for t in ids.split(",")] for ids in args.ids or []]
+    if args.prompt:
+        if task.tokenizer is None:
+            raise SystemExit("text prompts need a tokenizer: --tokenizer bytes")
+        prompts += [task.tokenizer.encode(p) for p in args.prompt]
+    if not prompts:
+        raise SystemExit("nothing to continue: give --ids or --prompt")
+    gen = task(prompts, args.max_new_tokens, key=args.seed, sampling=Sampling(temperature=args.temperature, top_k=args.top_k, top_p=args.top_p))
+    for r in range(len(prompts)):
+        row = {"prompt": prompts[r], "tokens": gen.new_tokens(r).tolist()}
+        if gen.text is not None:
+            row["text"] = gen.text[r]
+        print(json.dumps(row))
+    return 0
+
+
 def main(argv: Optional[Sequence[str]] = None) -> int:
     argv = list(sys.argv[1:] if argv is None else argv)
     if argv and argv[0] == "launch":
         from . import launch
         return launch.main(argv[1:])
+    if argv and argv[0] == "trace":
+        from . import trace
+        return trace.main(argv[1:])
     ap = argparse.ArgumentParser(prog="dewb")
     sub = ap.add_subparsers(dest="command", required=True)
     t = sub.add_parser("train"); t.add_argument("recipe"); t.add_argument("--set", action="append"); t.add_argument("--cpu", action="store_true")
@@ -242,7 +275,12 @@ def main(argv: Optional[Sequence[str]] = None) -> int:
     sv = sub.add_parser("serve"); sv.add_argument("checkpoint"); sv.add_argument("--host", default="127.0.0.1"); sv.add_argument("--port", type=int, default=8000)
     sv.add_argument("--slots", type=int, default=64); sv.add_argument("--capacity", type=int, default=2048); sv.add_argument("--page-size", type=int, default=16)
     sv.add_argument("--host-pages", type=int, default=0); sv.add_argument("--name", default=None); sv.add_argument("--cpu", action="store_true")
+    sv.add_argument("--tokenizer", default=None, choices=["bytes"])
     sv.add_argument("--max-seconds", type=float, default=None); sv.set_defaults(fn=cmd_serve)
+    gn = sub.add_parser("generate"); gn.add_argument("checkpoint"); gn.add_argument("--ids", action="append"); gn.add_argument("--prompt", action="append")
+    gn.add_argument("--max-new-tokens", type=int, default=32); gn.add_argument("--temperature", type=float, default=0.0); gn.add_argument("--top-k", type=int, default=None)
+    gn.add_argument("--top-p", type=float, default=1.0); gn.add_argument("--seed", type=int, default=0); gn.add_argument("--tokenizer", default=None, choices=["bytes"])
+    gn.add_argument("--dtype", default="bfloat16", choices=["bfloat16", "float32"]); gn.add_argument("--cpu", action="store_true"); gn.set_defaults(fn=cmd_generate)
     pl = sub.add_parser("plan"); pl.add_argument("recipe"); pl.add_argument("--set", action="append"); pl.add_argument("--devices", type=int, default=8)
     pl.set_defaults(fn=cmd_plan)
     args = ap.parse_args(argv)

@@ -62,13 +62,18 @@ class TextGeneration:
 
 def pipeline(source, *, mesh=None, layout=None, dtype=None, param_dtype=None, ema: Optional[bool] = None, step: Optional[int] = None,
              model=None, tokenizer=None, device=None):
-    """Build a task from a checkpoint directory (``run.json`` names the model), a ``TrainState`` + model, or a module."""
+    """Build a task from a checkpoint directory (``run.json`` names the model), a released checkpoint (``config.json`` + safetensors, any family
+    ``Pretrained.load`` reads), a ``TrainState`` + model, or a module."""
     import os
     from ..checkpoints import Checkpoints
     from ..utils.registry import lookup
     if isinstance(source, (str, os.PathLike)):
         ck = Checkpoints(source)
         run = ck.read_run() or {}
+        if model is None and not run and os.path.exists(os.path.join(source, "config.json")):
+            from ..interop.hf import Pretrained
+            model = Pretrained.load(source, dtype=dtype or param_dtype or torch.bfloat16, device=device or "cpu").eval()
+            return TextGeneration(model, None, tokenizer)
         if model is None:
             if "model" not in run:
                 raise FileNotFoundError(f"{source}/run.json does not describe a model; pass model=")

@@ -52,6 +52,13 @@ def read_ragenex_config(cfg: Mapping[str, Any]) -> TransformerConfig:
         loop=None if not loop else Loop(steps=int(loop["times"]), first=int(loop["start"]), end=int(loop["stop"])))
 
 
+def ragenex(dtype=None, device=None, **fields) -> CausalTransformer:
+    """A freshly initialised model from the fields of a ``config.json`` (the registry's name for the design)."""
+    model = CausalTransformer(read_ragenex_config(fields), dtype=dtype, device=device)
+    model.family = "ragenex"
+    return model
+
+
 def write_ragenex_config(c: TransformerConfig) -> Dict[str, Any]:
     names = {v: k for k, v in KINDS.items()}
     layers = []

@@ -277,6 +277,17 @@ def test_release_with_missing_or_unknown_tensors_is_refused(tmp_path):
         Pretrained.load(C.write(tmp_path / "d", bad, w))
 
 
+def test_command_line_and_registry(tmp_path, capsys):
+    from dew_b200.cli.main import main
+    from dew_b200.utils.registry import lookup
+    cfg, w, _ = C.load(tmp_path, "plain")
+    p = C.prompt(cfg, 5)
+    assert main(["generate", str(tmp_path / "model"), "--ids", ",".join(map(str, p)), "--max-new-tokens", "4", "--dtype", "float32", "--cpu"]) == 0
+    assert json.loads(capsys.readouterr().out) == {"prompt": p, "tokens": _greedy(cfg, w, p, 4)}
+    built = lookup("ragenex", "model")(**cfg)
+    assert built.config == Pretrained.load(tmp_path / "model").config and built.family == "ragenex"
+
+
 def test_too_many_tokens_are_refused(tmp_path):
     cfg, _, m = C.load(tmp_path, "plain")
     b = RowBatch(m, 1, 8)
