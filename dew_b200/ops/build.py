@@ -31,7 +31,7 @@ EXACT_MATH = ("residual_streams", "paged_attention", "decayed_recurrence")
 # Subsets of the library a program can build alone, as ``libdewb_<part>.so``: a process that only decodes needs neither the training nor
 # the multi-GPU kernels.
 PARTS = {
-    "decoder": ("elementwise", "decode_attention", "decode_attention_tma", "flash_fwd_sm100", "gemm_sm100", "gemm_pair_sm100", "sampling")
+    "decoder": ("elementwise", "decode_attention", "decode_attention_tma", "flash_fwd_sm100", "gemm_sm100", "gemm_pair_sm100")
     + EXACT_MATH,
 }
 

@@ -144,7 +144,7 @@ def gemm(a: torch.Tensor, b: torch.Tensor, *, a_mn: bool = False, b_mn: bool = F
     cell = ("decode",) if (M <= 128 and case["plain"] and bias is None) else (("skinny",) if tiles < 24 else None)
     if bias is not None:
         case["plain"] = False                                    # (the weight-streaming kernel has no bias epilogue)
-    if kernel is None and cell is None and tiles >= 148 and _pair_built():
+    if kernel is None and cell is None and tiles >= 148 and _pair_built() and all(case[x] % 8 == 0 for x in ("lda", "ldb", "ldd")) and case["aligned"]:
         # measured: the pair kernel is 5-15 % faster on the layer shapes; the single-CTA kernel keeps the very wide head.
         # With DEWB_TUNE=1 the two are timed once per shape and the pick is cached on disk (ops/tuning.py).
         first = "sm100_pair" if (LARGE_GEMM == "sm100_pair" and N <= 32768) else "sm100_tcgen05"

@@ -22,3 +22,13 @@ def test_every_kernel_builds_within_its_register_budget():
     for needle in ("flash_fwd_kernel", "flash_dq_kernel", "flash_dkv_kernel", "gemm_pair_kernel", "gdn_scan_fwd_kernel", "moe_push_kernel",
                    "paged_decode_tma_kernel", "rs_adamw_ag_kernel"):
         assert needle in names, needle
+
+
+def test_library_parts_name_kernel_files():
+    """A part's files exist and hold what the decoding path cannot do without."""
+    stems = {p.stem for p in B.sources()}
+    for part, names in B.PARTS.items():
+        assert set(names) <= stems, part
+    assert set(B.EXACT_MATH) <= set(B.PARTS["decoder"])
+    assert "--use_fast_math" not in B._flags(B.CSRC / "kernels" / "residual_streams.cu")
+    assert "--use_fast_math" in B._flags(B.CSRC / "kernels" / "elementwise.cu")
