@@ -70,7 +70,7 @@ class Server:
         self.spec = KVCache(spec.quantized, spec.page_size, pool, spec.groups, spec.offloaded)
         p = next(model.parameters())
         self.store = make_cache(model, slots, capacity, self.spec)
-        if self.store.recurrent:
+        if self.store.keeps_state:
             prefix_cache = False          # a recurrent state stands for a whole row: no page of another row brings it along
         if self.store.slots is not None and host_pages > 0:
             raise NotImplementedError("the host tier copies pages of caches whose layers all keep the same heads")

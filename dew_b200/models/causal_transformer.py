@@ -516,6 +516,8 @@ class CausalTransformer(nn.Module):
         """The looped trunk: returns the final-normed exit state of the last pass, or of every pass with ``passes``."""
         cfg, loop = self.config, self.config.loop
         steps = loop.steps if steps is None else steps
+        if cache is not None and getattr(cache, "layers", 0) < len(self.runs()):
+            raise NotImplementedError(f"a looped decoder keeps one cache per pass: {len(self.runs())} entries (sampling.text.make_cache builds them)")
         if cache is not None and (loop.messages > 0 or passes or steps != loop.steps):
             raise NotImplementedError("a looped decoder's cache holds its configured passes, each with keys and values of its own; cross-pass messages, "
                                       "per-pass exits and another number of passes run on whole sequences without a cache")
@@ -593,6 +595,11 @@ class CausalTransformer(nn.Module):
         if pos is not None and cache is None and tokens.shape[1] > pos.shape[0]:
             raise ValueError(f"{tokens.shape[1]} tokens do not fit the {pos.shape[0]} learned positions")
         runs = self.runs(steps)
+        if cache is not None:
+            if len(getattr(cache, "slots", None) or ()) != len(self.runs()):
+                raise ValueError("this decoder's layers differ in what they keep: its cache comes from sampling.text.make_cache")
+            if positions is None:
+                positions = torch.arange(tokens.shape[1], device=tokens.device)[None].expand(tokens.shape[0], -1)
         if cache is not None and steps is not None and steps != cfg.loop.steps:
             raise NotImplementedError("the cache holds the configured number of passes")
         H = ops_streams.embed_streams(tokens, positions, self.embed.weight, pos, cfg.hyper_connections)

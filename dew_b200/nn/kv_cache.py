@@ -143,7 +143,7 @@ class KVStore:
 
     # ------------------------------------------------------------------ layers that differ (CacheSlot)
     @property
-    def recurrent(self) -> bool:
+    def keeps_state(self) -> bool:
         """Whether some layer keeps a state (which no page holds: a prompt's prefix cannot be taken from another row's pages)."""
         return any(s.state is not None for s in self.slots or ())
 
