@@ -1,6 +1,7 @@
 // Optional attention variants shared by the forward and backward flash kernels.  The plain causal / full kernels are
 // compiled with VAR = false and contain none of this.
 //   window   : query i sees keys in (i + T - S - window, i + T - S]  (0 = no window)
+//   chunk    : query i sees no key from before the start of its chunk of `chunk` positions, counted from 0 (0 = no chunks; forward only)
 //   softcap  : scores become cap * tanh(score / cap)                 (0 = none)
 //   sinks    : one learned logit per query head that joins the softmax denominator only (forward; the backward kernels
 //              see it through the saved log-sum-exp)
@@ -18,6 +19,7 @@ struct Variant {
   const float* sinks;      // [Hq] or null
   const int* q_seg;        // [B, S] or null
   const int* k_seg;        // [B, T] or null
+  int chunk;
 };
 
 __device__ __forceinline__ float fast_tanh(float x) {
@@ -31,6 +33,7 @@ __device__ __forceinline__ int first_key_tile(const Variant& v, int b, int q0, i
   const int off = T - S;
   int lo = 0;
   if (v.window > 0) lo = max(0, (q0 + off - v.window + 1) / bn);
+  if (v.chunk > 0) lo = max(lo, (q0 + off) / v.chunk * v.chunk / bn);
   if (v.q_seg != nullptr && v.k_seg != nullptr) {
     const int first = v.q_seg[static_cast<long long>(b) * S + min(q0, S - 1)];
     const int* ks = v.k_seg + static_cast<long long>(b) * T;

@@ -8,10 +8,13 @@ namespace rows {
 
 using bf16 = __nv_bfloat16;
 
-// V consecutive values (8: bf16 only, 4 or 1) as fp32
+// V consecutive values (8, 4 or 1) as fp32
 template <int V>
 __device__ __forceinline__ void load_v(const float* p, float (&f)[V]) {
-  if constexpr (V == 4) {
+  if constexpr (V == 8) {
+    const float4 a = reinterpret_cast<const float4*>(p)[0], b = reinterpret_cast<const float4*>(p)[1];
+    f[0] = a.x; f[1] = a.y; f[2] = a.z; f[3] = a.w; f[4] = b.x; f[5] = b.y; f[6] = b.z; f[7] = b.w;
+  } else if constexpr (V == 4) {
     const float4 v = *reinterpret_cast<const float4*>(p);
     f[0] = v.x; f[1] = v.y; f[2] = v.z; f[3] = v.w;
   } else {

@@ -16,6 +16,8 @@
 #include <cuda_fp8.h>
 #include <cuda_runtime.h>
 
+#include "../common/key_range.cuh"
+
 namespace dewb {
 namespace decode {
 
@@ -56,7 +58,7 @@ paged_decode_kernel(const __nv_bfloat16* __restrict__ q, const void* __restrict_
                     const float* __restrict__ kscale, const float* __restrict__ vscale,
                     const int* __restrict__ page_table, const int* __restrict__ lengths, float* __restrict__ part_m,
                     float* __restrict__ part_l, float* __restrict__ part_acc, int Hq, int Hkv, int share, int page_size,
-                    int max_pages, int splits, float scale_log2, int window) {
+                    int max_pages, int splits, float scale_log2, int window, int chunk) {
   constexpr int DV = D / 32;                 // value elements per lane
   const int row = blockIdx.x, hk = blockIdx.y, split = blockIdx.z;
   const int kvh = hk / share;                  // `share` groups of query heads read the same KV head
@@ -75,7 +77,7 @@ paged_decode_kernel(const __nv_bfloat16* __restrict__ q, const void* __restrict_
   }
   __syncthreads();
   // keys of this split: [k_begin, k_end) in 32-key blocks, interleaved across the CTA's warps
-  const int first = (window > 0 && len > window) ? len - window : 0;
+  const int first = first_key(len, window, chunk);
   const int span = len - first;
   const int per_split = ((span + splits - 1) / splits + 31) / 32 * 32;
   const int k_begin = first + split * per_split;
@@ -311,7 +313,7 @@ extern "C" int dewb_paged_decode(const void* q, const void* kpool, const void* v
                                  const float* vscale, const int* page_table, const int* lengths, const float* sinks,
                                  void* out, float* lse, float* part_m, float* part_l, float* part_acc, int rows, int Hq,
                                  int Hkv, int share, int D, int page_size, int max_pages, int splits, float scale, int window,
-                                 int kv_kind, void* stream_ptr) {
+                                 int chunk, int kv_kind, void* stream_ptr) {
   if (rows <= 0) return 0;
   if ((D != 64 && D != 128 && D != 256) || share < 1 || Hkv < 1 || Hq % (Hkv * share) != 0 ||
       Hq / (Hkv * share) > MAX_G || splits < 1)
@@ -322,7 +324,7 @@ extern "C" int dewb_paged_decode(const void* q, const void* kpool, const void* v
   const __nv_bfloat16* qp = reinterpret_cast<const __nv_bfloat16*>(q);
   const int Gq = Hq / (Hkv * share);
 #define DEWB_DECODE_G(DD, KK, GG) paged_decode_kernel<DD, KK, GG><<<grid, WARPS * 32, 0, stream>>>( \
-    qp, kpool, vpool, kscale, vscale, page_table, lengths, part_m, part_l, part_acc, Hq, Hkv, share, page_size, max_pages, splits, scale_log2, window)
+    qp, kpool, vpool, kscale, vscale, page_table, lengths, part_m, part_l, part_acc, Hq, Hkv, share, page_size, max_pages, splits, scale_log2, window, chunk)
 #define DEWB_DECODE(DD, KK) do { if (Gq == 4) DEWB_DECODE_G(DD, KK, 4); else if (Gq == 8) DEWB_DECODE_G(DD, KK, 8); \
     else if (Gq == 1) DEWB_DECODE_G(DD, KK, 1); else if (Gq == 2) DEWB_DECODE_G(DD, KK, 2); else DEWB_DECODE_G(DD, KK, 0); } while (0)
 #define DEWB_DECODE_D(KK) do { if (D == 64) DEWB_DECODE(64, KK); else if (D == 128) DEWB_DECODE(128, KK); else DEWB_DECODE(256, KK); } while (0)

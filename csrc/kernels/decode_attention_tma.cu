@@ -12,6 +12,7 @@
 // The query count per KV head is far below the 64 rows tcgen05 needs, which is why this kernel uses the warp-level MMA.
 //
 // Capability parity: src/dew/nn/kernels/decode_attention.py (attend_paged), src/dew/nn/kernels/templates/attention_decode.py.
+#include "../common/key_range.cuh"
 #include "../common/ptx.cuh"
 #include "../common/tmap.h"
 
@@ -58,7 +59,7 @@ paged_decode_tma_kernel(const __grid_constant__ CUtensorMap tk, const __grid_con
                         const __nv_bfloat16* __restrict__ q, const int* __restrict__ page_table,
                         const int* __restrict__ lengths, float* __restrict__ part_m, float* __restrict__ part_l,
                         float* __restrict__ part_acc, int Hq, int Hkv, int page_size, int max_pages, int splits,
-                        float scale_log2, int window, long long q_row_stride, int* __restrict__ err,
+                        float scale_log2, int window, int chunk, long long q_row_stride, int* __restrict__ err,
                         __nv_bfloat16* __restrict__ out, const float* __restrict__ sinks, unsigned int* __restrict__ arrivals,
                         int chunk_tiles) {
   extern __shared__ __align__(1024) uint8_t smem[];
@@ -75,7 +76,7 @@ paged_decode_tma_kernel(const __grid_constant__ CUtensorMap tk, const __grid_con
   const int G = Hq / Hkv;
   const int len = lengths[row];
   // this split's keys, in whole 64-key tiles: [t_begin, t_end) tile indices of the row; keys outside [first, len) are masked
-  const int first = (window > 0 && len > window) ? len - window : 0;
+  const int first = first_key(len, window, chunk);
   const int tile_lo = first / TK, tile_hi = (len + TK - 1) / TK;
   // With `out` the kernel finishes the row itself: a row uses as many of the grid's splits as it has chunks of `chunk_tiles`
   // tiles (short rows take one CTA, the others leave at once), and the last split to arrive merges the partials.
@@ -307,7 +308,7 @@ struct Seg { int row, hk, part, eff, t_begin, ntiles, first, len; };
 
 // the segment that starts at tile `u` of the sequence and ends with its (row, head) or with the CTA's range `u1`
 __device__ __forceinline__ Seg locate(int u, int u1, const int* prefix, const int* __restrict__ lengths, int rows,
-                                      int per_head, int Q, int window) {
+                                      int per_head, int Q, int window, int chunk) {
   Seg sg;
   sg.hk = u / per_head;
   const int w = u - sg.hk * per_head;
@@ -320,7 +321,7 @@ __device__ __forceinline__ Seg locate(int u, int u1, const int* prefix, const in
   const int start = sg.hk * per_head + prefix[lo];          // the (row, head)'s first tile in the sequence
   const int n = prefix[lo + 1] - prefix[lo];
   sg.len = lengths[lo];
-  sg.first = (window > 0 && sg.len > window) ? sg.len - window : 0;
+  sg.first = first_key(sg.len, window, chunk);
   sg.t_begin = sg.first / TK + (u - start);
   sg.ntiles = min(u1, start + n) - u;
   const int first_cta = start / Q;
@@ -334,7 +335,7 @@ paged_decode_persist_kernel(const __grid_constant__ CUtensorMap tk, const __grid
                             const __nv_bfloat16* __restrict__ q, const int* __restrict__ page_table,
                             const int* __restrict__ lengths, float* __restrict__ part_m, float* __restrict__ part_l,
                             float* __restrict__ part_acc, int rows, int Hq, int Hkv, int page_size, int max_pages,
-                            int max_parts, float scale_log2, int window, long long q_row_stride, int* __restrict__ err,
+                            int max_parts, float scale_log2, int window, int chunk, long long q_row_stride, int* __restrict__ err,
                             __nv_bfloat16* __restrict__ out, const float* __restrict__ sinks,
                             unsigned int* __restrict__ arrivals, int min_tiles) {
   extern __shared__ __align__(1024) uint8_t smem[];
@@ -352,7 +353,7 @@ paged_decode_persist_kernel(const __grid_constant__ CUtensorMap tk, const __grid
   // tile counts of the rows, then their exclusive prefix sum (warp 0: each lane a contiguous run of rows)
   for (int r = tid; r < rows; r += THREADS) {
     const int len = lengths[r];
-    const int first = (window > 0 && len > window) ? len - window : 0;
+    const int first = first_key(len, window, chunk);
     const int tiles = max(0, (len + TK - 1) / TK - first / TK);
     prefix[r + 1] = tiles;
     if (tiles == 0 && (r % gridDim.x) == blockIdx.x)         // a row without keys: its output is zero
@@ -397,7 +398,7 @@ paged_decode_persist_kernel(const __grid_constant__ CUtensorMap tk, const __grid
       tma_prefetch_desc(&tv);
       bool ok = true;
       for (int u = u0; u < u1 && ok;) {
-        const Seg sg = locate(u, u1, prefix, lengths, rows, per_head, Q, window);
+        const Seg sg = locate(u, u1, prefix, lengths, rows, per_head, Q, window, chunk);
         const int* table = page_table + static_cast<long long>(sg.row) * max_pages;
         for (int t = 0; t < sg.ntiles; ++t, ++tg) {
           const int s = tg % STAGES;
@@ -425,7 +426,7 @@ paged_decode_persist_kernel(const __grid_constant__ CUtensorMap tk, const __grid
   const int g = lane >> 2, c = (lane & 3) * 2;
   bool ok = true;
   for (int u = u0; u < u1;) {
-    const Seg it = locate(u, u1, prefix, lengths, rows, per_head, Q, window);
+    const Seg it = locate(u, u1, prefix, lengths, rows, per_head, Q, window, chunk);
     u += it.ntiles;
     // Q fragments straight from global memory: A operand rows = heads; rows 8..15 do not exist (a1 = a3 = 0)
     uint32_t qa0[8], qa2[8];
@@ -583,7 +584,7 @@ paged_decode_persist_kernel(const __grid_constant__ CUtensorMap tk, const __grid
 extern "C" int dewb_paged_decode_stream(const void* q, const void* kpool, const void* vpool, long long pool_tokens,
                                         const int* page_table, const int* lengths, float* part_m, float* part_l,
                                         float* part_acc, int rows, int Hq, int Hkv, int page_size, int max_pages, int splits,
-                                        float scale, int window, long long q_row_stride, int* err, void* stream_ptr) {
+                                        float scale, int window, int chunk, long long q_row_stride, int* err, void* stream_ptr) {
   using namespace dewb::decode2;
   if (rows <= 0) return 0;
   if (Hq % Hkv != 0 || Hq / Hkv > 8 || page_size % TK != 0 || splits < 1 || pool_tokens <= 0) return -3;
@@ -597,7 +598,7 @@ extern "C" int dewb_paged_decode_stream(const void* q, const void* kpool, const 
   dim3 grid(rows, Hkv, splits);
   paged_decode_tma_kernel<<<grid, THREADS, SMEM, reinterpret_cast<cudaStream_t>(stream_ptr)>>>(
       tk, tv, reinterpret_cast<const __nv_bfloat16*>(q), page_table, lengths, part_m, part_l, part_acc, Hq, Hkv, page_size,
-      max_pages, splits, scale * 1.4426950408889634f, window, q_row_stride > 0 ? q_row_stride : static_cast<long long>(Hq) * D, err,
+      max_pages, splits, scale * 1.4426950408889634f, window, chunk, q_row_stride > 0 ? q_row_stride : static_cast<long long>(Hq) * D, err,
       nullptr, nullptr, nullptr, 0);
   return static_cast<int>(cudaGetLastError());
 }
@@ -609,7 +610,7 @@ extern "C" int dewb_paged_decode_fused(const void* q, const void* kpool, const v
                                        const int* page_table, const int* lengths, float* part_m, float* part_l,
                                        float* part_acc, unsigned int* arrivals, const float* sinks, void* out, int rows, int Hq,
                                        int Hkv, int page_size, int max_pages, int splits, int chunk_tiles, float scale,
-                                       int window, long long q_row_stride, int* err, void* stream_ptr) {
+                                       int window, int chunk, long long q_row_stride, int* err, void* stream_ptr) {
   using namespace dewb::decode2;
   if (rows <= 0) return 0;
   if (Hq % Hkv != 0 || Hq / Hkv > 8 || page_size % TK != 0 || splits < 1 || chunk_tiles < 1 || pool_tokens <= 0) return -3;
@@ -623,7 +624,7 @@ extern "C" int dewb_paged_decode_fused(const void* q, const void* kpool, const v
   dim3 grid(rows, Hkv, splits);
   paged_decode_tma_kernel<<<grid, THREADS, SMEM, reinterpret_cast<cudaStream_t>(stream_ptr)>>>(
       tk, tv, reinterpret_cast<const __nv_bfloat16*>(q), page_table, lengths, part_m, part_l, part_acc, Hq, Hkv, page_size,
-      max_pages, splits, scale * 1.4426950408889634f, window, q_row_stride > 0 ? q_row_stride : static_cast<long long>(Hq) * D, err,
+      max_pages, splits, scale * 1.4426950408889634f, window, chunk, q_row_stride > 0 ? q_row_stride : static_cast<long long>(Hq) * D, err,
       reinterpret_cast<__nv_bfloat16*>(out), sinks, arrivals, chunk_tiles);
   return static_cast<int>(cudaGetLastError());
 }
@@ -636,7 +637,7 @@ extern "C" int dewb_paged_decode_persist(const void* q, const void* kpool, const
                                          const int* page_table, const int* lengths, float* part_m, float* part_l,
                                          float* part_acc, unsigned int* arrivals, const float* sinks, void* out, int rows, int Hq,
                                          int Hkv, int page_size, int max_pages, int max_parts, int min_tiles, float scale,
-                                         int window, long long q_row_stride, int ctas, int* err, void* stream_ptr) {
+                                         int window, int chunk, long long q_row_stride, int ctas, int* err, void* stream_ptr) {
   using namespace dewb::decode2;
   if (rows <= 0) return 0;
   if (Hq % Hkv != 0 || Hq / Hkv > 8 || page_size % TK != 0 || max_parts < 2 || min_tiles < 1 || pool_tokens <= 0 ||
@@ -651,7 +652,7 @@ extern "C" int dewb_paged_decode_persist(const void* q, const void* kpool, const
   if (e != cudaSuccess) return static_cast<int>(e);
   paged_decode_persist_kernel<<<ctas, THREADS, P_SMEM, reinterpret_cast<cudaStream_t>(stream_ptr)>>>(
       tk, tv, reinterpret_cast<const __nv_bfloat16*>(q), page_table, lengths, part_m, part_l, part_acc, rows, Hq, Hkv, page_size,
-      max_pages, max_parts, scale * 1.4426950408889634f, window, q_row_stride > 0 ? q_row_stride : static_cast<long long>(Hq) * D, err,
+      max_pages, max_parts, scale * 1.4426950408889634f, window, chunk, q_row_stride > 0 ? q_row_stride : static_cast<long long>(Hq) * D, err,
       reinterpret_cast<__nv_bfloat16*>(out), sinks, arrivals, min_tiles);
   return static_cast<int>(cudaGetLastError());
 }

@@ -280,8 +280,10 @@ flash_fwd_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__
           for (int i = 0; i < HC; ++i) if (k0 + i > limit || k0 + i >= T) s[i] = -INFINITY;
         }
         if (VAR) {
-          if (var.window > 0) {
-            const int first = q0 + r + (T - S) - var.window + 1;   // first visible key of this row
+          if (var.window > 0 || var.chunk > 0) {
+            const int at = q0 + r + (T - S);
+            int first = var.window > 0 ? at - var.window + 1 : 0;   // first visible key of this row
+            if (var.chunk > 0) first = max(first, at / var.chunk * var.chunk);
             if (k0 < first) {
 #pragma unroll
               for (int i = 0; i < HC; ++i) if (k0 + i < first) s[i] = -INFINITY;
@@ -484,13 +486,13 @@ extern "C" int dewb_flash_set_variant(int variant) {
 
 // q [B,S,Hq,D], k/v [B,T,Hkv,D] (bf16, unit stride along D, other strides in elements: batch, sequence, head);
 // out [B,S,Hq,D] with its own strides; lse [B,Hq,S] fp32 (natural log), may be null.
-// Variants (each off at 0 / null): `window` keys visible behind each query, `softcap`, `sinks` [Hq] fp32, `q_seg` [B,S] /
+// Variants (each off at 0 / null): `window` keys visible behind each query, `chunk` positions a query sees no key from outside of, `softcap`, `sinks` [Hq] fp32, `q_seg` [B,S] /
 // `k_seg` [B,T] int32 segment ids of packed documents (non-decreasing along the sequence, rows 16-byte aligned: S, T % 4 == 0).
 extern "C" int dewb_flash_fwd_var(const void* q, const void* k, const void* v, void* out, float* lse, int B, int S, int T,
                                   int Hq, int Hkv, int D, long long q_sb, long long q_ss, long long q_sh, long long k_sb,
                                   long long k_ss, long long k_sh, long long v_sb, long long v_ss, long long v_sh,
                                   long long o_sb, long long o_ss, long long o_sh, float scale, int causal, int window,
-                                  float softcap, const float* sinks, const int* q_seg, const int* k_seg, int* err,
+                                  int chunk, float softcap, const float* sinks, const int* q_seg, const int* k_seg, int* err,
                                   void* stream_ptr) {
   using namespace dewb::attnfwd;
   if (D != 128 && D != 64) return -3;
@@ -500,7 +502,7 @@ extern "C" int dewb_flash_fwd_var(const void* q, const void* k, const void* v, v
     return -3;
   if ((q_seg != nullptr) != (k_seg != nullptr)) return -3;
   if (q_seg != nullptr && ((T % 4) || (reinterpret_cast<uintptr_t>(k_seg) & 15))) return -3;
-  if (window < 0 || softcap < 0.f) return -3;
+  if (window < 0 || chunk < 0 || softcap < 0.f) return -3;
   CUtensorMap tq, tk, tv;
   int r;
   if ((r = make_qkv_map(&tq, q, B, S, Hq, D, q_sb, q_ss, q_sh))) return 1000 + r;
@@ -508,8 +510,8 @@ extern "C" int dewb_flash_fwd_var(const void* q, const void* k, const void* v, v
   if ((r = make_qkv_map(&tv, v, B, T, Hkv, D, v_sb, v_ss, v_sh))) return 3000 + r;
   const float scale_log2 = scale * 1.4426950408889634f;
   cudaStream_t stream = reinterpret_cast<cudaStream_t>(stream_ptr);
-  const Variant var{window, softcap, sinks, q_seg, k_seg};
-  const bool any = window > 0 || softcap > 0.f || sinks != nullptr || q_seg != nullptr;
+  const Variant var{window, softcap, sinks, q_seg, k_seg, chunk};
+  const bool any = window > 0 || chunk > 0 || softcap > 0.f || sinks != nullptr || q_seg != nullptr;
 #define DEWB_FLASH_GO(DD, CC, PP, VV) launch<DD, CC, PP, VV>(tq, tk, tv, out, lse, B, S, T, Hq, Hkv, o_sb, o_ss, o_sh, scale_log2, var, err, stream)
   const bool pt = g_variant != 0;
   if (any) {
@@ -532,5 +534,5 @@ extern "C" int dewb_flash_fwd(const void* q, const void* k, const void* v, void*
                               long long o_sb, long long o_ss, long long o_sh, float scale, int causal, int* err,
                               void* stream_ptr) {
   return dewb_flash_fwd_var(q, k, v, out, lse, B, S, T, Hq, Hkv, D, q_sb, q_ss, q_sh, k_sb, k_ss, k_sh, v_sb, v_ss, v_sh, o_sb,
-                            o_ss, o_sh, scale, causal, 0, 0.f, nullptr, nullptr, nullptr, err, stream_ptr);
+                            o_ss, o_sh, scale, causal, 0, 0, 0.f, nullptr, nullptr, nullptr, err, stream_ptr);
 }

@@ -3,13 +3,19 @@
 //   qk_norm_append   from the packed projection [tokens, H dk + G dk + G dv]: RMS norm of q over all its heads at once and of k likewise
 //                    (weights may be null: no norm), the query temperature 1 + coef ln(floor((p + 1) / every) + 1), the copy into heads
 //                    of the cache's (padded) width, and the append of keys and values to the page pools
+//   head_norm_append   the same for per-head norms (one weight for all heads), with the projection's bias added on the way, rows that carry
+//                    more columns than the heads (gates), and layers that read another layer's keys and values (queries alone)
+//   head_gate        heads of the cache's width times a sigmoid of one number per head, packed to their own width
 //   paged_attend     causal attention of a call's tokens against everything the cache holds of their rows (any start positions; a decode
 //                    step is the case of one token per row); scores, softmax and sums in fp32 on the CUDA cores.  It is the fp32 form,
 //                    and takes the head widths the tensor-core kernels do not.
 //   paged_attend_mma   the same on the tensor cores for bf16 pools 64, 128 or 256 wide (a prompt's later portions, mixed start positions)
+//   Both take chunks (a query sees no key from before the start of its chunk of positions), a learned sink per head in the denominator, and
+//   a gate per head on the output.
 //
 // A query's row of work is (token, head of its group), so a group's heads share the key and value tiles.  Positions below 0 are padding:
 // nothing is appended for them and their outputs are zero.  Compiled without fast math.
+#include <climits>
 #include <cstdint>
 #include <cuda_bf16.h>
 #include <cuda_runtime.h>
@@ -94,13 +100,109 @@ qk_norm_append_kernel(const T* __restrict__ qkv, const T* __restrict__ qw, const
   }
 }
 
+// One group of LG lanes per (token, head); heads [0, H) queries, then G keys, then G values (G 0: queries alone).
+template <typename T, int V, int LG>
+__global__ void __launch_bounds__(256)
+head_norm_append_kernel(const T* __restrict__ qkv, long long row_stride, const T* __restrict__ bias, const T* __restrict__ qw, const T* __restrict__ kw,
+                        float eps, const int* __restrict__ positions, long long items, int S, int H, int G, int dk, int dv, int D,
+                        T* __restrict__ packed, T* __restrict__ kpool, T* __restrict__ vpool, Pool pool) {
+  const long long item = (static_cast<long long>(blockIdx.x) * 256 + threadIdx.x) / LG;
+  const int lane = threadIdx.x % LG;
+  const bool on = item < items;                      // every lane stays for the sums
+  const int heads = H + 2 * G;
+  const long long t = on ? item / heads : 0;
+  const int h = on ? static_cast<int>(item - t * heads) : 0;
+  const int part = h < H ? 0 : h < H + G ? 1 : 2, width = part == 2 ? dv : dk;
+  const int at = part == 2 ? (H + G) * dk + (h - H - G) * dv : h * dk;
+  const T* src = qkv + t * row_stride + at;
+  const T* b = bias == nullptr ? nullptr : bias + at;
+  const T* w = part == 0 ? qw : part == 1 ? kw : nullptr;
+  float ss = 0.f;
+  if (w != nullptr) {
+    for (int i = lane * V; i < width; i += LG * V) {
+      float a[V];
+      load_v<V>(src + i, a);
+      if (b != nullptr) {
+        float c[V];
+        load_v<V>(b + i, c);
+#pragma unroll
+        for (int j = 0; j < V; ++j) a[j] += c[j];
+      }
+#pragma unroll
+      for (int j = 0; j < V; ++j) ss += a[j] * a[j];
+    }
+  }
+#pragma unroll
+  for (int o = LG / 2; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+  if (!on) return;
+  const float r = w != nullptr ? 1.f / sqrtf(ss / width + eps) : 1.f;
+  T* dst = packed + item * D;
+  T* to_pool = nullptr;
+  if (part != 0 && positions[t] >= 0) {
+    const long long tok = pool_token(pool, static_cast<int>(t / S), positions[t]);
+    to_pool = (part == 1 ? kpool : vpool) + (tok * G + (part == 1 ? h - H : h - H - G)) * D;
+  }
+  for (int i = lane * V; i < D; i += LG * V) {
+    float a[V];
+#pragma unroll
+    for (int j = 0; j < V; ++j) a[j] = 0.f;
+    if (i < width) {
+      load_v<V>(src + i, a);
+      if (b != nullptr) {
+        float c[V];
+        load_v<V>(b + i, c);
+#pragma unroll
+        for (int j = 0; j < V; ++j) a[j] += c[j];
+      }
+      if (w != nullptr) {
+        float c[V];
+        load_v<V>(w + i, c);
+#pragma unroll
+        for (int j = 0; j < V; ++j) a[j] = a[j] * r * c[j];
+      }
+    }
+    store_v<V>(dst + i, a);
+    if (to_pool != nullptr) store_v<V>(to_pool + i, a);
+  }
+}
+
+__device__ __forceinline__ float sigmoid(float z) { return 1.f / (1.f + expf(-z)); }
+
+// grid (tokens, ceil(H dv / (256 V))): out [tokens, H, dv] = o [tokens, H, D] * sigmoid(gate [tokens, *] of the head)
+template <typename T, int V>
+__global__ void __launch_bounds__(256)
+head_gate_kernel(const T* __restrict__ o, const T* __restrict__ gate, long long gate_stride, T* __restrict__ out, int H, int dv, int D) {
+  const int i = (blockIdx.y * 256 + threadIdx.x) * V;
+  if (i >= H * dv) return;
+  const long long t = blockIdx.x;
+  const int h = i / dv;
+  float a[V];
+  load_v<V>(o + (t * H + h) * D + (i - h * dv), a);
+  const float s = sigmoid(ld(gate + t * gate_stride + h));
+#pragma unroll
+  for (int j = 0; j < V; ++j) a[j] *= s;
+  store_v<V>(out + t * H * dv + i, a);
+}
+
+// What a layer's attention adds to the causal softmax: each part off at 0 / null.
+template <typename T>
+struct Extras {
+  int chunk;               // a query sees no key from before the start of its chunk
+  const float* sinks;      // [H]: joins the denominator, has no value
+  const T* gate;           // [tokens, *]: head h's output times sigmoid(gate[token, h])
+  long long gate_stride;
+};
+
+__device__ __forceinline__ int chunk_start(int pos, int chunk) { return chunk > 0 && pos > 0 ? pos / chunk * chunk : 0; }
+
 constexpr int BQ = 32, BK = 32, THREADS = 256;
 
 // grid (query tiles, G, rows).  q [R, S, *, D] with a token stride; out [R, S, H, dv] contiguous.  NJ: value columns per thread / 4.
 template <typename T, int NJ>
 __global__ void __launch_bounds__(THREADS)
 paged_attend_kernel(const T* __restrict__ q, long long q_token_stride, const T* __restrict__ kpool, const T* __restrict__ vpool,
-                    const int* __restrict__ positions, int S, int H, int G, int dk, int dv, int D, float scale, T* __restrict__ out, Pool pool) {
+                    const int* __restrict__ positions, int S, int H, int G, int dk, int dv, int D, float scale, T* __restrict__ out, Pool pool,
+                    Extras<T> ex) {
   extern __shared__ __align__(16) float smem[];
   const int kst = ((dk + 3) & ~3) + 4, vst = NJ * 32 + 4;
   float* sq = smem;                     // [BQ][kst]
@@ -117,8 +219,11 @@ paged_attend_kernel(const T* __restrict__ q, long long q_token_stride, const T* 
     s_pos[tid] = r < rows ? positions[static_cast<long long>(row) * S + r / Gq] : -1;
   }
   __syncthreads();
-  int last = -1;
-  for (int i = 0; i < BQ; ++i) last = max(last, s_pos[i]);
+  int last = -1, lowest = INT_MAX;
+  for (int i = 0; i < BQ; ++i) {
+    last = max(last, s_pos[i]);
+    if (s_pos[i] >= 0) lowest = min(lowest, chunk_start(s_pos[i], ex.chunk));
+  }
   for (int i = tid; i < BQ * kst; i += THREADS) {
     const int r = i / kst, c = i - r * kst;
     float v = 0.f;
@@ -129,11 +234,11 @@ paged_attend_kernel(const T* __restrict__ q, long long q_token_stride, const T* 
     sq[i] = v;
   }
   const int qr = tid >> 3, ql = tid & 7;
-  const int my_pos = s_pos[qr];
+  const int my_pos = s_pos[qr], my_first = chunk_start(my_pos, ex.chunk);
   float m = -INFINITY, l = 0.f, acc[NJ][4];
 #pragma unroll
   for (int j = 0; j < NJ; ++j) { acc[j][0] = acc[j][1] = acc[j][2] = acc[j][3] = 0.f; }
-  for (int k0 = 0; k0 <= last; k0 += BK) {
+  for (int k0 = last < 0 ? 0 : lowest / BK * BK; k0 <= last; k0 += BK) {
     __syncthreads();
     if (tid < BK) s_tok[tid] = k0 + tid <= last ? pool_token(pool, row, k0 + tid) : -1;
     __syncthreads();
@@ -158,7 +263,7 @@ paged_attend_kernel(const T* __restrict__ q, long long q_token_stride, const T* 
     float bm = -INFINITY;
 #pragma unroll
     for (int j = 0; j < 4; ++j) {
-      if (k0 + ql + 8 * j > my_pos) s[j] = -INFINITY;
+      if (k0 + ql + 8 * j > my_pos || k0 + ql + 8 * j < my_first) s[j] = -INFINITY;
       bm = fmaxf(bm, s[j]);
     }
 #pragma unroll
@@ -190,7 +295,13 @@ paged_attend_kernel(const T* __restrict__ q, long long q_token_stride, const T* 
   }
   const int gr = r0 + qr;
   if (gr >= rows) return;
-  const float inv = l > 0.f ? 1.f / l : 0.f;
+  float inv = l > 0.f ? 1.f / l : 0.f;
+  const int head = g * Gq + gr % Gq;
+  if (ex.sinks != nullptr && l > 0.f) {
+    const float sink = ex.sinks[head], top = fmaxf(m, sink), f = expf(m - top);
+    inv = f / (l * f + expf(sink - top));
+  }
+  if (ex.gate != nullptr) inv *= sigmoid(ld(ex.gate + (static_cast<long long>(row) * S + gr / Gq) * ex.gate_stride + head));
   T* o = out + ((static_cast<long long>(row) * S + gr / Gq) * H + g * Gq + gr % Gq) * dv;
 #pragma unroll
   for (int j = 0; j < NJ; ++j)
@@ -213,7 +324,8 @@ __device__ __forceinline__ void cp16(uint32_t dst, const void* src, bool live) {
 template <int D>
 __global__ void __launch_bounds__(MTHREADS)
 paged_attend_mma_kernel(const bf16* __restrict__ q, long long q_token_stride, const bf16* __restrict__ kpool, const bf16* __restrict__ vpool,
-                        const int* __restrict__ positions, int S, int H, int G, int dv, float scale_log2, bf16* __restrict__ out, Pool pool) {
+                        const int* __restrict__ positions, int S, int H, int G, int dv, float scale_log2, bf16* __restrict__ out, Pool pool,
+                        Extras<bf16> ex) {
   using namespace mma16;
   constexpr int ST = D + 8;                        // smem row stride
   extern __shared__ __align__(16) uint8_t raw[];
@@ -229,9 +341,13 @@ paged_attend_mma_kernel(const bf16* __restrict__ q, long long q_token_stride, co
     s_pos[tid] = r < rows ? positions[static_cast<long long>(row) * S + r / Gq] : -1;
   }
   __syncthreads();
-  int last = -1;
-  for (int i = 0; i < MQ; ++i) last = max(last, s_pos[i]);
-  const int tiles = (last + MK) / MK;              // key tiles [0, last]
+  int last = -1, lowest = INT_MAX;
+  for (int i = 0; i < MQ; ++i) {
+    last = max(last, s_pos[i]);
+    if (s_pos[i] >= 0) lowest = min(lowest, chunk_start(s_pos[i], ex.chunk));
+  }
+  const int base = last < 0 ? 0 : lowest / MK * MK;
+  const int tiles = (last - base + MK) / MK;       // tiles of the keys [base, last]
   for (int i = tid; i < MQ * (D / 8); i += MTHREADS) {
     const int r = i / (D / 8), c = (i % (D / 8)) * 8, gr = r0 + r;
     const bool live = s_pos[r] >= 0;
@@ -242,7 +358,7 @@ paged_attend_mma_kernel(const bf16* __restrict__ q, long long q_token_stride, co
     bf16* dk_ = sk + (t & 1) * MK * ST;
     bf16* dv_ = sv + (t & 1) * MK * ST;
     for (int i = tid; i < MK * (D / 8); i += MTHREADS) {
-      const int r = i / (D / 8), c = (i % (D / 8)) * 8, key = t * MK + r;
+      const int r = i / (D / 8), c = (i % (D / 8)) * 8, key = base + t * MK + r;
       const bool live = key <= last;
       const long long off = live ? (pool_token(pool, row, key) * G + g) * D + c : 0;
       cp16(smem_addr(dk_ + r * ST + c), kpool + off, live);
@@ -252,6 +368,7 @@ paged_attend_mma_kernel(const bf16* __restrict__ q, long long q_token_stride, co
   };
   const int lg = lane >> 2, t2 = (lane & 3) * 2;
   const int p0 = s_pos[warp * 16 + lg], p1 = s_pos[warp * 16 + lg + 8];
+  const int f0_ = chunk_start(p0, ex.chunk), f1_ = chunk_start(p1, ex.chunk);        // first keys the rows see
   float m0 = -INFINITY, m1 = -INFINITY, l0 = 0.f, l1 = 0.f, o[D / 8][4];
 #pragma unroll
   for (int j = 0; j < D / 8; ++j) { o[j][0] = o[j][1] = o[j][2] = o[j][3] = 0.f; }
@@ -284,11 +401,11 @@ paged_attend_mma_kernel(const bf16* __restrict__ q, long long q_token_stride, co
     float x0 = -INFINITY, x1 = -INFINITY;
 #pragma unroll
     for (int j = 0; j < 8; ++j) {
-      const int key = t * MK + j * 8 + t2;
-      s[j][0] = key <= p0 ? s[j][0] * scale_log2 : -INFINITY;
-      s[j][1] = key + 1 <= p0 ? s[j][1] * scale_log2 : -INFINITY;
-      s[j][2] = key <= p1 ? s[j][2] * scale_log2 : -INFINITY;
-      s[j][3] = key + 1 <= p1 ? s[j][3] * scale_log2 : -INFINITY;
+      const int key = base + t * MK + j * 8 + t2;
+      s[j][0] = key <= p0 && key >= f0_ ? s[j][0] * scale_log2 : -INFINITY;
+      s[j][1] = key + 1 <= p0 && key + 1 >= f0_ ? s[j][1] * scale_log2 : -INFINITY;
+      s[j][2] = key <= p1 && key >= f1_ ? s[j][2] * scale_log2 : -INFINITY;
+      s[j][3] = key + 1 <= p1 && key + 1 >= f1_ ? s[j][3] * scale_log2 : -INFINITY;
       x0 = fmaxf(x0, fmaxf(s[j][0], s[j][1]));
       x1 = fmaxf(x1, fmaxf(s[j][2], s[j][3]));
     }
@@ -335,7 +452,13 @@ paged_attend_mma_kernel(const bf16* __restrict__ q, long long q_token_stride, co
   for (int e = 0; e < 2; ++e) {
     const int gr = r0 + warp * 16 + lg + 8 * e;
     if (gr >= rows) continue;
-    const float inv = e ? i1 : i0;
+    float inv = e ? i1 : i0;
+    const int head = g * Gq + gr % Gq;
+    if (ex.sinks != nullptr && inv > 0.f) {
+      const float m = e ? m1 : m0, l = e ? l1 : l0, sink = ex.sinks[head] * 1.4426950408889634f, top = fmaxf(m, sink), f = exp2f(m - top);
+      inv = f / (l * f + exp2f(sink - top));
+    }
+    if (ex.gate != nullptr) inv *= sigmoid(ld(ex.gate + (static_cast<long long>(row) * S + gr / Gq) * ex.gate_stride + head));
     bf16* dst = out + ((static_cast<long long>(row) * S + gr / Gq) * H + g * Gq + gr % Gq) * dv;
 #pragma unroll
     for (int j = 0; j < D / 8; ++j) {
@@ -348,34 +471,36 @@ paged_attend_mma_kernel(const bf16* __restrict__ q, long long q_token_stride, co
 
 template <int D>
 int attend_mma(const bf16* q, long long qs, const bf16* kpool, const bf16* vpool, const int* positions, int R, int S, int H, int G, int dv, float scale,
-               bf16* out, const Pool& pool, cudaStream_t stream) {
+               bf16* out, const Pool& pool, const Extras<bf16>& ex, cudaStream_t stream) {
   const int smem = (MQ + 4 * MK) * (D + 8) * 2;
   cudaError_t e = cudaFuncSetAttribute(paged_attend_mma_kernel<D>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
   if (e != cudaSuccess) return static_cast<int>(e);
   const long long tiles = (static_cast<long long>(S) * (H / G) + MQ - 1) / MQ;
   paged_attend_mma_kernel<D><<<dim3(static_cast<unsigned>(tiles), G, R), MTHREADS, smem, stream>>>(q, qs, kpool, vpool, positions, S, H, G, dv,
-                                                                                              scale * 1.4426950408889634f, out, pool);
+                                                                                              scale * 1.4426950408889634f, out, pool, ex);
   return static_cast<int>(cudaGetLastError());
 }
 
 template <typename T, int NJ>
 int attend(const T* q, long long qs, const T* kpool, const T* vpool, const int* positions, int R, int S, int H, int G, int dk, int dv, int D,
-           float scale, T* out, const Pool& pool, cudaStream_t stream) {
+           float scale, T* out, const Pool& pool, const Extras<T>& ex, cudaStream_t stream) {
   const int kst = ((dk + 3) & ~3) + 4, vst = NJ * 32 + 4;
   const size_t smem = static_cast<size_t>(BQ * kst + BK * kst + BK * vst + BQ * (BK + 1)) * 4;
   if (smem > 225 * 1024) return -3;
   cudaError_t e = cudaFuncSetAttribute(paged_attend_kernel<T, NJ>, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem));
   if (e != cudaSuccess) return static_cast<int>(e);
   const long long tiles = (static_cast<long long>(S) * (H / G) + BQ - 1) / BQ;
-  paged_attend_kernel<T, NJ><<<dim3(static_cast<unsigned>(tiles), G, R), THREADS, smem, stream>>>(q, qs, kpool, vpool, positions, S, H, G, dk, dv, D, scale, out, pool);
+  paged_attend_kernel<T, NJ><<<dim3(static_cast<unsigned>(tiles), G, R), THREADS, smem, stream>>>(q, qs, kpool, vpool, positions, S, H, G, dk, dv, D, scale, out,
+                                                                                             pool, ex);
   return static_cast<int>(cudaGetLastError());
 }
 
 template <typename T>
 int attend_any(const void* q, long long qs, const void* kpool, const void* vpool, const int* positions, int R, int S, int H, int G, int dk, int dv,
-               int D, float scale, void* out, const Pool& pool, cudaStream_t stream) {
+               int D, float scale, void* out, const Pool& pool, int chunk, const float* sinks, const void* gate, long long gate_stride, cudaStream_t stream) {
+  const Extras<T> ex{chunk, sinks, static_cast<const T*>(gate), gate_stride};
 #define DEWB_ATTEND(NN) attend<T, NN>(static_cast<const T*>(q), qs, static_cast<const T*>(kpool), static_cast<const T*>(vpool), positions, R, S, H, G, \
-                                      dk, dv, D, scale, static_cast<T*>(out), pool, stream)
+                                      dk, dv, D, scale, static_cast<T*>(out), pool, ex, stream)
   const int nj = (dv + 31) / 32;
   if (nj <= 1) return DEWB_ATTEND(1);
   if (nj <= 2) return DEWB_ATTEND(2);
@@ -411,31 +536,79 @@ extern "C" int dewb_qk_norm_append(const void* qkv, const void* qw, const void* 
   return static_cast<int>(cudaGetLastError());
 }
 
-extern "C" int dewb_paged_attend(const void* q, long long q_token_stride, const void* kpool, const void* vpool, const int* positions, int R, int S,
-                                 int H, int G, int dk, int dv, int D, float scale, void* out, const int* page_table, int page_size, int max_pages,
-                                 const int* row_ids, int fp32, void* stream_ptr) {
+// qkv [R * S, row_stride >= H dk + G dk + G dv] -> packed [R * S, H + 2 G, D] and the pools; per-head norms with the weights qw, kw [dk] (null: none),
+// bias [H dk + G dk + G dv] (null: none).  G 0: a layer without keys and values of its own (the pools are not touched).
+extern "C" int dewb_head_norm_append(const void* qkv, long long row_stride, const void* bias, const void* qw, const void* kw, float eps,
+                                     const int* positions, int R, int S, int H, int G, int dk, int dv, int D, void* packed, void* kpool,
+                                     void* vpool, const int* page_table, int page_size, int max_pages, const int* row_ids, int fp32,
+                                     void* stream_ptr) {
   if (R <= 0 || S <= 0) return 0;
-  if (H < 1 || G < 1 || H % G || dk < 1 || dv < 1 || D < dk || D < dv || page_size < 1 || max_pages < 1) return -3;
+  if (H < 1 || G < 0 || (G > 0 && H % G) || dk < 1 || dv < 1 || D < dk || D < dv || page_size < 1 || max_pages < 1 ||
+      row_stride < static_cast<long long>(H + G) * dk + static_cast<long long>(G) * dv)
+    return -3;
   cudaStream_t stream = reinterpret_cast<cudaStream_t>(stream_ptr);
   const Pool pool{page_table, page_size, max_pages, row_ids};
-  if (fp32) return attend_any<float>(q, q_token_stride, kpool, vpool, positions, R, S, H, G, dk, dv, D, scale, out, pool, stream);
-  return attend_any<bf16>(q, q_token_stride, kpool, vpool, positions, R, S, H, G, dk, dv, D, scale, out, pool, stream);
+  const bool vec = dk % 4 == 0 && dv % 4 == 0 && D % 4 == 0 && row_stride % 4 == 0 && aligned(qkv, 16) && aligned(bias, 16) && aligned(qw, 16) &&
+                   aligned(kw, 16) && aligned(packed, 16) && aligned(kpool, 16) && aligned(vpool, 16);
+  const long long items = static_cast<long long>(R) * S * (H + 2 * G);
+  const int lg = D <= 64 ? 16 : 32;
+  const long long blocks = (items * lg + 255) / 256;
+  if (blocks > 0x7fffffffll) return -3;
+#define DEWB_HEADS(TT, VV, LL) head_norm_append_kernel<TT, VV, LL><<<static_cast<unsigned>(blocks), 256, 0, stream>>>(static_cast<const TT*>(qkv),     row_stride, static_cast<const TT*>(bias), static_cast<const TT*>(qw), static_cast<const TT*>(kw), eps, positions, items, S, H, G, dk, dv, D,     static_cast<TT*>(packed), static_cast<TT*>(kpool), static_cast<TT*>(vpool), pool)
+#define DEWB_HEADS_L(TT, VV) do { if (lg == 16) DEWB_HEADS(TT, VV, 16); else DEWB_HEADS(TT, VV, 32); } while (0)
+  if (fp32) { if (vec) DEWB_HEADS_L(float, 4); else DEWB_HEADS_L(float, 1); }
+  else { if (vec) DEWB_HEADS_L(bf16, 4); else DEWB_HEADS_L(bf16, 1); }
+#undef DEWB_HEADS_L
+#undef DEWB_HEADS
+  return static_cast<int>(cudaGetLastError());
+}
+
+// o [tokens, H, D] -> out [tokens, H, dv], each head times sigmoid(gate[token * gate_stride + head])
+extern "C" int dewb_head_gate(const void* o, const void* gate, long long gate_stride, void* out, long long tokens, int H, int dv, int D, int fp32,
+                              void* stream_ptr) {
+  if (tokens <= 0) return 0;
+  if (H < 1 || dv < 1 || D < dv || gate_stride < H || gate == nullptr) return -3;
+  cudaStream_t stream = reinterpret_cast<cudaStream_t>(stream_ptr);
+  const bool vec = dv % 4 == 0 && D % 4 == 0 && aligned(o, 16) && aligned(out, 16);
+  const int v = vec && !fp32 && dv % 8 == 0 && D % 8 == 0 ? 8 : vec ? 4 : 1;
+  const int blocks = (H * dv + 256 * v - 1) / (256 * v);
+  if (blocks > 65535) return -3;
+  const dim3 grid(static_cast<unsigned>(tokens), blocks);
+#define DEWB_GATE(TT, VV) head_gate_kernel<TT, VV><<<grid, 256, 0, stream>>>(static_cast<const TT*>(o), static_cast<const TT*>(gate), gate_stride,     static_cast<TT*>(out), H, dv, D)
+  if (fp32) { if (v == 4) DEWB_GATE(float, 4); else DEWB_GATE(float, 1); }
+  else { if (v == 8) DEWB_GATE(bf16, 8); else if (v == 4) DEWB_GATE(bf16, 4); else DEWB_GATE(bf16, 1); }
+#undef DEWB_GATE
+  return static_cast<int>(cudaGetLastError());
+}
+
+// `chunk` 0, `sinks` null, `gate` null: off (see Extras).
+extern "C" int dewb_paged_attend(const void* q, long long q_token_stride, const void* kpool, const void* vpool, const int* positions, int R, int S,
+                                 int H, int G, int dk, int dv, int D, float scale, int chunk, const float* sinks, const void* gate,
+                                 long long gate_stride, void* out, const int* page_table, int page_size, int max_pages, const int* row_ids, int fp32,
+                                 void* stream_ptr) {
+  if (R <= 0 || S <= 0) return 0;
+  if (H < 1 || G < 1 || H % G || dk < 1 || dv < 1 || D < dk || D < dv || page_size < 1 || max_pages < 1 || chunk < 0) return -3;
+  cudaStream_t stream = reinterpret_cast<cudaStream_t>(stream_ptr);
+  const Pool pool{page_table, page_size, max_pages, row_ids};
+  if (fp32) return attend_any<float>(q, q_token_stride, kpool, vpool, positions, R, S, H, G, dk, dv, D, scale, out, pool, chunk, sinks, gate, gate_stride, stream);
+  return attend_any<bf16>(q, q_token_stride, kpool, vpool, positions, R, S, H, G, dk, dv, D, scale, out, pool, chunk, sinks, gate, gate_stride, stream);
 }
 
 // The tensor-core form (bf16; pools D = 64, 128 or 256 wide; q on 16-byte boundaries with a token stride of a multiple of 8).
 extern "C" int dewb_paged_attend_mma(const void* q, long long q_token_stride, const void* kpool, const void* vpool, const int* positions, int R, int S,
-                                     int H, int G, int dv, int D, float scale, void* out, const int* page_table, int page_size, int max_pages,
-                                     const int* row_ids, void* stream_ptr) {
+                                     int H, int G, int dv, int D, float scale, int chunk, const float* sinks, const void* gate, long long gate_stride,
+                                     void* out, const int* page_table, int page_size, int max_pages, const int* row_ids, void* stream_ptr) {
   if (R <= 0 || S <= 0) return 0;
-  if (H < 1 || G < 1 || H % G || dv < 1 || D < dv || page_size < 1 || max_pages < 1 || q_token_stride % 8 || !aligned(q, 16) || !aligned(kpool, 16) ||
+  if (H < 1 || G < 1 || H % G || dv < 1 || D < dv || page_size < 1 || max_pages < 1 || chunk < 0 || q_token_stride % 8 || !aligned(q, 16) || !aligned(kpool, 16) ||
       !aligned(vpool, 16))
     return -3;
   cudaStream_t stream = reinterpret_cast<cudaStream_t>(stream_ptr);
   const Pool pool{page_table, page_size, max_pages, row_ids};
   const bf16 *qp = static_cast<const bf16*>(q), *kp = static_cast<const bf16*>(kpool), *vp = static_cast<const bf16*>(vpool);
   bf16* op = static_cast<bf16*>(out);
-  if (D == 64) return attend_mma<64>(qp, q_token_stride, kp, vp, positions, R, S, H, G, dv, scale, op, pool, stream);
-  if (D == 128) return attend_mma<128>(qp, q_token_stride, kp, vp, positions, R, S, H, G, dv, scale, op, pool, stream);
-  if (D == 256) return attend_mma<256>(qp, q_token_stride, kp, vp, positions, R, S, H, G, dv, scale, op, pool, stream);
+  const Extras<bf16> ex{chunk, sinks, static_cast<const bf16*>(gate), gate_stride};
+  if (D == 64) return attend_mma<64>(qp, q_token_stride, kp, vp, positions, R, S, H, G, dv, scale, op, pool, ex, stream);
+  if (D == 128) return attend_mma<128>(qp, q_token_stride, kp, vp, positions, R, S, H, G, dv, scale, op, pool, ex, stream);
+  if (D == 256) return attend_mma<256>(qp, q_token_stride, kp, vp, positions, R, S, H, G, dv, scale, op, pool, ex, stream);
   return -3;
 }

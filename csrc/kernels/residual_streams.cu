@@ -4,9 +4,12 @@
 //   embed_streams   H[t, s, :] = embed[token t] (+ pos[position t]) for every stream s
 //   stream_step     one residual step between two sub-layers: the pending write of the sub-layer that just ran
 //                       H'[t] = sum_s mix[s, t] H[s] + out[t] * (scale . y)
-//                   (in place), the read of the next one, u = sum_s read[s] H'[s], and its norm (layer norm without a bias, or RMS norm)
+//                   (in place), the read of the next one, u = sum_s read[s] H'[s], and its norm (layer norm without a bias, or RMS norm);
+//                   y may pass an RMS norm of its own first (a block that normalises what its sub-layers return).  Without connection
+//                   weights the streams keep themselves and take y as it is: one such stream is the ordinary fp32 residual.
 //   clamped_glu     g sigmoid(alpha g) (u + 1) with g = min(gate, limit), u = clamp(up, -limit, limit)
 //   sigmoid_gated_norm   RMS norm over a whole row times a weight times sigmoid(gate)
+//   softcap         cap tanh(x / cap), fp32 out (logits)
 //
 // Activations are bf16 or fp32 (template T); the streams, the connection weights and every sum are fp32.  Compiled without fast math.
 #include <cstdint>
@@ -45,20 +48,32 @@ embed_streams_kernel(const long long* __restrict__ tokens, const int* __restrict
 // NS: the number of streams when it is small and known (registers sized for it), 0: any number up to MAX_STREAMS.
 template <typename T, int V, int NS>
 __global__ void __launch_bounds__(THREADS)
-stream_step_kernel(float* __restrict__ H, const T* __restrict__ y, const T* __restrict__ scale, const float* __restrict__ mix,
-                   const float* __restrict__ out, const float* __restrict__ read, const T* __restrict__ w, T* __restrict__ normed,
-                   int n_rt, int d, float eps, int rms) {
+stream_step_kernel(float* __restrict__ H, const T* __restrict__ y, const T* __restrict__ y_weight, const T* __restrict__ scale,
+                   const float* __restrict__ mix, const float* __restrict__ out, const float* __restrict__ read, const T* __restrict__ w,
+                   T* __restrict__ normed, int n_rt, int d, float y_eps, float eps, int rms) {
   constexpr int NM = NS ? NS : MAX_STREAMS;
   const int n = NS ? NS : n_rt;
-  extern __shared__ float su[];                      // u of this token
+  extern __shared__ float su[];                      // y, then u of this token
   __shared__ float s_mix[MAX_STREAMS * MAX_STREAMS], s_out[MAX_STREAMS], s_read[MAX_STREAMS], red[32];
   const long long t = blockIdx.x;
   if (y != nullptr) {
-    for (int i = threadIdx.x; i < n * n; i += THREADS) s_mix[i] = mix[i];
-    for (int i = threadIdx.x; i < n; i += THREADS) s_out[i] = out[i];
+    for (int i = threadIdx.x; i < n * n; i += THREADS) s_mix[i] = mix == nullptr ? (i % (n + 1) == 0 ? 1.f : 0.f) : mix[i];
+    for (int i = threadIdx.x; i < n; i += THREADS) s_out[i] = out == nullptr ? 1.f : out[i];
   }
-  for (int i = threadIdx.x; i < n; i += THREADS) s_read[i] = read[i];
+  for (int i = threadIdx.x; i < n; i += THREADS) s_read[i] = read == nullptr ? 1.f : read[i];
   __syncthreads();
+  float ry = 1.f;
+  if (y_weight != nullptr) {
+    float ss = 0.f;
+    for (int i = threadIdx.x * V; i < d; i += THREADS * V) {
+      float a[V];
+      load_v<V>(y + t * d + i, a);
+#pragma unroll
+      for (int j = 0; j < V; ++j) ss += a[j] * a[j];
+      store_v<V>(su + i, a);                         // this thread reads it back, and puts u there
+    }
+    ry = 1.f / sqrtf(block_sum(ss, red) / d + y_eps);
+  }
   float* Ht = H + t * n * d;
   float sum = 0.f;
   for (int i = threadIdx.x * V; i < d; i += THREADS * V) {
@@ -70,7 +85,15 @@ stream_step_kernel(float* __restrict__ H, const T* __restrict__ y, const T* __re
     for (int j = 0; j < V; ++j) u[j] = 0.f;
     if (y != nullptr) {
       float b[V];
-      load_v<V>(y + t * d + i, b);
+      if (y_weight != nullptr) {
+        float c[V];
+        load_v<V>(su + i, b);
+        load_v<V>(y_weight + i, c);
+#pragma unroll
+        for (int j = 0; j < V; ++j) b[j] = b[j] * ry * c[j];
+      } else {
+        load_v<V>(y + t * d + i, b);
+      }
       if (scale != nullptr) {
         float c[V];
         load_v<V>(scale + i, c);
@@ -179,6 +202,20 @@ sigmoid_gated_norm_kernel(const T* __restrict__ x, const T* __restrict__ gate, c
   }
 }
 
+// grid (rows, ceil(n / (THREADS V)))
+template <typename T, int V>
+__global__ void __launch_bounds__(THREADS)
+softcap_kernel(const T* __restrict__ x, float* __restrict__ out, int n, float cap) {
+  const int i = (blockIdx.y * THREADS + threadIdx.x) * V;
+  if (i >= n) return;
+  const long long at = static_cast<long long>(blockIdx.x) * n + i;
+  float a[V];
+  load_v<V>(x + at, a);
+#pragma unroll
+  for (int j = 0; j < V; ++j) a[j] = cap * tanhf(a[j] / cap);
+  store_v<V>(out + at, a);
+}
+
 template <typename K>
 int allow_smem(K kernel, size_t bytes) {
   if (bytes <= 48 * 1024) return 0;
@@ -187,13 +224,13 @@ int allow_smem(K kernel, size_t bytes) {
 }
 
 template <typename T>
-int step(float* H, const T* y, const T* scale, const float* mix, const float* out, const float* read, const T* w, T* normed, long long rows,
-         int n, int d, float eps, int rms, cudaStream_t stream) {
-  const bool vec = d % 4 == 0 && aligned(H, 16) && aligned(y, 4 * sizeof(T)) && aligned(scale, 4 * sizeof(T)) && aligned(w, 4 * sizeof(T)) &&
+int step(float* H, const T* y, const T* y_weight, const T* scale, const float* mix, const float* out, const float* read, const T* w, T* normed,
+         long long rows, int n, int d, float y_eps, float eps, int rms, cudaStream_t stream) {
+  const bool vec = d % 4 == 0 && aligned(H, 16) && aligned(y, 4 * sizeof(T)) && aligned(y_weight, 4 * sizeof(T)) && aligned(scale, 4 * sizeof(T)) && aligned(w, 4 * sizeof(T)) &&
                    aligned(normed, 4 * sizeof(T));
   const size_t smem = static_cast<size_t>(d) * 4;
 #define DEWB_STEP(VV, NN) do { const int r = allow_smem(stream_step_kernel<T, VV, NN>, smem); if (r) return r; \
-    stream_step_kernel<T, VV, NN><<<static_cast<unsigned>(rows), THREADS, smem, stream>>>(H, y, scale, mix, out, read, w, normed, n, d, eps, rms); } while (0)
+    stream_step_kernel<T, VV, NN><<<static_cast<unsigned>(rows), THREADS, smem, stream>>>(H, y, y_weight, scale, mix, out, read, w, normed, n, d, y_eps, eps, rms); } while (0)
   if (vec) {
     if (n == 1) DEWB_STEP(4, 1); else if (n == 2) DEWB_STEP(4, 2); else if (n == 3) DEWB_STEP(4, 3); else if (n == 4) DEWB_STEP(4, 4); else DEWB_STEP(1, 0);
   } else {
@@ -224,16 +261,34 @@ extern "C" int dewb_embed_streams(const long long* tokens, const int* positions,
   return static_cast<int>(cudaGetLastError());
 }
 
-// H [rows, n, d] fp32, updated in place when `y` [rows, d] is given; normed [rows, d] (null: write only).  mix is indexed [from, to].
-extern "C" int dewb_stream_step(float* H, const void* y, const void* scale, const float* mix, const float* out, const float* read, const void* w,
-                                void* normed, long long rows, int n, int d, float eps, int rms, int fp32, void* stream_ptr) {
+// H [rows, n, d] fp32, updated in place when `y` [rows, d] is given; normed [rows, d] (null: write only).  mix is indexed [from, to].  `mix`, `out`
+// and `read` may be null (each stream keeps itself, takes y, and is read with weight 1); y_weight [d]: y passes an RMS norm with that weight first.
+extern "C" int dewb_stream_step(float* H, const void* y, const void* y_weight, const void* scale, const float* mix, const float* out,
+                                const float* read, const void* w, void* normed, long long rows, int n, int d, float y_eps, float eps, int rms,
+                                int fp32, void* stream_ptr) {
   if (rows <= 0) return 0;
-  if (n < 1 || n > MAX_STREAMS || d < 1 || read == nullptr || (y != nullptr && (mix == nullptr || out == nullptr)) || (normed != nullptr && w == nullptr)) return -3;
+  if (n < 1 || n > MAX_STREAMS || d < 1 || (y == nullptr && y_weight != nullptr) || (normed != nullptr && w == nullptr)) return -3;
   cudaStream_t stream = reinterpret_cast<cudaStream_t>(stream_ptr);
-  if (fp32) return step<float>(H, static_cast<const float*>(y), static_cast<const float*>(scale), mix, out, read, static_cast<const float*>(w),
-                               static_cast<float*>(normed), rows, n, d, eps, rms, stream);
-  return step<bf16>(H, static_cast<const bf16*>(y), static_cast<const bf16*>(scale), mix, out, read, static_cast<const bf16*>(w),
-                    static_cast<bf16*>(normed), rows, n, d, eps, rms, stream);
+  if (fp32) return step<float>(H, static_cast<const float*>(y), static_cast<const float*>(y_weight), static_cast<const float*>(scale), mix, out, read,
+                               static_cast<const float*>(w), static_cast<float*>(normed), rows, n, d, y_eps, eps, rms, stream);
+  return step<bf16>(H, static_cast<const bf16*>(y), static_cast<const bf16*>(y_weight), static_cast<const bf16*>(scale), mix, out, read,
+                    static_cast<const bf16*>(w), static_cast<bf16*>(normed), rows, n, d, y_eps, eps, rms, stream);
+}
+
+// x [rows, n] -> out [rows, n] fp32
+extern "C" int dewb_softcap(const void* x, float* out, long long rows, int n, float cap, int fp32, void* stream_ptr) {
+  if (rows <= 0) return 0;
+  if (n < 1 || !(cap > 0.f)) return -3;
+  cudaStream_t stream = reinterpret_cast<cudaStream_t>(stream_ptr);
+  const int v = n % 4 == 0 && aligned(x, 16) && aligned(out, 16) ? 4 : 1;
+  const int blocks = (n + THREADS * v - 1) / (THREADS * v);
+  if (blocks > 65535) return -3;
+  const dim3 grid(static_cast<unsigned>(rows), blocks);
+#define DEWB_CAP(TT, VV) softcap_kernel<TT, VV><<<grid, THREADS, 0, stream>>>(static_cast<const TT*>(x), out, n, cap)
+  if (fp32) { if (v == 4) DEWB_CAP(float, 4); else DEWB_CAP(float, 1); }
+  else { if (v == 4) DEWB_CAP(bf16, 4); else DEWB_CAP(bf16, 1); }
+#undef DEWB_CAP
+  return static_cast<int>(cudaGetLastError());
 }
 
 // gu [rows, 2 F] (gate half, then linear half) -> out [rows, F]

@@ -151,9 +151,10 @@ class Pretrained:
     def load(directory: os.PathLike, dtype=None, device="cpu", strict: bool = True):
         """A ``CausalTransformer`` for the families of ``interop.families``; a ``ClassicDecoder`` for the older lineage of
         ``interop.classic`` (GPT-2, GPT-NeoX, Falcon, Phi, OPT, BLOOM, StarCoder2, GPTBigCode); Mamba and Mamba-2 releases through
-        ``interop.recurrent``; Ragenex through ``interop.ragenex``."""
+        ``interop.recurrent``; Ragenex and Fakonex through ``interop.ragenex`` and ``interop.fakonex``."""
         from .classic import CLASSIC, load_classic_state, read_classic_config
         from .families import family_of, load_state, read_config
+        from .fakonex import is_fakonex, load_fakonex_state, read_fakonex_config
         from .ragenex import is_ragenex, load_ragenex_state, read_ragenex_config
         from .release import GenerationConfig, Release
         rel = Release(directory, dtype=dtype or torch.bfloat16)
@@ -165,12 +166,14 @@ class Pretrained:
             model.generation_config = GenerationConfig.read(directory)
             model.family = fam.name
             return model
-        if is_ragenex(rel.config):
-            model = CausalTransformer(read_ragenex_config(rel.config), dtype=dtype, device=device)
-            model.unread_keys = load_ragenex_state(model, rel, strict=strict)
-            model.generation_config = GenerationConfig.read(directory)
-            model.family = "ragenex"
-            return model
+        for name, mine, read, load in (("ragenex", is_ragenex, read_ragenex_config, load_ragenex_state),
+                                       ("fakonex", is_fakonex, read_fakonex_config, load_fakonex_state)):
+            if mine(rel.config):
+                model = CausalTransformer(read(rel.config), dtype=dtype, device=device)
+                model.unread_keys = load(model, rel, strict=strict)
+                model.generation_config = GenerationConfig.read(directory)
+                model.family = name
+                return model
         if str(rel.config.get("model_type") or "").lower() in ("mamba", "mamba2"):
             from .recurrent import load_recurrent_state, read_recurrent_config
             model = CausalTransformer(read_recurrent_config(rel.config), dtype=dtype, device=device)
@@ -191,11 +194,15 @@ class Pretrained:
         from .families import FAMILIES, export_state, write_config
         from .release import save_release
         dtype = str(next(model.parameters()).dtype).replace("torch.", "")
-        if family is None and getattr(model, "family", None) == "ragenex":
-            family = "ragenex"
+        if family is None and getattr(model, "family", None) in ("ragenex", "fakonex"):
+            family = model.family
         if family == "ragenex":
             from .ragenex import export_ragenex_state, write_ragenex_config
             save_release(export_ragenex_state(model), write_ragenex_config(model.config), directory, max_shard_bytes, generation, fp8_blocks)
+            return
+        if family == "fakonex":
+            from .fakonex import export_fakonex_state, write_fakonex_config
+            save_release(export_fakonex_state(model), write_fakonex_config(model.config), directory, max_shard_bytes, generation, fp8_blocks)
             return
         if family is None:
             family = next((f.name for f in FAMILIES.values() if f.architecture == architecture), None)

@@ -11,6 +11,7 @@ from typing import Any, Dict, List, Mapping, Tuple
 import torch
 
 from ..models.causal_transformer import CausalTransformer, Loop, TransformerConfig
+from .layouts import copy_tensors
 
 ARCHITECTURE = "Ragenex"
 KINDS = {"attention": "nope", "lightning": "lightning"}
@@ -113,20 +114,7 @@ def _without_feed_forward(model: CausalTransformer) -> Tuple[str, ...]:
 
 def load_ragenex_state(model: CausalTransformer, tensors: Mapping[str, torch.Tensor], strict: bool = True) -> List[str]:
     """Copy a release's tensors into ``model``; returns the names nothing read (raises on them with ``strict``)."""
-    read = set()
-    for p, names in _tensors(model):
-        parts = [tensors[n] for n in names]
-        t = parts[0] if len(parts) == 1 else torch.cat(parts, 0)
-        if tuple(t.shape) != tuple(p.shape):
-            raise ValueError(f"{' | '.join(names)}: shape {tuple(t.shape)} on disk does not fit the parameter's {tuple(p.shape)}")
-        with torch.no_grad():
-            p.copy_(t.to(p.dtype))
-        read.update(names)
-    spare = _without_feed_forward(model)
-    left = sorted(k for k in tensors if k not in read and not (spare and k.startswith(spare)))
-    if strict and left:
-        raise KeyError(f"{len(left)} tensor(s) of the release were not read: {left[:6]}")
-    return left
+    return copy_tensors(_tensors(model), tensors, strict, _without_feed_forward(model))
 
 
 def export_ragenex_state(model: CausalTransformer) -> Dict[str, torch.Tensor]:

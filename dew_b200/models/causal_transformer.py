@@ -22,7 +22,7 @@ import torch.utils.checkpoint as ckpt
 from .. import ops
 from ..ops import streams as ops_streams
 from ..nn.attention import SelfAttention
-from ..nn.kv_cache import CacheSlot
+from ..nn.kv_cache import CacheSlot, Uncached
 from ..nn.layers import Embedding, LayerNorm, Linear, RMSNorm, declare
 from ..nn.mlp import ClampedGLU, SwiGLU
 from ..utils.registry import register
@@ -48,6 +48,7 @@ class Mixture:
     balance_rate: float = 1e-3
     groups: int = 1                                  # DeepSeek-V3's group-limited routing: experts in ``groups`` groups ...
     topk_groups: int = 1                             # ... of which each token may use the ``topk_groups`` best (by their top-2 sum)
+    group_fill: float = 0.0                          # choice score of the experts outside those groups (choice scores can be negative: -inf rules them out)
     style: str = "swiglu"                            # 'clamped_glu': GPT-OSS's biased router over the top logits and biased clamped-GLU experts
 
 
@@ -126,22 +127,30 @@ class TransformerConfig:
     query_temperature: Optional[Sequence[float]] = None    # (coef, every): queries times 1 + coef ln(floor((p + 1) / every) + 1)
     value_dim: Optional[int] = None                   # width of a head's values where it differs from head_dim
     mlp_limit: float = 7.0                            # mlp_activation 'clamped_glu': the clamp of both halves
+    fp32_residual: bool = False                       # the residual is kept in fp32 and fused with the norms around it (one plain stream of the static-stream stack)
+    attn_chunk: Optional[int] = None                  # a query sees no key from before the start of its chunk of this many positions
+    attn_head_gate: bool = False                      # each head's output times the sigmoid of one number from the layer's input
+    kv_from: Optional[int] = None                     # (per layer) read that earlier layer's keys and values instead of projecting its own
     layer_options: Optional[Sequence[Optional[Mapping]]] = None    # per layer, what differs from the fields above: num_heads, num_kv_heads, head_dim, value_dim,
-                                                      # query_scale, query_temperature, decay (lightning), mlp_features, mlp_limit
+                                                      # query_scale, query_temperature, attn_chunk, kv_from, decay (lightning), mlp_features, mlp_limit, mixture
 
     def __post_init__(self):
         if self.norm not in ("rms", "layer"):
             raise ValueError(f"unknown norm {self.norm!r}; known: rms, layer")
         if self.layer_options is not None and len(self.layer_options) != self.num_layers:
             raise ValueError(f"layer_options describes {len(self.layer_options)} layers of {self.num_layers}")
-        if self.static_streams:
-            if self.altup > 1 or self.mixture is not None or self.sandwich_norm or not self.pre_norm or self.residual_multiplier != 1.0 or self.remat \
-                    or self.depth_residual_block or self.engram or self.mtp_depth:
-                raise NotImplementedError("static hyper-connections are built for pre-norm layers with dense MLPs, without rematerialisation, AltUp, block "
-                                          "attention residuals, n-gram memories and multi-token prediction")
+        if self.fp32_residual and self.hyper_connections:
+            raise ValueError("fp32_residual is the residual without connections: static hyper-connections already keep their streams in fp32")
+        if self.fp32_stack:
+            if self.altup > 1 or not self.pre_norm or self.residual_multiplier != 1.0 or self.remat or self.depth_residual_block or self.engram or self.mtp_depth \
+                    or self.logit_divisor != 1.0:
+                raise NotImplementedError("fp32 residual streams are built for pre-norm layers, without rematerialisation, AltUp, residual and logit factors, "
+                                          "block attention residuals, n-gram memories and multi-token prediction")
         elif self.norm != "rms" or self.layer_scale or self.learned_positions:
-            raise NotImplementedError("layer norms, layer scale and learned positions belong to the static-stream stack (hyper_connections >= 1, "
-                                      "hyper_dynamic=False)")
+            raise NotImplementedError("layer norms, layer scale and learned positions belong to the static-stream stack (hyper_connections >= 1 with "
+                                      "hyper_dynamic=False, or fp32_residual)")
+        if self.kv_from is not None and self.layer_options is not None:
+            raise ValueError("kv_from belongs to a layer: give it in layer_options")
         if isinstance(self.mixture, Mapping):             # a run record (JSON) carries the mixture as a plain mapping
             self.mixture = Mixture(**self.mixture)
         if isinstance(self.loop, Mapping):
@@ -151,12 +160,18 @@ class TransformerConfig:
     def static_streams(self) -> bool:
         return self.hyper_connections >= 1 and not self.hyper_dynamic
 
+    @property
+    def fp32_stack(self) -> bool:
+        """Whether the layers run over fp32 residual streams (``CausalTransformer._static``)."""
+        return self.static_streams or self.fp32_residual
+
     def of_layer(self, index: int) -> "TransformerConfig":
         """The configuration as layer ``index`` sees it."""
         o = self.layer_options[index] if self.layer_options is not None else None
         if not o:
             return self
-        own = {"num_heads", "num_kv_heads", "head_dim", "value_dim", "query_scale", "query_temperature", "mlp_features", "mlp_limit"}
+        own = {"num_heads", "num_kv_heads", "head_dim", "value_dim", "query_scale", "query_temperature", "attn_chunk", "kv_from", "mlp_features", "mlp_limit",
+               "mixture"}
         if set(o) - own - {"decay"}:
             raise ValueError(f"unknown layer option(s) {sorted(set(o) - own - {'decay'})}; known: {sorted(own | {'decay'})}")
         mixer = {k: o[k] for k in ("num_heads", "head_dim", "value_dim", "decay") if k in o} if self.kinds()[index] == "lightning" else {}
@@ -178,7 +193,8 @@ def _mixer(cfg: TransformerConfig, kind: str, dtype, device, index: int = 0) -> 
                           causal=cfg.causal, window=cfg.window if kind == "local" or cfg.layer_types is None else None, bias=cfg.attn_bias,
                           softcap=cfg.attn_softcap, sinks=cfg.attention_sinks, norm_eps=cfg.norm_eps,
                           init_std=cfg.init_std, qkv_bias=cfg.qkv_bias, scale=cfg.query_scale, qk_norm_full=cfg.qk_norm_full,
-                          out_gate=cfg.attn_out_gate, value_dim=cfg.value_dim, temperature=cfg.query_temperature, dtype=dtype, device=device)
+                          out_gate=cfg.attn_out_gate, value_dim=cfg.value_dim, temperature=cfg.query_temperature,
+                          chunk=cfg.attn_chunk, head_gate=cfg.attn_head_gate, own_kv=cfg.kv_from is None, dtype=dtype, device=device)
         a.rotary = kind != "nope"                        # SmolLM3's every fourth layer attends without positions
         if kind == "local" and cfg.local_rope_theta is not None:
             a.own_rope = (float(cfg.local_rope_theta), None)
@@ -253,7 +269,7 @@ class DecoderLayer(nn.Module):
         self.has_mlp = True if cfg.layer_mlp is None else bool(list(cfg.layer_mlp)[index % len(cfg.layer_mlp)])
         if kind == "none" and not self.has_mlp:
             raise ValueError(f"layer {index} has neither a mixer nor an MLP")
-        if (kind == "none" or not self.has_mlp) and (cfg.sandwich_norm or not cfg.pre_norm or (cfg.hyper_connections > 1 and cfg.hyper_dynamic) or cfg.altup > 1):
+        if (kind == "none" or not self.has_mlp) and ((cfg.sandwich_norm and not cfg.fp32_stack) or not cfg.pre_norm or (cfg.hyper_connections > 1 and cfg.hyper_dynamic) or cfg.altup > 1):
             raise NotImplementedError("layers of one sub-layer are built for the plain pre-norm block")
         self.input_norm = _norm_of(cfg, dtype, device) if cfg.pre_norm else _NoNorm()
         self.mixer = None if kind == "none" else _mixer(cfg, kind, dtype, device, index)
@@ -276,18 +292,19 @@ class DecoderLayer(nn.Module):
             self.mlp = SwiGLU(cfg.emb_features, cfg.mlp_features or 4 * cfg.emb_features, init_std=cfg.init_std,
                               activation=cfg.mlp_activation, dtype=dtype, device=device)
         self.sparse = sparse
-        self.mixer_out_norm = RMSNorm(cfg.emb_features, cfg.norm_eps, dtype=dtype, device=device) if cfg.sandwich_norm else None
-        self.mlp_out_norm = RMSNorm(cfg.emb_features, cfg.norm_eps, dtype=dtype, device=device) if cfg.sandwich_norm else None
+        out_norm = lambda there: RMSNorm(cfg.emb_features, cfg.norm_eps, dtype=dtype, device=device) if cfg.sandwich_norm and there else None
+        self.mixer_out_norm, self.mlp_out_norm = out_norm(self.mixer is not None), out_norm(self.has_mlp)
         self.tp = None          # set by parallel.tp.tensor_parallelize: branches are then partial sums over ranks
         self.cross = None       # set by the model for the layers of a loop with messages: one merge per sub-layer input
         self.residual_multiplier = float(cfg.residual_multiplier)
         self.streams = None
         self.layer_scale = None
-        if cfg.static_streams:
+        if cfg.fp32_stack:
             from ..nn.streams import HyperConnections
             subs = int(self.mixer is not None) + int(self.mlp is not None)
-            self.streams = nn.ModuleList([HyperConnections(cfg.emb_features, cfg.hyper_connections, 2 * index + j, dynamic=False, device=device)
-                                          for j in range(subs)])
+            if cfg.static_streams:
+                self.streams = nn.ModuleList([HyperConnections(cfg.emb_features, cfg.hyper_connections, 2 * index + j, dynamic=False, device=device)
+                                              for j in range(subs)])
             if cfg.layer_scale:
                 self.layer_scale = nn.ParameterList([declare(nn.Parameter(torch.ones(cfg.emb_features, dtype=dtype, device=device)), ("norm",), "scale")
                                                      for _ in range(subs)])
@@ -302,6 +319,8 @@ class DecoderLayer(nn.Module):
     def _mix(self, n, cos, sin, positions, segment_ids, cache, slot: Optional[int]):
         """The mixer on its normalised input; ``slot`` is the cache entry of this run of the layer (None: the layer's own index)."""
         slot = self.index if slot is None else slot
+        if getattr(cache, "uncached", False) and self.kind not in ROTARY_KINDS:
+            cache = None
         if self.kind in ROTARY_KINDS:
             return self.mixer(n, cos, sin, positions, segment_ids, cache, slot)
         if getattr(cache, "slots", None) is not None:
@@ -310,15 +329,22 @@ class DecoderLayer(nn.Module):
 
     def forward_static(self, stack, cos, sin, positions, segment_ids, cache, slot: int) -> None:
         """The layer over a ``StreamStack``: each sub-layer's write is fused with the next one's read and norm."""
-        scale = self.layer_scale if self.layer_scale is not None else [None] * len(self.streams)
+        scale = self.layer_scale if self.layer_scale is not None else [None, None]
+        streams = self.streams if self.streams is not None else [None, None]
         q = 0
         if self.mixer is not None:
-            n = stack.enter(self.streams[q], self.input_norm)
-            stack.leave(self.streams[q], self._mix(n, cos, sin, positions, segment_ids, cache, slot), scale[q])
+            n = stack.enter(streams[q], self.input_norm)
+            stack.leave(streams[q], self._mix(n, cos, sin, positions, segment_ids, cache, slot), scale[q], self.mixer_out_norm)
             q += 1
         if self.mlp is not None:
-            n = stack.enter(self.streams[q], self.input_norm if q == 0 else self.post_norm)
-            stack.leave(self.streams[q], self.mlp(n), scale[q])
+            n = stack.enter(streams[q], self.input_norm if q == 0 else self.post_norm)
+            stack.leave(streams[q], self._feed_forward(n, positions, True), scale[q], self.mlp_out_norm)
+
+    def _feed_forward(self, n, positions, serving: bool):
+        from ..nn.moe import SparseMLP
+        if isinstance(self.mlp, SparseMLP):
+            return self.mlp(n, serving=serving and self.tp is None, positions=positions)
+        return self.mlp(n)
 
     def forward_streams(self, H, cos, sin, positions, segment_ids, cache):
         """The layer over several residual streams ``H [B,S,n,d]``: each sub-layer reads its input from the streams, and its
@@ -376,7 +402,7 @@ class DecoderLayer(nn.Module):
         if self.residual_multiplier != 1.0:
             a = a * self.residual_multiplier
         n, h = self._norm(self.post_norm, h, a)
-        m = self.mlp(n)
+        m = self._feed_forward(n, positions, cache is not None)
         m = m if self.mlp_out_norm is None else self.mlp_out_norm(m)
         return h, (m if self.residual_multiplier == 1.0 else m * self.residual_multiplier)
 
@@ -411,6 +437,7 @@ class CausalTransformer(nn.Module):
         self.vocab_size = cfg.vocab_size
         self.embed = Embedding(cfg.vocab_size, cfg.emb_features, cfg.init_std, dtype=dtype, device=device)
         kinds = cfg.kinds()
+        self._check_shared_keys()
         self.position_embed = Embedding(cfg.max_seq_len, cfg.emb_features, cfg.init_std, dtype=dtype, device=device) if cfg.learned_positions else None
         self.layers = nn.ModuleList([DecoderLayer(cfg, i, k, dtype, device) for i, k in enumerate(kinds)])
         self.final_norm = _norm_of(cfg, dtype, device)
@@ -439,6 +466,21 @@ class CausalTransformer(nn.Module):
             self.engrams = nn.ModuleDict({str(i): Engram(cfg.emb_features, cfg.vocab_size, layer=i, norm_eps=cfg.norm_eps, dtype=dtype, device=device, **fields)
                                           for i in cfg.engram.get("layers", (0,))})
         self._rope = None
+
+    def _check_shared_keys(self) -> None:
+        """A layer with ``kv_from`` needs an earlier attention layer with keys of its own, of the same heads."""
+        cfg, kinds = self.config, self.config.kinds()
+        for i in range(cfg.num_layers):
+            mine = cfg.of_layer(i)
+            if mine.kv_from is None:
+                continue
+            j = mine.kv_from
+            if not (0 <= j < i) or kinds[i] != "nope" or kinds[j] != "nope" or not cfg.fp32_stack:
+                raise ValueError(f"layer {i} cannot read the keys and values of layer {j}")
+            theirs = cfg.of_layer(j)
+            shape = lambda c: (c.num_kv_heads or c.num_heads, c.head_dim or c.emb_features // c.num_heads, c.value_dim or c.head_dim or c.emb_features // c.num_heads)
+            if theirs.kv_from is not None or shape(mine) != shape(theirs):
+                raise ValueError(f"layer {i} reads the keys and values of layer {j}, which has none of its own with the same heads")
 
     def mtp_hiddens(self, hidden: torch.Tensor, tokens: torch.Tensor, segment_ids=None) -> List[torch.Tensor]:
         """Hidden states of the multi-token-prediction depths.  ``hidden [B,S,d]`` is the trunk's final hidden state for the
@@ -474,15 +516,17 @@ class CausalTransformer(nn.Module):
         """One entry per layer run where the layers differ in what they keep (heads of their own widths, recurrent states); None where one
         shape of keys and values serves them all."""
         cfg, kinds = self.config, self.config.kinds()
-        if not (cfg.static_streams or cfg.layer_options is not None or cfg.query_temperature is not None or cfg.value_dim is not None):
+        if not (cfg.fp32_stack or cfg.layer_options is not None or cfg.query_temperature is not None or cfg.value_dim is not None or cfg.attn_chunk is not None
+                or cfg.attn_head_gate):
             return None
         if any(k not in ("nope", "lightning", "none") for k in kinds):
             raise NotImplementedError(f"per-layer caches are built for attention without rotation ('nope') and 'lightning' layers, not {sorted(set(kinds))}")
-        out = []
-        for i, _ in self.runs():
+        out, latest = [], {}
+        for i, slot in self.runs():
             m = self.layers[i].mixer
             if kinds[i] == "nope":
-                out.append(CacheSlot(m.num_kv_heads, m.head_dim, m.value_dim))
+                out.append(CacheSlot(m.num_kv_heads, m.head_dim, m.value_dim, source=None if m.own_kv else latest[cfg.of_layer(i).kv_from]))
+                latest[i] = slot if m.own_kv else out[-1].source
             else:
                 out.append(CacheSlot(state=(0,) if m is None else (m.h, m.d, m.dv)))
         return out
@@ -602,7 +646,9 @@ class CausalTransformer(nn.Module):
                 positions = torch.arange(tokens.shape[1], device=tokens.device)[None].expand(tokens.shape[0], -1)
         if cache is not None and steps is not None and steps != cfg.loop.steps:
             raise NotImplementedError("the cache holds the configured number of passes")
-        H = ops_streams.embed_streams(tokens, positions, self.embed.weight, pos, cfg.hyper_connections)
+        if cache is None and any(self.layers[i].mixer is not None and not getattr(self.layers[i].mixer, "own_kv", True) for i, _ in runs):
+            cache = Uncached(self.cache_slots())
+        H = ops_streams.embed_streams(tokens, positions, self.embed.weight, pos, max(1, cfg.hyper_connections))
         stack = StreamStack(H, self.embed.weight.dtype)
         cos, sin = (None, None) if all(k not in ROTARY_KINDS or k == "nope" for k in cfg.kinds()) else self.rope_tables(H.device)
         for r, (i, slot) in enumerate(runs):
@@ -616,9 +662,9 @@ class CausalTransformer(nn.Module):
         """``embeddings [B, S, d]``: input embeddings computed by the caller (a vision-language model splices image features into the
         token embeddings); they replace the table lookup of ``tokens`` and are scaled like it."""
         cfg = self.config
-        if cfg.static_streams:
+        if cfg.fp32_stack:
             if segment_ids is not None or embeddings is not None or passes:
-                raise NotImplementedError("static hyper-connections run on token rows without packed segments, given embeddings or per-pass exits")
+                raise NotImplementedError("fp32 residual streams run on token rows without packed segments, given embeddings or per-pass exits")
             return self._static(tokens, positions, cache, loop_steps).finish(self.final_norm)
         h = self.embed(tokens) if embeddings is None else embeddings
         if cfg.embed_scale:
@@ -683,7 +729,7 @@ class CausalTransformer(nn.Module):
         if self.config.logit_divisor != 1.0:
             out = out / self.config.logit_divisor
         if self.config.logit_softcap > 0:
-            out = self.config.logit_softcap * torch.tanh(out.float() / self.config.logit_softcap)
+            out = ops_streams.softcap(out, self.config.logit_softcap)
         return out
 
     def next_tokens_greedy(self, hidden: torch.Tensor) -> torch.Tensor:
@@ -715,7 +761,7 @@ class CausalTransformer(nn.Module):
             bias = layer.mlp.router.expert_bias
             if bias is not None:
                 effects[f"layers.{i}.mlp.router.expert_bias"] = load_balance_update(
-                    bias, last["counts"], self.config.mixture.balance_rate).detach()
+                    bias, last["counts"], layer.mlp.mix.balance_rate).detach()
             layer.mlp.last = {}
         if not losses:
             return {}
@@ -726,12 +772,11 @@ class CausalTransformer(nn.Module):
     # ------------------------------------------------------------------ accounting
     def param_count(self, active: bool = False) -> int:
         total = sum(p.numel() for p in self.parameters())
-        if active and self.config.mixture is not None:
-            mix = self.config.mixture
+        if active:
             for layer in self.layers:
                 if layer.sparse:
                     per = layer.mlp.experts.param_count_per_expert()
-                    total -= per * (mix.experts - mix.top_k)
+                    total -= per * (layer.mlp.mix.experts - layer.mlp.mix.top_k)
         return total
 
     def model_flops(self, tokens: int, seq_len: int) -> float:
@@ -746,10 +791,8 @@ class CausalTransformer(nn.Module):
             if ".mlp.experts." in name or name == "tp_head":
                 continue
             matmul_params += p.numel()
-        mix = cfg.mixture
-        if mix is not None:
-            sparse_layers = sum(1 for layer in self.layers if layer.sparse)
-            matmul_params += sparse_layers * mix.top_k * 3 * cfg.emb_features * (mix.expert_features or cfg.mlp_features or 4 * cfg.emb_features)
+        for mix in (layer.mlp.mix for layer in self.layers if layer.sparse):
+            matmul_params += mix.top_k * 3 * cfg.emb_features * (mix.expert_features or cfg.mlp_features or 4 * cfg.emb_features)
         if not cfg.tie_embeddings:
             matmul_params -= self.embed.weight.numel()
         n_attn = sum(1 for k in cfg.kinds() if k in ("attention", "local"))

@@ -19,7 +19,8 @@ class SelfAttention(nn.Module):
                  qk_norm: bool = False, bias: bool = False, causal: bool = True, window: Optional[int] = None,
                  softcap: float = 0.0, sinks: bool = False, norm_eps: float = 1e-6, out_zero_init: bool = False,
                  init_std: Optional[float] = None, qkv_bias: bool = False, scale: Optional[float] = None, qk_norm_full: bool = False,
-                 out_gate: bool = False, value_dim: Optional[int] = None, temperature=None, dtype=None, device=None):
+                 out_gate: bool = False, value_dim: Optional[int] = None, temperature=None, chunk: Optional[int] = None, head_gate: bool = False,
+                 own_kv: bool = True, dtype=None, device=None):
         super().__init__()
         self.features, self.num_heads = features, num_heads
         # a softmax scale other than head_dim ** -0.5 is folded into the queries (after the norm and the rotation)
@@ -31,9 +32,15 @@ class SelfAttention(nn.Module):
         self.scale = float(scale) if scale is not None else self.head_dim ** -0.5
         # queries grow with the position: (coef, every) multiplies them by 1 + coef ln(floor((p + 1) / every) + 1)
         self.temperature = None if temperature is None else (float(temperature[0]), int(temperature[1]))
-        self.heads = P.Heads(self.num_heads, self.num_kv_heads, self.head_dim, self.value_dim)
-        qkv_out = self.heads.packed
-        self.qkv_proj = Linear(features, qkv_out, bias=bias or qkv_bias, axes=("embed", "heads"), init_std=init_std, dtype=dtype, device=device)
+        # a query sees no key from before the start of its chunk of positions; head_gate: each head's output times the sigmoid of one number from
+        # the layer's input (its rows stand last in the projection); own_kv False: the layer reads another layer's keys and values
+        self.chunk, self.head_gate, self.own_kv = chunk, head_gate, own_kv
+        self.heads = P.Heads(self.num_heads, self.num_kv_heads, self.head_dim, self.value_dim, own_kv, head_gate)
+        self.qkv_proj = Linear(features, self.heads.row, bias=(bias or qkv_bias) and not head_gate, axes=("embed", "heads"), init_std=init_std, dtype=dtype,
+                               device=device)
+        # the gates have no bias
+        self.heads_bias = declare(nn.Parameter(torch.zeros(self.heads.packed, dtype=dtype, device=device)), ("heads",), "bias") \
+            if (bias or qkv_bias) and head_gate else None
         self.o_proj = Linear(self.num_heads * self.value_dim, features, bias=bias, axes=("heads", "embed"),
                              init_std=init_std, zero_init=out_zero_init, dtype=dtype, device=device)
         # Qwen3-Next: the heads' outputs pass a sigmoid gate computed from the layer's input, before the output projection
@@ -42,7 +49,7 @@ class SelfAttention(nn.Module):
         self.qk_norm_full = qk_norm_full
         qw, kw = (self.num_heads * self.head_dim, self.num_kv_heads * self.head_dim) if qk_norm_full else (self.head_dim, self.head_dim)
         self.q_norm = RMSNorm(qw, norm_eps, dtype=dtype, device=device) if (qk_norm or qk_norm_full) else None
-        self.k_norm = RMSNorm(kw, norm_eps, dtype=dtype, device=device) if (qk_norm or qk_norm_full) else None
+        self.k_norm = RMSNorm(kw, norm_eps, dtype=dtype, device=device) if (qk_norm or qk_norm_full) and own_kv else None
         self.sinks = declare(nn.Parameter(torch.zeros(num_heads, dtype=dtype, device=device)), ("heads",), "sinks") if sinks else None
         # a layer whose rotary table differs from the model's: (theta, scaling) builds its own; rotary False drops the rotation (NoPE)
         self.rotary, self.own_rope, self._own = True, None, None
@@ -94,25 +101,27 @@ class SelfAttention(nn.Module):
         return self._own
 
     def _general(self, x, positions, segment_ids, cache, layer):
-        """Heads of any widths, the query temperature, and caches whose layers differ; no rotation."""
+        """Heads of any widths, the query temperature, chunks, head gates, layers that share keys and values, and caches whose layers differ; no
+        rotation."""
+        from .kv_cache import Uncached
         B, S, _ = x.shape
-        if self.rotary or self.window is not None or self.softcap or self.sinks is not None or self.gate_proj is not None or segment_ids is not None \
-                or not self.causal or (self.q_norm is not None and not self.qk_norm_full):
-            raise NotImplementedError("a query temperature, values of another width and per-layer caches are built for causal attention without "
-                                      "rotation, window, soft cap, sinks, output gate or packed segments, with q / k norms over all heads or none")
-        qw, kw, eps = (None, None, 0.0) if self.q_norm is None else (self.q_norm.weight, self.k_norm.weight, self.q_norm.eps)
-        qkv = self.qkv_proj(x)
-        if cache is not None:
-            o = cache.attend_slot(layer, qkv, self.heads, positions, scale=self.scale, eps=eps, q_weight=qw, k_weight=kw, temperature=self.temperature)
-        else:
-            pos = torch.arange(S, device=x.device)[None].expand(B, S) if positions is None else positions
-            q, k, v = P.prepare_reference(qkv, self.heads, qw, kw, eps, self.temperature, pos)
-            o = ops.attention(q, k, v, causal=True, scale=self.scale)
+        if self.rotary or self.window is not None or self.softcap or self.gate_proj is not None or segment_ids is not None or not self.causal:
+            raise NotImplementedError("a query temperature, values of another width, chunks, head gates, shared keys and per-layer caches are built for "
+                                      "causal attention without rotation, window, soft cap, a full-width output gate or packed segments")
+        qw, eps = (None, 0.0) if self.q_norm is None else (self.q_norm.weight, self.q_norm.eps)
+        kw = None if self.k_norm is None else self.k_norm.weight
+        # the bias joins in fp32 where the heads are normalised
+        qkv = ops.linear(x, self.qkv_proj.weight) if type(self.qkv_proj) is Linear and self.qkv_proj.bias is not None else self.qkv_proj(x)
+        bias = self.qkv_proj.bias if type(self.qkv_proj) is Linear and self.qkv_proj.bias is not None else self.heads_bias
+        cache = Uncached(()) if cache is None else cache
+        o = cache.attend_slot(layer, qkv, self.heads, positions, scale=self.scale, eps=eps, q_weight=qw, k_weight=kw, temperature=self.temperature,
+                              bias=bias, chunk=self.chunk, sinks=self.sinks)
         return self.o_proj(o.reshape(B, S, self.num_heads * self.value_dim))
 
     def forward(self, x, cos=None, sin=None, positions=None, segment_ids=None, cache=None, layer: int = 0):
         B, S, _ = x.shape
-        if getattr(cache, "slots", None) is not None or self.temperature is not None or self.value_dim != self.head_dim:
+        if getattr(cache, "slots", None) is not None or self.temperature is not None or self.value_dim != self.head_dim or self.chunk is not None \
+                or self.head_gate or not self.own_kv:
             return self._general(x, positions, segment_ids, cache, layer)
         cos, sin = self._tables(cos, sin)
         if (cache is None and x.is_cuda and cos is not None and self.head_transform is None and self.gate_proj is None and self.q_norm is None and self.window is None and not self.softcap

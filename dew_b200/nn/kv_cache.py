@@ -13,8 +13,8 @@ from __future__ import annotations
 import ctypes
 import math
 import os
-from dataclasses import dataclass
-from typing import List, Optional, Sequence, Tuple
+from dataclasses import dataclass, field
+from typing import Dict, List, Optional, Sequence, Tuple
 
 import torch
 
@@ -41,11 +41,13 @@ class KVCache:
 
 @dataclass(frozen=True)
 class CacheSlot:
-    """What one run of a layer keeps per row: keys and values of its own head count and widths, or a recurrent state (a shape, fp32)."""
+    """What one run of a layer keeps per row: keys and values of its own head count and widths, a recurrent state (a shape, fp32), or nothing: it
+    reads the keys and values of the earlier slot ``source``."""
     kv_heads: int = 0
     head_dim: int = 0
     value_dim: int = 0
     state: Optional[Tuple[int, ...]] = None
+    source: Optional[int] = None
 
 
 @dataclass
@@ -61,6 +63,7 @@ class Call:
     row_ids: Optional[torch.Tensor]          # int32 store row of each call row, None: the same
     table: torch.Tensor                      # int32 [R, max_pages]: the call rows' page tables
     fresh: Optional[bool] = None             # every row starts at its first token (None: not looked at)
+    kept: Dict[int, torch.Tensor] = field(default_factory=dict)      # slot -> this call's packed heads, while later layers read its keys and values
 
 
 def pool_width(slot: CacheSlot, dtype) -> int:
@@ -123,8 +126,17 @@ class KVStore:
         if self.slots is not None:
             if self.kind:
                 raise NotImplementedError("quantised storage is built for caches whose layers all keep the same heads")
-            pool = lambda s: None if s.state is not None else torch.zeros(self.pages + 1, self.page_size, s.kv_heads, pool_width(s, dtype), dtype=dtype, device=device)
+            for i, s in enumerate(self.slots):
+                if s.source is not None and not (0 <= s.source < i and self.slots[s.source].source is None and self.slots[s.source].state is None):
+                    raise ValueError(f"slot {i} reads the keys and values of slot {s.source}, which keeps none of its own before it")
+            pool = lambda s: None if s.state is not None or s.source is not None else \
+                torch.zeros(self.pages + 1, self.page_size, s.kv_heads, pool_width(s, dtype), dtype=dtype, device=device)
             self.k, self.v = [pool(s) for s in self.slots], [pool(s) for s in self.slots]
+            for pools in (self.k, self.v):
+                for i, s in enumerate(self.slots):
+                    if s.source is not None:
+                        pools[i] = pools[s.source]
+            self.last_reader = {s.source: i for i, s in enumerate(self.slots) if s.source is not None}
             self.states = [None if s.state is None else torch.zeros(rows, *s.state, dtype=torch.float32, device=device) for s in self.slots]
             self.k_scale = self.v_scale = None
         else:
@@ -170,43 +182,65 @@ class KVStore:
         return c.fresh
 
     def attend_slot(self, slot: int, qkv: torch.Tensor, heads: P.Heads, positions: torch.Tensor, *, scale: float, eps: float = 1e-6, q_weight=None,
-                    k_weight=None, temperature=None) -> torch.Tensor:
-        """A layer's attention from its packed projection ``qkv [R, S, H dk + G dk + G dv]``: norms, temperature, append, causal attention
-        against everything the rows hold.  -> ``[R, S, H, dv]``.  A prompt from its first token takes the tcgen05 flash kernel, a decode
-        step the paged decode kernels, anything else (and fp32) the general paged kernel."""
+                    k_weight=None, temperature=None, bias=None, chunk: Optional[int] = None, sinks: Optional[torch.Tensor] = None) -> torch.Tensor:
+        """A layer's attention from its packed projection ``qkv [R, S, heads.row]``: bias, norms, temperature, append, causal attention against
+        everything the rows hold (of a query's own ``chunk`` of positions, with ``sinks``, times the heads' gates).  -> ``[R, S, H, dv]``.  A
+        prompt from its first token takes the tcgen05 flash kernel, a decode step the paged decode kernels, anything else (and fp32) the
+        general paged kernel.  A slot with a source appends nothing and reads the source's keys and values."""
         c = self.call(positions)
+        source = self.slots[slot].source
+        if (source is None) != heads.own:
+            raise ValueError(f"slot {slot}: the layer and the cache disagree on whether it has keys and values of its own")
         pages = P.Pages(self.k[slot], self.v[slot], self.page_table, self.page_size, c.row_ids)
-        packed = P.qk_norm_append(qkv, heads, q_weight, k_weight, eps, temperature, c.positions, pages)
+        packed = P.qk_norm_append(qkv, heads, q_weight, k_weight, eps, temperature, c.positions, pages, bias)
+        gate = qkv[..., heads.packed:] if heads.gated else None
+        visible = P.Visible(chunk, None if sinks is None else self._fp32_sinks(slot, sinks))
         R, S = positions.shape
         H, G = heads.q, heads.kv
         D = packed.shape[-1]
         q = packed[:, :, :H]
         if L.use_cuda(qkv) and qkv.dtype == torch.bfloat16:
             if S == 1 and D in (64, 128, 256):
-                return self._decode_slot(slot, packed, heads, c, scale)[:, None, :, :heads.dv]
+                return P.head_gate(self._decode_slot(slot, packed, heads, c, scale, visible)[:, None], gate, heads.dv)
             if D in (64, 128) and S % 128 == 0 and self.is_fresh(c):
-                from ..ops.flash import flash_fwd
-                out, _ = flash_fwd(q, packed[:, :, H:H + G], packed[:, :, H + G:], True, scale, need_lse=False)
-                return out[..., :heads.dv]
-        return P.paged_attend(q, heads, c.positions, pages, scale)
+                from ..ops.flash import Variants, flash_fwd
+                if slot in self.last_reader:
+                    c.kept[slot] = packed[:, :, H:]
+                kv = packed[:, :, H:] if source is None else c.kept.get(source)
+                if source is not None and self.last_reader[source] == slot:
+                    c.kept.pop(source, None)
+                if kv is not None:
+                    out, _ = flash_fwd(q, kv[:, :, :G], kv[:, :, G:], True, scale, need_lse=False, var=Variants(sinks=visible.sinks, chunk=chunk))
+                    return P.head_gate(out, gate, heads.dv)
+        return P.paged_attend(q, heads, c.positions, pages, scale, visible=visible, gate=gate)
 
-    def _decode_slot(self, slot: int, packed: torch.Tensor, heads: P.Heads, c: Call, scale: float) -> torch.Tensor:
+    def _fp32_sinks(self, slot: int, sinks: torch.Tensor) -> torch.Tensor:
+        """A layer's sinks as the kernels take them, converted once (again when the parameter changes)."""
+        bank = self.__dict__.setdefault("_sinks_of", {})
+        key = (sinks.data_ptr(), sinks._version)
+        if slot not in bank or bank[slot][0] != key:
+            bank[slot] = (key, sinks.detach().float().contiguous())
+        return bank[slot][1]
+
+    def _decode_slot(self, slot: int, packed: torch.Tensor, heads: P.Heads, c: Call, scale: float, visible: P.Visible = P.PLAIN) -> torch.Tensor:
         lib = L.load()
         R, D, H, G = packed.shape[0], packed.shape[-1], heads.q, heads.kv
         out = torch.empty(R, H, D, dtype=packed.dtype, device=packed.device)
         if D == 128 and self.page_size % 64 == 0 and H // G <= 8 and hasattr(lib, "dewb_paged_decode_persist"):
-            self._fused_decode(lib, slot, packed, (H + 2 * G) * D, c.lengths, R, H, D, None, None, out, scale=scale, kv_heads=G, table=c.table)
+            self._fused_decode(lib, slot, packed, packed.shape[2] * D, c.lengths, R, H, D, None, visible.sinks, out, scale=scale, kv_heads=G, table=c.table,
+                               chunk=visible.chunk)
             return out
         q = packed[:, 0, :H].contiguous()
         share = next(s for s in range(1, H // G + 1) if (H // G) % s == 0 and H // G // s <= 8)     # CTAs that share a key / value head
-        splits = 1
-        while splits < 16 and R * G * share * splits < 592 and self.max_len // (splits * 2) >= 256:
+        splits, longest = 1, min(self.max_len, visible.chunk or self.max_len)
+        while splits < 16 and R * G * share * splits < 592 and longest // (splits * 2) >= 256:
             splits *= 2
         pm, pl, pa = self._partials(R * H * splits, D, q.device)
         L.check(lib.dewb_paged_decode(L.ptr(q), L.ptr(self.k[slot]), L.ptr(self.v[slot]), L.ptr(None), L.ptr(None), L.ptr(c.table), L.ptr(c.lengths),
-                                      L.ptr(None), L.ptr(out), L.ptr(None), L.ptr(pm), L.ptr(pl), L.ptr(pa), ctypes.c_int(R), ctypes.c_int(H),
+                                      L.ptr(visible.sinks), L.ptr(out), L.ptr(None), L.ptr(pm), L.ptr(pl), L.ptr(pa), ctypes.c_int(R), ctypes.c_int(H),
                                       ctypes.c_int(G), ctypes.c_int(share), ctypes.c_int(D), ctypes.c_int(self.page_size), ctypes.c_int(self.max_pages),
-                                      ctypes.c_int(splits), ctypes.c_float(scale), ctypes.c_int(0), ctypes.c_int(0), L.stream_ptr()), "paged_decode")
+                                      ctypes.c_int(splits), ctypes.c_float(scale), ctypes.c_int(0), ctypes.c_int(visible.chunk or 0), ctypes.c_int(0), L.stream_ptr()),
+                "paged_decode")
         L.count_launches(2)
         return out
 
@@ -311,18 +345,19 @@ class KVStore:
     MIN_TILES = 4            # fewest 64-key tiles one CTA of the balanced decode kernel takes (bounds the parts a row is cut into)
 
     def _fused_decode(self, lib, layer: int, q, q_row_stride: int, lens32, R: int, Hq: int, D: int, window, sinks32, out,
-                      scale: Optional[float] = None, kv_heads: Optional[int] = None, table: Optional[torch.Tensor] = None) -> None:
+                      scale: Optional[float] = None, kv_heads: Optional[int] = None, table: Optional[torch.Tensor] = None,
+                      chunk: Optional[int] = None) -> None:
         """The streamed paged-attention kernel finishing its rows itself.  Up to 1024 rows take the balanced persistent form
         (every CTA moves the same number of tiles, whatever the rows' lengths); more rows take one CTA per (row, head, chunk)."""
-        longest = min(self.max_len, window) if window else self.max_len
+        longest = min(self.max_len, window or self.max_len, chunk or self.max_len)
         max_tiles = -(-longest // 64) + 1                                 # (+ 1: a window that straddles a tile boundary)
         persist = R <= 1024 and os.environ.get("DEWB_DECODE_PERSIST", "1") == "1"
         if persist:
             min_tiles = int(os.environ.get("DEWB_DECODE_MIN_TILES", self.MIN_TILES))
             splits = (max_tiles - 1) // min_tiles + 2
         else:
-            chunk = 8
-            splits = max(1, -(-max_tiles // chunk))
+            share = 8                                                     # tiles a CTA takes
+            splits = max(1, -(-max_tiles // share))
         n = R * Hq * splits
         scale = 1.0 / math.sqrt(D) if scale is None else scale
         kv_heads = self.kv_heads if kv_heads is None else kv_heads
@@ -337,11 +372,11 @@ class KVStore:
             if getattr(self, "_ctas", None) is None:
                 self._ctas = 2 * torch.cuda.get_device_properties(q.device).multi_processor_count
             L.check(lib.dewb_paged_decode_persist(*common, ctypes.c_int(min_tiles), ctypes.c_float(scale),
-                                                  ctypes.c_int(window or 0), ctypes.c_longlong(q_row_stride), ctypes.c_int(self._ctas),
+                                                  ctypes.c_int(window or 0), ctypes.c_int(chunk or 0), ctypes.c_longlong(q_row_stride), ctypes.c_int(self._ctas),
                                                   L.ptr(L.status(q.device)), L.stream_ptr()), "paged_decode_persist")
         else:
-            L.check(lib.dewb_paged_decode_fused(*common, ctypes.c_int(chunk), ctypes.c_float(scale),
-                                                ctypes.c_int(window or 0), ctypes.c_longlong(q_row_stride),
+            L.check(lib.dewb_paged_decode_fused(*common, ctypes.c_int(share), ctypes.c_float(scale),
+                                                ctypes.c_int(window or 0), ctypes.c_int(chunk or 0), ctypes.c_longlong(q_row_stride),
                                                 L.ptr(L.status(q.device)), L.stream_ptr()), "paged_decode_fused")
         L.count_launches()
 
@@ -410,7 +445,7 @@ class KVStore:
                                                      ctypes.c_longlong(self.pages * self.page_size), L.ptr(self.page_table), L.ptr(lens32),
                                                      L.ptr(pm), L.ptr(pl), L.ptr(pa), ctypes.c_int(R), ctypes.c_int(Hq),
                                                      ctypes.c_int(self.kv_heads), ctypes.c_int(self.page_size), ctypes.c_int(self.max_pages),
-                                                     ctypes.c_int(splits), ctypes.c_float(scale), ctypes.c_int(window or 0),
+                                                     ctypes.c_int(splits), ctypes.c_float(scale), ctypes.c_int(window or 0), ctypes.c_int(0),
                                                      ctypes.c_longlong(0), L.ptr(L.status(q.device)), L.stream_ptr()), "paged_decode_stream")
                 L.check(lib.dewb_decode_combine(L.ptr(pm), L.ptr(pl), L.ptr(pa), L.ptr(sinks32),
                                                 L.ptr(out), L.ptr(None), ctypes.c_int(R), ctypes.c_int(Hq), ctypes.c_int(D), ctypes.c_int(splits),
@@ -424,7 +459,7 @@ class KVStore:
                                           L.ptr(pm), L.ptr(pl), L.ptr(pa), ctypes.c_int(R), ctypes.c_int(Hq),
                                           ctypes.c_int(self.kv_heads), ctypes.c_int(1), ctypes.c_int(D), ctypes.c_int(self.page_size),
                                           ctypes.c_int(self.max_pages), ctypes.c_int(splits), ctypes.c_float(scale),
-                                          ctypes.c_int(window or 0), ctypes.c_int(self.kind), L.stream_ptr()), "paged_decode")
+                                          ctypes.c_int(window or 0), ctypes.c_int(0), ctypes.c_int(self.kind), L.stream_ptr()), "paged_decode")
             L.count_launches(2)
             return out
         return paged_attention_reference(self, layer, q, lengths, scale, window, sinks, softcap)
@@ -457,6 +492,32 @@ class KVStore:
         kc, vc = self.gather(layer, total, dtype=q.dtype)
         # bottom-right aligned causal attention of the chunk against everything cached so far (rows share `start`)
         return ops.attention_reference(q, kc, vc, causal=causal, window=window, softcap=softcap, sinks=sinks)
+
+
+class Uncached:
+    """Stands where a cache would in a forward call over whole sequences: ``attend_slot`` in plain differentiable form, remembering the keys
+    and values that later layers read."""
+    uncached = True
+
+    def __init__(self, slots: Sequence[CacheSlot]):
+        self.slots = list(slots)
+        self.sources = {s.source for s in slots if s.source is not None}
+        self.source_of = [s.source for s in slots]
+        self.kept: Dict[int, Tuple[torch.Tensor, torch.Tensor]] = {}
+
+    def attend_slot(self, slot: int, qkv, heads: P.Heads, positions, *, scale: float, eps: float = 1e-6, q_weight=None, k_weight=None, temperature=None,
+                    bias=None, chunk: Optional[int] = None, sinks=None) -> torch.Tensor:
+        R, S, _ = qkv.shape
+        pos = torch.arange(S, device=qkv.device)[None].expand(R, S) if positions is None else positions
+        q, k, v = P.prepare_reference(qkv, heads, q_weight, k_weight, eps, temperature, pos, bias)
+        if not heads.own:
+            k, v = self.kept[self.source_of[slot]]
+        elif slot in self.sources:
+            self.kept[slot] = (k, v)
+        # chunks counted from the first position: documents of the packed-segment form, with ids that start at 1
+        segments = None if not chunk else (torch.arange(S, device=qkv.device, dtype=torch.int32) // chunk + 1)[None].expand(R, S).contiguous()
+        o = ops.attention(q, k, v, causal=True, scale=scale, sinks=sinks, segment_ids=segments)
+        return P.head_gate_reference(o, qkv[..., heads.packed:] if heads.gated else None, heads.dv)
 
 
 def paged_attention_reference(store: KVStore, layer: int, q, lengths, scale, window=None, sinks=None, softcap=0.0):

@@ -17,6 +17,7 @@ import torch.nn.functional as F
 
 from .. import ops
 from ..ops import grouped as G
+from ..ops import moe_serve as serve
 from .layers import Linear, declare
 from .mlp import SwiGLU
 
@@ -30,6 +31,7 @@ class Router(nn.Module):
     def __init__(self, features: int, mix, dtype=None, device=None):
         super().__init__()
         self.mix = mix
+        self._split = None
         self.weight = declare(nn.Parameter(torch.empty(mix.experts, features, dtype=dtype, device=device)), ("experts", "embed"), "kernel")
         self.register_buffer("expert_bias", torch.zeros(mix.experts, dtype=torch.float32, device=device) if mix.bias else None, persistent=True)
         self.reset_parameters()
@@ -42,25 +44,28 @@ class Router(nn.Module):
         """``x2 [T, d]`` -> (weights [T, k] fp32, expert ids [T, k], scores [T, E] fp32)."""
         mix = self.mix
         logits = F.linear(x2.float(), self.weight.float())
-        grouped = getattr(mix, "groups", 1) > 1
-        if logits.is_cuda and mix.experts <= 256 and mix.top_k <= 16 and self.use_kernels and not grouped:
+        if logits.is_cuda and mix.experts <= 256 and mix.top_k <= 16 and self.use_kernels and mix.groups <= 1:
             from ..ops.routing import route
             return route(logits, self.expert_bias, mix.top_k, mix.score_function, mix.norm_topk_prob, mix.scaling)
-        scores = torch.softmax(logits, -1) if mix.score_function == "softmax" else torch.sigmoid(logits)
-        select = scores + self.expert_bias if self.expert_bias is not None else scores     # bias steers selection only
-        if grouped:
-            # group-limited routing (DeepSeek-V3): a group's score is the sum of its two best experts; experts outside the
-            # token's best ``topk_groups`` groups cannot be chosen
-            T, E = select.shape
-            per = E // mix.groups
-            gscore = select.view(T, mix.groups, per).topk(min(2, per), -1).values.sum(-1)
-            keep = torch.zeros_like(gscore).scatter_(1, gscore.topk(mix.topk_groups, -1).indices, 1.0).bool()
-            select = select.masked_fill(~keep[:, :, None].expand(T, mix.groups, per).reshape(T, E), 0.0)
-        _, ids = torch.topk(select, mix.top_k, dim=-1)
-        w = scores.gather(-1, ids)
-        if mix.norm_topk_prob:
-            w = w / w.sum(-1, keepdim=True).clamp_min(1e-20)
-        return w * mix.scaling, ids, scores
+        # the bias steers the selection only; group-limited routing (DeepSeek-V3): a group's score is the sum of its two best experts, and
+        # experts outside the token's best ``topk_groups`` groups cannot be chosen
+        return serve.select_reference(logits, self.expert_bias, self.selection)
+
+    @property
+    def selection(self) -> serve.Selection:
+        m = self.mix
+        return serve.Selection(m.experts, m.top_k, m.groups, m.topk_groups, m.group_fill, m.score_function, m.norm_topk_prob, m.scaling)
+
+    def split(self) -> serve.Split:
+        """The weights as bf16 rows for the tensor cores, made once per value of the parameter."""
+        key = (self.weight.data_ptr(), self.weight._version)
+        if self._split is None or self._split[0] != key:
+            self._split = (key, serve.split_weights(self.weight))
+        return self._split[1]
+
+    def train(self, mode: bool = True):
+        self._split = None                # (kernels that update the weights in place do not count as a change of their version)
+        return super().train(mode)
 
 
 def load_balance_update(bias: torch.Tensor, counts: torch.Tensor, rate: float) -> torch.Tensor:
@@ -130,11 +135,29 @@ class SparseMLP(nn.Module):
         self.ep = None            # set by dew_b200.parallel.ep.ExpertParallel when the experts are sharded over ranks
         self._exchange = None     # this layer's single-rank token exchange (created on first use on a GPU)
 
-    def forward(self, x: torch.Tensor) -> torch.Tensor:
+    def _serves(self, x2: torch.Tensor) -> bool:
+        return (not torch.is_grad_enabled() and not self.training and self.use_kernels and self.ep is None and self.mix.capacity_factor is None
+                and not self.keep_router_outputs and not self.experts.fp8 and type(self.experts) is ExpertMLP
+                and (self.shared_gate is None or type(self.shared_gate) is Linear) and serve.usable(x2, self.router.selection))
+
+    def _serve(self, x2: torch.Tensor, positions: Optional[torch.Tensor]) -> torch.Tensor:
+        """Forward alone: no statistics, and no expert runs for tokens at positions below 0."""
+        pos = None if positions is None else positions.reshape(-1).to(torch.int32)
+        r = serve.route(x2, self.router.weight, self.router.split() if x2.dtype == torch.bfloat16 else None, self.router.expert_bias, self.router.selection, pos)
+        s = serve.gather(x2, r, None if self.shared_gate is None else self.shared_gate.weight)
+        y = serve.product(serve.glu(serve.product(s.rows, self.experts.gate_up, s), s), self.experts.down, s)
+        return serve.combine(y, r, s, None if self.shared is None else self.shared(x2))
+
+    def forward(self, x: torch.Tensor, serving: bool = False, positions: Optional[torch.Tensor] = None) -> torch.Tensor:
+        """``serving``: a step of generation; on a GPU outside autograd it takes the kernels of ``ops.moe_serve``, which skip the tokens at
+        ``positions`` below 0 (padding)."""
         mix = self.mix
         shape = x.shape
         x2 = x.reshape(-1, shape[-1])
         T = x2.shape[0]
+        if serving and self._serves(x2):
+            self.last = {}
+            return self._serve(x2, positions).reshape(shape)
         self.router.use_kernels = self.use_kernels
         w, ids, scores = self.router(x2)
         if mix.capacity_factor is not None:

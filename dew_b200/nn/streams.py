@@ -9,12 +9,15 @@ streams (initialised to zero, so training starts from the static form).
 ``AltUp`` (K blocks): predict every block from all blocks (``P`` [K x K], identity at start), run the layer on ONE block
 (``layer % K``), and correct every block by its gate times the layer's innovation on the active block.
 
-``StreamStack`` runs a stack of static hyper-connections (``dynamic=False``: the weights alone, no input-dependent part) over fp32 streams.
+``StreamStack`` runs a stack of static hyper-connections (``dynamic=False``: the weights alone, no input-dependent part) over fp32 streams;
+without connections (None) and with one stream it is an ordinary residual kept in fp32.
 
 A stack of either with one stream / block reduces to the ordinary pre-norm residual stack.
 Reference: ``hyper_connections`` and ``altup`` fields of src/dew/nn/backbones/causal_transformer.py:165-423.
 """
 from __future__ import annotations
+
+from typing import Optional
 
 import torch
 import torch.nn as nn
@@ -71,22 +74,23 @@ class StreamStack:
     def __init__(self, H: torch.Tensor, dtype):
         self.H, self.dtype, self.pending = H, dtype, None
 
-    def enter(self, connection: "HyperConnections", norm: nn.Module) -> torch.Tensor:
+    def enter(self, connection: Optional["HyperConnections"], norm: nn.Module) -> torch.Tensor:
         """The next sub-layer's normalised input."""
-        return self._step(connection.alpha, norm)
+        return self._step(None if connection is None else connection.alpha, norm)
 
-    def leave(self, connection: "HyperConnections", y: torch.Tensor, scale=None) -> None:
-        """The sub-layer's output (times its layer scale), to be written back by the connection."""
-        self.pending = S.Write(y, scale, connection.mix, connection.beta)
+    def leave(self, connection: Optional["HyperConnections"], y: torch.Tensor, scale=None, norm: Optional[nn.Module] = None) -> None:
+        """The sub-layer's output (through an RMS ``norm`` of its own, times its layer scale), to be written back by the connection."""
+        mix, out = (None, None) if connection is None else (connection.mix, connection.beta)
+        self.pending = S.Write(y, scale, mix, out, *((None, 0.0) if norm is None else (norm.weight, norm.eps)))
 
     def finish(self, norm: nn.Module) -> torch.Tensor:
         """The final norm of the sum of the streams."""
-        return self._step(torch.ones(self.H.shape[-2], device=self.H.device), norm)
+        return self._step(None, norm)
 
     def total(self) -> torch.Tensor:
         """The sum of the streams after everything so far."""
         if self.pending is not None:
-            _, self.H = S.stream_step(self.H, self.pending, self.pending.out, None, 0.0, self.dtype)
+            _, self.H = S.stream_step(self.H, self.pending, None, None, 0.0, self.dtype)
             self.pending = None
         return self.H.sum(-2)
 

@@ -88,7 +88,7 @@ def _tgmm_reference(dy, x, layout: GroupLayout, groups: int):
 
 def gmm_forward(x, w, layout: GroupLayout, transpose_w: bool = False, out=None):
     """``out[rows of g] = x[rows of g] @ w[g]^T`` (``w [G, N, K]``) or ``@ w[g]`` (``w [G, K, N]``, ``transpose_w``)."""
-    if not L.use_cuda(x, w):
+    if not L.use_cuda(x, w) or x.dtype != torch.bfloat16:
         return _gmm_reference(x, w, layout, transpose_w)
     G = w.shape[0]
     M, K = x.shape
@@ -106,7 +106,7 @@ def gmm_forward(x, w, layout: GroupLayout, transpose_w: bool = False, out=None):
 
 def tgmm(dy, x, layout: GroupLayout, groups: int, out: Optional[torch.Tensor] = None, accumulate: bool = False):
     """Per-group ``dW[g] = dy[rows of g]^T @ x[rows of g]`` -> ``[G, N, K]`` (fp32 when accumulating into ``out``)."""
-    if not L.use_cuda(dy, x):
+    if not L.use_cuda(dy, x) or x.dtype != torch.bfloat16:
         r = _tgmm_reference(dy, x, layout, groups)
         if out is not None:
             out.add_(r.to(out.dtype)) if accumulate else out.copy_(r.to(out.dtype))

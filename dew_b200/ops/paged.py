@@ -1,9 +1,10 @@
-"""Attention of a call's tokens against a paged cache of any head widths (``csrc/kernels/paged_attention.cu``) and the projection
-epilogue in front of it (norm over all heads, query temperature, append), each with its plain PyTorch form."""
+"""Attention of a call's tokens against a paged cache of any head widths (``csrc/kernels/paged_attention.cu``), the projection epilogue in
+front of it (bias, norm over all heads or per head, query temperature, append) and the head gate behind it, each with its plain PyTorch form."""
 from __future__ import annotations
 
 import ctypes
-from typing import NamedTuple, Optional
+from dataclasses import dataclass
+from typing import Iterator, NamedTuple, Optional
 
 import torch
 
@@ -12,16 +13,40 @@ from . import library as L
 c_ll, c_int, c_float = ctypes.c_longlong, ctypes.c_int, ctypes.c_float
 
 
-class Heads(NamedTuple):
-    """The shape of one attention layer: query heads, key / value heads, key width, value width."""
+@dataclass(frozen=True)
+class Heads:
+    """The shape of one attention layer: query heads, key / value heads, key width, value width; ``own``: it projects keys and values of its
+    own (else it reads another layer's); ``gated``: its projection ends in one gate per query head."""
     q: int
     kv: int
     dk: int
     dv: int
+    own: bool = True
+    gated: bool = False
+
+    def __iter__(self) -> Iterator[int]:
+        """The four sizes."""
+        return iter((self.q, self.kv, self.dk, self.dv))
 
     @property
     def packed(self) -> int:
-        return (self.q + self.kv) * self.dk + self.kv * self.dv
+        """Columns of the heads in the projection."""
+        return self.q * self.dk + (self.kv * (self.dk + self.dv) if self.own else 0)
+
+    @property
+    def row(self) -> int:
+        """Columns of the projection."""
+        return self.packed + (self.q if self.gated else 0)
+
+
+class Visible(NamedTuple):
+    """What a layer's attention adds to the causal softmax: a query sees no key from before the start of its ``chunk`` of positions; ``sinks``
+    (fp32, one per query head) join the denominator only."""
+    chunk: Optional[int] = None
+    sinks: Optional[torch.Tensor] = None
+
+
+PLAIN = Visible()
 
 
 class Pages(NamedTuple):
@@ -45,14 +70,29 @@ def rms_norm_fp32(x: torch.Tensor, w: Optional[torch.Tensor], eps: float) -> tor
     return xf / torch.sqrt(xf.pow(2).mean(-1, keepdim=True) + eps) * w.float()
 
 
-def prepare_reference(qkv, heads: Heads, qw, kw, eps: float, temperature, positions):
-    """``q [R, S, H, dk]``, ``k [R, S, G, dk]``, ``v [R, S, G, dv]`` after the norms and the temperature, in the projection's dtype."""
+def per_head(heads: Heads, qw, kw) -> bool:
+    """Whether the norms' weights are of one head (shared by all) rather than of all heads at once."""
+    return (qw is not None and qw.numel() != heads.q * heads.dk) or (kw is not None and kw.numel() != heads.kv * heads.dk)
+
+
+def prepare_reference(qkv, heads: Heads, qw, kw, eps: float, temperature, positions, bias=None):
+    """``q [R, S, H, dk]``, ``k [R, S, G, dk]``, ``v [R, S, G, dv]`` after the bias, the norms and the temperature, in the projection's dtype (keys and
+    values None for a layer without its own)."""
     R, S, _ = qkv.shape
-    q, k, v = qkv.split([heads.q * heads.dk, heads.kv * heads.dk, heads.kv * heads.dv], -1)
-    q, k = rms_norm_fp32(q, qw, eps), rms_norm_fp32(k, kw, eps)
+    one = per_head(heads, qw, kw)
+
+    def norm(t, n, w):
+        t = t.reshape(R, S, n, heads.dk) if one else t
+        return rms_norm_fp32(t, w, eps).reshape(R, S, n, heads.dk)
+    x = qkv[..., :heads.packed]
+    x = x if bias is None else x.float() + bias.float()
+    q = norm(x[..., :heads.q * heads.dk], heads.q, qw)
     if temperature is not None:
-        q = q * query_temperature(positions.clamp_min(0), temperature[0], temperature[1]).unsqueeze(-1)
-    return (q.to(qkv.dtype).view(R, S, heads.q, heads.dk), k.to(qkv.dtype).view(R, S, heads.kv, heads.dk), v.reshape(R, S, heads.kv, heads.dv))
+        q = q * query_temperature(positions.clamp_min(0), temperature[0], temperature[1])[..., None, None]
+    if not heads.own:
+        return q.to(qkv.dtype), None, None
+    k, v = x[..., heads.q * heads.dk:].split([heads.kv * heads.dk, heads.kv * heads.dv], -1)
+    return q.to(qkv.dtype), norm(k, heads.kv, kw).to(qkv.dtype), v.reshape(R, S, heads.kv, heads.dv).to(qkv.dtype)
 
 
 def _slots(pages: Pages, positions: torch.Tensor) -> torch.Tensor:
@@ -62,14 +102,26 @@ def _slots(pages: Pages, positions: torch.Tensor) -> torch.Tensor:
     return pages.table[rows[:, None], p // pages.page_size].long() * pages.page_size + p % pages.page_size
 
 
-def qk_norm_append(qkv, heads: Heads, qw, kw, eps: float, temperature, positions, pages: Pages) -> torch.Tensor:
+def qk_norm_append(qkv, heads: Heads, qw, kw, eps: float, temperature, positions, pages: Pages, bias=None) -> torch.Tensor:
     """-> ``[R, S, H + 2 G, D]`` (normalised queries and keys, values; every head padded with zeros to the pool's width), with the keys and
-    values of the live positions written to the pools.  ``positions`` int32 ``[R, S]``, below 0 = padding."""
+    values of the live positions written to the pools; ``[R, S, H, D]`` and nothing written for a layer without its own keys and values.
+    ``positions`` int32 ``[R, S]``, below 0 = padding."""
     R, S, _ = qkv.shape
     D = pages.k.shape[-1]
     if L.use_cuda(qkv):
         qkv = qkv.contiguous()
-        qw, kw = (None if w is None else w.detach().to(qkv.dtype).contiguous() for w in (qw, kw))
+        qw, kw, bias = (None if w is None else w.detach().to(qkv.dtype).contiguous() for w in (qw, kw, bias))
+        if per_head(heads, qw, kw) or bias is not None or not heads.own or heads.gated:
+            if temperature is not None or not (per_head(heads, qw, kw) or qw is None or heads.q == heads.kv == 1):
+                raise NotImplementedError("a projection with a bias, gates or queries alone is built for norms per head and without a query temperature")
+            G = heads.kv if heads.own else 0
+            packed = torch.empty(R, S, heads.q + 2 * G, D, dtype=qkv.dtype, device=qkv.device)
+            L.check(L.load().dewb_head_norm_append(L.ptr(qkv), c_ll(qkv.shape[-1]), L.ptr(bias), L.ptr(qw), L.ptr(kw), c_float(eps), L.ptr(positions), c_int(R),
+                                                   c_int(S), c_int(heads.q), c_int(G), c_int(heads.dk), c_int(heads.dv), c_int(D), L.ptr(packed),
+                                                   L.ptr(pages.k), L.ptr(pages.v), L.ptr(pages.table), c_int(pages.page_size), c_int(pages.table.shape[1]),
+                                                   L.ptr(pages.row_ids), c_int(int(qkv.dtype == torch.float32)), L.stream_ptr()), "head_norm_append")
+            L.count_launches()
+            return packed
         packed = torch.empty(R, S, heads.q + 2 * heads.kv, D, dtype=qkv.dtype, device=qkv.device)
         coef, every = temperature if temperature is not None else (0.0, 0)
         L.check(L.load().dewb_qk_norm_append(L.ptr(qkv), L.ptr(qw), L.ptr(kw), c_float(eps), c_float(coef), c_int(every), L.ptr(positions), c_int(R),
@@ -78,8 +130,10 @@ def qk_norm_append(qkv, heads: Heads, qw, kw, eps: float, temperature, positions
                                              L.ptr(pages.row_ids), c_int(int(qkv.dtype == torch.float32)), L.stream_ptr()), "qk_norm_append")
         L.count_launches()
         return packed
-    q, k, v = prepare_reference(qkv, heads, qw, kw, eps, temperature, positions)
+    q, k, v = prepare_reference(qkv, heads, qw, kw, eps, temperature, positions, bias)
     pad = lambda t: torch.nn.functional.pad(t, (0, D - t.shape[-1]))
+    if not heads.own:
+        return pad(q)
     q, k, v = pad(q), pad(k), pad(v)
     slots, live = _slots(pages, positions), positions >= 0
     for pool, t in ((pages.k, k), (pages.v, v)):
@@ -87,7 +141,22 @@ def qk_norm_append(qkv, heads: Heads, qw, kw, eps: float, temperature, positions
     return torch.cat([q, k, v], 2)
 
 
-def paged_attend_reference(q, heads: Heads, positions, pages: Pages, scale: float) -> torch.Tensor:
+def seen_keys(positions: torch.Tensor, n: int, chunk: Optional[int]) -> torch.Tensor:
+    """``[R, S, n]``: which of the first ``n`` positions a query at ``positions [R, S]`` sees."""
+    j = torch.arange(n, device=positions.device)[None, None]
+    seen = j <= positions[..., None]
+    return seen if not chunk else seen & (j >= (positions.clamp_min(0) // chunk * chunk)[..., None])
+
+
+def softmax_with_sinks(s: torch.Tensor, sinks: Optional[torch.Tensor]) -> torch.Tensor:
+    """Softmax over the last axis of ``s [R, H, S, n]`` with each head's sink in the denominator; rows that see nothing give zeros."""
+    if sinks is None:
+        return torch.nan_to_num(torch.softmax(s, -1))
+    sink = sinks.float().view(1, -1, 1, 1).expand(*s.shape[:3], 1)
+    return torch.softmax(torch.cat([s, sink], -1), -1)[..., :-1]
+
+
+def paged_attend_reference(q, heads: Heads, positions, pages: Pages, scale: float, visible: Visible = PLAIN) -> torch.Tensor:
     R, S = positions.shape
     D = pages.k.shape[-1]
     n = int(positions.max()) + 1
@@ -96,32 +165,57 @@ def paged_attend_reference(q, heads: Heads, positions, pages: Pages, scale: floa
     slots = _slots(pages, torch.arange(n, device=q.device)[None].expand(R, n))
     kc = pages.k.view(-1, heads.kv, D)[slots].float().repeat_interleave(heads.q // heads.kv, 2)          # [R, n, H, D]
     vc = pages.v.view(-1, heads.kv, D)[slots][..., :heads.dv].float().repeat_interleave(heads.q // heads.kv, 2)
-    seen = torch.arange(n, device=q.device)[None, None] <= positions[..., None]                          # [R, S, n]
+    seen = seen_keys(positions, n, visible.chunk)                                                        # [R, S, n]
     # what the pool holds beyond a row's own tokens is another row's, or nothing: it must not reach the sums
     own = (torch.arange(n, device=q.device)[None] <= positions.amax(1, keepdim=True))[..., None, None]
     kc, vc = torch.where(own, kc, torch.zeros_like(kc)), torch.where(own, vc, torch.zeros_like(vc))
     s = torch.einsum("rshd,rnhd->rhsn", q[..., :D].float(), kc) * scale
-    p = torch.nan_to_num(torch.softmax(s.masked_fill(~seen[:, None], float("-inf")), -1))
+    p = softmax_with_sinks(s.masked_fill(~seen[:, None], float("-inf")), visible.sinks)
     return torch.einsum("rhsn,rnhd->rshd", p, vc).to(q.dtype)
 
 
-def paged_attend(q: torch.Tensor, heads: Heads, positions: torch.Tensor, pages: Pages, scale: float, kernel: Optional[str] = None) -> torch.Tensor:
-    """``q [R, S, H, D]`` (a view into the packed tensor will do: unit stride in a head, heads next to each other) -> ``[R, S, H, dv]``.
-    ``kernel`` forces ``mma`` (bf16 pools of 64, 128, 256) or ``general``."""
+def head_gate_reference(o: torch.Tensor, gate: Optional[torch.Tensor], dv: int) -> torch.Tensor:
+    o = o[..., :dv]
+    return o if gate is None else (o.float() * torch.sigmoid(gate.float()).unsqueeze(-1)).to(o.dtype)
+
+
+def head_gate(o: torch.Tensor, gate: Optional[torch.Tensor], dv: int) -> torch.Tensor:
+    """``o [..., H, D]`` times the sigmoid of ``gate [..., H]`` (columns of the projection will do), cut to ``dv`` values a head."""
+    if gate is None or not L.use_cuda(o):
+        return head_gate_reference(o, gate, dv)
+    o = o.contiguous()
+    H, D = o.shape[-2:]
+    tokens = o.numel() // (H * D)
+    if gate.stride(-1) != 1 or any(gate.shape[i] > 1 and gate.stride(i) != gate.stride(i + 1) * gate.shape[i + 1] for i in range(gate.dim() - 2)):
+        gate = gate.contiguous()
+    out = torch.empty(*o.shape[:-1], dv, dtype=o.dtype, device=o.device)
+    L.check(L.load().dewb_head_gate(L.ptr(o), L.ptr(gate), c_ll(gate.stride(-2)), L.ptr(out), c_ll(tokens), c_int(H), c_int(dv), c_int(D),
+                                    c_int(int(o.dtype == torch.float32)), L.stream_ptr()), "head_gate")
+    L.count_launches()
+    return out
+
+
+def paged_attend(q: torch.Tensor, heads: Heads, positions: torch.Tensor, pages: Pages, scale: float, kernel: Optional[str] = None,
+                 visible: Visible = PLAIN, gate: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """``q [R, S, H, D]`` (a view into the packed tensor will do: unit stride in a head, heads next to each other) -> ``[R, S, H, dv]``, times the
+    sigmoid of ``gate [R, S, H]`` where given.  ``kernel`` forces ``mma`` (bf16 pools of 64, 128, 256) or ``general``."""
     if not L.use_cuda(q):
-        return paged_attend_reference(q, heads, positions, pages, scale)
+        return head_gate_reference(paged_attend_reference(q, heads, positions, pages, scale, visible), gate, heads.dv)
     R, S, H, D = q.shape
     if q.stride(3) != 1 or q.stride(2) != D or (R > 1 and q.stride(0) != S * q.stride(1)):
         q = q.contiguous()
     out = torch.empty(R, S, H, heads.dv, dtype=q.dtype, device=q.device)
+    if gate is not None and (gate.stride(2) != 1 or (R > 1 and gate.stride(0) != S * gate.stride(1))):
+        gate = gate.contiguous()
+    extras = (c_int(visible.chunk or 0), L.ptr(visible.sinks), L.ptr(gate), c_ll(0 if gate is None else gate.stride(1)))
     if (kernel or ("mma" if q.dtype == torch.bfloat16 and D in (64, 128, 256) else "general")) == "mma":
         L.check(L.load().dewb_paged_attend_mma(L.ptr(q), c_ll(q.stride(1)), L.ptr(pages.k), L.ptr(pages.v), L.ptr(positions), c_int(R), c_int(S), c_int(H),
-                                               c_int(heads.kv), c_int(heads.dv), c_int(D), c_float(scale), L.ptr(out), L.ptr(pages.table),
+                                               c_int(heads.kv), c_int(heads.dv), c_int(D), c_float(scale), *extras, L.ptr(out), L.ptr(pages.table),
                                                c_int(pages.page_size), c_int(pages.table.shape[1]), L.ptr(pages.row_ids), L.stream_ptr()), "paged_attend_mma")
         L.count_launches()
         return out
     L.check(L.load().dewb_paged_attend(L.ptr(q), c_ll(q.stride(1)), L.ptr(pages.k), L.ptr(pages.v), L.ptr(positions), c_int(R), c_int(S), c_int(H),
-                                       c_int(heads.kv), c_int(heads.dk), c_int(heads.dv), c_int(D), c_float(scale), L.ptr(out), L.ptr(pages.table),
+                                       c_int(heads.kv), c_int(heads.dk), c_int(heads.dv), c_int(D), c_float(scale), *extras, L.ptr(out), L.ptr(pages.table),
                                        c_int(pages.page_size), c_int(pages.table.shape[1]), L.ptr(pages.row_ids),
                                        c_int(int(q.dtype == torch.float32)), L.stream_ptr()), "paged_attend")
     L.count_launches()

@@ -19,7 +19,7 @@ def _formula(logits, ids, score_function: str, norm: bool, scaling: float):
     scores = torch.softmax(logits, -1) if score_function == "softmax" else torch.sigmoid(logits)
     w = scores.gather(-1, ids)
     if norm:
-        w = w / w.sum(-1, keepdim=True).clamp_min(1e-20)
+        w = w / (w.sum(-1, keepdim=True) + 1e-20)
     return w * scaling, scores
 
 

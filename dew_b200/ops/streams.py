@@ -19,11 +19,14 @@ MAX_STREAMS = 16
 
 
 class Write(NamedTuple):
-    """A sub-layer's output on its way into the streams: ``H'[t] = sum_s mix[s, t] H[s] + out[t] * (scale * y)``."""
+    """A sub-layer's output on its way into the streams: ``H'[t] = sum_s mix[s, t] H[s] + out[t] * (scale * y)``.  Without ``mix`` and ``out``
+    every stream keeps itself and takes ``y``; with ``weight``, ``y`` passes an RMS norm (``weight``, ``eps``) first."""
     y: torch.Tensor
-    scale: Optional[torch.Tensor]
-    mix: torch.Tensor
-    out: torch.Tensor
+    scale: Optional[torch.Tensor] = None
+    mix: Optional[torch.Tensor] = None
+    out: Optional[torch.Tensor] = None
+    weight: Optional[torch.Tensor] = None
+    eps: float = 0.0
 
 
 def _kernel_ok(x: torch.Tensor, *others) -> bool:
@@ -68,35 +71,39 @@ def embed_streams(tokens: torch.Tensor, positions: Optional[torch.Tensor], embed
 def stream_step_reference(H, write: Optional[Write], read, weight, eps: float, dtype, norm: str = "layer"):
     if write is not None:
         y = write.y.float()
+        if write.weight is not None:
+            y = y / torch.sqrt(y.pow(2).mean(-1, keepdim=True) + write.eps) * write.weight.float()
         if write.scale is not None:
             y = y * write.scale.float()
-        H = torch.einsum("st,...sd->...td", write.mix.float(), H) + write.out.float()[:, None] * y.unsqueeze(-2)
+        kept = H if write.mix is None else torch.einsum("st,...sd->...td", write.mix.float(), H)
+        H = kept + (y.unsqueeze(-2) if write.out is None else write.out.float()[:, None] * y.unsqueeze(-2))
     if weight is None:
         return None, H
-    u = torch.einsum("s,...sd->...d", read.float(), H)
+    u = H.sum(-2) if read is None else torch.einsum("s,...sd->...d", read.float(), H)
     if norm == "layer":
         return layer_norm_reference(u, weight, eps).to(dtype), H
     return (u / torch.sqrt(u.pow(2).mean(-1, keepdim=True) + eps) * weight.float()).to(dtype), H
 
 
-def stream_step(H: torch.Tensor, write: Optional[Write], read: torch.Tensor, weight: Optional[torch.Tensor], eps: float, dtype,
+def stream_step(H: torch.Tensor, write: Optional[Write], read: Optional[torch.Tensor], weight: Optional[torch.Tensor], eps: float, dtype,
                 norm: str = "layer") -> Tuple[Optional[torch.Tensor], torch.Tensor]:
-    """``(norm(sum_s read[s] H'[s]) * weight, H')`` with ``H'`` the streams after ``write`` (None: as they are).  ``H [..., n, d]`` fp32;
+    """``(norm(sum_s read[s] H'[s]) * weight, H')`` with ``H'`` the streams after ``write`` (None: as they are); ``read`` None: all ones.  ``H [..., n, d]`` fp32;
     on a GPU outside autograd ``H`` is updated in place.  ``weight`` None: the write alone."""
     if norm not in ("layer", "rms"):
         raise ValueError(f"unknown norm {norm!r}; known: layer, rms")
     n, d = H.shape[-2:]
-    tensors = (weight, read) + (() if write is None else (write.y, write.scale, write.mix, write.out))
+    tensors = (weight, read) + (() if write is None else (write.y, write.scale, write.mix, write.out, write.weight))
     if n > MAX_STREAMS or not H.is_contiguous() or not _kernel_ok(H, *tensors) or dtype not in (torch.bfloat16, torch.float32):
         return stream_step_reference(H, write, read, weight, eps, dtype, norm)
     rows = H.numel() // (n * d)
     normed = None if weight is None else torch.empty(*H.shape[:-2], d, dtype=dtype, device=H.device)
-    y = scale = mix = out = None
+    y = y_weight = scale = mix = out = None
     if write is not None:
         y, scale, mix, out = _as(write.y, dtype), _as(write.scale, dtype), _as(write.mix, torch.float32), _as(write.out, torch.float32)
+        y_weight = _as(write.weight, dtype)
     r, w = _as(read, torch.float32), _as(weight, dtype)
-    L.check(L.load().dewb_stream_step(L.ptr(H), L.ptr(y), L.ptr(scale), L.ptr(mix), L.ptr(out), L.ptr(r), L.ptr(w), L.ptr(normed), c_ll(rows), c_int(n),
-                                      c_int(d), c_float(eps), c_int(int(norm == "rms")), c_int(int(dtype == torch.float32)), L.stream_ptr()), "stream_step")
+    L.check(L.load().dewb_stream_step(L.ptr(H), L.ptr(y), L.ptr(y_weight), L.ptr(scale), L.ptr(mix), L.ptr(out), L.ptr(r), L.ptr(w), L.ptr(normed), c_ll(rows),
+                                      c_int(n), c_int(d), c_float(0.0 if write is None else write.eps), c_float(eps), c_int(int(norm == "rms")), c_int(int(dtype == torch.float32)), L.stream_ptr()), "stream_step")
     L.count_launches()
     return normed, H
 
@@ -116,6 +123,23 @@ def clamped_glu(gu: torch.Tensor, limit: float, alpha: float = 1.702) -> torch.T
     out = torch.empty(*gu.shape[:-1], Fh, dtype=gu.dtype, device=gu.device)
     L.check(L.load().dewb_clamped_glu(L.ptr(gu), L.ptr(out), c_ll(gu.numel() // (2 * Fh)), c_int(Fh), c_float(limit), c_float(alpha),
                                       c_int(int(gu.dtype == torch.float32)), L.stream_ptr()), "clamped_glu")
+    L.count_launches()
+    return out
+
+
+def softcap_reference(x: torch.Tensor, cap: float) -> torch.Tensor:
+    return cap * torch.tanh(x.float() / cap)
+
+
+def softcap(x: torch.Tensor, cap: float) -> torch.Tensor:
+    """``cap tanh(x / cap)`` in fp32."""
+    if not _kernel_ok(x):
+        return softcap_reference(x, cap)
+    x = x.contiguous()
+    n = x.shape[-1]
+    out = torch.empty(x.shape, dtype=torch.float32, device=x.device)
+    L.check(L.load().dewb_softcap(L.ptr(x), L.ptr(out), c_ll(x.numel() // max(n, 1)), c_int(n), c_float(cap), c_int(int(x.dtype == torch.float32)),
+                                  L.stream_ptr()), "softcap")
     L.count_launches()
     return out
 

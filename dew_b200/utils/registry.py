@@ -48,7 +48,7 @@ _STATIC: Dict[str, Dict[str, str]] = {
         "autoencoder_kl": "dew_b200.models.latent_autoencoders:AutoencoderKL", "dc_ae": "dew_b200.models.latent_autoencoders:DCAE",
         "causal_video_vae": "dew_b200.models.latent_autoencoders:CausalVideoVAE",
         "classic_decoder": "dew_b200.models.classic_decoder:ClassicDecoder",
-        "ragenex": "dew_b200.interop.ragenex:ragenex",
+        "ragenex": "dew_b200.interop.ragenex:ragenex", "fakonex": "dew_b200.interop.fakonex:fakonex",
     },
     "objective": {
         "lm": "dew_b200.objectives.lm:LMObjective",
