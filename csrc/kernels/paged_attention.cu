@@ -100,27 +100,30 @@ qk_norm_append_kernel(const T* __restrict__ qkv, const T* __restrict__ qw, const
   }
 }
 
-// One group of LG lanes per (token, head); heads [0, H) queries, then G keys, then G values (G 0: queries alone).
-template <typename T, int V, int LG>
+// One group of LG lanes per (token, head); heads [0, H) queries, then G keys, then G values (G 0: queries alone).  ONE: a head is at most LG V
+// wide, so it is read once.
+template <typename T, int V, int LG, bool ONE>
 __global__ void __launch_bounds__(256)
 head_norm_append_kernel(const T* __restrict__ qkv, long long row_stride, const T* __restrict__ bias, const T* __restrict__ qw, const T* __restrict__ kw,
                         float eps, const int* __restrict__ positions, long long items, int S, int H, int G, int dk, int dv, int D,
                         T* __restrict__ packed, T* __restrict__ kpool, T* __restrict__ vpool, Pool pool) {
-  const long long item = (static_cast<long long>(blockIdx.x) * 256 + threadIdx.x) / LG;
+  const unsigned item = blockIdx.x * (256 / LG) + threadIdx.x / LG;
   const int lane = threadIdx.x % LG;
   const bool on = item < items;                      // every lane stays for the sums
-  const int heads = H + 2 * G;
-  const long long t = on ? item / heads : 0;
-  const int h = on ? static_cast<int>(item - t * heads) : 0;
+  const unsigned heads = H + 2 * G, tt = on ? item / heads : 0;
+  const long long t = tt;
+  const int h = on ? static_cast<int>(item - tt * heads) : 0;
   const int part = h < H ? 0 : h < H + G ? 1 : 2, width = part == 2 ? dv : dk;
   const int at = part == 2 ? (H + G) * dk + (h - H - G) * dv : h * dk;
   const T* src = qkv + t * row_stride + at;
   const T* b = bias == nullptr ? nullptr : bias + at;
   const T* w = part == 0 ? qw : part == 1 ? kw : nullptr;
-  float ss = 0.f;
-  if (w != nullptr) {
+  const int pos = part != 0 ? positions[t] : -1;
+  float ss = 0.f, a[V];
+#pragma unroll
+  for (int j = 0; j < V; ++j) a[j] = 0.f;
+  if (ONE || w != nullptr) {
     for (int i = lane * V; i < width; i += LG * V) {
-      float a[V];
       load_v<V>(src + i, a);
       if (b != nullptr) {
         float c[V];
@@ -136,23 +139,26 @@ head_norm_append_kernel(const T* __restrict__ qkv, long long row_stride, const T
   for (int o = LG / 2; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
   if (!on) return;
   const float r = w != nullptr ? 1.f / sqrtf(ss / width + eps) : 1.f;
-  T* dst = packed + item * D;
+  T* dst = packed + static_cast<long long>(item) * D;
   T* to_pool = nullptr;
-  if (part != 0 && positions[t] >= 0) {
-    const long long tok = pool_token(pool, static_cast<int>(t / S), positions[t]);
+  if (pos >= 0) {
+    const long long tok = pool_token(pool, static_cast<int>(tt / static_cast<unsigned>(S)), pos);
     to_pool = (part == 1 ? kpool : vpool) + (tok * G + (part == 1 ? h - H : h - H - G)) * D;
   }
   for (int i = lane * V; i < D; i += LG * V) {
-    float a[V];
+    if (!ONE) {
 #pragma unroll
-    for (int j = 0; j < V; ++j) a[j] = 0.f;
+      for (int j = 0; j < V; ++j) a[j] = 0.f;
+    }
     if (i < width) {
-      load_v<V>(src + i, a);
-      if (b != nullptr) {
-        float c[V];
-        load_v<V>(b + i, c);
+      if (!ONE) {
+        load_v<V>(src + i, a);
+        if (b != nullptr) {
+          float c[V];
+          load_v<V>(b + i, c);
 #pragma unroll
-        for (int j = 0; j < V; ++j) a[j] += c[j];
+          for (int j = 0; j < V; ++j) a[j] += c[j];
+        }
       }
       if (w != nullptr) {
         float c[V];
@@ -551,13 +557,16 @@ extern "C" int dewb_head_norm_append(const void* qkv, long long row_stride, cons
   const bool vec = dk % 4 == 0 && dv % 4 == 0 && D % 4 == 0 && row_stride % 4 == 0 && aligned(qkv, 16) && aligned(bias, 16) && aligned(qw, 16) &&
                    aligned(kw, 16) && aligned(packed, 16) && aligned(kpool, 16) && aligned(vpool, 16);
   const long long items = static_cast<long long>(R) * S * (H + 2 * G);
-  const int lg = D <= 64 ? 16 : 32;
+  const bool vec8 = vec && !fp32 && dk % 8 == 0 && dv % 8 == 0 && D % 8 == 0 && row_stride % 8 == 0;
+  const int v = vec8 ? 8 : vec ? 4 : 1, lg = D <= 8 * v ? 8 : D <= 16 * v ? 16 : 32;
+  const bool one = D <= lg * v;
   const long long blocks = (items * lg + 255) / 256;
-  if (blocks > 0x7fffffffll) return -3;
-#define DEWB_HEADS(TT, VV, LL) head_norm_append_kernel<TT, VV, LL><<<static_cast<unsigned>(blocks), 256, 0, stream>>>(static_cast<const TT*>(qkv),     row_stride, static_cast<const TT*>(bias), static_cast<const TT*>(qw), static_cast<const TT*>(kw), eps, positions, items, S, H, G, dk, dv, D,     static_cast<TT*>(packed), static_cast<TT*>(kpool), static_cast<TT*>(vpool), pool)
-#define DEWB_HEADS_L(TT, VV) do { if (lg == 16) DEWB_HEADS(TT, VV, 16); else DEWB_HEADS(TT, VV, 32); } while (0)
+  if (items > 0x7fffffffll) return -3;
+#define DEWB_HEADS(TT, VV, LL, OO) head_norm_append_kernel<TT, VV, LL, OO><<<static_cast<unsigned>(blocks), 256, 0, stream>>>(static_cast<const TT*>(qkv),     row_stride, static_cast<const TT*>(bias), static_cast<const TT*>(qw), static_cast<const TT*>(kw), eps, positions, items, S, H, G, dk, dv, D,     static_cast<TT*>(packed), static_cast<TT*>(kpool), static_cast<TT*>(vpool), pool)
+#define DEWB_HEADS_L(TT, VV) do { if (lg == 8) DEWB_HEADS(TT, VV, 8, true); else if (lg == 16) DEWB_HEADS(TT, VV, 16, true); \
+    else if (one) DEWB_HEADS(TT, VV, 32, true); else DEWB_HEADS(TT, VV, 32, false); } while (0)
   if (fp32) { if (vec) DEWB_HEADS_L(float, 4); else DEWB_HEADS_L(float, 1); }
-  else { if (vec) DEWB_HEADS_L(bf16, 4); else DEWB_HEADS_L(bf16, 1); }
+  else { if (vec8) DEWB_HEADS_L(bf16, 8); else if (vec) DEWB_HEADS_L(bf16, 4); else DEWB_HEADS_L(bf16, 1); }
 #undef DEWB_HEADS_L
 #undef DEWB_HEADS
   return static_cast<int>(cudaGetLastError());

@@ -6,7 +6,8 @@
 //                       H'[t] = sum_s mix[s, t] H[s] + out[t] * (scale . y)
 //                   (in place), the read of the next one, u = sum_s read[s] H'[s], and its norm (layer norm without a bias, or RMS norm);
 //                   y may pass an RMS norm of its own first (a block that normalises what its sub-layers return).  Without connection
-//                   weights the streams keep themselves and take y as it is: one such stream is the ordinary fp32 residual.
+//                   weights the streams keep themselves and take y as it is: one such stream is the ordinary fp32 residual, which has a
+//                   form of its own (residual_step).
 //   clamped_glu     g sigmoid(alpha g) (u + 1) with g = min(gate, limit), u = clamp(up, -limit, limit)
 //   sigmoid_gated_norm   RMS norm over a whole row times a weight times sigmoid(gate)
 //   softcap         cap tanh(x / cap), fp32 out (logits)
@@ -152,6 +153,66 @@ stream_step_kernel(float* __restrict__ H, const T* __restrict__ y, const T* __re
   }
 }
 
+// One plain stream (H += y, y through its RMS norm where it has a weight, then the norm of H): the whole row in registers, NI pieces of V values a
+// thread, every load in flight before the first sum.
+template <typename T, int V, int NI>
+__global__ void __launch_bounds__(THREADS)
+residual_step_kernel(float* __restrict__ H, const T* __restrict__ y, const T* __restrict__ y_weight, const T* __restrict__ w, T* __restrict__ normed,
+                     int d, float y_eps, float eps) {
+  __shared__ float red[32];
+  const long long at = static_cast<long long>(blockIdx.x) * d;
+  float x[NI][V], b[NI][V];
+#pragma unroll
+  for (int p = 0; p < NI; ++p) {
+    const int i = (p * THREADS + threadIdx.x) * V;
+#pragma unroll
+    for (int j = 0; j < V; ++j) x[p][j] = b[p][j] = 0.f;
+    if (i < d) {
+      load_v<V>(y + at + i, b[p]);
+      load_v<V>(H + at + i, x[p]);
+    }
+  }
+  if (y_weight != nullptr) {
+    float ss = 0.f;
+#pragma unroll
+    for (int p = 0; p < NI; ++p)
+#pragma unroll
+      for (int j = 0; j < V; ++j) ss += b[p][j] * b[p][j];
+    const float ry = 1.f / sqrtf(block_sum(ss, red) / d + y_eps);
+#pragma unroll
+    for (int p = 0; p < NI; ++p) {
+      const int i = (p * THREADS + threadIdx.x) * V;
+      if (i < d) {
+        float c[V];
+        load_v<V>(y_weight + i, c);
+#pragma unroll
+        for (int j = 0; j < V; ++j) b[p][j] = b[p][j] * ry * c[j];
+      }
+    }
+  }
+  float ss = 0.f;
+#pragma unroll
+  for (int p = 0; p < NI; ++p) {
+    const int i = (p * THREADS + threadIdx.x) * V;
+#pragma unroll
+    for (int j = 0; j < V; ++j) { x[p][j] += b[p][j]; ss += x[p][j] * x[p][j]; }
+    if (i < d) store_v<V>(H + at + i, x[p]);
+  }
+  if (normed == nullptr) return;
+  const float r = 1.f / sqrtf(block_sum(ss, red) / d + eps);
+#pragma unroll
+  for (int p = 0; p < NI; ++p) {
+    const int i = (p * THREADS + threadIdx.x) * V;
+    if (i < d) {
+      float c[V];
+      load_v<V>(w + i, c);
+#pragma unroll
+      for (int j = 0; j < V; ++j) c[j] *= x[p][j] * r;
+      store_v<V>(normed + at + i, c);
+    }
+  }
+}
+
 // x sigmoid(z) times a factor: fp32 models take the exact quotient, bf16 the approximate one (a few parts in 2^22)
 template <typename T>
 __device__ __forceinline__ float times_sigmoid(float x, float z) {
@@ -228,6 +289,13 @@ int step(float* H, const T* y, const T* y_weight, const T* scale, const float* m
          long long rows, int n, int d, float y_eps, float eps, int rms, cudaStream_t stream) {
   const bool vec = d % 4 == 0 && aligned(H, 16) && aligned(y, 4 * sizeof(T)) && aligned(y_weight, 4 * sizeof(T)) && aligned(scale, 4 * sizeof(T)) && aligned(w, 4 * sizeof(T)) &&
                    aligned(normed, 4 * sizeof(T));
+  if (vec && n == 1 && rms && y != nullptr && scale == nullptr && mix == nullptr && out == nullptr && read == nullptr && d <= 32 * THREADS) {
+    const int pieces = (d + THREADS * 4 - 1) / (THREADS * 4);
+#define DEWB_RES(NN) residual_step_kernel<T, 4, NN><<<static_cast<unsigned>(rows), THREADS, 0, stream>>>(H, y, y_weight, w, normed, d, y_eps, eps)
+    if (pieces <= 1) DEWB_RES(1); else if (pieces <= 2) DEWB_RES(2); else if (pieces <= 4) DEWB_RES(4); else DEWB_RES(8);
+#undef DEWB_RES
+    return static_cast<int>(cudaGetLastError());
+  }
   const size_t smem = static_cast<size_t>(d) * 4;
 #define DEWB_STEP(VV, NN) do { const int r = allow_smem(stream_step_kernel<T, VV, NN>, smem); if (r) return r; \
     stream_step_kernel<T, VV, NN><<<static_cast<unsigned>(rows), THREADS, smem, stream>>>(H, y, y_weight, scale, mix, out, read, w, normed, n, d, y_eps, eps, rms); } while (0)

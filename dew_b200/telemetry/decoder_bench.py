@@ -1,15 +1,15 @@
-"""Prefill and decode throughput of the Ragenex design beside this library's closest decoder of the same sizes (rotary attention and
-gated-delta-net layers in the same order, SwiGLU, one bf16 residual), and each of the design's kernels beside the like kernel of that decoder,
-as a fraction of its roofline.
+"""Prefill and decode throughput of a decoder design beside this library's closest decoder of the same sizes, and each of the design's kernels
+beside the like kernel of that decoder, as a fraction of its roofline: the Ragenex design here (closest: rotary attention and gated-delta-net
+layers in the same order, SwiGLU, one bf16 residual), the Fakonex design in ``telemetry.fakonex_bench``.
 
-``bench.py --decoder ragenex`` prints the result as one JSON line.  Weights are random.  Everything is timed on the device with CUDA events
+``bench.py --decoder ragenex | fakonex`` prints the result as one JSON line.  Weights are random.  Everything is timed on the device with CUDA events
 after warm-up; prefill activations and weights are larger than L2, and a decode step (one CUDA graph) streams all the weights.
 """
 from __future__ import annotations
 
 import json
 from pathlib import Path
-from typing import Callable, Dict, List
+from typing import Callable, Dict, List, Optional
 
 import torch
 
@@ -203,17 +203,24 @@ def kernels(s: dict, tokens: int, decode_rows: int, context: int, iters: int) ->
     return rows
 
 
-def run(sizes=("d2048", "d4096", "d2048h64"), rows: int = 4, prompt: int = 4096, decode_rows: int = 64, context: int = 4096, iters: int = 5) -> Dict[str, object]:
+def run(name: str = "ragenex", sizes=None, rows: int = 4, prompt: int = 4096, decode_rows: int = 64, context: Optional[int] = None, iters: int = 5) -> Dict[str, object]:
     torch.manual_seed(0)
+    if name == "fakonex":
+        from . import fakonex_bench as f
+        table, design, near, parts = f.SIZES, f.design, f.closest, f.kernels
+        context = 4095 if context is None else context           # the last position of a chunk: as many keys as the closest model's window holds
+    else:
+        table, design, near, parts = SIZES, ragenex, closest, kernels
+        context = 4096 if context is None else context
     out: Dict[str, object] = {"peaks": peaks(), "rows": rows, "prompt": prompt, "decode_rows": decode_rows, "context": context, "warmup": WARMUP,
                               "dtype": "bf16", "data": "synthetic (random token ids, random-init weights)", "sizes": {}}
-    for name in sizes:
-        s = SIZES[name]
+    for size in sizes or table:
+        s = table[size]
         line: Dict[str, object] = {"config": s}
-        for tag, make in (("ragenex", ragenex), ("closest", closest)):
+        for tag, make in ((name, design), ("closest", near)):
             line[tag] = throughput(make(s, prompt + 128), s, rows, prompt, decode_rows, context, iters)
             torch.cuda.empty_cache()
-        line["kernels"] = kernels(s, rows * prompt, decode_rows, context, iters)
+        line["kernels"] = parts(s, rows * prompt, decode_rows, context, iters)
         torch.cuda.empty_cache()
-        out["sizes"][name] = line
+        out["sizes"][size] = line
     return out
