@@ -134,6 +134,8 @@ __device__ __forceinline__ void choose(const Choice& c, long long t, bool live, 
   }
 }
 
+constexpr int SELECT_TOKENS = 32;      // tokens a block selects for: it takes its experts' places with one addition per expert
+
 // logits [T, ld] fp32; `rest` columns further on (0: none) holds what the weights' rounding to bf16 dropped, to be added
 template <int NI>
 __global__ void __launch_bounds__(THREADS)
@@ -141,7 +143,13 @@ moe_select_kernel(const float* __restrict__ logits, long long ld_, int rest, con
   extern __shared__ float smem[];
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   float* s_sel = smem + warp * (c.E + c.groups);
-  for (long long t = static_cast<long long>(blockIdx.x) * WARPS + warp; t < T; t += static_cast<long long>(gridDim.x) * WARPS) {
+  int* s_count = reinterpret_cast<int*>(smem + WARPS * (c.E + c.groups));
+  int* const counts = c.counts;
+  for (int e = threadIdx.x; e < c.E; e += THREADS) s_count[e] = 0;
+  __syncthreads();
+  c.counts = s_count;
+  const long long t0 = static_cast<long long>(blockIdx.x) * SELECT_TOKENS, t1 = t0 + SELECT_TOKENS < T ? t0 + SELECT_TOKENS : T;
+  for (long long t = t0 + warp; t < t1; t += WARPS) {
     float sc[NI];
 #pragma unroll
     for (int i = 0; i < NI; ++i) {
@@ -150,6 +158,12 @@ moe_select_kernel(const float* __restrict__ logits, long long ld_, int rest, con
     }
     choose<NI>(c, t, positions == nullptr || positions[t] >= 0, sc, s_sel, s_sel + c.E);
   }
+  __syncthreads();
+  for (int e = threadIdx.x; e < c.E; e += THREADS)
+    if (s_count[e] > 0) s_count[e] = atomicAdd(counts + e, s_count[e]);
+  __syncthreads();
+  for (long long t = t0 + warp; t < t1; t += WARPS)      // the lanes that wrote these places
+    if (lane < c.k && c.ids[t * c.k + lane] >= 0) c.rank[t * c.k + lane] += s_count[c.ids[t * c.k + lane]];
 }
 
 // x [T, d], w [E, d]
@@ -392,11 +406,10 @@ int allow_smem(K kernel, size_t bytes) {
 
 template <int NI>
 int select(const float* logits, long long ld_, int rest, const int* positions, int T, const Choice& c, cudaStream_t stream) {
-  const size_t smem = static_cast<size_t>(WARPS) * (c.E + c.groups) * 4;
+  const size_t smem = (static_cast<size_t>(WARPS) * (c.E + c.groups) + c.E) * 4;
   const int r = allow_smem(moe_select_kernel<NI>, smem);
   if (r) return r;
-  const int blocks = (T + WARPS - 1) / WARPS;
-  moe_select_kernel<NI><<<blocks < 148 * 8 ? blocks : 148 * 8, THREADS, smem, stream>>>(logits, ld_, rest, positions, T, c);
+  moe_select_kernel<NI><<<(T + SELECT_TOKENS - 1) / SELECT_TOKENS, THREADS, smem, stream>>>(logits, ld_, rest, positions, T, c);
   return static_cast<int>(cudaGetLastError());
 }
 
