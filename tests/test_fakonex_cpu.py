@@ -98,7 +98,7 @@ def test_head_gates_read_the_last_columns_of_the_projection():
         assert torch.allclose(got[..., h, :].to(D64), o[..., h, :5].to(D64) * O.sigmoid(z[..., 5 + h].to(D64))[..., None], atol=1e-6)
 
 
-@pytest.mark.parametrize("E,top,groups,keep", [(6, 2, 3, 2), (8, 4, 2, 1), (4, 2, 4, 2), (12, 3, 4, 1), (5, 5, 1, 1), (9, 1, 3, 3)])
+@pytest.mark.parametrize("E,top,groups,keep", [(6, 2, 3, 2), (10, 3, 2, 1), (4, 2, 4, 2), (12, 3, 4, 1), (5, 5, 1, 1), (9, 1, 3, 3)])
 def test_selection(E, top, groups, keep):
     z, b = rnd(40, E), rnd(E, seed=1) - 1.0
     s = moe_serve.Selection(E, top, groups, keep, float("-inf"), "sigmoid")

@@ -170,7 +170,7 @@ def test_decode_in_chunks_over_long_rows(D, Hq, Hkv):
 
 
 # ------------------------------------------------------------------------------------------------ experts
-SELECTIONS = [moe_serve.Selection(8, 4, 2, 1, float("-inf"), "sigmoid"), moe_serve.Selection(12, 2, 4, 2, float("-inf"), "sigmoid", True, 2.5),
+SELECTIONS = [moe_serve.Selection(10, 3, 2, 1, float("-inf"), "sigmoid"), moe_serve.Selection(12, 2, 4, 2, float("-inf"), "sigmoid", True, 2.5),
               moe_serve.Selection(5, 5, 1, 1, 0.0, "softmax", False), moe_serve.Selection(128, 8, 8, 4, 0.0, "sigmoid"),
               moe_serve.Selection(300, 20, 10, 3, float("-inf"), "softmax"), moe_serve.Selection(6, 3, 6, 4, float("-inf"), "sigmoid")]
 
