@@ -1,6 +1,7 @@
 // Optional attention variants shared by the forward and backward flash kernels.  The plain causal / full kernels are
 // compiled with VAR = false and contain none of this.
 //   window   : query i sees keys in (i + T - S - window, i + T - S]  (0 = no window)
+//   keep     : beside a window, the first `keep` keys stay visible (forward only)
 //   chunk    : query i sees no key from before the start of its chunk of `chunk` positions, counted from 0 (0 = no chunks; forward only)
 //   softcap  : scores become cap * tanh(score / cap)                 (0 = none)
 //   sinks    : one learned logit per query head that joins the softmax denominator only (forward; the backward kernels
@@ -20,13 +21,11 @@ struct Variant {
   const int* q_seg;        // [B, S] or null
   const int* k_seg;        // [B, T] or null
   int chunk;
+  int keep;
 };
 
-__device__ __forceinline__ float fast_tanh(float x) {
-  float y;
-  asm("tanh.approx.f32 %0, %1;" : "=f"(y) : "f"(x));
-  return y;
-}
+// tanh to fp32 accuracy relative to 1 (scores under a cap are fp32 quantities): 1 - 2 / (1 + e^2x)
+__device__ __forceinline__ float soft_tanh(float x) { return 1.f - __fdividef(2.f, 1.f + exp2f(x * 2.8853900817779268f)); }
 
 // First key tile (of `bn` keys) that a query tile starting at row q0 can see; `off` = T - S (bottom-right alignment).
 __device__ __forceinline__ int first_key_tile(const Variant& v, int b, int q0, int S, int T, int bn, int n_tiles) {

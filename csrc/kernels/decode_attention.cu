@@ -16,6 +16,7 @@
 #include <cuda_fp8.h>
 #include <cuda_runtime.h>
 
+#include "../common/attn_variant.cuh"
 #include "../common/key_range.cuh"
 
 namespace dewb {
@@ -58,7 +59,7 @@ paged_decode_kernel(const __nv_bfloat16* __restrict__ q, const void* __restrict_
                     const float* __restrict__ kscale, const float* __restrict__ vscale,
                     const int* __restrict__ page_table, const int* __restrict__ lengths, float* __restrict__ part_m,
                     float* __restrict__ part_l, float* __restrict__ part_acc, int Hq, int Hkv, int share, int page_size,
-                    int max_pages, int splits, float scale_log2, int window, int chunk) {
+                    int max_pages, int splits, float scale_log2, int window, int keep, int chunk, float cap_log2) {
   constexpr int DV = D / 32;                 // value elements per lane
   const int row = blockIdx.x, hk = blockIdx.y, split = blockIdx.z;
   const int kvh = hk / share;                  // `share` groups of query heads read the same KV head
@@ -78,10 +79,11 @@ paged_decode_kernel(const __nv_bfloat16* __restrict__ q, const void* __restrict_
   __syncthreads();
   // keys of this split: [k_begin, k_end) in 32-key blocks, interleaved across the CTA's warps
   const int first = first_key(len, window, chunk);
-  const int span = len - first;
+  const int kept = kept_keys(first, keep);     // the first keys that stay visible stand in front of the others
+  const int span = kept + len - first;
   const int per_split = ((span + splits - 1) / splits + 31) / 32 * 32;
-  const int k_begin = first + split * per_split;
-  const int k_end = min(len, k_begin + per_split);
+  const int k_begin = split * per_split;         // counted among the visible keys
+  const int k_end = min(span, k_begin + per_split);
   float m[GM], l[GM], acc[GM][DV];
 #pragma unroll
   for (int g = 0; g < GM; ++g) {
@@ -91,8 +93,8 @@ paged_decode_kernel(const __nv_bfloat16* __restrict__ q, const void* __restrict_
   }
   const int* table = page_table + static_cast<long long>(row) * max_pages;
   for (int kb = k_begin + warp * 32; kb < k_end; kb += WARPS * 32) {
-    const int key = kb + lane;
-    const bool live = key < k_end;
+    const bool live = kb + lane < k_end;
+    const int key = kb + lane < kept ? kb + lane : first + kb + lane - kept;
     float s[GM];
 #pragma unroll
     for (int g = 0; g < GM; ++g) s[g] = -INFINITY;
@@ -126,6 +128,10 @@ paged_decode_kernel(const __nv_bfloat16* __restrict__ q, const void* __restrict_
       const float ks = KIND == KV_BF16 ? 1.f : kscale[tok * Hkv + kvh];
 #pragma unroll
       for (int g = 0; g < GM; ++g) if (GT != 0 || g < G) s[g] = dot[g] * ks;
+      if (cap_log2 > 0.f) {
+#pragma unroll
+        for (int g = 0; g < GM; ++g) if (GT != 0 || g < G) s[g] = cap_log2 * attn::soft_tanh(s[g] / cap_log2);
+      }
     }
     // online softmax update (per query head), block maximum by warp reduction
     float p[GM];
@@ -313,10 +319,10 @@ extern "C" int dewb_paged_decode(const void* q, const void* kpool, const void* v
                                  const float* vscale, const int* page_table, const int* lengths, const float* sinks,
                                  void* out, float* lse, float* part_m, float* part_l, float* part_acc, int rows, int Hq,
                                  int Hkv, int share, int D, int page_size, int max_pages, int splits, float scale, int window,
-                                 int chunk, int kv_kind, void* stream_ptr) {
+                                 int keep, int chunk, float softcap, int kv_kind, void* stream_ptr) {
   if (rows <= 0) return 0;
   if ((D != 64 && D != 128 && D != 256) || share < 1 || Hkv < 1 || Hq % (Hkv * share) != 0 ||
-      Hq / (Hkv * share) > MAX_G || splits < 1)
+      Hq / (Hkv * share) > MAX_G || splits < 1 || keep < 0 || (keep > 0 && chunk > 0))
     return -3;
   cudaStream_t stream = reinterpret_cast<cudaStream_t>(stream_ptr);
   const float scale_log2 = scale * 1.4426950408889634f;
@@ -324,7 +330,7 @@ extern "C" int dewb_paged_decode(const void* q, const void* kpool, const void* v
   const __nv_bfloat16* qp = reinterpret_cast<const __nv_bfloat16*>(q);
   const int Gq = Hq / (Hkv * share);
 #define DEWB_DECODE_G(DD, KK, GG) paged_decode_kernel<DD, KK, GG><<<grid, WARPS * 32, 0, stream>>>( \
-    qp, kpool, vpool, kscale, vscale, page_table, lengths, part_m, part_l, part_acc, Hq, Hkv, share, page_size, max_pages, splits, scale_log2, window, chunk)
+    qp, kpool, vpool, kscale, vscale, page_table, lengths, part_m, part_l, part_acc, Hq, Hkv, share, page_size, max_pages, splits, scale_log2, window, keep, chunk, softcap * 1.4426950408889634f)
 #define DEWB_DECODE(DD, KK) do { if (Gq == 4) DEWB_DECODE_G(DD, KK, 4); else if (Gq == 8) DEWB_DECODE_G(DD, KK, 8); \
     else if (Gq == 1) DEWB_DECODE_G(DD, KK, 1); else if (Gq == 2) DEWB_DECODE_G(DD, KK, 2); else DEWB_DECODE_G(DD, KK, 0); } while (0)
 #define DEWB_DECODE_D(KK) do { if (D == 64) DEWB_DECODE(64, KK); else if (D == 128) DEWB_DECODE(128, KK); else DEWB_DECODE(256, KK); } while (0)

@@ -12,6 +12,7 @@
 // The query count per KV head is far below the 64 rows tcgen05 needs, which is why this kernel uses the warp-level MMA.
 //
 // Capability parity: src/dew/nn/kernels/decode_attention.py (attend_paged), src/dew/nn/kernels/templates/attention_decode.py.
+#include "../common/attn_variant.cuh"
 #include "../common/key_range.cuh"
 #include "../common/ptx.cuh"
 #include "../common/tmap.h"
@@ -59,7 +60,7 @@ paged_decode_tma_kernel(const __grid_constant__ CUtensorMap tk, const __grid_con
                         const __nv_bfloat16* __restrict__ q, const int* __restrict__ page_table,
                         const int* __restrict__ lengths, float* __restrict__ part_m, float* __restrict__ part_l,
                         float* __restrict__ part_acc, int Hq, int Hkv, int page_size, int max_pages, int splits,
-                        float scale_log2, int window, int chunk, long long q_row_stride, int* __restrict__ err,
+                        float scale_log2, int window, int keep, int chunk, float cap_log2, long long q_row_stride, int* __restrict__ err,
                         __nv_bfloat16* __restrict__ out, const float* __restrict__ sinks, unsigned int* __restrict__ arrivals,
                         int chunk_tiles) {
   extern __shared__ __align__(1024) uint8_t smem[];
@@ -75,20 +76,20 @@ paged_decode_tma_kernel(const __grid_constant__ CUtensorMap tk, const __grid_con
   const int row = blockIdx.x, hk = blockIdx.y, split = blockIdx.z;
   const int G = Hq / Hkv;
   const int len = lengths[row];
-  // this split's keys, in whole 64-key tiles: [t_begin, t_end) tile indices of the row; keys outside [first, len) are masked
-  const int first = first_key(len, window, chunk);
-  const int tile_lo = first / TK, tile_hi = (len + TK - 1) / TK;
+  // this split's keys, in whole 64-key tiles: [t_begin, t_end) of the row's walk; keys the query does not see are masked
+  const TileWalk walk(len, window, keep, chunk, TK);
+  const int first = walk.first;
   // With `out` the kernel finishes the row itself: a row uses as many of the grid's splits as it has chunks of `chunk_tiles`
   // tiles (short rows take one CTA, the others leave at once), and the last split to arrive merges the partials.
   int eff = splits;
   if (out != nullptr) {
-    eff = (max(0, tile_hi - tile_lo) + chunk_tiles - 1) / chunk_tiles;
+    eff = (walk.n + chunk_tiles - 1) / chunk_tiles;
     eff = max(1, min(splits, eff));
     if (split >= eff) return;
   }
-  const int per_split = (tile_hi - tile_lo + eff - 1) / eff;
-  const int t_begin = tile_lo + split * per_split;
-  const int t_end = min(tile_hi, t_begin + per_split);
+  const int per_split = (walk.n + eff - 1) / eff;
+  const int t_begin = split * per_split;
+  const int t_end = min(walk.n, t_begin + per_split);
   const int ntiles = max(0, t_end - t_begin);
 
   __nv_bfloat16* sQ = reinterpret_cast<__nv_bfloat16*>(smem + OFF_Q);
@@ -122,7 +123,7 @@ paged_decode_tma_kernel(const __grid_constant__ CUtensorMap tk, const __grid_con
         const int s = t % STAGES;
         const uint32_t ph = (t / STAGES) & 1;
         if (!mbar_wait(&bars->empty[s], ph ^ 1, abort_flag)) { atomicCAS(err, 0, ERR_WAIT_EMPTY); break; }
-        const int key0 = (t_begin + t) * TK;
+        const int key0 = walk.tile(t_begin + t) * TK;
         const int page = table[key0 / page_size];
         const int row0 = page * page_size + key0 % page_size;
         uint8_t* st = smem + s * STAGE_BYTES;
@@ -169,13 +170,15 @@ paged_decode_tma_kernel(const __grid_constant__ CUtensorMap tk, const __grid_con
         mma_16816(sc[1], qa0[ks], 0u, qa2[ks], 0u, b2, b3);
       }
       // mask and online softmax for head row lane / 4 (values of rows 8..15, sc[.][2..3], are ignored)
-      const int key_base = (t_begin + t) * TK + kw + (lane & 3) * 2;
+      const int key_base = walk.tile(t_begin + t) * TK + kw + (lane & 3) * 2;
       float pv[4];
       float mx = -INFINITY;
 #pragma unroll
       for (int i = 0; i < 4; ++i) {
         const int key = key_base + (i >> 1) * 8 + (i & 1);
-        const float v = (key >= first && key < len) ? sc[i >> 1][i & 1] * scale_log2 : -INFINITY;
+        float v = sc[i >> 1][i & 1] * scale_log2;
+        if (cap_log2 > 0.f) v = cap_log2 * attn::soft_tanh(v / cap_log2);
+        v = (key >= first || key < keep) && key < len ? v : -INFINITY;
         pv[i] = v;
         mx = fmaxf(mx, v);
       }
@@ -304,25 +307,22 @@ struct PBars {
 
 __device__ __forceinline__ void consumer_bar() { asm volatile("bar.sync 1, 128;" ::: "memory"); }
 
-struct Seg { int row, hk, part, eff, t_begin, ntiles, first, len; };
+struct Seg { int row, hk, part, eff, t_begin, ntiles, len; TileWalk walk; };
 
 // the segment that starts at tile `u` of the sequence and ends with its (row, head) or with the CTA's range `u1`
 __device__ __forceinline__ Seg locate(int u, int u1, const int* prefix, const int* __restrict__ lengths, int rows,
-                                      int per_head, int Q, int window, int chunk) {
-  Seg sg;
-  sg.hk = u / per_head;
-  const int w = u - sg.hk * per_head;
+                                      int per_head, int Q, int window, int keep, int chunk) {
+  const int hk = u / per_head;
+  const int w = u - hk * per_head;
   int lo = 0, hi = rows;                                   // largest r with prefix[r] <= w
   while (hi - lo > 1) {
     const int mid = (lo + hi) >> 1;
     if (prefix[mid] <= w) lo = mid; else hi = mid;
   }
-  sg.row = lo;
+  Seg sg{lo, hk, 0, 0, 0, 0, lengths[lo], TileWalk(lengths[lo], window, keep, chunk, TK)};
   const int start = sg.hk * per_head + prefix[lo];          // the (row, head)'s first tile in the sequence
   const int n = prefix[lo + 1] - prefix[lo];
-  sg.len = lengths[lo];
-  sg.first = first_key(sg.len, window, chunk);
-  sg.t_begin = sg.first / TK + (u - start);
+  sg.t_begin = u - start;                                   // counted in the row's walk
   sg.ntiles = min(u1, start + n) - u;
   const int first_cta = start / Q;
   sg.part = u / Q - first_cta;
@@ -335,7 +335,7 @@ paged_decode_persist_kernel(const __grid_constant__ CUtensorMap tk, const __grid
                             const __nv_bfloat16* __restrict__ q, const int* __restrict__ page_table,
                             const int* __restrict__ lengths, float* __restrict__ part_m, float* __restrict__ part_l,
                             float* __restrict__ part_acc, int rows, int Hq, int Hkv, int page_size, int max_pages,
-                            int max_parts, float scale_log2, int window, int chunk, long long q_row_stride, int* __restrict__ err,
+                            int max_parts, float scale_log2, int window, int keep, int chunk, float cap_log2, long long q_row_stride, int* __restrict__ err,
                             __nv_bfloat16* __restrict__ out, const float* __restrict__ sinks,
                             unsigned int* __restrict__ arrivals, int min_tiles) {
   extern __shared__ __align__(1024) uint8_t smem[];
@@ -353,8 +353,7 @@ paged_decode_persist_kernel(const __grid_constant__ CUtensorMap tk, const __grid
   // tile counts of the rows, then their exclusive prefix sum (warp 0: each lane a contiguous run of rows)
   for (int r = tid; r < rows; r += THREADS) {
     const int len = lengths[r];
-    const int first = first_key(len, window, chunk);
-    const int tiles = max(0, (len + TK - 1) / TK - first / TK);
+    const int tiles = TileWalk(len, window, keep, chunk, TK).n;
     prefix[r + 1] = tiles;
     if (tiles == 0 && (r % gridDim.x) == blockIdx.x)         // a row without keys: its output is zero
       for (int i = 0; i < Hq * D; ++i) out[static_cast<long long>(r) * Hq * D + i] = __float2bfloat16(0.f);
@@ -398,13 +397,13 @@ paged_decode_persist_kernel(const __grid_constant__ CUtensorMap tk, const __grid
       tma_prefetch_desc(&tv);
       bool ok = true;
       for (int u = u0; u < u1 && ok;) {
-        const Seg sg = locate(u, u1, prefix, lengths, rows, per_head, Q, window, chunk);
+        const Seg sg = locate(u, u1, prefix, lengths, rows, per_head, Q, window, keep, chunk);
         const int* table = page_table + static_cast<long long>(sg.row) * max_pages;
         for (int t = 0; t < sg.ntiles; ++t, ++tg) {
           const int s = tg % STAGES;
           const uint32_t ph = (tg / STAGES) & 1;
           if (!mbar_wait(&bars->empty[s], ph ^ 1, abort_flag)) { atomicCAS(err, 0, ERR_WAIT_EMPTY); ok = false; break; }
-          const int key0 = (sg.t_begin + t) * TK;
+          const int key0 = sg.walk.tile(sg.t_begin + t) * TK;
           const int page = table[key0 / page_size];
           const int row0 = page * page_size + key0 % page_size;
           uint8_t* st = smem + s * STAGE_BYTES;
@@ -426,7 +425,7 @@ paged_decode_persist_kernel(const __grid_constant__ CUtensorMap tk, const __grid
   const int g = lane >> 2, c = (lane & 3) * 2;
   bool ok = true;
   for (int u = u0; u < u1;) {
-    const Seg it = locate(u, u1, prefix, lengths, rows, per_head, Q, window, chunk);
+    const Seg it = locate(u, u1, prefix, lengths, rows, per_head, Q, window, keep, chunk);
     u += it.ntiles;
     // Q fragments straight from global memory: A operand rows = heads; rows 8..15 do not exist (a1 = a3 = 0)
     uint32_t qa0[8], qa2[8];
@@ -463,13 +462,15 @@ paged_decode_persist_kernel(const __grid_constant__ CUtensorMap tk, const __grid
         mma_16816(sc[0], qa0[ks], 0u, qa2[ks], 0u, b0, b1);
         mma_16816(sc[1], qa0[ks], 0u, qa2[ks], 0u, b2, b3);
       }
-      const int key_base = (it.t_begin + t) * TK + kw + (lane & 3) * 2;
+      const int key_base = it.walk.tile(it.t_begin + t) * TK + kw + (lane & 3) * 2;
       float pv[4];
       float mx = -INFINITY;
 #pragma unroll
       for (int i = 0; i < 4; ++i) {
         const int key = key_base + (i >> 1) * 8 + (i & 1);
-        const float v = (key >= it.first && key < it.len) ? sc[i >> 1][i & 1] * scale_log2 : -INFINITY;
+        float v = sc[i >> 1][i & 1] * scale_log2;
+        if (cap_log2 > 0.f) v = cap_log2 * attn::soft_tanh(v / cap_log2);
+        v = (key >= it.walk.first || key < keep) && key < it.len ? v : -INFINITY;
         pv[i] = v;
         mx = fmaxf(mx, v);
       }
@@ -584,10 +585,10 @@ paged_decode_persist_kernel(const __grid_constant__ CUtensorMap tk, const __grid
 extern "C" int dewb_paged_decode_stream(const void* q, const void* kpool, const void* vpool, long long pool_tokens,
                                         const int* page_table, const int* lengths, float* part_m, float* part_l,
                                         float* part_acc, int rows, int Hq, int Hkv, int page_size, int max_pages, int splits,
-                                        float scale, int window, int chunk, long long q_row_stride, int* err, void* stream_ptr) {
+                                        float scale, int window, int keep, int chunk, float softcap, long long q_row_stride, int* err, void* stream_ptr) {
   using namespace dewb::decode2;
   if (rows <= 0) return 0;
-  if (Hq % Hkv != 0 || Hq / Hkv > 8 || page_size % TK != 0 || splits < 1 || pool_tokens <= 0) return -3;
+  if (Hq % Hkv != 0 || Hq / Hkv > 8 || page_size % TK != 0 || keep < 0 || (keep > 0 && chunk > 0) || splits < 1 || pool_tokens <= 0) return -3;
   CUtensorMap tk, tv;
   int r;
   const uint64_t cols = static_cast<uint64_t>(Hkv) * D;
@@ -598,7 +599,7 @@ extern "C" int dewb_paged_decode_stream(const void* q, const void* kpool, const 
   dim3 grid(rows, Hkv, splits);
   paged_decode_tma_kernel<<<grid, THREADS, SMEM, reinterpret_cast<cudaStream_t>(stream_ptr)>>>(
       tk, tv, reinterpret_cast<const __nv_bfloat16*>(q), page_table, lengths, part_m, part_l, part_acc, Hq, Hkv, page_size,
-      max_pages, splits, scale * 1.4426950408889634f, window, chunk, q_row_stride > 0 ? q_row_stride : static_cast<long long>(Hq) * D, err,
+      max_pages, splits, scale * 1.4426950408889634f, window, keep, chunk, softcap * 1.4426950408889634f, q_row_stride > 0 ? q_row_stride : static_cast<long long>(Hq) * D, err,
       nullptr, nullptr, nullptr, 0);
   return static_cast<int>(cudaGetLastError());
 }
@@ -610,10 +611,10 @@ extern "C" int dewb_paged_decode_fused(const void* q, const void* kpool, const v
                                        const int* page_table, const int* lengths, float* part_m, float* part_l,
                                        float* part_acc, unsigned int* arrivals, const float* sinks, void* out, int rows, int Hq,
                                        int Hkv, int page_size, int max_pages, int splits, int chunk_tiles, float scale,
-                                       int window, int chunk, long long q_row_stride, int* err, void* stream_ptr) {
+                                       int window, int keep, int chunk, float softcap, long long q_row_stride, int* err, void* stream_ptr) {
   using namespace dewb::decode2;
   if (rows <= 0) return 0;
-  if (Hq % Hkv != 0 || Hq / Hkv > 8 || page_size % TK != 0 || splits < 1 || chunk_tiles < 1 || pool_tokens <= 0) return -3;
+  if (Hq % Hkv != 0 || Hq / Hkv > 8 || page_size % TK != 0 || keep < 0 || (keep > 0 && chunk > 0) || splits < 1 || chunk_tiles < 1 || pool_tokens <= 0) return -3;
   CUtensorMap tk, tv;
   int r;
   const uint64_t cols = static_cast<uint64_t>(Hkv) * D;
@@ -624,7 +625,7 @@ extern "C" int dewb_paged_decode_fused(const void* q, const void* kpool, const v
   dim3 grid(rows, Hkv, splits);
   paged_decode_tma_kernel<<<grid, THREADS, SMEM, reinterpret_cast<cudaStream_t>(stream_ptr)>>>(
       tk, tv, reinterpret_cast<const __nv_bfloat16*>(q), page_table, lengths, part_m, part_l, part_acc, Hq, Hkv, page_size,
-      max_pages, splits, scale * 1.4426950408889634f, window, chunk, q_row_stride > 0 ? q_row_stride : static_cast<long long>(Hq) * D, err,
+      max_pages, splits, scale * 1.4426950408889634f, window, keep, chunk, softcap * 1.4426950408889634f, q_row_stride > 0 ? q_row_stride : static_cast<long long>(Hq) * D, err,
       reinterpret_cast<__nv_bfloat16*>(out), sinks, arrivals, chunk_tiles);
   return static_cast<int>(cudaGetLastError());
 }
@@ -637,10 +638,10 @@ extern "C" int dewb_paged_decode_persist(const void* q, const void* kpool, const
                                          const int* page_table, const int* lengths, float* part_m, float* part_l,
                                          float* part_acc, unsigned int* arrivals, const float* sinks, void* out, int rows, int Hq,
                                          int Hkv, int page_size, int max_pages, int max_parts, int min_tiles, float scale,
-                                         int window, int chunk, long long q_row_stride, int ctas, int* err, void* stream_ptr) {
+                                         int window, int keep, int chunk, float softcap, long long q_row_stride, int ctas, int* err, void* stream_ptr) {
   using namespace dewb::decode2;
   if (rows <= 0) return 0;
-  if (Hq % Hkv != 0 || Hq / Hkv > 8 || page_size % TK != 0 || max_parts < 2 || min_tiles < 1 || pool_tokens <= 0 ||
+  if (Hq % Hkv != 0 || Hq / Hkv > 8 || page_size % TK != 0 || keep < 0 || (keep > 0 && chunk > 0) || max_parts < 2 || min_tiles < 1 || pool_tokens <= 0 ||
       rows > P_MAXROWS || ctas < 1)
     return -3;
   CUtensorMap tk, tv;
@@ -652,7 +653,7 @@ extern "C" int dewb_paged_decode_persist(const void* q, const void* kpool, const
   if (e != cudaSuccess) return static_cast<int>(e);
   paged_decode_persist_kernel<<<ctas, THREADS, P_SMEM, reinterpret_cast<cudaStream_t>(stream_ptr)>>>(
       tk, tv, reinterpret_cast<const __nv_bfloat16*>(q), page_table, lengths, part_m, part_l, part_acc, rows, Hq, Hkv, page_size,
-      max_pages, max_parts, scale * 1.4426950408889634f, window, chunk, q_row_stride > 0 ? q_row_stride : static_cast<long long>(Hq) * D, err,
+      max_pages, max_parts, scale * 1.4426950408889634f, window, keep, chunk, softcap * 1.4426950408889634f, q_row_stride > 0 ? q_row_stride : static_cast<long long>(Hq) * D, err,
       reinterpret_cast<__nv_bfloat16*>(out), sinks, arrivals, min_tiles);
   return static_cast<int>(cudaGetLastError());
 }

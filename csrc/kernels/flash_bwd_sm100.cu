@@ -28,7 +28,7 @@ constexpr int THREADS = 320;            // 8 softmax warps (two threads per TMEM
 constexpr int TMA_WARP = 8, MMA_WARP = 9;
 constexpr float LOG2E = 1.4426950408889634f;
 using attn::Variant;
-using attn::fast_tanh;
+using attn::soft_tanh;
 
 __device__ __forceinline__ void named_barrier_sync(int id, int threads) {
   asm volatile("bar.sync %0, %1;" ::"r"(id), "r"(threads) : "memory");
@@ -296,7 +296,7 @@ flash_dq_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__ 
             float x0 = __uint_as_float(sv[i]) * scale_log2, x1 = __uint_as_float(sv[i + 1]) * scale_log2;
             float f0 = 1.f, f1 = 1.f;               // d(capped score) / d(score)
             if (VAR && var.softcap > 0.f) {
-              const float t0 = fast_tanh(x0 * inv_cap2), t1 = fast_tanh(x1 * inv_cap2);
+              const float t0 = soft_tanh(x0 * inv_cap2), t1 = soft_tanh(x1 * inv_cap2);
               x0 = cap2 * t0; x1 = cap2 * t1;
               f0 = 1.f - t0 * t0; f1 = 1.f - t1 * t1;
             }
@@ -599,8 +599,8 @@ flash_dkv_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__
             float x2 = __uint_as_float(sv[i + 2]) * scale_log2, x3 = __uint_as_float(sv[i + 3]) * scale_log2;
             float f0 = 1.f, f1 = 1.f, f2 = 1.f, f3 = 1.f;       // d(capped score) / d(score)
             if (VAR && var.softcap > 0.f) {
-              const float t0 = fast_tanh(x0 * inv_cap2), t1 = fast_tanh(x1 * inv_cap2);
-              const float t2 = fast_tanh(x2 * inv_cap2), t3 = fast_tanh(x3 * inv_cap2);
+              const float t0 = soft_tanh(x0 * inv_cap2), t1 = soft_tanh(x1 * inv_cap2);
+              const float t2 = soft_tanh(x2 * inv_cap2), t3 = soft_tanh(x3 * inv_cap2);
               x0 = cap2 * t0; x1 = cap2 * t1; x2 = cap2 * t2; x3 = cap2 * t3;
               f0 = 1.f - t0 * t0; f1 = 1.f - t1 * t1; f2 = 1.f - t2 * t2; f3 = 1.f - t3 * t3;
             }

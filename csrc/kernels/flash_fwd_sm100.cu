@@ -1,4 +1,8 @@
-// Flash attention forward for sm_100a (head_dim 128 or 64, bf16, causal or full, GQA).
+// Flash attention forward for sm_100a (bf16, causal or full, GQA): queries and keys up to 64, 128 or 192 wide, values up to 64 or 128.
+//
+// Queries and keys may come in two parts of their own widths (latent attention: an unrotated part per head, a rotated part whose keys all heads
+// share); each part fills whole 64-column sub-tiles of the operand, the columns past its width read as zeros.  `gate` multiplies the output by a
+// sigmoid, element by element, before it is written.
 //
 // One CTA per (query tile of 128 rows, query head, batch); 320 threads:
 //   warps 0..7  softmax      : two threads per query row (warps w and w + 4 share TMEM lane quarter w & 3 and take 64
@@ -32,19 +36,30 @@ __device__ __forceinline__ void named_barrier_sync(int id, int threads) {
 }
 
 using attn::Variant;
-using attn::fast_tanh;
 
-template <int D>
+// DK: width of a query / key row in shared memory, DV: of a value row
+template <int DK, int DV>
 struct Cfg {
-  static constexpr int SUB = D / 64;                 // 64-column (128-byte) sub-tiles per row
-  static constexpr int Q_BYTES = BM * D * 2;
-  static constexpr int KV_BYTES = BN * D * 2;
-  static constexpr int P_BYTES = BM * BN * 2;
-  static constexpr int KSTAGES = 3;                  // K is consumed one tile ahead of V: it needs the deeper ring
-  static constexpr int TILE_BYTES = Q_BYTES + (KSTAGES + 2) * KV_BYTES + P_BYTES;
+  static constexpr int SUB = DK / 64;                // 64-column (128-byte) sub-tiles per query / key row
+  static constexpr int SUBV = DV / 64;
+  static constexpr int Q_BYTES = BM * DK * 2;
+  static constexpr int K_BYTES = BN * DK * 2;
+  static constexpr int V_BYTES = BN * DV * 2;
+  static constexpr int P_BYTES = DK > 128 ? 0 : BM * BN * 2;         // wide keys leave no room for P: tensor-memory form only
+  static constexpr int KSTAGES = DK > 128 ? 2 : 3;   // K is consumed one tile ahead of V: it needs the deeper ring where it fits
+  static constexpr int TILE_BYTES = Q_BYTES + KSTAGES * K_BYTES + 2 * V_BYTES + P_BYTES;
   static constexpr int SMEM = TILE_BYTES + 2560;      // + barriers and the row-maximum exchange (see Bars); no slack to spare
   static constexpr int TMEM_S0 = 0, TMEM_S1 = 128, TMEM_O = 256, TMEM_COLS = 512;
-  static constexpr int TMEM_QA = 384;                // PT: Q as a tensor-memory A operand (D / 2 packed columns)
+  static constexpr int TMEM_QA = 384;                // PT: Q as a tensor-memory A operand (DK / 2 packed columns)
+  static_assert(DV <= 128 && TMEM_QA + DK / 2 <= TMEM_COLS, "accumulator and queries must fit the tensor memory");
+};
+
+// Where the parts of the queries and keys lie, and what happens to the output.
+struct Parts {
+  int first;                       // sub-tiles that come from the first part (all of them when there is only one)
+  int dv;                          // value columns written, a multiple of 8
+  const __nv_bfloat16* gate;       // [B * S, *] or null: head h's columns start at h * dv
+  long long gate_stride;           // elements between its rows
 };
 
 struct Bars {
@@ -56,7 +71,7 @@ struct Bars {
   uint32_t tmem_base;
   int abort_flag;
   int poisoned;
-  int j_lo;                            // first key tile this query tile sees (variants only)
+  int j_lo;                            // first key tile this query tile sees (variants only), the kept first ones aside
   float xmax[2][2][BM];   // [tile parity][column half][row]: partial row maxima exchanged between the two halves; the
                           // parity the last tile did not use carries the partial row sums at the end
 };
@@ -67,13 +82,14 @@ static_assert(sizeof(Bars) <= 2560, "Bars must fit the space Cfg::SMEM leaves af
 // probabilities (tcgen05.st) and the P V product reads its A operand from there, so P never crosses shared memory (no
 // 32 KB store + 32 KB operand fetch per tile) and the softmax of the next tile need not wait for the product to drain
 // a shared buffer.  PT = false is the shared-memory form (P in the 128-byte-swizzled K-major layout).
-template <int D, bool CAUSAL, bool PT, bool VAR>
+template <int DK, int DV, bool CAUSAL, bool PT, bool VAR>
 __global__ void __launch_bounds__(THREADS, 1)
 flash_fwd_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__ CUtensorMap tk,
-                 const __grid_constant__ CUtensorMap tv, __nv_bfloat16* __restrict__ out, float* __restrict__ lse,
+                 const __grid_constant__ CUtensorMap tv, const __grid_constant__ CUtensorMap tq2, const __grid_constant__ CUtensorMap tk2,
+                 __nv_bfloat16* __restrict__ out, float* __restrict__ lse,
                  int S, int T, int Hq, int Hkv, long long o_stride_b, long long o_stride_s, long long o_stride_h,
-                 float scale_log2, Variant var, int* __restrict__ err) {
-  using C = Cfg<D>;
+                 float scale_log2, Variant var, Parts parts, int* __restrict__ err) {
+  using C = Cfg<DK, DV>;
   extern __shared__ __align__(1024) uint8_t smem_raw[];
   // The tiles fill 224 KiB, so this kernel has no static shared memory and no alignment slack: the dynamic window must
   // start on a 1024-byte boundary (the 128-byte swizzle atoms need it). If it ever did not, refuse instead of overrunning.
@@ -84,8 +100,8 @@ flash_fwd_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__
   uint8_t* smem = smem_raw;
   uint8_t* sQ = smem;
   uint8_t* sK = sQ + C::Q_BYTES;             // KSTAGES stages
-  uint8_t* sV = sK + C::KSTAGES * C::KV_BYTES;   // 2 stages
-  uint8_t* sP = sV + 2 * C::KV_BYTES;
+  uint8_t* sV = sK + C::KSTAGES * C::K_BYTES;   // 2 stages
+  uint8_t* sP = sV + 2 * C::V_BYTES;
   Bars* bars = reinterpret_cast<Bars*>(sP + C::P_BYTES);
   {
     // An earlier launch reported a timed-out wait: leave at once instead of queueing more waits behind it. One
@@ -125,35 +141,42 @@ flash_fwd_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__
   tc_fence_after();
   const uint32_t tmem = bars->tmem_base;
   volatile int* abort_flag = &bars->abort_flag;
-  // every role walks the key tiles j_lo .. n_all - 1; rings, phases and "first tile" tests count from j_lo
+  // every role walks the kept first tiles, then the key tiles j_lo .. n_all - 1; rings, phases and "first tile" tests count the walk
   const int j_lo = VAR ? bars->j_lo : 0;
-  const int n_tiles = n_all - j_lo;
+  const int n_kept = VAR ? min(j_lo, (var.keep + BN - 1) / BN) : 0;
+  const int n_tiles = n_kept + n_all - j_lo;
+  auto tile_of = [&](int j) { return VAR ? (j < n_kept ? j : j_lo + j - n_kept) : j; };
 
   if (warp == TMA_WARP) {
     // ------------------------------------------------------------------ TMA producer
     if (lane == 0) {
       mbar_expect_tx(&bars->q_full, C::Q_BYTES);
 #pragma unroll
-      for (int t = 0; t < C::SUB; ++t) tma_load_4d(sQ + t * (BM * 128), &tq, &bars->q_full, t * 64, h, q0, b);
+      for (int t = 0; t < C::SUB; ++t)
+        tma_load_4d(sQ + t * (BM * 128), t < parts.first ? &tq : &tq2, &bars->q_full, (t < parts.first ? t : t - parts.first) * 64, h, q0, b);
       bool ok = true;
       for (int j = 0; j < n_tiles && ok; ++j) {
         const int st = j & 1; const uint32_t ph = (j >> 1) & 1;
         const int ks = j % C::KSTAGES; const uint32_t kph = (j / C::KSTAGES) & 1;
         if (!mbar_wait(&bars->k_empty[ks], kph ^ 1, abort_flag)) { atomicCAS(err, 0, ERR_WAIT_EMPTY); ok = false; break; }
-        mbar_expect_tx(&bars->k_full[ks], C::KV_BYTES);
+        const int key0 = tile_of(j) * BN;
+        mbar_expect_tx(&bars->k_full[ks], C::K_BYTES);
 #pragma unroll
-        for (int t = 0; t < C::SUB; ++t) tma_load_4d(sK + ks * C::KV_BYTES + t * (BN * 128), &tk, &bars->k_full[ks], t * 64, hk, (j_lo + j) * BN, b);
+        for (int t = 0; t < C::SUB; ++t) {
+          const bool one = t < parts.first;
+          tma_load_4d(sK + ks * C::K_BYTES + t * (BN * 128), one ? &tk : &tk2, &bars->k_full[ks], (one ? t : t - parts.first) * 64, one ? hk : 0, key0, b);
+        }
         if (!mbar_wait(&bars->v_empty[st], ph ^ 1, abort_flag)) { atomicCAS(err, 0, ERR_WAIT_EMPTY); ok = false; break; }
-        mbar_expect_tx(&bars->v_full[st], C::KV_BYTES);
+        mbar_expect_tx(&bars->v_full[st], C::V_BYTES);
 #pragma unroll
-        for (int t = 0; t < C::SUB; ++t) tma_load_4d(sV + st * C::KV_BYTES + t * (BN * 128), &tv, &bars->v_full[st], t * 64, hk, (j_lo + j) * BN, b);
+        for (int t = 0; t < C::SUBV; ++t) tma_load_4d(sV + st * C::V_BYTES + t * (BN * 128), &tv, &bars->v_full[st], t * 64, hk, key0, b);
       }
     }
   } else if (warp == MMA_WARP) {
     // ------------------------------------------------------------------ MMA issuer
     // The whole warp runs this loop and waits together; one elected lane issues (see mbar_wait_warp).
     constexpr uint32_t idesc_qk = make_idesc(BM, BN, 1, 1, 0, 0);
-    constexpr uint32_t idesc_pv = make_idesc(BM, D, 1, 1, 0, 1);
+    constexpr uint32_t idesc_pv = make_idesc(BM, DV, 1, 1, 0, 1);
     // PT: Q is the A operand of every score product of the CTA, so the softmax warps copy it once to tensor memory and
     // the score products fetch only K from shared memory
     bool ok = mbar_wait_warp(PT ? &bars->qa_ready : &bars->q_full, 0, abort_flag);
@@ -168,11 +191,11 @@ flash_fwd_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__
       // this one and the tensor pipe runs one thread's products in order, so no barrier is needed.
       if (!PT && !mbar_wait_warp(&bars->s_empty[st], ph ^ 1, abort_flag)) { if (lane == 0) atomicCAS(err, 0, ERR_WAIT_TMEM_EMPTY); return false; }
       tc_fence_after();
-      const uint32_t ka = smem_u32(sK + ks * C::KV_BYTES);
+      const uint32_t ka = smem_u32(sK + ks * C::K_BYTES);
       const uint32_t ts = tmem + (st ? C::TMEM_S1 : C::TMEM_S0);
       if (elect_one()) {
 #pragma unroll
-        for (int kk = 0; kk < D / 16; ++kk) {
+        for (int kk = 0; kk < DK / 16; ++kk) {
           const uint32_t off = (kk >> 2) * (BM * 128) + (kk & 3) * 32;
           if (PT) umma_bf16_ts(ts, tmem + C::TMEM_QA + kk * 8, make_sdesc_sw128(ka + off, 16, 1024), idesc_qk, kk > 0 ? 1u : 0u);
           else umma_bf16_ss(ts, make_sdesc_sw128(qa + off, 16, 1024), make_sdesc_sw128(ka + off, 16, 1024), idesc_qk, kk > 0 ? 1u : 0u);
@@ -190,7 +213,7 @@ flash_fwd_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__
       if (!mbar_wait_warp(&bars->p_full, j & 1, abort_flag)) { if (lane == 0) atomicCAS(err, 0, ERR_WAIT_OTHER); ok = false; break; }
       if (!mbar_wait_warp(&bars->v_full[st], ph, abort_flag)) { if (lane == 0) atomicCAS(err, 0, ERR_WAIT_FULL); ok = false; break; }
       tc_fence_after();
-      const uint32_t va = smem_u32(sV + st * C::KV_BYTES);
+      const uint32_t va = smem_u32(sV + st * C::V_BYTES);
       const uint32_t tp = tmem + (st ? C::TMEM_S1 : C::TMEM_S0);
       if (elect_one()) {
 #pragma unroll
@@ -224,7 +247,7 @@ flash_fwd_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__
       const bool got = mbar_wait(&bars->q_full, 0, abort_flag);
       if (!__all_sync(0xffffffffu, got)) { atomicCAS(err, 0, ERR_WAIT_FULL); ok = false; }
       if (ok) {
-        constexpr int CH16 = D / 16;                  // 16-byte chunks (8 features, 4 columns) per thread
+        constexpr int CH16 = DK / 16;                 // 16-byte chunks (8 features, 4 columns) per thread
 #pragma unroll
         for (int g4 = 0; g4 < CH16 / 4; ++g4) {
           uint32_t w[16];
@@ -267,13 +290,13 @@ flash_fwd_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__
         tc_fence_before();
         __syncwarp();
         if (!PT && lane == 0) mbar_arrive(&bars->s_empty[st]);   // the score buffer may be overwritten by tile j + 2
-        const int k0 = (j_lo + j) * BN + half * HC;
+        const int k0 = tile_of(j) * BN + half * HC;
         const int limit = CAUSAL ? (q0 + r + (T - S)) : (T - 1);   // last visible key index for this row
         if (VAR && var.softcap > 0.f) {
           // cap * tanh(score / cap), kept in the log2 domain: scale_log2 = scale * log2(e)
           const float inv_cap = 1.f / (var.softcap * 1.4426950408889634f), cap2 = var.softcap * 1.4426950408889634f;
 #pragma unroll
-          for (int i = 0; i < HC; ++i) s[i] = cap2 * fast_tanh(s[i] * inv_cap);
+          for (int i = 0; i < HC; ++i) s[i] = cap2 * attn::soft_tanh(s[i] * inv_cap);
         }
         if (k0 + HC - 1 > limit || k0 + HC > T) {
 #pragma unroll
@@ -286,7 +309,7 @@ flash_fwd_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__
             if (var.chunk > 0) first = max(first, at / var.chunk * var.chunk);
             if (k0 < first) {
 #pragma unroll
-              for (int i = 0; i < HC; ++i) if (k0 + i < first) s[i] = -INFINITY;
+              for (int i = 0; i < HC; ++i) if (k0 + i < first && k0 + i >= var.keep) s[i] = -INFINITY;
             }
           }
           if (var.q_seg != nullptr && k0 < T) {
@@ -338,9 +361,9 @@ flash_fwd_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__
         if (need) { m_used = m_new; l *= alpha; }
         if (j > 0) {
 #pragma unroll
-          for (int c = 0; c < D / 32; ++c) {           // this thread's half of the output columns
+          for (int c = 0; c < DV / 32; ++c) {           // this thread's half of the output columns
             uint32_t v[16];
-            const uint32_t col = C::TMEM_O + half * (D / 2) + c * 16;
+            const uint32_t col = C::TMEM_O + half * (DV / 2) + c * 16;
             tmem_ld_32x32b_x16(tmem + lane_addr + col, v);
             tmem_ld_wait();
 #pragma unroll
@@ -410,11 +433,11 @@ flash_fwd_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__
     if (ok) {
       tc_fence_after();
       const int row = q0 + r;
-      __nv_bfloat16* orow = out + b * o_stride_b + static_cast<long long>(row) * o_stride_s + h * o_stride_h + half * (D / 2);
+      __nv_bfloat16* orow = out + b * o_stride_b + static_cast<long long>(row) * o_stride_s + h * o_stride_h + half * (DV / 2);
 #pragma unroll
-      for (int c = 0; c < D / 64; ++c) {
+      for (int c = 0; c < DV / 64; ++c) {
         uint32_t v[32];
-        if (n_tiles > 0) { tmem_ld_32x32b_x32(tmem + lane_addr + C::TMEM_O + half * (D / 2) + c * 32, v); tmem_ld_wait(); }
+        if (n_tiles > 0) { tmem_ld_32x32b_x32(tmem + lane_addr + C::TMEM_O + half * (DV / 2) + c * 32, v); tmem_ld_wait(); }
         else {
 #pragma unroll
           for (int i = 0; i < 32; ++i) v[i] = 0;
@@ -423,11 +446,25 @@ flash_fwd_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__
           uint4* o4 = reinterpret_cast<uint4*>(orow + c * 32);
 #pragma unroll
           for (int q = 0; q < 4; ++q) {
+            const int col = half * (DV / 2) + c * 32 + q * 8;
+            if (col >= parts.dv) continue;
+            float o[8];
+#pragma unroll
+            for (int i = 0; i < 8; ++i) o[i] = __uint_as_float(v[q * 8 + i]) * inv;
+            if (parts.gate != nullptr) {
+              const uint4 z = *reinterpret_cast<const uint4*>(parts.gate + (static_cast<long long>(b) * S + row) * parts.gate_stride + h * parts.dv + col);
+              const uint32_t zw[4] = {z.x, z.y, z.z, z.w};
+#pragma unroll
+              for (int i = 0; i < 4; ++i) {
+                o[2 * i] = __fdividef(o[2 * i], 1.f + __expf(-__uint_as_float(zw[i] << 16)));
+                o[2 * i + 1] = __fdividef(o[2 * i + 1], 1.f + __expf(-__uint_as_float(zw[i] & 0xffff0000u)));
+              }
+            }
             uint4 pk;
-            pk.x = pack_bf16(__uint_as_float(v[q * 8 + 0]) * inv, __uint_as_float(v[q * 8 + 1]) * inv);
-            pk.y = pack_bf16(__uint_as_float(v[q * 8 + 2]) * inv, __uint_as_float(v[q * 8 + 3]) * inv);
-            pk.z = pack_bf16(__uint_as_float(v[q * 8 + 4]) * inv, __uint_as_float(v[q * 8 + 5]) * inv);
-            pk.w = pack_bf16(__uint_as_float(v[q * 8 + 6]) * inv, __uint_as_float(v[q * 8 + 7]) * inv);
+            pk.x = pack_bf16(o[0], o[1]);
+            pk.y = pack_bf16(o[2], o[3]);
+            pk.z = pack_bf16(o[4], o[5]);
+            pk.w = pack_bf16(o[6], o[7]);
             o4[q] = pk;
           }
         }
@@ -448,16 +485,17 @@ flash_fwd_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__
   }
 }
 
-template <int D, bool CAUSAL, bool PT, bool VAR>
-static int launch(const CUtensorMap& tq, const CUtensorMap& tk, const CUtensorMap& tv, void* out, float* lse, int B,
-                  int S, int T, int Hq, int Hkv, long long osb, long long oss, long long osh, float scale_log2,
-                  const Variant& var, int* err, cudaStream_t stream) {
-  auto kern = flash_fwd_kernel<D, CAUSAL, PT, VAR>;
-  cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, Cfg<D>::SMEM);
+template <int DK, int DV, bool CAUSAL, bool PT, bool VAR>
+static int launch(const CUtensorMap& tq, const CUtensorMap& tk, const CUtensorMap& tv, const CUtensorMap& tq2, const CUtensorMap& tk2, void* out,
+                  float* lse, int B, int S, int T, int Hq, int Hkv, long long osb, long long oss, long long osh, float scale_log2,
+                  const Variant& var, const Parts& parts, int* err, cudaStream_t stream) {
+  static_assert(PT || Cfg<DK, DV>::P_BYTES > 0, "P has no shared memory here");
+  auto kern = flash_fwd_kernel<DK, DV, CAUSAL, PT, VAR>;
+  cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, Cfg<DK, DV>::SMEM);
   if (e != cudaSuccess) return static_cast<int>(e);
   dim3 grid((S + BM - 1) / BM, Hq, B);
-  kern<<<grid, THREADS, Cfg<D>::SMEM, stream>>>(tq, tk, tv, reinterpret_cast<__nv_bfloat16*>(out), lse, S, T, Hq, Hkv,
-                                                 osb, oss, osh, scale_log2, var, err);
+  kern<<<grid, THREADS, Cfg<DK, DV>::SMEM, stream>>>(tq, tk, tv, tq2, tk2, reinterpret_cast<__nv_bfloat16*>(out), lse, S, T, Hq, Hkv,
+                                                      osb, oss, osh, scale_log2, var, parts, err);
   return static_cast<int>(cudaGetLastError());
 }
 
@@ -486,13 +524,13 @@ extern "C" int dewb_flash_set_variant(int variant) {
 
 // q [B,S,Hq,D], k/v [B,T,Hkv,D] (bf16, unit stride along D, other strides in elements: batch, sequence, head);
 // out [B,S,Hq,D] with its own strides; lse [B,Hq,S] fp32 (natural log), may be null.
-// Variants (each off at 0 / null): `window` keys visible behind each query, `chunk` positions a query sees no key from outside of, `softcap`, `sinks` [Hq] fp32, `q_seg` [B,S] /
+// Variants (each off at 0 / null): `window` keys visible behind each query, `keep` first keys visible beside a window, `chunk` positions a query sees no key from outside of, `softcap`, `sinks` [Hq] fp32, `q_seg` [B,S] /
 // `k_seg` [B,T] int32 segment ids of packed documents (non-decreasing along the sequence, rows 16-byte aligned: S, T % 4 == 0).
 extern "C" int dewb_flash_fwd_var(const void* q, const void* k, const void* v, void* out, float* lse, int B, int S, int T,
                                   int Hq, int Hkv, int D, long long q_sb, long long q_ss, long long q_sh, long long k_sb,
                                   long long k_ss, long long k_sh, long long v_sb, long long v_ss, long long v_sh,
                                   long long o_sb, long long o_ss, long long o_sh, float scale, int causal, int window,
-                                  int chunk, float softcap, const float* sinks, const int* q_seg, const int* k_seg, int* err,
+                                  int keep, int chunk, float softcap, const float* sinks, const int* q_seg, const int* k_seg, int* err,
                                   void* stream_ptr) {
   using namespace dewb::attnfwd;
   if (D != 128 && D != 64) return -3;
@@ -502,7 +540,8 @@ extern "C" int dewb_flash_fwd_var(const void* q, const void* k, const void* v, v
     return -3;
   if ((q_seg != nullptr) != (k_seg != nullptr)) return -3;
   if (q_seg != nullptr && ((T % 4) || (reinterpret_cast<uintptr_t>(k_seg) & 15))) return -3;
-  if (window < 0 || chunk < 0 || softcap < 0.f) return -3;
+  if (window < 0 || keep < 0 || chunk < 0 || softcap < 0.f) return -3;
+  if (keep > 0 && (window == 0 || chunk > 0)) return -3;
   CUtensorMap tq, tk, tv;
   int r;
   if ((r = make_qkv_map(&tq, q, B, S, Hq, D, q_sb, q_ss, q_sh))) return 1000 + r;
@@ -510,9 +549,10 @@ extern "C" int dewb_flash_fwd_var(const void* q, const void* k, const void* v, v
   if ((r = make_qkv_map(&tv, v, B, T, Hkv, D, v_sb, v_ss, v_sh))) return 3000 + r;
   const float scale_log2 = scale * 1.4426950408889634f;
   cudaStream_t stream = reinterpret_cast<cudaStream_t>(stream_ptr);
-  const Variant var{window, softcap, sinks, q_seg, k_seg, chunk};
+  const Variant var{window, softcap, sinks, q_seg, k_seg, chunk, keep};
+  const Parts parts{D / 64, D, nullptr, 0};
   const bool any = window > 0 || chunk > 0 || softcap > 0.f || sinks != nullptr || q_seg != nullptr;
-#define DEWB_FLASH_GO(DD, CC, PP, VV) launch<DD, CC, PP, VV>(tq, tk, tv, out, lse, B, S, T, Hq, Hkv, o_sb, o_ss, o_sh, scale_log2, var, err, stream)
+#define DEWB_FLASH_GO(DD, CC, PP, VV) launch<DD, DD, CC, PP, VV>(tq, tk, tv, tq, tk, out, lse, B, S, T, Hq, Hkv, o_sb, o_ss, o_sh, scale_log2, var, parts, err, stream)
   const bool pt = g_variant != 0;
   if (any) {
     // the variants run the tensor-memory form only
@@ -534,5 +574,39 @@ extern "C" int dewb_flash_fwd(const void* q, const void* k, const void* v, void*
                               long long o_sb, long long o_ss, long long o_sh, float scale, int causal, int* err,
                               void* stream_ptr) {
   return dewb_flash_fwd_var(q, k, v, out, lse, B, S, T, Hq, Hkv, D, q_sb, q_ss, q_sh, k_sb, k_ss, k_sh, v_sb, v_ss, v_sh, o_sb,
-                            o_ss, o_sh, scale, causal, 0, 0, 0.f, nullptr, nullptr, nullptr, err, stream_ptr);
+                            o_ss, o_sh, scale, causal, 0, 0, 0, 0.f, nullptr, nullptr, nullptr, err, stream_ptr);
+}
+
+// Causal attention whose queries and keys come in two parts: q [B,S,H,da + db] and keys [B,T,H,da] per head (strides in elements: batch, sequence,
+// head) beside k2 [B,T,db], which all heads share; v [B,T,H,dv]; out [B,S,H,dv] contiguous, times sigmoid(gate [B*S, H dv], rows gate_stride apart)
+// where gate is not null.  Query i sees the keys up to i + T - S.  da, db, dv multiples of 8; whole sub-tiles of 64 columns for each part: three at
+// most together, dv <= 128.
+extern "C" int dewb_flash_fwd_parts(const void* q, const void* k, const void* k2, const void* v, const void* gate, long long gate_stride, void* out,
+                                    int B, int S, int T, int H, int da, int db, int dv, long long q_sb, long long q_ss, long long q_sh,
+                                    long long k_sb, long long k_ss, long long k_sh, long long k2_sb, long long k2_ss, long long v_sb,
+                                    long long v_ss, long long v_sh, float scale, int* err, void* stream_ptr) {
+  using namespace dewb::attnfwd;
+  if (B <= 0 || S <= 0 || H <= 0) return 0;
+  if (da < 8 || db < 8 || dv < 8 || da % 8 || db % 8 || dv % 8 || dv > 128 || T < S) return -3;
+  if ((q_ss % 8) || (q_sh % 8) || (q_sb % 8) || (k_ss % 8) || (k_sh % 8) || (k_sb % 8) || (k2_ss % 8) || (k2_sb % 8) || (v_ss % 8) || (v_sh % 8) || (v_sb % 8) ||
+      (gate_stride % 8) || (reinterpret_cast<uintptr_t>(gate) & 15) || (reinterpret_cast<uintptr_t>(out) & 15))
+    return -3;
+  const int first = (da + 63) / 64, sub = first + (db + 63) / 64;
+  if (sub > 3) return -3;
+  CUtensorMap tq, tk, tv, tq2, tk2;
+  int r;
+  if ((r = make_qkv_map(&tq, q, B, S, H, da, q_sb, q_ss, q_sh))) return 1000 + r;
+  if ((r = make_qkv_map(&tq2, static_cast<const __nv_bfloat16*>(q) + da, B, S, H, db, q_sb, q_ss, q_sh))) return 1500 + r;
+  if ((r = make_qkv_map(&tk, k, B, T, H, da, k_sb, k_ss, k_sh))) return 2000 + r;
+  if ((r = make_qkv_map(&tk2, k2, B, T, 1, db, k2_sb, k2_ss, k2_ss))) return 2500 + r;
+  if ((r = make_qkv_map(&tv, v, B, T, H, dv, v_sb, v_ss, v_sh))) return 3000 + r;
+  cudaStream_t stream = reinterpret_cast<cudaStream_t>(stream_ptr);
+  const Variant var{0, 0.f, nullptr, nullptr, nullptr, 0, 0};
+  const Parts parts{first, dv, static_cast<const __nv_bfloat16*>(gate), gate_stride};
+  const long long oss = static_cast<long long>(H) * dv, osb = oss * S;
+#define DEWB_PARTS_GO(KK, VV) launch<KK, VV, true, true, false>(tq, tk, tv, tq2, tk2, out, nullptr, B, S, T, H, H, osb, oss, dv, \
+    scale * 1.4426950408889634f, var, parts, err, stream)
+  if (sub == 2) return dv <= 64 ? DEWB_PARTS_GO(128, 64) : DEWB_PARTS_GO(128, 128);
+  return dv <= 64 ? DEWB_PARTS_GO(192, 64) : DEWB_PARTS_GO(192, 128);
+#undef DEWB_PARTS_GO
 }

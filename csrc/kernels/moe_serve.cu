@@ -8,7 +8,8 @@
 //   moe_glu       silu(gate) * up on the rows in use
 //   moe_combine   a token's rows times their weights, plus the shared expert's output times its gate, in fp32
 //
-// Selection: scores are a sigmoid or softmax of the logits; choice scores add a bias that steers the choice only; with groups, a group counts
+// Selection: logits may carry a bias; scores are a sigmoid or softmax of the logits, or the logits themselves, whose weights are then the softmax over
+// the chosen ones alone; choice scores add a bias that steers the choice only; with groups, a group counts
 // the sum of its two best choice scores and the experts outside a token's best groups are out of the choice (their choice scores become
 // `fill`); the weights are the chosen scores, divided by their sum where `norm` asks for it.  Tokens at positions below 0 are padding: no
 // expert runs for them.  A row's place among its expert's rows comes from an atomic counter, so it may differ from run to run; the rows of a
@@ -38,10 +39,11 @@ __device__ __forceinline__ float ld(const float* p) { return *p; }
 __device__ __forceinline__ float ld(const bf16* p) { return __bfloat162float(*p); }
 
 struct Choice {
-  const float* bias;       // [E] or null
+  const float* bias;       // [E] or null: steers the choice alone
+  const float* logit_bias;  // [E] or null: part of the logits
   int E, k, groups, keep;
   float fill;              // choice score of experts outside the kept groups
-  int sigmoid, norm;
+  int score, norm;         // score 0: softmax, 1: sigmoid, 2: the logits, weights by the softmax over the chosen ones
   float scaling;
   float* weights;          // [T, k]
   int* ids;                // [T, k], -1: padding
@@ -57,10 +59,14 @@ __device__ __forceinline__ void choose(const Choice& c, long long t, bool live, 
     if (lane < c.k) { c.weights[t * c.k + lane] = 0.f; c.ids[t * c.k + lane] = -1; }
     return;
   }
-  if (c.sigmoid) {
+  if (c.logit_bias != nullptr) {
+#pragma unroll
+    for (int i = 0; i < NI; ++i) if (lane + 32 * i < c.E) sc[i] += c.logit_bias[lane + 32 * i];
+  }
+  if (c.score == 1) {
 #pragma unroll
     for (int i = 0; i < NI; ++i) sc[i] = sigmoid(sc[i]);
-  } else {
+  } else if (c.score == 0) {
     float mx = -INFINITY, sum = 0.f;
 #pragma unroll
     for (int i = 0; i < NI; ++i) if (lane + 32 * i < c.E) mx = fmaxf(mx, sc[i]);
@@ -126,8 +132,16 @@ __device__ __forceinline__ void choose(const Choice& c, long long t, bool live, 
     wsum += bs;
     if (lane == j) { my_w = bs; my_id = bi; }
   }
+  if (c.score == 2) {
+    float mx = lane < c.k ? my_w : -INFINITY;
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(FULL, mx, o));
+    my_w = lane < c.k ? expf(my_w - mx) : 0.f;
+    my_w /= warp_sum(my_w);
+  } else if (c.norm) {
+    my_w = my_w / (wsum + 1e-20f);
+  }
   if (lane < c.k) {
-    if (c.norm) my_w = my_w / (wsum + 1e-20f);
     c.weights[t * c.k + lane] = my_w * c.scaling;
     c.ids[t * c.k + lane] = my_id;
     c.rank[t * c.k + lane] = atomicAdd(c.counts + my_id, 1);
@@ -393,7 +407,7 @@ moe_combine_kernel(const T* __restrict__ y, const float* __restrict__ weights, c
 }
 
 bool choice_ok(const Choice& c) {
-  return c.E >= 1 && c.E <= MAX_E && c.k >= 1 && c.k <= MAX_K && c.k <= c.E && c.groups >= 1 && c.E % c.groups == 0 && c.keep >= 1 && c.keep <= c.groups &&
+  return c.score >= 0 && c.score <= 2 && c.E >= 1 && c.E <= MAX_E && c.k >= 1 && c.k <= MAX_K && c.k <= c.E && c.groups >= 1 && c.E % c.groups == 0 && c.keep >= 1 && c.keep <= c.groups &&
          c.weights != nullptr && c.ids != nullptr && c.rank != nullptr && c.counts != nullptr;
 }
 
@@ -445,11 +459,11 @@ using namespace dewb::moeserve;
 
 // logits [T, ld] fp32 (plus logits[., rest + e] when rest > 0) -> weights, ids, rank [T, k], counts [E] (zero before the call).
 // `positions` [T] or null: below 0 = padding.
-extern "C" int dewb_moe_select(const float* logits, long long ld_, int rest, const float* bias, const int* positions, int T, int E, int k, int groups,
-                               int keep, float fill, int sigmoid, int norm, float scaling, float* weights, int* ids, int* rank, int* counts,
+extern "C" int dewb_moe_select(const float* logits, long long ld_, int rest, const float* bias, const float* logit_bias, const int* positions, int T,
+                               int E, int k, int groups, int keep, float fill, int score, int norm, float scaling, float* weights, int* ids, int* rank, int* counts,
                                void* stream_ptr) {
   if (T <= 0) return 0;
-  const Choice c{bias, E, k, groups, keep, fill, sigmoid, norm, scaling, weights, ids, rank, counts};
+  const Choice c{bias, logit_bias, E, k, groups, keep, fill, score, norm, scaling, weights, ids, rank, counts};
   if (!choice_ok(c) || ld_ < E || rest < 0 || (rest > 0 && ld_ < rest + E)) return -3;
   cudaStream_t stream = reinterpret_cast<cudaStream_t>(stream_ptr);
   if (E <= 128) return select<4>(logits, ld_, rest, positions, T, c, stream);
@@ -458,11 +472,11 @@ extern "C" int dewb_moe_select(const float* logits, long long ld_, int rest, con
 }
 
 // The same with the logits made here: x [T, d] (fp32 or bf16), w [E, d] (fp32, or bf16 beside a bf16 x).
-extern "C" int dewb_moe_router(const void* x, const void* w, const float* bias, const int* positions, int T, int d, int E, int k, int groups, int keep,
-                               float fill, int sigmoid, int norm, float scaling, float* weights, int* ids, int* rank, int* counts, int x_fp32,
+extern "C" int dewb_moe_router(const void* x, const void* w, const float* bias, const float* logit_bias, const int* positions, int T, int d, int E,
+                               int k, int groups, int keep, float fill, int score, int norm, float scaling, float* weights, int* ids, int* rank, int* counts, int x_fp32,
                                int w_fp32, void* stream_ptr) {
   if (T <= 0) return 0;
-  const Choice c{bias, E, k, groups, keep, fill, sigmoid, norm, scaling, weights, ids, rank, counts};
+  const Choice c{bias, logit_bias, E, k, groups, keep, fill, score, norm, scaling, weights, ids, rank, counts};
   if (!choice_ok(c) || d < 1 || (x_fp32 && !w_fp32)) return -3;
   cudaStream_t stream = reinterpret_cast<cudaStream_t>(stream_ptr);
   const bool vec = d % 4 == 0 && aligned(x, 16) && aligned(w, 16);

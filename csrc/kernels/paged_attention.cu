@@ -3,15 +3,17 @@
 //   qk_norm_append   from the packed projection [tokens, H dk + G dk + G dv]: RMS norm of q over all its heads at once and of k likewise
 //                    (weights may be null: no norm), the query temperature 1 + coef ln(floor((p + 1) / every) + 1), the copy into heads
 //                    of the cache's (padded) width, and the append of keys and values to the page pools
-//   head_norm_append   the same for per-head norms (one weight for all heads), with the projection's bias added on the way, rows that carry
-//                    more columns than the heads (gates), and layers that read another layer's keys and values (queries alone)
+//   head_norm_append   the same for per-head norms (one weight for all heads, or no weight), with the projection's bias added on the way, rows that
+//                    carry more columns than the heads (gates), layers that read another layer's keys and values (queries alone), and the rotation
+//                    of the first columns of every query and key head by a call's table of cosines and sines
+//   rotary_angles    that table, from the positions and the pairs' frequencies
 //   head_gate        heads of the cache's width times a sigmoid of one number per head, packed to their own width
 //   paged_attend     causal attention of a call's tokens against everything the cache holds of their rows (any start positions; a decode
 //                    step is the case of one token per row); scores, softmax and sums in fp32 on the CUDA cores.  It is the fp32 form,
 //                    and takes the head widths the tensor-core kernels do not.
 //   paged_attend_mma   the same on the tensor cores for bf16 pools 64, 128 or 256 wide (a prompt's later portions, mixed start positions)
-//   Both take chunks (a query sees no key from before the start of its chunk of positions), a learned sink per head in the denominator, and
-//   a gate per head on the output.
+//   Both take chunks (a query sees no key from before the start of its chunk of positions), a window beside which the row's first keys may stay
+//   visible, a soft cap on the scores, a learned sink per head in the denominator, and a gate per head on the output.
 //
 // A query's row of work is (token, head of its group), so a group's heads share the key and value tiles.  Positions below 0 are padding:
 // nothing is appended for them and their outputs are zero.  Compiled without fast math.
@@ -100,12 +102,93 @@ qk_norm_append_kernel(const T* __restrict__ qkv, const T* __restrict__ qw, const
   }
 }
 
-// One group of LG lanes per (token, head); heads [0, H) queries, then G keys, then G values (G 0: queries alone).  ONE: a head is at most LG V
-// wide, so it is read once.
-template <typename T, int V, int LG, bool ONE>
+// positions [n] -> out [n, half] (cosine, sine) of position * frequency[i]; the angle is formed in double precision
+__global__ void __launch_bounds__(256)
+rotary_angles_kernel(const int* __restrict__ positions, const double* __restrict__ frequency, float2* __restrict__ out, long long n, int half) {
+  const long long at = static_cast<long long>(blockIdx.x) * 256 + threadIdx.x;
+  if (at >= n * half) return;
+  const int p = positions[at / half];
+  double s, c;
+  sincos(static_cast<double>(p > 0 ? p : 0) * frequency[at % half], &s, &c);
+  out[at] = make_float2(static_cast<float>(c), static_cast<float>(s));
+}
+
+// The rotation of one call: the first `dims` columns of a head turn by `table` [tokens, dims / 2] (cosine, sine); null: none.
+struct Turn {
+  const float2* table;
+  int dims, interleaved;
+};
+
+// V consecutive columns of a head starting at `i`, the bias added and each times the head's `gain` and its weight, with the columns below
+// `turn.dims` rotated by this token's angles.  src, b, w point at the head's first column; every column that is read lies within the head.
+template <typename T, int V>
+__device__ __forceinline__ void head_columns(const T* src, const T* b, const T* w, float gain, int i, const float2* angle, int dims, int interleaved,
+                                             float (&a)[V]) {
+  auto column = [&](int c) {
+    float x = ld(src + c);
+    if (b != nullptr) x += ld(b + c);
+    return w != nullptr ? x * gain * ld(w + c) : x * gain;
+  };
+  auto columns = [&](int c, float (&x)[V]) {
+    load_v<V>(src + c, x);
+    if (b != nullptr) {
+      float y[V];
+      load_v<V>(b + c, y);
+#pragma unroll
+      for (int j = 0; j < V; ++j) x[j] += y[j];
+    }
+    if (w != nullptr) {
+      float y[V];
+      load_v<V>(w + c, y);
+#pragma unroll
+      for (int j = 0; j < V; ++j) x[j] = x[j] * gain * y[j];
+    } else {
+#pragma unroll
+      for (int j = 0; j < V; ++j) x[j] *= gain;
+    }
+  };
+  columns(i, a);
+  if (angle == nullptr || i >= dims) return;
+  const int half = dims / 2;
+  if (!interleaved && half % V == 0) {
+    float other[V];
+    const bool low = i < half;
+    columns(low ? i + half : i - half, other);
+    const float2* t = angle + (low ? i : i - half);
+#pragma unroll
+    for (int j = 0; j < V; ++j) a[j] = low ? a[j] * t[j].x - other[j] * t[j].y : a[j] * t[j].x + other[j] * t[j].y;
+    return;
+  }
+  if constexpr (V > 1) {
+    if (interleaved) {
+#pragma unroll
+      for (int j = 0; j < V; j += 2)
+        if (i + j < dims) {
+          const float2 t = angle[(i + j) / 2];
+          const float u = a[j], v = a[j + 1];
+          a[j] = u * t.x - v * t.y;
+          a[j + 1] = v * t.x + u * t.y;
+        }
+      return;
+    }
+  }
+#pragma unroll
+  for (int j = 0; j < V; ++j) {
+    const int c = i + j;
+    if (c >= dims) break;
+    const bool low = interleaved ? c % 2 == 0 : c < half;
+    const float other = column(interleaved ? (low ? c + 1 : c - 1) : low ? c + half : c - half);
+    const float2 t = angle[interleaved ? c / 2 : low ? c : c - half];
+    a[j] = low ? a[j] * t.x - other * t.y : a[j] * t.x + other * t.y;
+  }
+}
+
+// One group of LG lanes per (token, head); heads [0, H) queries, then G keys, then G values (G 0: queries alone).  Queries and keys pass an RMS norm
+// where they have a weight or `unit` asks for it (a rotation keeps a head's square sum, so one without a weight may stand before or behind it).
+template <typename T, int V, int LG>
 __global__ void __launch_bounds__(256)
 head_norm_append_kernel(const T* __restrict__ qkv, long long row_stride, const T* __restrict__ bias, const T* __restrict__ qw, const T* __restrict__ kw,
-                        float eps, const int* __restrict__ positions, long long items, int S, int H, int G, int dk, int dv, int D,
+                        float eps, int unit, Turn turn, const int* __restrict__ positions, long long items, int S, int H, int G, int dk, int dv, int D,
                         T* __restrict__ packed, T* __restrict__ kpool, T* __restrict__ vpool, Pool pool) {
   const unsigned item = blockIdx.x * (256 / LG) + threadIdx.x / LG;
   const int lane = threadIdx.x % LG;
@@ -118,12 +201,12 @@ head_norm_append_kernel(const T* __restrict__ qkv, long long row_stride, const T
   const T* src = qkv + t * row_stride + at;
   const T* b = bias == nullptr ? nullptr : bias + at;
   const T* w = part == 0 ? qw : part == 1 ? kw : nullptr;
+  const bool normed = part != 2 && (w != nullptr || unit);
   const int pos = part != 0 ? positions[t] : -1;
-  float ss = 0.f, a[V];
-#pragma unroll
-  for (int j = 0; j < V; ++j) a[j] = 0.f;
-  if (ONE || w != nullptr) {
+  float ss = 0.f;
+  if (normed) {
     for (int i = lane * V; i < width; i += LG * V) {
+      float a[V];
       load_v<V>(src + i, a);
       if (b != nullptr) {
         float c[V];
@@ -138,7 +221,8 @@ head_norm_append_kernel(const T* __restrict__ qkv, long long row_stride, const T
 #pragma unroll
   for (int o = LG / 2; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
   if (!on) return;
-  const float r = w != nullptr ? 1.f / sqrtf(ss / width + eps) : 1.f;
+  const float r = normed ? 1.f / sqrtf(ss / width + eps) : 1.f;
+  const float2* angle = part != 2 && turn.table != nullptr ? turn.table + t * (turn.dims / 2) : nullptr;
   T* dst = packed + static_cast<long long>(item) * D;
   T* to_pool = nullptr;
   if (pos >= 0) {
@@ -146,26 +230,12 @@ head_norm_append_kernel(const T* __restrict__ qkv, long long row_stride, const T
     to_pool = (part == 1 ? kpool : vpool) + (tok * G + (part == 1 ? h - H : h - H - G)) * D;
   }
   for (int i = lane * V; i < D; i += LG * V) {
-    if (!ONE) {
+    float a[V];
+    if (i < width) {
+      head_columns<T, V>(src, b, w, r, i, angle, turn.dims, turn.interleaved, a);
+    } else {
 #pragma unroll
       for (int j = 0; j < V; ++j) a[j] = 0.f;
-    }
-    if (i < width) {
-      if (!ONE) {
-        load_v<V>(src + i, a);
-        if (b != nullptr) {
-          float c[V];
-          load_v<V>(b + i, c);
-#pragma unroll
-          for (int j = 0; j < V; ++j) a[j] += c[j];
-        }
-      }
-      if (w != nullptr) {
-        float c[V];
-        load_v<V>(w + i, c);
-#pragma unroll
-        for (int j = 0; j < V; ++j) a[j] = a[j] * r * c[j];
-      }
     }
     store_v<V>(dst + i, a);
     if (to_pool != nullptr) store_v<V>(to_pool + i, a);
@@ -194,12 +264,20 @@ head_gate_kernel(const T* __restrict__ o, const T* __restrict__ gate, long long 
 template <typename T>
 struct Extras {
   int chunk;               // a query sees no key from before the start of its chunk
+  int window, keep;        // a query sees its last `window` keys (its own among them) and the row's first `keep`
+  float cap;               // scores become cap tanh(score / cap); the tensor-core form holds it in the log2 domain
   const float* sinks;      // [H]: joins the denominator, has no value
   const T* gate;           // [tokens, *]: head h's output times sigmoid(gate[token, h])
   long long gate_stride;
 };
 
-__device__ __forceinline__ int chunk_start(int pos, int chunk) { return chunk > 0 && pos > 0 ? pos / chunk * chunk : 0; }
+// First key a query sees, the kept ones aside.
+template <typename T>
+__device__ __forceinline__ int first_seen(int pos, const Extras<T>& ex) {
+  if (pos <= 0) return 0;
+  const int start = ex.chunk > 0 ? pos / ex.chunk * ex.chunk : 0;
+  return ex.window > 0 ? max(start, pos - ex.window + 1) : start;
+}
 
 constexpr int BQ = 32, BK = 32, THREADS = 256;
 
@@ -228,7 +306,7 @@ paged_attend_kernel(const T* __restrict__ q, long long q_token_stride, const T* 
   int last = -1, lowest = INT_MAX;
   for (int i = 0; i < BQ; ++i) {
     last = max(last, s_pos[i]);
-    if (s_pos[i] >= 0) lowest = min(lowest, chunk_start(s_pos[i], ex.chunk));
+    if (s_pos[i] >= 0) lowest = min(lowest, first_seen(s_pos[i], ex));
   }
   for (int i = tid; i < BQ * kst; i += THREADS) {
     const int r = i / kst, c = i - r * kst;
@@ -240,11 +318,14 @@ paged_attend_kernel(const T* __restrict__ q, long long q_token_stride, const T* 
     sq[i] = v;
   }
   const int qr = tid >> 3, ql = tid & 7;
-  const int my_pos = s_pos[qr], my_first = chunk_start(my_pos, ex.chunk);
+  const int my_pos = s_pos[qr], my_first = first_seen(my_pos, ex);
   float m = -INFINITY, l = 0.f, acc[NJ][4];
 #pragma unroll
   for (int j = 0; j < NJ; ++j) { acc[j][0] = acc[j][1] = acc[j][2] = acc[j][3] = 0.f; }
-  for (int k0 = last < 0 ? 0 : lowest / BK * BK; k0 <= last; k0 += BK) {
+  // the tiles of the kept first keys, then those from the lowest first key on
+  const int lo = last < 0 ? 0 : lowest / BK, kept = last < 0 ? 0 : min((ex.keep + BK - 1) / BK, lo), tiles = kept + (last + BK) / BK - lo;
+  for (int t = 0; t < tiles; ++t) {
+    const int k0 = (t < kept ? t : lo + t - kept) * BK;
     __syncthreads();
     if (tid < BK) s_tok[tid] = k0 + tid <= last ? pool_token(pool, row, k0 + tid) : -1;
     __syncthreads();
@@ -269,7 +350,9 @@ paged_attend_kernel(const T* __restrict__ q, long long q_token_stride, const T* 
     float bm = -INFINITY;
 #pragma unroll
     for (int j = 0; j < 4; ++j) {
-      if (k0 + ql + 8 * j > my_pos || k0 + ql + 8 * j < my_first) s[j] = -INFINITY;
+      if (ex.cap > 0.f) s[j] = ex.cap * tanhf(s[j] / ex.cap);
+      const int key = k0 + ql + 8 * j;
+      if (key > my_pos || (key < my_first && key >= ex.keep)) s[j] = -INFINITY;
       bm = fmaxf(bm, s[j]);
     }
 #pragma unroll
@@ -327,6 +410,9 @@ __device__ __forceinline__ void cp16(uint32_t dst, const void* src, bool live) {
   asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst), "l"(src), "r"(n) : "memory");
 }
 
+// tanh to fp32 accuracy relative to 1
+__device__ __forceinline__ float soft_tanh(float x) { return 1.f - __fdividef(2.f, 1.f + exp2f(x * 2.8853900817779268f)); }
+
 template <int D>
 __global__ void __launch_bounds__(MTHREADS)
 paged_attend_mma_kernel(const bf16* __restrict__ q, long long q_token_stride, const bf16* __restrict__ kpool, const bf16* __restrict__ vpool,
@@ -350,10 +436,11 @@ paged_attend_mma_kernel(const bf16* __restrict__ q, long long q_token_stride, co
   int last = -1, lowest = INT_MAX;
   for (int i = 0; i < MQ; ++i) {
     last = max(last, s_pos[i]);
-    if (s_pos[i] >= 0) lowest = min(lowest, chunk_start(s_pos[i], ex.chunk));
+    if (s_pos[i] >= 0) lowest = min(lowest, first_seen(s_pos[i], ex));
   }
-  const int base = last < 0 ? 0 : lowest / MK * MK;
-  const int tiles = (last - base + MK) / MK;       // tiles of the keys [base, last]
+  // the tiles of the kept first keys, then those from the lowest first key on
+  const int lo = last < 0 ? 0 : lowest / MK, kept = last < 0 ? 0 : min((ex.keep + MK - 1) / MK, lo), tiles = kept + (last + MK) / MK - lo;
+  auto first_key_of = [&](int t) { return (t < kept ? t : lo + t - kept) * MK; };
   for (int i = tid; i < MQ * (D / 8); i += MTHREADS) {
     const int r = i / (D / 8), c = (i % (D / 8)) * 8, gr = r0 + r;
     const bool live = s_pos[r] >= 0;
@@ -363,8 +450,9 @@ paged_attend_mma_kernel(const bf16* __restrict__ q, long long q_token_stride, co
   auto fetch = [&](int t) {
     bf16* dk_ = sk + (t & 1) * MK * ST;
     bf16* dv_ = sv + (t & 1) * MK * ST;
+    const int k0 = first_key_of(t);
     for (int i = tid; i < MK * (D / 8); i += MTHREADS) {
-      const int r = i / (D / 8), c = (i % (D / 8)) * 8, key = base + t * MK + r;
+      const int r = i / (D / 8), c = (i % (D / 8)) * 8, key = k0 + r;
       const bool live = key <= last;
       const long long off = live ? (pool_token(pool, row, key) * G + g) * D + c : 0;
       cp16(smem_addr(dk_ + r * ST + c), kpool + off, live);
@@ -374,7 +462,7 @@ paged_attend_mma_kernel(const bf16* __restrict__ q, long long q_token_stride, co
   };
   const int lg = lane >> 2, t2 = (lane & 3) * 2;
   const int p0 = s_pos[warp * 16 + lg], p1 = s_pos[warp * 16 + lg + 8];
-  const int f0_ = chunk_start(p0, ex.chunk), f1_ = chunk_start(p1, ex.chunk);        // first keys the rows see
+  const int f0_ = first_seen(p0, ex), f1_ = first_seen(p1, ex);        // first keys the rows see
   float m0 = -INFINITY, m1 = -INFINITY, l0 = 0.f, l1 = 0.f, o[D / 8][4];
 #pragma unroll
   for (int j = 0; j < D / 8; ++j) { o[j][0] = o[j][1] = o[j][2] = o[j][3] = 0.f; }
@@ -407,11 +495,14 @@ paged_attend_mma_kernel(const bf16* __restrict__ q, long long q_token_stride, co
     float x0 = -INFINITY, x1 = -INFINITY;
 #pragma unroll
     for (int j = 0; j < 8; ++j) {
-      const int key = base + t * MK + j * 8 + t2;
-      s[j][0] = key <= p0 && key >= f0_ ? s[j][0] * scale_log2 : -INFINITY;
-      s[j][1] = key + 1 <= p0 && key + 1 >= f0_ ? s[j][1] * scale_log2 : -INFINITY;
-      s[j][2] = key <= p1 && key >= f1_ ? s[j][2] * scale_log2 : -INFINITY;
-      s[j][3] = key + 1 <= p1 && key + 1 >= f1_ ? s[j][3] * scale_log2 : -INFINITY;
+      const int key = first_key_of(t) + j * 8 + t2;
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        float v = s[j][e] * scale_log2;
+        if (ex.cap > 0.f) v = ex.cap * soft_tanh(v / ex.cap);
+        const int at = key + (e & 1), p = e < 2 ? p0 : p1, f = e < 2 ? f0_ : f1_;
+        s[j][e] = at <= p && (at >= f || at < ex.keep) ? v : -INFINITY;
+      }
       x0 = fmaxf(x0, fmaxf(s[j][0], s[j][1]));
       x1 = fmaxf(x1, fmaxf(s[j][2], s[j][3]));
     }
@@ -503,8 +594,9 @@ int attend(const T* q, long long qs, const T* kpool, const T* vpool, const int* 
 
 template <typename T>
 int attend_any(const void* q, long long qs, const void* kpool, const void* vpool, const int* positions, int R, int S, int H, int G, int dk, int dv,
-               int D, float scale, void* out, const Pool& pool, int chunk, const float* sinks, const void* gate, long long gate_stride, cudaStream_t stream) {
-  const Extras<T> ex{chunk, sinks, static_cast<const T*>(gate), gate_stride};
+               int D, float scale, void* out, const Pool& pool, int chunk, int window, int keep, float softcap, const float* sinks, const void* gate,
+               long long gate_stride, cudaStream_t stream) {
+  const Extras<T> ex{chunk, window, keep, softcap, sinks, static_cast<const T*>(gate), gate_stride};
 #define DEWB_ATTEND(NN) attend<T, NN>(static_cast<const T*>(q), qs, static_cast<const T*>(kpool), static_cast<const T*>(vpool), positions, R, S, H, G, \
                                       dk, dv, D, scale, static_cast<T*>(out), pool, ex, stream)
   const int nj = (dv + 31) / 32;
@@ -542,29 +634,31 @@ extern "C" int dewb_qk_norm_append(const void* qkv, const void* qw, const void* 
   return static_cast<int>(cudaGetLastError());
 }
 
-// qkv [R * S, row_stride >= H dk + G dk + G dv] -> packed [R * S, H + 2 G, D] and the pools; per-head norms with the weights qw, kw [dk] (null: none),
-// bias [H dk + G dk + G dv] (null: none).  G 0: a layer without keys and values of its own (the pools are not touched).
-extern "C" int dewb_head_norm_append(const void* qkv, long long row_stride, const void* bias, const void* qw, const void* kw, float eps,
-                                     const int* positions, int R, int S, int H, int G, int dk, int dv, int D, void* packed, void* kpool,
-                                     void* vpool, const int* page_table, int page_size, int max_pages, const int* row_ids, int fp32,
-                                     void* stream_ptr) {
+// qkv [R * S, row_stride >= H dk + G dk + G dv] -> packed [R * S, H + 2 G, D] and the pools; per-head norms with the weights qw, kw [dk] (null: none;
+// `unit`: a norm without a weight), bias [H dk + G dk + G dv] (null: none); `table` [R * S, dims / 2, 2] (null: no rotation) turns the first `dims`
+// columns of the query and key heads.  G 0: a layer without keys and values of its own (the pools are not touched).
+extern "C" int dewb_head_norm_append(const void* qkv, long long row_stride, const void* bias, const void* qw, const void* kw, float eps, int unit,
+                                     const float* table, int dims, int interleaved, const int* positions, int R, int S, int H, int G, int dk, int dv,
+                                     int D, void* packed, void* kpool, void* vpool, const int* page_table, int page_size, int max_pages,
+                                     const int* row_ids, int fp32, void* stream_ptr) {
   if (R <= 0 || S <= 0) return 0;
   if (H < 1 || G < 0 || (G > 0 && H % G) || dk < 1 || dv < 1 || D < dk || D < dv || page_size < 1 || max_pages < 1 ||
-      row_stride < static_cast<long long>(H + G) * dk + static_cast<long long>(G) * dv)
+      row_stride < static_cast<long long>(H + G) * dk + static_cast<long long>(G) * dv || (table != nullptr && (dims < 2 || dims % 2 || dims > dk)))
     return -3;
   cudaStream_t stream = reinterpret_cast<cudaStream_t>(stream_ptr);
   const Pool pool{page_table, page_size, max_pages, row_ids};
+  const Turn turn{reinterpret_cast<const float2*>(table), table == nullptr ? 0 : dims, interleaved};
   const bool vec = dk % 4 == 0 && dv % 4 == 0 && D % 4 == 0 && row_stride % 4 == 0 && aligned(qkv, 16) && aligned(bias, 16) && aligned(qw, 16) &&
                    aligned(kw, 16) && aligned(packed, 16) && aligned(kpool, 16) && aligned(vpool, 16);
   const long long items = static_cast<long long>(R) * S * (H + 2 * G);
   const bool vec8 = vec && !fp32 && dk % 8 == 0 && dv % 8 == 0 && D % 8 == 0 && row_stride % 8 == 0;
   const int v = vec8 ? 8 : vec ? 4 : 1, lg = D <= 8 * v ? 8 : D <= 16 * v ? 16 : 32;
-  const bool one = D <= lg * v;
   const long long blocks = (items * lg + 255) / 256;
   if (items > 0x7fffffffll) return -3;
-#define DEWB_HEADS(TT, VV, LL, OO) head_norm_append_kernel<TT, VV, LL, OO><<<static_cast<unsigned>(blocks), 256, 0, stream>>>(static_cast<const TT*>(qkv),     row_stride, static_cast<const TT*>(bias), static_cast<const TT*>(qw), static_cast<const TT*>(kw), eps, positions, items, S, H, G, dk, dv, D,     static_cast<TT*>(packed), static_cast<TT*>(kpool), static_cast<TT*>(vpool), pool)
-#define DEWB_HEADS_L(TT, VV) do { if (lg == 8) DEWB_HEADS(TT, VV, 8, true); else if (lg == 16) DEWB_HEADS(TT, VV, 16, true); \
-    else if (one) DEWB_HEADS(TT, VV, 32, true); else DEWB_HEADS(TT, VV, 32, false); } while (0)
+#define DEWB_HEADS(TT, VV, LL) head_norm_append_kernel<TT, VV, LL><<<static_cast<unsigned>(blocks), 256, 0, stream>>>(static_cast<const TT*>(qkv), \
+    row_stride, static_cast<const TT*>(bias), static_cast<const TT*>(qw), static_cast<const TT*>(kw), eps, unit, turn, positions, items, S, H, G, dk, dv, D, \
+    static_cast<TT*>(packed), static_cast<TT*>(kpool), static_cast<TT*>(vpool), pool)
+#define DEWB_HEADS_L(TT, VV) do { if (lg == 8) DEWB_HEADS(TT, VV, 8); else if (lg == 16) DEWB_HEADS(TT, VV, 16); else DEWB_HEADS(TT, VV, 32); } while (0)
   if (fp32) { if (vec) DEWB_HEADS_L(float, 4); else DEWB_HEADS_L(float, 1); }
   else { if (vec8) DEWB_HEADS_L(bf16, 8); else if (vec) DEWB_HEADS_L(bf16, 4); else DEWB_HEADS_L(bf16, 1); }
 #undef DEWB_HEADS_L
@@ -590,32 +684,46 @@ extern "C" int dewb_head_gate(const void* o, const void* gate, long long gate_st
   return static_cast<int>(cudaGetLastError());
 }
 
-// `chunk` 0, `sinks` null, `gate` null: off (see Extras).
+// positions [n] (below 0: taken as 0), frequency [half] -> out [n, half, 2]
+extern "C" int dewb_rotary_angles(const int* positions, const double* frequency, float* out, long long n, int half, void* stream_ptr) {
+  if (n <= 0) return 0;
+  const long long blocks = (n * half + 255) / 256;
+  if (half < 1 || blocks > 0x7fffffffll) return -3;
+  rotary_angles_kernel<<<static_cast<unsigned>(blocks), 256, 0, reinterpret_cast<cudaStream_t>(stream_ptr)>>>(positions, frequency, reinterpret_cast<float2*>(out),
+                                                                                                              n, half);
+  return static_cast<int>(cudaGetLastError());
+}
+
+static bool range_ok(int chunk, int window, int keep, float softcap) {
+  return chunk >= 0 && window >= 0 && keep >= 0 && (keep == 0 || chunk == 0) && softcap >= 0.f;
+}
+
+// `chunk` 0, `window` 0 (and `keep` with it), `softcap` 0, `sinks` null, `gate` null: off (see Extras).
 extern "C" int dewb_paged_attend(const void* q, long long q_token_stride, const void* kpool, const void* vpool, const int* positions, int R, int S,
-                                 int H, int G, int dk, int dv, int D, float scale, int chunk, const float* sinks, const void* gate,
+                                 int H, int G, int dk, int dv, int D, float scale, int chunk, int window, int keep, float softcap, const float* sinks, const void* gate,
                                  long long gate_stride, void* out, const int* page_table, int page_size, int max_pages, const int* row_ids, int fp32,
                                  void* stream_ptr) {
   if (R <= 0 || S <= 0) return 0;
-  if (H < 1 || G < 1 || H % G || dk < 1 || dv < 1 || D < dk || D < dv || page_size < 1 || max_pages < 1 || chunk < 0) return -3;
+  if (H < 1 || G < 1 || H % G || dk < 1 || dv < 1 || D < dk || D < dv || page_size < 1 || max_pages < 1 || !range_ok(chunk, window, keep, softcap)) return -3;
   cudaStream_t stream = reinterpret_cast<cudaStream_t>(stream_ptr);
   const Pool pool{page_table, page_size, max_pages, row_ids};
-  if (fp32) return attend_any<float>(q, q_token_stride, kpool, vpool, positions, R, S, H, G, dk, dv, D, scale, out, pool, chunk, sinks, gate, gate_stride, stream);
-  return attend_any<bf16>(q, q_token_stride, kpool, vpool, positions, R, S, H, G, dk, dv, D, scale, out, pool, chunk, sinks, gate, gate_stride, stream);
+  if (fp32) return attend_any<float>(q, q_token_stride, kpool, vpool, positions, R, S, H, G, dk, dv, D, scale, out, pool, chunk, window, keep, softcap, sinks, gate, gate_stride, stream);
+  return attend_any<bf16>(q, q_token_stride, kpool, vpool, positions, R, S, H, G, dk, dv, D, scale, out, pool, chunk, window, keep, softcap, sinks, gate, gate_stride, stream);
 }
 
 // The tensor-core form (bf16; pools D = 64, 128 or 256 wide; q on 16-byte boundaries with a token stride of a multiple of 8).
 extern "C" int dewb_paged_attend_mma(const void* q, long long q_token_stride, const void* kpool, const void* vpool, const int* positions, int R, int S,
-                                     int H, int G, int dv, int D, float scale, int chunk, const float* sinks, const void* gate, long long gate_stride,
+                                     int H, int G, int dv, int D, float scale, int chunk, int window, int keep, float softcap, const float* sinks, const void* gate, long long gate_stride,
                                      void* out, const int* page_table, int page_size, int max_pages, const int* row_ids, void* stream_ptr) {
   if (R <= 0 || S <= 0) return 0;
-  if (H < 1 || G < 1 || H % G || dv < 1 || D < dv || page_size < 1 || max_pages < 1 || chunk < 0 || q_token_stride % 8 || !aligned(q, 16) || !aligned(kpool, 16) ||
+  if (H < 1 || G < 1 || H % G || dv < 1 || D < dv || page_size < 1 || max_pages < 1 || !range_ok(chunk, window, keep, softcap) || q_token_stride % 8 || !aligned(q, 16) || !aligned(kpool, 16) ||
       !aligned(vpool, 16))
     return -3;
   cudaStream_t stream = reinterpret_cast<cudaStream_t>(stream_ptr);
   const Pool pool{page_table, page_size, max_pages, row_ids};
   const bf16 *qp = static_cast<const bf16*>(q), *kp = static_cast<const bf16*>(kpool), *vp = static_cast<const bf16*>(vpool);
   bf16* op = static_cast<bf16*>(out);
-  const Extras<bf16> ex{chunk, sinks, static_cast<const bf16*>(gate), gate_stride};
+  const Extras<bf16> ex{chunk, window, keep, softcap * 1.4426950408889634f, sinks, static_cast<const bf16*>(gate), gate_stride};
   if (D == 64) return attend_mma<64>(qp, q_token_stride, kp, vp, positions, R, S, H, G, dv, scale, op, pool, ex, stream);
   if (D == 128) return attend_mma<128>(qp, q_token_stride, kp, vp, positions, R, S, H, G, dv, scale, op, pool, ex, stream);
   if (D == 256) return attend_mma<256>(qp, q_token_stride, kp, vp, positions, R, S, H, G, dv, scale, op, pool, ex, stream);

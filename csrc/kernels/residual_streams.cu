@@ -1,14 +1,16 @@
 // Row kernels of decoders whose residual is a bundle of fp32 streams, for sm_100a.  All are bandwidth bound: one pass over the operands,
 // 16-byte accesses, fp32 arithmetic.
 //
-//   embed_streams   H[t, s, :] = embed[token t] (+ pos[position t]) for every stream s
+//   embed_streams   H[t, s, :] = gain * embed[token t] (+ pos[position t]) for every stream s
 //   stream_step     one residual step between two sub-layers: the pending write of the sub-layer that just ran
-//                       H'[t] = sum_s mix[s, t] H[s] + out[t] * (scale . y)
-//                   (in place), the read of the next one, u = sum_s read[s] H'[s], and its norm (layer norm without a bias, or RMS norm);
-//                   y may pass an RMS norm of its own first (a block that normalises what its sub-layers return).  Without connection
+//                       H'[t] = sum_s mix[s, t] H[s] + out[t] * gain * (scale . y + scale2 . y2)
+//                   (in place), the read of the next one, u = sum_s read[s] H'[s], and its norm (layer norm without a bias, or RMS norm,
+//                   whose weights may be stored as their distance from `around`); y may pass an RMS norm of its own first (a block that
+//                   normalises what its sub-layers return); y2 is there when two sub-layers read the same norm and join together.  Without connection
 //                   weights the streams keep themselves and take y as it is: one such stream is the ordinary fp32 residual, which has a
 //                   form of its own (residual_step).
 //   clamped_glu     g sigmoid(alpha g) (u + 1) with g = min(gate, limit), u = clamp(up, -limit, limit)
+//   gelu_glu        gelu(gate) up, the tanh form of gelu
 //   sigmoid_gated_norm   RMS norm over a whole row times a weight times sigmoid(gate)
 //   softcap         cap tanh(x / cap), fp32 out (logits)
 //
@@ -29,13 +31,15 @@ constexpr int THREADS = 256;
 template <typename T, int V>
 __global__ void __launch_bounds__(THREADS)
 embed_streams_kernel(const long long* __restrict__ tokens, const int* __restrict__ positions, const T* __restrict__ embed,
-                     const T* __restrict__ pos, float* __restrict__ H, int n, int d, int vocab, int max_pos) {
+                     const T* __restrict__ pos, float* __restrict__ H, int n, int d, int vocab, int max_pos, float gain) {
   const long long t = blockIdx.x;
   const long long tok = min(max(tokens[t], 0ll), static_cast<long long>(vocab - 1));
   const int p = min(max(positions == nullptr ? 0 : positions[t], 0), max_pos - 1);
   for (int i = threadIdx.x * V; i < d; i += THREADS * V) {
     float a[V];
     load_v<V>(embed + tok * d + i, a);
+#pragma unroll
+    for (int j = 0; j < V; ++j) a[j] *= gain;
     if (pos != nullptr) {
       float b[V];
       load_v<V>(pos + static_cast<long long>(p) * d + i, b);
@@ -51,7 +55,8 @@ template <typename T, int V, int NS>
 __global__ void __launch_bounds__(THREADS)
 stream_step_kernel(float* __restrict__ H, const T* __restrict__ y, const T* __restrict__ y_weight, const T* __restrict__ scale,
                    const float* __restrict__ mix, const float* __restrict__ out, const float* __restrict__ read, const T* __restrict__ w,
-                   T* __restrict__ normed, int n_rt, int d, float y_eps, float eps, int rms) {
+                   T* __restrict__ normed, int n_rt, int d, float y_eps, float eps, int rms, const T* __restrict__ y2, const T* __restrict__ scale2,
+                   float gain, float around) {
   constexpr int NM = NS ? NS : MAX_STREAMS;
   const int n = NS ? NS : n_rt;
   extern __shared__ float su[];                      // y, then u of this token
@@ -101,6 +106,15 @@ stream_step_kernel(float* __restrict__ H, const T* __restrict__ y, const T* __re
 #pragma unroll
         for (int j = 0; j < V; ++j) b[j] *= c[j];
       }
+      if (y2 != nullptr) {
+        float b2[V], c[V];
+        load_v<V>(y2 + t * d + i, b2);
+        if (scale2 != nullptr) load_v<V>(scale2 + i, c);
+#pragma unroll
+        for (int j = 0; j < V; ++j) b[j] += scale2 != nullptr ? c[j] * b2[j] : b2[j];
+      }
+#pragma unroll
+      for (int j = 0; j < V; ++j) b[j] *= gain;
 #pragma unroll(NS ? NS : 1)
       for (int q = 0; q < NM; ++q) {
         if (NS || q < n) {
@@ -148,20 +162,21 @@ stream_step_kernel(float* __restrict__ H, const T* __restrict__ y, const T* __re
     float c[V], o[V];
     load_v<V>(w + i, c);
 #pragma unroll
-    for (int j = 0; j < V; ++j) o[j] = (su[i + j] - mean) * r * c[j];
+    for (int j = 0; j < V; ++j) o[j] = (su[i + j] - mean) * r * (around + c[j]);
     store_v<V>(normed + t * d + i, o);
   }
 }
 
-// One plain stream (H += y, y through its RMS norm where it has a weight, then the norm of H): the whole row in registers, NI pieces of V values a
-// thread, every load in flight before the first sum.
-template <typename T, int V, int NI>
+// One plain stream (H += gain (scale . y + scale2 . y2), y through its RMS norm where it has a weight, then the norm of H): the whole row in registers,
+// NI pieces of V values a thread, every load in flight before the first sum.  TWO: y2 is there.
+template <typename T, int V, int NI, bool TWO>
 __global__ void __launch_bounds__(THREADS)
 residual_step_kernel(float* __restrict__ H, const T* __restrict__ y, const T* __restrict__ y_weight, const T* __restrict__ w, T* __restrict__ normed,
-                     int d, float y_eps, float eps) {
+                     int d, float y_eps, float eps, const T* __restrict__ scale, const T* __restrict__ y2, const T* __restrict__ scale2, float gain,
+                     float around) {
   __shared__ float red[32];
   const long long at = static_cast<long long>(blockIdx.x) * d;
-  float x[NI][V], b[NI][V];
+  float x[NI][V], b[NI][V], b2[TWO ? NI : 1][V];
 #pragma unroll
   for (int p = 0; p < NI; ++p) {
     const int i = (p * THREADS + threadIdx.x) * V;
@@ -169,6 +184,7 @@ residual_step_kernel(float* __restrict__ H, const T* __restrict__ y, const T* __
     for (int j = 0; j < V; ++j) x[p][j] = b[p][j] = 0.f;
     if (i < d) {
       load_v<V>(y + at + i, b[p]);
+      if (TWO) load_v<V>(y2 + at + i, b2[p]);
       load_v<V>(H + at + i, x[p]);
     }
   }
@@ -190,6 +206,27 @@ residual_step_kernel(float* __restrict__ H, const T* __restrict__ y, const T* __
       }
     }
   }
+  if (scale != nullptr || TWO || gain != 1.f) {
+#pragma unroll
+    for (int p = 0; p < NI; ++p) {
+      const int i = (p * THREADS + threadIdx.x) * V;
+      if (i < d) {
+        float c[V];
+        if (scale != nullptr) {
+          load_v<V>(scale + i, c);
+#pragma unroll
+          for (int j = 0; j < V; ++j) b[p][j] *= c[j];
+        }
+        if (TWO) {
+          if (scale2 != nullptr) load_v<V>(scale2 + i, c);
+#pragma unroll
+          for (int j = 0; j < V; ++j) b[p][j] += scale2 != nullptr ? c[j] * b2[p][j] : b2[p][j];
+        }
+#pragma unroll
+        for (int j = 0; j < V; ++j) b[p][j] *= gain;
+      }
+    }
+  }
   float ss = 0.f;
 #pragma unroll
   for (int p = 0; p < NI; ++p) {
@@ -207,7 +244,7 @@ residual_step_kernel(float* __restrict__ H, const T* __restrict__ y, const T* __
       float c[V];
       load_v<V>(w + i, c);
 #pragma unroll
-      for (int j = 0; j < V; ++j) c[j] *= x[p][j] * r;
+      for (int j = 0; j < V; ++j) c[j] = (around + c[j]) * x[p][j] * r;
       store_v<V>(normed + at + i, c);
     }
   }
@@ -236,6 +273,21 @@ clamped_glu_kernel(const T* __restrict__ gu, T* __restrict__ out, int F, float l
     o[j] = times_sigmoid<T>(a, alpha * a) * (b + 1.f);
   }
   store_v<V>(out + r * F + i, o);
+}
+
+// gelu(z) = z sigmoid(2 sqrt(2 / pi) (z + 0.044715 z^3)); grid as above
+template <typename T, int V>
+__global__ void __launch_bounds__(THREADS)
+gelu_glu_kernel(const T* __restrict__ gu, T* __restrict__ out, int F) {
+  const long long r = blockIdx.x;
+  const int i = (blockIdx.y * THREADS + threadIdx.x) * V;
+  if (i >= F) return;
+  float g[V], u[V];
+  load_v<V>(gu + r * 2 * F + i, g);
+  load_v<V>(gu + r * 2 * F + F + i, u);
+#pragma unroll
+  for (int j = 0; j < V; ++j) u[j] *= times_sigmoid<T>(g[j], 1.5957691216057308f * (g[j] + 0.044715f * g[j] * g[j] * g[j]));
+  store_v<V>(out + r * F + i, u);
 }
 
 template <typename T, int V>
@@ -286,19 +338,22 @@ int allow_smem(K kernel, size_t bytes) {
 
 template <typename T>
 int step(float* H, const T* y, const T* y_weight, const T* scale, const float* mix, const float* out, const float* read, const T* w, T* normed,
-         long long rows, int n, int d, float y_eps, float eps, int rms, cudaStream_t stream) {
-  const bool vec = d % 4 == 0 && aligned(H, 16) && aligned(y, 4 * sizeof(T)) && aligned(y_weight, 4 * sizeof(T)) && aligned(scale, 4 * sizeof(T)) && aligned(w, 4 * sizeof(T)) &&
+         long long rows, int n, int d, float y_eps, float eps, int rms, const T* y2, const T* scale2, float gain, float around, cudaStream_t stream) {
+  const bool vec = aligned(y2, 4 * sizeof(T)) && aligned(scale2, 4 * sizeof(T)) && d % 4 == 0 && aligned(H, 16) && aligned(y, 4 * sizeof(T)) && aligned(y_weight, 4 * sizeof(T)) && aligned(scale, 4 * sizeof(T)) && aligned(w, 4 * sizeof(T)) &&
                    aligned(normed, 4 * sizeof(T));
-  if (vec && n == 1 && rms && y != nullptr && scale == nullptr && mix == nullptr && out == nullptr && read == nullptr && d <= 32 * THREADS) {
+  if (vec && n == 1 && rms && y != nullptr && mix == nullptr && out == nullptr && read == nullptr && d <= 32 * THREADS) {
     const int pieces = (d + THREADS * 4 - 1) / (THREADS * 4);
-#define DEWB_RES(NN) residual_step_kernel<T, 4, NN><<<static_cast<unsigned>(rows), THREADS, 0, stream>>>(H, y, y_weight, w, normed, d, y_eps, eps)
+#define DEWB_RES_T(NN, TT) residual_step_kernel<T, 4, NN, TT><<<static_cast<unsigned>(rows), THREADS, 0, stream>>>(H, y, y_weight, w, normed, d, y_eps, eps, \
+    scale, y2, scale2, gain, around)
+#define DEWB_RES(NN) do { if (y2 != nullptr) DEWB_RES_T(NN, true); else DEWB_RES_T(NN, false); } while (0)
     if (pieces <= 1) DEWB_RES(1); else if (pieces <= 2) DEWB_RES(2); else if (pieces <= 4) DEWB_RES(4); else DEWB_RES(8);
 #undef DEWB_RES
+#undef DEWB_RES_T
     return static_cast<int>(cudaGetLastError());
   }
   const size_t smem = static_cast<size_t>(d) * 4;
 #define DEWB_STEP(VV, NN) do { const int r = allow_smem(stream_step_kernel<T, VV, NN>, smem); if (r) return r; \
-    stream_step_kernel<T, VV, NN><<<static_cast<unsigned>(rows), THREADS, smem, stream>>>(H, y, y_weight, scale, mix, out, read, w, normed, n, d, y_eps, eps, rms); } while (0)
+    stream_step_kernel<T, VV, NN><<<static_cast<unsigned>(rows), THREADS, smem, stream>>>(H, y, y_weight, scale, mix, out, read, w, normed, n, d, y_eps, eps, rms, y2, scale2, gain, around); } while (0)
   if (vec) {
     if (n == 1) DEWB_STEP(4, 1); else if (n == 2) DEWB_STEP(4, 2); else if (n == 3) DEWB_STEP(4, 3); else if (n == 4) DEWB_STEP(4, 4); else DEWB_STEP(1, 0);
   } else {
@@ -315,14 +370,14 @@ using namespace dewb::streams;
 
 // `fp32`: activations and weights are fp32, else bf16.  `positions` / `pos` may be null.
 extern "C" int dewb_embed_streams(const long long* tokens, const int* positions, const void* embed, const void* pos, float* H, long long rows,
-                                  int n, int d, int vocab, int max_pos, int fp32, void* stream_ptr) {
+                                  int n, int d, int vocab, int max_pos, float gain, int fp32, void* stream_ptr) {
   if (rows <= 0) return 0;
   if (n < 1 || d < 1 || vocab < 1 || (pos != nullptr && (max_pos < 1 || positions == nullptr))) return -3;
   cudaStream_t stream = reinterpret_cast<cudaStream_t>(stream_ptr);
   const bool vec = d % 4 == 0 && aligned(H, 16) && aligned(embed, 16) && aligned(pos, 16);
   const unsigned grid = static_cast<unsigned>(rows);
 #define DEWB_EMBED(TT, VV) embed_streams_kernel<TT, VV><<<grid, THREADS, 0, stream>>>(tokens, positions, static_cast<const TT*>(embed), \
-    static_cast<const TT*>(pos), H, n, d, vocab, max_pos > 0 ? max_pos : 1)
+    static_cast<const TT*>(pos), H, n, d, vocab, max_pos > 0 ? max_pos : 1, gain)
   if (fp32) { if (vec) DEWB_EMBED(float, 4); else DEWB_EMBED(float, 1); }
   else { if (vec) DEWB_EMBED(bf16, 4); else DEWB_EMBED(bf16, 1); }
 #undef DEWB_EMBED
@@ -331,16 +386,19 @@ extern "C" int dewb_embed_streams(const long long* tokens, const int* positions,
 
 // H [rows, n, d] fp32, updated in place when `y` [rows, d] is given; normed [rows, d] (null: write only).  mix is indexed [from, to].  `mix`, `out`
 // and `read` may be null (each stream keeps itself, takes y, and is read with weight 1); y_weight [d]: y passes an RMS norm with that weight first.
+// `scale`, `scale2` [d], y2 [rows, d]: see stream_step above (null: absent); weights of the norm are `around` + w.
 extern "C" int dewb_stream_step(float* H, const void* y, const void* y_weight, const void* scale, const float* mix, const float* out,
                                 const float* read, const void* w, void* normed, long long rows, int n, int d, float y_eps, float eps, int rms,
-                                int fp32, void* stream_ptr) {
+                                const void* y2, const void* scale2, float gain, float around, int fp32, void* stream_ptr) {
   if (rows <= 0) return 0;
-  if (n < 1 || n > MAX_STREAMS || d < 1 || (y == nullptr && y_weight != nullptr) || (normed != nullptr && w == nullptr)) return -3;
+  if (n < 1 || n > MAX_STREAMS || d < 1 || (y == nullptr && (y_weight != nullptr || y2 != nullptr)) || (y_weight != nullptr && y2 != nullptr) || (normed != nullptr && w == nullptr)) return -3;
   cudaStream_t stream = reinterpret_cast<cudaStream_t>(stream_ptr);
   if (fp32) return step<float>(H, static_cast<const float*>(y), static_cast<const float*>(y_weight), static_cast<const float*>(scale), mix, out, read,
-                               static_cast<const float*>(w), static_cast<float*>(normed), rows, n, d, y_eps, eps, rms, stream);
+                               static_cast<const float*>(w), static_cast<float*>(normed), rows, n, d, y_eps, eps, rms, static_cast<const float*>(y2),
+                               static_cast<const float*>(scale2), gain, around, stream);
   return step<bf16>(H, static_cast<const bf16*>(y), static_cast<const bf16*>(y_weight), static_cast<const bf16*>(scale), mix, out, read,
-                    static_cast<const bf16*>(w), static_cast<bf16*>(normed), rows, n, d, y_eps, eps, rms, stream);
+                    static_cast<const bf16*>(w), static_cast<bf16*>(normed), rows, n, d, y_eps, eps, rms, static_cast<const bf16*>(y2),
+                    static_cast<const bf16*>(scale2), gain, around, stream);
 }
 
 // x [rows, n] -> out [rows, n] fp32
@@ -372,6 +430,23 @@ extern "C" int dewb_clamped_glu(const void* gu, void* out, long long rows, int F
   if (fp32) { if (v == 4) DEWB_GLU(float, 4); else DEWB_GLU(float, 1); }
   else { if (v == 8) DEWB_GLU(bf16, 8); else if (v == 4) DEWB_GLU(bf16, 4); else DEWB_GLU(bf16, 1); }
 #undef DEWB_GLU
+  return static_cast<int>(cudaGetLastError());
+}
+
+// gu [rows, 2 F] (gate half, then linear half) -> out [rows, F]
+extern "C" int dewb_gelu_glu(const void* gu, void* out, long long rows, int F, int fp32, void* stream_ptr) {
+  if (rows <= 0) return 0;
+  if (F < 1) return -3;
+  cudaStream_t stream = reinterpret_cast<cudaStream_t>(stream_ptr);
+  const bool a16 = aligned(gu, 16) && aligned(out, 16);
+  const int v = F % 8 == 0 && !fp32 && a16 ? 8 : F % 4 == 0 && a16 ? 4 : 1;
+  const int blocks = (F + THREADS * v - 1) / (THREADS * v);
+  if (blocks > 65535) return -3;
+  const dim3 grid(static_cast<unsigned>(rows), blocks);
+#define DEWB_GELU(TT, VV) gelu_glu_kernel<TT, VV><<<grid, THREADS, 0, stream>>>(static_cast<const TT*>(gu), static_cast<TT*>(out), F)
+  if (fp32) { if (v == 4) DEWB_GELU(float, 4); else DEWB_GELU(float, 1); }
+  else { if (v == 8) DEWB_GELU(bf16, 8); else if (v == 4) DEWB_GELU(bf16, 4); else DEWB_GELU(bf16, 1); }
+#undef DEWB_GELU
   return static_cast<int>(cudaGetLastError());
 }
 

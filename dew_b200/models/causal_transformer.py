@@ -25,6 +25,7 @@ from ..nn.attention import SelfAttention
 from ..nn.kv_cache import CacheSlot, Uncached
 from ..nn.layers import Embedding, LayerNorm, Linear, RMSNorm, declare
 from ..nn.mlp import ClampedGLU, SwiGLU
+from ..ops.rotary import Rotary
 from ..utils.registry import register
 
 
@@ -34,10 +35,11 @@ class Mixture:
     experts: int = 8
     top_k: int = 2
     layers: Optional[Sequence[int]] = None          # which layers are sparse (None = all)
-    score_function: str = "softmax"                  # softmax | sigmoid
+    score_function: str = "softmax"                  # softmax | sigmoid | top_softmax (the choice by the logits, the weights their softmax over the chosen)
     norm_topk_prob: bool = True
     scaling: float = 1.0
     bias: bool = False                               # aux-loss-free balancing bias (selection only)
+    router_bias: bool = False                        # a bias on the router's logits
     expert_features: Optional[int] = None
     shared_features: int = 0                         # total hidden width of the shared experts
     shared_gate: bool = False
@@ -131,8 +133,12 @@ class TransformerConfig:
     attn_chunk: Optional[int] = None                  # a query sees no key from before the start of its chunk of this many positions
     attn_head_gate: bool = False                      # each head's output times the sigmoid of one number from the layer's input
     kv_from: Optional[int] = None                     # (per layer) read that earlier layer's keys and values instead of projecting its own
-    layer_options: Optional[Sequence[Optional[Mapping]]] = None    # per layer, what differs from the fields above: num_heads, num_kv_heads, head_dim, value_dim,
-                                                      # query_scale, query_temperature, attn_chunk, kv_from, decay (lightning), mlp_features, mlp_limit, mixture
+    rotation: Optional[Rotary] = None                 # attention layers turn by this (their own angles, any positions) instead of the model's tables
+    keep_first: int = 0                               # with a window: keys from the row's start that stay visible
+    qk_unit_norm: bool = False                        # q and k over their root mean square per head, after the rotation and without a weight
+    parallel_block: bool = False                      # a layer's mixer and MLP read one norm and join the residual together
+    norm_around: float = 0.0                          # the weights of the residual's norms are stored as their distance from this
+    layer_options: Optional[Sequence[Optional[Mapping]]] = None    # per layer, what differs from the fields above: LAYER_OPTIONS, and decay (lightning)
 
     def __post_init__(self):
         if self.norm not in ("rms", "layer"):
@@ -142,19 +148,24 @@ class TransformerConfig:
         if self.fp32_residual and self.hyper_connections:
             raise ValueError("fp32_residual is the residual without connections: static hyper-connections already keep their streams in fp32")
         if self.fp32_stack:
-            if self.altup > 1 or not self.pre_norm or self.residual_multiplier != 1.0 or self.remat or self.depth_residual_block or self.engram or self.mtp_depth \
-                    or self.logit_divisor != 1.0:
-                raise NotImplementedError("fp32 residual streams are built for pre-norm layers, without rematerialisation, AltUp, residual and logit factors, "
-                                          "block attention residuals, n-gram memories and multi-token prediction")
-        elif self.norm != "rms" or self.layer_scale or self.learned_positions:
-            raise NotImplementedError("layer norms, layer scale and learned positions belong to the static-stream stack (hyper_connections >= 1 with "
-                                      "hyper_dynamic=False, or fp32_residual)")
+            if self.altup > 1 or not self.pre_norm or self.remat or self.depth_residual_block or self.engram or self.mtp_depth or self.logit_divisor != 1.0:
+                raise NotImplementedError("fp32 residual streams are built for pre-norm layers, without rematerialisation, AltUp, logit factors, block "
+                                          "attention residuals, n-gram memories and multi-token prediction")
+            if self.parallel_block and (self.hyper_connections or self.sandwich_norm):
+                raise NotImplementedError("layers whose sub-layers join together are built for one plain residual without norms on what joins")
+            if self.norm_around and self.norm != "rms":
+                raise NotImplementedError("norm weights stored around another value than 0 are built for RMS norms")
+        elif self.norm != "rms" or self.layer_scale or self.learned_positions or self.parallel_block or self.norm_around:
+            raise NotImplementedError("layer norms, layer scale, learned positions, parallel blocks and norm weights stored around a value belong to the "
+                                      "static-stream stack (hyper_connections >= 1 with hyper_dynamic=False, or fp32_residual)")
         if self.kv_from is not None and self.layer_options is not None:
             raise ValueError("kv_from belongs to a layer: give it in layer_options")
         if isinstance(self.mixture, Mapping):             # a run record (JSON) carries the mixture as a plain mapping
             self.mixture = Mixture(**self.mixture)
         if isinstance(self.loop, Mapping):
             self.loop = Loop(**self.loop)
+        if isinstance(self.rotation, Mapping):
+            self.rotation = Rotary(**self.rotation)
 
     @property
     def static_streams(self) -> bool:
@@ -170,12 +181,11 @@ class TransformerConfig:
         o = self.layer_options[index] if self.layer_options is not None else None
         if not o:
             return self
-        own = {"num_heads", "num_kv_heads", "head_dim", "value_dim", "query_scale", "query_temperature", "attn_chunk", "kv_from", "mlp_features", "mlp_limit",
-               "mixture"}
-        if set(o) - own - {"decay"}:
-            raise ValueError(f"unknown layer option(s) {sorted(set(o) - own - {'decay'})}; known: {sorted(own | {'decay'})}")
+        if set(o) - LAYER_OPTIONS - {"decay"}:
+            raise ValueError(f"unknown layer option(s) {sorted(set(o) - LAYER_OPTIONS - {'decay'})}; known: {sorted(LAYER_OPTIONS | {'decay'})}")
         mixer = {k: o[k] for k in ("num_heads", "head_dim", "value_dim", "decay") if k in o} if self.kinds()[index] == "lightning" else {}
-        return replace(self, layer_options=None, mixer_options={**self.mixer_options, **mixer}, **{k: v for k, v in o.items() if k in own})
+        return replace(self, layer_options=None, mixer_options={**self.mixer_options, **mixer, **o.get("mixer_options", {})},
+                       **{k: v for k, v in o.items() if k in LAYER_OPTIONS and k != "mixer_options"})
 
     def kinds(self) -> List[str]:
         if self.layer_types is None:
@@ -184,18 +194,22 @@ class TransformerConfig:
         return [pattern[i % len(pattern)] for i in range(self.num_layers)]
 
 
+LAYER_OPTIONS = frozenset({"num_heads", "num_kv_heads", "head_dim", "value_dim", "query_scale", "query_temperature", "attn_chunk", "kv_from", "window", "keep_first",
+                           "attn_softcap", "rotation", "attention_sinks", "qkv_bias", "qk_unit_norm", "mlp_features", "mlp_limit", "mlp_activation", "mixture",
+                           "mixer_options"})
 ROTARY_KINDS = ("attention", "local", "nope", "mla", "differential", "forgetting")      # mixers called with the rotary tables and positions
 
 
 def _mixer(cfg: TransformerConfig, kind: str, dtype, device, index: int = 0) -> nn.Module:
     if kind in ("attention", "local", "nope"):
         a = SelfAttention(cfg.emb_features, cfg.num_heads, cfg.num_kv_heads, cfg.head_dim, qk_norm=cfg.qk_norm,
-                          causal=cfg.causal, window=cfg.window if kind == "local" or cfg.layer_types is None else None, bias=cfg.attn_bias,
+                          causal=cfg.causal, window=cfg.window if kind == "local" or cfg.layer_types is None or cfg.rotation is not None else None, bias=cfg.attn_bias,
                           softcap=cfg.attn_softcap, sinks=cfg.attention_sinks, norm_eps=cfg.norm_eps,
                           init_std=cfg.init_std, qkv_bias=cfg.qkv_bias, scale=cfg.query_scale, qk_norm_full=cfg.qk_norm_full,
                           out_gate=cfg.attn_out_gate, value_dim=cfg.value_dim, temperature=cfg.query_temperature,
-                          chunk=cfg.attn_chunk, head_gate=cfg.attn_head_gate, own_kv=cfg.kv_from is None, dtype=dtype, device=device)
-        a.rotary = kind != "nope"                        # SmolLM3's every fourth layer attends without positions
+                          chunk=cfg.attn_chunk, head_gate=cfg.attn_head_gate, own_kv=cfg.kv_from is None, rotation=cfg.rotation if kind != "nope" else None, keep_first=cfg.keep_first, unit_qk=cfg.qk_unit_norm,
+                          dtype=dtype, device=device)
+        a.rotary = kind != "nope" and cfg.rotation is None      # SmolLM3's every fourth layer attends without positions
         if kind == "local" and cfg.local_rope_theta is not None:
             a.own_rope = (float(cfg.local_rope_theta), None)
         return a
@@ -245,7 +259,7 @@ def _mixer(cfg: TransformerConfig, kind: str, dtype, device, index: int = 0) -> 
 def _norm_of(cfg: TransformerConfig, dtype, device) -> nn.Module:
     if cfg.norm == "layer":
         return LayerNorm(cfg.emb_features, cfg.norm_eps, bias=False, dtype=dtype, device=device)
-    return RMSNorm(cfg.emb_features, cfg.norm_eps, dtype=dtype, device=device)
+    return RMSNorm(cfg.emb_features, cfg.norm_eps, dtype=dtype, device=device, around=cfg.norm_around)
 
 
 class _NoNorm(nn.Module):
@@ -273,7 +287,8 @@ class DecoderLayer(nn.Module):
             raise NotImplementedError("layers of one sub-layer are built for the plain pre-norm block")
         self.input_norm = _norm_of(cfg, dtype, device) if cfg.pre_norm else _NoNorm()
         self.mixer = None if kind == "none" else _mixer(cfg, kind, dtype, device, index)
-        one = kind == "none" or not self.has_mlp                  # one sub-layer: the input norm is its only norm
+        self.parallel = cfg.parallel_block
+        one = kind == "none" or not self.has_mlp or self.parallel      # one sub-layer, or two behind one norm: the input norm is the only norm
         self.post_norm = None if one else (_norm_of(cfg, dtype, device) if cfg.pre_norm else _NoNorm())
         mix = cfg.mixture
         sparse = self.has_mlp and mix is not None and (mix.layers is None or index in mix.layers)
@@ -331,14 +346,19 @@ class DecoderLayer(nn.Module):
         """The layer over a ``StreamStack``: each sub-layer's write is fused with the next one's read and norm."""
         scale = self.layer_scale if self.layer_scale is not None else [None, None]
         streams = self.streams if self.streams is not None else [None, None]
-        q = 0
+        q, gain = 0, self.residual_multiplier
+        if self.parallel and self.mixer is not None and self.mlp is not None:
+            n = stack.enter(None, self.input_norm)
+            stack.leave(None, self._mix(n, cos, sin, positions, segment_ids, cache, slot), scale[0], gain=gain, beside=self._feed_forward(n, positions, True),
+                        beside_scale=scale[1])
+            return
         if self.mixer is not None:
             n = stack.enter(streams[q], self.input_norm)
-            stack.leave(streams[q], self._mix(n, cos, sin, positions, segment_ids, cache, slot), scale[q], self.mixer_out_norm)
+            stack.leave(streams[q], self._mix(n, cos, sin, positions, segment_ids, cache, slot), scale[q], self.mixer_out_norm, gain)
             q += 1
         if self.mlp is not None:
             n = stack.enter(streams[q], self.input_norm if q == 0 else self.post_norm)
-            stack.leave(streams[q], self._feed_forward(n, positions, True), scale[q], self.mlp_out_norm)
+            stack.leave(streams[q], self._feed_forward(n, positions, True), scale[q], self.mlp_out_norm, gain)
 
     def _feed_forward(self, n, positions, serving: bool):
         from ..nn.moe import SparseMLP
@@ -517,14 +537,17 @@ class CausalTransformer(nn.Module):
         shape of keys and values serves them all."""
         cfg, kinds = self.config, self.config.kinds()
         if not (cfg.fp32_stack or cfg.layer_options is not None or cfg.query_temperature is not None or cfg.value_dim is not None or cfg.attn_chunk is not None
-                or cfg.attn_head_gate):
+                or cfg.attn_head_gate or cfg.rotation is not None or cfg.keep_first or cfg.qk_unit_norm):
             return None
-        if any(k not in ("nope", "lightning", "none") for k in kinds):
-            raise NotImplementedError(f"per-layer caches are built for attention without rotation ('nope') and 'lightning' layers, not {sorted(set(kinds))}")
+        if any(self._wants_tables(i) or k not in ("nope", "attention", "local", "mla", "lightning", "none") for i, k in enumerate(kinds)):
+            raise NotImplementedError("per-layer caches are built for attention without rotation ('nope') or with one of its own, 'mla' with one of its own and "
+                                      f"'lightning' layers, not {sorted(set(kinds))}")
         out, latest = [], {}
         for i, slot in self.runs():
             m = self.layers[i].mixer
-            if kinds[i] == "nope":
+            if kinds[i] == "mla":
+                out.append(CacheSlot(1, m.shape.row, m.shape.rank, latent=True))
+            elif kinds[i] in ("nope", "attention", "local"):
                 out.append(CacheSlot(m.num_kv_heads, m.head_dim, m.value_dim, source=None if m.own_kv else latest[cfg.of_layer(i).kv_from]))
                 latest[i] = slot if m.own_kv else out[-1].source
             else:
@@ -532,6 +555,13 @@ class CausalTransformer(nn.Module):
         return out
 
     # ------------------------------------------------------------------ helpers
+    def _wants_tables(self, i: int) -> bool:
+        """Whether layer ``i`` turns by the model's rotary tables."""
+        m, kind = self.layers[i].mixer, self.config.kinds()[i]
+        if kind not in ROTARY_KINDS or kind == "nope":
+            return False
+        return m.shape is None if kind == "mla" else getattr(m, "rotation", None) is None
+
     def head_weight(self) -> torch.Tensor:
         return self.embed.weight if self.head is None else self.head.weight
 
@@ -633,8 +663,7 @@ class CausalTransformer(nn.Module):
         """The stack over fp32 streams, up to the final norm; ``observe(run, total)`` sees the sum of the streams after every layer run."""
         from ..nn.streams import StreamStack
         cfg = self.config
-        if cfg.embed_scale or cfg.embed_multiplier is not None:
-            raise NotImplementedError("scaled embeddings are not built for the static-stream stack")
+        gain = (cfg.emb_features ** 0.5 if cfg.embed_scale else 1.0) * (1.0 if cfg.embed_multiplier is None else cfg.embed_multiplier)
         pos = None if self.position_embed is None else self.position_embed.weight
         if pos is not None and cache is None and tokens.shape[1] > pos.shape[0]:
             raise ValueError(f"{tokens.shape[1]} tokens do not fit the {pos.shape[0]} learned positions")
@@ -644,13 +673,15 @@ class CausalTransformer(nn.Module):
                 raise ValueError("this decoder's layers differ in what they keep: its cache comes from sampling.text.make_cache")
             if positions is None:
                 positions = torch.arange(tokens.shape[1], device=tokens.device)[None].expand(tokens.shape[0], -1)
+        if positions is not None and positions.shape != tokens.shape:
+            positions = positions.expand(tokens.shape)
         if cache is not None and steps is not None and steps != cfg.loop.steps:
             raise NotImplementedError("the cache holds the configured number of passes")
         if cache is None and any(self.layers[i].mixer is not None and not getattr(self.layers[i].mixer, "own_kv", True) for i, _ in runs):
             cache = Uncached(self.cache_slots())
-        H = ops_streams.embed_streams(tokens, positions, self.embed.weight, pos, max(1, cfg.hyper_connections))
+        H = ops_streams.embed_streams(tokens, positions, self.embed.weight, pos, max(1, cfg.hyper_connections), gain)
         stack = StreamStack(H, self.embed.weight.dtype)
-        cos, sin = (None, None) if all(k not in ROTARY_KINDS or k == "nope" for k in cfg.kinds()) else self.rope_tables(H.device)
+        cos, sin = self.rope_tables(H.device) if any(self._wants_tables(i) for i in range(len(self.layers))) else (None, None)
         for r, (i, slot) in enumerate(runs):
             self.layers[i].forward_static(stack, cos, sin, positions, None, cache, slot)
             if observe is not None:

@@ -20,7 +20,7 @@ class SelfAttention(nn.Module):
                  softcap: float = 0.0, sinks: bool = False, norm_eps: float = 1e-6, out_zero_init: bool = False,
                  init_std: Optional[float] = None, qkv_bias: bool = False, scale: Optional[float] = None, qk_norm_full: bool = False,
                  out_gate: bool = False, value_dim: Optional[int] = None, temperature=None, chunk: Optional[int] = None, head_gate: bool = False,
-                 own_kv: bool = True, dtype=None, device=None):
+                 own_kv: bool = True, rotation=None, keep_first: int = 0, unit_qk: bool = False, dtype=None, device=None):
         super().__init__()
         self.features, self.num_heads = features, num_heads
         # a softmax scale other than head_dim ** -0.5 is folded into the queries (after the norm and the rotation)
@@ -35,6 +35,15 @@ class SelfAttention(nn.Module):
         # a query sees no key from before the start of its chunk of positions; head_gate: each head's output times the sigmoid of one number from
         # the layer's input (its rows stand last in the projection); own_kv False: the layer reads another layer's keys and values
         self.chunk, self.head_gate, self.own_kv = chunk, head_gate, own_kv
+        # rotation: the layer's own (``ops.rotary.Rotary``) in place of the model's tables; keep_first: keys from the row's start that a window leaves
+        # visible; unit_qk: q and k over their root mean square per head, after the rotation and without a weight
+        self.rotation, self.keep_first, self.unit_qk = rotation, int(keep_first), unit_qk
+        if keep_first and window is None:
+            raise ValueError("keep_first belongs to a window")
+        if unit_qk and (qk_norm or qk_norm_full):
+            raise ValueError("q and k pass one norm: qk_norm (weights, in front of the rotation) or unit_qk (none, behind it)")
+        if rotation is not None and rotation.dims > self.head_dim:
+            raise ValueError(f"a rotation of {rotation.dims} dimensions does not fit heads of {self.head_dim}")
         self.heads = P.Heads(self.num_heads, self.num_kv_heads, self.head_dim, self.value_dim, own_kv, head_gate)
         self.qkv_proj = Linear(features, self.heads.row, bias=(bias or qkv_bias) and not head_gate, axes=("embed", "heads"), init_std=init_std, dtype=dtype,
                                device=device)
@@ -46,13 +55,13 @@ class SelfAttention(nn.Module):
         # Qwen3-Next: the heads' outputs pass a sigmoid gate computed from the layer's input, before the output projection
         self.gate_proj = Linear(features, self.num_heads * self.head_dim, axes=("embed", "heads"), init_std=init_std, dtype=dtype, device=device) if out_gate else None
         # OLMo-2 normalises q and k over all their heads at once (one weight of heads x head_dim); the usual form is per head
-        self.qk_norm_full = qk_norm_full
+        self.qk_norm_full, self.norm_eps = qk_norm_full, norm_eps
         qw, kw = (self.num_heads * self.head_dim, self.num_kv_heads * self.head_dim) if qk_norm_full else (self.head_dim, self.head_dim)
         self.q_norm = RMSNorm(qw, norm_eps, dtype=dtype, device=device) if (qk_norm or qk_norm_full) else None
         self.k_norm = RMSNorm(kw, norm_eps, dtype=dtype, device=device) if (qk_norm or qk_norm_full) and own_kv else None
         self.sinks = declare(nn.Parameter(torch.zeros(num_heads, dtype=dtype, device=device)), ("heads",), "sinks") if sinks else None
         # a layer whose rotary table differs from the model's: (theta, scaling) builds its own; rotary False drops the rotation (NoPE)
-        self.rotary, self.own_rope, self._own = True, None, None
+        self.rotary, self.own_rope, self._own = rotation is None, None, None
         self.head_transform = None     # a module applied to the heads' outputs [B, S, H, D] before the output projection (dew_b200.nn.dex)
         self.track_qk_max = False      # set by dew_b200.optim.qk_clip.watch: record each head's largest attention logit
         self.qk_max: Optional[torch.Tensor] = None
@@ -101,27 +110,30 @@ class SelfAttention(nn.Module):
         return self._own
 
     def _general(self, x, positions, segment_ids, cache, layer):
-        """Heads of any widths, the query temperature, chunks, head gates, layers that share keys and values, and caches whose layers differ; no
-        rotation."""
+        """Heads of any widths, the query temperature, chunks, head gates, windows that keep the first keys, layers that share keys and values, and
+        caches whose layers differ; a rotation is the layer's own."""
         from .kv_cache import Uncached
         B, S, _ = x.shape
-        if self.rotary or self.window is not None or self.softcap or self.gate_proj is not None or segment_ids is not None or not self.causal:
-            raise NotImplementedError("a query temperature, values of another width, chunks, head gates, shared keys and per-layer caches are built for "
-                                      "causal attention without rotation, window, soft cap, a full-width output gate or packed segments")
-        qw, eps = (None, 0.0) if self.q_norm is None else (self.q_norm.weight, self.q_norm.eps)
+        if self.rotary or self.gate_proj is not None or segment_ids is not None or not self.causal:
+            raise NotImplementedError("a query temperature, values of another width, chunks, head gates, kept first keys, shared keys and per-layer caches are "
+                                      "built for causal attention without the model's rotary tables, a full-width output gate or packed segments")
+        if self.temperature is not None and (self.rotation is not None or self.unit_qk):
+            raise NotImplementedError("a query temperature is built for layers without rotation and unit norms")
+        qw, eps = (None, self.norm_eps) if self.q_norm is None else (self.q_norm.weight, self.q_norm.eps)
         kw = None if self.k_norm is None else self.k_norm.weight
         # the bias joins in fp32 where the heads are normalised
         qkv = ops.linear(x, self.qkv_proj.weight) if type(self.qkv_proj) is Linear and self.qkv_proj.bias is not None else self.qkv_proj(x)
         bias = self.qkv_proj.bias if type(self.qkv_proj) is Linear and self.qkv_proj.bias is not None else self.heads_bias
         cache = Uncached(()) if cache is None else cache
         o = cache.attend_slot(layer, qkv, self.heads, positions, scale=self.scale, eps=eps, q_weight=qw, k_weight=kw, temperature=self.temperature,
-                              bias=bias, chunk=self.chunk, sinks=self.sinks)
+                              bias=bias, chunk=self.chunk, sinks=self.sinks, window=self.window, keep=self.keep_first, softcap=self.softcap, rot=self.rotation,
+                              unit=self.unit_qk)
         return self.o_proj(o.reshape(B, S, self.num_heads * self.value_dim))
 
     def forward(self, x, cos=None, sin=None, positions=None, segment_ids=None, cache=None, layer: int = 0):
         B, S, _ = x.shape
         if getattr(cache, "slots", None) is not None or self.temperature is not None or self.value_dim != self.head_dim or self.chunk is not None \
-                or self.head_gate or not self.own_kv:
+                or self.head_gate or not self.own_kv or self.rotation is not None or self.keep_first or self.unit_qk:
             return self._general(x, positions, segment_ids, cache, layer)
         cos, sin = self._tables(cos, sin)
         if (cache is None and x.is_cuda and cos is not None and self.head_transform is None and self.gate_proj is None and self.q_norm is None and self.window is None and not self.softcap

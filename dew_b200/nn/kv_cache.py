@@ -3,8 +3,8 @@
 Parity: src/dew/nn/kv_cache.py (``KVCache`` spec :362-408 - ``quantized``, ``page_size``, ``pages``, ``groups``,
 ``offloaded``; ``quantize`` / ``dequantize`` :411-446 per-token-per-head absmax scales; ``hadamard`` :465-479;
 ``KVStore.write / attend / decode`` :787-1180; pool layout :1297-1320; ``gather_cache_rows`` :1686).
-A decoder whose layers differ in what they keep (heads of other widths, recurrent states, a layer that runs several times) gives the store
-one ``CacheSlot`` per layer run; ``attend_slot`` and ``state`` then take the place of ``attend``.
+A decoder whose layers differ in what they keep (heads of other widths, latent rows, recurrent states, a layer that runs several times) gives the
+store one ``CacheSlot`` per layer run; ``attend_slot``, ``attend_latent`` and ``state`` then take the place of ``attend``.
 Pool layout here: ``[layers, pages, page_size, kv_heads, head_dim]`` for keys and for values, a page table
 ``[rows, max_pages]`` and ``lengths [rows]``; a dense cache is the special case of one page per row.
 """
@@ -19,8 +19,10 @@ from typing import Dict, List, Optional, Sequence, Tuple
 import torch
 
 from .. import ops
+from ..ops import latent as M
 from ..ops import library as L
 from ..ops import paged as P
+from ..ops import rotary
 
 LIMITS = {"int8": 127.0, "float8_e4m3fn": 448.0}
 KINDS = {None: 0, "int8": 1, "float8_e4m3fn": 2}
@@ -41,18 +43,19 @@ class KVCache:
 
 @dataclass(frozen=True)
 class CacheSlot:
-    """What one run of a layer keeps per row: keys and values of its own head count and widths, a recurrent state (a shape, fp32), or nothing: it
-    reads the keys and values of the earlier slot ``source``."""
+    """What one run of a layer keeps per row: keys and values of its own head count and widths (with ``latent``, rows of which the first ``value_dim``
+    columns are the values too), a recurrent state (a shape, fp32), or nothing: it reads the keys and values of the earlier slot ``source``."""
     kv_heads: int = 0
     head_dim: int = 0
     value_dim: int = 0
     state: Optional[Tuple[int, ...]] = None
     source: Optional[int] = None
+    latent: bool = False
 
 
 @dataclass
 class Call:
-    """The integers of one forward call, computed once for all its layers.  ``key`` holds the positions tensor itself, so its memory cannot
+    """The integers of one forward call, and its angles, computed once for all its layers.  ``key`` holds the positions tensor itself, so its memory cannot
     be handed to another tensor while this entry can still be found."""
     key: torch.Tensor
     version: int
@@ -64,10 +67,21 @@ class Call:
     table: torch.Tensor                      # int32 [R, max_pages]: the call rows' page tables
     fresh: Optional[bool] = None             # every row starts at its first token (None: not looked at)
     kept: Dict[int, torch.Tensor] = field(default_factory=dict)      # slot -> this call's packed heads, while later layers read its keys and values
+    angles: Dict[rotary.Rotary, torch.Tensor] = field(default_factory=dict)
+
+    def turned(self, rot: Optional[rotary.Rotary]) -> Optional[P.Turned]:
+        if rot is None:
+            return None
+        if rot not in self.angles:
+            self.angles[rot] = rotary.angles(self.positions, rot)
+        return P.Turned(rot, self.angles[rot])
 
 
 def pool_width(slot: CacheSlot, dtype) -> int:
-    """Width of a slot's pool heads: what the bf16 kernels are built for (64, 128, 256) where the head fits, else the head rounded up to 8."""
+    """Width of a slot's pool heads: what the bf16 kernels are built for (64, 128, 256) where the head fits, else the head rounded up to 8; latent rows
+    are rounded up to 16."""
+    if slot.latent:
+        return (slot.head_dim + 15) // 16 * 16
     w = max(slot.head_dim, slot.value_dim)
     if dtype == torch.bfloat16:
         for d in (64, 128, 256):
@@ -131,7 +145,8 @@ class KVStore:
                     raise ValueError(f"slot {i} reads the keys and values of slot {s.source}, which keeps none of its own before it")
             pool = lambda s: None if s.state is not None or s.source is not None else \
                 torch.zeros(self.pages + 1, self.page_size, s.kv_heads, pool_width(s, dtype), dtype=dtype, device=device)
-            self.k, self.v = [pool(s) for s in self.slots], [pool(s) for s in self.slots]
+            self.k = [pool(s) for s in self.slots]
+            self.v = [k if s.latent else pool(s) for k, s in zip(self.k, self.slots)]
             for pools in (self.k, self.v):
                 for i, s in enumerate(self.slots):
                     if s.source is not None:
@@ -152,6 +167,7 @@ class KVStore:
         self.row_ids: Optional[torch.Tensor] = None      # rows of the store addressed by the batch rows of a call
         self._scratch = None
         self.chunk_span: Optional[Tuple[int, int]] = None      # (first position, one past the last) of the prefill chunk in flight, when the caller knows
+        self.together = True         # whether every row of that chunk starts at its first position
 
     # ------------------------------------------------------------------ layers that differ (CacheSlot)
     @property
@@ -182,9 +198,10 @@ class KVStore:
         return c.fresh
 
     def attend_slot(self, slot: int, qkv: torch.Tensor, heads: P.Heads, positions: torch.Tensor, *, scale: float, eps: float = 1e-6, q_weight=None,
-                    k_weight=None, temperature=None, bias=None, chunk: Optional[int] = None, sinks: Optional[torch.Tensor] = None) -> torch.Tensor:
-        """A layer's attention from its packed projection ``qkv [R, S, heads.row]``: bias, norms, temperature, append, causal attention against
-        everything the rows hold (of a query's own ``chunk`` of positions, with ``sinks``, times the heads' gates).  -> ``[R, S, H, dv]``.  A
+                    k_weight=None, temperature=None, bias=None, chunk: Optional[int] = None, sinks: Optional[torch.Tensor] = None,
+                    window: Optional[int] = None, keep: int = 0, softcap: float = 0.0, rot: Optional[rotary.Rotary] = None, unit: bool = False) -> torch.Tensor:
+        """A layer's attention from its packed projection ``qkv [R, S, heads.row]``: bias, norms, rotation, temperature, append, causal attention
+        against everything the rows hold (or what ``paged.Visible`` leaves of it, times the heads' gates).  -> ``[R, S, H, dv]``.  A
         prompt from its first token takes the tcgen05 flash kernel, a decode step the paged decode kernels, anything else (and fp32) the
         general paged kernel.  A slot with a source appends nothing and reads the source's keys and values."""
         c = self.call(positions)
@@ -192,9 +209,9 @@ class KVStore:
         if (source is None) != heads.own:
             raise ValueError(f"slot {slot}: the layer and the cache disagree on whether it has keys and values of its own")
         pages = P.Pages(self.k[slot], self.v[slot], self.page_table, self.page_size, c.row_ids)
-        packed = P.qk_norm_append(qkv, heads, q_weight, k_weight, eps, temperature, c.positions, pages, bias)
+        packed = P.qk_norm_append(qkv, heads, q_weight, k_weight, eps, temperature, c.positions, pages, bias, c.turned(rot), unit)
         gate = qkv[..., heads.packed:] if heads.gated else None
-        visible = P.Visible(chunk, None if sinks is None else self._fp32_sinks(slot, sinks))
+        visible = P.Visible(chunk, None if sinks is None else self._fp32_sinks(slot, sinks), window, keep if window else 0, softcap)
         R, S = positions.shape
         H, G = heads.q, heads.kv
         D = packed.shape[-1]
@@ -210,7 +227,8 @@ class KVStore:
                 if source is not None and self.last_reader[source] == slot:
                     c.kept.pop(source, None)
                 if kv is not None:
-                    out, _ = flash_fwd(q, kv[:, :, :G], kv[:, :, G:], True, scale, need_lse=False, var=Variants(sinks=visible.sinks, chunk=chunk))
+                    out, _ = flash_fwd(q, kv[:, :, :G], kv[:, :, G:], True, scale, need_lse=False, var=Variants(visible.window, softcap, visible.sinks, chunk=chunk,
+                                                                                                                keep=visible.keep))
                     return P.head_gate(out, gate, heads.dv)
         return P.paged_attend(q, heads, c.positions, pages, scale, visible=visible, gate=gate)
 
@@ -227,28 +245,55 @@ class KVStore:
         R, D, H, G = packed.shape[0], packed.shape[-1], heads.q, heads.kv
         out = torch.empty(R, H, D, dtype=packed.dtype, device=packed.device)
         if D == 128 and self.page_size % 64 == 0 and H // G <= 8 and hasattr(lib, "dewb_paged_decode_persist"):
-            self._fused_decode(lib, slot, packed, packed.shape[2] * D, c.lengths, R, H, D, None, visible.sinks, out, scale=scale, kv_heads=G, table=c.table,
-                               chunk=visible.chunk)
+            self._fused_decode(lib, slot, packed, packed.shape[2] * D, c.lengths, R, H, D, visible.window, visible.sinks, out, scale=scale, kv_heads=G, table=c.table,
+                               visible=visible)
             return out
         q = packed[:, 0, :H].contiguous()
         share = next(s for s in range(1, H // G + 1) if (H // G) % s == 0 and H // G // s <= 8)     # CTAs that share a key / value head
-        splits, longest = 1, min(self.max_len, visible.chunk or self.max_len)
+        splits, longest = 1, min(self.max_len, visible.chunk or self.max_len, visible.window + visible.keep if visible.window else self.max_len)
         while splits < 16 and R * G * share * splits < 592 and longest // (splits * 2) >= 256:
             splits *= 2
         pm, pl, pa = self._partials(R * H * splits, D, q.device)
         L.check(lib.dewb_paged_decode(L.ptr(q), L.ptr(self.k[slot]), L.ptr(self.v[slot]), L.ptr(None), L.ptr(None), L.ptr(c.table), L.ptr(c.lengths),
                                       L.ptr(visible.sinks), L.ptr(out), L.ptr(None), L.ptr(pm), L.ptr(pl), L.ptr(pa), ctypes.c_int(R), ctypes.c_int(H),
                                       ctypes.c_int(G), ctypes.c_int(share), ctypes.c_int(D), ctypes.c_int(self.page_size), ctypes.c_int(self.max_pages),
-                                      ctypes.c_int(splits), ctypes.c_float(scale), ctypes.c_int(0), ctypes.c_int(visible.chunk or 0), ctypes.c_int(0), L.stream_ptr()),
+                                      ctypes.c_int(splits), ctypes.c_float(scale), ctypes.c_int(visible.window or 0), ctypes.c_int(visible.keep),
+                                      ctypes.c_int(visible.chunk or 0), ctypes.c_float(visible.softcap), ctypes.c_int(0), L.stream_ptr()),
                 "paged_decode")
         L.count_launches(2)
         return out
 
     def _partials(self, n: int, D: int, device):
-        if self._scratch is None or self._scratch[0].numel() < n or self._scratch[2].numel() < n * D:
-            self._scratch = (torch.empty(n, dtype=torch.float32, device=device), torch.empty(n, dtype=torch.float32, device=device),
-                             torch.empty(n * D, dtype=torch.float32, device=device))
+        """Scratch for ``n`` partial sums of ``D`` values.  The buffers grow apart and never shrink, so that layers of different shapes settle on one
+        set (a captured step keeps using what its warm-up left)."""
+        have = [0, 0, 0] if self._scratch is None else [t.numel() for t in self._scratch]
+        if any(h < w for h, w in zip(have, (n, n, n * D))):
+            self._scratch = tuple(t if t is not None and t.numel() >= w else torch.empty(w, dtype=torch.float32, device=device)
+                                  for t, w in zip(self._scratch or (None,) * 3, (n, n, n * D)))
         return self._scratch
+
+    def attend_latent(self, slot: int, z: torch.Tensor, queries, up: torch.Tensor, lat: M.Latent, positions: torch.Tensor, *, scale: float, eps: float,
+                      q_weight=None, kv_weight=None, gated: bool = False) -> torch.Tensor:
+        """A latent attention layer from its input projection ``z [R, S, q_rank | rank | rot_dim (| gate)]``: norms, rotation, append, causal attention
+        against everything the rows hold, up-projection, gate.  ``queries`` makes ``[R, S, H * width]`` of the normed query latent; ``up`` is the
+        keys' and values' up-projection ``[H * (dim + vdim), rank]``.  -> ``[R, S, H * vdim]``.  Portions whose rows start together form their keys
+        in full width and take the tcgen05 flash kernel; decode steps, mixed positions and fp32 stay in the latents' space."""
+        c = self.call(positions)
+        pages = P.Pages(self.k[slot], self.v[slot], self.page_table, self.page_size, c.row_ids)
+        table = c.turned(lat.rotary).table
+        cq, made = M.rows(z, lat, q_weight, kv_weight, eps, table, c.positions, pages)
+        R, S = positions.shape
+        q = queries(cq).view(R, S, lat.heads, lat.width)
+        gate = z[..., lat.q_rank + lat.row:] if gated else None
+        if L.use_cuda(z) and S > 1 and M.flash_ok(q, lat):
+            start = 0 if self.is_fresh(c) else self.chunk_span[0] if self.chunk_span is not None and self.together else None
+            if start is not None:
+                if start > 0:
+                    made = M.gather(lat, c.lengths, start + S, pages)
+                return M.flash(M.rotate(q, lat, table), made, up, lat, scale, gate)
+        o = M.attend(M.absorb(q, up, lat, table, self.k[slot].shape[-1]), lat, c.positions, pages, scale, self.max_len,
+                     lambda n, width: self._partials(n, width, z.device))
+        return M.expand(o, up, lat, gate)
 
     # ------------------------------------------------------------------ latent rows (multi-head latent attention)
     def latent(self, layer: int, width: int) -> torch.Tensor:
@@ -346,11 +391,11 @@ class KVStore:
 
     def _fused_decode(self, lib, layer: int, q, q_row_stride: int, lens32, R: int, Hq: int, D: int, window, sinks32, out,
                       scale: Optional[float] = None, kv_heads: Optional[int] = None, table: Optional[torch.Tensor] = None,
-                      chunk: Optional[int] = None) -> None:
+                      visible: P.Visible = P.PLAIN) -> None:
         """The streamed paged-attention kernel finishing its rows itself.  Up to 1024 rows take the balanced persistent form
         (every CTA moves the same number of tiles, whatever the rows' lengths); more rows take one CTA per (row, head, chunk)."""
-        longest = min(self.max_len, window or self.max_len, chunk or self.max_len)
-        max_tiles = -(-longest // 64) + 1                                 # (+ 1: a window that straddles a tile boundary)
+        longest = min(self.max_len, window + visible.keep if window else self.max_len, visible.chunk or self.max_len)
+        max_tiles = -(-longest // 64) + 1 + int(visible.keep > 0)         # (+ 1: a window, or kept first keys, that straddle a tile boundary)
         persist = R <= 1024 and os.environ.get("DEWB_DECODE_PERSIST", "1") == "1"
         if persist:
             min_tiles = int(os.environ.get("DEWB_DECODE_MIN_TILES", self.MIN_TILES))
@@ -372,11 +417,13 @@ class KVStore:
             if getattr(self, "_ctas", None) is None:
                 self._ctas = 2 * torch.cuda.get_device_properties(q.device).multi_processor_count
             L.check(lib.dewb_paged_decode_persist(*common, ctypes.c_int(min_tiles), ctypes.c_float(scale),
-                                                  ctypes.c_int(window or 0), ctypes.c_int(chunk or 0), ctypes.c_longlong(q_row_stride), ctypes.c_int(self._ctas),
+                                                  ctypes.c_int(window or 0), ctypes.c_int(visible.keep), ctypes.c_int(visible.chunk or 0),
+                                                ctypes.c_float(visible.softcap), ctypes.c_longlong(q_row_stride), ctypes.c_int(self._ctas),
                                                   L.ptr(L.status(q.device)), L.stream_ptr()), "paged_decode_persist")
         else:
             L.check(lib.dewb_paged_decode_fused(*common, ctypes.c_int(share), ctypes.c_float(scale),
-                                                ctypes.c_int(window or 0), ctypes.c_int(chunk or 0), ctypes.c_longlong(q_row_stride),
+                                                ctypes.c_int(window or 0), ctypes.c_int(visible.keep), ctypes.c_int(visible.chunk or 0),
+                                                ctypes.c_float(visible.softcap), ctypes.c_longlong(q_row_stride),
                                                 L.ptr(L.status(q.device)), L.stream_ptr()), "paged_decode_fused")
         L.count_launches()
 
@@ -446,7 +493,7 @@ class KVStore:
                                                      L.ptr(pm), L.ptr(pl), L.ptr(pa), ctypes.c_int(R), ctypes.c_int(Hq),
                                                      ctypes.c_int(self.kv_heads), ctypes.c_int(self.page_size), ctypes.c_int(self.max_pages),
                                                      ctypes.c_int(splits), ctypes.c_float(scale), ctypes.c_int(window or 0), ctypes.c_int(0),
-                                                     ctypes.c_longlong(0), L.ptr(L.status(q.device)), L.stream_ptr()), "paged_decode_stream")
+                                                     ctypes.c_int(0), ctypes.c_float(0.0), ctypes.c_longlong(0), L.ptr(L.status(q.device)), L.stream_ptr()), "paged_decode_stream")
                 L.check(lib.dewb_decode_combine(L.ptr(pm), L.ptr(pl), L.ptr(pa), L.ptr(sinks32),
                                                 L.ptr(out), L.ptr(None), ctypes.c_int(R), ctypes.c_int(Hq), ctypes.c_int(D), ctypes.c_int(splits),
                                                 L.stream_ptr()), "decode_combine")
@@ -459,7 +506,8 @@ class KVStore:
                                           L.ptr(pm), L.ptr(pl), L.ptr(pa), ctypes.c_int(R), ctypes.c_int(Hq),
                                           ctypes.c_int(self.kv_heads), ctypes.c_int(1), ctypes.c_int(D), ctypes.c_int(self.page_size),
                                           ctypes.c_int(self.max_pages), ctypes.c_int(splits), ctypes.c_float(scale),
-                                          ctypes.c_int(window or 0), ctypes.c_int(0), ctypes.c_int(self.kind), L.stream_ptr()), "paged_decode")
+                                          ctypes.c_int(window or 0), ctypes.c_int(0), ctypes.c_int(0), ctypes.c_float(0.0), ctypes.c_int(self.kind),
+                                          L.stream_ptr()), "paged_decode")
             L.count_launches(2)
             return out
         return paged_attention_reference(self, layer, q, lengths, scale, window, sinks, softcap)
@@ -506,18 +554,47 @@ class Uncached:
         self.kept: Dict[int, Tuple[torch.Tensor, torch.Tensor]] = {}
 
     def attend_slot(self, slot: int, qkv, heads: P.Heads, positions, *, scale: float, eps: float = 1e-6, q_weight=None, k_weight=None, temperature=None,
-                    bias=None, chunk: Optional[int] = None, sinks=None) -> torch.Tensor:
+                    bias=None, chunk: Optional[int] = None, sinks=None, window: Optional[int] = None, keep: int = 0, softcap: float = 0.0,
+                    rot: Optional[rotary.Rotary] = None, unit: bool = False) -> torch.Tensor:
         R, S, _ = qkv.shape
         pos = torch.arange(S, device=qkv.device)[None].expand(R, S) if positions is None else positions
-        q, k, v = P.prepare_reference(qkv, heads, q_weight, k_weight, eps, temperature, pos, bias)
+        turned = None if rot is None else P.Turned(rot, rotary.angles_reference(pos, rot))
+        q, k, v = P.prepare_reference(qkv, heads, q_weight, k_weight, eps, temperature, pos, bias, turned, unit)
         if not heads.own:
             k, v = self.kept[self.source_of[slot]]
         elif slot in self.sources:
             self.kept[slot] = (k, v)
         # chunks counted from the first position: documents of the packed-segment form, with ids that start at 1
         segments = None if not chunk else (torch.arange(S, device=qkv.device, dtype=torch.int32) // chunk + 1)[None].expand(R, S).contiguous()
-        o = ops.attention(q, k, v, causal=True, scale=scale, sinks=sinks, segment_ids=segments)
+        if keep and window:
+            o = visible_attention(q, k, v, scale, P.Visible(chunk, sinks, window, keep, softcap))
+        else:
+            o = ops.attention(q, k, v, causal=True, scale=scale, sinks=sinks, segment_ids=segments, window=window, softcap=softcap)
         return P.head_gate_reference(o, qkv[..., heads.packed:] if heads.gated else None, heads.dv)
+
+    def attend_latent(self, slot: int, z, queries, up, lat: M.Latent, positions, *, scale: float, eps: float, q_weight=None, kv_weight=None,
+                      gated: bool = False) -> torch.Tensor:
+        R, S, _ = z.shape
+        pos = torch.arange(S, device=z.device)[None].expand(R, S) if positions is None else positions
+        table = rotary.angles_reference(pos, lat.rotary)
+        cq, made = M.prepare_reference(z, lat, q_weight, kv_weight, eps, table)
+        q = queries(cq).view(R, S, lat.heads, lat.width)
+        q = torch.cat([q[..., :lat.dim], rotary.turn(q[..., lat.dim:], table, lat.rotary).to(q.dtype)], -1)
+        wk, wv = lat.split_up(up)
+        k = torch.einsum("rsl,hdl->rshd", made.c, wk)
+        k = torch.cat([k, made.key.unsqueeze(2).expand(R, S, lat.heads, lat.rot_dim)], -1)
+        o = ops.attention(q, k, torch.einsum("rsl,hvl->rshv", made.c, wv), causal=True, scale=scale)
+        return M.gate_reference(o.reshape(R, S, lat.heads * lat.vdim), z[..., lat.q_rank + lat.row:] if gated else None)
+
+
+def visible_attention(q, k, v, scale: float, visible: P.Visible) -> torch.Tensor:
+    """Causal attention over whole rows as ``visible`` limits it: ``q [R, S, H, dk]``, ``k, v [R, S, G, *]`` (plain, differentiable)."""
+    R, S, H, _ = q.shape
+    k, v = (t.float().repeat_interleave(H // t.shape[2], 2) for t in (k, v))
+    seen = P.seen_keys(torch.arange(S, device=q.device)[None].expand(R, S), S, visible)
+    s = torch.einsum("rshd,rnhd->rhsn", q.float(), k) * scale
+    s = s if not visible.softcap else visible.softcap * torch.tanh(s / visible.softcap)
+    return torch.einsum("rhsn,rnhd->rshd", P.softmax_with_sinks(s.masked_fill(~seen[:, None], float("-inf")), visible.sinks), v).to(q.dtype)
 
 
 def paged_attention_reference(store: KVStore, layer: int, q, lengths, scale, window=None, sinks=None, softcap=0.0):

@@ -63,17 +63,21 @@ class Embedding(nn.Module):
 
 
 class RMSNorm(nn.Module):
-    def __init__(self, features: int, eps: float = 1e-6, dtype=None, device=None):
+    """``around``: the weights are stored as their distance from it (built for the norms of fp32 residual streams, ``nn.streams``)."""
+
+    def __init__(self, features: int, eps: float = 1e-6, dtype=None, device=None, around: float = 0.0):
         super().__init__()
-        self.eps = eps
-        self.weight = declare(nn.Parameter(torch.ones(features, dtype=dtype, device=device)), ("norm",), "scale")
+        self.eps, self.around = eps, float(around)
+        self.weight = declare(nn.Parameter(torch.full((features,), 1.0 - around, dtype=dtype, device=device)), ("norm",), "scale")
 
     def reset_parameters(self, generator=None):
         with torch.no_grad():
-            self.weight.fill_(1.0)
+            self.weight.fill_(1.0 - self.around)
 
     def forward(self, x, branch=None):
         """With ``branch``: residual-stream form, returns ``(norm(x + branch), x + branch)``."""
+        if self.around:
+            raise NotImplementedError("norm weights stored around another value than 0 belong to fp32 residual streams")
         if branch is not None:
             return ops.stream_rms_norm(x, branch, self.weight, self.eps)
         return ops.rms_norm(x, self.weight, self.eps)

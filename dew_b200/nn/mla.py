@@ -1,6 +1,9 @@
 """Multi-head latent attention (DeepSeek-V2/V3): keys and values are reconstructed from a small shared latent (the KV
 cache holds the latent and one shared rotary key per token), queries optionally from their own latent; each head has a
-rotary part and a no-position part.  Reference: src/dew/nn/mla.py (1240 lines)."""
+rotary part and a no-position part.  Reference: src/dew/nn/mla.py (1240 lines).
+
+With a ``rotation`` of its own the layer belongs to decoders whose layers differ in what they keep: its input projections stand in one weight
+(query latent | latent | rotated key part | output gate), and its cache slot holds paged rows of latents (``ops.latent``)."""
 from __future__ import annotations
 
 from typing import Optional
@@ -9,24 +12,37 @@ import torch
 import torch.nn as nn
 
 from .. import ops
+from ..ops.latent import Latent
 from .layers import Linear, RMSNorm
 
 
 class MultiHeadLatentAttention(nn.Module):
     def __init__(self, features: int, num_heads: int, kv_latent: int = 512, q_latent: Optional[int] = None, nope_dim: int = 128,
                  rope_dim: int = 64, v_dim: int = 128, norm_eps: float = 1e-6, causal: bool = True, softmax_gain: float = 1.0,
-                 dtype=None, device=None):
+                 rotation=None, scale: Optional[float] = None, out_gate: bool = False, dtype=None, device=None):
         super().__init__()
+        if rotation is None and (out_gate or scale is not None):
+            raise NotImplementedError("an output gate and a configured scale are built for latent attention with a rotation of its own")
+        if rotation is not None and not causal:
+            raise NotImplementedError("latent attention with a rotation of its own is built for causal attention")
         # softmax_gain multiplies the (nope + rope) ** -0.5 scale: DeepSeek-V3's long-context releases raise it by YaRN's magnitude squared
         self.softmax_gain = float(softmax_gain)
         self.h, self.nope, self.rope, self.vd, self.causal = num_heads, nope_dim, rope_dim, v_dim, causal
         kw = dict(dtype=dtype, device=device)
         qd = num_heads * (nope_dim + rope_dim)
-        if q_latent:
+        self.shape = None if rotation is None else Latent(num_heads, nope_dim, rope_dim, v_dim, kv_latent, q_latent or 0, rotation)
+        if self.shape is not None:
+            self.scale = (nope_dim + rope_dim) ** -0.5 * self.softmax_gain if scale is None else float(scale)
+            self.out_gate = out_gate
+            self.in_proj = Linear(features, (q_latent or 0) + kv_latent + rope_dim + (num_heads * v_dim if out_gate else 0), axes=("embed", "heads"), **kw)
+            self.q_norm = RMSNorm(q_latent, norm_eps, **kw) if q_latent else None
+            self.q_up = Linear(q_latent or features, qd, **kw)
+        elif q_latent:
             self.q_down, self.q_norm, self.q_up = Linear(features, q_latent, **kw), RMSNorm(q_latent, norm_eps, **kw), Linear(q_latent, qd, **kw)
         else:
             self.q_down, self.q_norm, self.q_up = None, None, Linear(features, qd, **kw)
-        self.kv_down = Linear(features, kv_latent + rope_dim, **kw)          # latent | shared rotary key
+        if self.shape is None:
+            self.kv_down = Linear(features, kv_latent + rope_dim, **kw)      # latent | shared rotary key
         self.kv_norm = RMSNorm(kv_latent, norm_eps, **kw)
         self.kv_up = Linear(kv_latent, num_heads * (nope_dim + v_dim), **kw)
         self.o_proj = Linear(num_heads * v_dim, features, **kw)
@@ -72,9 +88,21 @@ class MultiHeadLatentAttention(nn.Module):
         o_lat = torch.einsum("rsht,rtl->rshl", p, c)
         return torch.einsum("rshl,hvl->rshv", o_lat, w_uv.float()).to(q_nope.dtype)
 
+    def _paged(self, x, positions, segment_ids, cache, layer: int):
+        if segment_ids is not None:
+            raise NotImplementedError("latent attention with a rotation of its own runs on token rows without packed segments")
+        from .kv_cache import Uncached
+        cache = Uncached(()) if cache is None else cache
+        queries = (lambda c: self.q_up(x)) if self.q_norm is None else self.q_up
+        o = cache.attend_latent(layer, self.in_proj(x), queries, self.kv_up.weight, self.shape, positions, scale=self.scale, eps=self.kv_norm.eps,
+                                q_weight=None if self.q_norm is None else self.q_norm.weight, kv_weight=self.kv_norm.weight, gated=self.out_gate)
+        return self.o_proj(o)
+
     def forward(self, x, cos=None, sin=None, positions=None, segment_ids=None, cache=None, layer: int = 0):
         B, T, _ = x.shape
         H = self.h
+        if self.shape is not None:
+            return self._paged(x, positions, segment_ids, cache, layer)
         q = self.q_up(x) if self.q_down is None else self.q_up(self.q_norm(self.q_down(x)))
         q = q.view(B, T, H, self.nope + self.rope)
         c, k_rope = self.latent(x)

@@ -29,9 +29,11 @@ class SwiGLU(nn.Module):
             if type(self.gate_up_proj).__name__ == "Linear" and self.gate_up_proj.bias is None:
                 return self.down_proj(ops.linear_swiglu(x, self.gate_up_proj.weight))
             return self.down_proj(ops.packed_swiglu(self.gate_up_proj(x)))
-        gu = self.gate_up_proj(x)
-        g, u = gu.chunk(2, -1)                                    # GeGLU (Gemma): the gate passes through GELU
-        return self.down_proj(F.gelu(g, approximate="tanh" if self.activation == "gelu_tanh" else "none") * u)
+        gu = self.gate_up_proj(x)                                 # GeGLU (Gemma): the gate passes through GELU
+        if self.activation == "gelu_tanh":
+            return self.down_proj(streams.gelu_glu(gu))
+        g, u = gu.chunk(2, -1)
+        return self.down_proj(F.gelu(g) * u)
 
 
 class ClampedGLU(nn.Module):

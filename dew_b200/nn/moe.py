@@ -33,18 +33,24 @@ class Router(nn.Module):
         self.mix = mix
         self._split = None
         self.weight = declare(nn.Parameter(torch.empty(mix.experts, features, dtype=dtype, device=device)), ("experts", "embed"), "kernel")
+        self.logit_bias = declare(nn.Parameter(torch.zeros(mix.experts, dtype=torch.float32, device=device)), ("experts",), "bias") if mix.router_bias else None
         self.register_buffer("expert_bias", torch.zeros(mix.experts, dtype=torch.float32, device=device) if mix.bias else None, persistent=True)
         self.reset_parameters()
 
     def reset_parameters(self, generator=None):
         with torch.no_grad():
             self.weight.normal_(0.0, 1.0 / math.sqrt(self.weight.shape[1]), generator=generator)
+            if self.logit_bias is not None:
+                self.logit_bias.zero_()
+
+    def logits(self, x2: torch.Tensor) -> torch.Tensor:
+        return F.linear(x2.float(), self.weight.float(), self.logit_bias)
 
     def forward(self, x2: torch.Tensor):
         """``x2 [T, d]`` -> (weights [T, k] fp32, expert ids [T, k], scores [T, E] fp32)."""
         mix = self.mix
-        logits = F.linear(x2.float(), self.weight.float())
-        if logits.is_cuda and mix.experts <= 256 and mix.top_k <= 16 and self.use_kernels and mix.groups <= 1:
+        logits = self.logits(x2)
+        if logits.is_cuda and mix.experts <= 256 and mix.top_k <= 16 and self.use_kernels and mix.groups <= 1 and mix.score_function != "top_softmax":
             from ..ops.routing import route
             return route(logits, self.expert_bias, mix.top_k, mix.score_function, mix.norm_topk_prob, mix.scaling)
         # the bias steers the selection only; group-limited routing (DeepSeek-V3): a group's score is the sum of its two best experts, and
@@ -143,7 +149,8 @@ class SparseMLP(nn.Module):
     def _serve(self, x2: torch.Tensor, positions: Optional[torch.Tensor]) -> torch.Tensor:
         """Forward alone: no statistics, and no expert runs for tokens at positions below 0."""
         pos = None if positions is None else positions.reshape(-1).to(torch.int32)
-        r = serve.route(x2, self.router.weight, self.router.split() if x2.dtype == torch.bfloat16 else None, self.router.expert_bias, self.router.selection, pos)
+        r = serve.route(x2, self.router.weight, self.router.split() if x2.dtype == torch.bfloat16 else None, self.router.expert_bias, self.router.selection, pos,
+                        logit_bias=self.router.logit_bias)
         s = serve.gather(x2, r, None if self.shared_gate is None else self.shared_gate.weight)
         y = serve.product(serve.glu(serve.product(s.rows, self.experts.gate_up, s), s), self.experts.down, s)
         return serve.combine(y, r, s, None if self.shared is None else self.shared(x2))
@@ -170,7 +177,7 @@ class SparseMLP(nn.Module):
         self.last = {"counts": counts, "balance_loss": mix.experts * (frac * scores.mean(0)).sum()}
         if self.keep_router_outputs:
             self.last.update(scores=scores, ids=ids, shape=(int(math.prod(shape[:-2])) if len(shape) > 2 else 1, int(shape[-2])),
-                             log_z=torch.logsumexp(F.linear(x2.float(), self.router.weight.float()), -1))
+                             log_z=torch.logsumexp(self.router.logits(x2), -1))
         if self.ep is not None:
             y = self.ep.dispatch_compute_combine(self, x2, w, ids)
         elif x2.is_cuda and x2.dtype == torch.bfloat16 and mix.experts <= 256 and mix.top_k <= 16 and self.use_kernels:

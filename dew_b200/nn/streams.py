@@ -78,10 +78,12 @@ class StreamStack:
         """The next sub-layer's normalised input."""
         return self._step(None if connection is None else connection.alpha, norm)
 
-    def leave(self, connection: Optional["HyperConnections"], y: torch.Tensor, scale=None, norm: Optional[nn.Module] = None) -> None:
-        """The sub-layer's output (through an RMS ``norm`` of its own, times its layer scale), to be written back by the connection."""
+    def leave(self, connection: Optional["HyperConnections"], y: torch.Tensor, scale=None, norm: Optional[nn.Module] = None, gain: float = 1.0,
+              beside: Optional[torch.Tensor] = None, beside_scale=None) -> None:
+        """The sub-layer's output (through an RMS ``norm`` of its own, times its layer scale), to be written back by the connection; ``beside`` is the
+        output of a second sub-layer that read the same norm, ``gain`` multiplies both."""
         mix, out = (None, None) if connection is None else (connection.mix, connection.beta)
-        self.pending = S.Write(y, scale, mix, out, *((None, 0.0) if norm is None else (norm.weight, norm.eps)))
+        self.pending = S.Write(y, scale, mix, out, *((None, 0.0) if norm is None else (norm.weight, norm.eps)), beside, beside_scale, gain)
 
     def finish(self, norm: nn.Module) -> torch.Tensor:
         """The final norm of the sum of the streams."""
@@ -96,7 +98,7 @@ class StreamStack:
 
     def _step(self, read, norm) -> torch.Tensor:
         kind = "layer" if isinstance(norm, LayerNorm) else "rms"
-        n, self.H = S.stream_step(self.H, self.pending, read, norm.weight, norm.eps, self.dtype, kind)
+        n, self.H = S.stream_step(self.H, self.pending, read, norm.weight, norm.eps, self.dtype, kind, getattr(norm, "around", 0.0))
         self.pending = None
         return n
 

@@ -17,14 +17,16 @@ def _strides(t):
 
 
 class Variants:
-    """The optional attention variants the kernels take: ``window`` (keys visible behind each query, None = all), ``chunk`` (a query sees no key
+    """The optional attention variants the kernels take: ``window`` (keys visible behind each query, None = all; with ``keep`` the first ``keep`` keys
+    stay visible beside it, forward only), ``chunk`` (a query sees no key
     from before the start of its chunk of that many positions; forward only), ``softcap``
     (scores become cap * tanh(score / cap)), ``sinks`` ([Hq] fp32 logits that join the softmax denominator only) and
     ``segments`` (int32 [B, S] ids of packed documents, non-decreasing along the sequence; 0 marks padding)."""
 
-    def __init__(self, window=None, softcap: float = 0.0, sinks=None, segments=None, chunk=None):
+    def __init__(self, window=None, softcap: float = 0.0, sinks=None, segments=None, chunk=None, keep: int = 0):
         self.window = int(window) if window else 0
         self.chunk = int(chunk) if chunk else 0
+        self.keep = int(keep) if window else 0
         self.softcap = float(softcap or 0.0)
         self.sinks = sinks.detach().to(torch.float32).contiguous() if sinks is not None else None
         self.segments = segments.to(torch.int32).contiguous() if segments is not None else None
@@ -43,7 +45,7 @@ def flash_fwd(q, k, v, causal: bool, scale: float, need_lse: bool = True, var: V
     lse = torch.empty((B, Hq, S), dtype=torch.float32, device=q.device) if need_lse else None
     rc = L.load().dewb_flash_fwd_var(L.ptr(q), L.ptr(k), L.ptr(v), L.ptr(out), L.ptr(lse), c_int(B), c_int(S), c_int(T),
                                      c_int(Hq), c_int(Hkv), c_int(D), *_strides(q), *_strides(k), *_strides(v),
-                                     *_strides(out), c_float(scale), c_int(int(causal)), c_int(var.window), c_int(var.chunk), c_float(var.softcap),
+                                     *_strides(out), c_float(scale), c_int(int(causal)), c_int(var.window), c_int(var.keep), c_int(var.chunk), c_float(var.softcap),
                                      L.ptr(var.sinks), L.ptr(var.segments), L.ptr(var.segments), L.ptr(L.status(q.device)),
                                      L.stream_ptr())
     L.check(rc, "flash_fwd")

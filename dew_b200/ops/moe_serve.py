@@ -14,12 +14,14 @@ from . import library as L
 
 c_ll, c_int, c_float = ctypes.c_longlong, ctypes.c_int, ctypes.c_float
 MAX_EXPERTS, MAX_TOP = 1024, 32
+SCORES = ("softmax", "sigmoid", "top_softmax")
 ROUTER_TOKENS = 512          # up to here the router's logits are formed token by token; past it, by a tensor-core product
 
 
 class Selection(NamedTuple):
     """How a router chooses: ``top`` of ``experts``; with ``groups`` > 1 only within the token's best ``keep`` groups (by the sum of their two
-    best choice scores), the others' choice scores becoming ``fill``; ``norm`` divides the weights by their sum."""
+    best choice scores), the others' choice scores becoming ``fill``; ``norm`` divides the weights by their sum.  ``score``: ``softmax`` or ``sigmoid``
+    of the logits, or ``top_softmax``: the choice runs on the logits, and the weights are the softmax over the chosen ones alone."""
     experts: int
     top: int
     groups: int = 1
@@ -44,6 +46,11 @@ def choice_scores(scores: torch.Tensor, bias: Optional[torch.Tensor], s: Selecti
 
 def select_reference(logits: torch.Tensor, bias: Optional[torch.Tensor], s: Selection) -> Tuple[torch.Tensor, torch.Tensor, torch.Tensor]:
     """fp32 ``logits [T, E]`` -> (weights ``[T, k]``, ids ``[T, k]``, scores ``[T, E]``)."""
+    if s.score not in SCORES:
+        raise ValueError(f"unknown router score {s.score!r}; known: {', '.join(SCORES)}")
+    if s.score == "top_softmax":
+        ids = torch.topk(choice_scores(logits, bias, s), s.top, dim=-1).indices
+        return torch.softmax(logits.gather(-1, ids), -1) * s.scaling, ids, torch.softmax(logits, -1)
     scores = torch.softmax(logits, -1) if s.score == "softmax" else torch.sigmoid(logits)
     ids = torch.topk(choice_scores(scores, bias, s), s.top, dim=-1).indices
     w = scores.gather(-1, ids)
@@ -79,16 +86,18 @@ class Routed(NamedTuple):
 
 
 def route(x2: torch.Tensor, weight: torch.Tensor, split: Optional[Split], bias: Optional[torch.Tensor], s: Selection,
-          positions: Optional[torch.Tensor] = None, kernel: Optional[str] = None) -> Routed:
-    """``x2 [T, d]``, the router's ``weight [E, d]`` (``split``: its bf16 rows, for a bf16 ``x2``).  ``kernel`` forces ``rows`` (logits token by
+          positions: Optional[torch.Tensor] = None, kernel: Optional[str] = None, logit_bias: Optional[torch.Tensor] = None) -> Routed:
+    """``x2 [T, d]``, the router's ``weight [E, d]`` (``split``: its bf16 rows, for a bf16 ``x2``), ``bias`` of the choice, ``logit_bias`` of the logits.  ``kernel`` forces ``rows`` (logits token by
     token) or ``product`` (a tensor-core product first)."""
     T, d = x2.shape
     E, k, dev = s.experts, s.top, x2.device
     out = Routed(torch.empty(T, k, dtype=torch.float32, device=dev), torch.empty(T, k, dtype=torch.int32, device=dev),
                  torch.empty(T, k, dtype=torch.int32, device=dev), torch.zeros(E, dtype=torch.int32, device=dev))
     x2, lib = x2.contiguous(), L.load()
-    b = None if bias is None else bias.detach().float().contiguous()
-    tail = (c_int(E), c_int(k), c_int(s.groups), c_int(s.keep), c_float(s.fill), c_int(int(s.score != "softmax")), c_int(int(s.norm)), c_float(s.scaling),
+    b, lb = (None if t is None else t.detach().float().contiguous() for t in (bias, logit_bias))
+    if positions is not None and positions.numel() != T:
+        raise ValueError(f"{positions.numel()} positions for {T} tokens")
+    tail = (c_int(E), c_int(k), c_int(s.groups), c_int(s.keep), c_float(s.fill), c_int(SCORES.index(s.score)), c_int(int(s.norm)), c_float(s.scaling),
             L.ptr(out.weights), L.ptr(out.ids), L.ptr(out.rank), L.ptr(out.counts))
     if (kernel or ("product" if T > ROUTER_TOKENS and x2.dtype == torch.bfloat16 and split is not None and d % 8 == 0 else "rows")) == "product":
         from .functional import gemm
@@ -96,13 +105,13 @@ def route(x2: torch.Tensor, weight: torch.Tensor, split: Optional[Split], bias: 
         ld = (n + 7) // 8 * 8
         logits = torch.empty(T, ld, dtype=torch.float32, device=dev)
         gemm(x2, split.rows, out=logits[:, :n], kernel="sm100_tcgen05")
-        L.check(lib.dewb_moe_select(L.ptr(logits), c_ll(ld), c_int(0 if split.exact else n - E), L.ptr(b), L.ptr(positions), c_int(T), *tail, L.stream_ptr()),
+        L.check(lib.dewb_moe_select(L.ptr(logits), c_ll(ld), c_int(0 if split.exact else n - E), L.ptr(b), L.ptr(lb), L.ptr(positions), c_int(T), *tail, L.stream_ptr()),
                 "moe_select")
         L.count_launches()
         return out
     w = split.rows if split is not None and split.exact and x2.dtype == torch.bfloat16 else weight.detach().float()
     w = w.contiguous()
-    L.check(lib.dewb_moe_router(L.ptr(x2), L.ptr(w), L.ptr(b), L.ptr(positions), c_int(T), c_int(d), *tail, c_int(int(x2.dtype == torch.float32)),
+    L.check(lib.dewb_moe_router(L.ptr(x2), L.ptr(w), L.ptr(b), L.ptr(lb), L.ptr(positions), c_int(T), c_int(d), *tail, c_int(int(x2.dtype == torch.float32)),
                                 c_int(int(w.dtype == torch.float32)), L.stream_ptr()), "moe_router")
     L.count_launches()
     return out

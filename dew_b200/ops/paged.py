@@ -1,5 +1,6 @@
 """Attention of a call's tokens against a paged cache of any head widths (``csrc/kernels/paged_attention.cu``), the projection epilogue in
-front of it (bias, norm over all heads or per head, query temperature, append) and the head gate behind it, each with its plain PyTorch form."""
+front of it (bias, norm over all heads or per head, rotation, query temperature, append) and the head gate behind it, each with its plain PyTorch
+form."""
 from __future__ import annotations
 
 import ctypes
@@ -9,6 +10,7 @@ from typing import Iterator, NamedTuple, Optional
 import torch
 
 from . import library as L
+from . import rotary as rotary_ops
 
 c_ll, c_int, c_float = ctypes.c_longlong, ctypes.c_int, ctypes.c_float
 
@@ -40,10 +42,14 @@ class Heads:
 
 
 class Visible(NamedTuple):
-    """What a layer's attention adds to the causal softmax: a query sees no key from before the start of its ``chunk`` of positions; ``sinks``
-    (fp32, one per query head) join the denominator only."""
+    """What a layer's attention adds to the causal softmax: a query sees no key from before the start of its ``chunk`` of positions; with a ``window``
+    it sees that many keys (its own included) and the row's first ``keep``; scores become ``softcap tanh(score / softcap)``; ``sinks`` (fp32, one per
+    query head) join the denominator only."""
     chunk: Optional[int] = None
     sinks: Optional[torch.Tensor] = None
+    window: Optional[int] = None
+    keep: int = 0
+    softcap: float = 0.0
 
 
 PLAIN = Visible()
@@ -56,6 +62,12 @@ class Pages(NamedTuple):
     table: torch.Tensor                   # [store rows, max_pages] int32
     page_size: int
     row_ids: Optional[torch.Tensor]       # int32 store row of each call row (None: the same)
+
+
+class Turned(NamedTuple):
+    """A call's rotation of the query and key heads: ``table`` of ``rotary.angles``."""
+    rot: rotary_ops.Rotary
+    table: torch.Tensor
 
 
 def query_temperature(positions: torch.Tensor, coef: float, every: int) -> torch.Tensor:
@@ -75,15 +87,18 @@ def per_head(heads: Heads, qw, kw) -> bool:
     return (qw is not None and qw.numel() != heads.q * heads.dk) or (kw is not None and kw.numel() != heads.kv * heads.dk)
 
 
-def prepare_reference(qkv, heads: Heads, qw, kw, eps: float, temperature, positions, bias=None):
-    """``q [R, S, H, dk]``, ``k [R, S, G, dk]``, ``v [R, S, G, dv]`` after the bias, the norms and the temperature, in the projection's dtype (keys and
-    values None for a layer without its own)."""
+def prepare_reference(qkv, heads: Heads, qw, kw, eps: float, temperature, positions, bias=None, turned: Optional[Turned] = None, unit: bool = False):
+    """``q [R, S, H, dk]``, ``k [R, S, G, dk]``, ``v [R, S, G, dv]`` after the bias, the norms, the rotation, (with ``unit``) the division of every head by
+    its root mean square, and the temperature, in the projection's dtype (keys and values None for a layer without its own)."""
     R, S, _ = qkv.shape
     one = per_head(heads, qw, kw)
 
     def norm(t, n, w):
         t = t.reshape(R, S, n, heads.dk) if one else t
-        return rms_norm_fp32(t, w, eps).reshape(R, S, n, heads.dk)
+        t = rms_norm_fp32(t, w, eps).reshape(R, S, n, heads.dk)
+        if turned is not None:
+            t = rotary_ops.turn(t, turned.table, turned.rot)
+        return t if not unit else t / torch.sqrt(t.pow(2).mean(-1, keepdim=True) + eps)
     x = qkv[..., :heads.packed]
     x = x if bias is None else x.float() + bias.float()
     q = norm(x[..., :heads.q * heads.dk], heads.q, qw)
@@ -102,8 +117,9 @@ def _slots(pages: Pages, positions: torch.Tensor) -> torch.Tensor:
     return pages.table[rows[:, None], p // pages.page_size].long() * pages.page_size + p % pages.page_size
 
 
-def qk_norm_append(qkv, heads: Heads, qw, kw, eps: float, temperature, positions, pages: Pages, bias=None) -> torch.Tensor:
-    """-> ``[R, S, H + 2 G, D]`` (normalised queries and keys, values; every head padded with zeros to the pool's width), with the keys and
+def qk_norm_append(qkv, heads: Heads, qw, kw, eps: float, temperature, positions, pages: Pages, bias=None, turned: Optional[Turned] = None,
+                   unit: bool = False) -> torch.Tensor:
+    """-> ``[R, S, H + 2 G, D]`` (queries and keys after ``prepare_reference``'s steps, values; every head padded with zeros to the pool's width), with the keys and
     values of the live positions written to the pools; ``[R, S, H, D]`` and nothing written for a layer without its own keys and values.
     ``positions`` int32 ``[R, S]``, below 0 = padding."""
     R, S, _ = qkv.shape
@@ -111,13 +127,18 @@ def qk_norm_append(qkv, heads: Heads, qw, kw, eps: float, temperature, positions
     if L.use_cuda(qkv):
         qkv = qkv.contiguous()
         qw, kw, bias = (None if w is None else w.detach().to(qkv.dtype).contiguous() for w in (qw, kw, bias))
-        if per_head(heads, qw, kw) or bias is not None or not heads.own or heads.gated:
+        if per_head(heads, qw, kw) or bias is not None or not heads.own or heads.gated or turned is not None or unit:
             if temperature is not None or not (per_head(heads, qw, kw) or qw is None or heads.q == heads.kv == 1):
-                raise NotImplementedError("a projection with a bias, gates or queries alone is built for norms per head and without a query temperature")
+                raise NotImplementedError("a projection with a bias, gates, a rotation or queries alone is built for norms per head and without a query "
+                                          "temperature")
+            if unit and (qw is not None or kw is not None):
+                raise NotImplementedError("heads pass one norm: with a weight in front of the rotation, or without one behind it")
+            rot, table = (None, None) if turned is None else turned
             G = heads.kv if heads.own else 0
             packed = torch.empty(R, S, heads.q + 2 * G, D, dtype=qkv.dtype, device=qkv.device)
-            L.check(L.load().dewb_head_norm_append(L.ptr(qkv), c_ll(qkv.shape[-1]), L.ptr(bias), L.ptr(qw), L.ptr(kw), c_float(eps), L.ptr(positions), c_int(R),
-                                                   c_int(S), c_int(heads.q), c_int(G), c_int(heads.dk), c_int(heads.dv), c_int(D), L.ptr(packed),
+            L.check(L.load().dewb_head_norm_append(L.ptr(qkv), c_ll(qkv.shape[-1]), L.ptr(bias), L.ptr(qw), L.ptr(kw), c_float(eps), c_int(int(unit)),
+                                                   L.ptr(table), c_int(0 if rot is None else rot.dims), c_int(int(rot is not None and rot.interleaved)),
+                                                   L.ptr(positions), c_int(R), c_int(S), c_int(heads.q), c_int(G), c_int(heads.dk), c_int(heads.dv), c_int(D), L.ptr(packed),
                                                    L.ptr(pages.k), L.ptr(pages.v), L.ptr(pages.table), c_int(pages.page_size), c_int(pages.table.shape[1]),
                                                    L.ptr(pages.row_ids), c_int(int(qkv.dtype == torch.float32)), L.stream_ptr()), "head_norm_append")
             L.count_launches()
@@ -130,7 +151,7 @@ def qk_norm_append(qkv, heads: Heads, qw, kw, eps: float, temperature, positions
                                              L.ptr(pages.row_ids), c_int(int(qkv.dtype == torch.float32)), L.stream_ptr()), "qk_norm_append")
         L.count_launches()
         return packed
-    q, k, v = prepare_reference(qkv, heads, qw, kw, eps, temperature, positions, bias)
+    q, k, v = prepare_reference(qkv, heads, qw, kw, eps, temperature, positions, bias, turned, unit)
     pad = lambda t: torch.nn.functional.pad(t, (0, D - t.shape[-1]))
     if not heads.own:
         return pad(q)
@@ -141,11 +162,15 @@ def qk_norm_append(qkv, heads: Heads, qw, kw, eps: float, temperature, positions
     return torch.cat([q, k, v], 2)
 
 
-def seen_keys(positions: torch.Tensor, n: int, chunk: Optional[int]) -> torch.Tensor:
+def seen_keys(positions: torch.Tensor, n: int, visible: Visible = PLAIN) -> torch.Tensor:
     """``[R, S, n]``: which of the first ``n`` positions a query at ``positions [R, S]`` sees."""
     j = torch.arange(n, device=positions.device)[None, None]
     seen = j <= positions[..., None]
-    return seen if not chunk else seen & (j >= (positions.clamp_min(0) // chunk * chunk)[..., None])
+    if visible.chunk:
+        seen = seen & (j >= (positions.clamp_min(0) // visible.chunk * visible.chunk)[..., None])
+    if visible.window:
+        seen = seen & ((j > positions[..., None] - visible.window) | (j < visible.keep))
+    return seen
 
 
 def softmax_with_sinks(s: torch.Tensor, sinks: Optional[torch.Tensor]) -> torch.Tensor:
@@ -165,11 +190,12 @@ def paged_attend_reference(q, heads: Heads, positions, pages: Pages, scale: floa
     slots = _slots(pages, torch.arange(n, device=q.device)[None].expand(R, n))
     kc = pages.k.view(-1, heads.kv, D)[slots].float().repeat_interleave(heads.q // heads.kv, 2)          # [R, n, H, D]
     vc = pages.v.view(-1, heads.kv, D)[slots][..., :heads.dv].float().repeat_interleave(heads.q // heads.kv, 2)
-    seen = seen_keys(positions, n, visible.chunk)                                                        # [R, S, n]
+    seen = seen_keys(positions, n, visible)                                                              # [R, S, n]
     # what the pool holds beyond a row's own tokens is another row's, or nothing: it must not reach the sums
     own = (torch.arange(n, device=q.device)[None] <= positions.amax(1, keepdim=True))[..., None, None]
     kc, vc = torch.where(own, kc, torch.zeros_like(kc)), torch.where(own, vc, torch.zeros_like(vc))
     s = torch.einsum("rshd,rnhd->rhsn", q[..., :D].float(), kc) * scale
+    s = s if not visible.softcap else visible.softcap * torch.tanh(s / visible.softcap)
     p = softmax_with_sinks(s.masked_fill(~seen[:, None], float("-inf")), visible.sinks)
     return torch.einsum("rhsn,rnhd->rshd", p, vc).to(q.dtype)
 
@@ -207,7 +233,7 @@ def paged_attend(q: torch.Tensor, heads: Heads, positions: torch.Tensor, pages: 
     out = torch.empty(R, S, H, heads.dv, dtype=q.dtype, device=q.device)
     if gate is not None and (gate.stride(2) != 1 or (R > 1 and gate.stride(0) != S * gate.stride(1))):
         gate = gate.contiguous()
-    extras = (c_int(visible.chunk or 0), L.ptr(visible.sinks), L.ptr(gate), c_ll(0 if gate is None else gate.stride(1)))
+    extras = (c_int(visible.chunk or 0), c_int(visible.window or 0), c_int(visible.keep), c_float(visible.softcap), L.ptr(visible.sinks), L.ptr(gate), c_ll(0 if gate is None else gate.stride(1)))
     if (kernel or ("mma" if q.dtype == torch.bfloat16 and D in (64, 128, 256) else "general")) == "mma":
         L.check(L.load().dewb_paged_attend_mma(L.ptr(q), c_ll(q.stride(1)), L.ptr(pages.k), L.ptr(pages.v), L.ptr(positions), c_int(R), c_int(S), c_int(H),
                                                c_int(heads.kv), c_int(heads.dv), c_int(D), c_float(scale), *extras, L.ptr(out), L.ptr(pages.table),

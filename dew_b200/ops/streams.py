@@ -19,14 +19,18 @@ MAX_STREAMS = 16
 
 
 class Write(NamedTuple):
-    """A sub-layer's output on its way into the streams: ``H'[t] = sum_s mix[s, t] H[s] + out[t] * (scale * y)``.  Without ``mix`` and ``out``
-    every stream keeps itself and takes ``y``; with ``weight``, ``y`` passes an RMS norm (``weight``, ``eps``) first."""
+    """A sub-layer's output on its way into the streams: ``H'[t] = sum_s mix[s, t] H[s] + out[t] * gain * (scale * y + scale2 * y2)``.  Without ``mix``
+    and ``out`` every stream keeps itself and takes ``y``; with ``weight``, ``y`` passes an RMS norm (``weight``, ``eps``) first; ``y2`` is the second
+    of two sub-layers that join together."""
     y: torch.Tensor
     scale: Optional[torch.Tensor] = None
     mix: Optional[torch.Tensor] = None
     out: Optional[torch.Tensor] = None
     weight: Optional[torch.Tensor] = None
     eps: float = 0.0
+    y2: Optional[torch.Tensor] = None
+    scale2: Optional[torch.Tensor] = None
+    gain: float = 1.0
 
 
 def _kernel_ok(x: torch.Tensor, *others) -> bool:
@@ -46,8 +50,9 @@ def layer_norm_reference(x: torch.Tensor, w: torch.Tensor, eps: float) -> torch.
     return dev / torch.sqrt(dev.pow(2).mean(-1, keepdim=True) + eps) * w.float()
 
 
-def embed_streams(tokens: torch.Tensor, positions: Optional[torch.Tensor], embed: torch.Tensor, pos: Optional[torch.Tensor], n: int) -> torch.Tensor:
-    """``[B, S]`` tokens (and positions, below 0 = padding) -> fp32 streams ``[B, S, n, d]``, all equal to the embedding plus the learned
+def embed_streams(tokens: torch.Tensor, positions: Optional[torch.Tensor], embed: torch.Tensor, pos: Optional[torch.Tensor], n: int,
+                  gain: float = 1.0) -> torch.Tensor:
+    """``[B, S]`` tokens (and positions, below 0 = padding) -> fp32 streams ``[B, S, n, d]``, all equal to ``gain`` times the embedding plus the learned
     position vector."""
     B, S = tokens.shape
     d = embed.shape[1]
@@ -59,51 +64,57 @@ def embed_streams(tokens: torch.Tensor, positions: Optional[torch.Tensor], embed
         p32 = None if pos is None else positions.to(torch.int32).contiguous()
         e, p = embed.detach().contiguous(), _as(pos, embed.dtype)
         L.check(L.load().dewb_embed_streams(L.ptr(tk), L.ptr(p32), L.ptr(e), L.ptr(p), L.ptr(H), c_ll(B * S), c_int(n), c_int(d), c_int(embed.shape[0]),
-                                            c_int(0 if pos is None else pos.shape[0]), c_int(int(embed.dtype == torch.float32)), L.stream_ptr()), "embed_streams")
+                                            c_int(0 if pos is None else pos.shape[0]), c_float(gain), c_int(int(embed.dtype == torch.float32)), L.stream_ptr()), "embed_streams")
         L.count_launches()
         return H
-    x = F.embedding(tokens, embed).float()
+    x = F.embedding(tokens, embed).float() * gain
     if pos is not None:
         x = x + F.embedding(positions.long().clamp_min(0), pos).float()
     return x.unsqueeze(2).expand(B, S, n, d).contiguous()
 
 
-def stream_step_reference(H, write: Optional[Write], read, weight, eps: float, dtype, norm: str = "layer"):
+def stream_step_reference(H, write: Optional[Write], read, weight, eps: float, dtype, norm: str = "layer", around: float = 0.0):
     if write is not None:
         y = write.y.float()
         if write.weight is not None:
             y = y / torch.sqrt(y.pow(2).mean(-1, keepdim=True) + write.eps) * write.weight.float()
         if write.scale is not None:
             y = y * write.scale.float()
+        if write.y2 is not None:
+            y = y + (write.y2.float() if write.scale2 is None else write.y2.float() * write.scale2.float())
+        y = y * write.gain
         kept = H if write.mix is None else torch.einsum("st,...sd->...td", write.mix.float(), H)
         H = kept + (y.unsqueeze(-2) if write.out is None else write.out.float()[:, None] * y.unsqueeze(-2))
     if weight is None:
         return None, H
     u = H.sum(-2) if read is None else torch.einsum("s,...sd->...d", read.float(), H)
+    weight = weight.float() + around
     if norm == "layer":
         return layer_norm_reference(u, weight, eps).to(dtype), H
     return (u / torch.sqrt(u.pow(2).mean(-1, keepdim=True) + eps) * weight.float()).to(dtype), H
 
 
 def stream_step(H: torch.Tensor, write: Optional[Write], read: Optional[torch.Tensor], weight: Optional[torch.Tensor], eps: float, dtype,
-                norm: str = "layer") -> Tuple[Optional[torch.Tensor], torch.Tensor]:
-    """``(norm(sum_s read[s] H'[s]) * weight, H')`` with ``H'`` the streams after ``write`` (None: as they are); ``read`` None: all ones.  ``H [..., n, d]`` fp32;
+                norm: str = "layer", around: float = 0.0) -> Tuple[Optional[torch.Tensor], torch.Tensor]:
+    """``(norm(sum_s read[s] H'[s]) * (around + weight), H')`` with ``H'`` the streams after ``write`` (None: as they are); ``read`` None: all ones.  ``H [..., n, d]`` fp32;
     on a GPU outside autograd ``H`` is updated in place.  ``weight`` None: the write alone."""
     if norm not in ("layer", "rms"):
         raise ValueError(f"unknown norm {norm!r}; known: layer, rms")
     n, d = H.shape[-2:]
-    tensors = (weight, read) + (() if write is None else (write.y, write.scale, write.mix, write.out, write.weight))
+    tensors = (weight, read) + (() if write is None else (write.y, write.scale, write.mix, write.out, write.weight, write.y2, write.scale2))
     if n > MAX_STREAMS or not H.is_contiguous() or not _kernel_ok(H, *tensors) or dtype not in (torch.bfloat16, torch.float32):
-        return stream_step_reference(H, write, read, weight, eps, dtype, norm)
+        return stream_step_reference(H, write, read, weight, eps, dtype, norm, around)
     rows = H.numel() // (n * d)
     normed = None if weight is None else torch.empty(*H.shape[:-2], d, dtype=dtype, device=H.device)
-    y = y_weight = scale = mix = out = None
+    y = y_weight = scale = mix = out = y2 = scale2 = None
     if write is not None:
         y, scale, mix, out = _as(write.y, dtype), _as(write.scale, dtype), _as(write.mix, torch.float32), _as(write.out, torch.float32)
-        y_weight = _as(write.weight, dtype)
+        y_weight, y2, scale2 = _as(write.weight, dtype), _as(write.y2, dtype), _as(write.scale2, dtype)
     r, w = _as(read, torch.float32), _as(weight, dtype)
     L.check(L.load().dewb_stream_step(L.ptr(H), L.ptr(y), L.ptr(y_weight), L.ptr(scale), L.ptr(mix), L.ptr(out), L.ptr(r), L.ptr(w), L.ptr(normed), c_ll(rows),
-                                      c_int(n), c_int(d), c_float(0.0 if write is None else write.eps), c_float(eps), c_int(int(norm == "rms")), c_int(int(dtype == torch.float32)), L.stream_ptr()), "stream_step")
+                                      c_int(n), c_int(d), c_float(0.0 if write is None else write.eps), c_float(eps), c_int(int(norm == "rms")),
+                                      L.ptr(y2), L.ptr(scale2), c_float(1.0 if write is None else write.gain), c_float(around),
+                                      c_int(int(dtype == torch.float32)), L.stream_ptr()), "stream_step")
     L.count_launches()
     return normed, H
 
@@ -123,6 +134,24 @@ def clamped_glu(gu: torch.Tensor, limit: float, alpha: float = 1.702) -> torch.T
     out = torch.empty(*gu.shape[:-1], Fh, dtype=gu.dtype, device=gu.device)
     L.check(L.load().dewb_clamped_glu(L.ptr(gu), L.ptr(out), c_ll(gu.numel() // (2 * Fh)), c_int(Fh), c_float(limit), c_float(alpha),
                                       c_int(int(gu.dtype == torch.float32)), L.stream_ptr()), "clamped_glu")
+    L.count_launches()
+    return out
+
+
+def gelu_glu_reference(gu: torch.Tensor) -> torch.Tensor:
+    g, u = gu.chunk(2, -1)
+    return F.gelu(g, approximate="tanh") * u
+
+
+def gelu_glu(gu: torch.Tensor) -> torch.Tensor:
+    """``[..., 2F]`` (gate half, then linear half) -> ``[..., F]``: ``gelu(gate) * up``, the tanh form."""
+    if not _kernel_ok(gu):
+        return gelu_glu_reference(gu)
+    gu = gu.contiguous()
+    Fh = gu.shape[-1] // 2
+    out = torch.empty(*gu.shape[:-1], Fh, dtype=gu.dtype, device=gu.device)
+    L.check(L.load().dewb_gelu_glu(L.ptr(gu), L.ptr(out), c_ll(gu.numel() // (2 * Fh)), c_int(Fh), c_int(int(gu.dtype == torch.float32)), L.stream_ptr()),
+            "gelu_glu")
     L.count_launches()
     return out
 

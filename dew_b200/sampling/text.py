@@ -177,10 +177,12 @@ class RowBatch:
             named = variables_for_call(model, params)
             self.call = lambda t, **kw: torch.func.functional_call(model, named, (t,), kw)
 
-    def forward(self, ids: torch.Tensor, positions: torch.Tensor, span: Optional[Tuple[int, int]] = None, pick: Optional[torch.Tensor] = None):
+    def forward(self, ids: torch.Tensor, positions: torch.Tensor, span: Optional[Tuple[int, int]] = None, pick: Optional[torch.Tensor] = None,
+                together: bool = True):
         """``ids, positions [rows, S]`` (positions below 0 = padding at a row's end) -> logits ``[n, V]`` at ``pick = (rows, places)`` or of
-        every position.  ``span``: where the tokens lie in every row, when the caller knows (saves the cache a device read)."""
-        self.store.chunk_span = span
+        every position.  ``span``: where the tokens lie in every row, when the caller knows (saves the cache a device read); ``together``: whether
+        every row starts at its first."""
+        self.store.chunk_span, self.store.together = span, together
         try:
             with torch.no_grad():
                 if self.splits_head:                         # the head runs on the picked positions alone
@@ -191,7 +193,7 @@ class RowBatch:
                 logits = self.call(ids, positions=positions, cache=self.store)
                 return logits if pick is None else logits[pick]
         finally:
-            self.store.chunk_span = None
+            self.store.chunk_span, self.store.together = None, True
 
     def prefill(self, tokens: torch.Tensor, lengths: torch.Tensor) -> torch.Tensor:
         """The prompts ``[rows, S]`` (right-padded), from their first token; returns last-position logits ``[rows, V]``."""
@@ -230,12 +232,13 @@ class RowBatch:
                 if added:
                     self.store.page_table[r, have:have + len(added)] = torch.tensor(added, dtype=torch.int32, device=self.device)
         live = {starts[r] for r, p in enumerate(pieces) if len(p)}
-        span = (live.pop(), max(starts[r] + len(p) for r, p in enumerate(pieces))) if len(live) == 1 else None
+        together = len(live) == 1
+        span = (live.pop(), max(starts[r] + len(p) for r, p in enumerate(pieces))) if together else None
         if span is None and self.store.slots is not None:
             span = (1, max(starts[r] + len(p) for r, p in enumerate(pieces)))     # rows at different places: not a fresh prompt
         wanted = [(r, w) for r, ws in enumerate(want or ()) for w in ws]
         pick = tuple(torch.tensor([x[j] for x in wanted], dtype=torch.long, device=self.device) for j in range(2))
-        out = self.forward(ids.to(self.device), pos.to(self.device), span, pick)
+        out = self.forward(ids.to(self.device), pos.to(self.device), span, pick, together)
         self.lengths = [n + len(p) for n, p in zip(starts, pieces)]
         return out if wanted else None
 
