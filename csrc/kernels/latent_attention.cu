@@ -1,5 +1,5 @@
-// Latent attention in generation, for sm_100a: a token leaves one row [latent | rotated key part] for all heads, in pages W values wide (rank + rot
-// padded with zeros to a multiple of 16).
+// Latent attention in generation, for sm_100a: a token leaves one row [latent | rotated key part] for all heads, in pages W values wide: rank + rot
+// padded with zeros to a multiple of 16, and 8 more, so that rows copied to shared memory as they lie start on different banks.
 //
 //   latent_rows      from the input projection [tokens, query latent | latent | key part | ...]: RMS norm of the query latent and of the latent, the
 //                    rotation of the key part (by the call's table of cosines and sines), and the append of the row to its page
@@ -8,7 +8,7 @@
 //                    them) and latents out of it, times the sigmoid of a gate.  bf16 on the tensor cores (mma.sync: a decode step has too few rows for
 //                    tcgen05), fp32 and ragged sizes on the CUDA cores
 //   latent_attend    causal attention of a call's tokens against the rows' latents (decode steps, mixed positions): 16 or 32 rows of work (token,
-//                    head) a CTA, tiles of 32 latents through a cp.async ring, each read once for scores and values, keys split over CTAs
+//                    head) a CTA, tiles of 32 latents through a ring of bulk copies, each read once for scores and values, keys split over CTAs
 //   latent_combine   merges the splits
 //   latent_gather    pages -> dense latents and key parts of every row (a prompt's later portions, whose keys are formed in full width)
 //
@@ -20,6 +20,7 @@
 #include <cuda_runtime.h>
 
 #include "../common/mma_bf16.cuh"
+#include "../common/ptx.cuh"
 #include "../common/rows.cuh"
 
 namespace dewb {
@@ -130,27 +131,32 @@ struct HeadProduct {
   int tokens, H, N, K;
   const float2* table;             // not null: columns [N, N + pad) of out are the rotated columns [K, K + rot) of a, then zeros
   int rot, pad, dims, interleaved;
+  int pairs;                       // columns of out and gate can be moved in pairs
 };
 
+// Part `part` of the tail: TAIL columns of up to 64 rows
+constexpr int TAIL = 16;
+
 template <typename T>
-__device__ __forceinline__ void tail_columns(const HeadProduct<T>& p, int t0, int rows, int h, int threads) {
-  for (int i = threadIdx.x; i < rows * p.pad; i += threads) {
-    const int r = i / p.pad, j = i - r * p.pad;
+__device__ __forceinline__ void tail_columns(const HeadProduct<T>& p, int t0, int part, int h, int threads) {
+  const int c0 = part * TAIL, n = min(TAIL, p.pad - c0), end = min(64, p.tokens - t0) * n;
+#pragma unroll 4
+  for (int i = threadIdx.x; i < end; i += threads) {
+    const int r = i / n, j = c0 + i - r * n;
     const long long t = t0 + r;
-    if (t >= p.tokens) break;
     const float v = j < p.rot ? turned(p.a + t * p.a_token + h * p.a_head + p.K, j, p.table + t * (p.dims / 2), p.dims, p.interleaved) : 0.f;
     st(p.out + t * p.out_token + h * p.out_head + p.N + j, v);
   }
 }
 
-// grid (ceil(N / 64) (+ 1 with a table), ceil(tokens / 64), H)
+// grid (ceil(N / 64) (+ ceil(pad / TAIL) with a table), ceil(tokens / 64), H)
 template <typename T, bool TRANS>
 __global__ void __launch_bounds__(256)
 head_product_kernel(HeadProduct<T> p) {
   constexpr int M = 64, NT = 64, KT = 16;
   __shared__ __align__(16) float sa[KT][M + 4], sw[KT][NT + 4];
   const int t0 = blockIdx.y * M, n0 = blockIdx.x * NT, h = blockIdx.z;
-  if (n0 >= p.N) { tail_columns(p, t0, M, h, 256); return; }
+  if (n0 >= p.N) { tail_columns(p, t0, blockIdx.x - (p.N + NT - 1) / NT, h, 256); return; }
   const int tx = threadIdx.x & 15, ty = threadIdx.x >> 4;
   float acc[4][4] = {};
   for (int k0 = 0; k0 < p.K; k0 += KT) {
@@ -208,7 +214,7 @@ head_product_mma_kernel(HeadProduct<bf16> p) {
   extern __shared__ __align__(16) uint8_t raw[];
   bf16* ring = reinterpret_cast<bf16*>(raw);
   const int t0 = blockIdx.y * 64, n0 = blockIdx.x * 64, h = blockIdx.z;
-  if (n0 >= p.N) { tail_columns(p, t0, 64, h, 128); return; }
+  if (n0 >= p.N) { tail_columns(p, t0, blockIdx.x - (p.N + 63) / 64, h, 128); return; }
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
   const int steps = (p.K + 63) / 64;
   auto fetch = [&](int s) {
@@ -256,6 +262,22 @@ head_product_mma_kernel(HeadProduct<bf16> p) {
   for (int e = 0; e < 2; ++e) {
     const long long t = t0 + warp * 16 + lg + 8 * e;
     if (t >= p.tokens) continue;
+    if (p.pairs) {                                     // pairs of columns; every gate is under way before the first is used
+      uint32_t z[8];
+#pragma unroll
+      for (int j = 0; j < 8; ++j) {
+        const int n = n0 + j * 8 + t2;
+        z[j] = p.gate != nullptr && n < p.N ? *reinterpret_cast<const uint32_t*>(p.gate + t * p.gate_token + static_cast<long long>(h) * p.N + n) : 0u;
+      }
+#pragma unroll
+      for (int j = 0; j < 8; ++j) {
+        const int n = n0 + j * 8 + t2;
+        float a = acc[j][2 * e], b = acc[j][2 * e + 1];
+        if (p.gate != nullptr) { a *= sigmoid(lo_f(z[j])); b *= sigmoid(hi_f(z[j])); }
+        if (n < p.N) *reinterpret_cast<uint32_t*>(p.out + t * p.out_token + h * p.out_head + n) = pack2(a, b);
+      }
+      continue;
+    }
 #pragma unroll
     for (int j = 0; j < 8; ++j)
 #pragma unroll
@@ -269,9 +291,13 @@ head_product_mma_kernel(HeadProduct<bf16> p) {
   }
 }
 
-// ---- attention against the latents.  Eight warps: for the scores a warp takes a quarter of the W columns and half of the tile's keys (partial scores
-// meet in shared memory), for the values a slice of NV * 8 latent columns.  KS: 16-column steps of a quarter; MT: tiles of 16 rows of work.
-constexpr int TK = 32, A_THREADS = 256, SST = TK + 4, PPT = TK + 8;
+// ---- attention against the latents: 17 warps.  Warp 16 brings tiles of 32 rows into a ring, one bulk copy a tile (a row, where pages do not hold whole
+// tiles).  Warps 0..7 form scores - a warp takes
+// a quarter of the W columns and half of the tile's keys, the partial scores meet in shared memory - and the online softmax.  Warps 8..15 keep the sums,
+// NV * 8 latent columns each, and free the stage.  Scores of one tile and values of the one before run at the same time.  KS: 16-column steps of a
+// quarter; MT: tiles of 16 rows of work (token, head).
+constexpr int TK = 32, GROUP = 256, A_THREADS = 2 * GROUP + 32, SST = TK + 8, PPT = TK + 8;
+constexpr uint32_t FULL = 0xffffffffu;
 
 struct Attend {
   const bf16* q;                   // [R * S, H, W]
@@ -281,153 +307,214 @@ struct Attend {
   float *part_m, *part_l, *part_acc;      // [R * S * H, splits] (log2 domain) and [..., rank]
   int S, H, W, rank, splits;
   float scale_log2;
+  int* err;
 };
 
 template <int MT>
-constexpr int attend_stages() { return MT == 1 ? 2 : 4; }
+constexpr int attend_stages() { return MT == 1 ? 5 : 4; }
+
+template <int STAGES>
+struct AttendBars {
+  uint64_t k_full[STAGES], k_empty[STAGES], p_full[2], p_empty[2];
+  int abort_flag, poisoned;
+};
 
 template <int KS, int NV, int MT>
-__global__ void __launch_bounds__(A_THREADS, MT == 1 ? 2 : 1)
+__global__ void __launch_bounds__(A_THREADS, 1)
 latent_attend_kernel(Attend p, Pool pages) {
-  constexpr int STAGES = attend_stages<MT>(), M = 16 * MT, TPR = A_THREADS / M, KPT = TK / TPR;
+  constexpr int STAGES = attend_stages<MT>(), M = 16 * MT, TPR = GROUP / M, KPT = TK / TPR;
   extern __shared__ __align__(16) uint8_t raw[];
-  const int ST = p.W + 8;
-  bf16* sk = reinterpret_cast<bf16*>(raw);                       // [STAGES][TK][ST]
-  float* ss = reinterpret_cast<float*>(sk + STAGES * TK * ST);   // [4][M][SST]
-  bf16* sp = reinterpret_cast<bf16*>(ss + 4 * M * SST);          // [M][PPT]
-  __shared__ float s_alpha[M], s_l[M], s_m[M];
+  const int ST = p.W;
+  bf16* sk = reinterpret_cast<bf16*>(raw);                       // [STAGES][TK][W]
+  float* ss = reinterpret_cast<float*>(sk + STAGES * TK * ST);   // [2][4][M][SST]
+  bf16* sp = reinterpret_cast<bf16*>(ss + 2 * 4 * M * SST);      // [2][M][PPT]
+  __shared__ AttendBars<STAGES> bars;
+  __shared__ float s_alpha[2][M], s_l[M], s_m[M];
   __shared__ int s_pos[M];
   const int row = blockIdx.y, split = blockIdx.z, w0 = blockIdx.x * M, work = p.S * p.H;
-  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, kq = warp & 3, kg = warp >> 2;
+  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+  if (tid == 0) {
+    bars.poisoned = *reinterpret_cast<volatile int*>(p.err);
+    bars.abort_flag = 0;
+    for (int i = 0; i < STAGES; ++i) { mbar_init(&bars.k_full[i], 1); mbar_init(&bars.k_empty[i], 8); }
+    for (int i = 0; i < 2; ++i) { mbar_init(&bars.p_full[i], 8); mbar_init(&bars.p_empty[i], 8); }
+    fence_barrier_init();
+    fence_proxy_async();
+  }
   if (tid < M) s_pos[tid] = w0 + tid < work ? p.positions[static_cast<long long>(row) * p.S + (w0 + tid) / p.H] : -1;
   __syncthreads();
+  if (bars.poisoned != 0) return;
+  volatile int* abort_flag = &bars.abort_flag;
   int last = -1;
   for (int i = 0; i < M; ++i) last = max(last, s_pos[i]);
   const int all = (last + TK) / TK, per = (all + p.splits - 1) / p.splits;
   const int begin = min(all, split * per), tiles = min(all, begin + per) - begin;
-  auto fetch = [&](int t) {
-    if (t < tiles) {
-      const int key0 = (begin + t) * TK + warp * 4;
-      long long mine = 0;
-      if (lane < 4 && key0 + lane <= last) mine = pool_token(pages, row, key0 + lane);
-      bf16* dst = sk + (t % STAGES) * TK * ST + warp * 4 * ST;
-#pragma unroll
-      for (int r = 0; r < 4; ++r) {
-        const long long tok = __shfl_sync(0xffffffffu, mine, r);
-        const bool live = key0 + r <= last;
-        const bf16* src = p.pool + tok * p.W;
-        for (int c = lane * 8; c < p.W; c += 256) cp16(smem_addr(dst + r * ST + c), live ? src + c : p.pool, live);
-      }
+  const int lg = lane >> 2, t2 = (lane & 3) * 2;
+  bool ok = true;
+  if (warp == 16) {
+    // ------------------------------------------------------------------ producer
+    // Tokens past the last one (a tile whole in a page brings them along, else the last is repeated) meet weights of zero.
+    const bool whole = pages.page_size % TK == 0;
+    auto source = [&](int t) { return pool_token(pages, row, whole ? (begin + t) * TK : min((begin + t) * TK + lane, last)); };
+    long long tok = tiles > 0 ? source(0) : 0;
+    int t = 0;
+    for (; t < tiles; ++t) {
+      const int st = t % STAGES;
+      if (!mbar_wait_warp(&bars.k_empty[st], ((t / STAGES) & 1) ^ 1, abort_flag)) { if (lane == 0) atomicCAS(p.err, 0, ERR_WAIT_EMPTY); break; }
+      if (lane == 0) mbar_expect_tx(&bars.k_full[st], TK * p.W * 2);
+      __syncwarp();
+      if (!whole) bulk_load_1d(sk + (st * TK + lane) * ST, p.pool + tok * p.W, p.W * 2, &bars.k_full[st]);
+      else if (lane == 0) bulk_load_1d(sk + st * TK * ST, p.pool + tok * p.W, TK * p.W * 2, &bars.k_full[st]);
+      if (t + 1 < tiles) tok = source(t + 1);          // the page's number is under way while the ring is full
     }
-    cp_commit();
-  };
-#pragma unroll
-  for (int t = 0; t < STAGES - 1; ++t) fetch(t);
-  // this warp's columns of the queries, as A operands
-  const int lg = lane >> 2, t2 = (lane & 3) * 2, steps = p.W / 16, first = kq * ((steps + 3) / 4), count = max(0, min((steps + 3) / 4, steps - first));
-  uint32_t qa[MT][KS][4];
-#pragma unroll
-  for (int m = 0; m < MT; ++m)
-#pragma unroll
-    for (int e = 0; e < 2; ++e) {
-      const int w = w0 + m * 16 + lg + 8 * e;
-      const bool live = w < work && s_pos[m * 16 + lg + 8 * e] >= 0;
-      const bf16* src = p.q + (static_cast<long long>(row) * work + w) * p.W;
-#pragma unroll
-      for (int k = 0; k < KS; ++k) {
-        qa[m][k][e] = live && k < count ? *reinterpret_cast<const uint32_t*>(src + (first + k) * 16 + t2) : 0u;
-        qa[m][k][2 + e] = live && k < count ? *reinterpret_cast<const uint32_t*>(src + (first + k) * 16 + 8 + t2) : 0u;
-      }
-    }
-  float o[MT][NV][4];
-#pragma unroll
-  for (int m = 0; m < MT; ++m)
-#pragma unroll
-    for (int n = 0; n < NV; ++n) { o[m][n][0] = o[m][n][1] = o[m][n][2] = o[m][n][3] = 0.f; }
-  const int srow = tid / TPR, skey = (tid % TPR) * KPT, my_pos = s_pos[srow];       // this thread's scores in the softmax
-  float m_run = -INFINITY, l_run = 0.f;
-  const int v0 = warp * NV * 8;
-  for (int t = 0; t < tiles; ++t) {
-    cp_wait<STAGES - 2>();
-    __syncthreads();
-    fetch(t + STAGES - 1);                           // into the stage whose values the last tile's products have read
-    const bf16* tile = sk + (t % STAGES) * TK * ST;
-    float s[MT][2][4];
+    if (t < tiles)                                     // gave up: the copies under way still land in this block's memory
+      for (int i = max(0, t - STAGES); i < t; ++i) mbar_wait_warp(&bars.k_full[i % STAGES], (i / STAGES) & 1, nullptr);
+  } else if (warp < 8) {
+    // ------------------------------------------------------------------ scores and softmax
+    const int kq = warp & 3, kg = warp >> 2, steps = (p.W - 8) / 16, quarter = (steps + 3) / 4, first = kq * quarter, count = max(0, min(quarter, steps - first));
+    uint32_t qa[MT][KS][4];                            // this warp's columns of the queries, as A operands
 #pragma unroll
     for (int m = 0; m < MT; ++m)
 #pragma unroll
-      for (int n = 0; n < 2; ++n) { s[m][n][0] = s[m][n][1] = s[m][n][2] = s[m][n][3] = 0.f; }
+      for (int e = 0; e < 2; ++e) {
+        const int w = w0 + m * 16 + lg + 8 * e;
+        const bool live = w < work && s_pos[m * 16 + lg + 8 * e] >= 0;
+        const bf16* src = p.q + (static_cast<long long>(row) * work + w) * p.W;
 #pragma unroll
-    for (int k = 0; k < KS; ++k)
-      if (k < count) {
-        uint32_t b[4];
-        ldsm4(b, smem_addr(tile + (kg * 16 + (lane & 7) + (lane >> 4) * 8) * ST + (first + k) * 16 + ((lane >> 3) & 1) * 8));
-#pragma unroll
-        for (int m = 0; m < MT; ++m) {
-          mma(s[m][0], qa[m][k], b[0], b[1]);
-          mma(s[m][1], qa[m][k], b[2], b[3]);
+        for (int k = 0; k < KS; ++k) {
+          qa[m][k][e] = live && k < count ? *reinterpret_cast<const uint32_t*>(src + (first + k) * 16 + t2) : 0u;
+          qa[m][k][2 + e] = live && k < count ? *reinterpret_cast<const uint32_t*>(src + (first + k) * 16 + 8 + t2) : 0u;
         }
       }
+    const int srow = tid / TPR, skey = (tid % TPR) * KPT, my_pos = s_pos[srow];       // this thread's scores in the softmax
+    const uint32_t kaddr = smem_addr(sk) + ((kg * 16 + (lane & 7) + (lane >> 4) * 8) * ST + first * 16 + ((lane >> 3) & 1) * 8) * 2;
+    float m_run = -INFINITY, l_run = 0.f;
+    for (int t = 0; t < tiles; ++t) {
+      const int st = t % STAGES, b = t & 1;
+      if (ok && !mbar_wait_warp(&bars.k_full[st], (t / STAGES) & 1, abort_flag)) { if (lane == 0) atomicCAS(p.err, 0, ERR_WAIT_FULL); ok = false; }
+      float* part = ss + b * 4 * M * SST;
+      if (ok) {
+        float s[MT][2][4];
 #pragma unroll
-    for (int m = 0; m < MT; ++m)
+        for (int m = 0; m < MT; ++m)
 #pragma unroll
-      for (int n = 0; n < 2; ++n) {
-        float* d = ss + (kq * M + m * 16 + lg) * SST + kg * 16 + n * 8 + t2;
-        *reinterpret_cast<float2*>(d) = make_float2(s[m][n][0], s[m][n][1]);
-        *reinterpret_cast<float2*>(d + 8 * SST) = make_float2(s[m][n][2], s[m][n][3]);
+          for (int n = 0; n < 2; ++n) { s[m][n][0] = s[m][n][1] = s[m][n][2] = s[m][n][3] = 0.f; }
+        const uint32_t at = kaddr + st * TK * ST * 2;
+#pragma unroll
+        for (int k = 0; k < KS; ++k)
+          if (k < count) {
+            uint32_t f[4];
+            ldsm4(f, at + k * 32);
+#pragma unroll
+            for (int m = 0; m < MT; ++m) {
+              mma(s[m][0], qa[m][k], f[0], f[1]);
+              mma(s[m][1], qa[m][k], f[2], f[3]);
+            }
+          }
+#pragma unroll
+        for (int m = 0; m < MT; ++m)
+#pragma unroll
+          for (int n = 0; n < 2; ++n) {
+            float* d = part + (kq * M + m * 16 + lg) * SST + kg * 16 + n * 8 + t2;
+            *reinterpret_cast<float2*>(d) = make_float2(s[m][n][0], s[m][n][1]);
+            *reinterpret_cast<float2*>(d + 8 * SST) = make_float2(s[m][n][2], s[m][n][3]);
+          }
       }
-    __syncthreads();
-    {
+      // the eight warps meet once a tile: the two buffers of partial scores take turns
+      asm volatile("bar.sync 1, 256;" ::: "memory");
+      if (ok && !mbar_wait_warp(&bars.p_empty[b], ((t >> 1) & 1) ^ 1, abort_flag)) { if (lane == 0) atomicCAS(p.err, 0, ERR_WAIT_OTHER); ok = false; }
+      if (!ok) continue;
       float v[KPT], mx = -INFINITY;
 #pragma unroll
+      for (int i = 0; i < KPT; ++i) v[i] = 0.f;
+#pragma unroll
+      for (int q = 0; q < 4; ++q)
+        {
+          float x[KPT];
+          const float* src = part + (q * M + srow) * SST + skey;
+          if constexpr (KPT == 4) load_v<4>(src, x);
+          else { const float2 y = *reinterpret_cast<const float2*>(src); x[0] = y.x; x[1] = y.y; }
+#pragma unroll
+          for (int i = 0; i < KPT; ++i) v[i] += x[i];
+        }
+#pragma unroll
       for (int i = 0; i < KPT; ++i) {
-        const int c = skey + i;
-        const float x = ss[srow * SST + c] + ss[(M + srow) * SST + c] + ss[(2 * M + srow) * SST + c] + ss[(3 * M + srow) * SST + c];
-        v[i] = (begin + t) * TK + c <= my_pos ? x * p.scale_log2 : -INFINITY;
+        v[i] = (begin + t) * TK + skey + i <= my_pos ? v[i] * p.scale_log2 : -INFINITY;
         mx = fmaxf(mx, v[i]);
       }
 #pragma unroll
-      for (int d = TPR / 2; d > 0; d >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, d));
+      for (int d = TPR / 2; d > 0; d >>= 1) mx = fmaxf(mx, __shfl_xor_sync(FULL, mx, d));
       const float mn = fmaxf(m_run, mx), base = mn == -INFINITY ? 0.f : mn, alpha = exp2f(m_run - base);
       float sum = 0.f;
 #pragma unroll
       for (int i = 0; i < KPT; ++i) { v[i] = exp2f(v[i] - base); sum += v[i]; }
 #pragma unroll
-      for (int d = TPR / 2; d > 0; d >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, d);
+      for (int d = TPR / 2; d > 0; d >>= 1) sum += __shfl_xor_sync(FULL, sum, d);
       l_run = l_run * alpha + sum;
       m_run = mn;
 #pragma unroll
-      for (int i = 0; i < KPT; i += 2) *reinterpret_cast<uint32_t*>(sp + srow * PPT + skey + i) = pack2(v[i], v[i + 1]);
-      if (tid % TPR == 0) s_alpha[srow] = alpha;
+      for (int i = 0; i < KPT; i += 2) *reinterpret_cast<uint32_t*>(sp + (b * M + srow) * PPT + skey + i) = pack2(v[i], v[i + 1]);
+      if (tid % TPR == 0) s_alpha[b][srow] = alpha;
+      __syncwarp();
+      if (lane == 0) mbar_arrive(&bars.p_full[b]);
     }
-    __syncthreads();
+    if (tid % TPR == 0) { s_l[srow] = l_run; s_m[srow] = m_run; }
+  }
+  float o[MT][NV][4];
+  const int v0 = (warp - 8) * NV * 8;
+  if (warp >= 8 && warp < 16) {
+    // ------------------------------------------------------------------ sums of latents
 #pragma unroll
-    for (int m = 0; m < MT; ++m) {
-      const float a0 = s_alpha[m * 16 + lg], a1 = s_alpha[m * 16 + lg + 8];
+    for (int m = 0; m < MT; ++m)
 #pragma unroll
-      for (int n = 0; n < NV; ++n) { o[m][n][0] *= a0; o[m][n][1] *= a0; o[m][n][2] *= a1; o[m][n][3] *= a1; }
-    }
+      for (int n = 0; n < NV; ++n) { o[m][n][0] = o[m][n][1] = o[m][n][2] = o[m][n][3] = 0.f; }
+    const uint32_t vaddr = smem_addr(sk) + ((lane & 15) * ST + v0 + (lane >> 4) * 8) * 2;
+    const uint32_t paddr = smem_addr(sp) + ((lane & 15) * PPT + (lane >> 4) * 8) * 2;
+    for (int t = 0; t < tiles && ok; ++t) {
+      const int st = t % STAGES, b = t & 1;
+      if (!mbar_wait_warp(&bars.p_full[b], (t >> 1) & 1, abort_flag) || !mbar_wait_warp(&bars.k_full[st], (t / STAGES) & 1, abort_flag)) {
+        if (lane == 0) atomicCAS(p.err, 0, ERR_WAIT_OTHER);
+        ok = false;
+        break;
+      }
 #pragma unroll
-    for (int kk = 0; kk < TK; kk += 16) {
-      uint32_t a[MT][4];
+      for (int m = 0; m < MT; ++m) {
+        const float a0 = s_alpha[b][m * 16 + lg], a1 = s_alpha[b][m * 16 + lg + 8];
+        if (__any_sync(FULL, a0 != 1.f || a1 != 1.f)) {
 #pragma unroll
-      for (int m = 0; m < MT; ++m) ldsm4(a[m], smem_addr(sp + (m * 16 + (lane & 15)) * PPT + kk + (lane >> 4) * 8));
-#pragma unroll
-      for (int n = 0; n < NV; n += 2)
-        if (v0 + n * 8 < p.rank) {
-          uint32_t b[4];
-          ldsm4_t(b, smem_addr(tile + (kk + (lane & 15)) * ST + v0 + n * 8 + (lane >> 4) * 8));
-#pragma unroll
-          for (int m = 0; m < MT; ++m) {
-            mma(o[m][n], a[m], b[0], b[1]);
-            mma(o[m][n + 1], a[m], b[2], b[3]);
-          }
+          for (int n = 0; n < NV; ++n) { o[m][n][0] *= a0; o[m][n][1] *= a0; o[m][n][2] *= a1; o[m][n][3] *= a1; }
         }
+      }
+#pragma unroll
+      for (int kk = 0; kk < TK; kk += 16) {
+        uint32_t a[MT][4];
+#pragma unroll
+        for (int m = 0; m < MT; ++m) ldsm4(a[m], paddr + ((b * M + m * 16) * PPT + kk) * 2);
+#pragma unroll
+        for (int n = 0; n < NV; n += 2)
+          if (v0 + n * 8 < p.rank) {
+            uint32_t f[4];
+            ldsm4_t(f, vaddr + ((st * TK + kk) * ST + n * 8) * 2);
+#pragma unroll
+            for (int m = 0; m < MT; ++m) {
+              mma(o[m][n], a[m], f[0], f[1]);
+              mma(o[m][n + 1], a[m], f[2], f[3]);
+            }
+          }
+      }
+      __syncwarp();
+      if (lane == 0) { mbar_arrive(&bars.p_empty[b]); mbar_arrive(&bars.k_empty[st]); }
     }
   }
-  cp_wait<0>();
-  if (tid % TPR == 0) { s_l[srow] = l_run; s_m[srow] = m_run; }
   __syncthreads();
+  if (warp < 8 || warp >= 16) {
+    if (p.splits > 1 && tid < M && w0 + tid < work) {
+      const long long at = (static_cast<long long>(row) * work + w0 + tid) * p.splits + split;
+      p.part_m[at] = s_m[tid];
+      p.part_l[at] = s_l[tid];
+    }
+    return;
+  }
 #pragma unroll
   for (int m = 0; m < MT; ++m)
 #pragma unroll
@@ -446,11 +533,6 @@ latent_attend_kernel(Attend p, Pool pages) {
           else p.part_acc[(at * p.splits + split) * p.rank + c] = o[m][n][2 * e + q];
         }
     }
-  if (p.splits > 1 && tid < M && w0 + tid < work) {
-    const long long at = (static_cast<long long>(row) * work + w0 + tid) * p.splits + split;
-    p.part_m[at] = s_m[tid];
-    p.part_l[at] = s_l[tid];
-  }
 }
 
 // a block a (token, head)
@@ -513,7 +595,7 @@ int rows_of(const void* z, long long stride, const void* qw, const void* cw, flo
 template <int KS, int NV, int MT>
 int attend(const Attend& p, const Pool& pages, int R, cudaStream_t stream) {
   constexpr int M = 16 * MT;
-  const int smem = attend_stages<MT>() * TK * (p.W + 8) * 2 + 4 * M * SST * 4 + M * PPT * 2;
+  const int smem = attend_stages<MT>() * TK * p.W * 2 + 2 * 4 * M * SST * 4 + 2 * M * PPT * 2;
   cudaError_t e = cudaFuncSetAttribute(latent_attend_kernel<KS, NV, MT>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
   if (e != cudaSuccess) return static_cast<int>(e);
   const long long blocks = (static_cast<long long>(p.S) * p.H + M - 1) / M;
@@ -525,8 +607,9 @@ int attend(const Attend& p, const Pool& pages, int R, cudaStream_t stream) {
 }
 
 template <typename T>
-int product(const HeadProduct<T>& p, int trans, cudaStream_t stream) {
-  const dim3 grid((p.N + 63) / 64 + (p.table != nullptr ? 1 : 0), (p.tokens + 63) / 64, p.H);
+int product(HeadProduct<T> p, int trans, cudaStream_t stream) {
+  p.pairs = p.N % 2 == 0 && p.out_token % 2 == 0 && p.out_head % 2 == 0 && p.gate_token % 2 == 0 && aligned(p.out, 4) && aligned(p.gate, 4);
+  const dim3 grid((p.N + 63) / 64 + (p.table != nullptr ? (p.pad + TAIL - 1) / TAIL : 0), (p.tokens + 63) / 64, p.H);
   if constexpr (sizeof(T) == 2) {
     const bool whole = p.K % 8 == 0 && (!trans || p.N % 8 == 0) && p.a_token % 8 == 0 && p.a_head % 8 == 0 && p.w_head % 8 == 0 && p.w_ld % 8 == 0 &&
                        aligned(p.a, 16) && aligned(p.w, 16);
@@ -590,27 +673,27 @@ extern "C" int dewb_head_product(const void* a, long long a_token, long long a_h
   const float2* t = reinterpret_cast<const float2*>(table);
   if (fp32) return product(HeadProduct<float>{static_cast<const float*>(a), a_token, a_head, static_cast<const float*>(w), w_head, w_ld,
                                               static_cast<const float*>(gate), gate_token, static_cast<float*>(out), out_token, out_head, tokens, H, N, K, t, rot,
-                                              pad, dims, interleaved}, trans, stream);
+                                              pad, dims, interleaved, 0}, trans, stream);
   return product(HeadProduct<dewb::rows::bf16>{static_cast<const dewb::rows::bf16*>(a), a_token, a_head, static_cast<const dewb::rows::bf16*>(w), w_head, w_ld,
                                                static_cast<const dewb::rows::bf16*>(gate), gate_token, static_cast<dewb::rows::bf16*>(out), out_token, out_head,
-                                               tokens, H, N, K, t, rot, pad, dims, interleaved}, trans, stream);
+                                               tokens, H, N, K, t, rot, pad, dims, interleaved, 0}, trans, stream);
 }
 
-// q [R * S, H, W] (bf16) against the rows' latents in pool [*, page_size, W] -> out [R * S, H, rank]; W a multiple of 16, at most 576, rank at most
-// 512.  Scratch for splits > 1 (fp32): part_m, part_l [R * S * H * splits], part_acc [... * rank].  `wide`: 32 rows of work a CTA.
+// q [R * S, H, W] (bf16) against the rows' latents in pool [*, page_size, W] -> out [R * S, H, rank]; W a multiple of 16 plus 8, at most 584, rank at
+// most 512.  Scratch for splits > 1 (fp32): part_m, part_l [R * S * H * splits], part_acc [... * rank].  `wide`: 32 rows of work a CTA.
 extern "C" int dewb_latent_attend(const void* q, const void* pool, const int* positions, int R, int S, int H, int W, int rank, float scale, int splits,
                                   int wide, float* part_m, float* part_l, float* part_acc, void* out, const int* page_table, int page_size,
-                                  int max_pages, const int* row_ids, void* stream_ptr) {
+                                  int max_pages, const int* row_ids, int* err, void* stream_ptr) {
   if (R <= 0 || S <= 0) return 0;
-  if (H < 1 || W < 16 || W % 16 || W > 576 || rank < 1 || rank > W || rank > 512 || splits < 1 || splits > 65535 || R > 65535 || page_size < 1 || max_pages < 1 ||
+  if (H < 1 || W < 24 || W % 16 != 8 || W > 584 || rank < 1 || rank > W || rank > 512 || splits < 1 || splits > 65535 || R > 65535 || page_size < 1 || max_pages < 1 ||
       !aligned(q, 16) || !aligned(pool, 16) || (splits > 1 && (part_m == nullptr || part_l == nullptr || part_acc == nullptr)))
     return -3;
   cudaStream_t stream = reinterpret_cast<cudaStream_t>(stream_ptr);
   const Pool pages{page_table, page_size, max_pages, row_ids};
   const Attend p{static_cast<const dewb::rows::bf16*>(q), static_cast<const dewb::rows::bf16*>(pool), positions, static_cast<dewb::rows::bf16*>(out), part_m, part_l,
-                 part_acc, S, H, W, rank, splits, scale * 1.4426950408889634f};
-  if (W <= 192 && rank <= 128) return wide ? attend<3, 2, 2>(p, pages, R, stream) : attend<3, 2, 1>(p, pages, R, stream);
-  if (W <= 320 && rank <= 256) return wide ? attend<5, 4, 2>(p, pages, R, stream) : attend<5, 4, 1>(p, pages, R, stream);
+                 part_acc, S, H, W, rank, splits, scale * 1.4426950408889634f, err};
+  if (W <= 200 && rank <= 128) return wide ? attend<3, 2, 2>(p, pages, R, stream) : attend<3, 2, 1>(p, pages, R, stream);
+  if (W <= 328 && rank <= 256) return wide ? attend<5, 4, 2>(p, pages, R, stream) : attend<5, 4, 1>(p, pages, R, stream);
   return wide ? attend<9, 8, 2>(p, pages, R, stream) : attend<9, 8, 1>(p, pages, R, stream);
 }
 

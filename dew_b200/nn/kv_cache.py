@@ -79,9 +79,9 @@ class Call:
 
 def pool_width(slot: CacheSlot, dtype) -> int:
     """Width of a slot's pool heads: what the bf16 kernels are built for (64, 128, 256) where the head fits, else the head rounded up to 8; latent rows
-    are rounded up to 16."""
+    are rounded up to 16, and 8 more (the kernel's bank spacing)."""
     if slot.latent:
-        return (slot.head_dim + 15) // 16 * 16
+        return (slot.head_dim + 15) // 16 * 16 + 8
     w = max(slot.head_dim, slot.value_dim)
     if dtype == torch.bfloat16:
         for d in (64, 128, 256):

@@ -21,7 +21,7 @@ from . import paged as P
 from .rotary import Rotary, turn
 
 c_ll, c_int, c_float = ctypes.c_longlong, ctypes.c_int, ctypes.c_float
-MAX_WIDTH, MAX_RANK = 576, 512          # what the tensor-core kernel against the latents takes; past them, the general paged kernel
+MAX_WIDTH, MAX_RANK = 584, 512          # what the tensor-core kernel against the latents takes; past them, the general paged kernel
 
 
 @dataclass(frozen=True)
@@ -156,7 +156,7 @@ def flat_gate(gate: torch.Tensor) -> torch.Tensor:
 
 
 def attend_kernel_ok(q: torch.Tensor, lat: Latent, W: int) -> bool:
-    return q.dtype == torch.bfloat16 and W % 16 == 0 and W <= MAX_WIDTH and lat.rank <= MAX_RANK
+    return q.dtype == torch.bfloat16 and W % 16 == 8 and W <= MAX_WIDTH and lat.rank <= MAX_RANK
 
 
 def attend(q: torch.Tensor, lat: Latent, positions: torch.Tensor, pages: P.Pages, scale: float, longest: int, scratch=None,
@@ -170,15 +170,15 @@ def attend(q: torch.Tensor, lat: Latent, positions: torch.Tensor, pages: P.Pages
     out = torch.empty(R, S, H, lat.rank, dtype=q.dtype, device=q.device)
     wide = S * H > 16
     blocks, tiles = R * -(-S * H // (32 if wide else 16)), -(-longest // 32)
-    ctas = 148 if wide else 296                                  # as many as are resident at once
-    splits = max(1, min(ctas // max(blocks, 1), tiles // 4, 32))
+    splits = max(1, min(148 // max(blocks, 1), tiles // 4, 32))      # one CTA an SM
     pm = pl = pa = None
     if splits > 1:
         n = R * S * H * splits
         pm, pl, pa = (scratch or fresh_scratch(q.device))(n, lat.rank)
     L.check(L.load().dewb_latent_attend(L.ptr(q), L.ptr(pages.k), L.ptr(positions), c_int(R), c_int(S), c_int(H), c_int(W), c_int(lat.rank), c_float(scale),
                                         c_int(splits), c_int(int(wide)), L.ptr(pm), L.ptr(pl), L.ptr(pa), L.ptr(out), L.ptr(pages.table),
-                                        c_int(pages.page_size), c_int(pages.table.shape[1]), L.ptr(pages.row_ids), L.stream_ptr()), "latent_attend")
+                                        c_int(pages.page_size), c_int(pages.table.shape[1]), L.ptr(pages.row_ids), L.ptr(L.status(q.device)), L.stream_ptr()),
+            "latent_attend")
     L.count_launches(1 + int(splits > 1))
     return out
 

@@ -1,9 +1,11 @@
 """Prefill and decode throughput of a decoder design beside this library's closest decoder of the same sizes, and each of the design's kernels
 beside the like kernel of that decoder, as a fraction of its roofline: the Ragenex design here (closest: rotary attention and gated-delta-net
-layers in the same order, SwiGLU, one bf16 residual), the Fakonex design in ``telemetry.fakonex_bench``.
+layers in the same order, SwiGLU, one bf16 residual), the Fakonex design in ``telemetry.fakonex_bench``, the Selivik design in
+``telemetry.selivik_bench``.
 
-``bench.py --decoder ragenex | fakonex`` prints the result as one JSON line.  Weights are random.  Everything is timed on the device with CUDA events
-after warm-up; prefill activations and weights are larger than L2, and a decode step (one CUDA graph) streams all the weights.
+``bench.py --decoder ragenex | fakonex | selivik`` prints the result as one JSON line.  Weights are random.  Everything is timed on the device with CUDA events
+after warm-up; prefill activations and weights are larger than L2, and a decode step (one CUDA graph, where the model's step can be captured) streams
+all the weights.
 """
 from __future__ import annotations
 
@@ -45,6 +47,17 @@ def timed(fn: Callable[[], object], iters: int) -> float:
     return a.elapsed_time(b) / iters
 
 
+def replayed(fn: Callable[[], object], iters: int, copies: int = 8) -> float:
+    """Milliseconds per call inside a CUDA graph of ``copies`` calls (kernels of a decode step, which launches from Python would hide)."""
+    fn()
+    torch.cuda.synchronize()
+    graph = torch.cuda.CUDAGraph()
+    with torch.cuda.graph(graph):
+        for _ in range(copies):
+            fn()
+    return timed(graph.replay, iters) / copies
+
+
 def ragenex(s: dict, max_len: int, device="cuda"):
     """The design at size ``s``: every fourth layer lightning attention."""
     from ..models.causal_transformer import CausalTransformer, TransformerConfig
@@ -69,6 +82,12 @@ def closest(s: dict, max_len: int, device="cuda"):
         dtype=torch.bfloat16, device=device).eval()
 
 
+def keeps_latents(model) -> bool:
+    """Whether some layer keeps its latents outside the pages (``KVStore.latent``): its cached step forms a prompt's score matrix and reads lengths on the
+    host, so a prompt is timed as a whole sequence without a cache and a decode step without a graph."""
+    return any(k == "mla" and layer.mixer.shape is None for k, layer in zip(model.config.kinds(), model.layers))
+
+
 @torch.no_grad()
 def throughput(model, s: dict, rows: int, prompt: int, decode_rows: int, context: int, iters: int) -> Dict[str, float]:
     from ..nn.kv_cache import KVCache
@@ -86,8 +105,11 @@ def throughput(model, s: dict, rows: int, prompt: int, decode_rows: int, context
     pos = torch.arange(prompt, device="cuda")[None].repeat(rows, 1)
     store, c = cache(rows, prompt)
     store.chunk_span = (0, prompt)
+    uncached = keeps_latents(model)
 
     def prefill():
+        if uncached:
+            return model.logits(model(ids, return_hidden=True)[:, -1])
         return model.logits(model(ids, positions=pos, cache=c, return_hidden=True)[:, -1])
     ms = timed(prefill, iters)
     out = {"prefill_tokens_per_s": rows * prompt / ms * 1e3, "prefill_ms": ms}
@@ -98,6 +120,12 @@ def throughput(model, s: dict, rows: int, prompt: int, decode_rows: int, context
 
     def step():
         return model.next_tokens_greedy(model(tok, positions=at, cache=c, return_hidden=True)[:, 0])
+    if uncached:
+        ms = timed(step, 2 * iters)
+        out.update(decode_tokens_per_s=decode_rows / ms * 1e3, decode_ms=ms, eager=True)
+        del store, c
+        torch.cuda.empty_cache()
+        return out
     side = torch.cuda.Stream()
     with torch.cuda.stream(side):
         step()
@@ -209,6 +237,10 @@ def run(name: str = "ragenex", sizes=None, rows: int = 4, prompt: int = 4096, de
         from . import fakonex_bench as f
         table, design, near, parts = f.SIZES, f.design, f.closest, f.kernels
         context = 4095 if context is None else context           # the last position of a chunk: as many keys as the closest model's window holds
+    elif name == "selivik":
+        from . import selivik_bench as f
+        table, design, near, parts = f.SIZES, f.design, f.closest, f.kernels
+        context = 4096 if context is None else context
     else:
         table, design, near, parts = SIZES, ragenex, closest, kernels
         context = 4096 if context is None else context
