@@ -44,10 +44,9 @@ def angle(p, i, dims, base, factor=1.0):
 def rotate_pairs(x, p, pairs, base, dims, factor=1.0):
     """``x`` with every pair ``(a, b)`` of places (the i-th of ``pairs``) turned by the i-th angle of position ``p``."""
     y = x.clone()
-    for i, (a, b) in enumerate(pairs):
-        t = angle(p, i, dims, base, factor)
-        c, s = math.cos(t), math.sin(t)
-        y[a], y[b] = x[a] * c - x[b] * s, x[b] * c + x[a] * s
+    t = torch.tensor([angle(p, i, dims, base, factor) for i in range(len(pairs))], dtype=F)
+    a, b = (torch.tensor([pair[j] for pair in pairs]) for j in range(2))
+    y[a], y[b] = (x[a] * t.cos() - x[b] * t.sin()).to(x.dtype), (x[b] * t.cos() + x[a] * t.sin()).to(x.dtype)
     return y
 
 
