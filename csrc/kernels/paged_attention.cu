@@ -279,7 +279,9 @@ __device__ __forceinline__ int first_seen(int pos, const Extras<T>& ex) {
   return ex.window > 0 ? max(start, pos - ex.window + 1) : start;
 }
 
-constexpr int BQ = 32, BK = 32, THREADS = 256;
+constexpr int BQ = 32, BK = 32, THREADS = 256, WIDE = 576;
+
+__host__ __device__ inline int key_piece(int dk) { return dk <= WIDE ? dk : 256; }
 
 // grid (query tiles, G, rows).  q [R, S, *, D] with a token stride; out [R, S, H, dv] contiguous.  NJ: value columns per thread / 4.
 template <typename T, int NJ>
@@ -288,14 +290,15 @@ paged_attend_kernel(const T* __restrict__ q, long long q_token_stride, const T* 
                     const int* __restrict__ positions, int S, int H, int G, int dk, int dv, int D, float scale, T* __restrict__ out, Pool pool,
                     Extras<T> ex) {
   extern __shared__ __align__(16) float smem[];
-  const int kst = ((dk + 3) & ~3) + 4, vst = NJ * 32 + 4;
+  // keys past WIDE columns go through shared memory (with their queries) in pieces; values past a block's columns are other blocks' work
+  const int kc = key_piece(dk), kst = ((kc + 3) & ~3) + 4, vst = NJ * 32 + 4;
   float* sq = smem;                     // [BQ][kst]
   float* sk = sq + BQ * kst;            // [BK][kst]
   float* sv = sk + BK * kst;            // [BK][vst]
   float* sp = sv + BK * vst;            // [BQ][BK + 1]
   __shared__ int s_pos[BQ];
   __shared__ long long s_tok[BK];
-  const int row = blockIdx.z, g = blockIdx.y, Gq = H / G;
+  const int parts = (dv + NJ * 32 - 1) / (NJ * 32), row = blockIdx.z, g = blockIdx.y / parts, v0 = (blockIdx.y - g * parts) * NJ * 32, Gq = H / G;
   const int r0 = blockIdx.x * BQ, rows = S * Gq;
   const int tid = threadIdx.x;
   if (tid < BQ) {
@@ -308,15 +311,18 @@ paged_attend_kernel(const T* __restrict__ q, long long q_token_stride, const T* 
     last = max(last, s_pos[i]);
     if (s_pos[i] >= 0) lowest = min(lowest, first_seen(s_pos[i], ex));
   }
-  for (int i = tid; i < BQ * kst; i += THREADS) {
-    const int r = i / kst, c = i - r * kst;
-    float v = 0.f;
-    if (c < dk && s_pos[r] >= 0) {
-      const int gr = r0 + r;
-      v = ld(q + (static_cast<long long>(row) * S + gr / Gq) * q_token_stride + static_cast<long long>(g * Gq + gr % Gq) * D + c) * scale;
+  auto load_queries = [&](int c0) {
+    for (int i = tid; i < BQ * kst; i += THREADS) {
+      const int r = i / kst, c = i - r * kst;
+      float v = 0.f;
+      if (c < kc && c0 + c < dk && s_pos[r] >= 0) {
+        const int gr = r0 + r;
+        v = ld(q + (static_cast<long long>(row) * S + gr / Gq) * q_token_stride + static_cast<long long>(g * Gq + gr % Gq) * D + c0 + c) * scale;
+      }
+      sq[i] = v;
     }
-    sq[i] = v;
-  }
+  };
+  if (kc == dk) load_queries(0);
   const int qr = tid >> 3, ql = tid & 7;
   const int my_pos = s_pos[qr], my_first = first_seen(my_pos, ex);
   float m = -INFINITY, l = 0.f, acc[NJ][4];
@@ -329,22 +335,28 @@ paged_attend_kernel(const T* __restrict__ q, long long q_token_stride, const T* 
     __syncthreads();
     if (tid < BK) s_tok[tid] = k0 + tid <= last ? pool_token(pool, row, k0 + tid) : -1;
     __syncthreads();
-    for (int i = tid; i < BK * kst; i += THREADS) {
-      const int r = i / kst, c = i - r * kst;
-      sk[i] = (c < dk && s_tok[r] >= 0) ? ld(kpool + (s_tok[r] * G + g) * D + c) : 0.f;
-    }
     for (int i = tid; i < BK * vst; i += THREADS) {
       const int r = i / vst, c = i - r * vst;
-      sv[i] = (c < dv && s_tok[r] >= 0) ? ld(vpool + (s_tok[r] * G + g) * D + c) : 0.f;
+      sv[i] = (v0 + c < dv && s_tok[r] >= 0) ? ld(vpool + (s_tok[r] * G + g) * D + v0 + c) : 0.f;
     }
-    __syncthreads();
     float s[4] = {0.f, 0.f, 0.f, 0.f};
-    for (int c = 0; c < kst - 4; c += 4) {
-      const float4 a = *reinterpret_cast<const float4*>(sq + qr * kst + c);
+    for (int c0 = 0; c0 < dk; c0 += kc) {
+      if (kc != dk) {
+        if (c0 > 0) __syncthreads();                 // the piece before has been read
+        load_queries(c0);
+      }
+      for (int i = tid; i < BK * kst; i += THREADS) {
+        const int r = i / kst, c = i - r * kst;
+        sk[i] = (c < kc && c0 + c < dk && s_tok[r] >= 0) ? ld(kpool + (s_tok[r] * G + g) * D + c0 + c) : 0.f;
+      }
+      __syncthreads();
+      for (int c = 0; c < kst - 4; c += 4) {
+        const float4 a = *reinterpret_cast<const float4*>(sq + qr * kst + c);
 #pragma unroll
-      for (int j = 0; j < 4; ++j) {
-        const float4 b = *reinterpret_cast<const float4*>(sk + (ql + 8 * j) * kst + c);
-        s[j] += a.x * b.x + a.y * b.y + a.z * b.z + a.w * b.w;
+        for (int j = 0; j < 4; ++j) {
+          const float4 b = *reinterpret_cast<const float4*>(sk + (ql + 8 * j) * kst + c);
+          s[j] += a.x * b.x + a.y * b.y + a.z * b.z + a.w * b.w;
+        }
       }
     }
     float bm = -INFINITY;
@@ -396,7 +408,7 @@ paged_attend_kernel(const T* __restrict__ q, long long q_token_stride, const T* 
   for (int j = 0; j < NJ; ++j)
 #pragma unroll
     for (int e = 0; e < 4; ++e) {
-      const int c = ql * 4 + 32 * j + e;
+      const int c = v0 + ql * 4 + 32 * j + e;
       if (c < dv) st(o + c, acc[j][e] * inv);
     }
 }
@@ -581,13 +593,13 @@ int attend_mma(const bf16* q, long long qs, const bf16* kpool, const bf16* vpool
 template <typename T, int NJ>
 int attend(const T* q, long long qs, const T* kpool, const T* vpool, const int* positions, int R, int S, int H, int G, int dk, int dv, int D,
            float scale, T* out, const Pool& pool, const Extras<T>& ex, cudaStream_t stream) {
-  const int kst = ((dk + 3) & ~3) + 4, vst = NJ * 32 + 4;
+  const int kst = ((key_piece(dk) + 3) & ~3) + 4, vst = NJ * 32 + 4, parts = (dv + NJ * 32 - 1) / (NJ * 32);
   const size_t smem = static_cast<size_t>(BQ * kst + BK * kst + BK * vst + BQ * (BK + 1)) * 4;
   if (smem > 225 * 1024) return -3;
   cudaError_t e = cudaFuncSetAttribute(paged_attend_kernel<T, NJ>, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem));
   if (e != cudaSuccess) return static_cast<int>(e);
   const long long tiles = (static_cast<long long>(S) * (H / G) + BQ - 1) / BQ;
-  paged_attend_kernel<T, NJ><<<dim3(static_cast<unsigned>(tiles), G, R), THREADS, smem, stream>>>(q, qs, kpool, vpool, positions, S, H, G, dk, dv, D, scale, out,
+  paged_attend_kernel<T, NJ><<<dim3(static_cast<unsigned>(tiles), G * parts, R), THREADS, smem, stream>>>(q, qs, kpool, vpool, positions, S, H, G, dk, dv, D, scale, out,
                                                                                              pool, ex);
   return static_cast<int>(cudaGetLastError());
 }
@@ -605,8 +617,8 @@ int attend_any(const void* q, long long qs, const void* kpool, const void* vpool
   if (nj <= 4) return DEWB_ATTEND(4);
   if (nj <= 8) return DEWB_ATTEND(8);
   if (nj <= 16) return DEWB_ATTEND(16);
+  return DEWB_ATTEND(8);
 #undef DEWB_ATTEND
-  return -3;
 }
 
 }  // namespace paged
