@@ -203,56 +203,61 @@ __device__ __forceinline__ void cp_commit() { asm volatile("cp.async.commit_grou
 template <int N>
 __device__ __forceinline__ void cp_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory"); }
 
-// The same on the tensor cores: 64 x 64 tiles, 4 warps of 16 rows, K in pieces of 64 through a three-stage ring.  Every 16-byte piece of the operands
+// The same on the tensor cores: 64 x 64 tiles, 8 warps of 16 rows and 32 columns, K in pieces of 128 through a ring.  Every 16-byte piece of the operands
 // is aligned and whole (K, and N for TRANS, multiples of 8).
-constexpr int PST = 72;                            // smem row stride
-constexpr int P_STAGES = 3, P_STAGE = 2 * 64 * PST;
+constexpr int PK = 128, PST = PK + 8, WST = 72;    // smem row strides: pieces of a and w, and of a TRANS w (its rows are columns of the product)
+constexpr int P_STAGES = 3, P_THREADS = 256, P_STAGE = 64 * PST + (64 * PST > PK * WST ? 64 * PST : PK * WST);
 
 template <bool TRANS>
-__global__ void __launch_bounds__(128)
+__global__ void __launch_bounds__(P_THREADS)
 head_product_mma_kernel(HeadProduct<bf16> p) {
   extern __shared__ __align__(16) uint8_t raw[];
   bf16* ring = reinterpret_cast<bf16*>(raw);
   const int t0 = blockIdx.y * 64, n0 = blockIdx.x * 64, h = blockIdx.z;
-  if (n0 >= p.N) { tail_columns(p, t0, blockIdx.x - (p.N + 63) / 64, h, 128); return; }
-  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
-  const int steps = (p.K + 63) / 64;
+  if (n0 >= p.N) { tail_columns(p, t0, blockIdx.x - (p.N + 63) / 64, h, P_THREADS); return; }
+  const int tid = threadIdx.x, lane = tid & 31, warp = (tid >> 5) & 3, half = tid >> 7;
+  const int steps = (p.K + PK - 1) / PK;
   auto fetch = [&](int s) {
     if (s < steps) {
       bf16* sa = ring + (s % P_STAGES) * P_STAGE;
       bf16* sw = sa + 64 * PST;
-      const int k0 = s * 64;
+      const int k0 = s * PK;
 #pragma unroll
-      for (int i = 0; i < 4; ++i) {
-        const int at = i * 128 + tid, r = at >> 3, c = (at & 7) * 8;
+      for (int i = 0; i < 64 * PK / 8 / P_THREADS; ++i) {
+        const int at = i * P_THREADS + tid, r = at / (PK / 8), c = at % (PK / 8) * 8;
         const bool la = t0 + r < p.tokens && k0 + c < p.K;
         cp16(smem_addr(sa + r * PST + c), la ? p.a + (t0 + r) * p.a_token + h * p.a_head + k0 + c : p.a, la);
-        const bool lw = TRANS ? k0 + r < p.K && n0 + c < p.N : n0 + r < p.N && k0 + c < p.K;
-        cp16(smem_addr(sw + r * PST + c), lw ? p.w + h * p.w_head + (TRANS ? (k0 + r) * p.w_ld + n0 + c : (n0 + r) * p.w_ld + k0 + c) : p.w, lw);
+        const int wr = TRANS ? at >> 3 : r, wc = TRANS ? (at & 7) * 8 : c;
+        const bool lw = TRANS ? k0 + wr < p.K && n0 + wc < p.N : n0 + wr < p.N && k0 + wc < p.K;
+        cp16(smem_addr(sw + wr * (TRANS ? WST : PST) + wc),
+             lw ? p.w + h * p.w_head + (TRANS ? (k0 + wr) * p.w_ld + n0 + wc : (n0 + wr) * p.w_ld + k0 + wc) : p.w, lw);
       }
     }
     cp_commit();
   };
-  float acc[8][4] = {};
-  fetch(0);
-  fetch(1);
+  float acc[4][4] = {};
+#pragma unroll
+  for (int s = 0; s < P_STAGES - 1; ++s) fetch(s);
   for (int s = 0; s < steps; ++s) {
-    cp_wait<1>();
+    cp_wait<P_STAGES - 2>();
     __syncthreads();
-    fetch(s + 2);
+    fetch(s + P_STAGES - 1);
     const bf16* sa = ring + (s % P_STAGES) * P_STAGE;
     const bf16* sw = sa + 64 * PST;
 #pragma unroll
-    for (int kk = 0; kk < 64; kk += 16) {
-      uint32_t a[4];
+    for (int kk = 0; kk < PK; kk += 16) {
+      uint32_t a[4], b[2][4];
       ldsm4(a, smem_addr(sa + (warp * 16 + (lane & 15)) * PST + kk + (lane >> 4) * 8));
 #pragma unroll
-      for (int j = 0; j < 4; ++j) {
-        uint32_t b[4];
-        if (TRANS) ldsm4_t(b, smem_addr(sw + (kk + (lane & 15)) * PST + j * 16 + (lane >> 4) * 8));
-        else ldsm4(b, smem_addr(sw + (j * 16 + (lane & 7) + (lane >> 4) * 8) * PST + kk + ((lane >> 3) & 1) * 8));
-        mma(acc[2 * j], a, b[0], b[1]);
-        mma(acc[2 * j + 1], a, b[2], b[3]);
+      for (int j = 0; j < 2; ++j) {
+        const int n = half * 32 + j * 16;
+        if (TRANS) ldsm4_t(b[j], smem_addr(sw + (kk + (lane & 15)) * WST + n + (lane >> 4) * 8));
+        else ldsm4(b[j], smem_addr(sw + (n + (lane & 7) + (lane >> 4) * 8) * PST + kk + ((lane >> 3) & 1) * 8));
+      }
+#pragma unroll
+      for (int j = 0; j < 2; ++j) {
+        mma(acc[2 * j], a, b[j][0], b[j][1]);
+        mma(acc[2 * j + 1], a, b[j][2], b[j][3]);
       }
     }
   }
@@ -263,15 +268,15 @@ head_product_mma_kernel(HeadProduct<bf16> p) {
     const long long t = t0 + warp * 16 + lg + 8 * e;
     if (t >= p.tokens) continue;
     if (p.pairs) {                                     // pairs of columns; every gate is under way before the first is used
-      uint32_t z[8];
+      uint32_t z[4];
 #pragma unroll
-      for (int j = 0; j < 8; ++j) {
-        const int n = n0 + j * 8 + t2;
+      for (int j = 0; j < 4; ++j) {
+        const int n = n0 + half * 32 + j * 8 + t2;
         z[j] = p.gate != nullptr && n < p.N ? *reinterpret_cast<const uint32_t*>(p.gate + t * p.gate_token + static_cast<long long>(h) * p.N + n) : 0u;
       }
 #pragma unroll
-      for (int j = 0; j < 8; ++j) {
-        const int n = n0 + j * 8 + t2;
+      for (int j = 0; j < 4; ++j) {
+        const int n = n0 + half * 32 + j * 8 + t2;
         float a = acc[j][2 * e], b = acc[j][2 * e + 1];
         if (p.gate != nullptr) { a *= sigmoid(lo_f(z[j])); b *= sigmoid(hi_f(z[j])); }
         if (n < p.N) *reinterpret_cast<uint32_t*>(p.out + t * p.out_token + h * p.out_head + n) = pack2(a, b);
@@ -279,10 +284,10 @@ head_product_mma_kernel(HeadProduct<bf16> p) {
       continue;
     }
 #pragma unroll
-    for (int j = 0; j < 8; ++j)
+    for (int j = 0; j < 4; ++j)
 #pragma unroll
       for (int q = 0; q < 2; ++q) {
-        const int n = n0 + j * 8 + t2 + q;
+        const int n = n0 + half * 32 + j * 8 + t2 + q;
         if (n >= p.N) continue;
         float v = acc[j][2 * e + q];
         if (p.gate != nullptr) v *= sigmoid(ld(p.gate + t * p.gate_token + static_cast<long long>(h) * p.N + n));
@@ -618,8 +623,8 @@ int product(HeadProduct<T> p, int trans, cudaStream_t stream) {
       cudaError_t e = trans ? cudaFuncSetAttribute(head_product_mma_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem)
                             : cudaFuncSetAttribute(head_product_mma_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
       if (e != cudaSuccess) return static_cast<int>(e);
-      if (trans) head_product_mma_kernel<true><<<grid, 128, smem, stream>>>(p);
-      else head_product_mma_kernel<false><<<grid, 128, smem, stream>>>(p);
+      if (trans) head_product_mma_kernel<true><<<grid, P_THREADS, smem, stream>>>(p);
+      else head_product_mma_kernel<false><<<grid, P_THREADS, smem, stream>>>(p);
       return static_cast<int>(cudaGetLastError());
     }
   }
