@@ -297,10 +297,9 @@ head_product_mma_kernel(HeadProduct<bf16> p) {
 }
 
 // ---- attention against the latents: 17 warps.  Warp 16 brings tiles of 32 rows into a ring, one bulk copy a tile (a row, where pages do not hold whole
-// tiles).  Warps 0..7 form scores - a warp takes
-// a quarter of the W columns and half of the tile's keys, the partial scores meet in shared memory - and the online softmax.  Warps 8..15 keep the sums,
-// NV * 8 latent columns each, and free the stage.  Scores of one tile and values of the one before run at the same time.  KS: 16-column steps of a
-// quarter; MT: tiles of 16 rows of work (token, head).
+// tiles).  Warps 0..7 form scores: a warp takes a quarter of the W columns and half of the tile's keys, and leaves its part in shared memory.  Warps 8..15
+// add the parts up, keep the online softmax and the sums (NV * 8 latent columns each), and free the stage.  Scores of one tile and softmax and values of
+// the one before run at the same time.  KS: 16-column steps of a quarter; MT: tiles of 16 rows of work (token, head).
 constexpr int TK = 32, GROUP = 256, A_THREADS = 2 * GROUP + 32, SST = TK + 8, PPT = TK + 8;
 constexpr uint32_t FULL = 0xffffffffu;
 
@@ -320,7 +319,7 @@ constexpr int attend_stages() { return MT == 1 ? 5 : 4; }
 
 template <int STAGES>
 struct AttendBars {
-  uint64_t k_full[STAGES], k_empty[STAGES], p_full[2], p_empty[2];
+  uint64_t k_full[STAGES], k_empty[STAGES], s_full[2], s_empty[2];
   int abort_flag, poisoned;
 };
 
@@ -342,7 +341,7 @@ latent_attend_kernel(Attend p, Pool pages) {
     bars.poisoned = *reinterpret_cast<volatile int*>(p.err);
     bars.abort_flag = 0;
     for (int i = 0; i < STAGES; ++i) { mbar_init(&bars.k_full[i], 1); mbar_init(&bars.k_empty[i], 8); }
-    for (int i = 0; i < 2; ++i) { mbar_init(&bars.p_full[i], 8); mbar_init(&bars.p_empty[i], 8); }
+    for (int i = 0; i < 2; ++i) { mbar_init(&bars.s_full[i], 8); mbar_init(&bars.s_empty[i], 8); }
     fence_barrier_init();
     fence_proxy_async();
   }
@@ -355,7 +354,6 @@ latent_attend_kernel(Attend p, Pool pages) {
   const int all = (last + TK) / TK, per = (all + p.splits - 1) / p.splits;
   const int begin = min(all, split * per), tiles = min(all, begin + per) - begin;
   const int lg = lane >> 2, t2 = (lane & 3) * 2;
-  bool ok = true;
   if (warp == 16) {
     // ------------------------------------------------------------------ producer
     // Tokens past the last one (a tile whole in a page brings them along, else the last is repeated) meet weights of zero.
@@ -375,7 +373,7 @@ latent_attend_kernel(Attend p, Pool pages) {
     if (t < tiles)                                     // gave up: the copies under way still land in this block's memory
       for (int i = max(0, t - STAGES); i < t; ++i) mbar_wait_warp(&bars.k_full[i % STAGES], (i / STAGES) & 1, nullptr);
   } else if (warp < 8) {
-    // ------------------------------------------------------------------ scores and softmax
+    // ------------------------------------------------------------------ scores
     const int kq = warp & 3, kg = warp >> 2, steps = (p.W - 8) / 16, quarter = (steps + 3) / 4, first = kq * quarter, count = max(0, min(quarter, steps - first));
     uint32_t qa[MT][KS][4];                            // this warp's columns of the queries, as A operands
 #pragma unroll
@@ -391,14 +389,12 @@ latent_attend_kernel(Attend p, Pool pages) {
           qa[m][k][2 + e] = live && k < count ? *reinterpret_cast<const uint32_t*>(src + (first + k) * 16 + 8 + t2) : 0u;
         }
       }
-    const int srow = tid / TPR, skey = (tid % TPR) * KPT, my_pos = s_pos[srow];       // this thread's scores in the softmax
     const uint32_t kaddr = smem_addr(sk) + ((kg * 16 + (lane & 7) + (lane >> 4) * 8) * ST + first * 16 + ((lane >> 3) & 1) * 8) * 2;
-    float m_run = -INFINITY, l_run = 0.f;
     for (int t = 0; t < tiles; ++t) {
       const int st = t % STAGES, b = t & 1;
-      if (ok && !mbar_wait_warp(&bars.k_full[st], (t / STAGES) & 1, abort_flag)) { if (lane == 0) atomicCAS(p.err, 0, ERR_WAIT_FULL); ok = false; }
+      if (!mbar_wait_warp(&bars.k_full[st], (t / STAGES) & 1, abort_flag)) { if (lane == 0) atomicCAS(p.err, 0, ERR_WAIT_FULL); break; }
       float* part = ss + b * 4 * M * SST;
-      if (ok) {
+      {
         float s[MT][2][4];
 #pragma unroll
         for (int m = 0; m < MT; ++m)
@@ -416,6 +412,7 @@ latent_attend_kernel(Attend p, Pool pages) {
               mma(s[m][1], qa[m][k], f[2], f[3]);
             }
           }
+        if (!mbar_wait_warp(&bars.s_empty[b], ((t >> 1) & 1) ^ 1, abort_flag)) { if (lane == 0) atomicCAS(p.err, 0, ERR_WAIT_OTHER); break; }
 #pragma unroll
         for (int m = 0; m < MT; ++m)
 #pragma unroll
@@ -425,16 +422,33 @@ latent_attend_kernel(Attend p, Pool pages) {
             *reinterpret_cast<float2*>(d + 8 * SST) = make_float2(s[m][n][2], s[m][n][3]);
           }
       }
-      // the eight warps meet once a tile: the two buffers of partial scores take turns
-      asm volatile("bar.sync 1, 256;" ::: "memory");
-      if (ok && !mbar_wait_warp(&bars.p_empty[b], ((t >> 1) & 1) ^ 1, abort_flag)) { if (lane == 0) atomicCAS(p.err, 0, ERR_WAIT_OTHER); ok = false; }
-      if (!ok) continue;
-      float v[KPT], mx = -INFINITY;
+      __syncwarp();
+      if (lane == 0) mbar_arrive(&bars.s_full[b]);
+    }
+  }
+  float o[MT][NV][4];
+  const int v0 = (warp - 8) * NV * 8;
+  if (warp >= 8 && warp < 16) {
+    // ------------------------------------------------------------------ softmax and sums of latents
+    const int bid = tid - GROUP, srow = bid / TPR, skey = (bid % TPR) * KPT, my_pos = s_pos[srow];      // this thread's scores
+    float m_run = -INFINITY, l_run = 0.f;
+    bool ok = true;
 #pragma unroll
-      for (int i = 0; i < KPT; ++i) v[i] = 0.f;
+    for (int m = 0; m < MT; ++m)
 #pragma unroll
-      for (int q = 0; q < 4; ++q)
-        {
+      for (int n = 0; n < NV; ++n) { o[m][n][0] = o[m][n][1] = o[m][n][2] = o[m][n][3] = 0.f; }
+    const uint32_t vaddr = smem_addr(sk) + ((lane & 15) * ST + v0 + (lane >> 4) * 8) * 2;
+    const uint32_t paddr = smem_addr(sp) + ((lane & 15) * PPT + (lane >> 4) * 8) * 2;
+    for (int t = 0; t < tiles; ++t) {
+      const int st = t % STAGES, b = t & 1;
+      const float* part = ss + b * 4 * M * SST;
+      if (ok && !mbar_wait_warp(&bars.s_full[b], (t >> 1) & 1, abort_flag)) { if (lane == 0) atomicCAS(p.err, 0, ERR_WAIT_OTHER); ok = false; }
+      if (ok) {
+        float v[KPT], mx = -INFINITY;
+#pragma unroll
+        for (int i = 0; i < KPT; ++i) v[i] = 0.f;
+#pragma unroll
+        for (int q = 0; q < 4; ++q) {
           float x[KPT];
           const float* src = part + (q * M + srow) * SST + skey;
           if constexpr (KPT == 4) load_v<4>(src, x);
@@ -442,46 +456,29 @@ latent_attend_kernel(Attend p, Pool pages) {
 #pragma unroll
           for (int i = 0; i < KPT; ++i) v[i] += x[i];
         }
+        __syncwarp();
+        if (lane == 0) mbar_arrive(&bars.s_empty[b]);
 #pragma unroll
-      for (int i = 0; i < KPT; ++i) {
-        v[i] = (begin + t) * TK + skey + i <= my_pos ? v[i] * p.scale_log2 : -INFINITY;
-        mx = fmaxf(mx, v[i]);
+        for (int i = 0; i < KPT; ++i) {
+          v[i] = (begin + t) * TK + skey + i <= my_pos ? v[i] * p.scale_log2 : -INFINITY;
+          mx = fmaxf(mx, v[i]);
+        }
+#pragma unroll
+        for (int d = TPR / 2; d > 0; d >>= 1) mx = fmaxf(mx, __shfl_xor_sync(FULL, mx, d));
+        const float mn = fmaxf(m_run, mx), base = mn == -INFINITY ? 0.f : mn, alpha = exp2f(m_run - base);
+        float sum = 0.f;
+#pragma unroll
+        for (int i = 0; i < KPT; ++i) { v[i] = exp2f(v[i] - base); sum += v[i]; }
+        l_run = l_run * alpha + sum;                     // (this thread's keys alone: the parts meet at the end)
+        m_run = mn;
+#pragma unroll
+        for (int i = 0; i < KPT; i += 2) *reinterpret_cast<uint32_t*>(sp + (b * M + srow) * PPT + skey + i) = pack2(v[i], v[i + 1]);
+        if (bid % TPR == 0) s_alpha[b][srow] = alpha;
       }
-#pragma unroll
-      for (int d = TPR / 2; d > 0; d >>= 1) mx = fmaxf(mx, __shfl_xor_sync(FULL, mx, d));
-      const float mn = fmaxf(m_run, mx), base = mn == -INFINITY ? 0.f : mn, alpha = exp2f(m_run - base);
-      float sum = 0.f;
-#pragma unroll
-      for (int i = 0; i < KPT; ++i) { v[i] = exp2f(v[i] - base); sum += v[i]; }
-#pragma unroll
-      for (int d = TPR / 2; d > 0; d >>= 1) sum += __shfl_xor_sync(FULL, sum, d);
-      l_run = l_run * alpha + sum;
-      m_run = mn;
-#pragma unroll
-      for (int i = 0; i < KPT; i += 2) *reinterpret_cast<uint32_t*>(sp + (b * M + srow) * PPT + skey + i) = pack2(v[i], v[i + 1]);
-      if (tid % TPR == 0) s_alpha[b][srow] = alpha;
-      __syncwarp();
-      if (lane == 0) mbar_arrive(&bars.p_full[b]);
-    }
-    if (tid % TPR == 0) { s_l[srow] = l_run; s_m[srow] = m_run; }
-  }
-  float o[MT][NV][4];
-  const int v0 = (warp - 8) * NV * 8;
-  if (warp >= 8 && warp < 16) {
-    // ------------------------------------------------------------------ sums of latents
-#pragma unroll
-    for (int m = 0; m < MT; ++m)
-#pragma unroll
-      for (int n = 0; n < NV; ++n) { o[m][n][0] = o[m][n][1] = o[m][n][2] = o[m][n][3] = 0.f; }
-    const uint32_t vaddr = smem_addr(sk) + ((lane & 15) * ST + v0 + (lane >> 4) * 8) * 2;
-    const uint32_t paddr = smem_addr(sp) + ((lane & 15) * PPT + (lane >> 4) * 8) * 2;
-    for (int t = 0; t < tiles && ok; ++t) {
-      const int st = t % STAGES, b = t & 1;
-      if (!mbar_wait_warp(&bars.p_full[b], (t >> 1) & 1, abort_flag) || !mbar_wait_warp(&bars.k_full[st], (t / STAGES) & 1, abort_flag)) {
-        if (lane == 0) atomicCAS(p.err, 0, ERR_WAIT_OTHER);
-        ok = false;
-        break;
-      }
+      // the eight warps meet once a tile: the two buffers of weights take turns
+      asm volatile("bar.sync 1, 256;" ::: "memory");
+      if (ok && !mbar_wait_warp(&bars.k_full[st], (t / STAGES) & 1, abort_flag)) { if (lane == 0) atomicCAS(p.err, 0, ERR_WAIT_FULL); ok = false; }
+      if (!ok) continue;
 #pragma unroll
       for (int m = 0; m < MT; ++m) {
         const float a0 = s_alpha[b][m * 16 + lg], a1 = s_alpha[b][m * 16 + lg + 8];
@@ -508,8 +505,11 @@ latent_attend_kernel(Attend p, Pool pages) {
           }
       }
       __syncwarp();
-      if (lane == 0) { mbar_arrive(&bars.p_empty[b]); mbar_arrive(&bars.k_empty[st]); }
+      if (lane == 0) mbar_arrive(&bars.k_empty[st]);
     }
+#pragma unroll
+    for (int d = TPR / 2; d > 0; d >>= 1) l_run += __shfl_xor_sync(FULL, l_run, d);
+    if (bid % TPR == 0) { s_l[srow] = l_run; s_m[srow] = m_run; }
   }
   __syncthreads();
   if (warp < 8 || warp >= 16) {
