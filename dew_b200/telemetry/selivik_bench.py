@@ -164,7 +164,7 @@ def kernels(s: dict, tokens: int, decode_rows: int, context: int, iters: int) ->
     qa = latent.absorb(q1, up, lat, t1, W)
     lend = lambda n, width: store._partials(n, width, "cuda")
     q0 = rand(B, H, D)
-    nb, nb2 = B * (context + 1) * W * 2, B * (context + 1) * 2 * G * D * 2
+    nb, nb2 = B * (context + 1) * lat.row * 2, B * (context + 1) * 2 * G * D * 2
     entry("decode: latent_attend", "decode attention", lambda: latent.attend(qa, lat, posd, pages, 0.1, store.max_len, lend), nb,
           2 * (lat.row + lat.rank) * LH * B * (context + 1), lambda: plain.decode_attention(0, q0, lens), nb2, 0)
     wk, wv = lat.split_up(up)
