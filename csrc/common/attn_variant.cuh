@@ -6,6 +6,8 @@
 //   softcap  : scores become cap * tanh(score / cap)                 (0 = none)
 //   sinks    : one learned logit per query head that joins the softmax denominator only (forward; the backward kernels
 //              see it through the saved log-sum-exp)
+//   gain     : each head's scores times a number of its own, in front of the cap (forward only)
+//   sig      : every visible key weighs sigmoid(score + sig[head]), and nothing is divided by the sum of the weights (forward only)
 //   segments : packed documents - a query sees a key only if both carry the same segment id; ids are non-decreasing
 //              along the sequence (0 = padding, allowed after the last document), which is what lets whole tiles be skipped
 #pragma once
@@ -22,6 +24,8 @@ struct Variant {
   const int* k_seg;        // [B, T] or null
   int chunk;
   int keep;
+  const float* gain;       // [Hq] or null
+  const float* sig;        // [Hq] or null
 };
 
 // tanh to fp32 accuracy relative to 1 (scores under a cap are fp32 quantities): 1 - 2 / (1 + e^2x)

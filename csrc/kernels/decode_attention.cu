@@ -59,7 +59,8 @@ paged_decode_kernel(const __nv_bfloat16* __restrict__ q, const void* __restrict_
                     const float* __restrict__ kscale, const float* __restrict__ vscale,
                     const int* __restrict__ page_table, const int* __restrict__ lengths, float* __restrict__ part_m,
                     float* __restrict__ part_l, float* __restrict__ part_acc, int Hq, int Hkv, int share, int page_size,
-                    int max_pages, int splits, float scale_log2, int window, int keep, int chunk, float cap_log2) {
+                    int max_pages, int splits, float scale_log2, int window, int keep, int chunk, float cap_log2, const float* __restrict__ gain,
+                    const float* __restrict__ sig) {
   constexpr int DV = D / 32;                 // value elements per lane
   const int row = blockIdx.x, hk = blockIdx.y, split = blockIdx.z;
   const int kvh = hk / share;                  // `share` groups of query heads read the same KV head
@@ -74,7 +75,7 @@ paged_decode_kernel(const __nv_bfloat16* __restrict__ q, const void* __restrict_
   const int len = lengths[row];
   for (int i = threadIdx.x; i < G * D; i += blockDim.x) {
     const int g = i / D, d = i - g * D;
-    sq[g][d] = __bfloat162float(q[(static_cast<long long>(row) * Hq + hk * G + g) * D + d]) * scale_log2;
+    sq[g][d] = __bfloat162float(q[(static_cast<long long>(row) * Hq + hk * G + g) * D + d]) * (gain != nullptr ? scale_log2 * gain[hk * G + g] : scale_log2);
   }
   __syncthreads();
   // keys of this split: [k_begin, k_end) in 32-key blocks, interleaved across the CTA's warps
@@ -133,8 +134,15 @@ paged_decode_kernel(const __nv_bfloat16* __restrict__ q, const void* __restrict_
         for (int g = 0; g < GM; ++g) if (GT != 0 || g < G) s[g] = cap_log2 * attn::soft_tanh(s[g] / cap_log2);
       }
     }
-    // online softmax update (per query head), block maximum by warp reduction
+    // online softmax update (per query head), block maximum by warp reduction; sigmoid weights need neither maximum nor sum
     float p[GM];
+    if (sig != nullptr) {
+#pragma unroll
+      for (int g = 0; g < GM; ++g) if (GT != 0 || g < G) {
+        p[g] = live ? __fdividef(1.f, 1.f + exp2f(-(s[g] + sig[hk * G + g] * 1.4426950408889634f))) : 0.f;
+        m[g] = 0.f;
+      }
+    } else
 #pragma unroll
     for (int g = 0; g < GM; ++g) {
       if (GT != 0 || g < G) {
@@ -244,11 +252,11 @@ paged_decode_kernel(const __nv_bfloat16* __restrict__ q, const void* __restrict_
   }
 }
 
-// out[row, h, :] = sum_s acc_s * 2^(m_s - M) / sum_s l_s * 2^(m_s - M); optional attention sink per head
+// out[row, h, :] = sum_s acc_s * 2^(m_s - M) / sum_s l_s * 2^(m_s - M); optional attention sink per head; `sums`: not divided (m is 0 then)
 template <int D>
 __global__ void decode_combine_kernel(const float* __restrict__ part_m, const float* __restrict__ part_l,
                                       const float* __restrict__ part_acc, const float* __restrict__ sinks,
-                                      __nv_bfloat16* __restrict__ out, float* __restrict__ lse, int Hq, int splits) {
+                                      __nv_bfloat16* __restrict__ out, float* __restrict__ lse, int Hq, int splits, bool sums) {
   const long long rh = blockIdx.x;          // row * Hq + h
   const int d = threadIdx.x;
   float M = -INFINITY;
@@ -268,7 +276,7 @@ __global__ void decode_combine_kernel(const float* __restrict__ part_m, const fl
     a *= f;
     M = Mn;
   }
-  if (d < D) out[rh * D + d] = __float2bfloat16(L > 0.f ? a / L : 0.f);
+  if (d < D) out[rh * D + d] = __float2bfloat16(sums ? a : L > 0.f ? a / L : 0.f);
   if (d == 0 && lse != nullptr) lse[rh] = L > 0.f ? (M + log2f(L)) * 0.6931471805599453f : -INFINITY;
 }
 
@@ -314,15 +322,16 @@ __global__ void kv_append_kernel(const __nv_bfloat16* __restrict__ k_new, const 
 
 using namespace dewb::decode;
 
+// `gain` [Hq] (null: none): a head's scores times it, in front of the cap; `sig` [Hq] (null: softmax): weights sigmoid(score + sig[head]), not divided.
 // Scratch (caller-provided fp32): part_m, part_l [rows * Hq * splits], part_acc [rows * Hq * splits * D].
 extern "C" int dewb_paged_decode(const void* q, const void* kpool, const void* vpool, const float* kscale,
                                  const float* vscale, const int* page_table, const int* lengths, const float* sinks,
                                  void* out, float* lse, float* part_m, float* part_l, float* part_acc, int rows, int Hq,
                                  int Hkv, int share, int D, int page_size, int max_pages, int splits, float scale, int window,
-                                 int keep, int chunk, float softcap, int kv_kind, void* stream_ptr) {
+                                 int keep, int chunk, float softcap, const float* gain, const float* sig, int kv_kind, void* stream_ptr) {
   if (rows <= 0) return 0;
   if ((D != 64 && D != 128 && D != 256) || share < 1 || Hkv < 1 || Hq % (Hkv * share) != 0 ||
-      Hq / (Hkv * share) > MAX_G || splits < 1 || keep < 0 || (keep > 0 && chunk > 0))
+      Hq / (Hkv * share) > MAX_G || splits < 1 || keep < 0 || (keep > 0 && chunk > 0) || (sig != nullptr && (sinks != nullptr || lse != nullptr)))
     return -3;
   cudaStream_t stream = reinterpret_cast<cudaStream_t>(stream_ptr);
   const float scale_log2 = scale * 1.4426950408889634f;
@@ -330,7 +339,7 @@ extern "C" int dewb_paged_decode(const void* q, const void* kpool, const void* v
   const __nv_bfloat16* qp = reinterpret_cast<const __nv_bfloat16*>(q);
   const int Gq = Hq / (Hkv * share);
 #define DEWB_DECODE_G(DD, KK, GG) paged_decode_kernel<DD, KK, GG><<<grid, WARPS * 32, 0, stream>>>( \
-    qp, kpool, vpool, kscale, vscale, page_table, lengths, part_m, part_l, part_acc, Hq, Hkv, share, page_size, max_pages, splits, scale_log2, window, keep, chunk, softcap * 1.4426950408889634f)
+    qp, kpool, vpool, kscale, vscale, page_table, lengths, part_m, part_l, part_acc, Hq, Hkv, share, page_size, max_pages, splits, scale_log2, window, keep, chunk, softcap * 1.4426950408889634f, gain, sig)
 #define DEWB_DECODE(DD, KK) do { if (Gq == 4) DEWB_DECODE_G(DD, KK, 4); else if (Gq == 8) DEWB_DECODE_G(DD, KK, 8); \
     else if (Gq == 1) DEWB_DECODE_G(DD, KK, 1); else if (Gq == 2) DEWB_DECODE_G(DD, KK, 2); else DEWB_DECODE_G(DD, KK, 0); } while (0)
 #define DEWB_DECODE_D(KK) do { if (D == 64) DEWB_DECODE(64, KK); else if (D == 128) DEWB_DECODE(128, KK); else DEWB_DECODE(256, KK); } while (0)
@@ -339,9 +348,9 @@ extern "C" int dewb_paged_decode(const void* q, const void* kpool, const void* v
 #undef DEWB_DECODE
 #undef DEWB_DECODE_G
   __nv_bfloat16* op = reinterpret_cast<__nv_bfloat16*>(out);
-  if (D == 64) decode_combine_kernel<64><<<rows * Hq, 64, 0, stream>>>(part_m, part_l, part_acc, sinks, op, lse, Hq, splits);
-  else if (D == 128) decode_combine_kernel<128><<<rows * Hq, 128, 0, stream>>>(part_m, part_l, part_acc, sinks, op, lse, Hq, splits);
-  else decode_combine_kernel<256><<<rows * Hq, 256, 0, stream>>>(part_m, part_l, part_acc, sinks, op, lse, Hq, splits);
+  if (D == 64) decode_combine_kernel<64><<<rows * Hq, 64, 0, stream>>>(part_m, part_l, part_acc, sinks, op, lse, Hq, splits, sig != nullptr);
+  else if (D == 128) decode_combine_kernel<128><<<rows * Hq, 128, 0, stream>>>(part_m, part_l, part_acc, sinks, op, lse, Hq, splits, sig != nullptr);
+  else decode_combine_kernel<256><<<rows * Hq, 256, 0, stream>>>(part_m, part_l, part_acc, sinks, op, lse, Hq, splits, sig != nullptr);
   return static_cast<int>(cudaGetLastError());
 }
 
@@ -430,8 +439,8 @@ extern "C" int dewb_decode_combine(const float* part_m, const float* part_l, con
   if (D != 64 && D != 128 && D != 256) return -3;
   cudaStream_t stream = reinterpret_cast<cudaStream_t>(stream_ptr);
   __nv_bfloat16* op = reinterpret_cast<__nv_bfloat16*>(out);
-  if (D == 64) decode_combine_kernel<64><<<rows * Hq, 64, 0, stream>>>(part_m, part_l, part_acc, sinks, op, lse, Hq, splits);
-  else if (D == 128) decode_combine_kernel<128><<<rows * Hq, 128, 0, stream>>>(part_m, part_l, part_acc, sinks, op, lse, Hq, splits);
-  else decode_combine_kernel<256><<<rows * Hq, 256, 0, stream>>>(part_m, part_l, part_acc, sinks, op, lse, Hq, splits);
+  if (D == 64) decode_combine_kernel<64><<<rows * Hq, 64, 0, stream>>>(part_m, part_l, part_acc, sinks, op, lse, Hq, splits, false);
+  else if (D == 128) decode_combine_kernel<128><<<rows * Hq, 128, 0, stream>>>(part_m, part_l, part_acc, sinks, op, lse, Hq, splits, false);
+  else decode_combine_kernel<256><<<rows * Hq, 256, 0, stream>>>(part_m, part_l, part_acc, sinks, op, lse, Hq, splits, false);
   return static_cast<int>(cudaGetLastError());
 }

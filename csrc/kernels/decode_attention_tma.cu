@@ -337,7 +337,7 @@ paged_decode_persist_kernel(const __grid_constant__ CUtensorMap tk, const __grid
                             float* __restrict__ part_acc, int rows, int Hq, int Hkv, int page_size, int max_pages,
                             int max_parts, float scale_log2, int window, int keep, int chunk, float cap_log2, long long q_row_stride, int* __restrict__ err,
                             __nv_bfloat16* __restrict__ out, const float* __restrict__ sinks,
-                            unsigned int* __restrict__ arrivals, int min_tiles) {
+                            unsigned int* __restrict__ arrivals, int min_tiles, const float* __restrict__ gain, const float* __restrict__ sig) {
   extern __shared__ __align__(1024) uint8_t smem[];
   if ((smem_u32(smem) & 1023u) != 0) {
     if (threadIdx.x == 0) atomicCAS(err, 0, ERR_BAD_ARG);
@@ -438,6 +438,9 @@ paged_decode_persist_kernel(const __grid_constant__ CUtensorMap tk, const __grid
       }
     }
     float m_run = -INFINITY, l_run = 0.f;
+    const int my_head = it.hk * G + min(g, G - 1);
+    const float my_scale = gain != nullptr ? scale_log2 * gain[my_head] : scale_log2;
+    const float my_sig = sig != nullptr ? sig[my_head] * 1.4426950408889634f : 0.f;
     float o[16][4];
 #pragma unroll
     for (int n = 0; n < 16; ++n) { o[n][0] = 0.f; o[n][1] = 0.f; o[n][2] = 0.f; o[n][3] = 0.f; }
@@ -468,25 +471,31 @@ paged_decode_persist_kernel(const __grid_constant__ CUtensorMap tk, const __grid
 #pragma unroll
       for (int i = 0; i < 4; ++i) {
         const int key = key_base + (i >> 1) * 8 + (i & 1);
-        float v = sc[i >> 1][i & 1] * scale_log2;
+        float v = sc[i >> 1][i & 1] * my_scale;
         if (cap_log2 > 0.f) v = cap_log2 * attn::soft_tanh(v / cap_log2);
         v = (key >= it.walk.first || key < keep) && key < it.len ? v : -INFINITY;
         pv[i] = v;
         mx = fmaxf(mx, v);
       }
-      mx = fmaxf(mx, __shfl_xor_sync(FULL, mx, 1));
-      mx = fmaxf(mx, __shfl_xor_sync(FULL, mx, 2));
-      const float m_new = fmaxf(m_run, mx);
-      const float alpha = (m_run == -INFINITY) ? 0.f : exp2f(m_run - m_new);
-      float ps = 0.f;
+      if (sig != nullptr) {                                    // sigmoid weights: neither maximum nor sum
 #pragma unroll
-      for (int i = 0; i < 4; ++i) { pv[i] = (m_new == -INFINITY) ? 0.f : exp2f(pv[i] - m_new); ps += pv[i]; }
-      ps += __shfl_xor_sync(FULL, ps, 1);
-      ps += __shfl_xor_sync(FULL, ps, 2);
-      l_run = l_run * alpha + ps;
-      m_run = m_new;
+        for (int i = 0; i < 4; ++i) pv[i] = pv[i] == -INFINITY ? 0.f : __fdividef(1.f, 1.f + exp2f(-(pv[i] + my_sig)));
+        m_run = 0.f;
+      } else {
+        mx = fmaxf(mx, __shfl_xor_sync(FULL, mx, 1));
+        mx = fmaxf(mx, __shfl_xor_sync(FULL, mx, 2));
+        const float m_new = fmaxf(m_run, mx);
+        const float alpha = (m_run == -INFINITY) ? 0.f : exp2f(m_run - m_new);
+        float ps = 0.f;
 #pragma unroll
-      for (int n = 0; n < 16; ++n) { o[n][0] *= alpha; o[n][1] *= alpha; }
+        for (int i = 0; i < 4; ++i) { pv[i] = (m_new == -INFINITY) ? 0.f : exp2f(pv[i] - m_new); ps += pv[i]; }
+        ps += __shfl_xor_sync(FULL, ps, 1);
+        ps += __shfl_xor_sync(FULL, ps, 2);
+        l_run = l_run * alpha + ps;
+        m_run = m_new;
+#pragma unroll
+        for (int n = 0; n < 16; ++n) { o[n][0] *= alpha; o[n][1] *= alpha; }
+      }
       const uint32_t pa0 = pack_bf16(pv[0], pv[1]), pa2 = pack_bf16(pv[2], pv[3]);
 #pragma unroll
       for (int nb2 = 0; nb2 < 8; ++nb2) {
@@ -530,7 +539,7 @@ paged_decode_persist_kernel(const __grid_constant__ CUtensorMap tk, const __grid
             ll = ll * f + exp2f(sk - mn);
             a *= f;
           }
-          out[(head0 + gg) * D + d] = __float2bfloat16(ll > 0.f ? a / ll : 0.f);
+          out[(head0 + gg) * D + d] = __float2bfloat16(sig != nullptr ? a : ll > 0.f ? a / ll : 0.f);
         } else {
           const long long oidx = (head0 + gg) * max_parts + it.part;
           part_acc[oidx * D + d] = a;
@@ -570,7 +579,7 @@ paged_decode_persist_kernel(const __grid_constant__ CUtensorMap tk, const __grid
         Lsum = Lsum * f + exp2f(sk - mn);
         a *= f;
       }
-      out[(head0 + gg) * D + d] = __float2bfloat16(Lsum > 0.f ? a / Lsum : 0.f);
+      out[(head0 + gg) * D + d] = __float2bfloat16(sig != nullptr ? a : Lsum > 0.f ? a / Lsum : 0.f);
     }
   }
 }
@@ -630,7 +639,7 @@ extern "C" int dewb_paged_decode_fused(const void* q, const void* kpool, const v
   return static_cast<int>(cudaGetLastError());
 }
 
-// Persistent, balanced form of the same operation (see the kernel's comment): one launch of `ctas` CTAs (two per SM) that
+// Persistent, balanced form of the same operation (see the kernel's comment; `gain` and `sig` as in dewb_paged_decode): one launch of `ctas` CTAs (two per SM) that
 // share out the tiles evenly.  A CTA's range is at least `min_tiles` tiles, so a (row, head) of n tiles is cut into at most
 // (n - 1) / min_tiles + 2 parts: `max_parts` (the stride of the partial buffers: part_m / part_l [rows * Hq * max_parts],
 // part_acc [... * 128]) must be at least that for the longest row.  rows <= 1024; `arrivals` uint32 [rows * Hkv], zero once.
@@ -638,11 +647,12 @@ extern "C" int dewb_paged_decode_persist(const void* q, const void* kpool, const
                                          const int* page_table, const int* lengths, float* part_m, float* part_l,
                                          float* part_acc, unsigned int* arrivals, const float* sinks, void* out, int rows, int Hq,
                                          int Hkv, int page_size, int max_pages, int max_parts, int min_tiles, float scale,
-                                         int window, int keep, int chunk, float softcap, long long q_row_stride, int ctas, int* err, void* stream_ptr) {
+                                         int window, int keep, int chunk, float softcap, const float* gain, const float* sig, long long q_row_stride, int ctas,
+                                         int* err, void* stream_ptr) {
   using namespace dewb::decode2;
   if (rows <= 0) return 0;
   if (Hq % Hkv != 0 || Hq / Hkv > 8 || page_size % TK != 0 || keep < 0 || (keep > 0 && chunk > 0) || max_parts < 2 || min_tiles < 1 || pool_tokens <= 0 ||
-      rows > P_MAXROWS || ctas < 1)
+      rows > P_MAXROWS || ctas < 1 || (sig != nullptr && sinks != nullptr))
     return -3;
   CUtensorMap tk, tv;
   int r;
@@ -654,6 +664,6 @@ extern "C" int dewb_paged_decode_persist(const void* q, const void* kpool, const
   paged_decode_persist_kernel<<<ctas, THREADS, P_SMEM, reinterpret_cast<cudaStream_t>(stream_ptr)>>>(
       tk, tv, reinterpret_cast<const __nv_bfloat16*>(q), page_table, lengths, part_m, part_l, part_acc, rows, Hq, Hkv, page_size,
       max_pages, max_parts, scale * 1.4426950408889634f, window, keep, chunk, softcap * 1.4426950408889634f, q_row_stride > 0 ? q_row_stride : static_cast<long long>(Hq) * D, err,
-      reinterpret_cast<__nv_bfloat16*>(out), sinks, arrivals, min_tiles);
+      reinterpret_cast<__nv_bfloat16*>(out), sinks, arrivals, min_tiles, gain, sig);
   return static_cast<int>(cudaGetLastError());
 }

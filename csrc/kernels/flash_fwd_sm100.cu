@@ -82,7 +82,8 @@ static_assert(sizeof(Bars) <= 2560, "Bars must fit the space Cfg::SMEM leaves af
 // probabilities (tcgen05.st) and the P V product reads its A operand from there, so P never crosses shared memory (no
 // 32 KB store + 32 KB operand fetch per tile) and the softmax of the next tile need not wait for the product to drain
 // a shared buffer.  PT = false is the shared-memory form (P in the 128-byte-swizzled K-major layout).
-template <int DK, int DV, bool CAUSAL, bool PT, bool VAR>
+// SIG: the weights are sigmoids (Variant::sig): no maxima, no sums, nothing to rescale.
+template <int DK, int DV, bool CAUSAL, bool PT, bool VAR, bool SIG>
 __global__ void __launch_bounds__(THREADS, 1)
 flash_fwd_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__ CUtensorMap tk,
                  const __grid_constant__ CUtensorMap tv, const __grid_constant__ CUtensorMap tq2, const __grid_constant__ CUtensorMap tk2,
@@ -241,6 +242,8 @@ flash_fwd_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__
     const uint32_t lane_addr = static_cast<uint32_t>(q4 * 32) << 16;
     float m_used = -INFINITY, l = 0.f;
     bool ok = true;
+    if (VAR && var.gain != nullptr) scale_log2 *= var.gain[h];
+    const float sig2 = SIG ? var.sig[h] * 1.4426950408889634f : 0.f;
     if (PT) {
       // this thread's half of its query row, from the swizzled shared tile to tensor memory: lane = row, 32-bit column w
       // = features 2w, 2w + 1 (the layout of a tensor-memory A operand)
@@ -334,6 +337,24 @@ flash_fwd_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__
             }
           }
         }
+        if constexpr (SIG) {
+          const uint32_t pbase = tmem + lane_addr + (st ? C::TMEM_S1 : C::TMEM_S0) + half * (HC / 2);
+          // the other thread of the row has its scores in registers before this one overwrites their columns
+          named_barrier_sync(1 + q4, 64);
+#pragma unroll
+          for (int c = 0; c < HC / 32; ++c) {
+            uint32_t pk[16];
+#pragma unroll
+            for (int i = 0; i < 16; ++i)
+              pk[i] = pack_bf16(__fdividef(1.f, 1.f + fast_exp2(-(s[c * 32 + 2 * i] + sig2))), __fdividef(1.f, 1.f + fast_exp2(-(s[c * 32 + 2 * i + 1] + sig2))));
+            tmem_st_32x32b_x16(pbase + c * 16, pk);
+          }
+          tmem_st_wait();
+          tc_fence_before();
+          __syncwarp();
+          if (lane == 0) mbar_arrive(&bars->p_full);
+          continue;
+        }
         {
           // four independent chains, not one of 64 dependent maxima
           float m0 = s[0], m1 = s[1], m2 = s[2], m3 = s[3];
@@ -341,6 +362,10 @@ flash_fwd_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__
           for (int i = 4; i < HC; i += 4) { m0 = fmaxf(m0, s[i]); m1 = fmaxf(m1, s[i + 1]); m2 = fmaxf(m2, s[i + 2]); m3 = fmaxf(m3, s[i + 3]); }
           mt = fmaxf(fmaxf(m0, m1), fmaxf(m2, m3));
         }
+      }
+      if constexpr (SIG) {                             // (a wait gave up: only the barrier's count is kept)
+        named_barrier_sync(1 + q4, 64);
+        continue;
       }
       // the row's maximum over all 128 columns: exchange with the thread that holds the other half of the row
       bars->xmax[j & 1][half][r] = mt;
@@ -420,8 +445,8 @@ flash_fwd_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__
     named_barrier_sync(1 + q4, 64);
     l += bars->xmax[n_tiles & 1][half ^ 1][r];
     float lse_shift = 0.f;     // log2 of the factor the sink adds to the denominator's scale
-    float inv = l > 0.f ? 1.f / l : 0.f;
-    if (VAR && var.sinks != nullptr) {
+    float inv = SIG ? 1.f : l > 0.f ? 1.f / l : 0.f;
+    if (VAR && !SIG && var.sinks != nullptr) {
       // the sink joins the denominator only: softmax over [scores, sink] with the sink's value column dropped
       const float sink2 = var.sinks[h] * 1.4426950408889634f;
       const float m_fin = fmaxf(m_used, sink2);
@@ -485,12 +510,13 @@ flash_fwd_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__
   }
 }
 
-template <int DK, int DV, bool CAUSAL, bool PT, bool VAR>
+template <int DK, int DV, bool CAUSAL, bool PT, bool VAR, bool SIG = false>
 static int launch(const CUtensorMap& tq, const CUtensorMap& tk, const CUtensorMap& tv, const CUtensorMap& tq2, const CUtensorMap& tk2, void* out,
                   float* lse, int B, int S, int T, int Hq, int Hkv, long long osb, long long oss, long long osh, float scale_log2,
                   const Variant& var, const Parts& parts, int* err, cudaStream_t stream) {
   static_assert(PT || Cfg<DK, DV>::P_BYTES > 0, "P has no shared memory here");
-  auto kern = flash_fwd_kernel<DK, DV, CAUSAL, PT, VAR>;
+  static_assert(!SIG || (PT && VAR), "sigmoid weights run the tensor-memory form of the variants");
+  auto kern = flash_fwd_kernel<DK, DV, CAUSAL, PT, VAR, SIG>;
   cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, Cfg<DK, DV>::SMEM);
   if (e != cudaSuccess) return static_cast<int>(e);
   dim3 grid((S + BM - 1) / BM, Hq, B);
@@ -524,14 +550,14 @@ extern "C" int dewb_flash_set_variant(int variant) {
 
 // q [B,S,Hq,D], k/v [B,T,Hkv,D] (bf16, unit stride along D, other strides in elements: batch, sequence, head);
 // out [B,S,Hq,D] with its own strides; lse [B,Hq,S] fp32 (natural log), may be null.
-// Variants (each off at 0 / null): `window` keys visible behind each query, `keep` first keys visible beside a window, `chunk` positions a query sees no key from outside of, `softcap`, `sinks` [Hq] fp32, `q_seg` [B,S] /
+// Variants (each off at 0 / null): `gain` [Hq] fp32 factors of the heads' scores, `sig` [Hq] fp32: sigmoid weights (causal, without lse and sinks), `window` keys visible behind each query, `keep` first keys visible beside a window, `chunk` positions a query sees no key from outside of, `softcap`, `sinks` [Hq] fp32, `q_seg` [B,S] /
 // `k_seg` [B,T] int32 segment ids of packed documents (non-decreasing along the sequence, rows 16-byte aligned: S, T % 4 == 0).
 extern "C" int dewb_flash_fwd_var(const void* q, const void* k, const void* v, void* out, float* lse, int B, int S, int T,
                                   int Hq, int Hkv, int D, long long q_sb, long long q_ss, long long q_sh, long long k_sb,
                                   long long k_ss, long long k_sh, long long v_sb, long long v_ss, long long v_sh,
                                   long long o_sb, long long o_ss, long long o_sh, float scale, int causal, int window,
-                                  int keep, int chunk, float softcap, const float* sinks, const int* q_seg, const int* k_seg, int* err,
-                                  void* stream_ptr) {
+                                  int keep, int chunk, float softcap, const float* sinks, const int* q_seg, const int* k_seg, const float* gain,
+                                  const float* sig, int* err, void* stream_ptr) {
   using namespace dewb::attnfwd;
   if (D != 128 && D != 64) return -3;
   if (Hq % Hkv != 0) return -3;
@@ -540,7 +566,7 @@ extern "C" int dewb_flash_fwd_var(const void* q, const void* k, const void* v, v
     return -3;
   if ((q_seg != nullptr) != (k_seg != nullptr)) return -3;
   if (q_seg != nullptr && ((T % 4) || (reinterpret_cast<uintptr_t>(k_seg) & 15))) return -3;
-  if (window < 0 || keep < 0 || chunk < 0 || softcap < 0.f) return -3;
+  if (window < 0 || keep < 0 || chunk < 0 || softcap < 0.f || (sig != nullptr && (sinks != nullptr || lse != nullptr || !causal))) return -3;
   if (keep > 0 && (window == 0 || chunk > 0)) return -3;
   CUtensorMap tq, tk, tv;
   int r;
@@ -549,11 +575,16 @@ extern "C" int dewb_flash_fwd_var(const void* q, const void* k, const void* v, v
   if ((r = make_qkv_map(&tv, v, B, T, Hkv, D, v_sb, v_ss, v_sh))) return 3000 + r;
   const float scale_log2 = scale * 1.4426950408889634f;
   cudaStream_t stream = reinterpret_cast<cudaStream_t>(stream_ptr);
-  const Variant var{window, softcap, sinks, q_seg, k_seg, chunk, keep};
+  const Variant var{window, softcap, sinks, q_seg, k_seg, chunk, keep, gain, sig};
   const Parts parts{D / 64, D, nullptr, 0};
-  const bool any = window > 0 || chunk > 0 || softcap > 0.f || sinks != nullptr || q_seg != nullptr;
+  const bool any = window > 0 || chunk > 0 || softcap > 0.f || sinks != nullptr || q_seg != nullptr || gain != nullptr || sig != nullptr;
 #define DEWB_FLASH_GO(DD, CC, PP, VV) launch<DD, DD, CC, PP, VV>(tq, tk, tv, tq, tk, out, lse, B, S, T, Hq, Hkv, o_sb, o_ss, o_sh, scale_log2, var, parts, err, stream)
   const bool pt = g_variant != 0;
+  if (sig != nullptr) {
+#define DEWB_FLASH_SIG(DD) launch<DD, DD, true, true, true, true>(tq, tk, tv, tq, tk, out, lse, B, S, T, Hq, Hkv, o_sb, o_ss, o_sh, scale_log2, var, parts, err, stream)
+    return D == 128 ? DEWB_FLASH_SIG(128) : DEWB_FLASH_SIG(64);
+#undef DEWB_FLASH_SIG
+  }
   if (any) {
     // the variants run the tensor-memory form only
     if (D == 128) return causal ? DEWB_FLASH_GO(128, true, true, true) : DEWB_FLASH_GO(128, false, true, true);
@@ -574,7 +605,7 @@ extern "C" int dewb_flash_fwd(const void* q, const void* k, const void* v, void*
                               long long o_sb, long long o_ss, long long o_sh, float scale, int causal, int* err,
                               void* stream_ptr) {
   return dewb_flash_fwd_var(q, k, v, out, lse, B, S, T, Hq, Hkv, D, q_sb, q_ss, q_sh, k_sb, k_ss, k_sh, v_sb, v_ss, v_sh, o_sb,
-                            o_ss, o_sh, scale, causal, 0, 0, 0, 0.f, nullptr, nullptr, nullptr, err, stream_ptr);
+                            o_ss, o_sh, scale, causal, 0, 0, 0, 0.f, nullptr, nullptr, nullptr, nullptr, nullptr, err, stream_ptr);
 }
 
 // Causal attention whose queries and keys come in two parts: q [B,S,H,da + db] and keys [B,T,H,da] per head (strides in elements: batch, sequence,
@@ -601,7 +632,7 @@ extern "C" int dewb_flash_fwd_parts(const void* q, const void* k, const void* k2
   if ((r = make_qkv_map(&tk2, k2, B, T, 1, db, k2_sb, k2_ss, k2_ss))) return 2500 + r;
   if ((r = make_qkv_map(&tv, v, B, T, H, dv, v_sb, v_ss, v_sh))) return 3000 + r;
   cudaStream_t stream = reinterpret_cast<cudaStream_t>(stream_ptr);
-  const Variant var{0, 0.f, nullptr, nullptr, nullptr, 0, 0};
+  const Variant var{0, 0.f, nullptr, nullptr, nullptr, 0, 0, nullptr, nullptr};
   const Parts parts{first, dv, static_cast<const __nv_bfloat16*>(gate), gate_stride};
   const long long oss = static_cast<long long>(H) * dv, osb = oss * S;
 #define DEWB_PARTS_GO(KK, VV) launch<KK, VV, true, true, false>(tq, tk, tv, tq2, tk2, out, nullptr, B, S, T, H, H, osb, oss, dv, \

@@ -10,7 +10,7 @@
 //
 // Selection: logits may carry a bias; scores are a sigmoid or softmax of the logits, or the logits themselves, whose weights are then the softmax over
 // the chosen ones alone; choice scores add a bias that steers the choice only; with groups, a group counts
-// the sum of its two best choice scores and the experts outside a token's best groups are out of the choice (their choice scores become
+// the sum of its two best choice scores (or its best one) and the experts outside a token's best groups are out of the choice (their choice scores become
 // `fill`); the weights are the chosen scores, divided by their sum where `norm` asks for it.  Tokens at positions below 0 are padding: no
 // expert runs for them.  A row's place among its expert's rows comes from an atomic counter, so it may differ from run to run; the rows of a
 // product do not depend on each other.  Compiled without fast math.
@@ -41,7 +41,7 @@ __device__ __forceinline__ float ld(const bf16* p) { return __bfloat162float(*p)
 struct Choice {
   const float* bias;       // [E] or null: steers the choice alone
   const float* logit_bias;  // [E] or null: part of the logits
-  int E, k, groups, keep;
+  int E, k, groups, keep, best;   // a group counts the sum of its `best` (1 or 2) best choice scores
   float fill;              // choice score of experts outside the kept groups
   int score, norm;         // score 0: softmax, 1: sigmoid, 2: the logits, weights by the softmax over the chosen ones
   float scaling;
@@ -95,7 +95,7 @@ __device__ __forceinline__ void choose(const Choice& c, long long t, bool live, 
         const float v = s_sel[e];
         if (v > a) { b = a; a = v; } else if (v > b) b = v;
       }
-      s_group[g] = per > 1 ? a + b : a;
+      s_group[g] = per > 1 && c.best > 1 ? a + b : a;
     }
     __syncwarp();
 #pragma unroll
@@ -460,10 +460,10 @@ using namespace dewb::moeserve;
 // logits [T, ld] fp32 (plus logits[., rest + e] when rest > 0) -> weights, ids, rank [T, k], counts [E] (zero before the call).
 // `positions` [T] or null: below 0 = padding.
 extern "C" int dewb_moe_select(const float* logits, long long ld_, int rest, const float* bias, const float* logit_bias, const int* positions, int T,
-                               int E, int k, int groups, int keep, float fill, int score, int norm, float scaling, float* weights, int* ids, int* rank, int* counts,
+                               int E, int k, int groups, int keep, int best, float fill, int score, int norm, float scaling, float* weights, int* ids, int* rank, int* counts,
                                void* stream_ptr) {
   if (T <= 0) return 0;
-  const Choice c{bias, logit_bias, E, k, groups, keep, fill, score, norm, scaling, weights, ids, rank, counts};
+  const Choice c{bias, logit_bias, E, k, groups, keep, best, fill, score, norm, scaling, weights, ids, rank, counts};
   if (!choice_ok(c) || ld_ < E || rest < 0 || (rest > 0 && ld_ < rest + E)) return -3;
   cudaStream_t stream = reinterpret_cast<cudaStream_t>(stream_ptr);
   if (E <= 128) return select<4>(logits, ld_, rest, positions, T, c, stream);
@@ -473,10 +473,10 @@ extern "C" int dewb_moe_select(const float* logits, long long ld_, int rest, con
 
 // The same with the logits made here: x [T, d] (fp32 or bf16), w [E, d] (fp32, or bf16 beside a bf16 x).
 extern "C" int dewb_moe_router(const void* x, const void* w, const float* bias, const float* logit_bias, const int* positions, int T, int d, int E,
-                               int k, int groups, int keep, float fill, int score, int norm, float scaling, float* weights, int* ids, int* rank, int* counts, int x_fp32,
+                               int k, int groups, int keep, int best, float fill, int score, int norm, float scaling, float* weights, int* ids, int* rank, int* counts, int x_fp32,
                                int w_fp32, void* stream_ptr) {
   if (T <= 0) return 0;
-  const Choice c{bias, logit_bias, E, k, groups, keep, fill, score, norm, scaling, weights, ids, rank, counts};
+  const Choice c{bias, logit_bias, E, k, groups, keep, best, fill, score, norm, scaling, weights, ids, rank, counts};
   if (!choice_ok(c) || d < 1 || (x_fp32 && !w_fp32)) return -3;
   cudaStream_t stream = reinterpret_cast<cudaStream_t>(stream_ptr);
   const bool vec = d % 4 == 0 && aligned(x, 16) && aligned(w, 16);

@@ -13,7 +13,8 @@
 //                    and takes the head widths the tensor-core kernels do not.
 //   paged_attend_mma   the same on the tensor cores for bf16 pools 64, 128 or 256 wide (a prompt's later portions, mixed start positions)
 //   Both take chunks (a query sees no key from before the start of its chunk of positions), a window beside which the row's first keys may stay
-//   visible, a soft cap on the scores, a learned sink per head in the denominator, and a gate per head on the output.
+//   visible, a factor per head on the scores, a soft cap on them, a learned sink per head in the denominator, and a gate per head on the output;
+//   instead of the softmax, every visible key may weigh the sigmoid of its score plus a number per head, with no sum over the keys.
 //
 // A query's row of work is (token, head of its group), so a group's heads share the key and value tiles.  Positions below 0 are padding:
 // nothing is appended for them and their outputs are zero.  Compiled without fast math.
@@ -269,6 +270,8 @@ struct Extras {
   const float* sinks;      // [H]: joins the denominator, has no value
   const T* gate;           // [tokens, *]: head h's output times sigmoid(gate[token, h])
   long long gate_stride;
+  const float* gain;       // [H]: the head's scores times it, in front of the cap
+  const float* sig;        // [H]: weights are sigmoid(score + sig[head]) instead of the softmax
 };
 
 // First key a query sees, the kept ones aside.
@@ -317,7 +320,9 @@ paged_attend_kernel(const T* __restrict__ q, long long q_token_stride, const T* 
       float v = 0.f;
       if (c < kc && c0 + c < dk && s_pos[r] >= 0) {
         const int gr = r0 + r;
-        v = ld(q + (static_cast<long long>(row) * S + gr / Gq) * q_token_stride + static_cast<long long>(g * Gq + gr % Gq) * D + c0 + c) * scale;
+        const int head = g * Gq + gr % Gq;
+        v = ld(q + (static_cast<long long>(row) * S + gr / Gq) * q_token_stride + static_cast<long long>(head) * D + c0 + c) *
+            (ex.gain != nullptr ? scale * ex.gain[head] : scale);
       }
       sq[i] = v;
     }
@@ -325,6 +330,7 @@ paged_attend_kernel(const T* __restrict__ q, long long q_token_stride, const T* 
   if (kc == dk) load_queries(0);
   const int qr = tid >> 3, ql = tid & 7;
   const int my_pos = s_pos[qr], my_first = first_seen(my_pos, ex);
+  const float my_sig = ex.sig != nullptr ? ex.sig[g * Gq + (r0 + qr) % Gq] : 0.f;
   float m = -INFINITY, l = 0.f, acc[NJ][4];
 #pragma unroll
   for (int j = 0; j < NJ; ++j) { acc[j][0] = acc[j][1] = acc[j][2] = acc[j][3] = 0.f; }
@@ -367,24 +373,31 @@ paged_attend_kernel(const T* __restrict__ q, long long q_token_stride, const T* 
       if (key > my_pos || (key < my_first && key >= ex.keep)) s[j] = -INFINITY;
       bm = fmaxf(bm, s[j]);
     }
+    if (ex.sig != nullptr) {
 #pragma unroll
-    for (int o = 4; o > 0; o >>= 1) bm = fmaxf(bm, __shfl_xor_sync(0xffffffffu, bm, o));
-    const float mn = fmaxf(m, bm);
-    const float alpha = m == -INFINITY ? 0.f : expf(m - mn);
-    float ps = 0.f;
+      for (int j = 0; j < 4; ++j) sp[qr * (BK + 1) + ql + 8 * j] = s[j] == -INFINITY ? 0.f : sigmoid(s[j] + my_sig);
+      l = 1.f;                                       // nothing to divide by
+      __syncwarp();
+    } else {
 #pragma unroll
-    for (int j = 0; j < 4; ++j) {
-      const float p = s[j] == -INFINITY ? 0.f : expf(s[j] - mn);
-      ps += p;
-      sp[qr * (BK + 1) + ql + 8 * j] = p;
+      for (int o = 4; o > 0; o >>= 1) bm = fmaxf(bm, __shfl_xor_sync(0xffffffffu, bm, o));
+      const float mn = fmaxf(m, bm);
+      const float alpha = m == -INFINITY ? 0.f : expf(m - mn);
+      float ps = 0.f;
+#pragma unroll
+      for (int j = 0; j < 4; ++j) {
+        const float p = s[j] == -INFINITY ? 0.f : expf(s[j] - mn);
+        ps += p;
+        sp[qr * (BK + 1) + ql + 8 * j] = p;
+      }
+#pragma unroll
+      for (int o = 4; o > 0; o >>= 1) ps += __shfl_xor_sync(0xffffffffu, ps, o);
+      l = l * alpha + ps;
+      m = mn;
+      __syncwarp();
+#pragma unroll
+      for (int j = 0; j < NJ; ++j) { acc[j][0] *= alpha; acc[j][1] *= alpha; acc[j][2] *= alpha; acc[j][3] *= alpha; }
     }
-#pragma unroll
-    for (int o = 4; o > 0; o >>= 1) ps += __shfl_xor_sync(0xffffffffu, ps, o);
-    l = l * alpha + ps;
-    m = mn;
-    __syncwarp();
-#pragma unroll
-    for (int j = 0; j < NJ; ++j) { acc[j][0] *= alpha; acc[j][1] *= alpha; acc[j][2] *= alpha; acc[j][3] *= alpha; }
     for (int k = 0; k < BK; ++k) {
       const float p = sp[qr * (BK + 1) + k];
 #pragma unroll
@@ -425,7 +438,8 @@ __device__ __forceinline__ void cp16(uint32_t dst, const void* src, bool live) {
 // tanh to fp32 accuracy relative to 1
 __device__ __forceinline__ float soft_tanh(float x) { return 1.f - __fdividef(2.f, 1.f + exp2f(x * 2.8853900817779268f)); }
 
-template <int D>
+// SIG: sigmoid weights
+template <int D, bool SIG>
 __global__ void __launch_bounds__(MTHREADS)
 paged_attend_mma_kernel(const bf16* __restrict__ q, long long q_token_stride, const bf16* __restrict__ kpool, const bf16* __restrict__ vpool,
                         const int* __restrict__ positions, int S, int H, int G, int dv, float scale_log2, bf16* __restrict__ out, Pool pool,
@@ -475,6 +489,9 @@ paged_attend_mma_kernel(const bf16* __restrict__ q, long long q_token_stride, co
   const int lg = lane >> 2, t2 = (lane & 3) * 2;
   const int p0 = s_pos[warp * 16 + lg], p1 = s_pos[warp * 16 + lg + 8];
   const int f0_ = first_seen(p0, ex), f1_ = first_seen(p1, ex);        // first keys the rows see
+  const int h0_ = g * Gq + (r0 + warp * 16 + lg) % Gq, h1_ = g * Gq + (r0 + warp * 16 + lg + 8) % Gq;
+  const float c0_ = ex.gain != nullptr ? scale_log2 * ex.gain[h0_] : scale_log2, c1_ = ex.gain != nullptr ? scale_log2 * ex.gain[h1_] : scale_log2;
+  const float b0_ = SIG ? ex.sig[h0_] * 1.4426950408889634f : 0.f, b1_ = SIG ? ex.sig[h1_] * 1.4426950408889634f : 0.f;
   float m0 = -INFINITY, m1 = -INFINITY, l0 = 0.f, l1 = 0.f, o[D / 8][4];
 #pragma unroll
   for (int j = 0; j < D / 8; ++j) { o[j][0] = o[j][1] = o[j][2] = o[j][3] = 0.f; }
@@ -510,14 +527,17 @@ paged_attend_mma_kernel(const bf16* __restrict__ q, long long q_token_stride, co
       const int key = first_key_of(t) + j * 8 + t2;
 #pragma unroll
       for (int e = 0; e < 4; ++e) {
-        float v = s[j][e] * scale_log2;
+        float v = s[j][e] * (e < 2 ? c0_ : c1_);
         if (ex.cap > 0.f) v = ex.cap * soft_tanh(v / ex.cap);
         const int at = key + (e & 1), p = e < 2 ? p0 : p1, f = e < 2 ? f0_ : f1_;
-        s[j][e] = at <= p && (at >= f || at < ex.keep) ? v : -INFINITY;
+        const bool seen = at <= p && (at >= f || at < ex.keep);
+        if (SIG) s[j][e] = seen ? __fdividef(1.f, 1.f + exp2f(-(v + (e < 2 ? b0_ : b1_)))) : 0.f;
+        else s[j][e] = seen ? v : -INFINITY;
       }
       x0 = fmaxf(x0, fmaxf(s[j][0], s[j][1]));
       x1 = fmaxf(x1, fmaxf(s[j][2], s[j][3]));
     }
+    if constexpr (!SIG) {
 #pragma unroll
     for (int d = 1; d < 4; d <<= 1) {
       x0 = fmaxf(x0, __shfl_xor_sync(0xffffffffu, x0, d));
@@ -536,6 +556,7 @@ paged_attend_mma_kernel(const bf16* __restrict__ q, long long q_token_stride, co
       s[j][2] = exp2f(s[j][2] - b1); s[j][3] = exp2f(s[j][3] - b1);
       l0 += s[j][0] + s[j][1];
       l1 += s[j][2] + s[j][3];
+    }
     }
 #pragma unroll
     for (int j = 0; j < 4; ++j) {
@@ -556,7 +577,7 @@ paged_attend_mma_kernel(const bf16* __restrict__ q, long long q_token_stride, co
     l0 += __shfl_xor_sync(0xffffffffu, l0, d);
     l1 += __shfl_xor_sync(0xffffffffu, l1, d);
   }
-  const float i0 = l0 > 0.f ? 1.f / l0 : 0.f, i1 = l1 > 0.f ? 1.f / l1 : 0.f;
+  const float i0 = SIG ? 1.f : l0 > 0.f ? 1.f / l0 : 0.f, i1 = SIG ? 1.f : l1 > 0.f ? 1.f / l1 : 0.f;
 #pragma unroll
   for (int e = 0; e < 2; ++e) {
     const int gr = r0 + warp * 16 + lg + 8 * e;
@@ -578,14 +599,14 @@ paged_attend_mma_kernel(const bf16* __restrict__ q, long long q_token_stride, co
   }
 }
 
-template <int D>
+template <int D, bool SIG>
 int attend_mma(const bf16* q, long long qs, const bf16* kpool, const bf16* vpool, const int* positions, int R, int S, int H, int G, int dv, float scale,
                bf16* out, const Pool& pool, const Extras<bf16>& ex, cudaStream_t stream) {
   const int smem = (MQ + 4 * MK) * (D + 8) * 2;
-  cudaError_t e = cudaFuncSetAttribute(paged_attend_mma_kernel<D>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
+  cudaError_t e = cudaFuncSetAttribute(paged_attend_mma_kernel<D, SIG>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
   if (e != cudaSuccess) return static_cast<int>(e);
   const long long tiles = (static_cast<long long>(S) * (H / G) + MQ - 1) / MQ;
-  paged_attend_mma_kernel<D><<<dim3(static_cast<unsigned>(tiles), G, R), MTHREADS, smem, stream>>>(q, qs, kpool, vpool, positions, S, H, G, dv,
+  paged_attend_mma_kernel<D, SIG><<<dim3(static_cast<unsigned>(tiles), G, R), MTHREADS, smem, stream>>>(q, qs, kpool, vpool, positions, S, H, G, dv,
                                                                                               scale * 1.4426950408889634f, out, pool, ex);
   return static_cast<int>(cudaGetLastError());
 }
@@ -607,8 +628,8 @@ int attend(const T* q, long long qs, const T* kpool, const T* vpool, const int* 
 template <typename T>
 int attend_any(const void* q, long long qs, const void* kpool, const void* vpool, const int* positions, int R, int S, int H, int G, int dk, int dv,
                int D, float scale, void* out, const Pool& pool, int chunk, int window, int keep, float softcap, const float* sinks, const void* gate,
-               long long gate_stride, cudaStream_t stream) {
-  const Extras<T> ex{chunk, window, keep, softcap, sinks, static_cast<const T*>(gate), gate_stride};
+               long long gate_stride, const float* gain, const float* sig, cudaStream_t stream) {
+  const Extras<T> ex{chunk, window, keep, softcap, sinks, static_cast<const T*>(gate), gate_stride, gain, sig};
 #define DEWB_ATTEND(NN) attend<T, NN>(static_cast<const T*>(q), qs, static_cast<const T*>(kpool), static_cast<const T*>(vpool), positions, R, S, H, G, \
                                       dk, dv, D, scale, static_cast<T*>(out), pool, ex, stream)
   const int nj = (dv + 31) / 32;
@@ -710,34 +731,37 @@ static bool range_ok(int chunk, int window, int keep, float softcap) {
   return chunk >= 0 && window >= 0 && keep >= 0 && (keep == 0 || chunk == 0) && softcap >= 0.f;
 }
 
-// `chunk` 0, `window` 0 (and `keep` with it), `softcap` 0, `sinks` null, `gate` null: off (see Extras).
+// `chunk` 0, `window` 0 (and `keep` with it), `softcap` 0, `sinks`, `gate`, `gain` and `sig` null: off (see Extras).
 extern "C" int dewb_paged_attend(const void* q, long long q_token_stride, const void* kpool, const void* vpool, const int* positions, int R, int S,
                                  int H, int G, int dk, int dv, int D, float scale, int chunk, int window, int keep, float softcap, const float* sinks, const void* gate,
-                                 long long gate_stride, void* out, const int* page_table, int page_size, int max_pages, const int* row_ids, int fp32,
-                                 void* stream_ptr) {
+                                 long long gate_stride, const float* gain, const float* sig, void* out, const int* page_table, int page_size, int max_pages,
+                                 const int* row_ids, int fp32, void* stream_ptr) {
   if (R <= 0 || S <= 0) return 0;
-  if (H < 1 || G < 1 || H % G || dk < 1 || dv < 1 || D < dk || D < dv || page_size < 1 || max_pages < 1 || !range_ok(chunk, window, keep, softcap)) return -3;
+  if (H < 1 || G < 1 || H % G || dk < 1 || dv < 1 || D < dk || D < dv || page_size < 1 || max_pages < 1 || !range_ok(chunk, window, keep, softcap) || (sig != nullptr && sinks != nullptr)) return -3;
   cudaStream_t stream = reinterpret_cast<cudaStream_t>(stream_ptr);
   const Pool pool{page_table, page_size, max_pages, row_ids};
-  if (fp32) return attend_any<float>(q, q_token_stride, kpool, vpool, positions, R, S, H, G, dk, dv, D, scale, out, pool, chunk, window, keep, softcap, sinks, gate, gate_stride, stream);
-  return attend_any<bf16>(q, q_token_stride, kpool, vpool, positions, R, S, H, G, dk, dv, D, scale, out, pool, chunk, window, keep, softcap, sinks, gate, gate_stride, stream);
+  if (fp32) return attend_any<float>(q, q_token_stride, kpool, vpool, positions, R, S, H, G, dk, dv, D, scale, out, pool, chunk, window, keep, softcap, sinks, gate, gate_stride, gain, sig, stream);
+  return attend_any<bf16>(q, q_token_stride, kpool, vpool, positions, R, S, H, G, dk, dv, D, scale, out, pool, chunk, window, keep, softcap, sinks, gate, gate_stride, gain, sig, stream);
 }
 
 // The tensor-core form (bf16; pools D = 64, 128 or 256 wide; q on 16-byte boundaries with a token stride of a multiple of 8).
 extern "C" int dewb_paged_attend_mma(const void* q, long long q_token_stride, const void* kpool, const void* vpool, const int* positions, int R, int S,
                                      int H, int G, int dv, int D, float scale, int chunk, int window, int keep, float softcap, const float* sinks, const void* gate, long long gate_stride,
-                                     void* out, const int* page_table, int page_size, int max_pages, const int* row_ids, void* stream_ptr) {
+                                     const float* gain, const float* sig, void* out, const int* page_table, int page_size, int max_pages, const int* row_ids, void* stream_ptr) {
   if (R <= 0 || S <= 0) return 0;
-  if (H < 1 || G < 1 || H % G || dv < 1 || D < dv || page_size < 1 || max_pages < 1 || !range_ok(chunk, window, keep, softcap) || q_token_stride % 8 || !aligned(q, 16) || !aligned(kpool, 16) ||
+  if (H < 1 || G < 1 || H % G || dv < 1 || D < dv || page_size < 1 || max_pages < 1 || !range_ok(chunk, window, keep, softcap) || (sig != nullptr && sinks != nullptr) ||
+      q_token_stride % 8 || !aligned(q, 16) || !aligned(kpool, 16) ||
       !aligned(vpool, 16))
     return -3;
   cudaStream_t stream = reinterpret_cast<cudaStream_t>(stream_ptr);
   const Pool pool{page_table, page_size, max_pages, row_ids};
   const bf16 *qp = static_cast<const bf16*>(q), *kp = static_cast<const bf16*>(kpool), *vp = static_cast<const bf16*>(vpool);
   bf16* op = static_cast<bf16*>(out);
-  const Extras<bf16> ex{chunk, window, keep, softcap * 1.4426950408889634f, sinks, static_cast<const bf16*>(gate), gate_stride};
-  if (D == 64) return attend_mma<64>(qp, q_token_stride, kp, vp, positions, R, S, H, G, dv, scale, op, pool, ex, stream);
-  if (D == 128) return attend_mma<128>(qp, q_token_stride, kp, vp, positions, R, S, H, G, dv, scale, op, pool, ex, stream);
-  if (D == 256) return attend_mma<256>(qp, q_token_stride, kp, vp, positions, R, S, H, G, dv, scale, op, pool, ex, stream);
+  const Extras<bf16> ex{chunk, window, keep, softcap * 1.4426950408889634f, sinks, static_cast<const bf16*>(gate), gate_stride, gain, sig};
+#define DEWB_MMA(DD, SS) attend_mma<DD, SS>(qp, q_token_stride, kp, vp, positions, R, S, H, G, dv, scale, op, pool, ex, stream)
+  if (D == 64) return sig != nullptr ? DEWB_MMA(64, true) : DEWB_MMA(64, false);
+  if (D == 128) return sig != nullptr ? DEWB_MMA(128, true) : DEWB_MMA(128, false);
+  if (D == 256) return sig != nullptr ? DEWB_MMA(256, true) : DEWB_MMA(256, false);
+#undef DEWB_MMA
   return -3;
 }

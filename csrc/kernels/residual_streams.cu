@@ -3,12 +3,13 @@
 //
 //   embed_streams   H[t, s, :] = gain * embed[token t] (+ pos[position t]) for every stream s
 //   stream_step     one residual step between two sub-layers: the pending write of the sub-layer that just ran
-//                       H'[t] = sum_s mix[s, t] H[s] + out[t] * gain * (scale . y + scale2 . y2)
+//                       H'[t] = sum_s mix[s, t] H[s] + out[t] * (gain scale . y + gain2 scale2 . y2)
 //                   (in place), the read of the next one, u = sum_s read[s] H'[s], and its norm (layer norm without a bias, or RMS norm,
 //                   whose weights may be stored as their distance from `around`); y may pass an RMS norm of its own first (a block that
 //                   normalises what its sub-layers return); y2 is there when two sub-layers read the same norm and join together.  Without connection
 //                   weights the streams keep themselves and take y as it is: one such stream is the ordinary fp32 residual, which has a
-//                   form of its own (residual_step).
+//                   form of its own (residual_step).  What else joins the one stream on the way (Join): the token's embedding again, and a vector
+//                   (a looped block of layers takes them in front of each pass).  The norm's weight may be one number for all coordinates.
 //   clamped_glu     g sigmoid(alpha g) (u + 1) with g = min(gate, limit), u = clamp(up, -limit, limit)
 //   gelu_glu        gelu(gate) up, the tanh form of gelu
 //   sigmoid_gated_norm   RMS norm over a whole row times a weight times sigmoid(gate)
@@ -50,13 +51,52 @@ embed_streams_kernel(const long long* __restrict__ tokens, const int* __restrict
   }
 }
 
+// What joins the residual beside the sub-layers: add [d] and gain * table[token] (null: neither).
+template <typename T>
+struct Join {
+  const T* add;
+  const T* table;
+  const long long* tokens;
+  int vocab;
+  float gain;
+  __host__ __device__ __forceinline__ bool any() const { return add != nullptr || table != nullptr; }
+  template <int V>
+  __device__ __forceinline__ void to(float (&x)[V], long long t, int i, int d) const {
+    if (table != nullptr) {
+      float e[V];
+      load_v<V>(table + min(max(tokens[t], 0ll), static_cast<long long>(vocab - 1)) * d + i, e);
+#pragma unroll
+      for (int j = 0; j < V; ++j) x[j] += gain * e[j];
+    }
+    if (add != nullptr) {
+      float e[V];
+      load_v<V>(add + i, e);
+#pragma unroll
+      for (int j = 0; j < V; ++j) x[j] += e[j];
+    }
+  }
+};
+
+// V weights of a norm: `one` - the same number for every coordinate
+template <typename T, int V>
+__device__ __forceinline__ void load_weight(const T* w, int one, int i, float (&c)[V]) {
+  if (one) {
+    float x[1];
+    load_v<1>(w, x);
+#pragma unroll
+    for (int j = 0; j < V; ++j) c[j] = x[0];
+  } else {
+    load_v<V>(w + i, c);
+  }
+}
+
 // NS: the number of streams when it is small and known (registers sized for it), 0: any number up to MAX_STREAMS.
 template <typename T, int V, int NS>
 __global__ void __launch_bounds__(THREADS)
 stream_step_kernel(float* __restrict__ H, const T* __restrict__ y, const T* __restrict__ y_weight, const T* __restrict__ scale,
                    const float* __restrict__ mix, const float* __restrict__ out, const float* __restrict__ read, const T* __restrict__ w,
                    T* __restrict__ normed, int n_rt, int d, float y_eps, float eps, int rms, const T* __restrict__ y2, const T* __restrict__ scale2,
-                   float gain, float around) {
+                   float gain, float gain2, float around, int w_one, Join<T> join) {
   constexpr int NM = NS ? NS : MAX_STREAMS;
   const int n = NS ? NS : n_rt;
   extern __shared__ float su[];                      // y, then u of this token
@@ -106,15 +146,15 @@ stream_step_kernel(float* __restrict__ H, const T* __restrict__ y, const T* __re
 #pragma unroll
         for (int j = 0; j < V; ++j) b[j] *= c[j];
       }
+#pragma unroll
+      for (int j = 0; j < V; ++j) b[j] *= gain;
       if (y2 != nullptr) {
         float b2[V], c[V];
         load_v<V>(y2 + t * d + i, b2);
         if (scale2 != nullptr) load_v<V>(scale2 + i, c);
 #pragma unroll
-        for (int j = 0; j < V; ++j) b[j] += scale2 != nullptr ? c[j] * b2[j] : b2[j];
+        for (int j = 0; j < V; ++j) b[j] += gain2 * (scale2 != nullptr ? c[j] * b2[j] : b2[j]);
       }
-#pragma unroll
-      for (int j = 0; j < V; ++j) b[j] *= gain;
 #pragma unroll(NS ? NS : 1)
       for (int q = 0; q < NM; ++q) {
         if (NS || q < n) {
@@ -128,6 +168,7 @@ stream_step_kernel(float* __restrict__ H, const T* __restrict__ y, const T* __re
 #pragma unroll
               for (int j = 0; j < V; ++j) a[j] += m * x[s][j];
             }
+          if (join.any()) join.template to<V>(a, t, i, d);
           store_v<V>(Ht + static_cast<long long>(q) * d + i, a);
 #pragma unroll
           for (int j = 0; j < V; ++j) u[j] += s_read[q] * a[j];
@@ -137,6 +178,10 @@ stream_step_kernel(float* __restrict__ H, const T* __restrict__ y, const T* __re
 #pragma unroll
       for (int s = 0; s < NM; ++s)
         if (NS || s < n) {
+          if (join.any()) {
+            join.template to<V>(x[s], t, i, d);
+            store_v<V>(Ht + static_cast<long long>(s) * d + i, x[s]);
+          }
 #pragma unroll
           for (int j = 0; j < V; ++j) u[j] += s_read[s] * x[s][j];
         }
@@ -160,20 +205,20 @@ stream_step_kernel(float* __restrict__ H, const T* __restrict__ y, const T* __re
   const float r = 1.f / sqrtf(var + eps);
   for (int i = threadIdx.x * V; i < d; i += THREADS * V) {
     float c[V], o[V];
-    load_v<V>(w + i, c);
+    load_weight<T, V>(w, w_one, i, c);
 #pragma unroll
     for (int j = 0; j < V; ++j) o[j] = (su[i + j] - mean) * r * (around + c[j]);
     store_v<V>(normed + t * d + i, o);
   }
 }
 
-// One plain stream (H += gain (scale . y + scale2 . y2), y through its RMS norm where it has a weight, then the norm of H): the whole row in registers,
+// One plain stream (H += gain scale . y + gain2 scale2 . y2 and what joins, y through its RMS norm where it has a weight, then the norm of H): the whole row in registers,
 // NI pieces of V values a thread, every load in flight before the first sum.  TWO: y2 is there.
 template <typename T, int V, int NI, bool TWO>
 __global__ void __launch_bounds__(THREADS)
 residual_step_kernel(float* __restrict__ H, const T* __restrict__ y, const T* __restrict__ y_weight, const T* __restrict__ w, T* __restrict__ normed,
                      int d, float y_eps, float eps, const T* __restrict__ scale, const T* __restrict__ y2, const T* __restrict__ scale2, float gain,
-                     float around) {
+                     float gain2, float around, int w_one, Join<T> join) {
   __shared__ float red[32];
   const long long at = static_cast<long long>(blockIdx.x) * d;
   float x[NI][V], b[NI][V], b2[TWO ? NI : 1][V];
@@ -183,7 +228,7 @@ residual_step_kernel(float* __restrict__ H, const T* __restrict__ y, const T* __
 #pragma unroll
     for (int j = 0; j < V; ++j) x[p][j] = b[p][j] = 0.f;
     if (i < d) {
-      load_v<V>(y + at + i, b[p]);
+      if (y != nullptr) load_v<V>(y + at + i, b[p]);
       if (TWO) load_v<V>(y2 + at + i, b2[p]);
       load_v<V>(H + at + i, x[p]);
     }
@@ -217,14 +262,21 @@ residual_step_kernel(float* __restrict__ H, const T* __restrict__ y, const T* __
 #pragma unroll
           for (int j = 0; j < V; ++j) b[p][j] *= c[j];
         }
+#pragma unroll
+        for (int j = 0; j < V; ++j) b[p][j] *= gain;
         if (TWO) {
           if (scale2 != nullptr) load_v<V>(scale2 + i, c);
 #pragma unroll
-          for (int j = 0; j < V; ++j) b[p][j] += scale2 != nullptr ? c[j] * b2[p][j] : b2[p][j];
+          for (int j = 0; j < V; ++j) b[p][j] += gain2 * (scale2 != nullptr ? c[j] * b2[p][j] : b2[p][j]);
         }
-#pragma unroll
-        for (int j = 0; j < V; ++j) b[p][j] *= gain;
       }
+    }
+  }
+  if (join.any()) {
+#pragma unroll
+    for (int p = 0; p < NI; ++p) {
+      const int i = (p * THREADS + threadIdx.x) * V;
+      if (i < d) join.template to<V>(b[p], blockIdx.x, i, d);
     }
   }
   float ss = 0.f;
@@ -242,7 +294,7 @@ residual_step_kernel(float* __restrict__ H, const T* __restrict__ y, const T* __
     const int i = (p * THREADS + threadIdx.x) * V;
     if (i < d) {
       float c[V];
-      load_v<V>(w + i, c);
+      load_weight<T, V>(w, w_one, i, c);
 #pragma unroll
       for (int j = 0; j < V; ++j) c[j] = (around + c[j]) * x[p][j] * r;
       store_v<V>(normed + at + i, c);
@@ -338,13 +390,14 @@ int allow_smem(K kernel, size_t bytes) {
 
 template <typename T>
 int step(float* H, const T* y, const T* y_weight, const T* scale, const float* mix, const float* out, const float* read, const T* w, T* normed,
-         long long rows, int n, int d, float y_eps, float eps, int rms, const T* y2, const T* scale2, float gain, float around, cudaStream_t stream) {
-  const bool vec = aligned(y2, 4 * sizeof(T)) && aligned(scale2, 4 * sizeof(T)) && d % 4 == 0 && aligned(H, 16) && aligned(y, 4 * sizeof(T)) && aligned(y_weight, 4 * sizeof(T)) && aligned(scale, 4 * sizeof(T)) && aligned(w, 4 * sizeof(T)) &&
+         long long rows, int n, int d, float y_eps, float eps, int rms, const T* y2, const T* scale2, float gain, float gain2, float around, int w_one,
+         const Join<T>& join, cudaStream_t stream) {
+  const bool vec = aligned(join.add, 4 * sizeof(T)) && aligned(join.table, 4 * sizeof(T)) && aligned(y2, 4 * sizeof(T)) && aligned(scale2, 4 * sizeof(T)) && d % 4 == 0 && aligned(H, 16) && aligned(y, 4 * sizeof(T)) && aligned(y_weight, 4 * sizeof(T)) && aligned(scale, 4 * sizeof(T)) && (w_one || aligned(w, 4 * sizeof(T))) &&
                    aligned(normed, 4 * sizeof(T));
-  if (vec && n == 1 && rms && y != nullptr && mix == nullptr && out == nullptr && read == nullptr && d <= 32 * THREADS) {
+  if (vec && n == 1 && rms && (y != nullptr || join.any()) && mix == nullptr && out == nullptr && read == nullptr && d <= 32 * THREADS) {
     const int pieces = (d + THREADS * 4 - 1) / (THREADS * 4);
 #define DEWB_RES_T(NN, TT) residual_step_kernel<T, 4, NN, TT><<<static_cast<unsigned>(rows), THREADS, 0, stream>>>(H, y, y_weight, w, normed, d, y_eps, eps, \
-    scale, y2, scale2, gain, around)
+    scale, y2, scale2, gain, gain2, around, w_one, join)
 #define DEWB_RES(NN) do { if (y2 != nullptr) DEWB_RES_T(NN, true); else DEWB_RES_T(NN, false); } while (0)
     if (pieces <= 1) DEWB_RES(1); else if (pieces <= 2) DEWB_RES(2); else if (pieces <= 4) DEWB_RES(4); else DEWB_RES(8);
 #undef DEWB_RES
@@ -353,7 +406,7 @@ int step(float* H, const T* y, const T* y_weight, const T* scale, const float* m
   }
   const size_t smem = static_cast<size_t>(d) * 4;
 #define DEWB_STEP(VV, NN) do { const int r = allow_smem(stream_step_kernel<T, VV, NN>, smem); if (r) return r; \
-    stream_step_kernel<T, VV, NN><<<static_cast<unsigned>(rows), THREADS, smem, stream>>>(H, y, y_weight, scale, mix, out, read, w, normed, n, d, y_eps, eps, rms, y2, scale2, gain, around); } while (0)
+    stream_step_kernel<T, VV, NN><<<static_cast<unsigned>(rows), THREADS, smem, stream>>>(H, y, y_weight, scale, mix, out, read, w, normed, n, d, y_eps, eps, rms, y2, scale2, gain, gain2, around, w_one, join); } while (0)
   if (vec) {
     if (n == 1) DEWB_STEP(4, 1); else if (n == 2) DEWB_STEP(4, 2); else if (n == 3) DEWB_STEP(4, 3); else if (n == 4) DEWB_STEP(4, 4); else DEWB_STEP(1, 0);
   } else {
@@ -386,19 +439,25 @@ extern "C" int dewb_embed_streams(const long long* tokens, const int* positions,
 
 // H [rows, n, d] fp32, updated in place when `y` [rows, d] is given; normed [rows, d] (null: write only).  mix is indexed [from, to].  `mix`, `out`
 // and `read` may be null (each stream keeps itself, takes y, and is read with weight 1); y_weight [d]: y passes an RMS norm with that weight first.
-// `scale`, `scale2` [d], y2 [rows, d]: see stream_step above (null: absent); weights of the norm are `around` + w.
+// `scale`, `scale2` [d], y2 [rows, d]: see stream_step above (null: absent); weights of the norm are `around` + w, w [d] or (`w_one`) one number.  `add` [d]
+// and `table_gain` times `table` [vocab, d] at the row's token join the one stream (n 1) as well (null: neither).
 extern "C" int dewb_stream_step(float* H, const void* y, const void* y_weight, const void* scale, const float* mix, const float* out,
                                 const float* read, const void* w, void* normed, long long rows, int n, int d, float y_eps, float eps, int rms,
-                                const void* y2, const void* scale2, float gain, float around, int fp32, void* stream_ptr) {
+                                const void* y2, const void* scale2, float gain, float gain2, float around, int w_one, const void* add, const void* table,
+                                const long long* tokens, int vocab, float table_gain, int fp32, void* stream_ptr) {
   if (rows <= 0) return 0;
-  if (n < 1 || n > MAX_STREAMS || d < 1 || (y == nullptr && (y_weight != nullptr || y2 != nullptr)) || (y_weight != nullptr && y2 != nullptr) || (normed != nullptr && w == nullptr)) return -3;
+  if (n < 1 || n > MAX_STREAMS || d < 1 || (y == nullptr && (y_weight != nullptr || y2 != nullptr)) || (y_weight != nullptr && y2 != nullptr) || (normed != nullptr && w == nullptr) ||
+      ((add != nullptr || table != nullptr) && n != 1) || (table != nullptr && (tokens == nullptr || vocab < 1)))
+    return -3;
   cudaStream_t stream = reinterpret_cast<cudaStream_t>(stream_ptr);
   if (fp32) return step<float>(H, static_cast<const float*>(y), static_cast<const float*>(y_weight), static_cast<const float*>(scale), mix, out, read,
                                static_cast<const float*>(w), static_cast<float*>(normed), rows, n, d, y_eps, eps, rms, static_cast<const float*>(y2),
-                               static_cast<const float*>(scale2), gain, around, stream);
+                               static_cast<const float*>(scale2), gain, gain2, around, w_one,
+                               Join<float>{static_cast<const float*>(add), static_cast<const float*>(table), tokens, vocab, table_gain}, stream);
   return step<bf16>(H, static_cast<const bf16*>(y), static_cast<const bf16*>(y_weight), static_cast<const bf16*>(scale), mix, out, read,
                     static_cast<const bf16*>(w), static_cast<bf16*>(normed), rows, n, d, y_eps, eps, rms, static_cast<const bf16*>(y2),
-                    static_cast<const bf16*>(scale2), gain, around, stream);
+                    static_cast<const bf16*>(scale2), gain, gain2, around, w_one,
+                    Join<bf16>{static_cast<const bf16*>(add), static_cast<const bf16*>(table), tokens, vocab, table_gain}, stream);
 }
 
 // x [rows, n] -> out [rows, n] fp32

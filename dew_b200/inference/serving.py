@@ -303,11 +303,10 @@ class Server:
         if any_live:
             if self.cuda_graph and greedy:
                 if self._graph is None:
-                    kept = [None if t is None else t.clone() for t in self.store.states]
+                    kept = [(t, t.clone()) for t in self.store.kept_states()]
                     self._decode_program(True)                      # warm-up (allocations, lazy initialisation)
-                    for t, old in zip(self.store.states, kept):     # a recurrent state, unlike a cache slot, must not take the token twice
-                        if t is not None:
-                            t.copy_(old)
+                    for t, old in kept:                             # a recurrent state, unlike a cache slot, must not take the token twice
+                        t.copy_(old)
                     torch.cuda.synchronize()
                     # the warm-up advanced the cache by one token for every row; replaying the same positions
                     # rewrites the same slots with the same values, so the cache stays consistent

@@ -151,11 +151,13 @@ class Pretrained:
     def load(directory: os.PathLike, dtype=None, device="cpu", strict: bool = True):
         """A ``CausalTransformer`` for the families of ``interop.families``; a ``ClassicDecoder`` for the older lineage of
         ``interop.classic`` (GPT-2, GPT-NeoX, Falcon, Phi, OPT, BLOOM, StarCoder2, GPTBigCode); Mamba and Mamba-2 releases through
-        ``interop.recurrent``; Ragenex, Fakonex and Selivik through ``interop.ragenex``, ``interop.fakonex`` and ``interop.selivik``."""
+        ``interop.recurrent``; Ragenex, Fakonex, Selivik and Rarelorn through ``interop.ragenex``, ``interop.fakonex``, ``interop.selivik`` and
+        ``interop.rarelorn``."""
         from .classic import CLASSIC, load_classic_state, read_classic_config
         from .families import family_of, load_state, read_config
         from .fakonex import is_fakonex, load_fakonex_state, read_fakonex_config
         from .ragenex import is_ragenex, load_ragenex_state, read_ragenex_config
+        from .rarelorn import is_rarelorn, load_rarelorn_state, read_rarelorn_config
         from .release import GenerationConfig, Release
         from .selivik import is_selivik, load_selivik_state, read_selivik_config
         rel = Release(directory, dtype=dtype or torch.bfloat16)
@@ -169,7 +171,8 @@ class Pretrained:
             return model
         for name, mine, read, load in (("ragenex", is_ragenex, read_ragenex_config, load_ragenex_state),
                                        ("fakonex", is_fakonex, read_fakonex_config, load_fakonex_state),
-                                       ("selivik", is_selivik, read_selivik_config, load_selivik_state)):
+                                       ("selivik", is_selivik, read_selivik_config, load_selivik_state),
+                                       ("rarelorn", is_rarelorn, lambda cfg: read_rarelorn_config(cfg, rel), load_rarelorn_state)):
             if mine(rel.config):
                 model = CausalTransformer(read(rel.config), dtype=dtype, device=device)
                 model.unread_keys = load(model, rel, strict=strict)
@@ -196,7 +199,7 @@ class Pretrained:
         from .families import FAMILIES, export_state, write_config
         from .release import save_release
         dtype = str(next(model.parameters()).dtype).replace("torch.", "")
-        if family is None and getattr(model, "family", None) in ("ragenex", "fakonex", "selivik"):
+        if family is None and getattr(model, "family", None) in ("ragenex", "fakonex", "selivik", "rarelorn"):
             family = model.family
         if family == "ragenex":
             from .ragenex import export_ragenex_state, write_ragenex_config
@@ -209,6 +212,10 @@ class Pretrained:
         if family == "selivik":
             from .selivik import export_selivik_state, write_selivik_config
             save_release(export_selivik_state(model), write_selivik_config(model.config), directory, max_shard_bytes, generation, fp8_blocks)
+            return
+        if family == "rarelorn":
+            from .rarelorn import export_rarelorn_state, write_rarelorn_config
+            save_release(export_rarelorn_state(model), write_rarelorn_config(model.config), directory, max_shard_bytes, generation, fp8_blocks)
             return
         if family is None:
             family = next((f.name for f in FAMILIES.values() if f.architecture == architecture), None)

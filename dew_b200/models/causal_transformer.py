@@ -49,7 +49,8 @@ class Mixture:
     fp8: Any = False                                 # True: block-scaled MXFP8 expert GEMMs (1 x 32 blocks); 'row': row / channel scaled e4m3
     balance_rate: float = 1e-3
     groups: int = 1                                  # DeepSeek-V3's group-limited routing: experts in ``groups`` groups ...
-    topk_groups: int = 1                             # ... of which each token may use the ``topk_groups`` best (by their top-2 sum)
+    topk_groups: int = 1                             # ... of which each token may use the ``topk_groups`` best (by the sum of their ...
+    group_best: int = 2                              # ... ``group_best`` best scores: 2 or 1)
     group_fill: float = 0.0                          # choice score of the experts outside those groups (choice scores can be negative: -inf rules them out)
     style: str = "swiglu"                            # 'clamped_glu': GPT-OSS's biased router over the top logits and biased clamped-GLU experts
 
@@ -67,12 +68,21 @@ class Loop:
     backprop_steps: Optional[int] = None
     messages: int = 0                # n > 0: cross-pass messages - every pass starts from the prelude's output and reads the summaries the pass
     message_rank: int = 16           # before left of every block of n looped layers, merged into each sub-layer's input (nn/cross_pass.py)
+    restate: bool = False            # the embedding output joins the residual again in front of every pass but the first (fp32 residual)
+    step_vectors: bool = False       # a learned vector of each pass joins the residual in front of it (fp32 residual)
 
     def __post_init__(self):
         if self.steps < 1 or self.first < 0 or (self.end is not None and self.end <= self.first):
             raise ValueError("a loop runs layers [first, end) at least once")
+        if (self.restate or self.step_vectors) and (self.exit_gate or self.messages):
+            raise NotImplementedError("what joins in front of a pass is built for loops without exit gates and messages")
         if self.backprop_steps is not None and not 1 <= self.backprop_steps <= self.steps:
             raise ValueError("backprop_steps counts the last passes that carry a gradient: between 1 and steps")
+
+
+    @property
+    def joins(self) -> bool:
+        return self.restate or self.step_vectors
 
 
 @dataclass
@@ -94,7 +104,7 @@ class TransformerConfig:
     attn_softcap: float = 0.0
     logit_softcap: float = 0.0
     window: Optional[int] = None
-    layer_types: Optional[Sequence[str]] = None      # per layer: attention | local | nope | gdn | mamba2 | mamba | mamba3 | kda | mla | lightning | differential | forgetting | gla | delta | rwkv7 | memory | none
+    layer_types: Optional[Sequence[str]] = None      # per layer: attention | local | nope | gdn | mamba2 | mamba | mamba3 | kda | mla | lightning | mlstm | rwkv6 | pair | differential | forgetting | gla | delta | rwkv7 | memory | none
     mixture: Optional[Mixture] = None
     mixer_options: Dict[str, Any] = field(default_factory=dict)
     remat: bool = False
@@ -138,6 +148,10 @@ class TransformerConfig:
     qk_unit_norm: bool = False                        # q and k over their root mean square per head, after the rotation and without a weight
     parallel_block: bool = False                      # a layer's mixer and MLP read one norm and join the residual together
     norm_around: float = 0.0                          # the weights of the residual's norms are stored as their distance from this
+    norm_one: bool = False                            # the weights of the residual's norms are one number each
+    attn_conv: int = 0                                # q, k and v pass a causal convolution of this many taps per channel, in front of the rotation
+    attn_weighting: str = "softmax"                   # sigmoid: a visible key weighs the sigmoid of its score plus a number per head
+    attn_head_temperature: bool = False               # a head's scores times a learned number of its own
     layer_options: Optional[Sequence[Optional[Mapping]]] = None    # per layer, what differs from the fields above: LAYER_OPTIONS, and decay (lightning)
 
     def __post_init__(self):
@@ -158,6 +172,12 @@ class TransformerConfig:
         elif self.norm != "rms" or self.layer_scale or self.learned_positions or self.parallel_block or self.norm_around:
             raise NotImplementedError("layer norms, layer scale, learned positions, parallel blocks and norm weights stored around a value belong to the "
                                       "static-stream stack (hyper_connections >= 1 with hyper_dynamic=False, or fp32_residual)")
+            if self.norm_one and (self.norm != "rms" or self.static_streams):
+                raise NotImplementedError("norms with one number for all coordinates are RMS norms of the fp32 residual")
+            if self.loop is not None and self.static_streams and (Loop(**self.loop) if isinstance(self.loop, Mapping) else self.loop).joins:
+                raise NotImplementedError("what joins in front of a pass is built for one plain residual")
+        elif self.norm_one or (self.loop is not None and (Loop(**self.loop) if isinstance(self.loop, Mapping) else self.loop).joins):
+            raise NotImplementedError("norms with one number and what joins in front of a loop's passes belong to fp32_residual")
         if self.kv_from is not None and self.layer_options is not None:
             raise ValueError("kv_from belongs to a layer: give it in layer_options")
         if isinstance(self.mixture, Mapping):             # a run record (JSON) carries the mixture as a plain mapping
@@ -195,7 +215,7 @@ class TransformerConfig:
 
 
 LAYER_OPTIONS = frozenset({"num_heads", "num_kv_heads", "head_dim", "value_dim", "query_scale", "query_temperature", "attn_chunk", "kv_from", "window", "keep_first",
-                           "attn_softcap", "rotation", "attention_sinks", "qkv_bias", "qk_unit_norm", "mlp_features", "mlp_limit", "mlp_activation", "mixture",
+                           "attn_softcap", "rotation", "attention_sinks", "attn_bias", "attn_conv", "attn_weighting", "attn_head_temperature", "qkv_bias", "qk_unit_norm", "mlp_features", "mlp_limit", "mlp_activation", "mixture",
                            "mixer_options"})
 ROTARY_KINDS = ("attention", "local", "nope", "mla", "differential", "forgetting")      # mixers called with the rotary tables and positions
 
@@ -208,14 +228,15 @@ def _mixer(cfg: TransformerConfig, kind: str, dtype, device, index: int = 0) -> 
                           init_std=cfg.init_std, qkv_bias=cfg.qkv_bias, scale=cfg.query_scale, qk_norm_full=cfg.qk_norm_full,
                           out_gate=cfg.attn_out_gate, value_dim=cfg.value_dim, temperature=cfg.query_temperature,
                           chunk=cfg.attn_chunk, head_gate=cfg.attn_head_gate, own_kv=cfg.kv_from is None, rotation=cfg.rotation if kind != "nope" else None, keep_first=cfg.keep_first, unit_qk=cfg.qk_unit_norm,
-                          dtype=dtype, device=device)
+                          conv=cfg.attn_conv, weighting=cfg.attn_weighting, head_temperature=cfg.attn_head_temperature, dtype=dtype, device=device)
         a.rotary = kind != "nope" and cfg.rotation is None      # SmolLM3's every fourth layer attends without positions
         if kind == "local" and cfg.local_rope_theta is not None:
             a.own_rope = (float(cfg.local_rope_theta), None)
         return a
     if kind == "gdn":
         from ..nn.linear_attention import GatedDeltaNet
-        return GatedDeltaNet(cfg.emb_features, dtype=dtype, device=device, **cfg.mixer_options)
+        own = {"norm_eps": cfg.norm_eps} if cfg.fp32_stack else {}             # (elsewhere the heads' norm keeps its default unless the options say otherwise)
+        return GatedDeltaNet(cfg.emb_features, dtype=dtype, device=device, **{**own, **cfg.mixer_options})
     if kind == "mamba2":
         from ..nn.mamba2 import Mamba2
         return Mamba2(cfg.emb_features, dtype=dtype, device=device, **cfg.mixer_options)
@@ -234,6 +255,22 @@ def _mixer(cfg: TransformerConfig, kind: str, dtype, device, index: int = 0) -> 
     if kind == "lightning":
         from ..nn.recurrent_mixers import LightningAttention
         return LightningAttention(cfg.emb_features, layers=cfg.num_layers, norm_eps=cfg.norm_eps, dtype=dtype, device=device, **cfg.mixer_options)
+    if kind == "mlstm":
+        from ..nn.recurrent_mixers import MatrixMemory
+        return MatrixMemory(cfg.emb_features, norm_eps=cfg.norm_eps, dtype=dtype, device=device, **cfg.mixer_options)
+    if kind == "rwkv6":
+        from ..nn.recurrent_mixers import RWKV6
+        return RWKV6(cfg.emb_features, norm_eps=cfg.norm_eps, dtype=dtype, device=device, **cfg.mixer_options)
+    if kind == "pair":
+        # mixer_options: {'left' | 'right': (kind, what differs from this configuration), 'left_scale' | 'right_scale': factors}
+        from ..nn.mixer_pair import MixerPair
+        o = dict(cfg.mixer_options)
+        (lk, lo), (rk, ro) = o.pop("left"), o.pop("right")
+        side = lambda k, d: _mixer(replace(cfg, layer_options=None, layer_types=(k,), **{"mixer_options": {}, **d}), k, dtype, device, index)
+        pair = MixerPair(side(lk, lo), side(rk, ro), lk in ROTARY_KINDS, rk in ROTARY_KINDS, **o)
+        if any(r and getattr(m, "rotary", True) for m, r in zip((pair.left, pair.right), pair.rotary)):
+            raise NotImplementedError("mixers side by side carry their own rotation, or none ('nope')")
+        return pair
     if kind == "mamba3":
         from ..nn.recurrent_mixers import Mamba3
         return Mamba3(cfg.emb_features, dtype=dtype, device=device, **cfg.mixer_options)
@@ -252,14 +289,14 @@ def _mixer(cfg: TransformerConfig, kind: str, dtype, device, index: int = 0) -> 
     if kind == "rwkv7":
         from ..nn.linear_mixers import RWKV7
         return RWKV7(cfg.emb_features, layer_index=0, **({"num_heads": cfg.num_heads, **cfg.mixer_options})).to(device=device, dtype=dtype)
-    raise ValueError(f"unknown layer type {kind!r}; known: attention, local, gdn, mamba2, mamba, mamba3, kda, mla, lightning, differential, forgetting, "
+    raise ValueError(f"unknown layer type {kind!r}; known: attention, local, gdn, mamba2, mamba, mamba3, kda, mla, lightning, mlstm, rwkv6, pair, differential, forgetting, "
                      "gla, delta, rwkv7")
 
 
 def _norm_of(cfg: TransformerConfig, dtype, device) -> nn.Module:
     if cfg.norm == "layer":
         return LayerNorm(cfg.emb_features, cfg.norm_eps, bias=False, dtype=dtype, device=device)
-    return RMSNorm(cfg.emb_features, cfg.norm_eps, dtype=dtype, device=device, around=cfg.norm_around)
+    return RMSNorm(cfg.emb_features, cfg.norm_eps, dtype=dtype, device=device, around=cfg.norm_around, one=cfg.norm_one)
 
 
 class _NoNorm(nn.Module):
@@ -352,7 +389,12 @@ class DecoderLayer(nn.Module):
             stack.leave(None, self._mix(n, cos, sin, positions, segment_ids, cache, slot), scale[0], gain=gain, beside=self._feed_forward(n, positions, True),
                         beside_scale=scale[1])
             return
-        if self.mixer is not None:
+        if self.kind == "pair" and self.mixer_out_norm is None:
+            n = stack.enter(streams[q], self.input_norm)
+            a, b = self.mixer.branches(n, None, cache, slot, positions)
+            stack.leave(streams[q], a, scale[q], None, gain * self.mixer.left_scale, b, scale[q], gain * self.mixer.right_scale)
+            q += 1
+        elif self.mixer is not None:
             n = stack.enter(streams[q], self.input_norm)
             stack.leave(streams[q], self._mix(n, cos, sin, positions, segment_ids, cache, slot), scale[q], self.mixer_out_norm, gain)
             q += 1
@@ -463,6 +505,8 @@ class CausalTransformer(nn.Module):
         self.final_norm = _norm_of(cfg, dtype, device)
         self.head = None if cfg.tie_embeddings else Linear(cfg.emb_features, cfg.vocab_size, axes=("embed", "vocab"),
                                                            init_std=cfg.init_std, dtype=dtype, device=device)
+        self.pass_vectors = declare(nn.Parameter(torch.zeros(cfg.loop.steps, cfg.emb_features, dtype=dtype, device=device)), (None, "embed"), "scale") \
+            if cfg.loop is not None and cfg.loop.step_vectors else None
         self.mtp = nn.ModuleList([MTPBlock(cfg, i, dtype, device) for i in range(cfg.mtp_depth)]) if cfg.mtp_depth > 0 else None
         self.early_exit_gate = Linear(cfg.emb_features, 1, bias=True, init_std=cfg.init_std, dtype=dtype, device=device) \
             if cfg.loop is not None and cfg.loop.exit_gate else None
@@ -539,17 +583,19 @@ class CausalTransformer(nn.Module):
         if not (cfg.fp32_stack or cfg.layer_options is not None or cfg.query_temperature is not None or cfg.value_dim is not None or cfg.attn_chunk is not None
                 or cfg.attn_head_gate or cfg.rotation is not None or cfg.keep_first or cfg.qk_unit_norm):
             return None
-        if any(self._wants_tables(i) or k not in ("nope", "attention", "local", "mla", "lightning", "none") for i, k in enumerate(kinds)):
-            raise NotImplementedError("per-layer caches are built for attention without rotation ('nope') or with one of its own, 'mla' with one of its own and "
-                                      f"'lightning' layers, not {sorted(set(kinds))}")
+        if any(self._wants_tables(i) or not (k in ("mla", "lightning", "none") or hasattr(self.layers[i].mixer, "cache_slot")) for i, k in enumerate(kinds)):
+            raise NotImplementedError("per-layer caches are built for attention without rotation ('nope') or with one of its own, 'mla' with one of its own, "
+                                      f"'lightning', 'gdn', 'mlstm', 'rwkv6' and 'pair' layers, not {sorted(set(kinds))}")
         out, latest = [], {}
         for i, slot in self.runs():
             m = self.layers[i].mixer
             if kinds[i] == "mla":
                 out.append(CacheSlot(1, m.shape.row, m.shape.rank, latent=True))
             elif kinds[i] in ("nope", "attention", "local"):
-                out.append(CacheSlot(m.num_kv_heads, m.head_dim, m.value_dim, source=None if m.own_kv else latest[cfg.of_layer(i).kv_from]))
+                out.append(m.cache_slot(None if m.own_kv else latest[cfg.of_layer(i).kv_from]))
                 latest[i] = slot if m.own_kv else out[-1].source
+            elif hasattr(m, "cache_slot"):
+                out.append(m.cache_slot())
             else:
                 out.append(CacheSlot(state=(0,) if m is None else (m.h, m.d, m.dv)))
         return out
@@ -668,8 +714,10 @@ class CausalTransformer(nn.Module):
         if pos is not None and cache is None and tokens.shape[1] > pos.shape[0]:
             raise ValueError(f"{tokens.shape[1]} tokens do not fit the {pos.shape[0]} learned positions")
         runs = self.runs(steps)
+        if self.pass_vectors is not None and steps is not None and steps != cfg.loop.steps:
+            raise NotImplementedError(f"the loop has vectors for {cfg.loop.steps} passes")
         if cache is not None:
-            if len(getattr(cache, "slots", None) or ()) != len(self.runs()):
+            if getattr(cache, "layer_runs", 0) != len(self.runs()):
                 raise ValueError("this decoder's layers differ in what they keep: its cache comes from sampling.text.make_cache")
             if positions is None:
                 positions = torch.arange(tokens.shape[1], device=tokens.device)[None].expand(tokens.shape[0], -1)
@@ -682,7 +730,14 @@ class CausalTransformer(nn.Module):
         H = ops_streams.embed_streams(tokens, positions, self.embed.weight, pos, max(1, cfg.hyper_connections), gain)
         stack = StreamStack(H, self.embed.weight.dtype)
         cos, sin = self.rope_tables(H.device) if any(self._wants_tables(i) for i in range(len(self.layers))) else (None, None)
+        loop, passes = cfg.loop, 0
         for r, (i, slot) in enumerate(runs):
+            if loop is not None and loop.joins and i == loop.first:              # a pass begins
+                table = self.embed.weight if loop.restate and passes > 0 else None
+                vector = self.pass_vectors[passes] if self.pass_vectors is not None else None
+                if table is not None or vector is not None:
+                    stack.join(ops_streams.Join(vector, table, tokens, gain))
+                passes += 1
             self.layers[i].forward_static(stack, cos, sin, positions, None, cache, slot)
             if observe is not None:
                 observe(r, stack.total())

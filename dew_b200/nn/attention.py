@@ -11,6 +11,7 @@ import torch.nn as nn
 
 from .. import ops
 from ..ops import paged as P
+from ..ops import token_mix
 from .layers import Linear, RMSNorm, declare
 
 
@@ -20,7 +21,8 @@ class SelfAttention(nn.Module):
                  softcap: float = 0.0, sinks: bool = False, norm_eps: float = 1e-6, out_zero_init: bool = False,
                  init_std: Optional[float] = None, qkv_bias: bool = False, scale: Optional[float] = None, qk_norm_full: bool = False,
                  out_gate: bool = False, value_dim: Optional[int] = None, temperature=None, chunk: Optional[int] = None, head_gate: bool = False,
-                 own_kv: bool = True, rotation=None, keep_first: int = 0, unit_qk: bool = False, dtype=None, device=None):
+                 own_kv: bool = True, rotation=None, keep_first: int = 0, unit_qk: bool = False, conv: int = 0, weighting: str = "softmax",
+                 head_temperature: bool = False, dtype=None, device=None):
         super().__init__()
         self.features, self.num_heads = features, num_heads
         # a softmax scale other than head_dim ** -0.5 is folded into the queries (after the norm and the rotation)
@@ -38,6 +40,13 @@ class SelfAttention(nn.Module):
         # rotation: the layer's own (``ops.rotary.Rotary``) in place of the model's tables; keep_first: keys from the row's start that a window leaves
         # visible; unit_qk: q and k over their root mean square per head, after the rotation and without a weight
         self.rotation, self.keep_first, self.unit_qk = rotation, int(keep_first), unit_qk
+        # conv: q, k and v pass a causal convolution of that many taps per channel, behind the projection's bias; weighting 'sigmoid': a visible key weighs
+        # the sigmoid of its score plus a number per head, with no sum over the keys; head_temperature: a head's scores times a number of its own
+        self.weighting = weighting
+        if weighting not in ("softmax", "sigmoid"):
+            raise ValueError(f"unknown attention weighting {weighting!r}; known: softmax, sigmoid")
+        if weighting == "sigmoid" and sinks:
+            raise ValueError("a sink joins a softmax's denominator: sigmoid weights have none")
         if keep_first and window is None:
             raise ValueError("keep_first belongs to a window")
         if unit_qk and (qk_norm or qk_norm_full):
@@ -50,6 +59,14 @@ class SelfAttention(nn.Module):
         # the gates have no bias
         self.heads_bias = declare(nn.Parameter(torch.zeros(self.heads.packed, dtype=dtype, device=device)), ("heads",), "bias") \
             if (bias or qkv_bias) and head_gate else None
+        if conv and not (own_kv and not head_gate and causal):
+            raise NotImplementedError("a convolution on q, k and v is built for layers with keys and values of their own and without head gates")
+        self.conv = None
+        if conv:
+            from .linear_attention import ShortConv
+            self.conv = ShortConv(self.heads.packed, conv, activation=False, dtype=dtype, device=device)
+        per_head = lambda there, value: declare(nn.Parameter(torch.full((num_heads,), value, dtype=dtype, device=device)), ("heads",), "scale") if there else None
+        self.head_temperature, self.score_bias = per_head(head_temperature, 1.0), per_head(weighting == "sigmoid", 0.0)
         self.o_proj = Linear(self.num_heads * self.value_dim, features, bias=bias, axes=("heads", "embed"),
                              init_std=init_std, zero_init=out_zero_init, dtype=dtype, device=device)
         # Qwen3-Next: the heads' outputs pass a sigmoid gate computed from the layer's input, before the output projection
@@ -65,6 +82,11 @@ class SelfAttention(nn.Module):
         self.head_transform = None     # a module applied to the heads' outputs [B, S, H, D] before the output projection (dew_b200.nn.dex)
         self.track_qk_max = False      # set by dew_b200.optim.qk_clip.watch: record each head's largest attention logit
         self.qk_max: Optional[torch.Tensor] = None
+
+    def cache_slot(self, source: Optional[int] = None):
+        from .kv_cache import CacheSlot
+        more = () if self.conv is None or self.conv.kernel_size < 2 else (("conv", (self.heads.packed, self.conv.kernel_size - 1)),)
+        return CacheSlot(self.num_kv_heads, self.head_dim, self.value_dim, source=source, more=more)
 
     @torch.no_grad()
     def _record_qk_max(self, q, k):
@@ -125,15 +147,20 @@ class SelfAttention(nn.Module):
         qkv = ops.linear(x, self.qkv_proj.weight) if type(self.qkv_proj) is Linear and self.qkv_proj.bias is not None else self.qkv_proj(x)
         bias = self.qkv_proj.bias if type(self.qkv_proj) is Linear and self.qkv_proj.bias is not None else self.heads_bias
         cache = Uncached(()) if cache is None else cache
+        if self.conv is not None:
+            kept = getattr(cache, "more", None)
+            rows = cache.call(positions).rows if kept is not None else None
+            qkv, bias = token_mix.conv_tokens(qkv, self.conv.weight, bias, False, rows, None if kept is None else kept[layer].get("conv")), None
         o = cache.attend_slot(layer, qkv, self.heads, positions, scale=self.scale, eps=eps, q_weight=qw, k_weight=kw, temperature=self.temperature,
                               bias=bias, chunk=self.chunk, sinks=self.sinks, window=self.window, keep=self.keep_first, softcap=self.softcap, rot=self.rotation,
-                              unit=self.unit_qk)
+                              unit=self.unit_qk, gain=self.head_temperature, sigmoid=self.score_bias)
         return self.o_proj(o.reshape(B, S, self.num_heads * self.value_dim))
 
     def forward(self, x, cos=None, sin=None, positions=None, segment_ids=None, cache=None, layer: int = 0):
         B, S, _ = x.shape
         if getattr(cache, "slots", None) is not None or self.temperature is not None or self.value_dim != self.head_dim or self.chunk is not None \
-                or self.head_gate or not self.own_kv or self.rotation is not None or self.keep_first or self.unit_qk:
+                or self.head_gate or not self.own_kv or self.rotation is not None or self.keep_first or self.unit_qk or self.conv is not None \
+                or self.weighting != "softmax" or self.head_temperature is not None:
             return self._general(x, positions, segment_ids, cache, layer)
         cos, sin = self._tables(cos, sin)
         if (cache is None and x.is_cuda and cos is not None and self.head_transform is None and self.gate_proj is None and self.q_norm is None and self.window is None and not self.softcap

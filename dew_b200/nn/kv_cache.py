@@ -22,7 +22,7 @@ from .. import ops
 from ..ops import latent as M
 from ..ops import library as L
 from ..ops import paged as P
-from ..ops import rotary
+from ..ops import rotary, token_mix
 
 LIMITS = {"int8": 127.0, "float8_e4m3fn": 448.0}
 KINDS = {None: 0, "int8": 1, "float8_e4m3fn": 2}
@@ -44,13 +44,22 @@ class KVCache:
 @dataclass(frozen=True)
 class CacheSlot:
     """What one run of a layer keeps per row: keys and values of its own head count and widths (with ``latent``, rows of which the first ``value_dim``
-    columns are the values too), a recurrent state (a shape, fp32), or nothing: it reads the keys and values of the earlier slot ``source``."""
+    columns are the values too), a recurrent state (a shape, fp32), or nothing: it reads the keys and values of the earlier slot ``source``.  ``more`` names
+    further fp32 tensors of a row (the inputs a convolution still needs, a normaliser); ``beside`` is what a second mixer of the same layer keeps, in a slot
+    of its own behind those of the layers (``KVStore.beside``)."""
     kv_heads: int = 0
     head_dim: int = 0
     value_dim: int = 0
     state: Optional[Tuple[int, ...]] = None
     source: Optional[int] = None
     latent: bool = False
+    more: Tuple[Tuple[str, Tuple[int, ...]], ...] = ()
+    beside: Optional["CacheSlot"] = None
+
+    @property
+    def stateful(self) -> bool:
+        """Whether a row keeps something here that no page holds."""
+        return self.state is not None or bool(self.more)
 
 
 @dataclass
@@ -68,6 +77,10 @@ class Call:
     fresh: Optional[bool] = None             # every row starts at its first token (None: not looked at)
     kept: Dict[int, torch.Tensor] = field(default_factory=dict)      # slot -> this call's packed heads, while later layers read its keys and values
     angles: Dict[rotary.Rotary, torch.Tensor] = field(default_factory=dict)
+
+    @property
+    def rows(self) -> token_mix.Rows:
+        return token_mix.Rows(self.positions, self.lengths, self.row_ids)
 
     def turned(self, rot: Optional[rotary.Rotary]) -> Optional[P.Turned]:
         if rot is None:
@@ -127,6 +140,12 @@ class KVStore:
                  dtype=torch.bfloat16, device="cpu", slots: Optional[Sequence[CacheSlot]] = None):
         self.spec = spec
         self.slots = None if slots is None else list(slots)
+        self.layer_runs = 0 if slots is None else len(self.slots)
+        self.beside: Dict[int, int] = {}             # slot of a layer run -> slot of the second mixer's share of it
+        for i in range(self.layer_runs):
+            if self.slots[i].beside is not None:
+                self.beside[i] = len(self.slots)
+                self.slots.append(self.slots[i].beside)
         self.layers, self.rows, self.max_len, self.kv_heads, self.head_dim = layers, rows, max_len, kv_heads, head_dim
         self.page_size = spec.page_size or max_len
         self.max_pages = (max_len + self.page_size - 1) // self.page_size
@@ -136,6 +155,7 @@ class KVStore:
         # one page beyond the addressable pool: writes of padding positions land there, so that a write needs no data-dependent
         # shapes (and therefore no host synchronisation); no page table entry ever names it
         self.states: List[Optional[torch.Tensor]] = []
+        self.more: List[Dict[str, torch.Tensor]] = []
         self._call: Optional[Call] = None
         if self.slots is not None:
             if self.kind:
@@ -153,6 +173,7 @@ class KVStore:
                         pools[i] = pools[s.source]
             self.last_reader = {s.source: i for i, s in enumerate(self.slots) if s.source is not None}
             self.states = [None if s.state is None else torch.zeros(rows, *s.state, dtype=torch.float32, device=device) for s in self.slots]
+            self.more = [{n: torch.zeros(rows, *shape, dtype=torch.float32, device=device) for n, shape in s.more} for s in self.slots]
             self.k_scale = self.v_scale = None
         else:
             shape = (layers, self.pages + 1, self.page_size, kv_heads, head_dim)
@@ -173,7 +194,11 @@ class KVStore:
     @property
     def keeps_state(self) -> bool:
         """Whether some layer keeps a state (which no page holds: a prompt's prefix cannot be taken from another row's pages)."""
-        return any(s.state is not None for s in self.slots or ())
+        return any(s.stateful for s in self.slots or ())
+
+    def kept_states(self) -> List[torch.Tensor]:
+        """Every tensor of the store that a step moves on instead of adding to."""
+        return [t for t in self.states if t is not None] + [t for named in self.more for t in named.values()]
 
     def call(self, positions: torch.Tensor) -> Call:
         """The integers of the call whose layers pass ``positions [R, S]``: made by the first layer, found by the others."""
@@ -199,7 +224,8 @@ class KVStore:
 
     def attend_slot(self, slot: int, qkv: torch.Tensor, heads: P.Heads, positions: torch.Tensor, *, scale: float, eps: float = 1e-6, q_weight=None,
                     k_weight=None, temperature=None, bias=None, chunk: Optional[int] = None, sinks: Optional[torch.Tensor] = None,
-                    window: Optional[int] = None, keep: int = 0, softcap: float = 0.0, rot: Optional[rotary.Rotary] = None, unit: bool = False) -> torch.Tensor:
+                    window: Optional[int] = None, keep: int = 0, softcap: float = 0.0, rot: Optional[rotary.Rotary] = None, unit: bool = False,
+                    gain: Optional[torch.Tensor] = None, sigmoid: Optional[torch.Tensor] = None) -> torch.Tensor:
         """A layer's attention from its packed projection ``qkv [R, S, heads.row]``: bias, norms, rotation, temperature, append, causal attention
         against everything the rows hold (or what ``paged.Visible`` leaves of it, times the heads' gates).  -> ``[R, S, H, dv]``.  A
         prompt from its first token takes the tcgen05 flash kernel, a decode step the paged decode kernels, anything else (and fp32) the
@@ -211,7 +237,8 @@ class KVStore:
         pages = P.Pages(self.k[slot], self.v[slot], self.page_table, self.page_size, c.row_ids)
         packed = P.qk_norm_append(qkv, heads, q_weight, k_weight, eps, temperature, c.positions, pages, bias, c.turned(rot), unit)
         gate = qkv[..., heads.packed:] if heads.gated else None
-        visible = P.Visible(chunk, None if sinks is None else self._fp32_sinks(slot, sinks), window, keep if window else 0, softcap)
+        fp32 = lambda name, t: None if t is None else self._fp32_of(slot, name, t)
+        visible = P.Visible(chunk, fp32("sinks", sinks), window, keep if window else 0, softcap, fp32("gain", gain), fp32("sigmoid", sigmoid))
         R, S = positions.shape
         H, G = heads.q, heads.kv
         D = packed.shape[-1]
@@ -228,23 +255,25 @@ class KVStore:
                     c.kept.pop(source, None)
                 if kv is not None:
                     out, _ = flash_fwd(q, kv[:, :, :G], kv[:, :, G:], True, scale, need_lse=False, var=Variants(visible.window, softcap, visible.sinks, chunk=chunk,
-                                                                                                                keep=visible.keep))
+                                                                                                                keep=visible.keep, gain=visible.gain,
+                                                                                                                sigmoid=visible.sigmoid))
                     return P.head_gate(out, gate, heads.dv)
         return P.paged_attend(q, heads, c.positions, pages, scale, visible=visible, gate=gate)
 
-    def _fp32_sinks(self, slot: int, sinks: torch.Tensor) -> torch.Tensor:
-        """A layer's sinks as the kernels take them, converted once (again when the parameter changes)."""
-        bank = self.__dict__.setdefault("_sinks_of", {})
-        key = (sinks.data_ptr(), sinks._version)
-        if slot not in bank or bank[slot][0] != key:
-            bank[slot] = (key, sinks.detach().float().contiguous())
-        return bank[slot][1]
+    def _fp32_of(self, slot: int, name: str, t: torch.Tensor) -> torch.Tensor:
+        """A layer's numbers per head (sinks, factors, biases) as the kernels take them, converted once (again when the parameter changes)."""
+        bank = self.__dict__.setdefault("_per_head", {})
+        key = (t.data_ptr(), t._version)
+        if (slot, name) not in bank or bank[slot, name][0] != key:
+            bank[slot, name] = (key, t.detach().float().contiguous())
+        return bank[slot, name][1]
 
     def _decode_slot(self, slot: int, packed: torch.Tensor, heads: P.Heads, c: Call, scale: float, visible: P.Visible = P.PLAIN) -> torch.Tensor:
         lib = L.load()
         R, D, H, G = packed.shape[0], packed.shape[-1], heads.q, heads.kv
         out = torch.empty(R, H, D, dtype=packed.dtype, device=packed.device)
-        if D == 128 and self.page_size % 64 == 0 and H // G <= 8 and hasattr(lib, "dewb_paged_decode_persist"):
+        factors = visible.gain is not None or visible.sigmoid is not None
+        if D == 128 and self.page_size % 64 == 0 and H // G <= 8 and hasattr(lib, "dewb_paged_decode_persist") and (R <= 1024 or not factors):
             self._fused_decode(lib, slot, packed, packed.shape[2] * D, c.lengths, R, H, D, visible.window, visible.sinks, out, scale=scale, kv_heads=G, table=c.table,
                                visible=visible)
             return out
@@ -258,8 +287,8 @@ class KVStore:
                                       L.ptr(visible.sinks), L.ptr(out), L.ptr(None), L.ptr(pm), L.ptr(pl), L.ptr(pa), ctypes.c_int(R), ctypes.c_int(H),
                                       ctypes.c_int(G), ctypes.c_int(share), ctypes.c_int(D), ctypes.c_int(self.page_size), ctypes.c_int(self.max_pages),
                                       ctypes.c_int(splits), ctypes.c_float(scale), ctypes.c_int(visible.window or 0), ctypes.c_int(visible.keep),
-                                      ctypes.c_int(visible.chunk or 0), ctypes.c_float(visible.softcap), ctypes.c_int(0), L.stream_ptr()),
-                "paged_decode")
+                                      ctypes.c_int(visible.chunk or 0), ctypes.c_float(visible.softcap), L.ptr(visible.gain), L.ptr(visible.sigmoid), ctypes.c_int(0),
+                                      L.stream_ptr()), "paged_decode")
         L.count_launches(2)
         return out
 
@@ -396,7 +425,8 @@ class KVStore:
         (every CTA moves the same number of tiles, whatever the rows' lengths); more rows take one CTA per (row, head, chunk)."""
         longest = min(self.max_len, window + visible.keep if window else self.max_len, visible.chunk or self.max_len)
         max_tiles = -(-longest // 64) + 1 + int(visible.keep > 0)         # (+ 1: a window, or kept first keys, that straddle a tile boundary)
-        persist = R <= 1024 and os.environ.get("DEWB_DECODE_PERSIST", "1") == "1"
+        # (factors and sigmoid weights are built for the balanced form)
+        persist = visible.gain is not None or visible.sigmoid is not None or (R <= 1024 and os.environ.get("DEWB_DECODE_PERSIST", "1") == "1")
         if persist:
             min_tiles = int(os.environ.get("DEWB_DECODE_MIN_TILES", self.MIN_TILES))
             splits = (max_tiles - 1) // min_tiles + 2
@@ -418,7 +448,8 @@ class KVStore:
                 self._ctas = 2 * torch.cuda.get_device_properties(q.device).multi_processor_count
             L.check(lib.dewb_paged_decode_persist(*common, ctypes.c_int(min_tiles), ctypes.c_float(scale),
                                                   ctypes.c_int(window or 0), ctypes.c_int(visible.keep), ctypes.c_int(visible.chunk or 0),
-                                                ctypes.c_float(visible.softcap), ctypes.c_longlong(q_row_stride), ctypes.c_int(self._ctas),
+                                                ctypes.c_float(visible.softcap), L.ptr(visible.gain), L.ptr(visible.sigmoid), ctypes.c_longlong(q_row_stride),
+                                                ctypes.c_int(self._ctas),
                                                   L.ptr(L.status(q.device)), L.stream_ptr()), "paged_decode_persist")
         else:
             L.check(lib.dewb_paged_decode_fused(*common, ctypes.c_int(share), ctypes.c_float(scale),
@@ -506,7 +537,7 @@ class KVStore:
                                           L.ptr(pm), L.ptr(pl), L.ptr(pa), ctypes.c_int(R), ctypes.c_int(Hq),
                                           ctypes.c_int(self.kv_heads), ctypes.c_int(1), ctypes.c_int(D), ctypes.c_int(self.page_size),
                                           ctypes.c_int(self.max_pages), ctypes.c_int(splits), ctypes.c_float(scale),
-                                          ctypes.c_int(window or 0), ctypes.c_int(0), ctypes.c_int(0), ctypes.c_float(0.0), ctypes.c_int(self.kind),
+                                          ctypes.c_int(window or 0), ctypes.c_int(0), ctypes.c_int(0), ctypes.c_float(0.0), L.ptr(None), L.ptr(None), ctypes.c_int(self.kind),
                                           L.stream_ptr()), "paged_decode")
             L.count_launches(2)
             return out
@@ -555,7 +586,7 @@ class Uncached:
 
     def attend_slot(self, slot: int, qkv, heads: P.Heads, positions, *, scale: float, eps: float = 1e-6, q_weight=None, k_weight=None, temperature=None,
                     bias=None, chunk: Optional[int] = None, sinks=None, window: Optional[int] = None, keep: int = 0, softcap: float = 0.0,
-                    rot: Optional[rotary.Rotary] = None, unit: bool = False) -> torch.Tensor:
+                    rot: Optional[rotary.Rotary] = None, unit: bool = False, gain=None, sigmoid=None) -> torch.Tensor:
         R, S, _ = qkv.shape
         pos = torch.arange(S, device=qkv.device)[None].expand(R, S) if positions is None else positions
         turned = None if rot is None else P.Turned(rot, rotary.angles_reference(pos, rot))
@@ -566,8 +597,8 @@ class Uncached:
             self.kept[slot] = (k, v)
         # chunks counted from the first position: documents of the packed-segment form, with ids that start at 1
         segments = None if not chunk else (torch.arange(S, device=qkv.device, dtype=torch.int32) // chunk + 1)[None].expand(R, S).contiguous()
-        if keep and window:
-            o = visible_attention(q, k, v, scale, P.Visible(chunk, sinks, window, keep, softcap))
+        if (keep and window) or gain is not None or sigmoid is not None:
+            o = visible_attention(q, k, v, scale, P.Visible(chunk, sinks, window, keep, softcap, gain, sigmoid))
         else:
             o = ops.attention(q, k, v, causal=True, scale=scale, sinks=sinks, segment_ids=segments, window=window, softcap=softcap)
         return P.head_gate_reference(o, qkv[..., heads.packed:] if heads.gated else None, heads.dv)
@@ -592,9 +623,7 @@ def visible_attention(q, k, v, scale: float, visible: P.Visible) -> torch.Tensor
     R, S, H, _ = q.shape
     k, v = (t.float().repeat_interleave(H // t.shape[2], 2) for t in (k, v))
     seen = P.seen_keys(torch.arange(S, device=q.device)[None].expand(R, S), S, visible)
-    s = torch.einsum("rshd,rnhd->rhsn", q.float(), k) * scale
-    s = s if not visible.softcap else visible.softcap * torch.tanh(s / visible.softcap)
-    return torch.einsum("rhsn,rnhd->rshd", P.softmax_with_sinks(s.masked_fill(~seen[:, None], float("-inf")), visible.sinks), v).to(q.dtype)
+    return torch.einsum("rhsn,rnhd->rshd", P.weights_of(torch.einsum("rshd,rnhd->rhsn", q.float(), k) * scale, seen, visible), v).to(q.dtype)
 
 
 def paged_attention_reference(store: KVStore, layer: int, q, lengths, scale, window=None, sinks=None, softcap=0.0):

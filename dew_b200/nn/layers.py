@@ -63,12 +63,13 @@ class Embedding(nn.Module):
 
 
 class RMSNorm(nn.Module):
-    """``around``: the weights are stored as their distance from it (built for the norms of fp32 residual streams, ``nn.streams``)."""
+    """``around``: the weights are stored as their distance from it; ``one``: the weight is one number for all coordinates (both built for the norms of
+    fp32 residual streams, ``nn.streams``)."""
 
-    def __init__(self, features: int, eps: float = 1e-6, dtype=None, device=None, around: float = 0.0):
+    def __init__(self, features: int, eps: float = 1e-6, dtype=None, device=None, around: float = 0.0, one: bool = False):
         super().__init__()
-        self.eps, self.around = eps, float(around)
-        self.weight = declare(nn.Parameter(torch.full((features,), 1.0 - around, dtype=dtype, device=device)), ("norm",), "scale")
+        self.eps, self.around, self.one = eps, float(around), one
+        self.weight = declare(nn.Parameter(torch.full(() if one else (features,), 1.0 - around, dtype=dtype, device=device)), () if one else ("norm",), "scale")
 
     def reset_parameters(self, generator=None):
         with torch.no_grad():
@@ -76,8 +77,8 @@ class RMSNorm(nn.Module):
 
     def forward(self, x, branch=None):
         """With ``branch``: residual-stream form, returns ``(norm(x + branch), x + branch)``."""
-        if self.around:
-            raise NotImplementedError("norm weights stored around another value than 0 belong to fp32 residual streams")
+        if self.around or self.one:
+            raise NotImplementedError("norm weights stored around another value than 0, or as one number, belong to fp32 residual streams")
         if branch is not None:
             return ops.stream_rms_norm(x, branch, self.weight, self.eps)
         return ops.rms_norm(x, self.weight, self.eps)

@@ -16,7 +16,7 @@ import torch.nn as nn
 import torch.nn.functional as F
 
 from .. import ops
-from ..ops import scan
+from ..ops import recurrence, scan, token_mix
 from .layers import Linear, declare
 
 
@@ -78,7 +78,26 @@ class GatedDeltaNet(nn.Module):
                 self.dt_bias.copy_((dt + torch.log(-torch.expm1(-dt))).to(dev))
                 self.norm_weight.fill_(1.0)
 
-    def forward(self, x, segment_ids=None, cache=None, layer: int = 0):
+    def cache_slot(self):
+        from .kv_cache import CacheSlot
+        conv = (("conv", (2 * self.key_dim + self.value_dim, self.conv1d.kernel_size - 1)),) if self.conv1d.kernel_size > 1 else ()
+        return CacheSlot(state=(self.hv, self.dk, self.dv), more=conv)
+
+    def _in_slot(self, x, cache, slot: int, positions):
+        """A call's tokens with the state in the cache's slot: convolution, then norms, gates and recurrence in one kernel, then the heads' norm and gate."""
+        if self.qk_eps != 1e-6:
+            raise NotImplementedError("per-layer caches are built for q and k normalised with 1e-6 under the root (qk_eps=1e-6)")
+        rows = cache.call(positions).rows
+        qkvz, inner = self.in_proj_qkvz(x), 2 * self.key_dim + self.value_dim
+        qkv = token_mix.conv_tokens(qkvz[..., :inner], self.conv1d.weight, self.conv1d.bias, self.conv1d.activation, rows, cache.more[slot].get("conv"))
+        q, k, v = qkv.split([self.key_dim, self.key_dim, self.value_dim], -1)
+        o = recurrence.delta_rule(q, k, v, token_mix.narrow_product(x, self.in_proj_ba.weight), self.A_log, self.dt_bias, self.hv, self.hk, None, rows,
+                                  cache.states[slot])
+        return self.out_proj(token_mix.head_gated_norm(o, qkvz[..., inner:], self.norm_weight, self.norm_eps))
+
+    def forward(self, x, segment_ids=None, cache=None, layer: int = 0, positions=None):
+        if getattr(cache, "slots", None) is not None:
+            return self._in_slot(x, cache, layer, positions)
         B, T, _ = x.shape
         qkvz = self.in_proj_qkvz(x)
         ba = self.in_proj_ba(x).float()

@@ -53,14 +53,14 @@ class Router(nn.Module):
         if logits.is_cuda and mix.experts <= 256 and mix.top_k <= 16 and self.use_kernels and mix.groups <= 1 and mix.score_function != "top_softmax":
             from ..ops.routing import route
             return route(logits, self.expert_bias, mix.top_k, mix.score_function, mix.norm_topk_prob, mix.scaling)
-        # the bias steers the selection only; group-limited routing (DeepSeek-V3): a group's score is the sum of its two best experts, and
+        # the bias steers the selection only; group-limited routing (DeepSeek-V3): a group's score is the sum of its ``group_best`` (two, or one) best experts, and
         # experts outside the token's best ``topk_groups`` groups cannot be chosen
         return serve.select_reference(logits, self.expert_bias, self.selection)
 
     @property
     def selection(self) -> serve.Selection:
         m = self.mix
-        return serve.Selection(m.experts, m.top_k, m.groups, m.topk_groups, m.group_fill, m.score_function, m.norm_topk_prob, m.scaling)
+        return serve.Selection(m.experts, m.top_k, m.groups, m.topk_groups, m.group_fill, m.score_function, m.norm_topk_prob, m.scaling, m.group_best)
 
     def split(self) -> serve.Split:
         """The weights as bf16 rows for the tensor cores, made once per value of the parameter."""

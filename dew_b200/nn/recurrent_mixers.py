@@ -1,5 +1,5 @@
-"""More recurrent mixers: lightning attention (MiniMax), the S5 diagonal state space layer, and Mamba-3's single-input
-single-output recurrence (exponential-trapezoidal discretisation, complex state).
+"""More recurrent mixers: lightning attention (MiniMax), the matrix memory of xLSTM, RWKV-6-style time mixing, the S5 diagonal state space layer, and
+Mamba-3's single-input single-output recurrence (exponential-trapezoidal discretisation, complex state).
 
 Each has the step-by-step recurrence as its oracle and a parallel form that is what training runs:
 * lightning attention is the SSD recurrence with a constant decay per head (``dt = 1``, ``A = -rate``), so on a GPU with
@@ -22,7 +22,7 @@ import torch.nn as nn
 import torch.nn.functional as F
 
 from .. import ops
-from ..ops import decayed, scan, streams
+from ..ops import decayed, recurrence, scan, streams, token_mix
 from .layers import Linear, declare
 
 
@@ -114,6 +114,88 @@ class LightningAttention(nn.Module):
     def fresh_state(self, batch: int) -> dict:
         p = self.out_proj.weight
         return {"S": torch.zeros(batch, self.h, self.d, self.dv, dtype=torch.float32, device=p.device)}
+
+
+# ---------------------------------------------------------------------------------------------------------------
+# matrix memory and time mixing
+
+
+class MatrixMemory(nn.Module):
+    """The mLSTM of xLSTM: a matrix state per head with exponential input gates and sigmoid forget gates (their logits soft-capped), a normaliser and a
+    running maximum, the heads' outputs normed and gated."""
+
+    def __init__(self, features: int, num_heads: int = 4, head_dim: int = 64, value_dim: Optional[int] = None, gate_cap: float = 15.0, norm_eps: float = 1e-6,
+                 dtype=None, device=None):
+        super().__init__()
+        self.h, self.d, self.dv, self.cap, self.eps = num_heads, head_dim, value_dim or head_dim, float(gate_cap), norm_eps
+        inner = self.h * self.dv
+        self.in_proj = Linear(features, 2 * self.h * self.d + 2 * inner, axes=("embed", "heads"), dtype=dtype, device=device)       # q | k | v | gate
+        self.gate_proj = Linear(features, 2 * self.h, axes=("embed", "heads"), dtype=dtype, device=device)                          # input | forget
+        fp32 = lambda value: declare(nn.Parameter(torch.full((self.h,), value, dtype=torch.float32, device=device)), ("heads",), "bias")
+        self.i_bias, self.f_bias = fp32(0.0), fp32(3.0)
+        self.norm_weight = declare(nn.Parameter(torch.ones(inner, dtype=dtype, device=device)), ("norm",), "scale")
+        self.out_proj = Linear(inner, features, axes=("heads", "embed"), dtype=dtype, device=device)
+
+    def cache_slot(self):
+        from .kv_cache import CacheSlot
+        return CacheSlot(state=(self.h, self.d, self.dv), more=(("n", (self.h, self.d)), ("m", (self.h,))))
+
+    def forward(self, x, segment_ids=None, cache=None, layer: int = 0, positions=None):
+        if segment_ids is not None:
+            raise NotImplementedError("the matrix memory runs over rows without packed segments")
+        rows = memory = None
+        if getattr(cache, "slots", None) is not None:
+            rows = cache.call(positions).rows
+            memory = recurrence.Memory(cache.states[layer], cache.more[layer]["n"], cache.more[layer]["m"])
+        key, inner = self.h * self.d, self.h * self.dv
+        z = self.in_proj(x)
+        q, k, v, g = z.split([key, key, inner, inner], -1)
+        o = recurrence.matrix_memory(q, k, v, token_mix.narrow_product(x, self.gate_proj.weight), self.i_bias, self.f_bias, self.h, self.cap, None, rows, memory)
+        return self.out_proj(token_mix.head_gated_norm(o, g, self.norm_weight, self.eps, "sigmoid"))
+
+
+class RWKV6(nn.Module):
+    """Time mixing in the manner of RWKV-6: every projection reads its own mix of a token and the one before it, the state of a head decays per key channel by
+    an amount that the token chooses through a bottleneck, and a token reads itself through a bonus."""
+
+    MIXES = ("r", "k", "v", "g", "w")
+
+    def __init__(self, features: int, num_heads: int = 4, head_dim: int = 64, decay_rank: int = 64, norm_eps: float = 1e-6, dtype=None, device=None):
+        super().__init__()
+        self.features, self.h, self.d, self.eps = features, num_heads, head_dim, norm_eps
+        inner = num_heads * head_dim
+        new = lambda value, *shape, axes, kind: declare(nn.Parameter(torch.full(shape, value, dtype=dtype, device=device)), axes, kind)
+        self.mu = new(0.5, len(self.MIXES), features, axes=(None, "embed"), kind="scale")
+        self.rkvg = declare(nn.Parameter(torch.empty(4, inner, features, dtype=dtype, device=device)), (None, "heads", "embed"), "kernel")
+        self.decay_in = Linear(features, decay_rank, axes=("embed", None), dtype=dtype, device=device)
+        self.decay_out = Linear(decay_rank, inner, axes=(None, "heads"), dtype=dtype, device=device)
+        self.decay_base = new(-1.0, inner, axes=("heads",), kind="bias")
+        self.bonus = new(0.0, num_heads, head_dim, axes=("heads", None), kind="scale")
+        self.norm_weight = new(1.0, inner, axes=("norm",), kind="scale")
+        self.out_proj = Linear(inner, features, axes=("heads", "embed"), dtype=dtype, device=device)
+        self._own_reset = True
+        self.reset_parameters()
+
+    def reset_parameters(self, generator=None):
+        with torch.no_grad():
+            self.rkvg.normal_(0.0, self.features ** -0.5, generator=generator)
+
+    def cache_slot(self):
+        from .kv_cache import CacheSlot
+        return CacheSlot(state=(self.h, self.d, self.d), more=(("before", (self.features,)),))
+
+    def forward(self, x, segment_ids=None, cache=None, layer: int = 0, positions=None):
+        if segment_ids is not None:
+            raise NotImplementedError("time mixing runs over rows without packed segments")
+        rows = state = before = None
+        if getattr(cache, "slots", None) is not None:
+            rows, state, before = cache.call(positions).rows, cache.states[layer], cache.more[layer]["before"]
+        R, S, _ = x.shape
+        mixed = token_mix.shift_tokens(x, self.mu, rows, before)
+        r, k, v, g = token_mix.own_products(mixed[:4], self.rkvg)
+        decay = token_mix.low_rank_decay(token_mix.narrow_product(mixed[4], self.decay_in.weight), self.decay_out.weight, self.decay_base)
+        o = recurrence.bonus_decay(r, k, v, decay, self.bonus, self.h, rows, state)
+        return self.out_proj(token_mix.head_gated_norm(o, g, self.norm_weight, self.eps))
 
 
 # ---------------------------------------------------------------------------------------------------------------

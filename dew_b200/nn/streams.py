@@ -72,18 +72,22 @@ class StreamStack:
     write, read and norm are one pass over the streams (``ops.streams.stream_step``)."""
 
     def __init__(self, H: torch.Tensor, dtype):
-        self.H, self.dtype, self.pending = H, dtype, None
+        self.H, self.dtype, self.pending, self.joining = H, dtype, None, None
 
     def enter(self, connection: Optional["HyperConnections"], norm: nn.Module) -> torch.Tensor:
         """The next sub-layer's normalised input."""
         return self._step(None if connection is None else connection.alpha, norm)
 
     def leave(self, connection: Optional["HyperConnections"], y: torch.Tensor, scale=None, norm: Optional[nn.Module] = None, gain: float = 1.0,
-              beside: Optional[torch.Tensor] = None, beside_scale=None) -> None:
+              beside: Optional[torch.Tensor] = None, beside_scale=None, beside_gain: Optional[float] = None) -> None:
         """The sub-layer's output (through an RMS ``norm`` of its own, times its layer scale), to be written back by the connection; ``beside`` is the
-        output of a second sub-layer that read the same norm, ``gain`` multiplies both."""
+        output of a second sub-layer that read the same norm; ``gain`` multiplies both, or the first alone where ``beside_gain`` is given."""
         mix, out = (None, None) if connection is None else (connection.mix, connection.beta)
-        self.pending = S.Write(y, scale, mix, out, *((None, 0.0) if norm is None else (norm.weight, norm.eps)), beside, beside_scale, gain)
+        self.pending = S.Write(y, scale, mix, out, *((None, 0.0) if norm is None else (norm.weight, norm.eps)), beside, beside_scale, gain, beside_gain)
+
+    def join(self, join: S.Join) -> None:
+        """What the stream takes in in front of the next sub-layer's norm, beside the pending write."""
+        self.joining = join
 
     def finish(self, norm: nn.Module) -> torch.Tensor:
         """The final norm of the sum of the streams."""
@@ -98,8 +102,8 @@ class StreamStack:
 
     def _step(self, read, norm) -> torch.Tensor:
         kind = "layer" if isinstance(norm, LayerNorm) else "rms"
-        n, self.H = S.stream_step(self.H, self.pending, read, norm.weight, norm.eps, self.dtype, kind, getattr(norm, "around", 0.0))
-        self.pending = None
+        n, self.H = S.stream_step(self.H, self.pending, read, norm.weight, norm.eps, self.dtype, kind, getattr(norm, "around", 0.0), self.joining)
+        self.pending = self.joining = None
         return n
 
 

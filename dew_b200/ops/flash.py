@@ -20,19 +20,23 @@ class Variants:
     """The optional attention variants the kernels take: ``window`` (keys visible behind each query, None = all; with ``keep`` the first ``keep`` keys
     stay visible beside it, forward only), ``chunk`` (a query sees no key
     from before the start of its chunk of that many positions; forward only), ``softcap``
-    (scores become cap * tanh(score / cap)), ``sinks`` ([Hq] fp32 logits that join the softmax denominator only) and
-    ``segments`` (int32 [B, S] ids of packed documents, non-decreasing along the sequence; 0 marks padding)."""
+    (scores become cap * tanh(score / cap)), ``sinks`` ([Hq] fp32 logits that join the softmax denominator only),
+    ``segments`` (int32 [B, S] ids of packed documents, non-decreasing along the sequence; 0 marks padding), ``gain`` ([Hq] fp32: factors of the
+    heads' scores, in front of the cap; forward only) and ``sigmoid`` ([Hq] fp32: a visible key weighs sigmoid(score + sigmoid[head]), with no softmax;
+    forward only)."""
 
-    def __init__(self, window=None, softcap: float = 0.0, sinks=None, segments=None, chunk=None, keep: int = 0):
+    def __init__(self, window=None, softcap: float = 0.0, sinks=None, segments=None, chunk=None, keep: int = 0, gain=None, sigmoid=None):
         self.window = int(window) if window else 0
         self.chunk = int(chunk) if chunk else 0
         self.keep = int(keep) if window else 0
         self.softcap = float(softcap or 0.0)
         self.sinks = sinks.detach().to(torch.float32).contiguous() if sinks is not None else None
         self.segments = segments.to(torch.int32).contiguous() if segments is not None else None
+        self.gain, self.sigmoid = (None if t is None else t.detach().to(torch.float32).contiguous() for t in (gain, sigmoid))
 
     def any(self) -> bool:
-        return bool(self.window or self.chunk or self.softcap or self.sinks is not None or self.segments is not None)
+        return bool(self.window or self.chunk or self.softcap or self.sinks is not None or self.segments is not None or self.gain is not None
+                    or self.sigmoid is not None)
 
 
 NONE = Variants()
@@ -46,7 +50,7 @@ def flash_fwd(q, k, v, causal: bool, scale: float, need_lse: bool = True, var: V
     rc = L.load().dewb_flash_fwd_var(L.ptr(q), L.ptr(k), L.ptr(v), L.ptr(out), L.ptr(lse), c_int(B), c_int(S), c_int(T),
                                      c_int(Hq), c_int(Hkv), c_int(D), *_strides(q), *_strides(k), *_strides(v),
                                      *_strides(out), c_float(scale), c_int(int(causal)), c_int(var.window), c_int(var.keep), c_int(var.chunk), c_float(var.softcap),
-                                     L.ptr(var.sinks), L.ptr(var.segments), L.ptr(var.segments), L.ptr(L.status(q.device)),
+                                     L.ptr(var.sinks), L.ptr(var.segments), L.ptr(var.segments), L.ptr(var.gain), L.ptr(var.sigmoid), L.ptr(L.status(q.device)),
                                      L.stream_ptr())
     L.check(rc, "flash_fwd")
     L.count_launches()

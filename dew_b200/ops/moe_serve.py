@@ -19,8 +19,8 @@ ROUTER_TOKENS = 512          # up to here the router's logits are formed token b
 
 
 class Selection(NamedTuple):
-    """How a router chooses: ``top`` of ``experts``; with ``groups`` > 1 only within the token's best ``keep`` groups (by the sum of their two
-    best choice scores), the others' choice scores becoming ``fill``; ``norm`` divides the weights by their sum.  ``score``: ``softmax`` or ``sigmoid``
+    """How a router chooses: ``top`` of ``experts``; with ``groups`` > 1 only within the token's best ``keep`` groups (by the sum of their ``best``,
+    one or two, best choice scores), the others' choice scores becoming ``fill``; ``norm`` divides the weights by their sum.  ``score``: ``softmax`` or ``sigmoid``
     of the logits, or ``top_softmax``: the choice runs on the logits, and the weights are the softmax over the chosen ones alone."""
     experts: int
     top: int
@@ -30,6 +30,7 @@ class Selection(NamedTuple):
     score: str = "softmax"
     norm: bool = True
     scaling: float = 1.0
+    best: int = 2
 
 
 def choice_scores(scores: torch.Tensor, bias: Optional[torch.Tensor], s: Selection) -> torch.Tensor:
@@ -38,7 +39,7 @@ def choice_scores(scores: torch.Tensor, bias: Optional[torch.Tensor], s: Selecti
     if s.groups > 1:
         T, E = select.shape
         per = E // s.groups
-        best = select.view(T, s.groups, per).topk(min(2, per), -1).values.sum(-1)
+        best = select.view(T, s.groups, per).topk(min(s.best, per), -1).values.sum(-1)
         keep = torch.zeros_like(best).scatter_(1, best.topk(s.keep, -1).indices, 1.0).bool()
         select = select.masked_fill(~keep[:, :, None].expand(T, s.groups, per).reshape(T, E), s.fill)
     return select
@@ -97,7 +98,7 @@ def route(x2: torch.Tensor, weight: torch.Tensor, split: Optional[Split], bias: 
     b, lb = (None if t is None else t.detach().float().contiguous() for t in (bias, logit_bias))
     if positions is not None and positions.numel() != T:
         raise ValueError(f"{positions.numel()} positions for {T} tokens")
-    tail = (c_int(E), c_int(k), c_int(s.groups), c_int(s.keep), c_float(s.fill), c_int(SCORES.index(s.score)), c_int(int(s.norm)), c_float(s.scaling),
+    tail = (c_int(E), c_int(k), c_int(s.groups), c_int(s.keep), c_int(s.best), c_float(s.fill), c_int(SCORES.index(s.score)), c_int(int(s.norm)), c_float(s.scaling),
             L.ptr(out.weights), L.ptr(out.ids), L.ptr(out.rank), L.ptr(out.counts))
     if (kernel or ("product" if T > ROUTER_TOKENS and x2.dtype == torch.bfloat16 and split is not None and d % 8 == 0 else "rows")) == "product":
         from .functional import gemm

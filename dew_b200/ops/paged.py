@@ -43,13 +43,16 @@ class Heads:
 
 class Visible(NamedTuple):
     """What a layer's attention adds to the causal softmax: a query sees no key from before the start of its ``chunk`` of positions; with a ``window``
-    it sees that many keys (its own included) and the row's first ``keep``; scores become ``softcap tanh(score / softcap)``; ``sinks`` (fp32, one per
-    query head) join the denominator only."""
+    it sees that many keys (its own included) and the row's first ``keep``; scores are multiplied by ``gain`` (fp32, one per query head) and become
+    ``softcap tanh(score / softcap)``; ``sinks`` (fp32, one per query head) join the denominator only.  With ``sigmoid`` (fp32, one per query head) there is
+    no softmax: a visible key weighs ``sigmoid(score + sigmoid[head])``."""
     chunk: Optional[int] = None
     sinks: Optional[torch.Tensor] = None
     window: Optional[int] = None
     keep: int = 0
     softcap: float = 0.0
+    gain: Optional[torch.Tensor] = None
+    sigmoid: Optional[torch.Tensor] = None
 
 
 PLAIN = Visible()
@@ -181,6 +184,17 @@ def softmax_with_sinks(s: torch.Tensor, sinks: Optional[torch.Tensor]) -> torch.
     return torch.softmax(torch.cat([s, sink], -1), -1)[..., :-1]
 
 
+def weights_of(s: torch.Tensor, seen: torch.Tensor, visible: Visible) -> torch.Tensor:
+    """The keys' weights from their scaled scores ``s [R, H, S, n]`` and ``seen [R, S, n]``."""
+    if visible.gain is not None:
+        s = s * visible.gain.float().view(1, -1, 1, 1)
+    if visible.softcap:
+        s = visible.softcap * torch.tanh(s / visible.softcap)
+    if visible.sigmoid is not None:
+        return torch.sigmoid(s + visible.sigmoid.float().view(1, -1, 1, 1)) * seen[:, None]
+    return softmax_with_sinks(s.masked_fill(~seen[:, None], float("-inf")), visible.sinks)
+
+
 def paged_attend_reference(q, heads: Heads, positions, pages: Pages, scale: float, visible: Visible = PLAIN) -> torch.Tensor:
     R, S = positions.shape
     D = pages.k.shape[-1]
@@ -194,9 +208,7 @@ def paged_attend_reference(q, heads: Heads, positions, pages: Pages, scale: floa
     # what the pool holds beyond a row's own tokens is another row's, or nothing: it must not reach the sums
     own = (torch.arange(n, device=q.device)[None] <= positions.amax(1, keepdim=True))[..., None, None]
     kc, vc = torch.where(own, kc, torch.zeros_like(kc)), torch.where(own, vc, torch.zeros_like(vc))
-    s = torch.einsum("rshd,rnhd->rhsn", q[..., :D].float(), kc) * scale
-    s = s if not visible.softcap else visible.softcap * torch.tanh(s / visible.softcap)
-    p = softmax_with_sinks(s.masked_fill(~seen[:, None], float("-inf")), visible.sinks)
+    p = weights_of(torch.einsum("rshd,rnhd->rhsn", q[..., :D].float(), kc) * scale, seen, visible)
     return torch.einsum("rhsn,rnhd->rshd", p, vc).to(q.dtype)
 
 
@@ -233,7 +245,8 @@ def paged_attend(q: torch.Tensor, heads: Heads, positions: torch.Tensor, pages: 
     out = torch.empty(R, S, H, heads.dv, dtype=q.dtype, device=q.device)
     if gate is not None and (gate.stride(2) != 1 or (R > 1 and gate.stride(0) != S * gate.stride(1))):
         gate = gate.contiguous()
-    extras = (c_int(visible.chunk or 0), c_int(visible.window or 0), c_int(visible.keep), c_float(visible.softcap), L.ptr(visible.sinks), L.ptr(gate), c_ll(0 if gate is None else gate.stride(1)))
+    extras = (c_int(visible.chunk or 0), c_int(visible.window or 0), c_int(visible.keep), c_float(visible.softcap), L.ptr(visible.sinks), L.ptr(gate), c_ll(0 if gate is None else gate.stride(1)),
+              L.ptr(visible.gain), L.ptr(visible.sigmoid))
     if (kernel or ("mma" if q.dtype == torch.bfloat16 and D in (64, 128, 256) else "general")) == "mma":
         L.check(L.load().dewb_paged_attend_mma(L.ptr(q), c_ll(q.stride(1)), L.ptr(pages.k), L.ptr(pages.v), L.ptr(positions), c_int(R), c_int(S), c_int(H),
                                                c_int(heads.kv), c_int(heads.dv), c_int(D), c_float(scale), *extras, L.ptr(out), L.ptr(pages.table),

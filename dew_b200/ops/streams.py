@@ -19,9 +19,9 @@ MAX_STREAMS = 16
 
 
 class Write(NamedTuple):
-    """A sub-layer's output on its way into the streams: ``H'[t] = sum_s mix[s, t] H[s] + out[t] * gain * (scale * y + scale2 * y2)``.  Without ``mix``
-    and ``out`` every stream keeps itself and takes ``y``; with ``weight``, ``y`` passes an RMS norm (``weight``, ``eps``) first; ``y2`` is the second
-    of two sub-layers that join together."""
+    """A sub-layer's output on its way into the streams: ``H'[t] = sum_s mix[s, t] H[s] + out[t] * (gain * scale * y + gain2 * scale2 * y2)``.  Without
+    ``mix`` and ``out`` every stream keeps itself and takes ``y``; with ``weight``, ``y`` passes an RMS norm (``weight``, ``eps``) first; ``y2`` is the second
+    of two sub-layers that join together (``gain2`` None: ``gain``)."""
     y: torch.Tensor
     scale: Optional[torch.Tensor] = None
     mix: Optional[torch.Tensor] = None
@@ -30,6 +30,19 @@ class Write(NamedTuple):
     eps: float = 0.0
     y2: Optional[torch.Tensor] = None
     scale2: Optional[torch.Tensor] = None
+    gain: float = 1.0
+    gain2: Optional[float] = None
+
+    @property
+    def second(self) -> float:
+        return self.gain if self.gain2 is None else self.gain2
+
+
+class Join(NamedTuple):
+    """What joins one plain stream beside the sub-layers' outputs: ``add [d]``, and ``gain`` times the rows of ``table [vocab, d]`` at ``tokens [...]``."""
+    add: Optional[torch.Tensor] = None
+    table: Optional[torch.Tensor] = None
+    tokens: Optional[torch.Tensor] = None
     gain: float = 1.0
 
 
@@ -73,18 +86,23 @@ def embed_streams(tokens: torch.Tensor, positions: Optional[torch.Tensor], embed
     return x.unsqueeze(2).expand(B, S, n, d).contiguous()
 
 
-def stream_step_reference(H, write: Optional[Write], read, weight, eps: float, dtype, norm: str = "layer", around: float = 0.0):
+def stream_step_reference(H, write: Optional[Write], read, weight, eps: float, dtype, norm: str = "layer", around: float = 0.0, join: Optional[Join] = None):
     if write is not None:
         y = write.y.float()
         if write.weight is not None:
             y = y / torch.sqrt(y.pow(2).mean(-1, keepdim=True) + write.eps) * write.weight.float()
         if write.scale is not None:
             y = y * write.scale.float()
-        if write.y2 is not None:
-            y = y + (write.y2.float() if write.scale2 is None else write.y2.float() * write.scale2.float())
         y = y * write.gain
+        if write.y2 is not None:
+            y = y + write.second * (write.y2.float() if write.scale2 is None else write.y2.float() * write.scale2.float())
         kept = H if write.mix is None else torch.einsum("st,...sd->...td", write.mix.float(), H)
         H = kept + (y.unsqueeze(-2) if write.out is None else write.out.float()[:, None] * y.unsqueeze(-2))
+    if join is not None:
+        if join.table is not None:
+            H = H + join.gain * F.embedding(join.tokens, join.table).float().unsqueeze(-2)
+        if join.add is not None:
+            H = H + join.add.float()
     if weight is None:
         return None, H
     u = H.sum(-2) if read is None else torch.einsum("s,...sd->...d", read.float(), H)
@@ -95,15 +113,19 @@ def stream_step_reference(H, write: Optional[Write], read, weight, eps: float, d
 
 
 def stream_step(H: torch.Tensor, write: Optional[Write], read: Optional[torch.Tensor], weight: Optional[torch.Tensor], eps: float, dtype,
-                norm: str = "layer", around: float = 0.0) -> Tuple[Optional[torch.Tensor], torch.Tensor]:
+                norm: str = "layer", around: float = 0.0, join: Optional[Join] = None) -> Tuple[Optional[torch.Tensor], torch.Tensor]:
     """``(norm(sum_s read[s] H'[s]) * (around + weight), H')`` with ``H'`` the streams after ``write`` (None: as they are); ``read`` None: all ones.  ``H [..., n, d]`` fp32;
-    on a GPU outside autograd ``H`` is updated in place.  ``weight`` None: the write alone."""
+    on a GPU outside autograd ``H`` is updated in place.  ``weight`` None: the write alone; a ``weight`` of one number counts for all coordinates.  ``join``:
+    what else comes in behind the write (one stream)."""
     if norm not in ("layer", "rms"):
         raise ValueError(f"unknown norm {norm!r}; known: layer, rms")
     n, d = H.shape[-2:]
-    tensors = (weight, read) + (() if write is None else (write.y, write.scale, write.mix, write.out, write.weight, write.y2, write.scale2))
+    if join is not None and n != 1:
+        raise NotImplementedError("what joins beside the sub-layers is built for one stream")
+    tensors = (weight, read) + (() if write is None else (write.y, write.scale, write.mix, write.out, write.weight, write.y2, write.scale2)) + \
+        (() if join is None else (join.add, join.table))
     if n > MAX_STREAMS or not H.is_contiguous() or not _kernel_ok(H, *tensors) or dtype not in (torch.bfloat16, torch.float32):
-        return stream_step_reference(H, write, read, weight, eps, dtype, norm, around)
+        return stream_step_reference(H, write, read, weight, eps, dtype, norm, around, join)
     rows = H.numel() // (n * d)
     normed = None if weight is None else torch.empty(*H.shape[:-2], d, dtype=dtype, device=H.device)
     y = y_weight = scale = mix = out = y2 = scale2 = None
@@ -111,9 +133,13 @@ def stream_step(H: torch.Tensor, write: Optional[Write], read: Optional[torch.Te
         y, scale, mix, out = _as(write.y, dtype), _as(write.scale, dtype), _as(write.mix, torch.float32), _as(write.out, torch.float32)
         y_weight, y2, scale2 = _as(write.weight, dtype), _as(write.y2, dtype), _as(write.scale2, dtype)
     r, w = _as(read, torch.float32), _as(weight, dtype)
+    add, table, tokens = (None, None, None) if join is None else (_as(join.add, dtype), _as(join.table, dtype), join.tokens)
+    tokens = None if tokens is None else tokens.to(torch.int64).contiguous()
     L.check(L.load().dewb_stream_step(L.ptr(H), L.ptr(y), L.ptr(y_weight), L.ptr(scale), L.ptr(mix), L.ptr(out), L.ptr(r), L.ptr(w), L.ptr(normed), c_ll(rows),
                                       c_int(n), c_int(d), c_float(0.0 if write is None else write.eps), c_float(eps), c_int(int(norm == "rms")),
-                                      L.ptr(y2), L.ptr(scale2), c_float(1.0 if write is None else write.gain), c_float(around),
+                                      L.ptr(y2), L.ptr(scale2), c_float(1.0 if write is None else write.gain), c_float(1.0 if write is None else write.second),
+                                      c_float(around), c_int(int(w is not None and w.dim() == 0)), L.ptr(add), L.ptr(table), L.ptr(tokens),
+                                      c_int(0 if table is None else table.shape[0]), c_float(1.0 if join is None else join.gain),
                                       c_int(int(dtype == torch.float32)), L.stream_ptr()), "stream_step")
     L.count_launches()
     return normed, H

@@ -49,7 +49,7 @@ _STATIC: Dict[str, Dict[str, str]] = {
         "causal_video_vae": "dew_b200.models.latent_autoencoders:CausalVideoVAE",
         "classic_decoder": "dew_b200.models.classic_decoder:ClassicDecoder",
         "ragenex": "dew_b200.interop.ragenex:ragenex", "fakonex": "dew_b200.interop.fakonex:fakonex",
-        "selivik": "dew_b200.interop.selivik:selivik",
+        "selivik": "dew_b200.interop.selivik:selivik", "rarelorn": "dew_b200.interop.rarelorn:rarelorn",
     },
     "objective": {
         "lm": "dew_b200.objectives.lm:LMObjective",
