@@ -166,7 +166,7 @@ def main() -> None:
     ap.add_argument("--others", default="auto", choices=["auto", "none"],
                     help="auto: the default (dense) run also times 3 steps of the moe and hybrid configurations in child processes "
                          "and reports them under `others`")
-    ap.add_argument("--decoder", default=None, choices=["ragenex", "fakonex", "selivik"],
+    ap.add_argument("--decoder", default=None, choices=["ragenex", "fakonex", "selivik", "rarelorn"],
                     help="instead of the training benchmark: prefill and decode throughput of this decoder design beside the closest existing model of equal "
                          "size, and its kernels beside theirs (dew_b200/telemetry/decoder_bench.py)")
     ap.add_argument("--compile", action="store_true", help="torch_nccl arm only: torch.compile each decoder layer")

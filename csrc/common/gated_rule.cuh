@@ -70,7 +70,7 @@ __device__ __forceinline__ float softplus(float x) { return fmaxf(x, 0.f) + log1
 template <typename T>
 __device__ __forceinline__ void delta_log_gates(const Args<T>& p, long long token, int h, float& log_decay, float& beta) {
   const float* z = p.gates + token * 2 * p.H + h;
-  beta = 1.f / (1.f + expf(-z[0]));
+  beta = __fdividef(1.f, 1.f + expf(-z[0]));
   log_decay = -expf(p.bias0[h]) * softplus(z[p.H] + p.bias1[h]);
 }
 template <typename T>
@@ -83,8 +83,9 @@ __device__ __forceinline__ void delta_gates(const Args<T>& p, long long token, i
 template <typename T>
 __device__ __forceinline__ void memory_gates(const Args<T>& p, long long token, int h, float& in, float& forget) {
   const float* z = p.gates + token * 2 * p.H + h;
-  in = p.cap * tanhf((z[0] + p.bias0[h]) / p.cap);
-  forget = -softplus(-p.cap * tanhf((z[p.H] + p.bias1[h]) / p.cap));
+  const float inv = __fdividef(1.f, p.cap);
+  in = p.cap * tanhf((z[0] + p.bias0[h]) * inv);
+  forget = -softplus(-p.cap * tanhf((z[p.H] + p.bias1[h]) * inv));
 }
 
 }  // namespace gated

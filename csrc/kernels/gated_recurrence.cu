@@ -25,7 +25,7 @@ constexpr int STEP_THREADS = 256;
 // grid (H, column tiles, rows); a block walks its column tiles (memory: one block per row and head, which also owns n and m).  A thread owns V columns of
 // the key rows group, group + GROUPS, ..., U of them.
 template <int MODE, typename T, int V, int LANES, int U>
-__global__ void __launch_bounds__(STEP_THREADS)
+__global__ void __launch_bounds__(STEP_THREADS, U * V > 32 ? 2 : 3)
 gated_step_kernel(Args<T> p) {
   constexpr int GROUPS = STEP_THREADS / LANES, TILE = LANES * V;
   extern __shared__ float sm[];                 // q [dk], k [dk], w [dk] (wkv), partial [GROUPS][TILE], u [TILE]
@@ -60,7 +60,7 @@ gated_step_kernel(Args<T> p) {
   if (MODE == DELTA) {
     s0 = rows::block_sum(s0, red);
     s1 = rows::block_sum(s1, red);
-    const float fq = p.scale / sqrtf(s0 + 1e-6f), fk = 1.f / sqrtf(s1 + 1e-6f);
+    const float fq = p.scale * rsqrtf(s0 + 1e-6f), fk = rsqrtf(s1 + 1e-6f);
     delta_gates(p, row, h, a, b);               // decay, beta
     for (int i = threadIdx.x; i < dk; i += STEP_THREADS) { sq[i] *= fq; sk[i] *= fk; }
   } else if (MODE == MEMORY) {
@@ -78,7 +78,7 @@ gated_step_kernel(Args<T> p) {
       dot += x * sq[i];
     }
     dot = rows::block_sum(dot, red);            // (every thread has read m by here)
-    c = 1.f / (fmaxf(fabsf(dot), expf(-top)) + 1e-6f);
+    c = __fdividef(1.f, fmaxf(fabsf(dot), expf(-top)) + 1e-6f);
     if (threadIdx.x == 0) p.m[rh] = top;
   } else {
     c = rows::block_sum(s0, red);               // the bonus
@@ -224,7 +224,7 @@ gated_sequence_kernel(Args<T> p) {
 #pragma unroll
         for (int q = 16; q > 0; q >>= 1) { s0 += __shfl_xor_sync(0xffffffffu, s0, q); s1 += __shfl_xor_sync(0xffffffffu, s1, q); }
         if (MODE == DELTA) {
-          const float fq = p.scale / sqrtf(s0 + 1e-6f), fk = 1.f / sqrtf(s1 + 1e-6f);
+          const float fq = p.scale * rsqrtf(s0 + 1e-6f), fk = rsqrtf(s1 + 1e-6f);
           for (int c = lane; c < dk; c += 32) { sq[t * DK + c] *= fq; sk[t * DK + c] *= fk; }
           if (lane == 0) delta_gates(p, t_row + t0 + t, h, sc[t * 4], sc[t * 4 + 1]);
         } else if (lane == 0) {
@@ -274,7 +274,7 @@ gated_sequence_kernel(Args<T> p) {
         if (MODE == MEMORY) den += __shfl_xor_sync(0xffffffffu, den, q);
       }
       if (MODE == WKV) out += a * v;
-      if (MODE == MEMORY) out /= fmaxf(fabsf(den), sc[t * 4 + 2]) + 1e-6f;
+      if (MODE == MEMORY) out = __fdividef(out, fmaxf(fabsf(den), sc[t * 4 + 2]) + 1e-6f);
       if (rl == 0) sv[t * COLS + cl] = out;     // (the column's lanes have read their value: the shuffles stand between)
     }
     if (MODE == MEMORY) m = sc[(cnt - 1) * 4 + 3];

@@ -63,34 +63,42 @@ conv_tokens_kernel(const T* __restrict__ x, long long row_stride, const T* __res
   auto finish = [&](int t, float (&o)[V]) {
     if (act) {
 #pragma unroll
-      for (int j = 0; j < V; ++j) o[j] = o[j] * sigmoid(o[j]);
+      for (int j = 0; j < V; ++j) o[j] = sizeof(T) == 2 ? __fdividef(o[j], 1.f + __expf(-o[j])) : o[j] * sigmoid(o[j]);
     }
     store_v<V>(yr + static_cast<long long>(t) * C, o);
   };
   const int t1 = min(S, t0 + RUN);
   if constexpr (TAPS > 0) {
-    float wt[V][TAPS], u[TAPS][V];
+    constexpr int AHEAD = 4;                      // tokens fetched together
+    float wt[V][TAPS], u[TAPS + AHEAD - 1][V];
 #pragma unroll
     for (int j = 0; j < V; ++j)
 #pragma unroll
       for (int q = 0; q < TAPS; ++q) wt[j][q] = ld(w + static_cast<long long>(c + j) * TAPS + q);
 #pragma unroll
-    for (int q = 1; q < TAPS; ++q) input(t0 - TAPS + q, u[q]);
-    for (int t = t0; t < t1; ++t) {
-      float o[V];
+    for (int q = 0; q + 1 < TAPS; ++q) input(t0 - TAPS + 1 + q, u[AHEAD + q]);
+    for (int t = t0; t < t1; t += AHEAD) {
 #pragma unroll
       for (int q = 0; q + 1 < TAPS; ++q)
 #pragma unroll
-        for (int j = 0; j < V; ++j) u[q][j] = u[q + 1][j];
-      input(t, u[TAPS - 1]);
+        for (int j = 0; j < V; ++j) u[q][j] = u[q + AHEAD][j];
 #pragma unroll
-      for (int j = 0; j < V; ++j) {
-        o[j] = 0.f;
+      for (int s = 0; s < AHEAD; ++s)
+        if (t + s < t1) input(t + s, u[TAPS - 1 + s]);
 #pragma unroll
-        for (int q = 0; q < TAPS; ++q) o[j] += wt[j][q] * u[q][j];
-        if (pos[t] < 0) o[j] = 0.f;
+      for (int s = 0; s < AHEAD; ++s) {
+        if (t + s >= t1) break;
+        float o[V];
+        const bool live = pos[t + s] >= 0;
+#pragma unroll
+        for (int j = 0; j < V; ++j) {
+          o[j] = 0.f;
+#pragma unroll
+          for (int q = 0; q < TAPS; ++q) o[j] += wt[j][q] * u[q + s][j];
+          if (!live) o[j] = 0.f;
+        }
+        finish(t + s, o);
       }
-      finish(t, o);
     }
   } else {
     for (int t = t0; t < t1; ++t) {
@@ -178,35 +186,43 @@ shift_tokens_kernel(const T* __restrict__ x, const T* __restrict__ mu, float* __
   if (S == 1 && live && s != nullptr) store_v<V>(s, a);
 }
 
-// out [T, n] fp32 = x [T, d] w [n, d]^T: a warp per output, TOK tokens at a time.  grid (ceil(n / 8), ceil(T / TOK)).
-constexpr int TOK = 8;
+// out [T, n] fp32 = x [T, d] w [n, d]^T.  A block forms NOUT outputs of NTOK tokens; its warps share the reduction.  grid (ceil(n / NOUT), ceil(T / NTOK)).
+constexpr int NTOK = 4, NOUT = 4;
 template <typename T, int V>
 __global__ void __launch_bounds__(256)
 narrow_product_kernel(const T* __restrict__ x, const T* __restrict__ w, float* __restrict__ out, long long tokens, int n, int d) {
-  const int lane = threadIdx.x & 31, e = blockIdx.x * 8 + (threadIdx.x >> 5);
-  if (e >= n) return;
-  const long long t0 = static_cast<long long>(blockIdx.y) * TOK;
-  float acc[TOK];
+  __shared__ float part[8][NTOK * NOUT];
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, e0 = blockIdx.x * NOUT;
+  const long long t0 = static_cast<long long>(blockIdx.y) * NTOK;
+  float acc[NTOK][NOUT] = {};
+  for (int c = threadIdx.x * V; c < d; c += 256 * V) {
+    float a[NTOK][V], b[NOUT][V];
 #pragma unroll
-  for (int i = 0; i < TOK; ++i) acc[i] = 0.f;
-  for (int c = lane * V; c < d; c += 32 * V) {
-    float b[V];
-    load_v<V>(w + static_cast<long long>(e) * d + c, b);
+    for (int i = 0; i < NTOK; ++i) load_v<V>(x + min(t0 + i, tokens - 1) * d + c, a[i]);
 #pragma unroll
-    for (int i = 0; i < TOK; ++i) {
-      if (t0 + i < tokens) {
-        float a[V];
-        load_v<V>(x + (t0 + i) * d + c, a);
+    for (int e = 0; e < NOUT; ++e) load_v<V>(w + static_cast<long long>(min(e0 + e, n - 1)) * d + c, b[e]);
 #pragma unroll
-        for (int j = 0; j < V; ++j) acc[i] += a[j] * b[j];
-      }
-    }
+    for (int i = 0; i < NTOK; ++i)
+#pragma unroll
+      for (int e = 0; e < NOUT; ++e)
+#pragma unroll
+        for (int j = 0; j < V; ++j) acc[i][e] += a[i][j] * b[e][j];
   }
 #pragma unroll
-  for (int i = 0; i < TOK; ++i) {
+  for (int i = 0; i < NTOK; ++i)
 #pragma unroll
-    for (int o = 16; o > 0; o >>= 1) acc[i] += __shfl_xor_sync(0xffffffffu, acc[i], o);
-    if (lane == 0 && t0 + i < tokens) out[(t0 + i) * n + e] = acc[i];
+    for (int e = 0; e < NOUT; ++e) {
+#pragma unroll
+      for (int o = 16; o > 0; o >>= 1) acc[i][e] += __shfl_xor_sync(0xffffffffu, acc[i][e], o);
+      if (lane == 0) part[warp][i * NOUT + e] = acc[i][e];
+    }
+  __syncthreads();
+  if (threadIdx.x < NTOK * NOUT) {
+    const int i = threadIdx.x / NOUT, e = e0 + threadIdx.x % NOUT;
+    float s = 0.f;
+#pragma unroll
+    for (int q = 0; q < 8; ++q) s += part[q][threadIdx.x];
+    if (t0 + i < tokens && e < n) out[(t0 + i) * n + e] = s;
   }
 }
 
@@ -383,10 +399,10 @@ extern "C" int dewb_shift_tokens(const void* x, const void* mu, float* state, co
 // out [tokens, n] fp32 = x [tokens, d] w [n, d]^T
 extern "C" int dewb_narrow_product(const void* x, const void* w, float* out, long long tokens, int n, int d, int fp32, void* stream_ptr) {
   if (tokens <= 0) return 0;
-  const long long groups = (tokens + TOK - 1) / TOK;
+  const long long groups = (tokens + NTOK - 1) / NTOK;
   if (n < 1 || d < 1 || groups > 65535) return -3;
   cudaStream_t stream = reinterpret_cast<cudaStream_t>(stream_ptr);
-  const dim3 grid((n + 7) / 8, static_cast<unsigned>(groups));
+  const dim3 grid((n + NOUT - 1) / NOUT, static_cast<unsigned>(groups));
   const bool a16 = aligned(x, 16) && aligned(w, 16);
 #define DEWB_NARROW(TT, VV) narrow_product_kernel<TT, VV><<<grid, 256, 0, stream>>>(static_cast<const TT*>(x), static_cast<const TT*>(w), out, tokens, n, d)
   if (fp32) { if (a16 && d % 4 == 0) DEWB_NARROW(float, 4); else DEWB_NARROW(float, 1); }

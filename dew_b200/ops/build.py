@@ -26,7 +26,7 @@ NVCC_FLAGS = ["-O3", "-std=c++17", "-lineinfo", "--use_fast_math", "-Xcompiler",
               "--expt-relaxed-constexpr"]
 
 # Files whose 32-bit arithmetic has to hold up on its own (decoders that run in fp32): compiled without fast math.
-EXACT_MATH = ("residual_streams", "paged_attention", "latent_attention", "decayed_recurrence", "gated_recurrence", "token_mix", "moe_serve")
+EXACT_MATH = ("residual_streams", "paged_attention", "latent_attention", "decayed_recurrence", "gated_recurrence", "gated_chunks", "token_mix", "moe_serve")
 
 # Subsets of the library a program can build alone, as ``libdewb_<part>.so``: a process that only decodes needs neither the training nor
 # the multi-GPU kernels.

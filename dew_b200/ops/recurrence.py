@@ -1,4 +1,5 @@
-"""Recurrences over a matrix state per head whose decays come from the token (``csrc/kernels/gated_recurrence.cu``, whose head gives the equations): the gated
+"""Recurrences over a matrix state per head whose decays come from the token (``csrc/kernels/gated_recurrence.cu``, whose head gives the equations, and
+``gated_chunks.cu``, the tensor-core form for several tokens in bf16): the gated
 delta rule, the matrix memory with exponential gates, and the state with a decay per key channel and a bonus for the token itself.  Each takes a call's
 tokens as ``Rows`` and keeps its state between calls; the plain forms go token by token and autograd differentiates them.
 """
@@ -39,15 +40,24 @@ def _launch(mode: int, q, k, v, rows: Optional[Rows], H: int, G: int, dk: int, d
     rows = whole(R, S, q.device) if rows is None else rows
     q, k, v = rows_of(q), rows_of(k), rows_of(v)
     out = torch.empty(R, S, H, dv, dtype=q.dtype, device=q.device)
-    before = (None, None) if memory is None or S == 1 else (memory.n.clone(), memory.m.clone())      # read by every block of a head while one writes
+    # ``kernel`` forces ``chunks`` (tensor cores, bf16) or ``sequence`` (token after token in fp32, any widths)
+    before = (None, None) if memory is None or (S == 1 and kernel != "chunks") else (memory.n.clone(), memory.m.clone())      # read by every block of a head while one writes
     f32 = lambda t: None if t is None else t.detach().float().contiguous()
     gates, bias0, bias1, log_decay, u = f32(gates), f32(bias0), f32(bias1), f32(log_decay), same(u, q.dtype)
     at = lambda t: 0 if t is None else t.data_ptr()
     n, m = (None, None) if memory is None else (memory.n, memory.m)
+    whole_pieces = q.dtype == torch.bfloat16 and dk <= 128 and not any(n % 8 for n in (dk, dv, q.stride(1), k.stride(1), v.stride(1))) \
+        and not any(at(t) % 16 for t in (q, k, v, log_decay))
+    chunks = (kernel or ("chunks" if S > 1 and whole_pieces else "sequence")) == "chunks"
+    if chunks and not whole_pieces:
+        raise ValueError("the chunked form takes bf16 heads of whole 16-byte pieces, keys up to 128 wide")
     args = _Args(at(q), at(k), at(v), q.stride(1), k.stride(1), v.stride(1), at(gates), at(bias0), at(bias1), at(log_decay), at(u), at(state), at(n), at(m),
                  at(before[0]), at(before[1]), at(rows.positions), at(rows.lengths), at(rows.row_ids), at(out), scale, cap, R, S, H, G, dk, dv)
-    fn = L.load().dewb_gated_recurrence
-    L.check(fn(ctypes.c_int(mode), ctypes.byref(args), ctypes.c_int(int(q.dtype == torch.float32)), L.stream_ptr()), "gated_recurrence")
+    if chunks:
+        L.check(L.load().dewb_gated_chunks(ctypes.c_int(mode), ctypes.byref(args), L.stream_ptr()), "gated_chunks")
+    else:
+        L.check(L.load().dewb_gated_recurrence(ctypes.c_int(mode), ctypes.byref(args), ctypes.c_int(int(q.dtype == torch.float32)), L.stream_ptr()),
+                "gated_recurrence")
     L.count_launches()
     return out
 
@@ -92,14 +102,15 @@ def delta_rule_reference(q, k, v, gates, A_log, dt_bias, H: int, G: int, scale: 
     return _tokens(rows, [state], [qf.new_zeros(R, H, dk, dv)], body, (R, S, H, dv), v.dtype)
 
 
-def delta_rule(q, k, v, gates, A_log, dt_bias, H: int, G: int, scale: Optional[float] = None, rows: Optional[Rows] = None, state=None) -> torch.Tensor:
+def delta_rule(q, k, v, gates, A_log, dt_bias, H: int, G: int, scale: Optional[float] = None, rows: Optional[Rows] = None, state=None,
+               kernel: Optional[str] = None) -> torch.Tensor:
     """The gated delta rule: ``q, k [R, S, G dk]`` (behind their activation; they are normalised here), ``v [R, S, H dv]``, ``gates [R, S, 2 H]`` fp32 (step
     logits, then decay logits), ``A_log, dt_bias [H]`` -> ``[R, S, H, dv]``; head h uses q and k of head ``h // (H // G)``.  ``state [rows, H, dk, dv]``."""
     dk, dv = q.shape[-1] // G, v.shape[-1] // H
     scale = dk ** -0.5 if scale is None else float(scale)
     if not kernel_ok(q, k, v, gates, A_log, dt_bias):
         return delta_rule_reference(q, k, v, gates, A_log, dt_bias, H, G, scale, rows, state)
-    return _launch(DELTA, q, k, v, rows, H, G, dk, dv, state, scale, gates=gates, bias0=A_log, bias1=dt_bias)
+    return _launch(DELTA, q, k, v, rows, H, G, dk, dv, state, scale, gates=gates, bias0=A_log, bias1=dt_bias, kernel=kernel)
 
 
 def matrix_memory_reference(q, k, v, gates, i_bias, f_bias, H: int, cap: float, scale: float, rows: Optional[Rows] = None, memory: Optional[Memory] = None):
@@ -125,14 +136,14 @@ def matrix_memory_reference(q, k, v, gates, i_bias, f_bias, H: int, cap: float, 
 
 
 def matrix_memory(q, k, v, gates, i_bias, f_bias, H: int, cap: float, scale: Optional[float] = None, rows: Optional[Rows] = None,
-                  memory: Optional[Memory] = None) -> torch.Tensor:
+                  memory: Optional[Memory] = None, kernel: Optional[str] = None) -> torch.Tensor:
     """The matrix memory with exponential gates: ``q, k [R, S, H dk]``, ``v [R, S, H dv]``, ``gates [R, S, 2 H]`` fp32 (input logits, then forget logits),
     their biases ``[H]`` -> ``[R, S, H, dv]``."""
     dk, dv = q.shape[-1] // H, v.shape[-1] // H
     scale = dk ** -0.5 if scale is None else float(scale)
     if not kernel_ok(q, k, v, gates, i_bias, f_bias):
         return matrix_memory_reference(q, k, v, gates, i_bias, f_bias, H, cap, scale, rows, memory)
-    return _launch(MEMORY, q, k, v, rows, H, H, dk, dv, None if memory is None else memory.S, scale, float(cap), gates, i_bias, f_bias, memory=memory)
+    return _launch(MEMORY, q, k, v, rows, H, H, dk, dv, None if memory is None else memory.S, scale, float(cap), gates, i_bias, f_bias, memory=memory, kernel=kernel)
 
 
 def bonus_decay_reference(r, k, v, log_decay, u, H: int, rows: Optional[Rows] = None, state=None):
@@ -149,10 +160,10 @@ def bonus_decay_reference(r, k, v, log_decay, u, H: int, rows: Optional[Rows] = 
     return _tokens(rows, [state], [rf.new_zeros(R, H, dk, dv)], body, (R, S, H, dv), v.dtype)
 
 
-def bonus_decay(r, k, v, log_decay, u, H: int, rows: Optional[Rows] = None, state=None) -> torch.Tensor:
+def bonus_decay(r, k, v, log_decay, u, H: int, rows: Optional[Rows] = None, state=None, kernel: Optional[str] = None) -> torch.Tensor:
     """The state with a decay per key channel: ``r, k [R, S, H dk]``, ``v [R, S, H dv]``, ``log_decay [R, S, H dk]`` fp32, the bonus ``u [H, dk]`` with which a token
     reads itself -> ``[R, S, H, dv]``."""
     dk, dv = r.shape[-1] // H, v.shape[-1] // H
     if not kernel_ok(r, k, v, log_decay, u):
         return bonus_decay_reference(r, k, v, log_decay, u, H, rows, state)
-    return _launch(WKV, r, k, v, rows, H, H, dk, dv, state, log_decay=log_decay, u=u)
+    return _launch(WKV, r, k, v, rows, H, H, dk, dv, state, log_decay=log_decay, u=u, kernel=kernel)

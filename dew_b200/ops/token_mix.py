@@ -135,8 +135,8 @@ def narrow_product(x: torch.Tensor, w: torch.Tensor) -> torch.Tensor:
         gemm(x2, wk, out=out, kernel="sm100_tcgen05")
         return out.contiguous().view(*x.shape[:-1], n)
     out = torch.empty(T, n, dtype=torch.float32, device=x.device)
-    for t0 in range(0, T, 1 << 18):
-        t1 = min(T, t0 + (1 << 18))
+    for t0 in range(0, T, 1 << 17):
+        t1 = min(T, t0 + (1 << 17))
         L.check(L.load().dewb_narrow_product(L.ptr(x2[t0:t1]), L.ptr(wk), L.ptr(out[t0:t1]), c_ll(t1 - t0), c_int(n), c_int(d),
                                              c_int(int(x.dtype == torch.float32)), L.stream_ptr()), "narrow_product")
         L.count_launches()

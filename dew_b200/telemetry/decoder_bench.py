@@ -1,9 +1,9 @@
 """Prefill and decode throughput of a decoder design beside this library's closest decoder of the same sizes, and each of the design's kernels
 beside the like kernel of that decoder, as a fraction of its roofline: the Ragenex design here (closest: rotary attention and gated-delta-net
 layers in the same order, SwiGLU, one bf16 residual), the Fakonex design in ``telemetry.fakonex_bench``, the Selivik design in
-``telemetry.selivik_bench``.
+``telemetry.selivik_bench``, the Rarelorn design in ``telemetry.rarelorn_bench``.
 
-``bench.py --decoder ragenex | fakonex | selivik`` prints the result as one JSON line.  Weights are random.  Everything is timed on the device with CUDA events
+``bench.py --decoder ragenex | fakonex | selivik | rarelorn`` prints the result as one JSON line.  Weights are random.  Everything is timed on the device with CUDA events
 after warm-up; prefill activations and weights are larger than L2, and a decode step (one CUDA graph, where the model's step can be captured) streams
 all the weights.
 """
@@ -127,6 +127,7 @@ def throughput(model, s: dict, rows: int, prompt: int, decode_rows: int, context
         torch.cuda.empty_cache()
         return out
     side = torch.cuda.Stream()
+    torch.cuda.synchronize()                      # (the inputs above are made on the other stream)
     with torch.cuda.stream(side):
         step()
         step()
@@ -237,8 +238,11 @@ def run(name: str = "ragenex", sizes=None, rows: int = 4, prompt: int = 4096, de
         from . import fakonex_bench as f
         table, design, near, parts = f.SIZES, f.design, f.closest, f.kernels
         context = 4095 if context is None else context           # the last position of a chunk: as many keys as the closest model's window holds
-    elif name == "selivik":
-        from . import selivik_bench as f
+    elif name in ("selivik", "rarelorn"):
+        if name == "selivik":
+            from . import selivik_bench as f
+        else:
+            from . import rarelorn_bench as f
         table, design, near, parts = f.SIZES, f.design, f.closest, f.kernels
         context = 4096 if context is None else context
     else:
