@@ -68,24 +68,28 @@ __device__ __forceinline__ float softplus(float x) { return fmaxf(x, 0.f) + log1
 
 // The logarithm of a head's decay, and its step.
 template <typename T>
-__device__ __forceinline__ void delta_log_gates(const Args<T>& p, long long token, int h, float& log_decay, float& beta) {
-  const float* z = p.gates + token * 2 * p.H + h;
-  beta = __fdividef(1.f, 1.f + expf(-z[0]));
-  log_decay = -expf(p.bias0[h]) * softplus(z[p.H] + p.bias1[h]);
+__device__ __forceinline__ void delta_log_gates(const Args<T>& p, int h, float zb, float za, float& log_decay, float& beta) {
+  beta = __fdividef(1.f, 1.f + expf(-zb));
+  log_decay = -expf(p.bias0[h]) * softplus(za + p.bias1[h]);
 }
 template <typename T>
 __device__ __forceinline__ void delta_gates(const Args<T>& p, long long token, int h, float& decay, float& beta) {
-  delta_log_gates(p, token, h, decay, beta);
+  const float* z = p.gates + token * 2 * p.H + h;
+  delta_log_gates(p, h, z[0], z[p.H], decay, beta);
   decay = expf(decay);
 }
 
 // Logarithms of the input and the forget gate.
 template <typename T>
+__device__ __forceinline__ void memory_gates(const Args<T>& p, int h, float zi, float zf, float& in, float& forget) {
+  const float inv = __fdividef(1.f, p.cap);
+  in = p.cap * tanhf((zi + p.bias0[h]) * inv);
+  forget = -softplus(-p.cap * tanhf((zf + p.bias1[h]) * inv));
+}
+template <typename T>
 __device__ __forceinline__ void memory_gates(const Args<T>& p, long long token, int h, float& in, float& forget) {
   const float* z = p.gates + token * 2 * p.H + h;
-  const float inv = __fdividef(1.f, p.cap);
-  in = p.cap * tanhf((z[0] + p.bias0[h]) * inv);
-  forget = -softplus(-p.cap * tanhf((z[p.H] + p.bias1[h]) * inv));
+  memory_gates(p, h, z[0], z[p.H], in, forget);
 }
 
 }  // namespace gated

@@ -1,6 +1,6 @@
 // The recurrences of gated_recurrence.cu over a call's tokens in chunks on the tensor cores, for sm_100a (bf16, dk up to 128, widths in multiples of 8).
 //
-// One block of four warps walks a (row, head, 64 value columns) chunk by chunk.  A warp keeps the state of 16 value columns, transposed ([value, key], fp32
+// One block walks a (row, head, 64 or 128 value columns) chunk by chunk, the next chunk's rows on their way (cp.async).  A warp keeps the state of 16 value columns, transposed ([value, key], fp32
 // accumulators) for the whole call: a fragment of it turns into an operand without leaving the registers, and once a chunk's scores lie in shared memory a warp
 // needs nothing from the others.  Everything that is not a bf16 activation - the state, decayed scores, what the delta rule writes - enters its products as a
 // pair of bf16 (value and rounding rest: 16 bits of mantissa); weights of a token or a channel are fp32 factors.  No exponent is above 0 by construction.
@@ -25,23 +25,36 @@ namespace gated {
 
 using namespace mma16;
 
-constexpr int CT = 64, VT = 64, CTHREADS = 128;
+constexpr int CT = 64;              // tokens per chunk
 
-template <int MODE, int DK>
+template <int MODE, int DK, int NW>
 struct ChunkSmem {
-  bf16 q[CT][DK + 8], k[CT][DK + 8], v[CT][VT + 8];
+  static constexpr int VT = NW * 16;
+  bf16 q[2][CT][DK + 8], k[2][CT][DK + 8], v[2][CT][VT + 8];  // two stages
   bf16 p[2][CT][CT + 8];                                     // scores as the outputs take them: value, rest
   bf16 a[MODE == DELTA ? 2 : 1][MODE == DELTA ? CT : 1][CT + 8];   // delta: -A below the diagonal blocks
   bf16 t[2][4][16][MODE == DELTA ? 24 : 8];                  // delta: the diagonal blocks of (I + A)^-1
-  float diag[MODE == DELTA ? 4 : 1][16][17];
+  float diag[MODE == DELTA ? 4 : 1][16][16];                 // ... of A, by columns
   float x0[CT], x1[CT], x2[CT], x3[CT], x4[CT], x5[CT], x6[CT];   // of the tokens, see below
   float part[MODE == MEMORY ? CT : 1][4];                    // memory: sums of a row's scores, by block of 16 keys
-  float n[MODE == MEMORY ? DK : 1];
+  float n[MODE == MEMORY ? NW * 32 : 1];                     // memory: the normaliser, in the parts their threads own
   float end[2];
 };
 
 // 16 bytes of a token's row, zeros past its columns
 __device__ __forceinline__ uint4 row16(const bf16* p, bool ok) { return ok ? *reinterpret_cast<const uint4*>(p) : make_uint4(0, 0, 0, 0); }
+
+// 16 bytes into shared memory, zeros where there is nothing to read (the address has to be valid all the same)
+__device__ __forceinline__ void cp16(void* dst, const void* src, bool live) {
+  const int n = live ? 16 : 0;
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(smem_addr(dst)), "l"(src), "r"(n) : "memory");
+}
+
+// d += a b for two tiles of eight columns, b [16, 16]
+__device__ __forceinline__ void mma2(float (&d0)[4], float (&d1)[4], const uint32_t (&a)[4], const uint32_t (&b)[4]) {
+  mma(d0, a, b[0], b[1]);
+  mma(d1, a, b[2], b[3]);
+}
 
 // c [16 values, 16 tokens] as an operand whose rows are values and whose reduction runs over the tokens
 __device__ __forceinline__ void as_operand(const float (&lo)[4], const float (&hi)[4], uint32_t (&big)[4], uint32_t (&rest)[4]) {
@@ -68,12 +81,13 @@ __device__ __forceinline__ float warp_max_scan(float v, int lane) {
   return v;
 }
 
-// grid (H, ceil(dv / VT), rows)
-template <int MODE, int DK>
-__global__ void __launch_bounds__(CTHREADS, 2)
+// grid (H, ceil(dv / VT), rows), NW warps
+template <int MODE, int DK, int NW>
+__global__ void __launch_bounds__(NW * 32, NW == 4 ? 2 : 1)
 gated_chunks_kernel(Args<bf16> p) {
   extern __shared__ __align__(16) uint8_t raw[];
-  ChunkSmem<MODE, DK>& sm = *reinterpret_cast<ChunkSmem<MODE, DK>*>(raw);
+  ChunkSmem<MODE, DK, NW>& sm = *reinterpret_cast<ChunkSmem<MODE, DK, NW>*>(raw);
+  constexpr int CTHREADS = NW * 32, VT = NW * 16;
   constexpr int NK = DK / 8;                       // 8-column tiles of the state
   const int dk = p.dk, dv = p.dv, S_len = p.S, h = blockIdx.x, row = blockIdx.z, c0 = blockIdx.y * VT;
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, lg = lane >> 2, t2 = (lane & 3) * 2;
@@ -86,7 +100,7 @@ gated_chunks_kernel(Args<bf16> p) {
   const long long o_stride = static_cast<long long>(p.H) * dv;
   float* S = p.state == nullptr ? nullptr : p.state + rh * dk * dv;
   const bool held = S != nullptr && first > 0;
-  const int w0 = warp * 16;                        // this warp's value columns, and its share of the scores
+  const int w0 = warp * 16;                        // this warp's value columns
   float st_acc[NK][4];
 #pragma unroll
   for (int n = 0; n < NK; ++n)
@@ -97,63 +111,96 @@ gated_chunks_kernel(Args<bf16> p) {
     }
   float m = MODE == MEMORY && held ? p.m_before[rh] : 0.f;
   if (MODE == MEMORY)
-    for (int i = tid; i < DK; i += CTHREADS) sm.n[i] = held && i < dk ? p.n_before[rh * dk + i] : 0.f;
+    for (int i = tid; i < CTHREADS; i += CTHREADS) sm.n[i] = held && i < dk ? p.n_before[rh * dk + i] : 0.f;
   const int vcols = min(VT, dv - c0);
-  for (int t0 = 0; t0 < len; t0 += CT) {
-    const int n = min(CT, len - t0);
-    __syncthreads();                               // the chunk before has been read
-#pragma unroll 4
-    for (int i = tid; i < CT * (DK / 8); i += CTHREADS) {
-      const int t = i / (DK / 8), c = (i % (DK / 8)) * 8;
-      const bool ok = t < n && c < dk;
-      *reinterpret_cast<uint4*>(&sm.q[t][c]) = row16(qb + (t0 + t) * p.q_stride + c, ok);
-      *reinterpret_cast<uint4*>(&sm.k[t][c]) = row16(kb + (t0 + t) * p.k_stride + c, ok);
+  auto fetch = [&](int t0, int s) {
+    constexpr int PK = DK / 8, PV = VT / 8;        // 16-byte pieces of a row
+    const int ck = (tid % PK) * 8, cv = (tid % PV) * 8;
+#pragma unroll
+    for (int t = tid / PK; t < CT; t += CTHREADS / PK) {
+      const bool ok = t0 + t < len && ck < dk;
+      cp16(&sm.q[s][t][ck], ok ? qb + (t0 + t) * p.q_stride + ck : p.q, ok);
+      cp16(&sm.k[s][t][ck], ok ? kb + (t0 + t) * p.k_stride + ck : p.k, ok);
     }
-    for (int i = tid; i < CT * (VT / 8); i += CTHREADS) {
-      const int t = i / (VT / 8), c = (i % (VT / 8)) * 8;
-      *reinterpret_cast<uint4*>(&sm.v[t][c]) = row16(vb + (t0 + t) * p.v_stride + c, t < n && c < vcols);
+#pragma unroll
+    for (int t = tid / PV; t < CT; t += CTHREADS / PV) {
+      const bool ok = t0 + t < len && cv < vcols;
+      cp16(&sm.v[s][t][cv], ok ? vb + (t0 + t) * p.v_stride + cv : p.v, ok);
     }
-    if (tid < CT) {                                // what lies past the end neither writes nor forgets
-      float a = MODE == MEMORY ? -INFINITY : 0.f, b = 0.f;
-      if (tid < n) {
-        if (MODE == MEMORY) memory_gates(p, t_row + t0 + tid, h, a, b);
-        else delta_log_gates(p, t_row + t0 + tid, h, b, a);
+    asm volatile("cp.async.commit_group;" ::: "memory");
+  };
+  // the first warp's gates, a chunk ahead: tokens lane and lane + 32
+  float z0[2] = {0.f, 0.f}, z1[2] = {0.f, 0.f};
+  auto gates = [&](int t0) {
+#pragma unroll
+    for (int x = 0; x < 2; ++x)
+      if (t0 + lane + 32 * x < len) {
+        const float* z = p.gates + (t_row + t0 + lane + 32 * x) * 2 * p.H + h;
+        z0[x] = z[0];
+        z1[x] = z[p.H];
       }
-      sm.x0[tid] = a;                              // memory: log input gate; delta: beta
-      sm.x1[tid] = b;                              // log forget gate / log decay
-    }
-    __syncthreads();
+  };
+  if (len > 0) {
+    fetch(0, 0);
+    if (warp == 0) gates(0);
+  }
+  for (int t0 = 0, stage = 0; t0 < len; t0 += CT, stage ^= 1) {
+    const int n = min(CT, len - t0);
+    asm volatile("cp.async.wait_group 0;" ::: "memory");
+    __syncthreads();                               // this chunk is there, the one before has been read
+    if (t0 + CT < len) fetch(t0 + CT, stage ^ 1);
+    const bf16 (&sq_)[CT][DK + 8] = sm.q[stage], (&sk_)[CT][DK + 8] = sm.k[stage];
+    bf16 (&sv_)[CT][VT + 8] = sm.v[stage];
     // ---- scalars of the tokens.  memory: x0 = g, x1 = M, x2 = scale e^(m - M), x3 = e^-(F + M), x4 = q . n, x5 = e^(g - M_end);
     //      delta: x0 = beta, x1 = G, x2, x3 = factors of q and k, x4 = x2 e^G, x5 = x3 e^(G_end - G), x6 = beta x3 e^G
     {
-      const int t = tid >> 1, half = (tid & 1) * (DK / 2);
+      constexpr int PER = CTHREADS / CT, PARTS = CTHREADS / DK;        // threads per token; parts of the normaliser
+      const int t = tid / PER, c0_ = (tid % PER) * 8;
       float s0 = 0.f, s1 = 0.f;
 #pragma unroll
-      for (int c = 0; c < DK / 2; c += 8) {
+      for (int c = c0_; c < DK; c += 8 * PER) {
         float a[8], b[8];
-        rows::load_v<8>(&sm.q[t][half + c], a);
-        if (MODE == DELTA) rows::load_v<8>(&sm.k[t][half + c], b);
+        rows::load_v<8>(&sq_[t][c], a);
+        if (MODE == DELTA) rows::load_v<8>(&sk_[t][c], b);
 #pragma unroll
         for (int j = 0; j < 8; ++j) {
-          if (MODE == DELTA) { s0 += a[j] * a[j]; s1 += b[j] * b[j]; }
-          else s0 += a[j] * sm.n[half + c + j];
+          if (MODE == DELTA) {
+            s0 += a[j] * a[j];
+            s1 += b[j] * b[j];
+          } else {
+#pragma unroll
+            for (int x = 0; x < PARTS; ++x) s0 += a[j] * sm.n[x * DK + c + j];
+          }
         }
       }
-      s0 += __shfl_xor_sync(0xffffffffu, s0, 1);
-      s1 += __shfl_xor_sync(0xffffffffu, s1, 1);
-      if ((tid & 1) == 0) {
+#pragma unroll
+      for (int x = PER / 2; x > 0; x >>= 1) {
+        s0 += __shfl_xor_sync(0xffffffffu, s0, x);
+        s1 += __shfl_xor_sync(0xffffffffu, s1, x);
+      }
+      if (tid % PER == 0) {
         if (MODE == DELTA) { sm.x2[t] = p.scale * rsqrtf(s0 + 1e-6f); sm.x3[t] = rsqrtf(s1 + 1e-6f); }
         else sm.x4[t] = s0;
       }
     }
     if (warp == 0) {
-      const float a = sm.x1[lane], b = sm.x1[lane + 32];
-      const float F0 = warp_scan(a, lane), F1 = warp_scan(b, lane) + __shfl_sync(0xffffffffu, F0, 31);
+      float a[2], b[2];                            // beta or log input gate; log decay or log forget gate
+#pragma unroll
+      for (int x = 0; x < 2; ++x) {                // what lies past the end neither writes nor forgets
+        a[x] = MODE == MEMORY ? -INFINITY : 0.f;
+        b[x] = 0.f;
+        if (lane + 32 * x < n) {
+          if (MODE == MEMORY) memory_gates(p, h, z0[x], z1[x], a[x], b[x]);
+          else delta_log_gates(p, h, z0[x], z1[x], b[x], a[x]);
+        }
+      }
+      gates(t0 + CT);
+      const float F0 = warp_scan(b[0], lane), F1 = warp_scan(b[1], lane) + __shfl_sync(0xffffffffu, F0, 31);
       if (MODE == DELTA) {
-        sm.x1[lane] = F0;
-        sm.x1[lane + 32] = F1;
+        sm.x0[lane] = a[0]; sm.x0[lane + 32] = a[1];
+        sm.x1[lane] = F0; sm.x1[lane + 32] = F1;
       } else {
-        const float g0 = sm.x0[lane] - F0, g1 = sm.x0[lane + 32] - F1;
+        const float g0 = a[0] - F0, g1 = a[1] - F1;
         const float M0 = fmaxf(m, warp_max_scan(g0, lane)), M1 = fmaxf(__shfl_sync(0xffffffffu, M0, 31), warp_max_scan(g1, lane));
         sm.x0[lane] = g0; sm.x0[lane + 32] = g1;
         sm.x1[lane] = M0; sm.x1[lane + 32] = M1;
@@ -174,23 +221,29 @@ gated_chunks_kernel(Args<bf16> p) {
       }
     }
     // ---- scores: the ten 16 x 16 blocks on and below the diagonal, the diagonal ones first
-    for (int blk = warp; blk < 10; blk += 4) {
+    // (eight warps: a diagonal one each for four of them, the others deal out the rest)
+    for (int blk = warp; blk < 10; blk += NW == 8 && warp < 4 ? 10 : 4) {
       const int off = blk - 4;                     // 0..5: (1,0) (2,0) (2,1) (3,0) (3,1) (3,2)
       const int bi = blk < 4 ? blk : off < 1 ? 1 : off < 3 ? 2 : 3, bj = blk < 4 ? blk : off < 1 ? 0 : off < 3 ? off - 1 : off - 3;
       const int i0 = bi * 16, j0 = bj * 16;
-      float sq[2][4] = {}, sk[2][4] = {};
+      float sq[2][4], sk[2][4];
+      {
+        float s[2][2][4] = {}, z[2][2][4] = {};    // even and odd steps apart: their products do not wait for each other
 #pragma unroll
-      for (int kk = 0; kk < DK; kk += 16) {
-        uint32_t qa[4], ka[4], b[4];
-        ldsm4(b, smem_addr(&sm.k[j0 + (lane & 7) + (lane >> 4) * 8][kk + ((lane >> 3) & 1) * 8]));
-        ldsm4(qa, smem_addr(&sm.q[i0 + (lane & 15)][kk + (lane >> 4) * 8]));
-        mma(sq[0], qa, b[0], b[1]);
-        mma(sq[1], qa, b[2], b[3]);
-        if (MODE == DELTA) {
-          ldsm4(ka, smem_addr(&sm.k[i0 + (lane & 15)][kk + (lane >> 4) * 8]));
-          mma(sk[0], ka, b[0], b[1]);
-          mma(sk[1], ka, b[2], b[3]);
+        for (int kk = 0; kk < DK; kk += 16) {
+          uint32_t qa[4], ka[4], b[4];
+          ldsm4(b, smem_addr(&sk_[j0 + (lane & 7) + (lane >> 4) * 8][kk + ((lane >> 3) & 1) * 8]));
+          ldsm4(qa, smem_addr(&sq_[i0 + (lane & 15)][kk + (lane >> 4) * 8]));
+          mma2(s[kk / 16 & 1][0], s[kk / 16 & 1][1], qa, b);
+          if (MODE == DELTA) {
+            ldsm4(ka, smem_addr(&sk_[i0 + (lane & 15)][kk + (lane >> 4) * 8]));
+            mma2(z[kk / 16 & 1][0], z[kk / 16 & 1][1], ka, b);
+          }
         }
+#pragma unroll
+        for (int x = 0; x < 2; ++x)
+#pragma unroll
+          for (int e = 0; e < 4; ++e) { sq[x][e] = s[0][x][e] + s[1][x][e]; sk[x][e] = z[0][x][e] + z[1][x][e]; }
       }
       float sum[2] = {0.f, 0.f};
 #pragma unroll
@@ -203,10 +256,10 @@ gated_chunks_kernel(Args<bf16> p) {
           for (int z = 0; z < 2; ++z) {
             const bool on = j + z <= i;
             if (MODE == MEMORY) {
-              x[z] = on ? sq[half][2 * e + z] * p.scale * expf(sm.x0[j + z] - sm.x1[i]) : 0.f;
+              x[z] = on ? sq[half][2 * e + z] * p.scale * __expf(sm.x0[j + z] - sm.x1[i]) : 0.f;
               sum[e] += x[z];
             } else {
-              const float w = on ? sm.x3[j + z] * expf(sm.x1[i] - sm.x1[j + z]) : 0.f;
+              const float w = on ? sm.x3[j + z] * __expf(sm.x1[i] - sm.x1[j + z]) : 0.f;
               x[z] = sq[half][2 * e + z] * w * sm.x2[i];
               y[z] = j + z < i ? sk[half][2 * e + z] * w * sm.x3[i] * sm.x0[i] : 0.f;
             }
@@ -217,8 +270,8 @@ gated_chunks_kernel(Args<bf16> p) {
           *reinterpret_cast<uint32_t*>(&sm.p[1][i][j]) = rest;
           if constexpr (MODE == DELTA) {
             if (bi == bj) {
-              sm.diag[bi][i - i0][j - j0] = y[0];
-              sm.diag[bi][i - i0][j - j0 + 1] = y[1];
+              sm.diag[bi][j - j0][i - i0] = y[0];
+              sm.diag[bi][j - j0 + 1][i - i0] = y[1];
             } else {
               split2(-y[0], -y[1], big, rest);
               *reinterpret_cast<uint32_t*>(&sm.a[0][i][j]) = big;
@@ -238,12 +291,14 @@ gated_chunks_kernel(Args<bf16> p) {
         float x[16];
         const int c = lane & 15;
 #pragma unroll
-        for (int i = 0; i < 16; ++i) {
-          float s = i == c ? 1.f : 0.f;
+        for (int i = 0; i < 16; ++i) x[i] = i == c ? 1.f : 0.f;
 #pragma unroll
-          for (int j = 0; j < i; ++j) s -= sm.diag[bi][i][j] * x[j];
-          x[i] = s;
-        }
+        for (int j = 0; j < 15; ++j)
+#pragma unroll
+          for (int i = (j + 1) & ~3; i < 16; i += 4) {
+            const float4 d = *reinterpret_cast<const float4*>(&sm.diag[bi][j][i]);      // (zeros on and above the diagonal)
+            x[i] -= d.x * x[j]; x[i + 1] -= d.y * x[j]; x[i + 2] -= d.z * x[j]; x[i + 3] -= d.w * x[j];
+          }
         if (lane < 16) {
 #pragma unroll
           for (int i = 0; i < 16; ++i) {
@@ -266,21 +321,34 @@ gated_chunks_kernel(Args<bf16> p) {
     for (int kk = 0; kk < DK; kk += 16) {
       uint32_t big[4], rest[4];
       as_operand(st_acc[kk / 8], st_acc[kk / 8 + 1], big, rest);
+      auto rows_at = [&](const bf16 (&m)[CT][DK + 8], int j, uint32_t (&b)[4]) {
+        ldsm4(b, smem_addr(&m[j * 16 + (lane & 7) + (lane >> 4) * 8][kk + ((lane >> 3) & 1) * 8]));
+      };
+      if constexpr (MODE == DELTA) {               // eight sums between a product and the next one into the same sum
 #pragma unroll
-      for (int j = 0; j < 4; ++j) {
-        uint32_t b[4];
-        ldsm4(b, smem_addr(&sm.q[j * 16 + (lane & 7) + (lane >> 4) * 8][kk + ((lane >> 3) & 1) * 8]));
-        mma(acc[2 * j], big, b[0], b[1]);
-        mma(acc[2 * j + 1], big, b[2], b[3]);
-        mma(acc[2 * j], rest, b[0], b[1]);
-        mma(acc[2 * j + 1], rest, b[2], b[3]);
-        if constexpr (MODE == DELTA) {
-          ldsm4(b, smem_addr(&sm.k[j * 16 + (lane & 7) + (lane >> 4) * 8][kk + ((lane >> 3) & 1) * 8]));
-          mma(u[2 * j], big, b[0], b[1]);
-          mma(u[2 * j + 1], big, b[2], b[3]);
-          mma(u[2 * j], rest, b[0], b[1]);
-          mma(u[2 * j + 1], rest, b[2], b[3]);
+        for (int j = 0; j < 4; j += 2) {
+          uint32_t b0[4], b1[4], c0_[4], c1[4];
+          rows_at(sq_, j, b0);
+          rows_at(sk_, j, c0_);
+          rows_at(sq_, j + 1, b1);
+          rows_at(sk_, j + 1, c1);
+          mma2(acc[2 * j], acc[2 * j + 1], big, b0);
+          mma2(u[2 * j], u[2 * j + 1], big, c0_);
+          mma2(acc[2 * j + 2], acc[2 * j + 3], big, b1);
+          mma2(u[2 * j + 2], u[2 * j + 3], big, c1);
+          mma2(acc[2 * j], acc[2 * j + 1], rest, b0);
+          mma2(u[2 * j], u[2 * j + 1], rest, c0_);
+          mma2(acc[2 * j + 2], acc[2 * j + 3], rest, b1);
+          mma2(u[2 * j + 2], u[2 * j + 3], rest, c1);
         }
+      } else {
+        uint32_t b[4][4];
+#pragma unroll
+        for (int j = 0; j < 4; ++j) rows_at(sq_, j, b[j]);
+#pragma unroll
+        for (int j = 0; j < 4; ++j) mma2(acc[2 * j], acc[2 * j + 1], big, b[j]);
+#pragma unroll
+        for (int j = 0; j < 4; ++j) mma2(acc[2 * j], acc[2 * j + 1], rest, b[j]);
       }
     }
 #pragma unroll
@@ -297,7 +365,7 @@ gated_chunks_kernel(Args<bf16> p) {
 #pragma unroll
       for (int b = 0; b < 4; ++b) {
         uint32_t vt[4];
-        ldsm4_t(vt, smem_addr(&sm.v[b * 16 + (lane & 7) + (lane >> 4) * 8][w0 + ((lane >> 3) & 1) * 8]));
+        ldsm4_t(vt, smem_addr(&sv_[b * 16 + (lane & 7) + (lane >> 4) * 8][w0 + ((lane >> 3) & 1) * 8]));
 #pragma unroll
         for (int x = 0; x < 4; ++x) {              // (an operand of values over tokens has the places of a result)
           float (&d)[4] = u[2 * b + (x >> 1)];
@@ -309,50 +377,57 @@ gated_chunks_kernel(Args<bf16> p) {
       }
 #pragma unroll
       for (int b = 0; b < 4; ++b) {
-        uint32_t big[4], rest[4], x[4], y[4];
+        uint32_t big[4], rest[4];
+        auto block = [&](const bf16 (&m)[CT][CT + 8], int i, uint32_t (&x)[4]) {
+          ldsm4(x, smem_addr(&m[i * 16 + (lane & 7) + (lane >> 4) * 8][b * 16 + ((lane >> 3) & 1) * 8]));
+        };
+        {
+          uint32_t x[4], y[4];
+          float d[2][4] = {}, e[2][4] = {}, f[2][4] = {};
+          ldsm4(x, smem_addr(&sm.t[0][b][(lane & 7) + (lane >> 4) * 8][((lane >> 3) & 1) * 8]));
+          ldsm4(y, smem_addr(&sm.t[1][b][(lane & 7) + (lane >> 4) * 8][((lane >> 3) & 1) * 8]));
+          as_operand(u[2 * b], u[2 * b + 1], big, rest);
+          mma2(d[0], d[1], big, x);
+          mma2(e[0], e[1], rest, x);
+          mma2(f[0], f[1], big, y);
 #pragma unroll
-        for (int a = 0; a < b; ++a) {
-          as_operand(u[2 * a], u[2 * a + 1], big, rest);
-          ldsm4(x, smem_addr(&sm.a[0][b * 16 + (lane & 7) + (lane >> 4) * 8][a * 16 + ((lane >> 3) & 1) * 8]));
-          ldsm4(y, smem_addr(&sm.a[1][b * 16 + (lane & 7) + (lane >> 4) * 8][a * 16 + ((lane >> 3) & 1) * 8]));
-          mma(u[2 * b], big, x[0], x[1]);
-          mma(u[2 * b + 1], big, x[2], x[3]);
-          mma(u[2 * b], rest, x[0], x[1]);
-          mma(u[2 * b + 1], rest, x[2], x[3]);
-          mma(u[2 * b], big, y[0], y[1]);
-          mma(u[2 * b + 1], big, y[2], y[3]);
+          for (int z = 0; z < 2; ++z)
+#pragma unroll
+            for (int q = 0; q < 4; ++q) u[2 * b + z][q] = d[z][q] + (e[z][q] + f[z][q]);
         }
         as_operand(u[2 * b], u[2 * b + 1], big, rest);
-        ldsm4(x, smem_addr(&sm.t[0][b][(lane & 7) + (lane >> 4) * 8][((lane >> 3) & 1) * 8]));
-        ldsm4(y, smem_addr(&sm.t[1][b][(lane & 7) + (lane >> 4) * 8][((lane >> 3) & 1) * 8]));
+        // what the block means for the later right-hand sides, then for the outputs
 #pragma unroll
-        for (int z = 0; z < 2; ++z) {
-          float (&d)[4] = u[2 * b + z];
-          d[0] = d[1] = d[2] = d[3] = 0.f;
-          mma(d, big, x[2 * z], x[2 * z + 1]);
-          mma(d, rest, x[2 * z], x[2 * z + 1]);
-          mma(d, big, y[2 * z], y[2 * z + 1]);
+        for (int i = b + 1; i < 4; ++i) {
+          uint32_t x[4], y[4];
+          block(sm.a[0], i, x);
+          block(sm.a[1], i, y);
+          mma2(u[2 * i], u[2 * i + 1], big, x);
+          mma2(u[2 * i], u[2 * i + 1], rest, x);
+          mma2(u[2 * i], u[2 * i + 1], big, y);
+        }
+#pragma unroll
+        for (int i = b; i < 4; ++i) {
+          uint32_t x[4], y[4];
+          block(sm.p[0], i, x);
+          block(sm.p[1], i, y);
+          mma2(acc[2 * i], acc[2 * i + 1], big, x);
+          mma2(acc[2 * i], acc[2 * i + 1], rest, x);
+          mma2(acc[2 * i], acc[2 * i + 1], big, y);
         }
       }
     }
-    // ---- from the chunk: values (or writes) times scores
+    if constexpr (MODE == MEMORY) {                // ---- from the chunk: values times scores
 #pragma unroll
-    for (int b = 0; b < 4; ++b) {
-      uint32_t big[4], rest[4];
-      if constexpr (MODE == DELTA) as_operand(u[2 * b], u[2 * b + 1], big, rest);
-      else ldsm4_t(big, smem_addr(&sm.v[b * 16 + (lane & 7) + (lane >> 4) * 8][w0 + ((lane >> 3) & 1) * 8]));
+      for (int b = 0; b < 4; ++b) {
+        uint32_t vt[4], x[4][4];
+        ldsm4_t(vt, smem_addr(&sv_[b * 16 + (lane & 7) + (lane >> 4) * 8][w0 + ((lane >> 3) & 1) * 8]));
 #pragma unroll
-      for (int i = b; i < 4; ++i) {
-        uint32_t x[4], y[4];
-        ldsm4(x, smem_addr(&sm.p[0][i * 16 + (lane & 7) + (lane >> 4) * 8][b * 16 + ((lane >> 3) & 1) * 8]));
-        ldsm4(y, smem_addr(&sm.p[1][i * 16 + (lane & 7) + (lane >> 4) * 8][b * 16 + ((lane >> 3) & 1) * 8]));
-        mma(acc[2 * i], big, x[0], x[1]);
-        mma(acc[2 * i + 1], big, x[2], x[3]);
-        mma(acc[2 * i], big, y[0], y[1]);
-        mma(acc[2 * i + 1], big, y[2], y[3]);
-        if constexpr (MODE == DELTA) {
-          mma(acc[2 * i], rest, x[0], x[1]);
-          mma(acc[2 * i + 1], rest, x[2], x[3]);
+        for (int part = 0; part < 2; ++part) {
+#pragma unroll
+          for (int i = b; i < 4; ++i) ldsm4(x[i], smem_addr(&sm.p[part][i * 16 + (lane & 7) + (lane >> 4) * 8][b * 16 + ((lane >> 3) & 1) * 8]));
+#pragma unroll
+          for (int i = b; i < 4; ++i) mma2(acc[2 * i], acc[2 * i + 1], vt, x[i]);
         }
       }
     }
@@ -368,7 +443,7 @@ gated_chunks_kernel(Args<bf16> p) {
         const int i = b * 16 + t2;
         if constexpr (MODE == MEMORY) {
           uint32_t vt[4];
-          ldsm4_t(vt, smem_addr(&sm.v[b * 16 + (lane & 7) + (lane >> 4) * 8][w0 + ((lane >> 3) & 1) * 8]));
+          ldsm4_t(vt, smem_addr(&sv_[b * 16 + (lane & 7) + (lane >> 4) * 8][w0 + ((lane >> 3) & 1) * 8]));
 #pragma unroll
           for (int x = 0; x < 4; ++x) {
             const int j = i + (x >> 1) * 8;
@@ -383,13 +458,14 @@ gated_chunks_kernel(Args<bf16> p) {
           }
         }
 #pragma unroll
-        for (int j = 0; j < NK / 2; ++j) {
-          uint32_t x[4];
-          ldsm4_t(x, smem_addr(&sm.k[b * 16 + (lane & 15)][j * 16 + (lane >> 4) * 8]));
-          mma(st_acc[2 * j], big, x[0], x[1]);
-          mma(st_acc[2 * j + 1], big, x[2], x[3]);
-          mma(st_acc[2 * j], rest, x[0], x[1]);
-          mma(st_acc[2 * j + 1], rest, x[2], x[3]);
+        for (int j = 0; j < NK / 2; j += 4) {
+          uint32_t x[4][4];
+#pragma unroll
+          for (int z = 0; z < 4; ++z) ldsm4_t(x[z], smem_addr(&sk_[b * 16 + (lane & 15)][(j + z) * 16 + (lane >> 4) * 8]));
+#pragma unroll
+          for (int z = 0; z < 4; ++z) mma2(st_acc[2 * (j + z)], st_acc[2 * (j + z) + 1], big, x[z]);
+#pragma unroll
+          for (int z = 0; z < 4; ++z) mma2(st_acc[2 * (j + z)], st_acc[2 * (j + z) + 1], rest, x[z]);
         }
       }
     }
@@ -407,11 +483,11 @@ gated_chunks_kernel(Args<bf16> p) {
           acc[j][z] *= den;
           acc[j][z + 2] *= den;
         }
-      for (int c = tid; c < DK; c += CTHREADS) {
-        float s = sm.n[c] * keep;
-        for (int j = 0; j < n; ++j) s += sm.x5[j] * __bfloat162float(sm.k[j][c]);
-        sm.n[c] = s;
-      }
+      constexpr int PARTS = CTHREADS / DK;         // a part takes every PARTS-th token
+      float s = sm.n[tid] * keep;
+#pragma unroll 8
+      for (int j = tid / DK; j < n; j += PARTS) s += sm.x5[j] * __bfloat162float(sk_[j][tid % DK]);
+      sm.n[tid] = s;
       m = sm.end[1];
     }
     // ---- outputs: this warp's columns of the value tile hold them for wide stores (no other warp reads those columns)
@@ -419,12 +495,12 @@ gated_chunks_kernel(Args<bf16> p) {
 #pragma unroll
     for (int j = 0; j < 8; ++j)
 #pragma unroll
-      for (int e = 0; e < 4; ++e) sm.v[j * 8 + t2 + (e & 1)][w0 + lg + (e >> 1) * 8] = __float2bfloat16(acc[j][e]);
+      for (int e = 0; e < 4; ++e) sv_[j * 8 + t2 + (e & 1)][w0 + lg + (e >> 1) * 8] = __float2bfloat16(acc[j][e]);
     __syncwarp();
 #pragma unroll
     for (int i = lane; i < CT * 2; i += 32) {
       const int t = i >> 1, c = w0 + (i & 1) * 8;
-      if (t < n && c < vcols) *reinterpret_cast<uint4*>(o + (t0 + t) * o_stride + c) = *reinterpret_cast<const uint4*>(&sm.v[t][c]);
+      if (t < n && c < vcols) *reinterpret_cast<uint4*>(o + (t0 + t) * o_stride + c) = *reinterpret_cast<const uint4*>(&sv_[t][c]);
     }
   }
   if (S != nullptr && len > 0) {
@@ -437,7 +513,12 @@ gated_chunks_kernel(Args<bf16> p) {
       }
     if (MODE == MEMORY && blockIdx.y == 0) {
       __syncthreads();
-      for (int i = tid; i < dk; i += CTHREADS) p.n[rh * dk + i] = sm.n[i];
+      if (tid < dk) {
+        float s = 0.f;
+#pragma unroll
+        for (int x = 0; x < CTHREADS / DK; ++x) s += sm.n[x * DK + tid];
+        p.n[rh * dk + tid] = s;
+      }
       if (tid == 0) p.m[rh] = m;
     }
   }
@@ -448,7 +529,7 @@ gated_chunks_kernel(Args<bf16> p) {
 }
 
 // ---------------------------------------------------------------------------------------------------------------- wkv
-constexpr int WT = 16;             // tokens per chunk
+constexpr int WT = 16, VT = 64, CTHREADS = 128;             // tokens per chunk; value columns and threads of a block
 
 template <int DK>
 struct WkvSmem {
@@ -491,6 +572,9 @@ wkv_chunks_kernel(Args<bf16> p) {
     sm.u[c] = c < dk ? ld(p.u + h * dk + c) : 0.f;
     sm.L[0][c] = 0.f;
   }
+  int my_i = 1;                                    // this thread's pair of tokens
+  while (my_i < WT - 1 && my_i * (my_i + 1) / 2 <= tid) ++my_i;
+  const int my_j = tid - my_i * (my_i - 1) / 2;
   // the next chunk's rows wait in registers
   constexpr int QV = WT * DK / 8 / CTHREADS > 0 ? WT * DK / 8 / CTHREADS : 1, LV = WT * DK / 4 / CTHREADS;
   uint4 rq[QV], rk[QV], rv;
@@ -552,60 +636,61 @@ wkv_chunks_kernel(Args<bf16> p) {
       *reinterpret_cast<uint32_t*>(&sm.ks[0][t][c]) = big;
       *reinterpret_cast<uint32_t*>(&sm.ks[1][t][c]) = rest;
     }
-    // a pair per thread: 120 below the diagonal, 16 on it (two rounds for eight of them)
-    for (int x = tid; x < WT * (WT + 1) / 2; x += CTHREADS) {
-      int i = static_cast<int>((sqrtf(8.f * x + 1.f) - 1.f) * 0.5f);
-      while ((i + 1) * (i + 2) / 2 <= x) ++i;
-      while (i * (i + 1) / 2 > x) --i;
-      const int j = x - i * (i + 1) / 2;
-      float s0 = 0.f, s1 = 0.f;
-      if (i == j) {
-#pragma unroll 4
-        for (int c = 0; c < DK; c += 2) {
-          const uint32_t qq = *reinterpret_cast<const uint32_t*>(&sm.q[i][c]), kk = *reinterpret_cast<const uint32_t*>(&sm.k[i][c]);
-          s0 += lo_f(qq) * lo_f(kk) * sm.u[c];
-          s1 += hi_f(qq) * hi_f(kk) * sm.u[c + 1];
-        }
-      } else {
-#pragma unroll 4
-        for (int c = 0; c < DK; c += 2) {
-          const uint32_t qq = *reinterpret_cast<const uint32_t*>(&sm.q[i][c]), kk = *reinterpret_cast<const uint32_t*>(&sm.k[j][c]);
-          const float2 a = *reinterpret_cast<const float2*>(&sm.L[i][c]), b = *reinterpret_cast<const float2*>(&sm.L[j + 1][c]);
-          s0 += lo_f(qq) * lo_f(kk) * __expf(a.x - b.x);
-          s1 += hi_f(qq) * hi_f(kk) * __expf(a.y - b.y);
-        }
-      }
-      const float s = s0 + s1;
+    auto score = [&](int i, int j, float s) {
       const bf16 big = __float2bfloat16(s);
       sm.p[0][i][j] = big;
       sm.p[1][i][j] = __float2bfloat16(s - __bfloat162float(big));
-      if (i != j) sm.p[0][j][i] = sm.p[1][j][i] = __float2bfloat16(0.f);
+    };
+    if (tid < WT * (WT - 1) / 2) {                 // a pair below the diagonal per thread
+      const int i = my_i, j = my_j;
+      float s[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll 4
+      for (int c = 0; c < DK; c += 4) {
+        const uint2 qq = *reinterpret_cast<const uint2*>(&sm.q[i][c]), kk = *reinterpret_cast<const uint2*>(&sm.k[j][c]);
+        const float4 a = *reinterpret_cast<const float4*>(&sm.L[i][c]), b = *reinterpret_cast<const float4*>(&sm.L[j + 1][c]);
+        s[0] += lo_f(qq.x) * lo_f(kk.x) * __expf(a.x - b.x);
+        s[1] += hi_f(qq.x) * hi_f(kk.x) * __expf(a.y - b.y);
+        s[2] += lo_f(qq.y) * lo_f(kk.y) * __expf(a.z - b.z);
+        s[3] += hi_f(qq.y) * hi_f(kk.y) * __expf(a.w - b.w);
+      }
+      score(i, j, (s[0] + s[1]) + (s[2] + s[3]));
+      sm.p[0][j][i] = sm.p[1][j][i] = __float2bfloat16(0.f);
+    }
+    {                                              // the token itself: eight threads each
+      const int i = tid >> 3;
+      float s = 0.f;
+#pragma unroll
+      for (int c = (tid & 7) * 2; c < DK; c += 16) {
+        const uint32_t qq = *reinterpret_cast<const uint32_t*>(&sm.q[i][c]), kk = *reinterpret_cast<const uint32_t*>(&sm.k[i][c]);
+        s += lo_f(qq) * lo_f(kk) * sm.u[c] + hi_f(qq) * hi_f(kk) * sm.u[c + 1];
+      }
+#pragma unroll
+      for (int q = 4; q > 0; q >>= 1) s += __shfl_xor_sync(0xffffffffu, s, q);
+      if ((tid & 7) == 0) score(i, i, s);
     }
     __syncthreads();
     // ---- outputs [16 values, 16 tokens]
-    float acc[2][4] = {};
+    float acc[2][4] = {}, acc1[2][4] = {}, acc2[2][4] = {};
 #pragma unroll
     for (int kk = 0; kk < DK; kk += 16) {
       uint32_t big[4], rest[4], x[4], y[4];
       as_operand(st_acc[kk / 8], st_acc[kk / 8 + 1], big, rest);
       ldsm4(x, smem_addr(&sm.qs[0][(lane & 7) + (lane >> 4) * 8][kk + ((lane >> 3) & 1) * 8]));
       ldsm4(y, smem_addr(&sm.qs[1][(lane & 7) + (lane >> 4) * 8][kk + ((lane >> 3) & 1) * 8]));
-#pragma unroll
-      for (int z = 0; z < 2; ++z) {
-        mma(acc[z], big, x[2 * z], x[2 * z + 1]);
-        mma(acc[z], rest, x[2 * z], x[2 * z + 1]);
-        mma(acc[z], big, y[2 * z], y[2 * z + 1]);
-      }
+      mma2(acc[0], acc[1], big, x);
+      mma2(acc1[0], acc1[1], rest, x);
+      mma2(acc2[0], acc2[1], big, y);
     }
     uint32_t vt[4], x[4], y[4];
     ldsm4_t(vt, smem_addr(&sm.v[(lane & 7) + (lane >> 4) * 8][w0 + ((lane >> 3) & 1) * 8]));
     ldsm4(x, smem_addr(&sm.p[0][(lane & 7) + (lane >> 4) * 8][((lane >> 3) & 1) * 8]));
     ldsm4(y, smem_addr(&sm.p[1][(lane & 7) + (lane >> 4) * 8][((lane >> 3) & 1) * 8]));
+    mma2(acc[0], acc[1], vt, x);
+    mma2(acc1[0], acc1[1], vt, y);
 #pragma unroll
-    for (int z = 0; z < 2; ++z) {
-      mma(acc[z], vt, x[2 * z], x[2 * z + 1]);
-      mma(acc[z], vt, y[2 * z], y[2 * z + 1]);
-    }
+    for (int z = 0; z < 2; ++z)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) acc[z][e] += acc1[z][e] + acc2[z][e];
     // ---- the state after the chunk
 #pragma unroll
     for (int j = 0; j < NK; ++j) {
@@ -613,14 +698,12 @@ wkv_chunks_kernel(Args<bf16> p) {
       st_acc[j][0] *= w.x; st_acc[j][1] *= w.y; st_acc[j][2] *= w.x; st_acc[j][3] *= w.y;
     }
 #pragma unroll
-    for (int j = 0; j < NK / 2; ++j) {
-      ldsm4_t(x, smem_addr(&sm.ks[0][lane & 15][j * 16 + (lane >> 4) * 8]));
-      ldsm4_t(y, smem_addr(&sm.ks[1][lane & 15][j * 16 + (lane >> 4) * 8]));
-      mma(st_acc[2 * j], vt, x[0], x[1]);
-      mma(st_acc[2 * j + 1], vt, x[2], x[3]);
-      mma(st_acc[2 * j], vt, y[0], y[1]);
-      mma(st_acc[2 * j + 1], vt, y[2], y[3]);
-    }
+    for (int part = 0; part < 2; ++part)
+#pragma unroll
+      for (int j = 0; j < NK / 2; ++j) {
+        ldsm4_t(x, smem_addr(&sm.ks[part][lane & 15][j * 16 + (lane >> 4) * 8]));
+        mma2(st_acc[2 * j], st_acc[2 * j + 1], vt, x);
+      }
     __syncwarp();
 #pragma unroll
     for (int z = 0; z < 2; ++z)
@@ -648,12 +731,18 @@ wkv_chunks_kernel(Args<bf16> p) {
 }
 
 template <typename K>
-int chunks_go(K kernel, size_t smem, const Args<bf16>& p, cudaStream_t stream) {
+int chunks_go(K kernel, size_t smem, int columns, const Args<bf16>& p, cudaStream_t stream) {
   if (smem > 225 * 1024) return -3;
   cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem));
   if (e != cudaSuccess) return static_cast<int>(e);
-  kernel<<<dim3(p.H, (p.dv + VT - 1) / VT, p.R), CTHREADS, smem, stream>>>(p);
+  kernel<<<dim3(p.H, (p.dv + columns - 1) / columns, p.R), columns * 2, smem, stream>>>(p);
   return static_cast<int>(cudaGetLastError());
+}
+
+template <int MODE, int DK>
+int chunks_of(const Args<bf16>& p, cudaStream_t stream) {
+  if (p.dv > 64) return chunks_go(gated_chunks_kernel<MODE, DK, 8>, sizeof(ChunkSmem<MODE, DK, 8>), 128, p, stream);
+  return chunks_go(gated_chunks_kernel<MODE, DK, 4>, sizeof(ChunkSmem<MODE, DK, 4>), 64, p, stream);
 }
 
 }  // namespace gated
@@ -667,15 +756,12 @@ extern "C" int dewb_gated_chunks(int mode, const dewb_gated_args* a, void* strea
   if (a->R <= 0 || a->S <= 0) return 0;
   if (!args_ok(mode, *a) || a->dk % 8 || a->dv % 8 || a->dk > 128 || a->q_stride % 8 || a->k_stride % 8 || a->v_stride % 8) return -3;
   if (!dewb::rows::aligned(a->q, 16) || !dewb::rows::aligned(a->k, 16) || !dewb::rows::aligned(a->v, 16) || !dewb::rows::aligned(a->out, 16) ||
-      !dewb::rows::aligned(a->log_decay, 16) || (a->dv + VT - 1) / VT > 65535 || (mode == MEMORY && a->state != nullptr && a->n_before == nullptr))
+      !dewb::rows::aligned(a->log_decay, 16) || (a->dv + 63) / 64 > 65535 || (mode == MEMORY && a->state != nullptr && a->n_before == nullptr))
     return -3;
   cudaStream_t stream = reinterpret_cast<cudaStream_t>(stream_ptr);
   const Args<bf16> p(*a);
   const bool wide = p.dk > 64;
-  if (mode == WKV) return wide ? chunks_go(wkv_chunks_kernel<128>, sizeof(WkvSmem<128>), p, stream) : chunks_go(wkv_chunks_kernel<64>, sizeof(WkvSmem<64>), p, stream);
-  if (mode == MEMORY)
-    return wide ? chunks_go(gated_chunks_kernel<MEMORY, 128>, sizeof(ChunkSmem<MEMORY, 128>), p, stream)
-                : chunks_go(gated_chunks_kernel<MEMORY, 64>, sizeof(ChunkSmem<MEMORY, 64>), p, stream);
-  return wide ? chunks_go(gated_chunks_kernel<DELTA, 128>, sizeof(ChunkSmem<DELTA, 128>), p, stream)
-              : chunks_go(gated_chunks_kernel<DELTA, 64>, sizeof(ChunkSmem<DELTA, 64>), p, stream);
+  if (mode == WKV) return wide ? chunks_go(wkv_chunks_kernel<128>, sizeof(WkvSmem<128>), VT, p, stream) : chunks_go(wkv_chunks_kernel<64>, sizeof(WkvSmem<64>), VT, p, stream);
+  if (mode == MEMORY) return wide ? chunks_of<MEMORY, 128>(p, stream) : chunks_of<MEMORY, 64>(p, stream);
+  return wide ? chunks_of<DELTA, 128>(p, stream) : chunks_of<DELTA, 64>(p, stream);
 }

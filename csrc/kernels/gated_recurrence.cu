@@ -25,7 +25,7 @@ constexpr int STEP_THREADS = 256;
 // grid (H, column tiles, rows); a block walks its column tiles (memory: one block per row and head, which also owns n and m).  A thread owns V columns of
 // the key rows group, group + GROUPS, ..., U of them.
 template <int MODE, typename T, int V, int LANES, int U>
-__global__ void __launch_bounds__(STEP_THREADS, U * V > 32 ? 2 : 3)
+__global__ void __launch_bounds__(STEP_THREADS, U > 16 ? 1 : U * V > 32 ? 2 : 3)
 gated_step_kernel(Args<T> p) {
   constexpr int GROUPS = STEP_THREADS / LANES, TILE = LANES * V;
   extern __shared__ float sm[];                 // q [dk], k [dk], w [dk] (wkv), partial [GROUPS][TILE], u [TILE]

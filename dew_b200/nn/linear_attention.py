@@ -83,21 +83,24 @@ class GatedDeltaNet(nn.Module):
         conv = (("conv", (2 * self.key_dim + self.value_dim, self.conv1d.kernel_size - 1)),) if self.conv1d.kernel_size > 1 else ()
         return CacheSlot(state=(self.hv, self.dk, self.dv), more=conv)
 
-    def _in_slot(self, x, cache, slot: int, positions):
-        """A call's tokens with the state in the cache's slot: convolution, then norms, gates and recurrence in one kernel, then the heads' norm and gate."""
+    def _in_slot(self, x, cache=None, slot: int = 0, positions=None):
+        """A call's tokens with the state in the cache's slot (no cache: whole rows): convolution, then norms, gates and recurrence in one kernel, then
+        the heads' norm and gate."""
         if self.qk_eps != 1e-6:
             raise NotImplementedError("per-layer caches are built for q and k normalised with 1e-6 under the root (qk_eps=1e-6)")
-        rows = cache.call(positions).rows
+        rows, state, more = (None, None, {}) if cache is None else (cache.call(positions).rows, cache.states[slot], cache.more[slot])
         qkvz, inner = self.in_proj_qkvz(x), 2 * self.key_dim + self.value_dim
-        qkv = token_mix.conv_tokens(qkvz[..., :inner], self.conv1d.weight, self.conv1d.bias, self.conv1d.activation, rows, cache.more[slot].get("conv"))
+        qkv = token_mix.conv_tokens(qkvz[..., :inner], self.conv1d.weight, self.conv1d.bias, self.conv1d.activation, rows, more.get("conv"))
         q, k, v = qkv.split([self.key_dim, self.key_dim, self.value_dim], -1)
         o = recurrence.delta_rule(q, k, v, token_mix.narrow_product(x, self.in_proj_ba.weight), self.A_log, self.dt_bias, self.hv, self.hk, None, rows,
-                                  cache.states[slot])
+                                  state)
         return self.out_proj(token_mix.head_gated_norm(o, qkvz[..., inner:], self.norm_weight, self.norm_eps))
 
     def forward(self, x, segment_ids=None, cache=None, layer: int = 0, positions=None):
         if getattr(cache, "slots", None) is not None:
             return self._in_slot(x, cache, layer, positions)
+        if cache is None and x.is_cuda and x.dtype == torch.float32 and self.qk_eps == 1e-6 and segment_ids is None and not torch.is_grad_enabled():
+            return self._in_slot(x)                # (the training kernels form their products in bf16)
         B, T, _ = x.shape
         qkvz = self.in_proj_qkvz(x)
         ba = self.in_proj_ba(x).float()

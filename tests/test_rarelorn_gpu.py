@@ -69,7 +69,7 @@ def test_short_convolution(dtype, C_, taps, wide):
         one, two = (torch.full((4, C_, taps - 1), 9.0, device=DEV) for _ in range(2))
         against(lambda rows, cut: token_mix.conv_tokens(cut(x)[..., :C_], w, bias, silu, rows, one),
                 lambda rows, cut: token_mix.conv_tokens_reference(cut(x).float()[..., :C_], w, bias, silu, rows, two), fine(dtype))
-        assert close(one, two, 1e-6)
+        assert taps == 1 or close(one, two, 1e-6)
         assert close(token_mix.conv_tokens(x[..., :C_], w, bias, silu), token_mix.conv_tokens_reference(x.float()[..., :C_], w, bias, silu), fine(dtype))
 
 
