@@ -741,7 +741,10 @@ int chunks_go(K kernel, size_t smem, int columns, const Args<bf16>& p, cudaStrea
 
 template <int MODE, int DK>
 int chunks_of(const Args<bf16>& p, cudaStream_t stream) {
-  if (p.dv > 64) return chunks_go(gated_chunks_kernel<MODE, DK, 8>, sizeof(ChunkSmem<MODE, DK, 8>), 128, p, stream);
+  // wide blocks form a head's scores once instead of twice; narrow ones pay while both halves find an SM each
+  constexpr long long HALF_THE_SMS = 74;
+  if (p.dv > 64 && static_cast<long long>(p.R) * p.H * ((p.dv + 127) / 128) > HALF_THE_SMS)
+    return chunks_go(gated_chunks_kernel<MODE, DK, 8>, sizeof(ChunkSmem<MODE, DK, 8>), 128, p, stream);
   return chunks_go(gated_chunks_kernel<MODE, DK, 4>, sizeof(ChunkSmem<MODE, DK, 4>), 64, p, stream);
 }
 

@@ -117,7 +117,8 @@ def test_residual_step_with_a_norm_of_one_number(dtype, d):
 
 
 # ------------------------------------------------------------------------------------------------ recurrences
-SIZES = [(4, 2, 64, 64), (3, 3, 32, 48), (2, 1, 128, 128), (2, 2, 96, 72), (3, 1, 8, 136), (2, 2, 5, 7), (2, 2, 20, 33), (1, 1, 200, 40), (1, 1, 300, 9)]
+SIZES = [(4, 2, 64, 64), (3, 3, 32, 48), (2, 1, 128, 128), (2, 2, 96, 72), (3, 1, 8, 136), (2, 2, 5, 7), (2, 2, 20, 33), (1, 1, 200, 40), (1, 1, 300, 9),
+         (26, 13, 64, 72), (25, 25, 128, 128)]        # (the last two: enough heads for the wide blocks)
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
