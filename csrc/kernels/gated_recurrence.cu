@@ -1,10 +1,11 @@
 // Recurrences over a matrix state per head whose decays come from the token, for sm_100a.  k and q have dk entries, v has dv, S is [dk, dv] in fp32.
 //
-//   delta    q, k over their lengths (sqrt(sum + 1e-6)), q times `scale`;  beta = sigmoid(b), g = exp(-exp(A_log) softplus(a + dt_bias)) per head
-//            S <- g S;  u = beta (v - S^T k);  S <- S + k u^T;  o = S^T q.   A group of heads may share q and k.
-//   memory   q times `scale`; log gates per head: i = cap tanh((zi + bi) / cap), f = logsigmoid(cap tanh((zf + bf) / cap)); a running maximum m from 0 on
-//            m' = max(f + m, i);  S <- e^(f + m - m') S + e^(i - m') k v^T, n likewise with k alone;  o = S^T q / (max(|n . q|, e^-m') + 1e-6)
-//   wkv      a decay per key channel, given by its logarithm;  o = (S + diag(u) k v^T)^T q;  S <- diag(w) S + k v^T
+//   delta    k^ = k / sqrt(|k|^2 + 1e-6), q^ likewise times `scale`; a step beta = sigmoid(zb) and a decay g = exp(-e^A_log softplus(za + dt_bias)) per head:
+//            S' = g S + k^ (x) beta (v - g k^ S),   o = q^ S'.   A group of heads may share q and k.
+//   memory   log gates per head, soft-capped: i = cap tanh((zi + bi) / cap) and f = log sigmoid(cap tanh((zf + bf) / cap)).  With M' = max(f + M, i), M = 0 at
+//            first, the old state keeps e^(f + M - M') and k (x) v enters with e^(i - M'); the normaliser n goes the same way with k alone;
+//            o = scale q S' / (max(|scale q n'|, e^-M') + 1e-6)
+//   wkv      a decay w per key channel, given by its logarithm, and a bonus u for the token itself:  o = q S + (sum_c q_c u_c k_c) v,   S' = w . S + k (x) v
 //
 //   gated_step      one token per row: the state is read and written once
 //   gated_sequence  a call's tokens one after another in fp32, any head widths up to 512 (the exact form; it serves fp32 models)

@@ -89,7 +89,7 @@ def test_small_products_and_gated_norms(dtype, T):
     for d, n in ((64, 8), (37, 3), (4096, 64), (200, 130)):
         x, w = rnd(1, T, d, dtype=dtype), rnd(n, d, seed=1, dtype=dtype)
         assert close(token_mix.narrow_product(x, w).double(), torch.nn.functional.linear(x.double(), w.double()), 1e-5)
-    for rank, C_ in ((16, 192), (6, 37), (64, 256), (5, 70), (33, 8)):
+    for rank, C_ in ((16, 176), (6, 37), (64, 256), (5, 70), (33, 8)):
         z, w2, w0 = rnd(1, T, rank), rnd(C_, rank, seed=1, dtype=dtype) * rank ** -0.5, rnd(C_, seed=2, dtype=dtype) - 2
         want = -torch.exp(torch.nn.functional.linear(torch.tanh(z.double()), w2.double(), w0.double()))
         assert float(((token_mix.low_rank_decay(z, w2, w0).double() - want) / want).abs().max()) < 1e-4
